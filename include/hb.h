@@ -172,7 +172,7 @@ int hb_paged_decode_attention_static(void* stream, void* out, const void* q, con
 
 /* Y[M,N] = X[M,K] . W[N,K]^T  (weights stored [out,in] and applied as x.W^T, as every
  * matmul of the path does: src/engine/arch/llama_tp.rs:232-234,327,335-337,354).
- * bf16 with K%64==0 and N%8==0 runs on tcgen05 tensor cores (swap-AB: the weight's
+ * bf16 with K%8==0 runs on tcgen05 tensor cores (swap-AB: the weight's
  * output dim fills the 128-row UMMA M, the batch is the UMMA N; split-K fills the
  * SMs); other dtypes/shapes run a SIMT kernel.  `workspace` (may be NULL when
  * hb_gemm_workspace_bytes()==0) holds split-K partials and tile counters; it must be
@@ -181,7 +181,7 @@ size_t hb_gemm_workspace_bytes(int64_t M, int64_t N, int64_t K, hb_dtype dtype);
 int hb_gemm(void* stream, void* Y, const void* X, const void* W, int64_t M, int64_t N, int64_t K,
             hb_dtype dtype, void* workspace);
 
-/* The same GEMM with the epilogues the decode step fuses into it (bf16, K%64==0 only):
+/* The same GEMM with the epilogues the decode step fuses into it (bf16, K%8==0 only):
  *   epilogue 0: Y[M,N] = X.W^T, as bf16 or (out_f32 != 0) as fp32 — the logits GEMM;
  *   epilogue 1: W = [gate (N/2 rows) ; up (N/2 rows)], Y[M,N/2] = silu(X.gate^T) * (X.up^T)
  *               — gate, up, SiLU and the product of ffn_partial
@@ -429,6 +429,7 @@ typedef struct hb_model_config {
   int64_t num_kv_blocks;    /* 0 = derive from max_seq_len * max_batch */
   int max_batch;            /* largest B of hb_decode_batch (0 = 256) */
   int force_f32;            /* 1: keep F32 weights (the reference's CPU dtype) for tight parity */
+  int max_seqs;             /* models with recurrent state: sequences that may be live (0 = max_batch) */
 } hb_model_config;
 
 /* Shape of a model for hb_engine_create_random (no files involved). */
@@ -460,6 +461,10 @@ int hb_engine_load(const hb_model_config* cfg, hb_world* world, hb_engine** out)
 int hb_engine_create_random(const hb_model_shape* shape, const hb_model_config* cfg,
                             hb_world* world, uint64_t seed, float std, int norm_ones,
                             hb_engine** out);
+/* An engine with random weights for a model described by a config.json text (any registered
+ * design; the Llama family as well).  Matrices are N(0, std), norms and mixing vectors neutral. */
+int hb_engine_create_random_config(const char* config_json, const hb_model_config* cfg, uint64_t seed, float std,
+                                   hb_engine** out);
 int hb_engine_free(hb_engine* e);
 int64_t hb_engine_num_layers(const hb_engine* e);  /* loader.rs:331 */
 int64_t hb_engine_vocab_size(const hb_engine* e);  /* loader.rs:334 */
@@ -496,6 +501,26 @@ int hb_forward(hb_engine* e, hb_seq* s, const uint32_t* ids, size_t n, size_t se
  * [B, vocab]) may be NULL.  Copies in and out happen inside the call. */
 int hb_decode_batch(hb_engine* e, hb_seq* const* seqs, size_t B, const uint32_t* last_tokens,
                     uint32_t* next_tokens, float* logits_opt);
+/* One step over any mix of prompt portions and decoded tokens: entry i feeds its n_tokens next
+ * tokens (positions hb_seq_len(seq) ..) of its sequence, and asks for the logits at the places
+ * want[0..n_want) among them (ascending; may be empty).  All entries form one batch (cut only
+ * where they exceed max_batch rows).  Results lie in the order of the entries and of `want`:
+ * next_tokens (HOST uint32, greedy arg-max; may be NULL) and logits_out (HOST f32 [wanted, vocab];
+ * may be NULL).  A sequence appears once per step and may be left out of steps. */
+typedef struct hb_step_entry {
+  hb_seq* seq;
+  const uint32_t* tokens;
+  size_t n_tokens;
+  const uint32_t* want;
+  size_t n_want;
+} hb_step_entry;
+int hb_step(hb_engine* e, const hb_step_entry* entries, size_t n, uint32_t* next_tokens, float* logits_out);
+/* Draws one token from each of the first n rows of logits the last step left on the device, in the
+ * order of its wanted places (hb_decode_batch: its sequences), with hb_sample's pipeline.
+ * seeds / tokens: HOST [n]. */
+int hb_engine_sample(hb_engine* e, size_t n, const uint64_t* seeds, float temperature, float top_p, uint32_t* tokens);
+/* State slots not taken by a live sequence (0 for a model without recurrent state). */
+int hb_engine_num_free_state_slots(const hb_engine* e);
 /* ---- the step driven by a scheduler's block tables.  The reference's scheduler computes
  * block tables, copy-on-write pairs and swap lists every step (SchedulerOutputs,
  * src/scheduler/mod.rs:40-61,203-208; BlockManager::append_slot / swap_in / swap_out,
@@ -542,8 +567,8 @@ int hb_kv_swap_blocks(hb_engine* e, const int64_t* pairs, size_t n_pairs, int to
  * 0 QKV projection, 1 decode attention, 2 RoPE + KV write, 3 (add +) RMSNorm, 4 embedding /
  * argmax / SwiGLU gate, 5 all-reduce, 6 o_proj, 7 gate|up projection, 8 down_proj,
  * 9 lm_head (6 and 8 include the fused all-reduce + residual + norm when that kernel
- * runs).  The step counts like any other decode step. */
-#define HB_PROFILE_KINDS 10
+ * runs), 10 linear recurrence.  The step counts like any other decode step. */
+#define HB_PROFILE_KINDS 11
 int hb_engine_profile_step(hb_engine* e, hb_seq* const* seqs, size_t B,
                            const uint32_t* last_tokens, uint32_t* next_tokens, float* ms_by_kind);
 /* Algorithmic bytes all GEMM launches of one decode step move for batch B on this rank

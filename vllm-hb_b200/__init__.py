@@ -63,6 +63,18 @@ class ModelConfig(C.Structure):
         ("num_kv_blocks", C.c_int64),
         ("max_batch", C.c_int),
         ("force_f32", C.c_int),
+        ("max_seqs", C.c_int),
+    ]
+
+
+class StepEntry(C.Structure):
+    """hb_step_entry: the next tokens of one sequence and the places whose logits are wanted."""
+    _fields_ = [
+        ("seq", C.c_void_p),
+        ("tokens", C.c_void_p),
+        ("n_tokens", C.c_size_t),
+        ("want", C.c_void_p),
+        ("n_want", C.c_size_t),
     ]
 
 
@@ -155,6 +167,10 @@ _SIGS = {
     "hb_slot_for_position": (_i64, [_vp, _i64, _i64]),
     "hb_engine_load": (_i, [_vp, _vp, _vp]),
     "hb_engine_create_random": (_i, [_vp, _vp, _vp, _u64, _f, _i, _vp]),
+    "hb_engine_create_random_config": (_i, [C.c_char_p, _vp, _u64, _f, _vp]),
+    "hb_step": (_i, [_vp, _vp, _sz, _vp, _vp]),
+    "hb_engine_sample": (_i, [_vp, _sz, _vp, _f, _f, _vp]),
+    "hb_engine_num_free_state_slots": (_i, [_vp]),
     "hb_engine_free": (_i, [_vp]),
     "hb_engine_num_layers": (_i64, [_vp]),
     "hb_engine_vocab_size": (_i64, [_vp]),
@@ -790,19 +806,33 @@ class Engine:
 
     @staticmethod
     def _config(model_path: Optional[str], max_seq_len: int, bf16: bool, tp: int, num_kv_blocks: int,
-                max_batch: int, force_f32: bool) -> ModelConfig:
+                max_batch: int, force_f32: bool, max_seqs: int = 0) -> ModelConfig:
         return ModelConfig(model_path.encode() if model_path else None, max_seq_len, 0.9, int(bf16), tp,
-                           num_kv_blocks, max_batch, int(force_f32))
+                           num_kv_blocks, max_batch, int(force_f32), max_seqs)
 
     @classmethod
     def load(cls, model_path: str, *, max_seq_len: int = 2048, bf16: bool = True,
              tensor_parallel_size: int = 1, world: Optional[TpWorld] = None, num_kv_blocks: int = 0,
-             max_batch: int = 64, force_f32: bool = False) -> "Engine":
+             max_batch: int = 64, force_f32: bool = False, max_seqs: int = 0) -> "Engine":
+        """Any registered model family, chosen by config.json.  max_batch: rows of one step;
+        max_seqs: live sequences of a model with recurrent state (0 = max_batch)."""
         cfg = cls._config(model_path, max_seq_len, bf16, tensor_parallel_size, num_kv_blocks, max_batch,
-                          force_f32)
+                          force_f32, max_seqs)
         h = C.c_void_p()
         check(lib.hb_engine_load(C.byref(cfg), world.handle if world else None, C.byref(h)))
         return cls(h.value, world)
+
+    @classmethod
+    def create_random_config(cls, config: dict, *, seed: int = 1, std: float = 0.02, max_seq_len: int = 2048,
+                             bf16: bool = True, num_kv_blocks: int = 0, max_batch: int = 64, force_f32: bool = False,
+                             max_seqs: int = 0) -> "Engine":
+        """Random weights for a model described by its config.json as a dict."""
+        import json
+
+        cfg = cls._config(None, max_seq_len, bf16, 1, num_kv_blocks, max_batch, force_f32, max_seqs)
+        h = C.c_void_p()
+        check(lib.hb_engine_create_random_config(json.dumps(config).encode(), C.byref(cfg), seed, std, C.byref(h)))
+        return cls(h.value, None)
 
     @classmethod
     def create_random(cls, shape: dict, *, seed: int = 1, std: float = 0.02, norm_ones: bool = True,
@@ -868,6 +898,34 @@ class Engine:
                                   logits.ctypes.data if logits is not None else None))
         return next_tokens
 
+    def step(self, entries: Sequence[tuple], logits: bool = True) -> tuple[np.ndarray, Optional[np.ndarray]]:
+        """One step over any mix of prompt portions and decoded tokens.  entries: (cache, tokens,
+        want) with `want` the ascending places among `tokens` whose logits are asked for.
+        Returns (greedy next tokens [wanted], logits [wanted, vocab] or None)."""
+        arr = (StepEntry * len(entries))()
+        keep, n_want = [], 0
+        for i, (seq, tokens, want) in enumerate(entries):
+            t = np.ascontiguousarray(np.asarray(tokens, dtype=np.uint32))
+            w = np.ascontiguousarray(np.asarray(want, dtype=np.uint32))
+            keep.append((t, w))
+            arr[i] = StepEntry(seq.handle, t.ctypes.data, len(t), w.ctypes.data if len(w) else None, len(w))
+            n_want += len(w)
+        nxt = np.empty(n_want, dtype=np.uint32)
+        out = np.empty((n_want, self.vocab_size()), dtype=np.float32) if logits else None
+        check(lib.hb_step(self.handle, arr, len(entries), nxt.ctypes.data if n_want else None,
+                          out.ctypes.data if out is not None and n_want else None))
+        return nxt, out
+
+    def sample(self, seeds, temperature: float, top_p: float = 1.0) -> np.ndarray:
+        """One token per row of the last step's wanted logits, drawn on the device."""
+        s = np.ascontiguousarray(np.asarray(seeds, dtype=np.uint64))
+        out = np.empty(len(s), dtype=np.uint32)
+        check(lib.hb_engine_sample(self.handle, len(s), s.ctypes.data, float(temperature), float(top_p), out.ctypes.data))
+        return out
+
+    def num_free_state_slots(self) -> int:
+        return lib.hb_engine_num_free_state_slots(self.handle)
+
     # --- the step driven by a scheduler's block tables
     def decode_batch_tables(self, last_tokens, positions, block_tables, copy_pairs=(), logits=None) -> np.ndarray:
         """One decode step for rows whose KV lives in the caller's block tables
@@ -917,7 +975,7 @@ class Engine:
         check(lib.hb_kv_swap_blocks(self.handle, p.ctypes.data if len(p) else None, len(p), 1 if to_cpu else 0))
 
     PROFILE_KINDS = ("gemm_qkv", "attention", "rope_kv", "norm", "other", "all_reduce",
-                     "gemm_o_proj", "gemm_gate_up", "gemm_down", "gemm_lm_head")
+                     "gemm_o_proj", "gemm_gate_up", "gemm_down", "gemm_lm_head", "recurrence")
 
     def profile_step(self, seqs: Sequence[Sequence_], last_tokens: np.ndarray) -> tuple[np.ndarray, dict]:
         """One eager decode step with per-kernel-kind device times (ms)."""

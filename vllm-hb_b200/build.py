@@ -77,10 +77,12 @@ def build(force: bool = False, verbose: bool = False, variant: str = "") -> Path
     with cf.ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 1)) as ex:
         objs = list(ex.map(lambda s: _compile(s, force, verbose, obj_dir, defines), srcs))
     if force or not lib.exists() or any(o.stat().st_mtime > lib.stat().st_mtime for o in objs):
-        cmd = [_nvcc(), "-shared", "-o", str(lib), *map(str, objs), "-ldl", "-lpthread"]
+        part = lib.with_suffix(".part.so")
+        cmd = [_nvcc(), "-shared", "-o", str(part), *map(str, objs), "-ldl", "-lpthread"]
         res = subprocess.run(cmd, capture_output=True, text=True)
         if res.returncode != 0:
             raise RuntimeError(f"link failed:\n{res.stdout}\n{res.stderr}")
+        os.replace(part, lib)  # a library that exists is complete
     return lib
 
 

@@ -11,138 +11,15 @@
 //     cat-grown cache: src/worker/mod.rs:280-293, llama_tp.rs:245-259);
 //   - no allocation and no host round trip inside a step: all buffers are created at
 //     load, the step is captured once per batch size into a CUDA graph and replayed.
-#include <cmath>
-#include <deque>
-#include <map>
-#include <memory>
-#include <string>
-#include <vector>
-
-#include "comm.h"
-#include "common.h"
-#include "gemm.h"
-#include "json.h"
-#include "ops.h"
-#include "rowpar.h"
-#include "safetensors.h"
-
-struct hb_seq {
-  uint64_t id = 0;
-  std::vector<int64_t> blocks;  // physical block ids, table[pos / 16]
-  int64_t len = 0;              // tokens whose K/V are in the pool
-};
-
-namespace hb {
-
-struct LayerWeights {
-  void* wqkv = nullptr;   // [(hq_l + 2*hkv_l) * hd, H]   rows: q | k | v (column-parallel)
-  void* wo = nullptr;     // [H, hq_l * hd]               (row-parallel)
-  // Dense FFN: E = 1.  Mixture of experts: the experts' weights are concatenated, gate
-  // (w1) rows of all experts first, then their up (w3) rows; down (w2) along K.
-  void* wgu = nullptr;    // [2 * E * I_l, H]             rows: gate_0..gate_{E-1} | up_0..up_{E-1}
-  void* wdown = nullptr;  // [H, E * I_l]                 columns: expert e at [e * I_l, (e+1) * I_l)
-  void* wgate = nullptr;  // [E, H] router (replicated), null for a dense FFN
-  void* norm_in = nullptr;
-  void* norm_post = nullptr;
-};
-
-struct NamedTensor {
-  void* ptr;
-  int64_t rows, cols;
-  int64_t ld = 0;  // row stride in elements (0 = cols): expert down-projections are column blocks
-};
-
-enum GemmKind { kQkv = 0, kO = 1, kGateUp = 2, kDown = 3, kLmHead = 4 };
-constexpr int kPairCap = 1024;  // block pairs per copy launch
-
-struct StepPlans {
-  std::vector<TcGemmPlan> layer;  // [L * 4]
-  TcGemmPlan lm_head;
-  int attn_splits = 1;
-  int q_group = 1;          // prefill chunks: consecutive positions that share an attention CTA
-  bool defer_norm = false;  // add + norm folded into the GEMM epilogues (TcNormLink)
-  bool mm = false;          // exchange through the NVLink switch (multicast window of the world)
-  const void* mm_window = nullptr;  // the window the plans (and the captured graph) were made for
-  bool rope_epi = false;    // RoPE + KV write folded into the q|k|v GEMM epilogue (TcNormLink)
-  bool push = false;        // o_proj / down_proj epilogues push their partials to the reducing ranks (kEpiPush)
-  PushGeometry geo_o, geo_down;
-  int64_t launches = 0;  // kernels in one step (fixed per batch size)
-  cudaGraphExec_t graph = nullptr;
-};
-
-}  // namespace hb
-
-struct hb_engine {
-  int device = 0;
-  cudaStream_t stream = nullptr;
-  hb_world* world = nullptr;
-  int rank = 0, ws = 1;
-  hb_dtype dtype = HB_BF16;
-  size_t es = 2;
-  // shape
-  int64_t H = 0, I = 0, L = 0, hq = 0, hkv = 0, hd = 0, V = 0;
-  double eps = 1e-5, theta = 10000.0;
-  int64_t hq_l = 0, hkv_l = 0, I_l = 0, qkv_rows = 0;
-  // mixture of experts (mixtral.rs:40-57): E experts, top-k routing, sliding window; I_e = E * I_l
-  int64_t E = 1, topk = 1, window = 0, I_e = 0;
-  bool moe = false;
-  float* d_scale = nullptr;  // [max_batch, E] routing weights of the step
-  float* d_rowsq = nullptr;  // [max_batch, rowsq_stride] row sums of the deferred norm
-  float2* d_rope_cs = nullptr;  // [max_batch, hd/2] (cos, sin) of the step's positions
-  int rowsq_stride = 0;
-  // weights
-  void* embed = nullptr;
-  void* lm_head = nullptr;
-  void* final_norm = nullptr;
-  std::vector<hb::LayerWeights> layers;
-  std::map<std::string, hb::NamedTensor> named;
-  std::vector<void*> allocations;
-  // KV pool
-  int64_t num_blocks = 0;
-  std::vector<void*> kc, vc;
-  std::deque<int64_t> free_blocks;  // FIFO: pop front / push back (block_manager.rs:58,63-83)
-  uint64_t next_seq_id = 0;
-  // step buffers
-  int max_batch = 0;
-  int64_t max_blocks_per_seq = 0;
-  uint8_t* d_inputs = nullptr;  // [ids | positions | ctx | pad | slots | tables]
-  uint8_t* h_inputs = nullptr;  // pinned mirror
-  size_t inputs_bytes = 0;
-  size_t off_ids = 0, off_pos = 0, off_ctx = 0, off_slots = 0, off_tables = 0;
-  void *d_h = nullptr, *d_x = nullptr, *d_qkv = nullptr, *d_attn = nullptr, *d_gu = nullptr,
-       *d_act = nullptr, *d_proj = nullptr;
-  float* d_logits = nullptr;
-  uint32_t* d_next = nullptr;
-  uint32_t* h_next = nullptr;  // pinned
-  float* d_inv_freq = nullptr;
-  void* d_attn_ws = nullptr;
-  size_t attn_ws_bytes = 0;
-  void* d_gemm_ws = nullptr;
-  size_t gemm_ws_bytes = 0;
-  int* d_err = nullptr;
-  int64_t* d_pairs = nullptr;   // (src, dst) block ids of a copy request, kPairCap pairs at a time
-  uint8_t* h_swap = nullptr;    // pinned CPU block pool [cpu_blocks][L][K|V][block bytes] (hb_engine_reserve_cpu_blocks)
-  int64_t cpu_blocks = 0;
-  bool use_tc = false, use_graph = true, fused_swiglu = true;
-  std::map<int, hb::StepPlans> plans;
-  cudaEvent_t ev0 = nullptr, ev1 = nullptr;
-  float last_ms = -1.f;
-  int64_t last_launches = 0;
-  // per-kernel-kind timing of one eager step (hb_engine_profile_step)
-  bool profiling = false;
-  bool prof_capture = false;  // the profiled step is being captured: events become graph nodes
-  std::vector<cudaEvent_t> prof_events;
-  std::vector<int> prof_cats;
-  size_t prof_used = 0;
-  float prof_ms[16] = {0};
-};
+#include "engine.h"
 
 namespace hb {
 
 // ------------------------------------------------------------------ host helpers
-static int dev_alloc(hb_engine* e, void** p, size_t bytes) {
+int dev_alloc(hb_engine* e, void** p, size_t bytes, bool zero) {
   HB_CUDA_CHECK(cudaMalloc(p, bytes ? bytes : 16));
   e->allocations.push_back(*p);
+  if (zero) HB_CUDA_CHECK(cudaMemsetAsync(*p, 0, bytes ? bytes : 16, e->stream));
   return HB_OK;
 }
 
@@ -154,7 +31,7 @@ static hb_dtype st_dtype(const std::string& s) { return s == "F32" ? HB_F32 : s 
 
 // Rows [r0, r0+nr) x cols [c0, c0+nc) of a [rows, cols] tensor of the memory-mapped
 // checkpoint go to device memory at dst (row-major [nr, nc], row stride dst_ld elements) in
-// the engine dtype — the narrow() of column_shard / row_shard (src/parallel/shard.rs:46-74)
+// `dst_dtype` (the engine's for matrices) — the narrow() of column_shard / row_shard (src/parallel/shard.rs:46-74)
 // followed by to_device, without the reference's full CPU copy in the target dtype
 // (llama_tp.rs:367-377): only this rank's slice leaves the page cache, as one strided copy
 // straight from the mapping, and a checkpoint in another dtype is converted on the device.
@@ -165,15 +42,15 @@ struct UploadStage {
   ~UploadStage() { if (buf) cudaFree(buf); }
 };
 
-static int upload_slice(hb_engine* e, void* dst, const StTensor& t, int64_t cols, int64_t r0,
+static int upload_slice(hb_engine* e, void* dst, hb_dtype dst_dtype, const StTensor& t, int64_t cols, int64_t r0,
                         int64_t nr, int64_t c0, int64_t nc, UploadStage* stage, int64_t dst_ld = 0) {
   const size_t src_es = t.dtype == "F32" ? 4 : 2;
   const uint8_t* src = t.data + ((size_t)r0 * cols + c0) * src_es;
   if (dst_ld <= 0) dst_ld = nc;
   // every copy and conversion is ordered on the engine's stream; hb_engine_load synchronises it
   // before the mapping goes away
-  if (same_dtype(t.dtype, e->dtype)) {
-    HB_CUDA_CHECK(cudaMemcpy2DAsync(dst, (size_t)dst_ld * e->es, src, (size_t)cols * src_es, (size_t)nc * src_es,
+  if (same_dtype(t.dtype, dst_dtype)) {
+    HB_CUDA_CHECK(cudaMemcpy2DAsync(dst, (size_t)dst_ld * src_es, src, (size_t)cols * src_es, (size_t)nc * src_es,
                                     (size_t)nr, cudaMemcpyHostToDevice, e->stream));
     return HB_OK;
   }
@@ -188,11 +65,78 @@ static int upload_slice(hb_engine* e, void* dst, const StTensor& t, int64_t cols
   }
   HB_CUDA_CHECK(cudaMemcpy2DAsync(stage->buf, (size_t)nc * src_es, src, (size_t)cols * src_es, (size_t)nc * src_es,
                                   (size_t)nr, cudaMemcpyHostToDevice, e->stream));
-  int rc = convert_2d(e->stream, dst, e->dtype, dst_ld, stage->buf, st_dtype(t.dtype), nr, nc);
+  int rc = convert_2d(e->stream, dst, dst_dtype, dst_ld, stage->buf, st_dtype(t.dtype), nr, nc);
   if (rc) return rc;
   HB_CUDA_CHECK(cudaStreamSynchronize(e->stream));  // the stage is reused by the next slice
   return HB_OK;
 }
+
+// The *.safetensors shards of a model folder, memory-mapped.
+class CheckpointSource : public TensorSource {
+ public:
+  explicit CheckpointSource(hb_engine* e) : e_(e) {}
+  int open(const std::string& dir) {
+    std::vector<std::string> files;
+    int rc = list_safetensors(dir, &files);
+    if (rc) return rc;
+    for (auto& f : files) {
+      shards_.emplace_back(new SafetensorsFile);
+      if ((rc = shards_.back()->open(f))) return rc;
+      for (auto& kv : shards_.back()->tensors()) all_[kv.first] = &kv.second;
+    }
+    return HB_OK;
+  }
+  bool has(const std::string& name) const override { return all_.count(name) != 0; }
+  std::vector<int64_t> shape(const std::string& name) const override {
+    auto it = all_.find(name);
+    return it == all_.end() ? std::vector<int64_t>() : it->second->shape;
+  }
+  int fetch(const std::string& name, int64_t rows, int64_t cols, int64_t r0, int64_t nr, int64_t c0, int64_t nc, void* dst,
+            hb_dtype dst_dtype, int64_t dst_ld) override {
+    auto it = all_.find(name);
+    if (it == all_.end()) return fail(HB_ERR_IO, "Weight not found: %s", name.c_str());  // llama_tp.rs:380-385
+    const StTensor* s = it->second;
+    if (s->dtype != "F32" && s->dtype != "F16" && s->dtype != "BF16")
+      return fail(HB_ERR_UNSUPPORTED_DTYPE, "%s has dtype %s", name.c_str(), s->dtype.c_str());
+    // the shape itself, not only the element count: a transposed matrix must not be sharded
+    const bool shape_ok = (s->shape.size() == 2 && s->shape[0] == rows && s->shape[1] == cols) ||
+                          (rows == 1 && s->shape.size() == 1 && s->shape[0] == cols);
+    if (!shape_ok)
+      return fail(HB_ERR_IO, "%s has %lld elements in a shape other than the expected [%lld, %lld]", name.c_str(),
+                  (long long)s->numel(), (long long)rows, (long long)cols);
+    const size_t src_es = s->dtype == "F32" ? 4 : 2;
+    if (s->nbytes != (size_t)(rows * cols) * src_es)
+      return fail(HB_ERR_IO, "%s holds %zu bytes, [%lld, %lld] of %s needs %zu", name.c_str(), s->nbytes,
+                  (long long)rows, (long long)cols, s->dtype.c_str(), (size_t)(rows * cols) * src_es);
+    return upload_slice(e_, dst, dst_dtype, *s, cols, r0, nr, c0, nc, &stage_, dst_ld);
+  }
+
+ private:
+  hb_engine* e_;
+  UploadStage stage_;
+  std::vector<std::unique_ptr<SafetensorsFile>> shards_;
+  std::map<std::string, const StTensor*> all_;
+};
+
+// Weights drawn on the device: N(0, std), every tensor from a stream keyed by its name.
+class RandomSource : public TensorSource {
+ public:
+  RandomSource(hb_engine* e, uint64_t seed, float std) : e_(e), seed_(seed), std_(std) {}
+  bool has(const std::string&) const override { return true; }
+  std::vector<int64_t> shape(const std::string&) const override { return {}; }
+  bool generated() const override { return true; }
+  int fetch(const std::string& name, int64_t rows, int64_t cols, int64_t r0, int64_t nr, int64_t c0, int64_t nc, void* dst,
+            hb_dtype dst_dtype, int64_t dst_ld) override {
+    uint64_t id = 1469598103934665603ull;
+    for (char c : name) id = (id ^ (uint8_t)c) * 1099511628211ull;
+    return fill_normal(e_->stream, dst, dst_dtype, nr, nc, r0, c0, cols, seed_, id, std_, dst_ld);
+  }
+
+ private:
+  hb_engine* e_;
+  uint64_t seed_;
+  float std_;
+};
 
 static int check_divisibility(const hb_engine* e) {
   // TpLlamaBackend::load (src/engine/arch/llama_tp.rs:407-427)
@@ -325,7 +269,10 @@ static int alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
     HB_CUDA_CHECK(cudaMemset(e->kc[l], 0, blk_bytes * e->num_blocks));
     HB_CUDA_CHECK(cudaMemset(e->vc[l], 0, blk_bytes * e->num_blocks));
   }
+  e->k_block_bytes.assign(e->L, blk_bytes);
+  e->v_block_bytes.assign(e->L, blk_bytes);
   for (int64_t b = 0; b < e->num_blocks; ++b) e->free_blocks.push_back(b);
+  e->max_logits_rows = e->max_batch;
 
   const int B = e->max_batch;
   auto align16 = [](size_t v) { return (v + 15) / 16 * 16; };
@@ -367,6 +314,24 @@ static int alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
 }
 
 // ------------------------------------------------------------------ step
+int ensure_gemm_workspace(hb_engine* e, size_t ws) {
+  if (ws <= e->gemm_ws_bytes) return HB_OK;
+  // grows only when a new batch size needs more; never inside a captured step
+  void* p = nullptr;
+  HB_CUDA_CHECK(cudaMalloc(&p, ws));
+  HB_CUDA_CHECK(cudaMemset(p, 0, ws));
+  e->allocations.push_back(p);
+  e->d_gemm_ws = p;
+  e->gemm_ws_bytes = ws;
+  // graphs captured with the old scratch are dropped (it stays allocated until the engine goes)
+  for (auto& kv : e->plans)
+    if (kv.second.graph) { cudaGraphExecDestroy(kv.second.graph); kv.second.graph = nullptr; }
+  if (e->lm)
+    for (auto& kv : e->lm->graphs)
+      if (kv.second.exec) { cudaGraphExecDestroy(kv.second.exec); kv.second.exec = nullptr; }
+  return HB_OK;
+}
+
 static int pick_attn_splits(const hb_engine* e, int B) {
   DeviceInfo di;
   if (device_info(e->device, &di)) return 1;
@@ -479,17 +444,9 @@ static int ensure_plans(hb_engine* e, int B, bool chunk, StepPlans** out) {
       }
     }
   }
-  if (ws > e->gemm_ws_bytes) {
-    // grows only when a new batch size needs more; never inside a captured step
-    void* p = nullptr;
-    HB_CUDA_CHECK(cudaMalloc(&p, ws));
-    HB_CUDA_CHECK(cudaMemset(p, 0, ws));
-    e->allocations.push_back(p);
-    e->d_gemm_ws = p;
-    e->gemm_ws_bytes = ws;
-    // plans made for other batch sizes keep pointing at buffers that stay allocated
-    for (auto& kv : e->plans)
-      if (kv.second.graph) { cudaGraphExecDestroy(kv.second.graph); kv.second.graph = nullptr; }
+  {
+    const int rc = ensure_gemm_workspace(e, ws);
+    if (rc) return rc;
   }
   auto ins = e->plans.emplace(key, std::move(sp));
   *out = &ins.first->second;
@@ -506,12 +463,8 @@ static int run_gemm(hb_engine* e, StepPlans* sp, int64_t l, int kind, void* Y, c
   return gemm_simt(e->stream, Y, X, W, B, N, K, e->dtype, out_f32);
 }
 
-// kCatGemm is the QKV projection; the other projections have kinds of their own
-enum ProfCat { kCatGemm = 0, kCatAttention = 1, kCatRopeKv = 2, kCatNorm = 3, kCatOther = 4, kCatComm = 5,
-               kCatGemmO = 6, kCatGemmGateUp = 7, kCatGemmDown = 8, kCatGemmLmHead = 9, kNumCats = 10 };
-
 // While profiling, every call opens a timed segment of kind `cat` on the stream.
-static void prof_mark(hb_engine* e, int cat) {
+void prof_mark(hb_engine* e, int cat) {
   if (!e->profiling) return;
   if (e->prof_used == e->prof_events.size()) {
     cudaEvent_t ev = nullptr;
@@ -737,25 +690,29 @@ static int seq_ensure_block(hb_engine* e, hb_seq* s, int64_t pos) {
   return HB_OK;
 }
 
-// One row of a step: token `tok` of sequence `s` at position `pos`.  A decode step has one
-// row per sequence; a prefill chunk has consecutive positions of ONE sequence as its rows
-// (row i then attends to the keys of rows 0..i, which the same step wrote before its
-// attention kernel runs: causal attention over the growing cache, llama_tp.rs:313-316).
-struct StepRow {
-  const int64_t* blocks;  // the sequence's block table (ids into the KV pool), table[pos / 16]
-  size_t n_blocks;
-  int64_t pos;
-  uint32_t tok;
-};
+// Blocks (and, for a model with recurrent state, the state slot) that the next `n` tokens of a
+// sequence need.
+static int seq_reserve(hb_engine* e, hb_seq* s, int64_t n) {
+  if (e->max_positions > 0 && s->len + n > e->max_positions)
+    return fail(HB_ERR_INVALID_ARG, "sequence of %lld tokens exceeds the model's %lld positions", (long long)(s->len + n),
+                (long long)e->max_positions);
+  int rc = seq_ensure_block(e, s, s->len + n - 1);
+  if (rc) return rc;
+  if (e->num_state_slots > 0 && s->state_slot < 0) {
+    if (e->free_slots.empty())
+      return fail(HB_ERR_OOM_BLOCKS, "no free state slot (%d sequences may be live)", e->num_state_slots);
+    s->state_slot = e->free_slots.front();
+    e->free_slots.pop_front();
+  }
+  return HB_OK;
+}
 
-static int run_rows(hb_engine* e, const StepRow* rows, int B, uint32_t* next_tokens, float* logits_out,
-                    int logits_row0, bool chunk = false);
+static int run_step(hb_engine* e, const StepBatch& batch, uint32_t* next_tokens, float* logits_out);
 
 static int decode_step(hb_engine* e, hb_seq* const* seqs, int B, const uint32_t* tokens,
                        uint32_t* next_tokens, float* logits_out /* host [B, V] or null */) {
   if (B <= 0 || B > e->max_batch)
     return fail(HB_ERR_INVALID_ARG, "batch %d outside [1, %d]", B, e->max_batch);
-  std::vector<StepRow> rows((size_t)B);
   for (int b = 0; b < B; ++b) {
     hb_seq* s = seqs[b];
     if (!s) return fail(HB_ERR_INVALID_ARG, "null sequence at index %d", b);
@@ -763,11 +720,16 @@ static int decode_step(hb_engine* e, hb_seq* const* seqs, int B, const uint32_t*
       if (seqs[j] == s) return fail(HB_ERR_INVALID_ARG, "sequence repeated in one batch");
   }
   int rc;
+  StepBatch batch;
+  batch.segs.reserve((size_t)B);
+  batch.want.resize((size_t)B);
   for (int b = 0; b < B; ++b)
-    if ((rc = seq_ensure_block(e, seqs[b], seqs[b]->len))) return rc;
-  for (int b = 0; b < B; ++b) rows[b] = {seqs[b]->blocks.data(), seqs[b]->blocks.size(), seqs[b]->len, tokens[b]};
-  rc = run_rows(e, rows.data(), B, next_tokens, logits_out, 0);
-  if (rc) return rc;
+    if ((rc = seq_reserve(e, seqs[b], 1))) return rc;
+  for (int b = 0; b < B; ++b) {
+    batch.add(seqs[b]->blocks.data(), seqs[b]->blocks.size(), seqs[b]->len, tokens + b, 1, seqs[b]->state_slot);
+    batch.want[b] = b;
+  }
+  if ((rc = run_step(e, batch, next_tokens, logits_out))) return rc;
   for (int b = 0; b < B; ++b) seqs[b]->len += 1;
   return HB_OK;
 }
@@ -776,90 +738,119 @@ static int decode_step(hb_engine* e, hb_seq* const* seqs, int B, const uint32_t*
 // logits of the last token go to logits_out (host [V]) when it is not null.
 static int prefill(hb_engine* e, hb_seq* s, const uint32_t* ids, size_t n, float* logits_out,
                    bool all_positions = false) {
-  std::vector<StepRow> rows;
   size_t done = 0;
+  const size_t cap = (size_t)(all_positions ? std::min(e->max_batch, e->max_logits_rows) : e->max_batch);
   while (done < n) {
-    const int c = (int)std::min<size_t>(n - done, (size_t)e->max_batch);
-    rows.resize((size_t)c);
+    const int c = (int)std::min<size_t>(n - done, cap);
     int rc;
-    if ((rc = seq_ensure_block(e, s, s->len + c - 1))) return rc;
-    for (int i = 0; i < c; ++i) rows[i] = {s->blocks.data(), s->blocks.size(), s->len + i, ids[done + i]};
+    if ((rc = seq_reserve(e, s, c))) return rc;
+    StepBatch batch;
+    batch.add(s->blocks.data(), s->blocks.size(), s->len, ids + done, c, s->state_slot);
     const bool last = done + (size_t)c == n;
-    if (all_positions) rc = run_rows(e, rows.data(), c, nullptr, logits_out + done * (size_t)e->V, 0, true);
-    else rc = run_rows(e, rows.data(), c, nullptr, last ? logits_out : nullptr, c - 1, true);
-    if (rc) return rc;
+    if (all_positions) for (int i = 0; i < c; ++i) batch.want.push_back(i);
+    else if (last && logits_out) batch.want.push_back(c - 1);
+    if ((rc = run_step(e, batch, nullptr, all_positions ? logits_out + done * (size_t)e->V : logits_out))) return rc;
     s->len += c;
     done += (size_t)c;
   }
   return HB_OK;
 }
 
-static int run_rows(hb_engine* e, const StepRow* rows, int B, uint32_t* next_tokens, float* logits_out,
-                    int logits_row0, bool chunk) {
-  HB_CUDA_CHECK(cudaSetDevice(e->device));
-  int rc;
+// Llama family: every batch row has its own position, context length, KV slot and block table.
+static int llama_prepare(hb_engine* e, const StepBatch& batch, StepExec* x) {
   uint32_t* h_ids = (uint32_t*)(e->h_inputs + e->off_ids);
   int32_t* h_pos = (int32_t*)(e->h_inputs + e->off_pos);
   int32_t* h_ctx = (int32_t*)(e->h_inputs + e->off_ctx);
   int64_t* h_slots = (int64_t*)(e->h_inputs + e->off_slots);
   int32_t* h_tables = (int32_t*)(e->h_inputs + e->off_tables);
-  for (int b = 0; b < B; ++b) {
-    const StepRow& r = rows[b];
-    const int64_t pos = r.pos;
-    // the reference's embedding lookup fails on an id outside the vocabulary
-    // (index_select, llama_tp.rs:213-216); so does this
-    if ((int64_t)r.tok >= e->V)
-      return fail(HB_ERR_INVALID_ARG, "token id %u at row %d is outside the vocabulary of %lld", r.tok, b,
-                  (long long)e->V);
-    const int64_t need = pos / HB_BLOCK_SIZE + 1;
-    if (pos < 0 || (int64_t)r.n_blocks < need || need > e->max_blocks_per_seq)
-      return fail(HB_ERR_INVALID_ARG, "row %d: a block table of %zu block(s) does not cover position %lld", b,
-                  r.n_blocks, (long long)pos);
-    for (int64_t i = 0; i < need; ++i)
-      if (r.blocks[i] < 0 || r.blocks[i] >= e->num_blocks)
-        return fail(HB_ERR_INVALID_ARG, "row %d: block id %lld outside the pool of %lld", b, (long long)r.blocks[i],
-                    (long long)e->num_blocks);
-    h_ids[b] = r.tok;
-    h_pos[b] = (int32_t)pos;
-    h_ctx[b] = (int32_t)(pos + 1);
-    h_slots[b] = r.blocks[pos / HB_BLOCK_SIZE] * HB_BLOCK_SIZE + pos % HB_BLOCK_SIZE;
-    int32_t* row = h_tables + (size_t)b * e->max_blocks_per_seq;
-    for (int64_t i = 0; i < need; ++i) row[i] = (int32_t)r.blocks[i];
-  }
-  StepPlans* sp = nullptr;
-  if ((rc = ensure_plans(e, B, chunk, &sp))) return rc;
+  for (const StepSeg& g : batch.segs)
+    for (int i = 0; i < g.n; ++i) {
+      const int b = g.row0 + i;
+      const int64_t pos = g.pos0 + i, need = pos / HB_BLOCK_SIZE + 1;
+      h_ids[b] = g.tokens[i];
+      h_pos[b] = (int32_t)pos;
+      h_ctx[b] = (int32_t)(pos + 1);
+      h_slots[b] = g.blocks[pos / HB_BLOCK_SIZE] * HB_BLOCK_SIZE + pos % HB_BLOCK_SIZE;
+      int32_t* row = h_tables + (size_t)b * e->max_blocks_per_seq;
+      for (int64_t k = 0; k < need; ++k) row[k] = (int32_t)g.blocks[k];
+    }
+  // rows that are consecutive positions of ONE sequence may share the attention's K/V stream
+  const bool chunk = batch.segs.size() == 1 && batch.rows > 1;
+  int rc = ensure_plans(e, batch.rows, chunk, &x->plans);
+  if (rc) return rc;
+  x->rows = batch.rows;
   // only the used prefix of each region matters; one copy of the whole block is simplest
-  HB_CUDA_CHECK(cudaMemcpyAsync(e->d_inputs, e->h_inputs, e->inputs_bytes, cudaMemcpyHostToDevice, e->stream));
-  if (e->use_graph && !e->profiling) {
-    if (!sp->graph) {
+  x->input_bytes = e->inputs_bytes;
+  x->graph = &x->plans->graph;
+  x->graph_launches = &x->plans->launches;
+  x->logits_compact = false;
+  return HB_OK;
+}
+
+static int llama_issue(hb_engine* e, const StepExec& x) { return issue_step(e, x.plans, x.rows); }
+
+// One step of any model family: the batch is checked, its inputs are uploaded in one copy, the
+// kernels replay from a graph (or are issued on the stream), the wanted rows come back.
+static int run_step(hb_engine* e, const StepBatch& batch, uint32_t* next_tokens, float* logits_out) {
+  HB_CUDA_CHECK(cudaSetDevice(e->device));
+  int rc;
+  const int n_want = (int)batch.want.size();
+  if (batch.rows < 1 || batch.rows > e->max_batch)
+    return fail(HB_ERR_INVALID_ARG, "batch %d outside [1, %d]", batch.rows, e->max_batch);
+  if (n_want > e->max_logits_rows)
+    return fail(HB_ERR_INVALID_ARG, "logits of %d rows asked for, %d at most", n_want, e->max_logits_rows);
+  for (const StepSeg& g : batch.segs) {
+    for (int i = 0; i < g.n; ++i)
+      // the reference's embedding lookup fails on an id outside the vocabulary
+      // (index_select, llama_tp.rs:213-216); so does this
+      if ((int64_t)g.tokens[i] >= e->V)
+        return fail(HB_ERR_INVALID_ARG, "token id %u at row %d is outside the vocabulary of %lld", g.tokens[i], g.row0 + i,
+                    (long long)e->V);
+    const int64_t last = g.pos0 + g.n - 1, need = last / HB_BLOCK_SIZE + 1;
+    if (g.pos0 < 0 || (int64_t)g.n_blocks < need || need > e->max_blocks_per_seq)
+      return fail(HB_ERR_INVALID_ARG, "row %d: a block table of %zu block(s) does not cover position %lld", g.row0 + g.n - 1,
+                  g.n_blocks, (long long)last);
+    for (int64_t i = 0; i < need; ++i)
+      if (g.blocks[i] < 0 || g.blocks[i] >= e->num_blocks)
+        return fail(HB_ERR_INVALID_ARG, "row %d: block id %lld outside the pool of %lld", g.row0, (long long)g.blocks[i],
+                    (long long)e->num_blocks);
+    if (e->num_state_slots > 0 && (g.state_slot < 0 || g.state_slot >= e->num_state_slots))
+      return fail(HB_ERR_INVALID_ARG, "row %d: this model keeps recurrent state; its sequences need engine handles", g.row0);
+  }
+  StepExec x;
+  if ((rc = e->family->prepare(e, batch, &x))) return rc;
+  HB_CUDA_CHECK(cudaMemcpyAsync(e->d_inputs, e->h_inputs, x.input_bytes, cudaMemcpyHostToDevice, e->stream));
+  if (e->use_graph && !e->profiling && x.graph) {
+    if (!*x.graph) {
       cudaGraph_t g = nullptr;
       HB_CUDA_CHECK(cudaStreamBeginCapture(e->stream, cudaStreamCaptureModeThreadLocal));
-      rc = issue_step(e, sp, B);
-      sp->launches = e->last_launches;
+      e->last_launches = 0;
+      rc = e->family->issue(e, x);
+      *x.graph_launches = e->last_launches;
       cudaError_t ce = cudaStreamEndCapture(e->stream, &g);
       if (rc) { if (g) cudaGraphDestroy(g); return rc; }
       if (ce != cudaSuccess) return fail(HB_ERR_CUDA, "graph capture failed: %s", cudaGetErrorString(ce));
-      ce = cudaGraphInstantiate(&sp->graph, g, 0);
+      ce = cudaGraphInstantiate(x.graph, g, 0);
       cudaGraphDestroy(g);
       if (ce != cudaSuccess) return fail(HB_ERR_CUDA, "graph instantiate failed: %s", cudaGetErrorString(ce));
     }
-    e->last_launches = sp->launches;
+    e->last_launches = *x.graph_launches;
     HB_CUDA_CHECK(cudaEventRecord(e->ev0, e->stream));
-    HB_CUDA_CHECK(cudaGraphLaunch(sp->graph, e->stream));
+    HB_CUDA_CHECK(cudaGraphLaunch(*x.graph, e->stream));
     HB_CUDA_CHECK(cudaEventRecord(e->ev1, e->stream));
   } else {
     // Profiling.  With graphs enabled the step is captured once more with an event-record
     // node between the kernels and replayed, so that the per-kind times are those of the
     // kernels inside a graph (a failed capture: kernel by kernel
     // on the stream, which adds the launch gaps).
-    const bool eager_only = false;
     bool done = false;
-    if (e->profiling && e->use_graph && !eager_only) {
+    e->last_launches = 0;
+    if (e->profiling && e->use_graph) {
       cudaGraph_t g = nullptr;
       cudaGraphExec_t ge = nullptr;
       if (cudaStreamBeginCapture(e->stream, cudaStreamCaptureModeThreadLocal) == cudaSuccess) {
         e->prof_capture = true;
-        rc = issue_step(e, sp, B);
+        rc = e->family->issue(e, x);
         e->prof_capture = false;
         cudaError_t ce = cudaStreamEndCapture(e->stream, &g);
         if (!rc && ce == cudaSuccess && cudaGraphInstantiate(&ge, g, 0) == cudaSuccess) {
@@ -873,18 +864,30 @@ static int run_rows(hb_engine* e, const StepRow* rows, int B, uint32_t* next_tok
         if (g) cudaGraphDestroy(g);
         cudaGetLastError();
       }
-      if (!done) { e->prof_used = 0; e->prof_cats.clear(); }
+      if (!done) { e->prof_used = 0; e->prof_cats.clear(); e->last_launches = 0; }
     }
     if (!done) {
       HB_CUDA_CHECK(cudaEventRecord(e->ev0, e->stream));
-      if ((rc = issue_step(e, sp, B))) return rc;
+      if ((rc = e->family->issue(e, x))) return rc;
       HB_CUDA_CHECK(cudaEventRecord(e->ev1, e->stream));
     }
   }
-  HB_CUDA_CHECK(cudaMemcpyAsync(e->h_next, e->d_next, (size_t)B * 4, cudaMemcpyDeviceToHost, e->stream));
-  if (logits_out)
-    HB_CUDA_CHECK(cudaMemcpyAsync(logits_out, e->d_logits + (size_t)logits_row0 * e->V,
-                                  (size_t)(B - logits_row0) * e->V * 4, cudaMemcpyDeviceToHost, e->stream));
+  // wanted rows back to the host: runs of neighbouring logits rows go as one copy
+  auto row_of = [&](int i) { return x.logits_compact ? i : batch.want[i]; };
+  e->last_rows.clear();
+  if (n_want > 0) {
+    const int n_rows = x.logits_compact ? n_want : batch.rows;
+    if (next_tokens)
+      HB_CUDA_CHECK(cudaMemcpyAsync(e->h_next, e->d_next, (size_t)n_rows * 4, cudaMemcpyDeviceToHost, e->stream));
+    if (logits_out)
+      for (int i = 0; i < n_want;) {
+        int j = i + 1;
+        while (j < n_want && row_of(j) == row_of(j - 1) + 1) ++j;
+        HB_CUDA_CHECK(cudaMemcpyAsync(logits_out + (size_t)i * e->V, e->d_logits + (size_t)row_of(i) * e->V,
+                                      (size_t)(j - i) * e->V * 4, cudaMemcpyDeviceToHost, e->stream));
+        i = j;
+      }
+  }
   int h_err = 0;
   HB_CUDA_CHECK(cudaMemcpyAsync(&h_err, e->d_err, 4, cudaMemcpyDeviceToHost, e->stream));
   HB_CUDA_CHECK(cudaStreamSynchronize(e->stream));
@@ -907,10 +910,161 @@ static int run_rows(hb_engine* e, const StepRow* rows, int B, uint32_t* next_tok
     const int stw = hb_world_status(e->world);
     if (stw) return fail(stw, "a peer did not arrive in the all-reduce of the decode step");
   }
-  for (int b = 0; b < B; ++b)
-    if (next_tokens) next_tokens[b] = e->h_next[b];
+  if (next_tokens)
+    for (int i = 0; i < n_want; ++i) next_tokens[i] = e->h_next[row_of(i)];
+  for (int i = 0; i < n_want; ++i) e->last_rows.push_back(row_of(i));
   return HB_OK;
 }
+
+// Any mix of prompt portions and decoded tokens, one entry per sequence.  Entries whose rows (or
+// wanted rows) exceed what one step can hold are cut; everything else is one batch.
+static int mixed_step(hb_engine* e, const hb_step_entry* entries, size_t n, uint32_t* next_tokens, float* logits_out) {
+  for (size_t i = 0; i < n; ++i) {
+    const hb_step_entry& t = entries[i];
+    if (!t.seq || !t.tokens) return fail(HB_ERR_INVALID_ARG, "hb_step: null sequence or tokens at entry %zu", i);
+    if (t.n_tokens == 0) return fail(HB_ERR_EMPTY, "hb_step: entry %zu brings no tokens", i);
+    for (size_t j = 0; j < i; ++j)
+      if (entries[j].seq == t.seq) return fail(HB_ERR_INVALID_ARG, "hb_step: sequence repeated in one step");
+    for (size_t k = 0; k < t.n_want; ++k)
+      if (t.want[k] >= t.n_tokens || (k && t.want[k] <= t.want[k - 1]))
+        return fail(HB_ERR_INVALID_ARG, "hb_step: wanted places of entry %zu must ascend below %zu", i, t.n_tokens);
+    for (size_t k = 0; k < t.n_tokens; ++k)
+      if ((int64_t)t.tokens[k] >= e->V)
+        return fail(HB_ERR_INVALID_ARG, "token id %u of entry %zu is outside the vocabulary of %lld", t.tokens[k], i,
+                    (long long)e->V);
+  }
+  size_t i = 0, off = 0, w = 0, out = 0;  // entry, its next token, its next wanted place, results so far
+  while (i < n) {
+    StepBatch batch;
+    std::vector<std::pair<hb_seq*, int>> fed;
+    const size_t out0 = out;
+    while (i < n && batch.rows < e->max_batch && (int)batch.segs.size() < e->max_batch) {
+      const hb_step_entry& t = entries[i];
+      int64_t c = std::min<int64_t>((int64_t)(t.n_tokens - off), e->max_batch - batch.rows);
+      // no more wanted rows than the logits buffer holds
+      const size_t room = (size_t)e->max_logits_rows - batch.want.size();
+      if (w + room < t.n_want) c = std::min<int64_t>(c, (int64_t)t.want[w + room] - (int64_t)off);
+      if (c <= 0) break;
+      int rc = seq_reserve(e, t.seq, c);
+      if (rc) return rc;
+      for (; w < t.n_want && t.want[w] < off + (size_t)c; ++w, ++out)
+        batch.want.push_back(batch.rows + (int)(t.want[w] - off));
+      batch.add(t.seq->blocks.data(), t.seq->blocks.size(), t.seq->len, t.tokens + off, (int)c, t.seq->state_slot);
+      fed.emplace_back(t.seq, (int)c);
+      off += (size_t)c;
+      if (off < t.n_tokens) break;
+      ++i;
+      off = w = 0;
+    }
+    int rc = run_step(e, batch, next_tokens ? next_tokens + out0 : nullptr,
+                      logits_out ? logits_out + out0 * (size_t)e->V : nullptr);
+    if (rc) return rc;
+    for (auto& f : fed) f.first->len += f.second;
+  }
+  return HB_OK;
+}
+
+static double llama_step_bytes(const hb_engine* e, const int32_t* ctx_lens, int64_t n_seqs) {
+  const double es = (double)e->es;
+  double w = 0.0;
+  w += (double)e->L * ((double)e->qkv_rows * e->H + (double)e->H * e->hq_l * e->hd +
+                       3.0 * (double)e->I_e * e->H + (e->moe ? (double)e->E * e->H : 0.0) + 2.0 * e->H) * es;
+  w += ((double)e->V * e->H + e->H) * es;    // lm_head + final norm
+  w += (double)n_seqs * e->H * es;            // embedding rows
+  double kv = 0.0;
+  for (int64_t i = 0; i < n_seqs; ++i)
+    kv += (double)(ctx_lens ? ctx_lens[i] : 0) * e->L * 2.0 * e->hkv_l * e->hd * es;  // read
+  kv += (double)n_seqs * e->L * 2.0 * e->hkv_l * e->hd * es;                           // write
+  return w + kv;
+}
+
+static double llama_gemm_bytes(const hb_engine* e, int64_t B) {
+  const double es = (double)e->es, b = (double)B;
+  const double qkv = (double)e->qkv_rows, o_in = (double)e->hq_l * e->hd, H = (double)e->H,
+               Il = (double)e->I_e, V = (double)e->V;
+  double per_layer = (qkv * H + b * H + b * qkv) * es        // q|k|v projection
+                     + (H * o_in + b * o_in + b * H) * es    // o_proj
+                     + (2 * Il * H + b * H + b * Il) * es    // gate|up with the SwiGLU epilogue
+                     + (H * Il + b * Il + b * H) * es;       // down_proj
+  return (double)e->L * per_layer + (V * H + b * H) * es + b * V * 4.0;  // + lm_head, fp32 logits
+}
+
+// ------------------------------------------------------------------ Llama family: load
+static bool llama_serves(const Json& root) { return !root.get("architecture"); }
+
+static int llama_configure(hb_engine* e, const Json& root) {
+  const std::string mt = root.string_or("model_type", "llama");
+  if (mt != "llama" && mt != "mistral" && mt != "mixtral")
+    return fail(HB_ERR_INVALID_ARG, "model_type '%s' is not served by this path (llama, mistral, mixtral)",
+                    mt.c_str());
+  const bool mixtral = mt == "mixtral";
+  hb_model_shape sh;
+  memset(&sh, 0, sizeof(sh));
+  sh.hidden_size = (int64_t)root.number_or("hidden_size", 0);
+  sh.intermediate_size = (int64_t)root.number_or("intermediate_size", 0);
+  sh.num_hidden_layers = (int64_t)root.number_or("num_hidden_layers", 0);
+  sh.num_attention_heads = (int64_t)root.number_or("num_attention_heads", 0);
+  sh.num_key_value_heads = (int64_t)root.number_or("num_key_value_heads", 0);
+  sh.vocab_size = (int64_t)root.number_or("vocab_size", 0);
+  sh.rms_norm_eps = root.number_or("rms_norm_eps", 1e-5);     // llama_tp.rs:68-70
+  sh.rope_theta = root.number_or("rope_theta", mixtral ? 1000000.0 : 10000.0);  // llama_tp.rs:71-73, mixtral.rs:56-58
+  if (mixtral) {  // mixtral.rs:40-57
+    sh.num_local_experts = (int64_t)root.number_or("num_local_experts", 0);
+    sh.num_experts_per_tok = (int64_t)root.number_or("num_experts_per_tok", 0);
+    sh.sliding_window = (int64_t)root.number_or("sliding_window", 4096);
+    if (sh.num_local_experts < 1 || sh.num_experts_per_tok < 1)
+      return fail(HB_ERR_INVALID_ARG, "mixtral config.json needs num_local_experts and num_experts_per_tok");
+  }
+  return setup_shape(e, sh);
+}
+
+static int llama_load(hb_engine* g, TensorSource& src) {
+  int rc = alloc_weights(g);
+  if (rc) return rc;
+  const hb_dtype dt = g->dtype;
+  const int r = g->rank;
+  if ((rc = src.fetch("model.embed_tokens.weight", g->V, g->H, 0, g->V, 0, g->H, g->embed, dt, 0))) return rc;
+  if ((rc = src.fetch("lm_head.weight", g->V, g->H, 0, g->V, 0, g->H, g->lm_head, dt, 0))) return rc;  // no tied-embedding fallback (llama_tp.rs:488)
+  if ((rc = src.fetch("model.norm.weight", 1, g->H, 0, 1, 0, g->H, g->final_norm, dt, 0))) return rc;
+  const size_t rowb = (size_t)g->H * g->es;
+  for (int64_t l = 0; l < g->L; ++l) {
+    const std::string pf = "model.layers." + std::to_string(l);
+    auto& w = g->layers[l];
+    const int64_t qr = g->hq_l * g->hd, kr = g->hkv_l * g->hd, qd = g->hq * g->hd;
+    uint8_t* qkv = (uint8_t*)w.wqkv;
+    if ((rc = src.fetch(pf + ".self_attn.q_proj.weight", qd, g->H, r * qr, qr, 0, g->H, qkv, dt, 0))) return rc;
+    if ((rc = src.fetch(pf + ".self_attn.k_proj.weight", g->hkv * g->hd, g->H, r * kr, kr, 0, g->H, qkv + (size_t)qr * rowb, dt, 0))) return rc;
+    if ((rc = src.fetch(pf + ".self_attn.v_proj.weight", g->hkv * g->hd, g->H, r * kr, kr, 0, g->H, qkv + (size_t)(qr + kr) * rowb, dt, 0))) return rc;
+    if ((rc = src.fetch(pf + ".self_attn.o_proj.weight", g->H, qd, 0, g->H, r * qr, qr, w.wo, dt, 0))) return rc;
+    if (!g->moe) {
+      if ((rc = src.fetch(pf + ".mlp.gate_proj.weight", g->I, g->H, r * g->I_l, g->I_l, 0, g->H, w.wgu, dt, 0))) return rc;
+      if ((rc = src.fetch(pf + ".mlp.up_proj.weight", g->I, g->H, r * g->I_l, g->I_l, 0, g->H, (uint8_t*)w.wgu + (size_t)g->I_l * rowb, dt, 0))) return rc;
+      if ((rc = src.fetch(pf + ".mlp.down_proj.weight", g->H, g->I, 0, g->H, r * g->I_l, g->I_l, w.wdown, dt, 0))) return rc;
+    } else {
+      // mixtral.rs:330-333,354-363: w1 (gate) and w3 (up) column-parallel, w2 (down)
+      // row-parallel over the expert's intermediate size; the router is replicated
+      if ((rc = src.fetch(pf + ".block_sparse_moe.gate.weight", g->E, g->H, 0, g->E, 0, g->H, w.wgate, dt, 0))) return rc;
+      for (int64_t x = 0; x < g->E; ++x) {
+        const std::string ex = pf + ".block_sparse_moe.experts." + std::to_string(x);
+        uint8_t* w1 = (uint8_t*)w.wgu + (size_t)(x * g->I_l) * rowb;
+        uint8_t* w3 = (uint8_t*)w.wgu + (size_t)(g->I_e + x * g->I_l) * rowb;
+        uint8_t* w2 = (uint8_t*)w.wdown + (size_t)(x * g->I_l) * g->es;
+        if ((rc = src.fetch(ex + ".w1.weight", g->I, g->H, r * g->I_l, g->I_l, 0, g->H, w1, dt, 0))) return rc;
+        if ((rc = src.fetch(ex + ".w3.weight", g->I, g->H, r * g->I_l, g->I_l, 0, g->H, w3, dt, 0))) return rc;
+        if ((rc = src.fetch(ex + ".w2.weight", g->H, g->I, 0, g->H, r * g->I_l, g->I_l, w2, dt, g->I_e))) return rc;
+      }
+    }
+    if ((rc = src.fetch(pf + ".input_layernorm.weight", 1, g->H, 0, 1, 0, g->H, w.norm_in, dt, 0))) return rc;
+    if ((rc = src.fetch(pf + ".post_attention_layernorm.weight", 1, g->H, 0, 1, 0, g->H, w.norm_post, dt, 0))) return rc;
+  }
+  return HB_OK;
+}
+
+const ModelFamily kLlamaFamily = {"llama", llama_serves, llama_configure, llama_load, alloc_runtime,
+                                  llama_prepare, llama_issue, llama_step_bytes, llama_gemm_bytes};
+
+// The registry: the first family that serves a config.json loads it.
+static const ModelFamily* const kFamilies[] = {&kLlamaFamily, &kLayeredFamily};
 
 }  // namespace hb
 
@@ -992,6 +1146,17 @@ int hb_engine_create_random(const hb_model_shape* shape, const hb_model_config* 
   return HB_OK;
 }
 
+// The family that serves the parsed config.json, its shapes and checks.
+static int configure_family(hb_engine* e, const hb::Json& root) {
+  for (const hb::ModelFamily* f : hb::kFamilies)
+    if (f->serves(root)) {
+      e->family = f;
+      return f->configure(e, root);
+    }
+  return hb::fail(HB_ERR_INVALID_ARG, "architecture '%s' is not served by this library",
+                  root.string_or("architecture", "").c_str());
+}
+
 int hb_engine_load(const hb_model_config* cfg, hb_world* world, hb_engine** out) {
   HB_CHECK_ARG(cfg && out && cfg->model_path, "hb_engine_load: null argument");
   std::unique_ptr<hb_engine, int (*)(hb_engine*)> e(new hb_engine, hb_engine_free);
@@ -1004,116 +1169,32 @@ int hb_engine_load(const hb_model_config* cfg, hb_world* world, hb_engine** out)
   std::string err;
   hb::JsonParser jp(text.data(), text.size());
   if (!jp.parse(&root, &err)) return hb::fail(HB_ERR_IO, "config.json: %s", err.c_str());
-  const std::string mt = root.string_or("model_type", "llama");
-  if (mt != "llama" && mt != "mistral" && mt != "mixtral")
-    return hb::fail(HB_ERR_INVALID_ARG, "model_type '%s' is not served by this path (llama, mistral, mixtral)",
-                    mt.c_str());
-  const bool mixtral = mt == "mixtral";
-  hb_model_shape sh;
-  memset(&sh, 0, sizeof(sh));
-  sh.hidden_size = (int64_t)root.number_or("hidden_size", 0);
-  sh.intermediate_size = (int64_t)root.number_or("intermediate_size", 0);
-  sh.num_hidden_layers = (int64_t)root.number_or("num_hidden_layers", 0);
-  sh.num_attention_heads = (int64_t)root.number_or("num_attention_heads", 0);
-  sh.num_key_value_heads = (int64_t)root.number_or("num_key_value_heads", 0);
-  sh.vocab_size = (int64_t)root.number_or("vocab_size", 0);
-  sh.rms_norm_eps = root.number_or("rms_norm_eps", 1e-5);     // llama_tp.rs:68-70
-  sh.rope_theta = root.number_or("rope_theta", mixtral ? 1000000.0 : 10000.0);  // llama_tp.rs:71-73, mixtral.rs:56-58
-  if (mixtral) {  // mixtral.rs:40-57
-    sh.num_local_experts = (int64_t)root.number_or("num_local_experts", 0);
-    sh.num_experts_per_tok = (int64_t)root.number_or("num_experts_per_tok", 0);
-    sh.sliding_window = (int64_t)root.number_or("sliding_window", 4096);
-    if (sh.num_local_experts < 1 || sh.num_experts_per_tok < 1)
-      return hb::fail(HB_ERR_INVALID_ARG, "mixtral config.json needs num_local_experts and num_experts_per_tok");
-  }
-  if ((rc = hb::setup_shape(e.get(), sh))) return rc;
-  if ((rc = hb::alloc_weights(e.get()))) return rc;
+  if ((rc = configure_family(e.get(), root))) return rc;
+  hb::CheckpointSource ckpt(e.get());
+  if ((rc = ckpt.open(dir))) return rc;
+  if ((rc = e->family->load(e.get(), ckpt))) return rc;
+  HB_CUDA_CHECK(cudaStreamSynchronize(e->stream));  // the mapped files are closed when this function returns
+  if ((rc = e->family->alloc_runtime(e.get(), cfg))) return rc;
+  HB_CUDA_CHECK(cudaStreamSynchronize(e->stream));
+  *out = e.release();
+  return HB_OK;
+}
 
-  std::vector<std::string> files;
-  if ((rc = hb::list_safetensors(dir, &files))) return rc;
-  std::vector<std::unique_ptr<hb::SafetensorsFile>> shards;
-  std::map<std::string, const hb::StTensor*> all;
-  for (auto& f : files) {
-    shards.emplace_back(new hb::SafetensorsFile);
-    if ((rc = shards.back()->open(f))) return rc;
-    for (auto& kv : shards.back()->tensors()) all[kv.first] = &kv.second;
-  }
-  hb_engine* g = e.get();
-  hb::UploadStage scratch;
-  auto get = [&](const std::string& name, int64_t rows, int64_t cols, const hb::StTensor** t) -> int {
-    auto it = all.find(name);
-    if (it == all.end()) return hb::fail(HB_ERR_IO, "Weight not found: %s", name.c_str());  // llama_tp.rs:380-385
-    const hb::StTensor* s = it->second;
-    if (s->dtype != "F32" && s->dtype != "F16" && s->dtype != "BF16")
-      return hb::fail(HB_ERR_UNSUPPORTED_DTYPE, "%s has dtype %s", name.c_str(), s->dtype.c_str());
-    // the shape itself, not only the element count: a transposed matrix must not be sharded
-    const bool shape_ok = rows == 1 ? ((s->shape.size() == 1 && s->shape[0] == cols) ||
-                                       (s->shape.size() == 2 && s->shape[0] == 1 && s->shape[1] == cols))
-                                    : (s->shape.size() == 2 && s->shape[0] == rows && s->shape[1] == cols);
-    if (!shape_ok)
-      return hb::fail(HB_ERR_IO, "%s has %lld elements in a shape other than the expected [%lld, %lld]", name.c_str(),
-                      (long long)s->numel(), (long long)rows, (long long)cols);
-    const size_t src_es = s->dtype == "F32" ? 4 : 2;
-    if (s->nbytes != (size_t)(rows * cols) * src_es)
-      return hb::fail(HB_ERR_IO, "%s holds %zu bytes, [%lld, %lld] of %s needs %zu", name.c_str(), s->nbytes,
-                      (long long)rows, (long long)cols, s->dtype.c_str(), (size_t)(rows * cols) * src_es);
-    *t = s;
-    return HB_OK;
-  };
-  const int r = g->rank;
-  const hb::StTensor* t = nullptr;
-  if ((rc = get("model.embed_tokens.weight", g->V, g->H, &t))) return rc;
-  if ((rc = hb::upload_slice(g, g->embed, *t, g->H, 0, g->V, 0, g->H, &scratch))) return rc;
-  if ((rc = get("lm_head.weight", g->V, g->H, &t))) return rc;  // no tied-embedding fallback (llama_tp.rs:488)
-  if ((rc = hb::upload_slice(g, g->lm_head, *t, g->H, 0, g->V, 0, g->H, &scratch))) return rc;
-  if ((rc = get("model.norm.weight", 1, g->H, &t))) return rc;
-  if ((rc = hb::upload_slice(g, g->final_norm, *t, g->H, 0, 1, 0, g->H, &scratch))) return rc;
-  const size_t rowb = (size_t)g->H * g->es;
-  for (int64_t l = 0; l < g->L; ++l) {
-    const std::string pf = "model.layers." + std::to_string(l);
-    auto& w = g->layers[l];
-    const int64_t qr = g->hq_l * g->hd, kr = g->hkv_l * g->hd, qd = g->hq * g->hd;
-    uint8_t* qkv = (uint8_t*)w.wqkv;
-    if ((rc = get(pf + ".self_attn.q_proj.weight", qd, g->H, &t))) return rc;
-    if ((rc = hb::upload_slice(g, qkv, *t, g->H, r * qr, qr, 0, g->H, &scratch))) return rc;
-    if ((rc = get(pf + ".self_attn.k_proj.weight", g->hkv * g->hd, g->H, &t))) return rc;
-    if ((rc = hb::upload_slice(g, qkv + (size_t)qr * rowb, *t, g->H, r * kr, kr, 0, g->H, &scratch))) return rc;
-    if ((rc = get(pf + ".self_attn.v_proj.weight", g->hkv * g->hd, g->H, &t))) return rc;
-    if ((rc = hb::upload_slice(g, qkv + (size_t)(qr + kr) * rowb, *t, g->H, r * kr, kr, 0, g->H, &scratch))) return rc;
-    if ((rc = get(pf + ".self_attn.o_proj.weight", g->H, qd, &t))) return rc;
-    if ((rc = hb::upload_slice(g, w.wo, *t, qd, 0, g->H, r * qr, qr, &scratch))) return rc;
-    if (!g->moe) {
-      if ((rc = get(pf + ".mlp.gate_proj.weight", g->I, g->H, &t))) return rc;
-      if ((rc = hb::upload_slice(g, w.wgu, *t, g->H, r * g->I_l, g->I_l, 0, g->H, &scratch))) return rc;
-      if ((rc = get(pf + ".mlp.up_proj.weight", g->I, g->H, &t))) return rc;
-      if ((rc = hb::upload_slice(g, (uint8_t*)w.wgu + (size_t)g->I_l * rowb, *t, g->H, r * g->I_l, g->I_l, 0, g->H, &scratch))) return rc;
-      if ((rc = get(pf + ".mlp.down_proj.weight", g->H, g->I, &t))) return rc;
-      if ((rc = hb::upload_slice(g, w.wdown, *t, g->I, 0, g->H, r * g->I_l, g->I_l, &scratch))) return rc;
-    } else {
-      // mixtral.rs:330-333,354-363: w1 (gate) and w3 (up) column-parallel, w2 (down)
-      // row-parallel over the expert's intermediate size; the router is replicated
-      if ((rc = get(pf + ".block_sparse_moe.gate.weight", g->E, g->H, &t))) return rc;
-      if ((rc = hb::upload_slice(g, w.wgate, *t, g->H, 0, g->E, 0, g->H, &scratch))) return rc;
-      for (int64_t x = 0; x < g->E; ++x) {
-        const std::string ex = pf + ".block_sparse_moe.experts." + std::to_string(x);
-        uint8_t* w1 = (uint8_t*)w.wgu + (size_t)(x * g->I_l) * rowb;
-        uint8_t* w3 = (uint8_t*)w.wgu + (size_t)(g->I_e + x * g->I_l) * rowb;
-        uint8_t* w2 = (uint8_t*)w.wdown + (size_t)(x * g->I_l) * g->es;
-        if ((rc = get(ex + ".w1.weight", g->I, g->H, &t))) return rc;
-        if ((rc = hb::upload_slice(g, w1, *t, g->H, r * g->I_l, g->I_l, 0, g->H, &scratch))) return rc;
-        if ((rc = get(ex + ".w3.weight", g->I, g->H, &t))) return rc;
-        if ((rc = hb::upload_slice(g, w3, *t, g->H, r * g->I_l, g->I_l, 0, g->H, &scratch))) return rc;
-        if ((rc = get(ex + ".w2.weight", g->H, g->I, &t))) return rc;
-        if ((rc = hb::upload_slice(g, w2, *t, g->I, 0, g->H, r * g->I_l, g->I_l, &scratch, g->I_e))) return rc;
-      }
-    }
-    if ((rc = get(pf + ".input_layernorm.weight", 1, g->H, &t))) return rc;
-    if ((rc = hb::upload_slice(g, w.norm_in, *t, g->H, 0, 1, 0, g->H, &scratch))) return rc;
-    if ((rc = get(pf + ".post_attention_layernorm.weight", 1, g->H, &t))) return rc;
-    if ((rc = hb::upload_slice(g, w.norm_post, *t, g->H, 0, 1, 0, g->H, &scratch))) return rc;
-  }
-  HB_CUDA_CHECK(cudaStreamSynchronize(g->stream));  // the mapped files are closed when this function returns
-  if ((rc = hb::alloc_runtime(g, cfg))) return rc;
+int hb_engine_create_random_config(const char* config_json, const hb_model_config* cfg, uint64_t seed, float std,
+                                   hb_engine** out) {
+  HB_CHECK_ARG(config_json && cfg && out, "hb_engine_create_random_config: null argument");
+  std::unique_ptr<hb_engine, int (*)(hb_engine*)> e(new hb_engine, hb_engine_free);
+  int rc;
+  if ((rc = hb::setup_common(e.get(), cfg, nullptr))) return rc;
+  hb::Json root;
+  std::string err;
+  hb::JsonParser jp(config_json, strlen(config_json));
+  if (!jp.parse(&root, &err)) return hb::fail(HB_ERR_IO, "config: %s", err.c_str());
+  if ((rc = configure_family(e.get(), root))) return rc;
+  hb::RandomSource src(e.get(), seed, std);
+  if ((rc = e->family->load(e.get(), src))) return rc;
+  if ((rc = e->family->alloc_runtime(e.get(), cfg))) return rc;
+  HB_CUDA_CHECK(cudaStreamSynchronize(e->stream));
   *out = e.release();
   return HB_OK;
 }
@@ -1123,6 +1204,7 @@ int64_t hb_engine_vocab_size(const hb_engine* e) { return e ? e->V : -1; }
 int64_t hb_engine_hidden_size(const hb_engine* e) { return e ? e->H : -1; }
 int64_t hb_engine_param_count(const hb_engine* e) {
   if (!e) return -1;
+  if (e->lm) return e->lm->params;
   // Engine::param_count (src/engine/loader.rs:323-329)
   const int64_t attn = 4 * e->H * e->H, ffn = 3 * e->H * e->I;
   return e->V * e->H + e->L * (attn + ffn) + e->V * e->H;
@@ -1133,18 +1215,7 @@ float hb_engine_last_step_ms(hb_engine* e) { return e ? e->last_ms : -1.f; }
 int64_t hb_engine_last_step_launches(const hb_engine* e) { return e ? e->last_launches : -1; }
 
 double hb_engine_step_bytes(const hb_engine* e, const int32_t* ctx_lens, int64_t n_seqs) {
-  if (!e) return -1.0;
-  const double es = (double)e->es;
-  double w = 0.0;
-  w += (double)e->L * ((double)e->qkv_rows * e->H + (double)e->H * e->hq_l * e->hd +
-                       3.0 * (double)e->I_e * e->H + (e->moe ? (double)e->E * e->H : 0.0) + 2.0 * e->H) * es;
-  w += ((double)e->V * e->H + e->H) * es;    // lm_head + final norm
-  w += (double)n_seqs * e->H * es;            // embedding rows
-  double kv = 0.0;
-  for (int64_t i = 0; i < n_seqs; ++i)
-    kv += (double)(ctx_lens ? ctx_lens[i] : 0) * e->L * 2.0 * e->hkv_l * e->hd * es;  // read
-  kv += (double)n_seqs * e->L * 2.0 * e->hkv_l * e->hd * es;                           // write
-  return w + kv;
+  return e ? e->family->step_bytes(e, ctx_lens, n_seqs) : -1.0;
 }
 
 int64_t hb_engine_get_tensor(hb_engine* e, const char* name, float* out, int64_t cap) {
@@ -1157,7 +1228,8 @@ int64_t hb_engine_get_tensor(hb_engine* e, const char* name, float* out, int64_t
   cudaSetDevice(e->device);
   float* tmp = nullptr;
   if (cudaMalloc((void**)&tmp, (size_t)n * 4) != cudaSuccess) return hb::fail(HB_ERR_CUDA, "cudaMalloc failed");
-  int rc = hb::to_f32(e->stream, tmp, it->second.ptr, e->dtype, n, it->second.cols, it->second.ld);
+  const hb_dtype dt = it->second.dtype >= 0 ? (hb_dtype)it->second.dtype : e->dtype;
+  int rc = hb::to_f32(e->stream, tmp, it->second.ptr, dt, n, it->second.cols, it->second.ld);
   if (!rc && cudaMemcpyAsync(out, tmp, (size_t)n * 4, cudaMemcpyDeviceToHost, e->stream) != cudaSuccess) rc = HB_ERR_CUDA;
   cudaStreamSynchronize(e->stream);
   cudaFree(tmp);
@@ -1176,6 +1248,7 @@ int hb_seq_free(hb_engine* e, hb_seq* s) {
   if (!s) return HB_OK;
   HB_CHECK_ARG(e, "hb_seq_free: null engine");
   for (int64_t b : s->blocks) e->free_blocks.push_back(b);
+  if (s->state_slot >= 0) e->free_slots.push_back(s->state_slot);
   delete s;
   return HB_OK;
 }
@@ -1185,6 +1258,10 @@ int64_t hb_seq_len(const hb_seq* s) { return s ? s->len : -1; }
 int hb_seq_truncate(hb_engine* e, hb_seq* s, int64_t new_len) {
   HB_CHECK_ARG(e && s, "hb_seq_truncate: null argument");
   HB_CHECK_ARG(new_len >= 0 && new_len <= s->len, "hb_seq_truncate: length %lld outside [0, %lld]", (long long)new_len,
+               (long long)s->len);
+  // a recurrent state cannot be wound back; forgetting everything is always possible
+  HB_CHECK_ARG(e->num_state_slots == 0 || new_len == 0 || new_len == s->len,
+               "hb_seq_truncate: the model's recurrent state cannot be cut to %lld of %lld tokens", (long long)new_len,
                (long long)s->len);
   s->len = new_len;
   // blocks that hold no token any more go back to the free list (FIFO, as freed blocks do)
@@ -1224,7 +1301,7 @@ int hb_decode_batch(hb_engine* e, hb_seq* const* seqs, size_t B, const uint32_t*
 int hb_kv_copy_blocks(hb_engine* e, const int64_t* pairs, size_t n_pairs) {
   HB_CHECK_ARG(e && (pairs || n_pairs == 0), "hb_kv_copy_blocks: null argument");
   HB_CUDA_CHECK(cudaSetDevice(e->device));
-  const int64_t block_bytes = e->hkv_l * HB_BLOCK_SIZE * e->hd * (int64_t)e->es;
+  HB_CHECK_ARG(e->num_state_slots == 0, "hb_kv_copy_blocks: this model keeps recurrent state besides its blocks");
   for (size_t i = 0; i < 2 * n_pairs; ++i)
     if (pairs[i] < 0 || pairs[i] >= e->num_blocks)
       return hb::fail(HB_ERR_INVALID_ARG, "hb_kv_copy_blocks: block id %lld outside the pool of %lld",
@@ -1232,8 +1309,9 @@ int hb_kv_copy_blocks(hb_engine* e, const int64_t* pairs, size_t n_pairs) {
   for (size_t done = 0; done < n_pairs; done += hb::kPairCap) {
     const size_t n = std::min<size_t>(hb::kPairCap, n_pairs - done);
     HB_CUDA_CHECK(cudaMemcpyAsync(e->d_pairs, pairs + 2 * done, n * 2 * sizeof(int64_t), cudaMemcpyHostToDevice, e->stream));
-    for (int64_t l = 0; l < e->L; ++l) {
-      int rc = hb::kv_copy_blocks(e->stream, e->kc[l], e->vc[l], e->d_pairs, (int64_t)n, block_bytes, e->num_blocks);
+    for (size_t l = 0; l < e->kc.size(); ++l) {
+      int rc = hb::kv_copy_blocks(e->stream, e->kc[l], e->vc[l], e->d_pairs, (int64_t)n, (int64_t)e->k_block_bytes[l],
+                                  e->num_blocks);
       if (rc) return rc;
     }
     HB_CUDA_CHECK(cudaStreamSynchronize(e->stream));  // `pairs` and d_pairs may be reused
@@ -1246,8 +1324,10 @@ int hb_engine_reserve_cpu_blocks(hb_engine* e, int64_t n_blocks) {
   HB_CUDA_CHECK(cudaSetDevice(e->device));
   if (e->h_swap) { cudaFreeHost(e->h_swap); e->h_swap = nullptr; e->cpu_blocks = 0; }
   if (n_blocks == 0) return HB_OK;
-  const size_t block_bytes = (size_t)e->hkv_l * HB_BLOCK_SIZE * e->hd * e->es;
-  HB_CUDA_CHECK(cudaMallocHost((void**)&e->h_swap, (size_t)n_blocks * e->L * 2 * block_bytes));
+  HB_CHECK_ARG(e->num_state_slots == 0, "hb_engine_reserve_cpu_blocks: this model keeps recurrent state besides its blocks");
+  size_t per_block = 0;
+  for (size_t l = 0; l < e->kc.size(); ++l) per_block += e->k_block_bytes[l] + e->v_block_bytes[l];
+  HB_CUDA_CHECK(cudaMallocHost((void**)&e->h_swap, (size_t)n_blocks * per_block));
   e->cpu_blocks = n_blocks;
   return HB_OK;
 }
@@ -1255,7 +1335,6 @@ int hb_engine_reserve_cpu_blocks(hb_engine* e, int64_t n_blocks) {
 int hb_kv_swap_blocks(hb_engine* e, const int64_t* pairs, size_t n_pairs, int to_cpu) {
   HB_CHECK_ARG(e && (pairs || n_pairs == 0), "hb_kv_swap_blocks: null argument");
   HB_CUDA_CHECK(cudaSetDevice(e->device));
-  const size_t block_bytes = (size_t)e->hkv_l * HB_BLOCK_SIZE * e->hd * e->es;
   for (size_t i = 0; i < n_pairs; ++i) {
     // swap_out pairs are (gpu, cpu), swap_in pairs (cpu, gpu): block_manager.rs:359-406
     const int64_t g = to_cpu ? pairs[2 * i] : pairs[2 * i + 1], c = to_cpu ? pairs[2 * i + 1] : pairs[2 * i];
@@ -1265,12 +1344,16 @@ int hb_kv_swap_blocks(hb_engine* e, const int64_t* pairs, size_t n_pairs, int to
   }
   for (size_t i = 0; i < n_pairs; ++i) {
     const int64_t g = to_cpu ? pairs[2 * i] : pairs[2 * i + 1], c = to_cpu ? pairs[2 * i + 1] : pairs[2 * i];
-    for (int64_t l = 0; l < e->L; ++l)
+    size_t per_block = 0;
+    for (size_t l = 0; l < e->kc.size(); ++l) per_block += e->k_block_bytes[l] + e->v_block_bytes[l];
+    uint8_t* host = e->h_swap + (size_t)c * per_block;
+    for (size_t l = 0; l < e->kc.size(); ++l)
       for (int kv = 0; kv < 2; ++kv) {
+        const size_t block_bytes = kv ? e->v_block_bytes[l] : e->k_block_bytes[l];
         uint8_t* dev = (uint8_t*)(kv ? e->vc[l] : e->kc[l]) + (size_t)g * block_bytes;
-        uint8_t* host = e->h_swap + (((size_t)c * e->L + l) * 2 + kv) * block_bytes;
         if (to_cpu) HB_CUDA_CHECK(cudaMemcpyAsync(host, dev, block_bytes, cudaMemcpyDeviceToHost, e->stream));
         else HB_CUDA_CHECK(cudaMemcpyAsync(dev, host, block_bytes, cudaMemcpyHostToDevice, e->stream));
+        host += block_bytes;
       }
   }
   HB_CUDA_CHECK(cudaStreamSynchronize(e->stream));
@@ -1286,23 +1369,27 @@ int hb_decode_batch_tables(hb_engine* e, size_t B, const uint32_t* last_tokens, 
   int rc;
   // blocks_to_copy first: a sequence that shared its last block writes into its own copy
   if (n_copies && (rc = hb_kv_copy_blocks(e, copy_pairs, n_copies))) return rc;
-  std::vector<hb::StepRow> rows(B);
+  hb::StepBatch batch;
   for (size_t b = 0; b < B; ++b) {
     if (positions[b] < 0) return hb::fail(HB_ERR_INVALID_ARG, "row %zu: negative position", b);
     const size_t covered = std::min<size_t>(table_stride, (size_t)(positions[b] / HB_BLOCK_SIZE + 1));
-    rows[b] = {block_tables + b * table_stride, covered, positions[b], last_tokens[b]};
+    batch.add(block_tables + b * table_stride, covered, positions[b], last_tokens + b, 1);
+    batch.want.push_back((int32_t)b);
   }
   // two rows of one decode step are two sequences: they never write the same KV slot
+  auto slot_of = [](const hb::StepSeg& g, int64_t* slot) {
+    if (g.n_blocks * HB_BLOCK_SIZE <= (size_t)g.pos0) return false;  // reported by run_step
+    *slot = g.blocks[g.pos0 / HB_BLOCK_SIZE] * HB_BLOCK_SIZE + g.pos0 % HB_BLOCK_SIZE;
+    return true;
+  };
   for (size_t b = 0; b < B; ++b) {
-    if (rows[b].n_blocks * HB_BLOCK_SIZE <= (size_t)rows[b].pos) continue;  // reported by run_rows
-    const int64_t slot = rows[b].blocks[rows[b].pos / HB_BLOCK_SIZE] * HB_BLOCK_SIZE + rows[b].pos % HB_BLOCK_SIZE;
-    for (size_t j = 0; j < b; ++j) {
-      if (rows[j].n_blocks * HB_BLOCK_SIZE <= (size_t)rows[j].pos) continue;
-      if (rows[j].blocks[rows[j].pos / HB_BLOCK_SIZE] * HB_BLOCK_SIZE + rows[j].pos % HB_BLOCK_SIZE == slot)
+    int64_t slot = 0, other = 0;
+    if (!slot_of(batch.segs[b], &slot)) continue;
+    for (size_t j = 0; j < b; ++j)
+      if (slot_of(batch.segs[j], &other) && other == slot)
         return hb::fail(HB_ERR_INVALID_ARG, "rows %zu and %zu write the same KV slot %lld", j, b, (long long)slot);
-    }
   }
-  return hb::run_rows(e, rows.data(), (int)B, next_tokens, logits_opt, 0);
+  return hb::run_step(e, batch, next_tokens, logits_opt);
 }
 
 int hb_forward_tables(hb_engine* e, const uint32_t* ids, size_t n, size_t seq_pos, const int64_t* block_table,
@@ -1311,19 +1398,58 @@ int hb_forward_tables(hb_engine* e, const uint32_t* ids, size_t n, size_t seq_po
   HB_CHECK_ARG(e && ids && block_table && logits_out, "hb_forward_tables: null argument");
   // chunks of consecutive positions, as hb_forward; positions below seq_pos must already hold
   // this sequence's K/V in the table's blocks (a prefix-cache hit: block_manager.rs:213-234)
-  std::vector<hb::StepRow> rows;
   size_t done = 0;
   while (done < n) {
     const int c = (int)std::min<size_t>(n - done, (size_t)e->max_batch);
-    rows.resize((size_t)c);
-    for (int i = 0; i < c; ++i) rows[i] = {block_table, table_len, (int64_t)(seq_pos + done) + i, ids[done + i]};
-    const bool last = done + (size_t)c == n;
-    int rc = hb::run_rows(e, rows.data(), c, nullptr, last ? logits_out : nullptr, c - 1, true);
+    hb::StepBatch batch;
+    batch.add(block_table, table_len, (int64_t)(seq_pos + done), ids + done, c);
+    if (done + (size_t)c == n) batch.want.push_back(c - 1);
+    int rc = hb::run_step(e, batch, nullptr, logits_out);
     if (rc) return rc;
     done += (size_t)c;
   }
   return HB_OK;
 }
+
+int hb_step(hb_engine* e, const hb_step_entry* entries, size_t n, uint32_t* next_tokens, float* logits_out) {
+  HB_CHECK_ARG(e && (entries || n == 0), "hb_step: null argument");
+  return hb::mixed_step(e, entries, n, next_tokens, logits_out);
+}
+
+int hb_engine_sample(hb_engine* e, size_t n, const uint64_t* seeds, float temperature, float top_p, uint32_t* tokens) {
+  HB_CHECK_ARG(e && seeds && tokens, "hb_engine_sample: null argument");
+  HB_CHECK_ARG(n > 0 && n <= e->last_rows.size(), "hb_engine_sample: %zu rows asked for, the last step left %zu", n,
+               e->last_rows.size());
+  HB_CUDA_CHECK(cudaSetDevice(e->device));
+  if ((int)n > e->sample_rows) {
+    const int rows = std::min(e->max_logits_rows, std::max((int)n, 2 * e->sample_rows));
+    int rc;
+    if ((rc = hb::dev_alloc(e, (void**)&e->d_probs, (size_t)rows * e->V * 4))) return rc;
+    if ((rc = hb::dev_alloc(e, (void**)&e->d_picked, (size_t)rows * e->V * 4))) return rc;
+    if ((rc = hb::dev_alloc(e, (void**)&e->d_seeds, (size_t)rows * 8))) return rc;
+    if ((rc = hb::dev_alloc(e, (void**)&e->d_sampled, (size_t)rows * 4))) return rc;
+    e->sample_rows = rows;
+  }
+  HB_CUDA_CHECK(cudaMemcpyAsync(e->d_seeds, seeds, n * 8, cudaMemcpyHostToDevice, e->stream));
+  // wanted rows that lie apart (Llama family: one logits row per batch row) are gathered first
+  const float* logits = e->d_logits;
+  bool in_place = true;
+  for (size_t i = 0; i < n && in_place; ++i) in_place = e->last_rows[i] == (int)i;
+  if (!in_place) {
+    for (size_t i = 0; i < n; ++i)
+      HB_CUDA_CHECK(cudaMemcpyAsync(e->d_picked + i * e->V, e->d_logits + (size_t)e->last_rows[i] * e->V, (size_t)e->V * 4,
+                                    cudaMemcpyDeviceToDevice, e->stream));
+    logits = e->d_picked;
+  }
+  int rc = hb_sample(e->stream, e->d_sampled, e->d_probs, logits, nullptr, e->d_seeds, (int64_t)n, e->V, temperature,
+                     top_p, 0.f, 0.f);
+  if (rc) return rc;
+  HB_CUDA_CHECK(cudaMemcpyAsync(tokens, e->d_sampled, n * 4, cudaMemcpyDeviceToHost, e->stream));
+  HB_CUDA_CHECK(cudaStreamSynchronize(e->stream));
+  return HB_OK;
+}
+
+int hb_engine_num_free_state_slots(const hb_engine* e) { return e ? (int)e->free_slots.size() : -1; }
 
 int hb_engine_profile_step(hb_engine* e, hb_seq* const* seqs, size_t B, const uint32_t* last_tokens,
                            uint32_t* next_tokens, float* ms_by_kind) {
@@ -1336,17 +1462,7 @@ int hb_engine_profile_step(hb_engine* e, hb_seq* const* seqs, size_t B, const ui
   return HB_OK;
 }
 
-double hb_engine_gemm_bytes(const hb_engine* e, int64_t B) {
-  if (!e) return -1.0;
-  const double es = (double)e->es, b = (double)B;
-  const double qkv = (double)e->qkv_rows, o_in = (double)e->hq_l * e->hd, H = (double)e->H,
-               Il = (double)e->I_e, V = (double)e->V;
-  double per_layer = (qkv * H + b * H + b * qkv) * es        // q|k|v projection
-                     + (H * o_in + b * o_in + b * H) * es    // o_proj
-                     + (2 * Il * H + b * H + b * Il) * es    // gate|up with the SwiGLU epilogue
-                     + (H * Il + b * Il + b * H) * es;       // down_proj
-  return (double)e->L * per_layer + (V * H + b * H) * es + b * V * 4.0;  // + lm_head, fp32 logits
-}
+double hb_engine_gemm_bytes(const hb_engine* e, int64_t B) { return e ? e->family->gemm_bytes(e, B) : -1.0; }
 
 int hb_forward(hb_engine* e, hb_seq* s, const uint32_t* ids, size_t n, size_t seq_pos,
                float* logits_out) {

@@ -1,4 +1,4 @@
-// hb_gemm: the public GEMM entry point.  bf16 problems with K % 64 == 0 go to the
+// hb_gemm: the public GEMM entry point.  bf16 problems with K % 8 == 0 go to the
 // tcgen05 kernel, everything else to the CUDA-core kernel.
 #include "common.h"
 #include "gemm.h"
@@ -53,7 +53,7 @@ int hb_gemm_ex(void* stream, void* Y, const void* X, const void* W, int64_t M, i
   HB_CHECK_ARG(Y && X && W, "hb_gemm_ex: null pointer");
   HB_CHECK_ARG(epilogue == hb::kEpiStore || epilogue == hb::kEpiSwiGLU, "hb_gemm_ex: unknown epilogue %d", epilogue);
   HB_CHECK_ARG(hb::gemm_tc_supported(M, N, K, HB_BF16),
-               "hb_gemm_ex: bf16 with K %% 64 == 0 only (M=%lld N=%lld K=%lld)", (long long)M,
+               "hb_gemm_ex: bf16 with K %% 8 == 0 only (M=%lld N=%lld K=%lld)", (long long)M,
                (long long)N, (long long)K);
   int dev = 0;
   HB_CUDA_CHECK(cudaGetDevice(&dev));

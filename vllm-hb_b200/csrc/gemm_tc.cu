@@ -840,7 +840,9 @@ static int encode_out_map(CUtensorMap* tm, void* ptr, int64_t rows, int64_t cols
 }
 
 bool gemm_tc_supported(int64_t M, int64_t N, int64_t K, hb_dtype dtype) {
-  return dtype == HB_BF16 && M >= 1 && N >= 1 && K >= kTileK && K % kTileK == 0 &&
+  // K need not fill its last 64-wide chunk: the tensor maps deliver zeros past the end of a row
+  // (rows must be 16-byte multiples)
+  return dtype == HB_BF16 && M >= 1 && N >= 1 && K >= 8 && K % 8 == 0 &&
          N < (1ll << 30) && M < (1ll << 30);
 }
 
@@ -894,7 +896,7 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
   const int64_t m_eff = std::min<int64_t>(M, m_cap);
   pl.m_pad = (int)std::max<int64_t>(16, (m_eff + 15) / 16 * 16);
   pl.n_tiles = (int)((n_rows + kTileN - 1) / kTileN);
-  const int k_chunks = (int)(K / kTileK);
+  const int k_chunks = (int)((K + kTileK - 1) / kTileK);
   const bool want_cluster = true;  // split-K partners reduce on chip; global scratch only where a cluster cannot form
   const bool tuned = want_cluster && force_splits <= 0;
   // Few weights under a wide batch (o_proj and q|k|v at high tensor-parallel degrees): the
@@ -1063,7 +1065,7 @@ int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, voi
 #endif
   p.M = (int)pl.M; p.N = (int)pl.N;
   p.m_pad = pl.m_pad; p.splits = pl.splits; p.stages = pl.stages; p.tmem_cols = pl.tmem_cols;
-  p.k_chunks = (int)(pl.K / kTileK);
+  p.k_chunks = (int)((pl.K + kTileK - 1) / kTileK);
   p.n_tiles = pl.n_tiles;
   p.epilogue = pl.epilogue; p.out_f32 = pl.out_f32 ? 1 : 0;
   p.ldy = ldy;

@@ -1,0 +1,535 @@
+// The layered family: weights, pools and the step of models described by a LayeredSpec.
+#include <algorithm>
+#include <cstring>
+
+#include "engine.h"
+#include "layered_ops.h"
+
+namespace hb {
+
+LayeredModel::~LayeredModel() {
+  for (auto& kv : graphs)
+    if (kv.second.exec) cudaGraphExecDestroy(kv.second.exec);
+}
+
+static int64_t pad8(int64_t n) { return (n + 7) / 8 * 8; }
+static int64_t pad_to(int64_t n, int64_t m) { return (n + m - 1) / m * m; }
+
+// ------------------------------------------------------------------------------- load
+static bool layered_serves(const Json& config) { return is_latarax(config); }
+
+static int layered_configure(hb_engine* e, const Json& config) {
+  if (e->ws > 1) return fail(HB_ERR_INVALID_ARG, "this design runs on one rank");
+  if (e->dtype == HB_F16) return fail(HB_ERR_UNSUPPORTED_DTYPE, "this design runs in bf16 or f32, not f16");
+  e->lm.reset(new LayeredModel);
+  int rc = read_latarax(config, &e->lm->spec);
+  if (rc) return rc;
+  const LayeredSpec& s = e->lm->spec;
+  if (s.streams < 1 || s.streams > kMaxStreams)
+    return fail(HB_ERR_INVALID_ARG, "%d residual streams (1 to %d)", s.streams, kMaxStreams);
+  e->H = s.width; e->V = s.vocab; e->L = (int64_t)s.layers.size();
+  e->eps = s.eps;
+  e->max_positions = s.max_positions;
+  e->use_tc = e->dtype == HB_BF16;
+  const char* g = getenv("HB_GEMM");
+  if (g && std::string(g) == "simt") e->use_tc = false;
+  return HB_OK;
+}
+
+namespace {
+struct Loader {
+  hb_engine* e;
+  LayeredModel* m;
+  TensorSource& src;
+
+  // [rows, cols] rows of `name` at row r0 of a matrix, columns zero-padded to its K
+  int part(const LayeredLinear& lin, const std::string& name, int64_t r0, int64_t rows, int64_t cols) {
+    uint8_t* dst = (uint8_t*)lin.w + (size_t)r0 * lin.K * e->es;
+    int rc = src.fetch_all(name, rows, cols, dst, e->dtype, lin.K);
+    e->named[name] = {dst, rows, cols, lin.K};
+    m->params += rows * cols;
+    return rc;
+  }
+  int alloc(LayeredLinear* lin, int64_t n, int64_t k) {
+    lin->N = n;
+    lin->K = pad8(k);
+    return dev_alloc(e, &lin->w, (size_t)n * lin->K * e->es, true);
+  }
+  int linear(LayeredLinear* lin, const std::string& name, int64_t n, int64_t k) {
+    int rc = alloc(lin, pad8(n), k);
+    return rc ? rc : part(*lin, name, 0, n, k);
+  }
+  // fp32 vector or small matrix; generated weights take `neutral` (mix: the identity)
+  int small(float** dst, const std::string& name, int64_t rows, int64_t cols, float neutral, bool identity = false) {
+    int rc = dev_alloc(e, (void**)dst, (size_t)rows * cols * 4);
+    if (rc) return rc;
+    e->named[name] = {*dst, rows, cols, 0, HB_F32};
+    m->params += rows * cols;
+    if (!src.generated()) return src.fetch_all(name, rows, cols, *dst, HB_F32);
+    return identity ? constant(*dst, rows, cols) : fill_const(e->stream, *dst, HB_F32, rows * cols, neutral);
+  }
+  int constant(float* dst, int64_t rows, int64_t cols) {
+    std::vector<float> v((size_t)(rows * cols), 0.f);
+    for (int64_t i = 0; i < std::min(rows, cols); ++i) v[(size_t)(i * cols + i)] = 1.f;
+    return upload(dst, v);
+  }
+  int upload(float* dst, const std::vector<float>& v) {
+    HB_CUDA_CHECK(cudaMemcpyAsync(dst, v.data(), v.size() * 4, cudaMemcpyHostToDevice, e->stream));
+    HB_CUDA_CHECK(cudaStreamSynchronize(e->stream));
+    return HB_OK;
+  }
+  int sublayer(SublayerMix* q, const std::string& in, const std::string& out, const std::string& mix,
+               const std::string& norm) {
+    const int S = m->spec.streams;
+    int rc;
+    if (in.empty()) {  // one plain stream: x += y
+      const std::vector<float> one(1, 1.f);
+      for (float** p : {&q->in, &q->out, &q->mix}) {
+        if ((rc = dev_alloc(e, (void**)p, 4))) return rc;
+        if ((rc = upload(*p, one))) return rc;
+      }
+    } else {
+      if ((rc = small(&q->in, in, 1, S, 1.f / S))) return rc;
+      if ((rc = small(&q->out, out, 1, S, 1.f))) return rc;
+      if ((rc = small(&q->mix, mix, S, S, 0.f, true))) return rc;
+    }
+    return small(&q->norm, norm, 1, m->spec.width, 0.f);
+  }
+};
+}  // namespace
+
+static int layered_load(hb_engine* e, TensorSource& src) {
+  LayeredModel* m = e->lm.get();
+  LayeredSpec& s = m->spec;
+  Loader ld{e, m, src};
+  const int64_t W = s.width;
+  int rc;
+  m->Hp = pad8(W);
+  if ((rc = dev_alloc(e, &m->embed, (size_t)s.vocab * W * e->es))) return rc;
+  if ((rc = src.fetch_all(s.embed, s.vocab, W, m->embed, e->dtype))) return rc;
+  e->named[s.embed] = {m->embed, s.vocab, W};
+  if ((rc = dev_alloc(e, &m->pos, (size_t)s.max_positions * W * e->es))) return rc;
+  if ((rc = src.fetch_all(s.pos, s.max_positions, W, m->pos, e->dtype))) return rc;
+  e->named[s.pos] = {m->pos, s.max_positions, W};
+  m->params += (s.vocab + s.max_positions) * W;
+  if ((rc = ld.alloc(&m->head, s.vocab, W))) return rc;
+  if ((rc = ld.part(m->head, s.head, 0, s.vocab, W))) return rc;
+  if ((rc = ld.small(&m->final_norm, s.final_norm, 1, W, 0.f))) return rc;
+  m->layers.resize(s.layers.size());
+  for (size_t i = 0; i < s.layers.size(); ++i) {
+    LayerSpec& sp = s.layers[i];
+    LayeredLayer& l = m->layers[i];
+    MixerSpec& mx = sp.mixer;
+    if (mx.has_rec && mx.rec.low_rank_decay) {
+      const std::vector<int64_t> shape = src.shape(mx.ra1.tensor);
+      if (!src.generated() && shape.size() != 2) return fail(HB_ERR_IO, "Weight not found: %s", mx.ra1.tensor.c_str());
+      mx.rec.rank = src.generated() ? 16 : (int)shape[0];  // the low rank is the tensor's own
+      mx.ra1.rows = mx.rec.rank;
+      if (mx.rec.rank < 1) return fail(HB_ERR_IO, "%s is empty", mx.ra1.tensor.c_str());
+    }
+    int64_t n = 0;
+    const ProjPart* parts[] = {&mx.aq, &mx.ak, &mx.av, &mx.rq, &mx.rk, &mx.rv, &mx.rg, &mx.ra1};
+    for (const ProjPart* p : parts)
+      if (p->rows) n = std::max(n, p->offset + p->rows);
+    if ((rc = ld.alloc(&l.proj, pad8(n), W))) return rc;
+    for (const ProjPart* p : parts)
+      if (p->rows && (rc = ld.part(l.proj, p->tensor, p->offset, p->rows, W))) return rc;
+    if (mx.has_attn) {
+      if ((rc = ld.linear(&l.attn_o, mx.attn_o, W, (int64_t)mx.attn.heads * mx.attn.vdim))) return rc;
+    }
+    if (mx.has_rec) {
+      const RecurrenceSpec& r = mx.rec;
+      const int64_t hd = (int64_t)r.heads * r.dim, hv = (int64_t)r.heads * r.vdim;
+      if ((rc = ld.linear(&l.rec_o, mx.rec_o, W, hv))) return rc;
+      if ((rc = ld.small(&l.rec_norm, mx.rec_norm, 1, r.norm_per_head ? r.vdim : hv, 1.f))) return rc;
+      if (r.low_rank_decay) {
+        if ((rc = dev_alloc(e, (void**)&l.a2, (size_t)hd * r.rank * 4))) return rc;
+        if ((rc = src.fetch_all(mx.rec_a2, hd, r.rank, l.a2, HB_F32))) return rc;
+        e->named[mx.rec_a2] = {l.a2, hd, r.rank, 0, HB_F32};
+        m->params += hd * r.rank;
+        if ((rc = ld.small(&l.a2_bias, mx.rec_a2_bias, 1, hd, 1.f))) return rc;
+      } else {
+        if ((rc = dev_alloc(e, (void**)&l.decay, (size_t)r.heads * 4))) return rc;
+        if ((rc = ld.upload(l.decay, std::vector<float>(r.decay.begin(), r.decay.end())))) return rc;
+      }
+    }
+    if (mx.has_attn && mx.has_rec) {
+      if ((rc = ld.small(&l.attn_out_norm, mx.attn_out_norm, 1, W, 1.f))) return rc;
+      if ((rc = ld.small(&l.rec_out_norm, mx.rec_out_norm, 1, W, 1.f))) return rc;
+    }
+    if ((rc = ld.sublayer(&l.sub1, sp.hc1_in, sp.hc1_out, sp.hc1_mix, sp.norm1))) return rc;
+    if (sp.ff) {
+      l.ffp = pad8(sp.ff);
+      if ((rc = ld.alloc(&l.gate_up, 2 * l.ffp, W))) return rc;
+      if ((rc = ld.part(l.gate_up, sp.gate, 0, sp.ff, W))) return rc;
+      if ((rc = ld.part(l.gate_up, sp.up, l.ffp, sp.ff, W))) return rc;
+      if ((rc = ld.linear(&l.down, sp.down, W, sp.ff))) return rc;
+      if ((rc = ld.sublayer(&l.sub2, sp.hc2_in, sp.hc2_out, sp.hc2_mix, sp.norm2))) return rc;
+    }
+  }
+  return HB_OK;
+}
+
+// --------------------------------------------------------------------------- runtime
+struct InputLayout {
+  size_t bytes = 0;
+  size_t take(size_t n) {
+    const size_t at = bytes;
+    bytes = (bytes + n + 15) / 16 * 16;
+    return at;
+  }
+};
+
+static size_t layered_layout(const hb_engine* e, LayeredStep* s) {
+  InputLayout l;
+  s->off_ids = l.take((size_t)s->rows * 4);
+  s->off_pos = l.take((size_t)s->rows * 4);
+  s->off_slots = l.take((size_t)s->rows * 8);
+  s->off_row_seg = l.take((size_t)s->rows * 4);
+  s->off_want = l.take((size_t)s->want * 4);
+  s->off_seg = l.take((size_t)s->segs * sizeof(SegInfo));
+  s->off_short = l.take((size_t)s->n_short * 4);
+  s->off_long = l.take((size_t)s->n_long * 4);
+  s->off_chunk = l.take((size_t)s->n_chunks * sizeof(RowRange));
+  s->off_tile = l.take((size_t)s->n_tiles * sizeof(RowRange));
+  s->off_attn_rows = l.take((size_t)s->n_attn_rows * 4);
+  s->off_tables = l.take((size_t)s->segs * e->max_blocks_per_seq * 4);
+  return l.bytes;
+}
+
+static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
+  LayeredModel* m = e->lm.get();
+  const LayeredSpec& s = m->spec;
+  const size_t es = e->es;
+  int rc;
+  e->max_batch = cfg->max_batch > 0 ? cfg->max_batch : 256;
+  int64_t max_seq = cfg->max_seq_len > 0 ? (int64_t)cfg->max_seq_len : 2048;
+  max_seq = std::min(max_seq, s.max_positions);
+  e->max_blocks_per_seq = (max_seq + HB_BLOCK_SIZE - 1) / HB_BLOCK_SIZE;
+  m->max_segs = std::min(e->max_batch, cfg->max_seqs > 0 ? cfg->max_seqs : e->max_batch);
+  e->num_blocks = cfg->num_kv_blocks > 0 ? cfg->num_kv_blocks : e->max_blocks_per_seq * m->max_segs;
+  for (int64_t b = 0; b < e->num_blocks; ++b) e->free_blocks.push_back(b);
+  const int64_t R = pad_to(e->max_batch, 128);
+  m->row_cap = R;
+  int64_t max_attn = 0, max_rec = 0, max_o = 0, max_ffp = 0;
+  for (size_t i = 0; i < s.layers.size(); ++i) {
+    LayeredLayer& l = m->layers[i];
+    const MixerSpec& mx = s.layers[i].mixer;
+    m->max_proj = std::max(m->max_proj, l.proj.N);
+    max_ffp = std::max(max_ffp, l.ffp);
+    if (mx.has_attn) {
+      const AttentionSpec& a = mx.attn;
+      l.kv_pool = (int)e->kc.size();
+      const size_t kb = (size_t)a.kv_heads * HB_BLOCK_SIZE * a.dim * es, vb = (size_t)a.kv_heads * HB_BLOCK_SIZE * a.vdim * es;
+      void *k = nullptr, *v = nullptr;
+      // unwritten slots may be fetched (and masked): keep them finite
+      if ((rc = dev_alloc(e, &k, kb * e->num_blocks, true))) return rc;
+      if ((rc = dev_alloc(e, &v, vb * e->num_blocks, true))) return rc;
+      e->kc.push_back(k);
+      e->vc.push_back(v);
+      e->k_block_bytes.push_back(kb);
+      e->v_block_bytes.push_back(vb);
+      max_attn = std::max(max_attn, l.attn_o.K);
+    }
+    if (mx.has_rec) {
+      const RecurrenceSpec& r = mx.rec;
+      e->num_state_slots = m->max_segs;
+      if ((rc = dev_alloc(e, (void**)&l.state, (size_t)m->max_segs * r.heads * r.dim * r.vdim * 4, true))) return rc;
+      max_rec = std::max(max_rec, l.rec_o.K);
+      max_o = std::max(max_o, (int64_t)r.heads * r.vdim);
+    }
+  }
+  for (int i = 0; i < e->num_state_slots; ++i) e->free_slots.push_back(i);
+  e->max_logits_rows = (int)std::min<int64_t>(e->max_batch, std::max<int64_t>(64, (1ll << 28) / s.vocab));
+  const int64_t LR = pad_to(e->max_logits_rows, 16);
+  if ((rc = dev_alloc(e, (void**)&m->x, (size_t)R * s.streams * s.width * 4, true))) return rc;
+  if ((rc = dev_alloc(e, &m->h, (size_t)R * m->Hp * es, true))) return rc;
+  if ((rc = dev_alloc(e, &m->proj, (size_t)R * m->max_proj * es, true))) return rc;
+  if ((rc = dev_alloc(e, &m->attn, (size_t)R * max_attn * es, true))) return rc;
+  if ((rc = dev_alloc(e, &m->rec, (size_t)R * max_rec * es, true))) return rc;
+  if ((rc = dev_alloc(e, (void**)&m->o, (size_t)R * max_o * 4, true))) return rc;
+  if ((rc = dev_alloc(e, (void**)&m->y1, (size_t)R * m->Hp * 4, true))) return rc;
+  if ((rc = dev_alloc(e, (void**)&m->y2, (size_t)R * m->Hp * 4, true))) return rc;
+  if (!e->use_tc && (rc = dev_alloc(e, &m->gu, (size_t)R * 2 * max_ffp * es, true))) return rc;
+  if ((rc = dev_alloc(e, &m->act, (size_t)R * max_ffp * es, true))) return rc;
+  if ((rc = dev_alloc(e, &m->hf, (size_t)LR * m->Hp * es, true))) return rc;
+  if ((rc = dev_alloc(e, (void**)&e->d_logits, (size_t)LR * s.vocab * 4))) return rc;
+  if ((rc = dev_alloc(e, (void**)&e->d_next, (size_t)LR * 4, true))) return rc;
+  HB_CUDA_CHECK(cudaMallocHost((void**)&e->h_next, (size_t)LR * 4));
+  if ((rc = dev_alloc(e, (void**)&e->d_err, 16, true))) return rc;
+  // the largest step: every list at its longest
+  LayeredStep cap;
+  cap.rows = e->max_batch;
+  cap.want = e->max_batch;
+  cap.segs = cap.n_short = cap.n_long = m->max_segs;
+  cap.n_chunks = cap.n_tiles = e->max_batch + m->max_segs;
+  cap.n_attn_rows = e->max_batch;
+  e->inputs_bytes = layered_layout(e, &cap);
+  if ((rc = dev_alloc(e, (void**)&e->d_inputs, e->inputs_bytes, true))) return rc;
+  HB_CUDA_CHECK(cudaMallocHost((void**)&e->h_inputs, e->inputs_bytes));
+  return HB_OK;
+}
+
+// ------------------------------------------------------------------------------- step
+// Matrix products are planned for a bucket of rows, so that steps of similar size share plans;
+// the rows above the step's own are scratch.
+static int row_bucket(int rows) { return (int)(rows <= 256 ? pad_to(rows, 16) : pad_to(rows, 128)); }
+
+static int layered_plans(hb_engine* e, int rows, LayeredPlans** out) {
+  LayeredModel* m = e->lm.get();
+  const int M = row_bucket(rows);
+  auto it = m->plans.find(M);
+  if (it != m->plans.end()) { *out = &it->second; return HB_OK; }
+  LayeredPlans p;
+  const size_t L = m->layers.size();
+  p.proj.resize(L); p.attn_o.resize(L); p.rec_o.resize(L); p.gate_up.resize(L); p.down.resize(L);
+  size_t ws = 0;
+  int rc;
+  auto plan = [&](TcGemmPlan* pl, const void* X, const LayeredLinear& w, int epi, bool f32) -> int {
+    if (!w.w) return HB_OK;
+    const int r = gemm_tc_plan(pl, X, w.w, M, w.N, w.K, epi, f32, e->device);
+    if (!r) ws = std::max(ws, pl->workspace_bytes());
+    return r;
+  };
+  for (size_t i = 0; i < L; ++i) {
+    LayeredLayer& l = m->layers[i];
+    if ((rc = plan(&p.proj[i], m->h, l.proj, kEpiStore, false))) return rc;
+    if ((rc = plan(&p.attn_o[i], m->attn, l.attn_o, kEpiStore, true))) return rc;
+    if ((rc = plan(&p.rec_o[i], m->rec, l.rec_o, kEpiStore, true))) return rc;
+    if ((rc = plan(&p.gate_up[i], m->h, l.gate_up, kEpiSwiGLU, false))) return rc;
+    if ((rc = plan(&p.down[i], m->act, l.down, kEpiStore, true))) return rc;
+  }
+  if ((rc = ensure_gemm_workspace(e, ws))) return rc;
+  *out = &m->plans.emplace(M, std::move(p)).first->second;
+  return HB_OK;
+}
+
+static int layered_head_plan(hb_engine* e, int want, TcGemmPlan** out) {
+  LayeredModel* m = e->lm.get();
+  const int M = (int)std::min<int64_t>(row_bucket(want), pad_to(e->max_logits_rows, 16));
+  auto it = m->head_plans.find(M);
+  if (it != m->head_plans.end()) { *out = &it->second; return HB_OK; }
+  TcGemmPlan p;
+  int rc = gemm_tc_plan(&p, m->hf, m->head.w, M, m->head.N, m->head.K, kEpiStore, true, e->device);
+  if (rc) return rc;
+  if ((rc = ensure_gemm_workspace(e, p.workspace_bytes()))) return rc;
+  *out = &m->head_plans.emplace(M, p).first->second;
+  return HB_OK;
+}
+
+static int layered_prepare(hb_engine* e, const StepBatch& batch, StepExec* x) {
+  LayeredModel* m = e->lm.get();
+  if ((int)batch.segs.size() > m->max_segs)
+    return fail(HB_ERR_INVALID_ARG, "%zu sequences in one step, %d at most", batch.segs.size(), m->max_segs);
+  LayeredStep& s = x->layered;
+  s.rows = batch.rows;
+  s.segs = (int)batch.segs.size();
+  s.want = (int)batch.want.size();
+  s.decode = s.rows == s.segs;
+  s.n_short = s.segs;
+  s.n_attn_rows = s.rows;
+  x->rows = batch.rows;
+  x->logits_compact = true;
+  x->input_bytes = layered_layout(e, &s);
+  if (x->input_bytes > e->inputs_bytes) return fail(HB_ERR_INVALID_ARG, "step inputs of %zu bytes", x->input_bytes);
+  uint8_t* in = e->h_inputs;
+  uint32_t* ids = (uint32_t*)(in + s.off_ids);
+  int32_t* pos = (int32_t*)(in + s.off_pos);
+  int64_t* slots = (int64_t*)(in + s.off_slots);
+  int32_t* row_seg = (int32_t*)(in + s.off_row_seg);
+  SegInfo* seg = (SegInfo*)(in + s.off_seg);
+  int32_t* shorts = (int32_t*)(in + s.off_short);
+  int32_t* attn_rows = (int32_t*)(in + s.off_attn_rows);
+  int32_t* tables = (int32_t*)(in + s.off_tables);
+  for (int g = 0; g < s.segs; ++g) {
+    const StepSeg& t = batch.segs[g];
+    seg[g] = {t.row0, t.n, (int32_t)t.pos0, t.state_slot};
+    shorts[g] = g;
+    for (int i = 0; i < t.n; ++i) {
+      const int64_t p = t.pos0 + i;
+      ids[t.row0 + i] = t.tokens[i];
+      pos[t.row0 + i] = (int32_t)p;
+      slots[t.row0 + i] = t.blocks[p / HB_BLOCK_SIZE] * HB_BLOCK_SIZE + p % HB_BLOCK_SIZE;
+      row_seg[t.row0 + i] = g;
+      attn_rows[t.row0 + i] = t.row0 + i;
+    }
+    const int64_t need = (t.pos0 + t.n - 1) / HB_BLOCK_SIZE + 1;
+    int32_t* row = tables + (size_t)g * e->max_blocks_per_seq;
+    for (int64_t k = 0; k < need; ++k) row[k] = (int32_t)t.blocks[k];
+  }
+  std::copy(batch.want.begin(), batch.want.end(), (int32_t*)(in + s.off_want));
+  if (e->use_tc) {
+    int rc;
+    if ((rc = layered_plans(e, s.rows, &s.plans))) return rc;
+    if (s.want && (rc = layered_head_plan(e, s.want, &s.head_plan))) return rc;
+  }
+  // a step of decoded tokens whose logits are all wanted replays from a graph
+  if (s.decode && s.want == s.rows) {
+    LayeredGraph& g = m->graphs[s.rows];
+    x->graph = &g.exec;
+    x->graph_launches = &g.launches;
+  }
+  return HB_OK;
+}
+
+static int layered_issue(hb_engine* e, const StepExec& x) {
+  LayeredModel* m = e->lm.get();
+  const LayeredSpec& sp = m->spec;
+  const LayeredStep& s = x.layered;
+  cudaStream_t st = e->stream;
+  const uint8_t* in = e->d_inputs;
+  const uint32_t* ids = (const uint32_t*)(in + s.off_ids);
+  const int32_t* pos = (const int32_t*)(in + s.off_pos);
+  const int64_t* slots = (const int64_t*)(in + s.off_slots);
+  const int32_t* row_seg = (const int32_t*)(in + s.off_row_seg);
+  const SegInfo* seg = (const SegInfo*)(in + s.off_seg);
+  const int S = sp.streams;
+  const int64_t W = sp.width, rows = s.rows;
+  const size_t es = e->es;
+  int rc;
+  auto gemm = [&](const std::vector<TcGemmPlan>* plans, size_t i, void* Y, const void* X, const LayeredLinear& w,
+                  bool f32) -> int {
+    ++e->last_launches;
+    if (e->use_tc) return gemm_tc_run((*plans)[i], st, Y, (*plans)[i].N, e->d_gemm_ws, e->d_err);
+    return gemm_simt(st, Y, X, w.w, rows, w.N, w.K, e->dtype, f32);
+  };
+  const LayeredPlans* pl = s.plans;
+  auto at = [&](void* p, int64_t elements) { return (void*)((uint8_t*)p + (size_t)elements * es); };
+
+  prof_mark(e, kCatOther);
+  if ((rc = streams_embed(st, m->x, m->h, m->embed, m->pos, ids, pos, m->layers[0].sub1.in, m->layers[0].sub1.norm, rows, S, W,
+                          m->Hp, sp.vocab, sp.max_positions, sp.eps, e->dtype))) return rc;
+  ++e->last_launches;
+  for (size_t i = 0; i < m->layers.size(); ++i) {
+    LayeredLayer& l = m->layers[i];
+    const LayerSpec& lsp = sp.layers[i];
+    const MixerSpec& mx = lsp.mixer;
+    prof_mark(e, kCatGemm);
+    if ((rc = gemm(pl ? &pl->proj : nullptr, i, m->proj, m->h, l.proj, false))) return rc;
+    const int64_t ldp = l.proj.N;
+    float* y = m->y1;
+    if (mx.has_attn) {
+      const AttentionSpec& as = mx.attn;
+      SpanAttention a;
+      a.q = at(m->proj, mx.aq.offset); a.ld_q = ldp;
+      a.out = m->attn; a.ld_out = l.attn_o.K;
+      a.kc = e->kc[l.kv_pool]; a.vc = e->vc[l.kv_pool];
+      a.tables = (const int32_t*)(in + s.off_tables);
+      a.max_blocks = e->max_blocks_per_seq; a.num_blocks = e->num_blocks;
+      a.row_seg = row_seg; a.pos = pos;
+      a.heads = as.heads; a.kv_heads = as.kv_heads; a.dim = as.dim; a.vdim = as.vdim;
+      a.window = as.window; a.keep_first = as.keep_first; a.scale = as.scale;
+      prof_mark(e, kCatRopeKv);
+      if ((rc = span_kv_write(st, a, at(m->proj, mx.ak.offset), at(m->proj, mx.av.offset), ldp, slots, rows, e->dtype))) return rc;
+      prof_mark(e, kCatAttention);
+      if ((rc = span_attention_rows(st, a, (const int32_t*)(in + s.off_attn_rows), s.n_attn_rows, e->dtype))) return rc;
+      prof_mark(e, kCatGemmO);
+      if ((rc = gemm(pl ? &pl->attn_o : nullptr, i, y, m->attn, l.attn_o, true))) return rc;
+      e->last_launches += 2;
+      y = m->y2;
+    }
+    if (mx.has_rec) {
+      const RecurrenceSpec& rs = mx.rec;
+      Recurrence r;
+      r.p = m->proj; r.ld = ldp;
+      r.off_q = (int)mx.rq.offset; r.off_k = (int)mx.rk.offset; r.off_v = (int)mx.rv.offset; r.off_a1 = (int)mx.ra1.offset;
+      r.heads = rs.heads; r.dim = rs.dim; r.vdim = rs.vdim;
+      r.q_scale = rs.q_scale; r.silu_qkv = rs.silu_qkv ? 1 : 0;
+      r.decay = l.decay; r.a2 = l.a2; r.a2_bias = l.a2_bias; r.rank = rs.rank; r.inv_tau = (float)(1.0 / rs.tau);
+      r.state = l.state; r.o = m->o; r.ld_o = (int64_t)rs.heads * rs.vdim; r.segs = seg;
+      prof_mark(e, kCatRecurrence);
+      if ((rc = recurrence_tokens(st, r, (const int32_t*)(in + s.off_short), s.n_short, e->dtype))) return rc;
+      prof_mark(e, kCatNorm);
+      const int groups = rs.norm_per_head ? rs.heads : 1, size = rs.norm_per_head ? rs.vdim : rs.heads * rs.vdim;
+      if ((rc = gated_group_norm(st, m->rec, l.rec_o.K, m->o, r.ld_o, at(m->proj, mx.rg.offset), ldp, l.rec_norm, rows, groups,
+                                 size, rs.gate_silu, sp.eps, e->dtype))) return rc;
+      prof_mark(e, kCatGemmO);
+      if ((rc = gemm(pl ? &pl->rec_o : nullptr, i, y, m->rec, l.rec_o, true))) return rc;
+      e->last_launches += 2;
+    }
+    const bool both = mx.has_attn && mx.has_rec;
+    const SublayerMix* next = lsp.ff ? &l.sub2 : (i + 1 < m->layers.size() ? &m->layers[i + 1].sub1 : nullptr);
+    auto boundary = [&](const SublayerMix& q, bool two) -> int {
+      StreamMix sm;
+      sm.mix = q.mix; sm.out = q.out;
+      sm.next_in = next ? next->in : nullptr;
+      sm.next_norm = next ? next->norm : nullptr;
+      sm.w1 = l.attn_out_norm; sm.w2 = l.rec_out_norm;
+      ++e->last_launches;
+      prof_mark(e, kCatNorm);
+      return streams_mix(st, m->x, m->h, m->y1, two ? m->y2 : nullptr, m->Hp, sm, rows, S, W, m->Hp, sp.eps, e->dtype);
+    };
+    if ((rc = boundary(l.sub1, both))) return rc;
+    if (lsp.ff) {
+      prof_mark(e, kCatGemmGateUp);
+      if (e->use_tc) {
+        if ((rc = gemm(&pl->gate_up, i, m->act, m->h, l.gate_up, false))) return rc;
+      } else {
+        if ((rc = gemm(nullptr, i, m->gu, m->h, l.gate_up, false))) return rc;
+        if ((rc = hb_silu_mul(st, m->act, m->gu, rows, l.ffp, e->dtype))) return rc;
+        ++e->last_launches;
+      }
+      prof_mark(e, kCatGemmDown);
+      if ((rc = gemm(pl ? &pl->down : nullptr, i, m->y1, m->act, l.down, true))) return rc;
+      next = i + 1 < m->layers.size() ? &m->layers[i + 1].sub1 : nullptr;
+      if ((rc = boundary(l.sub2, false))) return rc;
+    }
+  }
+  if (s.want) {
+    prof_mark(e, kCatNorm);
+    if ((rc = streams_final(st, m->hf, m->x, (const int32_t*)(in + s.off_want), m->final_norm, s.want, S, W, m->Hp, sp.eps,
+                            e->dtype))) return rc;
+    prof_mark(e, kCatGemmLmHead);
+    if (e->use_tc) rc = gemm_tc_run(*s.head_plan, st, e->d_logits, sp.vocab, e->d_gemm_ws, e->d_err);
+    else rc = gemm_simt(st, e->d_logits, m->hf, m->head.w, s.want, m->head.N, m->head.K, e->dtype, true);
+    if (rc) return rc;
+    prof_mark(e, kCatOther);
+    if ((rc = hb_argmax(st, e->d_next, e->d_logits, s.want, sp.vocab, HB_F32))) return rc;
+    e->last_launches += 3;
+  }
+  prof_mark(e, -1);
+  return HB_OK;
+}
+
+// Bytes one decode step moves: weights once, K/V and recurrent states of the sequences, streams.
+static double layered_step_bytes(const hb_engine* e, const int32_t* ctx_lens, int64_t n_seqs) {
+  const LayeredModel* m = e->lm.get();
+  const LayeredSpec& s = m->spec;
+  const double es = (double)e->es, n = (double)n_seqs;
+  double w = (double)m->head.N * m->head.K * es + 2.0 * n * s.width * es;
+  for (size_t i = 0; i < s.layers.size(); ++i) {
+    const LayeredLayer& l = m->layers[i];
+    for (const LayeredLinear* q : {&l.proj, &l.attn_o, &l.rec_o, &l.gate_up, &l.down}) w += (double)q->N * q->K * es;
+    const MixerSpec& mx = s.layers[i].mixer;
+    if (mx.has_attn) {
+      const AttentionSpec& a = mx.attn;
+      for (int64_t k = 0; k < n_seqs; ++k) {
+        const int64_t ctx = ctx_lens ? ctx_lens[k] : 0;
+        int64_t seen = ctx;
+        if (a.window > 0) seen = std::min<int64_t>(ctx, (int64_t)a.window + std::min<int64_t>(a.keep_first, std::max<int64_t>(0, ctx - a.window)));
+        w += ((double)seen + 1.0) * a.kv_heads * (a.dim + a.vdim) * es;
+      }
+    }
+    if (mx.has_rec) w += n * 2.0 * mx.rec.heads * mx.rec.dim * mx.rec.vdim * 4.0;
+    w += n * (s.layers[i].ff ? 2.0 : 1.0) * 2.0 * s.streams * s.width * 4.0;
+  }
+  return w;
+}
+
+static double layered_gemm_bytes(const hb_engine* e, int64_t rows) {
+  const LayeredModel* m = e->lm.get();
+  const double es = (double)e->es, b = (double)rows;
+  auto lin = [&](const LayeredLinear& q, double n_out, double out_es) {
+    return q.w ? ((double)q.N * q.K + b * q.K) * es + b * n_out * out_es : 0.0;
+  };
+  double t = lin(m->head, (double)m->head.N, 4.0);
+  for (const LayeredLayer& l : m->layers)
+    t += lin(l.proj, (double)l.proj.N, es) + lin(l.attn_o, (double)l.attn_o.N, 4.0) + lin(l.rec_o, (double)l.rec_o.N, 4.0) +
+         lin(l.gate_up, (double)l.ffp, es) + lin(l.down, (double)l.down.N, 4.0);
+  return t;
+}
+
+const ModelFamily kLayeredFamily = {"layered", layered_serves, layered_configure, layered_load, layered_alloc_runtime,
+                                    layered_prepare, layered_issue, layered_step_bytes, layered_gemm_bytes};
+
+}  // namespace hb

@@ -1,0 +1,166 @@
+// Models described layer by layer: every layer has a mixer (attention, a gated linear
+// recurrence, or both side by side) and possibly a gated feed-forward, over one or several
+// residual streams held in fp32.  The mechanisms and their constants are data (LayeredSpec); a
+// design's reader (latarax.cc) turns its config.json and tensor names into it.
+#pragma once
+
+#include <cstdint>
+#include <map>
+#include <memory>
+#include <string>
+#include <vector>
+
+#include "common.h"
+#include "gemm.h"
+
+namespace hb {
+
+struct Json;
+
+// Softmax attention over a paged K/V cache: per-head sizes of keys and values may differ;
+// position i sees j <= i with i - j < window (0 = all) or j < keep_first.
+struct AttentionSpec {
+  int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
+  float scale = 1.f;
+  int window = 0, keep_first = 0;
+};
+
+// S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per head, fp32 state of [dim, vdim].
+struct RecurrenceSpec {
+  int heads = 0, dim = 0, vdim = 0;
+  float q_scale = 1.f;
+  bool silu_qkv = false;            // q, k and v pass through SiLU
+  // decay: a constant per head, or sigmoid(W2 (W1 h) + bias)^(1/tau) per key channel
+  bool low_rank_decay = false;
+  std::vector<double> decay;        // [heads]
+  double tau = 1.0;
+  int rank = 0;
+  // the outputs are RMS-normed per head (weight [vdim]) or all heads together (weight
+  // [heads * vdim]) and multiplied by a gate
+  bool norm_per_head = false;
+  bool gate_silu = false;           // gate activation: SiLU, else sigmoid
+};
+
+// Rows of the layer's input projection that come from one checkpoint tensor.
+struct ProjPart {
+  std::string tensor;
+  int64_t rows = 0;
+  int64_t offset = 0;  // first column of the projection's output (a multiple of 8)
+};
+
+struct MixerSpec {
+  bool has_attn = false, has_rec = false;
+  AttentionSpec attn;
+  RecurrenceSpec rec;
+  // tensors: projections that read h, concatenated into one matrix
+  ProjPart aq, ak, av;                       // attention
+  ProjPart rq, rk, rv, rg, ra1;              // recurrence (ra1: low-rank decay)
+  std::string attn_o, rec_o, rec_norm, rec_a2, rec_a2_bias;
+  std::string attn_out_norm, rec_out_norm;   // both branches: each normed, then averaged
+};
+
+struct LayerSpec {
+  std::string prefix;                        // tensor name prefix, "l0."
+  MixerSpec mixer;
+  std::string norm1, norm2;
+  std::string hc1_in, hc1_out, hc1_mix, hc2_in, hc2_out, hc2_mix;  // empty: one plain residual stream
+  int64_t ff = 0;                            // 0: no feed-forward
+  std::string gate, up, down;
+};
+
+struct LayeredSpec {
+  std::string design;
+  int64_t width = 0, vocab = 0, max_positions = 0;
+  int streams = 1;
+  float eps = 1e-6f;
+  std::string embed, pos, final_norm, head;
+  std::vector<LayerSpec> layers;
+};
+
+// Design readers: config.json (and, for sizes it does not give, tensor shapes) -> spec.
+bool is_latarax(const Json& config);
+int read_latarax(const Json& config, LayeredSpec* out);
+
+// ---------------------------------------------------------------------------- weights
+struct LayeredLinear {
+  void* w = nullptr;        // [N, K] engine dtype; N, K are padded to multiples of 8 with zeros
+  int64_t N = 0, K = 0;
+};
+
+struct SublayerMix {        // how a sublayer's output goes back into the streams (fp32, device)
+  float* in = nullptr;      // [streams]
+  float* out = nullptr;     // [streams]
+  float* mix = nullptr;     // [streams from, streams to]
+  float* norm = nullptr;    // [width], stored around zero
+};
+
+struct LayeredLayer {
+  LayeredLinear proj;                        // all projections of h
+  LayeredLinear attn_o, rec_o, gate_up, down;
+  int64_t ffp = 0;                           // padded feed-forward width
+  float *decay = nullptr;                    // [heads] (constant decay)
+  float *a2 = nullptr, *a2_bias = nullptr;   // [heads * dim, rank], [heads * dim]
+  float *rec_norm = nullptr, *attn_out_norm = nullptr, *rec_out_norm = nullptr;
+  int kv_pool = -1;                          // index into hb_engine::kc / vc
+  float* state = nullptr;                    // [slots, heads, dim, vdim]
+  SublayerMix sub1, sub2;
+};
+
+// Plans of all matrix products for one bucket of batch rows.
+struct LayeredPlans {
+  std::vector<TcGemmPlan> proj, attn_o, rec_o, gate_up, down;
+};
+
+struct LayeredGraph {
+  cudaGraphExec_t exec = nullptr;
+  int64_t launches = 0;
+};
+
+// Where a step's inputs lie in the (pinned and device) input block, and what it contains.
+struct LayeredStep {
+  int rows = 0, segs = 0, want = 0;
+  int n_short = 0;        // segments the token-by-token recurrence kernel takes
+  int n_chunks = 0;       // chunks of the longer segments (chunked recurrence kernels)
+  int n_long = 0;         // longer segments
+  int n_tiles = 0;        // query tiles of the tiled attention kernel
+  int n_attn_rows = 0;    // rows the per-token attention kernel takes
+  bool decode = false;    // every segment is one token
+  size_t off_ids = 0, off_pos = 0, off_slots = 0, off_row_seg = 0, off_want = 0, off_seg = 0, off_short = 0,
+         off_long = 0, off_chunk = 0, off_tile = 0, off_attn_rows = 0, off_tables = 0;
+  LayeredPlans* plans = nullptr;
+  TcGemmPlan* head_plan = nullptr;
+};
+
+struct LayeredModel {
+  LayeredSpec spec;
+  std::vector<LayeredLayer> layers;
+  void *embed = nullptr, *pos = nullptr;     // [vocab, width], [max_positions, width] engine dtype, dense rows
+  LayeredLinear head;                        // [vocab (padded), width (padded)]
+  float* final_norm = nullptr;
+  float* ones = nullptr;                     // [streams] of 1
+  int64_t Hp = 0;                            // width padded to a multiple of 8
+  int64_t params = 0;                        // elements of all tensors
+  int64_t row_cap = 0;                       // rows of the step buffers
+  // buffers
+  int64_t max_proj = 0;                      // widest projection row
+  float* x = nullptr;                        // [rows, streams, width]
+  void* h = nullptr;                         // [rows, Hp]
+  void* proj = nullptr;                      // [rows, max_proj]
+  void *attn = nullptr, *rec = nullptr;      // branch outputs before their output projection
+  float* o = nullptr;                        // [rows, heads * vdim] recurrence outputs
+  float *y1 = nullptr, *y2 = nullptr;        // [rows, Hp] sublayer outputs
+  void *gu = nullptr, *act = nullptr;        // feed-forward
+  void* hf = nullptr;                        // [logits rows, Hp] final normed rows
+  float* cum = nullptr;                      // [rows, heads * dim] cumulative log decay inside a chunk
+  float* chunk_state = nullptr;              // [chunks, heads, dim, vdim]
+  float* chunk_decay = nullptr;              // [chunks, heads * dim] log decay over a whole chunk
+  float* attn_part = nullptr;                // split partials of the per-token attention
+  int max_segs = 0, max_chunks = 0, attn_splits_cap = 1;
+  size_t inputs_cap = 0;
+  std::map<int, LayeredPlans> plans;         // by rows bucket
+  std::map<int, TcGemmPlan> head_plans;      // by wanted-rows bucket
+  std::map<int, LayeredGraph> graphs;        // by number of decoded sequences
+  ~LayeredModel();
+};
+
+}  // namespace hb

@@ -1,0 +1,92 @@
+// Launchers of the kernels the layered family is made of.  Every constant of a mechanism is a
+// parameter; rows of a step belong to segments (StepSeg) and carry their position and KV slot.
+#pragma once
+
+#include "common.h"
+
+namespace hb {
+
+// One segment of a step on the device: rows [row0, row0 + n), positions pos0 .., state slot.
+struct SegInfo {
+  int32_t row0, n, pos0, slot;
+};
+// A chunk of a longer segment (chunked recurrence) or a tile of query positions (tiled
+// attention): `n` consecutive rows from `row0`, part of segment `seg`; `index` counts the chunks of
+// the segment from 0.
+struct RowRange {
+  int32_t seg, row0, n, index;
+};
+
+// ------------------------------------------------------------------ residual streams (streams.cu)
+constexpr int kMaxStreams = 16;
+// x[r, s, :] = embed[ids[r]] + pos_table[pos[r]] for every stream s (fp32), then
+// h[r] = rms(sum_s in[s] x[r, s]) * (1 + norm).
+int streams_embed(cudaStream_t st, float* x, void* h, const void* embed, const void* pos_table, const uint32_t* ids,
+                  const int32_t* pos, const float* in, const float* norm, int64_t rows, int streams, int64_t width,
+                  int64_t ld_h, int64_t vocab, int64_t max_positions, float eps, hb_dtype dtype);
+// One sublayer boundary: y (fp32 rows of stride ld_y) goes back into the streams,
+//   x[r, t] = sum_s mix[s, t] x[r, s] + out[t] y[r],
+// and the next sublayer's input is read: h[r] = rms(sum_t next_in[t] x[r, t]) * (1 + next_norm)
+// (next_norm null: no further sublayer).  With y2, y is the mean of two branch outputs, each
+// RMS-normed over the width with its plain weight: (rms(y) w1 + rms(y2) w2) / 2.
+struct StreamMix {
+  const float *mix, *out, *next_in, *next_norm;
+  const float *w1 = nullptr, *w2 = nullptr;
+};
+int streams_mix(cudaStream_t st, float* x, void* h, const float* y, const float* y2, int64_t ld_y, const StreamMix& m,
+                int64_t rows, int streams, int64_t width, int64_t ld_h, float eps, hb_dtype dtype);
+// h[i] = rms(sum_s x[want[i], s]) * (1 + norm)
+int streams_final(cudaStream_t st, void* h, const float* x, const int32_t* want, const float* norm, int64_t n_want,
+                  int streams, int64_t width, int64_t ld_h, float eps, hb_dtype dtype);
+// out[r, g * size + i] = rms over the group of o[r, g, :] * weight * act(gate[r, g * size + i]);
+// weight [size] is shared by the groups; act = SiLU or sigmoid.
+int gated_group_norm(cudaStream_t st, void* out, int64_t ld_out, const float* o, int64_t ld_o, const void* gate,
+                     int64_t ld_gate, const float* weight, int64_t rows, int groups, int size, bool gate_silu, float eps,
+                     hb_dtype dtype);
+
+// --------------------------------------------------------------- attention (attention_span.cu)
+// Paged attention whose queries see the last `window` positions (0 = all) and the first
+// `keep_first`; keys and values of different widths.  Pools per layer:
+// K [num_blocks, kv_heads, 16, dim], V [num_blocks, kv_heads, 16, vdim].
+struct SpanAttention {
+  const void* q = nullptr;     // row r, head h at q + r * ld_q + h * dim
+  int64_t ld_q = 0;
+  void* out = nullptr;         // row r, head h at out + r * ld_out + h * vdim
+  int64_t ld_out = 0;
+  void *kc = nullptr, *vc = nullptr;
+  const int32_t* tables = nullptr;   // [segs, max_blocks]
+  int64_t max_blocks = 0, num_blocks = 0;
+  const int32_t* row_seg = nullptr;  // segment of a row
+  const int32_t* pos = nullptr;      // position of a row
+  int heads = 0, kv_heads = 0, dim = 0, vdim = 0, window = 0, keep_first = 0;
+  float scale = 1.f;
+};
+// K/V of the step's rows to their slots (slot = block * 16 + offset; negative: skipped).
+int span_kv_write(cudaStream_t st, const SpanAttention& a, const void* k, const void* v, int64_t ld_kv, const int64_t* slots,
+                  int64_t rows, hb_dtype dtype);
+// One CTA per (row of `row_list`, kv head): any dtype and any sizes.
+int span_attention_rows(cudaStream_t st, const SpanAttention& a, const int32_t* row_list, int n_rows, hb_dtype dtype);
+
+// ------------------------------------------------------------ linear recurrence (recurrence.cu)
+struct Recurrence {
+  const void* p = nullptr;     // projection rows: q, k, v (and the low-rank decay input) at offsets
+  int64_t ld = 0;
+  int off_q = 0, off_k = 0, off_v = 0, off_a1 = 0;
+  int heads = 0, dim = 0, vdim = 0;
+  float q_scale = 1.f;
+  int silu_qkv = 0;
+  const float* decay = nullptr;      // [heads] constant decay, or null:
+  const float* a2 = nullptr;         // [heads * dim, rank] low-rank decay
+  const float* a2_bias = nullptr;    // [heads * dim]
+  int rank = 0;
+  float inv_tau = 1.f;
+  float* state = nullptr;            // [slots, heads, dim, vdim]
+  float* o = nullptr;                // [rows, heads * vdim]
+  int64_t ld_o = 0;
+  const SegInfo* segs = nullptr;
+};
+// Token by token, state in and out of HBM once per segment where it fits the registers:
+// decoded tokens and short portions.  `list` holds segment numbers.
+int recurrence_tokens(cudaStream_t st, const Recurrence& a, const int32_t* list, int n_list, hb_dtype dtype);
+
+}  // namespace hb
