@@ -226,6 +226,86 @@ int hb_sample(void* stream, uint32_t* tokens, float* probs_workspace, const floa
               const uint32_t* token_counts, const uint64_t* seeds, int64_t n, int64_t vocab, float temperature,
               float top_p, float presence_penalty, float frequency_penalty);
 
+/* ---------------------------------------------- mechanisms of the layered models
+ * Kernels of the models described layer by layer (hb_engine_load of config.json files that name an
+ * "architecture"); bf16 or f32.  Rows of a batch belong to segments: runs of consecutive tokens of
+ * one sequence.  Ranges are int32 quadruples in device memory. */
+
+/* Paged attention whose queries at position p see the keys j <= p with p - j < window
+ * (window 0: all) or j < keep_first; keys and values may differ in width.
+ * q row r, head h at q + r*ld_q + h*dim; out likewise with vdim; K pool [num_blocks, kv_heads, 16,
+ * dim], V pool [num_blocks, kv_heads, 16, vdim]; softmax(scale * q.k) v, scores and weights in fp32.
+ * tiles {segment, first row, rows, -}: up to hb_span_attention_tile_positions() consecutive
+ * positions each (0: these sizes are not taken, give rows); rows: single rows.  n_splits > 1 cuts
+ * the keys of a row over several CTAs; workspace: n_rows*heads*n_splits*(vdim+2) floats. */
+typedef struct hb_span_attention_args {
+  const void* q;
+  int64_t ld_q;
+  void* out;
+  int64_t ld_out;
+  void *k_cache, *v_cache;
+  const int32_t* block_tables; /* [segments, max_blocks] */
+  int64_t max_blocks, num_blocks;
+  const int32_t* row_segment;
+  const int32_t* positions;
+  int heads, kv_heads, dim, vdim, window, keep_first;
+  float scale;
+} hb_span_attention_args;
+int hb_span_attention_tile_positions(const hb_span_attention_args* a, hb_dtype dtype);
+int hb_span_attention(void* stream, const hb_span_attention_args* a, const int32_t* tiles, int n_tiles, const int32_t* rows,
+                      int n_rows, int n_splits, float* workspace, hb_dtype dtype);
+/* K and V rows (stride ld elements) to their slots (block*16 + offset; negative: skipped). */
+int hb_span_kv_write(void* stream, const hb_span_attention_args* a, const void* k, const void* v, int64_t ld,
+                     const int64_t* slots, int64_t rows, hb_dtype dtype);
+
+/* S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per head, state and outputs fp32.
+ * p holds q, k (heads*dim), v (heads*vdim) and, for a low-rank decay, rank columns, at the given
+ * column offsets; q is scaled by q_scale, q, k and v pass through SiLU when silu_qkv.  Decay:
+ * `decay` [heads], or (decay NULL) sigmoid(a2 . p[off_a1..] + a2_bias)^(1/tau) per key channel.
+ * segments {first row, rows, first position, state slot}: position 0 starts from a zero state.
+ * `list`: segments that go token by token; `chunks` {segment, first row, rows <= 64, index} and
+ * `long_segments` {segment, first chunk, chunks, -}: segments that go in chunks on tensor cores
+ * (bf16; hb_linear_recurrence_chunked tells whether these sizes are taken); their workspaces are
+ * cum: rows*heads*dim floats and chunk_state: n_chunks*heads*dim*vdim floats. */
+typedef struct hb_linear_recurrence_args {
+  const void* p;
+  int64_t ld;
+  int off_q, off_k, off_v, off_a1, heads, dim, vdim;
+  float q_scale;
+  int silu_qkv;
+  const float *decay, *a2, *a2_bias;
+  int rank;
+  float tau;
+  float* state; /* [slots, heads, dim, vdim] */
+  float* o;     /* row r, head h at o + r*ld_o + h*vdim */
+  int64_t ld_o;
+  const int32_t* segments;
+} hb_linear_recurrence_args;
+int hb_linear_recurrence_chunked(const hb_linear_recurrence_args* a, hb_dtype dtype);
+int hb_linear_recurrence(void* stream, const hb_linear_recurrence_args* a, const int32_t* list, int n_list,
+                         const int32_t* chunks, int n_chunks, const int32_t* long_segments, int n_long, float* cum,
+                         float* chunk_state, hb_dtype dtype);
+
+/* Several residual streams x [rows, streams, width] in fp32.
+ * hb_streams_embed: every stream = embed[ids] + pos_table[positions]; h = rms(sum_s in[s] x_s) *
+ * (1 + norm).  hb_streams_mix: x_t = sum_s mix[s,t] x_s + out[t] y, then h = rms(sum_t
+ * next_in[t] x_t) * (1 + next_norm) (next_norm NULL: no h).  With y2 (and weights w1, w2) y is
+ * (rms(y) w1 + rms(y2) w2) / 2.  hb_streams_final: h_i = rms(sum_s x[want_i, s]) * (1 + norm).
+ * Vectors fp32; h rows of stride ld_h and the tables in `dtype`; y rows of stride ld_y, fp32. */
+int hb_streams_embed(void* stream, float* x, void* h, const void* embed, const void* pos_table, const uint32_t* ids,
+                     const int32_t* positions, const float* in, const float* norm, int64_t rows, int streams, int64_t width,
+                     int64_t ld_h, int64_t vocab, int64_t max_positions, float eps, hb_dtype dtype);
+int hb_streams_mix(void* stream, float* x, void* h, const float* y, const float* y2, int64_t ld_y, const float* mix,
+                   const float* out, const float* next_in, const float* next_norm, const float* w1, const float* w2,
+                   int64_t rows, int streams, int64_t width, int64_t ld_h, float eps, hb_dtype dtype);
+int hb_streams_final(void* stream, void* h, const float* x, const int32_t* want, const float* norm, int64_t n_want,
+                     int streams, int64_t width, int64_t ld_h, float eps, hb_dtype dtype);
+/* out[r, g*size + i] = o / rms over group g * weight[i] * act(gate); the weight [size] is shared by the
+ * groups; act: SiLU, or sigmoid when gate_silu is 0. */
+int hb_gated_group_norm(void* stream, void* out, int64_t ld_out, const float* o, int64_t ld_o, const void* gate,
+                        int64_t ld_gate, const float* weight, int64_t rows, int groups, int size, int gate_silu, float eps,
+                        hb_dtype dtype);
+
 /* --------------------------------------------------------------- comm surface */
 
 /* One rank's membership of a tensor-parallel group: the replacement of TpWorld

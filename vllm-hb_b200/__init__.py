@@ -94,6 +94,27 @@ class ModelShape(C.Structure):
     ]
 
 
+class SpanAttentionArgs(C.Structure):
+    """hb_span_attention_args: paged attention over a window and the first kept positions."""
+    _fields_ = [
+        ("q", C.c_void_p), ("ld_q", C.c_int64), ("out", C.c_void_p), ("ld_out", C.c_int64),
+        ("k_cache", C.c_void_p), ("v_cache", C.c_void_p), ("block_tables", C.c_void_p),
+        ("max_blocks", C.c_int64), ("num_blocks", C.c_int64), ("row_segment", C.c_void_p), ("positions", C.c_void_p),
+        ("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("window", C.c_int),
+        ("keep_first", C.c_int), ("scale", C.c_float),
+    ]
+
+
+class LinearRecurrenceArgs(C.Structure):
+    """hb_linear_recurrence_args: gated linear recurrence with a matrix state per head."""
+    _fields_ = [
+        ("p", C.c_void_p), ("ld", C.c_int64), ("off_q", C.c_int), ("off_k", C.c_int), ("off_v", C.c_int),
+        ("off_a1", C.c_int), ("heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("q_scale", C.c_float),
+        ("silu_qkv", C.c_int), ("decay", C.c_void_p), ("a2", C.c_void_p), ("a2_bias", C.c_void_p), ("rank", C.c_int),
+        ("tau", C.c_float), ("state", C.c_void_p), ("o", C.c_void_p), ("ld_o", C.c_int64), ("segments", C.c_void_p),
+    ]
+
+
 _vp, _i, _i64, _f, _sz, _u64 = C.c_void_p, C.c_int, C.c_int64, C.c_float, C.c_size_t, C.c_uint64
 
 _SIGS = {
@@ -113,6 +134,15 @@ _SIGS = {
     "hb_moe_route": (_i, [_vp, _vp, _vp, _vp, _i64, _i64, _i, _i, _i]),
     "hb_paged_decode_attention_static_max_bytes": (_sz, []),
     "hb_paged_decode_attention_static": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i, _i, _i, _i64, _i64, _i, _i]),
+    "hb_span_attention_tile_positions": (_i, [_vp, _i]),
+    "hb_span_attention": (_i, [_vp, _vp, _vp, _i, _vp, _i, _i, _vp, _i]),
+    "hb_span_kv_write": (_i, [_vp, _vp, _vp, _vp, _i64, _vp, _i64, _i]),
+    "hb_linear_recurrence_chunked": (_i, [_vp, _i]),
+    "hb_linear_recurrence": (_i, [_vp, _vp, _vp, _i, _vp, _i, _vp, _i, _vp, _vp, _i]),
+    "hb_streams_embed": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i, _i64, _i64, _i64, _i64, _f, _i]),
+    "hb_streams_mix": (_i, [_vp, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i, _i64, _i64, _f, _i]),
+    "hb_streams_final": (_i, [_vp, _vp, _vp, _vp, _vp, _i64, _i, _i64, _i64, _f, _i]),
+    "hb_gated_group_norm": (_i, [_vp, _vp, _i64, _vp, _i64, _vp, _i64, _vp, _i64, _i, _i, _i, _f, _i]),
     "hb_gemm_workspace_bytes": (_sz, [_i64, _i64, _i64, _i]),
     "hb_gemm": (_i, [_vp, _vp, _vp, _vp, _i64, _i64, _i64, _i, _vp]),
     "hb_gemm_ex_workspace_bytes": (_sz, [_i64, _i64, _i64, _i, _i]),

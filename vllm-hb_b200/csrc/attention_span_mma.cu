@@ -1,0 +1,485 @@
+// Span attention (see attention_span.cu) on tensor cores: bf16, key and value widths that are
+// multiples of 8.  S = Q K^T with bf16 operands and fp32 accumulation, softmax in fp32, and
+// O += P V with P as a pair of bf16 numbers (P = hi + lo), so that the weights keep fp32-like
+// precision.
+//
+//   tiles  (prompt portions): CTA = 64 rows = up to 64 / R consecutive positions of one segment x
+//          the R query heads of a kv head; four warps of 16 rows share every 64-key tile.
+//   tokens (decoded tokens): CTA = one row and kv head, the R <= 16 query heads padded to 16 MMA
+//          rows; each of four warps streams every fourth 16-key block through a ring of its own
+//          and the warps' (m, l, O) meet in shared memory.
+//
+// Both read only the 16-key blocks that some row of the CTA sees: those of the first kept tokens
+// and those from the earliest window on.  Rows of shared memory are padded by 8 elements, so that
+// ldmatrix is conflict-free for every width.  Value widths above 256 are cut into slices (grid.z).
+#include <algorithm>
+#include <climits>
+
+#include "layered_ops.h"
+#include "mma_sync.cuh"
+#include "tc_core.cuh"
+
+namespace hb {
+
+namespace {
+constexpr int kThreads = 128;
+constexpr int kWarps = 4;
+constexpr int kRows = 64;      // query rows of a tile
+constexpr int kKeys = 64;      // keys of a tile step
+constexpr int kBS = HB_BLOCK_SIZE;
+constexpr int kSlice = 256;    // widest value slice
+constexpr int kRing = 3;       // 16-key stages of a warp (token kernel)
+
+__host__ __device__ constexpr int pad16(int n) { return (n + 15) / 16 * 16; }
+
+// The blocks a CTA reads: [0, na) of the kept tokens, then [b0, b1].
+struct BlockRuns {
+  int na, b0, n;
+  __device__ __forceinline__ int block(int i) const { return i < na ? i : b0 + (i - na); }
+};
+__device__ __forceinline__ BlockRuns block_runs(int first_pos, int last_pos, int window, int keep_first) {
+  BlockRuns r;
+  const int lo = window > 0 ? max(0, first_pos - window + 1) : 0;
+  r.b0 = lo / kBS;
+  r.na = min((min(keep_first, lo) + kBS - 1) / kBS, r.b0);
+  r.n = r.na + last_pos / kBS - r.b0 + 1;
+  return r;
+}
+__device__ __forceinline__ bool visible(int key, int pos, int window, int keep_first) {
+  return key <= pos && (window <= 0 || pos - key < window || key < keep_first);
+}
+}  // namespace
+
+// NV: 16-column pairs of n-tiles, i.e. the value slice is at most 16 * NV wide.
+template <int NV>
+__global__ void __launch_bounds__(kThreads)
+span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ tiles, int stages) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  const int R = a.heads / a.kv_heads, D = a.dim, DP = pad16(D), KS = DP + 8;
+  const int v0 = blockIdx.z * kSlice, VW = min(kSlice, a.vdim - v0), VP = pad16(VW), VS = VP + 8;
+  __nv_bfloat16* s_q = (__nv_bfloat16*)smem;           // [64][KS]
+  __nv_bfloat16* s_k = s_q + kRows * KS;               // [stages][64][KS]
+  __nv_bfloat16* s_v = s_k + stages * kKeys * KS;      // [stages][64][VS]
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gi = lane >> 2, t = lane & 3, kvh = blockIdx.y;
+  // padding columns stay zero
+  for (int i = tid; i < (kRows + stages * kKeys) * KS / 8; i += kThreads)
+    if (i % (KS / 8) * 8 >= D) reinterpret_cast<uint4*>(s_q)[i] = make_uint4(0, 0, 0, 0);
+  for (int i = tid; i < stages * kKeys * VS / 8; i += kThreads)
+    if (i % (VS / 8) * 8 >= VW) reinterpret_cast<uint4*>(s_v)[i] = make_uint4(0, 0, 0, 0);
+  pdl_grid_wait();
+  const RowRange tile = tiles[blockIdx.x];
+  const int first_pos = a.pos[tile.row0], last_pos = first_pos + tile.n - 1;
+  const BlockRuns runs = block_runs(first_pos, last_pos, a.window, a.keep_first);
+  const int32_t* table = a.tables + (int64_t)tile.seg * a.max_blocks;
+  const int n_rows = tile.n * R, n_steps = (runs.n + kKeys / kBS - 1) / (kKeys / kBS);
+
+  const __nv_bfloat16* q = (const __nv_bfloat16*)a.q + (int64_t)kvh * R * D;
+  for (int i = tid; i < kRows * (D / 8); i += kThreads) {
+    const int m = i / (D / 8), c = i % (D / 8) * 8;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (m < n_rows) v = *reinterpret_cast<const uint4*>(q + (int64_t)(tile.row0 + m / R) * a.ld_q + (m % R) * D + c);
+    *reinterpret_cast<uint4*>(s_q + m * KS + c) = v;
+  }
+  auto load = [&](int step) {
+    const int s = step % stages;
+    const uint32_t dk = smem_u32(s_k + s * kKeys * KS), dv = smem_u32(s_v + s * kKeys * VS);
+    const int kc = D / 8, vc = VW / 8;
+    for (int i = tid; i < kKeys * (kc + vc); i += kThreads) {
+      const bool is_k = i < kKeys * kc;
+      const int w = is_k ? kc : vc, e = is_k ? i : i - kKeys * kc, j = e / w, c = e % w * 8;
+      const int vb = step * (kKeys / kBS) + j / kBS;
+      // past the last block: any block will do, its keys are masked (positions beyond the row's)
+      const int lb = runs.block(min(vb, runs.n - 1));
+      int64_t phys = lb < a.max_blocks ? table[lb] : 0;
+      if (phys < 0 || phys >= a.num_blocks) phys = 0;  // never outside the pool
+      const int64_t slot = (phys * a.kv_heads + kvh) * kBS + j % kBS;
+      if (is_k) cp_async_16(dk + (j * KS + c) * 2, (const __nv_bfloat16*)a.kc + slot * D + c);
+      else cp_async_16(dv + (j * VS + c) * 2, (const __nv_bfloat16*)a.vc + slot * a.vdim + v0 + c);
+    }
+    cp_async_commit();
+  };
+  load(0);
+
+  const int r0 = warp * 16 + gi, r1 = r0 + 8;
+  const int p0 = first_pos + r0 / R, p1 = first_pos + r1 / R;
+  const bool live = warp * 16 < n_rows;  // warps without rows only help to load
+  float o[2 * NV][4];
+#pragma unroll
+  for (int i = 0; i < 2 * NV; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+  const float sc = a.scale * 1.4426950408889634f;  // scores in units of log2
+  const uint32_t q_addr = smem_u32(s_q + (warp * 16 + (lane & 15)) * KS + (lane >> 4) * 8);
+
+  for (int step = 0; step < n_steps; ++step) {
+    if (stages > 1 && step + 1 < n_steps) {
+      load(step + 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    if (live) {
+      const __nv_bfloat16* kt = s_k + step % stages * kKeys * KS;
+      const __nv_bfloat16* vt = s_v + step % stages * kKeys * VS;
+      float s[8][4];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+      // lanes 0-7 / 8-15 / 16-23 / 24-31 address keys 0-7 k-low, 0-7 k-high, 8-15 k-low, 8-15 k-high
+      const uint32_t k_addr = smem_u32(kt + ((lane & 7) + (lane >> 4) * 8) * KS + ((lane >> 3) & 1) * 8);
+      for (int ks = 0; ks < DP / 16; ++ks) {
+        uint32_t qa[4];
+        ldsm_x4(q_addr + ks * 32, qa[0], qa[1], qa[2], qa[3]);
+#pragma unroll
+        for (int nk = 0; nk < 4; ++nk) {
+          uint32_t b0, b1, b2, b3;
+          ldsm_x4(k_addr + (nk * 16 * KS + ks * 16) * 2, b0, b1, b2, b3);
+          mma_bf16_16816(s[2 * nk], qa, b0, b1);
+          mma_bf16_16816(s[2 * nk + 1], qa, b2, b3);
+        }
+      }
+      float x0 = -INFINITY, x1 = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const int vb = step * (kKeys / kBS) + i / 2;
+        const int key = vb < runs.n ? runs.block(vb) * kBS + (i & 1) * 8 + 2 * t : INT_MAX - 1;
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          s[i][c] = visible(key + c, p0, a.window, a.keep_first) ? s[i][c] * sc : -INFINITY;
+          s[i][2 + c] = visible(key + c, p1, a.window, a.keep_first) ? s[i][2 + c] * sc : -INFINITY;
+          x0 = fmaxf(x0, s[i][c]);
+          x1 = fmaxf(x1, s[i][2 + c]);
+        }
+      }
+      x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 1)); x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 2));
+      x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 1)); x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
+      const float n0 = fmaxf(m0, x0), n1 = fmaxf(m1, x1);
+      const float e0 = n0 == -INFINITY ? 0.f : n0, e1 = n1 == -INFINITY ? 0.f : n1;  // nothing visible yet
+      const float al0 = exp2f(m0 - e0), al1 = exp2f(m1 - e1);
+      m0 = n0; m1 = n1;
+      l0 *= al0; l1 *= al1;
+#pragma unroll
+      for (int i = 0; i < 2 * NV; ++i) { o[i][0] *= al0; o[i][1] *= al0; o[i][2] *= al1; o[i][3] *= al1; }
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        s[i][0] = exp2f(s[i][0] - e0); s[i][1] = exp2f(s[i][1] - e0);
+        s[i][2] = exp2f(s[i][2] - e1); s[i][3] = exp2f(s[i][3] - e1);
+        l0 += s[i][0] + s[i][1];
+        l1 += s[i][2] + s[i][3];
+      }
+      const uint32_t v_addr = smem_u32(vt + (lane & 15) * VS + (lane >> 4) * 8);
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk) {
+        uint32_t hi[4], lo[4];
+        split_bf16(s[2 * kk][0], s[2 * kk][1], hi[0], lo[0]);
+        split_bf16(s[2 * kk][2], s[2 * kk][3], hi[1], lo[1]);
+        split_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1], hi[2], lo[2]);
+        split_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3], hi[3], lo[3]);
+#pragma unroll
+        for (int nv = 0; nv < NV; ++nv) {
+          if (nv * 16 < VP) {
+            uint32_t b0, b1, b2, b3;
+            ldsm_x4_trans(v_addr + (kk * 16 * VS + nv * 16) * 2, b0, b1, b2, b3);
+            mma_bf16_16816(o[2 * nv], hi, b0, b1);
+            mma_bf16_16816(o[2 * nv + 1], hi, b2, b3);
+            mma_bf16_16816(o[2 * nv], lo, b0, b1);
+            mma_bf16_16816(o[2 * nv + 1], lo, b2, b3);
+          }
+        }
+      }
+    }
+    __syncthreads();
+    if (stages == 1 && step + 1 < n_steps) load(step + 1);
+  }
+  pdl_trigger();
+  if (!live) return;
+  l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
+  l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+  const float i0 = 1.f / l0, i1 = 1.f / l1;
+  __nv_bfloat16* out = (__nv_bfloat16*)a.out + (int64_t)kvh * R * a.vdim + v0;
+  __nv_bfloat16* w0 = out + (int64_t)(tile.row0 + r0 / R) * a.ld_out + (r0 % R) * a.vdim;
+  __nv_bfloat16* w1 = out + (int64_t)(tile.row0 + r1 / R) * a.ld_out + (r1 % R) * a.vdim;
+#pragma unroll
+  for (int i = 0; i < 2 * NV; ++i) {
+    const int c = i * 8 + 2 * t;
+    if (c < VW) {
+      if (r0 < n_rows) *reinterpret_cast<uint32_t*>(w0 + c) = pack_bf16(o[i][0] * i0, o[i][1] * i0);
+      if (r1 < n_rows) *reinterpret_cast<uint32_t*>(w1 + c) = pack_bf16(o[i][2] * i1, o[i][3] * i1);
+    }
+  }
+}
+
+// n_splits > 1: every CTA takes its share of the row's blocks and writes (m, l, O) partials.
+template <int NV>
+__global__ void __launch_bounds__(kThreads)
+span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, int n_splits, float* __restrict__ part) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  const int R = a.heads / a.kv_heads, D = a.dim, DP = pad16(D), KS = DP + 8;
+  const int slices = (a.vdim + kSlice - 1) / kSlice;
+  const int v0 = (int)(blockIdx.z % slices) * kSlice, VW = min(kSlice, a.vdim - v0), VP = pad16(VW), VS = VP + 8;
+  const int split = blockIdx.z / slices;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gi = lane >> 2, t = lane & 3, kvh = blockIdx.y;
+  const int stage_elems = kBS * (KS + VS);
+  __nv_bfloat16* s_q = (__nv_bfloat16*)smem;                                  // [16][KS]
+  __nv_bfloat16* ring = s_q + 16 * KS + (size_t)warp * kRing * stage_elems;   // [kRing][K 16 x KS | V 16 x VS]
+  for (int s = 0; s < kRing; ++s) {
+    for (int i = lane; i < kBS; i += 32) {
+      for (int c = D; c < KS; c += 8) *reinterpret_cast<uint4*>(ring + s * stage_elems + i * KS + c) = make_uint4(0, 0, 0, 0);
+      for (int c = VW; c < VS; c += 8)
+        *reinterpret_cast<uint4*>(ring + s * stage_elems + kBS * KS + i * VS + c) = make_uint4(0, 0, 0, 0);
+    }
+  }
+  pdl_grid_wait();
+  const int64_t row = rows[blockIdx.x];
+  const int pos = a.pos[row];
+  const int32_t* table = a.tables + (int64_t)a.row_seg[row] * a.max_blocks;
+  const BlockRuns runs = block_runs(pos, pos, a.window, a.keep_first);
+  const int per = (runs.n + n_splits - 1) / n_splits, s_lo = split * per, s_hi = min(runs.n, s_lo + per);
+  const int n_w = s_hi - s_lo > warp ? (s_hi - s_lo - warp + kWarps - 1) / kWarps : 0;  // this warp's blocks
+
+  int tab_base = 0, tab = 0;
+  auto load_tab = [&](int base) {  // block table entries of this warp, 32 at a time, one per lane
+    tab_base = base;
+    const int i = base + lane;
+    const int lb = i < n_w ? runs.block(s_lo + warp + kWarps * i) : 0;
+    tab = lb < a.max_blocks ? table[lb] : 0;
+    if (tab < 0 || tab >= a.num_blocks) tab = 0;  // never outside the pool
+  };
+  auto load = [&](int i) {
+    if (i < n_w) {
+      if (i >= tab_base + 32) load_tab(i);
+      const int64_t slot = ((int64_t)__shfl_sync(0xffffffffu, tab, i - tab_base) * a.kv_heads + kvh) * kBS;
+      const uint32_t dst = smem_u32(ring + i % kRing * stage_elems);
+      const __nv_bfloat16* k = (const __nv_bfloat16*)a.kc + slot * D;
+      const __nv_bfloat16* v = (const __nv_bfloat16*)a.vc + slot * a.vdim + v0;
+      for (int e = lane; e < kBS * (D / 8); e += 32) {
+        const int j = e / (D / 8), c = e % (D / 8) * 8;
+        cp_async_16(dst + (j * KS + c) * 2, k + j * D + c);
+      }
+      for (int e = lane; e < kBS * (VW / 8); e += 32) {
+        const int j = e / (VW / 8), c = e % (VW / 8) * 8;
+        cp_async_16(dst + (kBS * KS + j * VS + c) * 2, v + (int64_t)j * a.vdim + c);
+      }
+    }
+    cp_async_commit();
+  };
+  load_tab(0);
+  for (int i = 0; i < kRing - 1; ++i) load(i);
+  const __nv_bfloat16* q = (const __nv_bfloat16*)a.q + row * a.ld_q + (int64_t)kvh * R * D;
+  for (int i = tid; i < 16 * (KS / 8); i += kThreads) {
+    const int m = i / (KS / 8), c = i % (KS / 8) * 8;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (m < R && c < D) v = *reinterpret_cast<const uint4*>(q + m * D + c);
+    *reinterpret_cast<uint4*>(s_q + m * KS + c) = v;
+  }
+  __syncthreads();
+  float o[2 * NV][4];
+#pragma unroll
+  for (int i = 0; i < 2 * NV; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+  const float sc = a.scale * 1.4426950408889634f;
+  const uint32_t q_addr = smem_u32(s_q + (lane & 15) * KS + (lane >> 4) * 8);
+  for (int i = 0; i < n_w; ++i) {
+    load(i + kRing - 1);
+    cp_async_wait<kRing - 1>();
+    __syncwarp();
+    const __nv_bfloat16* kt = ring + i % kRing * stage_elems;
+    const __nv_bfloat16* vt = kt + kBS * KS;
+    float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+    const uint32_t k_addr = smem_u32(kt + ((lane & 7) + (lane >> 4) * 8) * KS + ((lane >> 3) & 1) * 8);
+    for (int ks = 0; ks < DP / 16; ++ks) {
+      uint32_t qa[4], b0, b1, b2, b3;
+      ldsm_x4(q_addr + ks * 32, qa[0], qa[1], qa[2], qa[3]);
+      ldsm_x4(k_addr + ks * 32, b0, b1, b2, b3);
+      mma_bf16_16816(s[0], qa, b0, b1);
+      mma_bf16_16816(s[1], qa, b2, b3);
+    }
+    const int key0 = runs.block(s_lo + warp + kWarps * i) * kBS;
+    float x0 = -INFINITY, x1 = -INFINITY;
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int c = 0; c < 2; ++c) {
+        const bool vis = visible(key0 + n * 8 + 2 * t + c, pos, a.window, a.keep_first);
+        s[n][c] = vis ? s[n][c] * sc : -INFINITY;
+        s[n][2 + c] = vis ? s[n][2 + c] * sc : -INFINITY;
+        x0 = fmaxf(x0, s[n][c]);
+        x1 = fmaxf(x1, s[n][2 + c]);
+      }
+    x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 1)); x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 2));
+    x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 1)); x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
+    const float n0 = fmaxf(m0, x0), n1 = fmaxf(m1, x1);
+    const float e0 = n0 == -INFINITY ? 0.f : n0, e1 = n1 == -INFINITY ? 0.f : n1;
+    const float al0 = exp2f(m0 - e0), al1 = exp2f(m1 - e1);
+    m0 = n0; m1 = n1;
+    l0 *= al0; l1 *= al1;
+#pragma unroll
+    for (int n = 0; n < 2 * NV; ++n) { o[n][0] *= al0; o[n][1] *= al0; o[n][2] *= al1; o[n][3] *= al1; }
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
+      s[n][0] = exp2f(s[n][0] - e0); s[n][1] = exp2f(s[n][1] - e0);
+      s[n][2] = exp2f(s[n][2] - e1); s[n][3] = exp2f(s[n][3] - e1);
+      l0 += s[n][0] + s[n][1];
+      l1 += s[n][2] + s[n][3];
+    }
+    uint32_t hi[4], lo[4];
+    split_bf16(s[0][0], s[0][1], hi[0], lo[0]);
+    split_bf16(s[0][2], s[0][3], hi[1], lo[1]);
+    split_bf16(s[1][0], s[1][1], hi[2], lo[2]);
+    split_bf16(s[1][2], s[1][3], hi[3], lo[3]);
+    const uint32_t v_addr = smem_u32(vt + (lane & 15) * VS + (lane >> 4) * 8);
+#pragma unroll
+    for (int nv = 0; nv < NV; ++nv) {
+      if (nv * 16 < VP) {
+        uint32_t b0, b1, b2, b3;
+        ldsm_x4_trans(v_addr + nv * 32, b0, b1, b2, b3);
+        mma_bf16_16816(o[2 * nv], hi, b0, b1);
+        mma_bf16_16816(o[2 * nv + 1], hi, b2, b3);
+        mma_bf16_16816(o[2 * nv], lo, b0, b1);
+        mma_bf16_16816(o[2 * nv + 1], lo, b2, b3);
+      }
+    }
+    __syncwarp();  // the stage is refilled by the next iteration's load
+  }
+  cp_async_wait<0>();
+  pdl_trigger();
+  l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
+  l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+  // the warps' results meet in shared memory (the rings are idle now)
+  __syncthreads();
+  const int OS = VP + 2;
+  float* s_o = (float*)(s_q + 16 * KS);          // [kWarps][R][OS]
+  float* s_ml = s_o + (size_t)kWarps * R * OS;   // [kWarps][R][2]
+  auto put = [&](int m, float mm, float ll, int half) {
+    if (m >= R) return;
+    float* dst = s_o + ((size_t)warp * R + m) * OS;
+#pragma unroll
+    for (int n = 0; n < 2 * NV; ++n)
+      if (n * 8 < VP) *reinterpret_cast<float2*>(dst + n * 8 + 2 * t) = make_float2(o[n][half], o[n][half + 1]);
+    if (t == 0) { s_ml[(warp * R + m) * 2] = mm; s_ml[(warp * R + m) * 2 + 1] = ll; }
+  };
+  put(gi, m0, l0, 0);
+  put(gi + 8, m1, l1, 2);
+  __syncthreads();
+  for (int i = tid; i < R * VW; i += kThreads) {
+    const int m = i / VW, c = i % VW;
+    float mx = -INFINITY, l = 0.f, acc = 0.f;
+#pragma unroll
+    for (int w = 0; w < kWarps; ++w) mx = fmaxf(mx, s_ml[(w * R + m) * 2]);
+#pragma unroll
+    for (int w = 0; w < kWarps; ++w) {
+      const float mw = s_ml[(w * R + m) * 2];
+      const float f = mw == -INFINITY ? 0.f : exp2f(mw - mx);
+      l = fmaf(f, s_ml[(w * R + m) * 2 + 1], l);
+      acc = fmaf(f, s_o[((size_t)w * R + m) * OS + c], acc);
+    }
+    const int64_t head = (int64_t)kvh * R + m;
+    if (n_splits == 1) {
+      ((__nv_bfloat16*)a.out)[row * a.ld_out + head * a.vdim + v0 + c] = __float2bfloat16_rn(acc / l);
+    } else {
+      float* p = part + (((int64_t)blockIdx.x * a.heads + head) * n_splits + split) * (a.vdim + 2);
+      p[v0 + c] = acc;
+      if (c == 0 && v0 == 0) { p[a.vdim] = mx; p[a.vdim + 1] = l; }
+    }
+  }
+}
+
+// Sum of a row's split partials, weighted by their maxima.
+__global__ void __launch_bounds__(kThreads)
+span_attention_merge_kernel(const SpanAttention a, const int32_t* __restrict__ rows, int n_splits, const float* __restrict__ part) {
+  pdl_trigger();
+  pdl_grid_wait();
+  const int64_t row = rows[blockIdx.x];
+  const int head = blockIdx.y;
+  const float* p = part + ((int64_t)blockIdx.x * a.heads + head) * n_splits * (a.vdim + 2);
+  float mx = -INFINITY, l = 0.f;
+  for (int s = 0; s < n_splits; ++s) mx = fmaxf(mx, p[s * (a.vdim + 2) + a.vdim]);
+  for (int s = 0; s < n_splits; ++s) {
+    const float m = p[s * (a.vdim + 2) + a.vdim];
+    if (m != -INFINITY) l = fmaf(exp2f(m - mx), p[s * (a.vdim + 2) + a.vdim + 1], l);
+  }
+  for (int c = threadIdx.x; c < a.vdim; c += kThreads) {
+    float acc = 0.f;
+    for (int s = 0; s < n_splits; ++s) {
+      const float m = p[s * (a.vdim + 2) + a.vdim];
+      if (m != -INFINITY) acc = fmaf(exp2f(m - mx), p[s * (a.vdim + 2) + c], acc);
+    }
+    ((__nv_bfloat16*)a.out)[row * a.ld_out + (int64_t)head * a.vdim + c] = __float2bfloat16_rn(acc / l);
+  }
+}
+
+static size_t tiles_smem(const SpanAttention& a, int stages) {
+  const int KS = pad16(a.dim) + 8, VS = pad16(std::min(a.vdim, kSlice)) + 8;
+  return (size_t)(kRows * KS + stages * kKeys * (KS + VS)) * 2;
+}
+static size_t tokens_smem(const SpanAttention& a) {
+  const int R = a.heads / a.kv_heads, KS = pad16(a.dim) + 8, VP = pad16(std::min(a.vdim, kSlice)), VS = VP + 8;
+  const size_t ring = (size_t)kWarps * kRing * kBS * (KS + VS) * 2;
+  const size_t merge = (size_t)kWarps * R * (VP + 4) * sizeof(float);
+  return (size_t)16 * KS * 2 + std::max(ring, merge);
+}
+constexpr size_t kSmemCap = 224 * 1024;
+
+static bool span_mma_ok(const SpanAttention& a, hb_dtype dtype) {
+  auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  static const bool simt = [] { const char* e = getenv("HB_ATTN"); return e && e[0] == 's'; }();
+  return !simt && dtype == HB_BF16 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ld_q % 8 == 0 && a.ld_out % 2 == 0 && al(a.q) &&
+         al(a.out);
+}
+
+int span_attention_tile_positions(const SpanAttention& a, hb_dtype dtype) {
+  const int R = a.heads / a.kv_heads;
+  if (!span_mma_ok(a, dtype) || R > kRows || tiles_smem(a, 1) > kSmemCap) return 0;
+  return kRows / R;
+}
+bool span_attention_tokens_supported(const SpanAttention& a, hb_dtype dtype) {
+  return span_mma_ok(a, dtype) && a.heads / a.kv_heads <= 16 && tokens_smem(a) <= kSmemCap;
+}
+
+template <typename K>
+static int opt_in(K kernel, size_t smem) {
+  if (smem > 48 * 1024) HB_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemCap));
+  return HB_OK;
+}
+
+int span_attention_tiles(cudaStream_t st, const SpanAttention& a, const RowRange* tiles, int n_tiles) {
+  if (n_tiles == 0) return HB_OK;
+  const int stages = tiles_smem(a, 2) <= kSmemCap ? 2 : 1;
+  const size_t smem = tiles_smem(a, stages);
+  const dim3 grid((unsigned)n_tiles, (unsigned)a.kv_heads, (unsigned)((a.vdim + kSlice - 1) / kSlice));
+  auto launch = [&](auto* k) -> int {
+    int rc = opt_in(k, smem);
+    if (rc) return rc;
+    HB_CUDA_CHECK(launch_pdl(k, grid, dim3(kThreads), smem, st, a, tiles, stages));
+    return HB_OK;
+  };
+  const int vw = std::min(a.vdim, kSlice);
+  if (vw <= 64) return launch(span_attention_tiles_kernel<4>);
+  if (vw <= 128) return launch(span_attention_tiles_kernel<8>);
+  if (vw <= 192) return launch(span_attention_tiles_kernel<12>);
+  return launch(span_attention_tiles_kernel<16>);
+}
+
+int span_attention_tokens(cudaStream_t st, const SpanAttention& a, const int32_t* rows, int n_rows, int n_splits, float* part) {
+  if (n_rows == 0) return HB_OK;
+  const size_t smem = tokens_smem(a);
+  const int slices = (a.vdim + kSlice - 1) / kSlice;
+  const dim3 grid((unsigned)n_rows, (unsigned)a.kv_heads, (unsigned)(slices * n_splits));
+  auto launch = [&](auto* k) -> int {
+    int rc = opt_in(k, smem);
+    if (rc) return rc;
+    HB_CUDA_CHECK(launch_pdl(k, grid, dim3(kThreads), smem, st, a, rows, n_splits, part));
+    return HB_OK;
+  };
+  const int vw = std::min(a.vdim, kSlice);
+  int rc;
+  if (vw <= 64) rc = launch(span_attention_tokens_kernel<4>);
+  else if (vw <= 128) rc = launch(span_attention_tokens_kernel<8>);
+  else if (vw <= 192) rc = launch(span_attention_tokens_kernel<12>);
+  else rc = launch(span_attention_tokens_kernel<16>);
+  if (rc || n_splits == 1) return rc;
+  HB_CUDA_CHECK(launch_pdl(span_attention_merge_kernel, dim3((unsigned)n_rows, (unsigned)a.heads), dim3(kThreads), 0, st, a, rows,
+                           n_splits, (const float*)part));
+  return HB_OK;
+}
+
+}  // namespace hb

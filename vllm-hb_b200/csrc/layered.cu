@@ -188,13 +188,78 @@ static size_t layered_layout(const hb_engine* e, LayeredStep* s) {
   s->off_row_seg = l.take((size_t)s->rows * 4);
   s->off_want = l.take((size_t)s->want * 4);
   s->off_seg = l.take((size_t)s->segs * sizeof(SegInfo));
-  s->off_short = l.take((size_t)s->n_short * 4);
-  s->off_long = l.take((size_t)s->n_long * 4);
+  s->off_short = l.take((size_t)s->segs * 4);
+  s->off_long = l.take((size_t)s->n_long * sizeof(RowRange));
   s->off_chunk = l.take((size_t)s->n_chunks * sizeof(RowRange));
   s->off_tile = l.take((size_t)s->n_tiles * sizeof(RowRange));
-  s->off_attn_rows = l.take((size_t)s->n_attn_rows * 4);
+  s->off_row_list = l.take((size_t)s->rows * 4);
   s->off_tables = l.take((size_t)s->segs * e->max_blocks_per_seq * 4);
   return l.bytes;
+}
+
+// Segments of up to this many tokens go through the recurrence token by token.
+constexpr int kShortSegment = 8;
+// Decoded tokens: with fewer (row, kv head) units than this the keys are split over several CTAs.
+constexpr int kSplitUnits = 296;
+
+static SpanAttention span_args(const hb_engine* e, size_t i, const LayeredStep& s) {
+  const LayeredModel* m = e->lm.get();
+  const MixerSpec& mx = m->spec.layers[i].mixer;
+  const AttentionSpec& as = mx.attn;
+  const LayeredLayer& l = m->layers[i];
+  SpanAttention a;
+  a.q = (const uint8_t*)m->proj + mx.aq.offset * e->es; a.ld_q = l.proj.N;
+  a.out = m->attn; a.ld_out = l.attn_o.K;
+  a.kc = e->kc[l.kv_pool]; a.vc = e->vc[l.kv_pool];
+  a.tables = (const int32_t*)(e->d_inputs + s.off_tables);
+  a.max_blocks = e->max_blocks_per_seq; a.num_blocks = e->num_blocks;
+  a.row_seg = (const int32_t*)(e->d_inputs + s.off_row_seg);
+  a.pos = (const int32_t*)(e->d_inputs + s.off_pos);
+  a.heads = as.heads; a.kv_heads = as.kv_heads; a.dim = as.dim; a.vdim = as.vdim;
+  a.window = as.window; a.keep_first = as.keep_first; a.scale = as.scale;
+  return a;
+}
+
+// Prompt portions as tiles, decoded tokens as rows; sizes the tensor-core kernels do not take go
+// row by row.
+static int issue_attention(hb_engine* e, const SpanAttention& a, const LayeredStep& s) {
+  LayeredModel* m = e->lm.get();
+  cudaStream_t st = e->stream;
+  const int32_t* rows = (const int32_t*)(e->d_inputs + s.off_row_list);
+  int rc;
+  if (!m->tile_positions || span_attention_tile_positions(a, e->dtype) < m->tile_positions) {
+    ++e->last_launches;
+    return span_attention_rows(st, a, rows, s.rows, e->dtype);
+  }
+  if (s.n_tiles) {
+    ++e->last_launches;
+    if ((rc = span_attention_tiles(st, a, (const RowRange*)(e->d_inputs + s.off_tile), s.n_tiles))) return rc;
+  }
+  if (!s.n_token_rows) return HB_OK;
+  ++e->last_launches;
+  if (!span_attention_tokens_supported(a, e->dtype)) return span_attention_rows(st, a, rows, s.n_token_rows, e->dtype);
+  // the longest span a row can have decides the split: it is the same in every replay of a graph
+  const int64_t longest = a.window > 0 ? (int64_t)a.window + a.keep_first : a.max_blocks * HB_BLOCK_SIZE;
+  const int64_t blocks = std::min<int64_t>(longest / HB_BLOCK_SIZE + 2, a.max_blocks), units = (int64_t)s.n_token_rows * a.kv_heads;
+  int64_t splits = units < kSplitUnits / 2 ? std::min((kSplitUnits + units - 1) / units, (blocks + 15) / 16) : 1;
+  splits = std::max<int64_t>(1, std::min<int64_t>(splits, 16));
+  if (splits > 1) ++e->last_launches;
+  return span_attention_tokens(st, a, rows, s.n_token_rows, (int)splits, m->attn_part);
+}
+
+static int issue_recurrence(hb_engine* e, const Recurrence& r, const LayeredStep& s) {
+  LayeredModel* m = e->lm.get();
+  const int32_t* list = (const int32_t*)(e->d_inputs + s.off_short);
+  const bool chunked = e->use_tc && recurrence_chunks_supported(r, e->dtype);
+  const int n_list = chunked ? s.n_short : s.segs;  // short segments first, longer ones after them
+  if (n_list) ++e->last_launches;
+  int rc = recurrence_tokens(e->stream, r, list, n_list, e->dtype);
+  if (rc || !chunked) return rc;
+  RecurrenceChunks c;
+  c.chunks = (const RowRange*)(e->d_inputs + s.off_chunk); c.n_chunks = s.n_chunks;
+  c.segs = (const RowRange*)(e->d_inputs + s.off_long); c.n_segs = s.n_long;
+  c.cum = m->cum; c.state = m->chunk_state;
+  return recurrence_chunks(e->stream, r, c, &e->last_launches);
 }
 
 static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
@@ -211,7 +276,8 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   for (int64_t b = 0; b < e->num_blocks; ++b) e->free_blocks.push_back(b);
   const int64_t R = pad_to(e->max_batch, 128);
   m->row_cap = R;
-  int64_t max_attn = 0, max_rec = 0, max_o = 0, max_ffp = 0;
+  m->max_chunks = e->max_batch / kRecChunk + std::min(m->max_segs, e->max_batch / (kShortSegment + 1)) + 1;
+  int64_t max_attn = 0, max_rec = 0, max_o = 0, max_ffp = 0, max_cum = 0, max_state = 0, max_part = 0;
   for (size_t i = 0; i < s.layers.size(); ++i) {
     LayeredLayer& l = m->layers[i];
     const MixerSpec& mx = s.layers[i].mixer;
@@ -230,6 +296,7 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
       e->k_block_bytes.push_back(kb);
       e->v_block_bytes.push_back(vb);
       max_attn = std::max(max_attn, l.attn_o.K);
+      max_part = std::max(max_part, (int64_t)kSplitUnits * 2 * (a.heads / a.kv_heads) * (a.vdim + 2));
     }
     if (mx.has_rec) {
       const RecurrenceSpec& r = mx.rec;
@@ -237,6 +304,8 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
       if ((rc = dev_alloc(e, (void**)&l.state, (size_t)m->max_segs * r.heads * r.dim * r.vdim * 4, true))) return rc;
       max_rec = std::max(max_rec, l.rec_o.K);
       max_o = std::max(max_o, (int64_t)r.heads * r.vdim);
+      if (r.low_rank_decay) max_cum = std::max(max_cum, (int64_t)r.heads * r.dim);
+      max_state = std::max(max_state, (int64_t)r.heads * r.dim * r.vdim);
     }
   }
   for (int i = 0; i < e->num_state_slots; ++i) e->free_slots.push_back(i);
@@ -248,6 +317,16 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   if ((rc = dev_alloc(e, &m->attn, (size_t)R * max_attn * es, true))) return rc;
   if ((rc = dev_alloc(e, &m->rec, (size_t)R * max_rec * es, true))) return rc;
   if ((rc = dev_alloc(e, (void**)&m->o, (size_t)R * max_o * 4, true))) return rc;
+  if (e->use_tc) {
+    if ((rc = dev_alloc(e, (void**)&m->cum, (size_t)R * max_cum * 4))) return rc;
+    if ((rc = dev_alloc(e, (void**)&m->chunk_state, (size_t)m->max_chunks * max_state * 4))) return rc;
+    if ((rc = dev_alloc(e, (void**)&m->attn_part, (size_t)max_part * 4))) return rc;
+  }
+  for (size_t i = 0; i < s.layers.size(); ++i)
+    if (s.layers[i].mixer.has_attn) {
+      const int tp = span_attention_tile_positions(span_args(e, i, LayeredStep()), e->dtype);
+      if (tp > 0) m->tile_positions = m->tile_positions ? std::min(m->tile_positions, tp) : tp;
+    }
   if ((rc = dev_alloc(e, (void**)&m->y1, (size_t)R * m->Hp * 4, true))) return rc;
   if ((rc = dev_alloc(e, (void**)&m->y2, (size_t)R * m->Hp * 4, true))) return rc;
   if (!e->use_tc && (rc = dev_alloc(e, &m->gu, (size_t)R * 2 * max_ffp * es, true))) return rc;
@@ -261,9 +340,9 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   LayeredStep cap;
   cap.rows = e->max_batch;
   cap.want = e->max_batch;
-  cap.segs = cap.n_short = cap.n_long = m->max_segs;
-  cap.n_chunks = cap.n_tiles = e->max_batch + m->max_segs;
-  cap.n_attn_rows = e->max_batch;
+  cap.segs = cap.n_long = m->max_segs;
+  cap.n_chunks = m->max_chunks;
+  cap.n_tiles = e->max_batch + m->max_segs;
   e->inputs_bytes = layered_layout(e, &cap);
   if ((rc = dev_alloc(e, (void**)&e->d_inputs, e->inputs_bytes, true))) return rc;
   HB_CUDA_CHECK(cudaMallocHost((void**)&e->h_inputs, e->inputs_bytes));
@@ -326,8 +405,12 @@ static int layered_prepare(hb_engine* e, const StepBatch& batch, StepExec* x) {
   s.segs = (int)batch.segs.size();
   s.want = (int)batch.want.size();
   s.decode = s.rows == s.segs;
-  s.n_short = s.segs;
-  s.n_attn_rows = s.rows;
+  for (const StepSeg& t : batch.segs) {
+    if (t.n <= kShortSegment) ++s.n_short;
+    else { ++s.n_long; s.n_chunks += (t.n + kRecChunk - 1) / kRecChunk; }
+    if (t.n == 1) ++s.n_token_rows;
+    else if (m->tile_positions) s.n_tiles += (t.n + m->tile_positions - 1) / m->tile_positions;
+  }
   x->rows = batch.rows;
   x->logits_compact = true;
   x->input_bytes = layered_layout(e, &s);
@@ -339,19 +422,34 @@ static int layered_prepare(hb_engine* e, const StepBatch& batch, StepExec* x) {
   int32_t* row_seg = (int32_t*)(in + s.off_row_seg);
   SegInfo* seg = (SegInfo*)(in + s.off_seg);
   int32_t* shorts = (int32_t*)(in + s.off_short);
-  int32_t* attn_rows = (int32_t*)(in + s.off_attn_rows);
+  RowRange* longs = (RowRange*)(in + s.off_long);
+  RowRange* chunks = (RowRange*)(in + s.off_chunk);
+  RowRange* tiles = (RowRange*)(in + s.off_tile);
+  int32_t* row_list = (int32_t*)(in + s.off_row_list);
+  int at_short = 0, at_long = s.n_short, n_long = 0, n_chunks = 0, n_tiles = 0, at_token = 0, at_row = s.n_token_rows;
   int32_t* tables = (int32_t*)(in + s.off_tables);
   for (int g = 0; g < s.segs; ++g) {
     const StepSeg& t = batch.segs[g];
     seg[g] = {t.row0, t.n, (int32_t)t.pos0, t.state_slot};
-    shorts[g] = g;
+    if (t.n <= kShortSegment) {
+      shorts[at_short++] = g;
+    } else {
+      shorts[at_long++] = g;
+      RowRange& l = longs[n_long++];
+      l = {g, n_chunks, 0, 0};
+      for (int i = 0; i < t.n; i += kRecChunk)
+        chunks[n_chunks++] = {g, t.row0 + i, std::min(kRecChunk, t.n - i), l.n++};
+    }
+    if (t.n > 1 && m->tile_positions)
+      for (int i = 0; i < t.n; i += m->tile_positions)
+        tiles[n_tiles++] = {g, t.row0 + i, std::min(m->tile_positions, t.n - i), i / m->tile_positions};
     for (int i = 0; i < t.n; ++i) {
       const int64_t p = t.pos0 + i;
       ids[t.row0 + i] = t.tokens[i];
       pos[t.row0 + i] = (int32_t)p;
       slots[t.row0 + i] = t.blocks[p / HB_BLOCK_SIZE] * HB_BLOCK_SIZE + p % HB_BLOCK_SIZE;
       row_seg[t.row0 + i] = g;
-      attn_rows[t.row0 + i] = t.row0 + i;
+      row_list[t.n == 1 ? at_token++ : at_row++] = t.row0 + i;
     }
     const int64_t need = (t.pos0 + t.n - 1) / HB_BLOCK_SIZE + 1;
     int32_t* row = tables + (size_t)g * e->max_blocks_per_seq;
@@ -381,7 +479,6 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
   const uint32_t* ids = (const uint32_t*)(in + s.off_ids);
   const int32_t* pos = (const int32_t*)(in + s.off_pos);
   const int64_t* slots = (const int64_t*)(in + s.off_slots);
-  const int32_t* row_seg = (const int32_t*)(in + s.off_row_seg);
   const SegInfo* seg = (const SegInfo*)(in + s.off_seg);
   const int S = sp.streams;
   const int64_t W = sp.width, rows = s.rows;
@@ -409,23 +506,14 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
     const int64_t ldp = l.proj.N;
     float* y = m->y1;
     if (mx.has_attn) {
-      const AttentionSpec& as = mx.attn;
-      SpanAttention a;
-      a.q = at(m->proj, mx.aq.offset); a.ld_q = ldp;
-      a.out = m->attn; a.ld_out = l.attn_o.K;
-      a.kc = e->kc[l.kv_pool]; a.vc = e->vc[l.kv_pool];
-      a.tables = (const int32_t*)(in + s.off_tables);
-      a.max_blocks = e->max_blocks_per_seq; a.num_blocks = e->num_blocks;
-      a.row_seg = row_seg; a.pos = pos;
-      a.heads = as.heads; a.kv_heads = as.kv_heads; a.dim = as.dim; a.vdim = as.vdim;
-      a.window = as.window; a.keep_first = as.keep_first; a.scale = as.scale;
+      const SpanAttention a = span_args(e, i, s);
       prof_mark(e, kCatRopeKv);
       if ((rc = span_kv_write(st, a, at(m->proj, mx.ak.offset), at(m->proj, mx.av.offset), ldp, slots, rows, e->dtype))) return rc;
       prof_mark(e, kCatAttention);
-      if ((rc = span_attention_rows(st, a, (const int32_t*)(in + s.off_attn_rows), s.n_attn_rows, e->dtype))) return rc;
+      if ((rc = issue_attention(e, a, s))) return rc;
       prof_mark(e, kCatGemmO);
       if ((rc = gemm(pl ? &pl->attn_o : nullptr, i, y, m->attn, l.attn_o, true))) return rc;
-      e->last_launches += 2;
+      ++e->last_launches;  // the K/V write
       y = m->y2;
     }
     if (mx.has_rec) {
@@ -438,14 +526,14 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
       r.decay = l.decay; r.a2 = l.a2; r.a2_bias = l.a2_bias; r.rank = rs.rank; r.inv_tau = (float)(1.0 / rs.tau);
       r.state = l.state; r.o = m->o; r.ld_o = (int64_t)rs.heads * rs.vdim; r.segs = seg;
       prof_mark(e, kCatRecurrence);
-      if ((rc = recurrence_tokens(st, r, (const int32_t*)(in + s.off_short), s.n_short, e->dtype))) return rc;
+      if ((rc = issue_recurrence(e, r, s))) return rc;
       prof_mark(e, kCatNorm);
       const int groups = rs.norm_per_head ? rs.heads : 1, size = rs.norm_per_head ? rs.vdim : rs.heads * rs.vdim;
       if ((rc = gated_group_norm(st, m->rec, l.rec_o.K, m->o, r.ld_o, at(m->proj, mx.rg.offset), ldp, l.rec_norm, rows, groups,
                                  size, rs.gate_silu, sp.eps, e->dtype))) return rc;
       prof_mark(e, kCatGemmO);
       if ((rc = gemm(pl ? &pl->rec_o : nullptr, i, y, m->rec, l.rec_o, true))) return rc;
-      e->last_launches += 2;
+      ++e->last_launches;  // the gated norm
     }
     const bool both = mx.has_attn && mx.has_rec;
     const SublayerMix* next = lsp.ff ? &l.sub2 : (i + 1 < m->layers.size() ? &m->layers[i + 1].sub1 : nullptr);

@@ -123,10 +123,10 @@ struct LayeredStep {
   int n_chunks = 0;       // chunks of the longer segments (chunked recurrence kernels)
   int n_long = 0;         // longer segments
   int n_tiles = 0;        // query tiles of the tiled attention kernel
-  int n_attn_rows = 0;    // rows the per-token attention kernel takes
+  int n_token_rows = 0;   // rows that are single decoded tokens (first in the list of rows)
   bool decode = false;    // every segment is one token
   size_t off_ids = 0, off_pos = 0, off_slots = 0, off_row_seg = 0, off_want = 0, off_seg = 0, off_short = 0,
-         off_long = 0, off_chunk = 0, off_tile = 0, off_attn_rows = 0, off_tables = 0;
+         off_long = 0, off_chunk = 0, off_tile = 0, off_row_list = 0, off_tables = 0;
   LayeredPlans* plans = nullptr;
   TcGemmPlan* head_plan = nullptr;
 };
@@ -151,12 +151,11 @@ struct LayeredModel {
   float *y1 = nullptr, *y2 = nullptr;        // [rows, Hp] sublayer outputs
   void *gu = nullptr, *act = nullptr;        // feed-forward
   void* hf = nullptr;                        // [logits rows, Hp] final normed rows
-  float* cum = nullptr;                      // [rows, heads * dim] cumulative log decay inside a chunk
+  float* cum = nullptr;                      // [rows, heads * dim] running log2 decay inside a chunk
   float* chunk_state = nullptr;              // [chunks, heads, dim, vdim]
-  float* chunk_decay = nullptr;              // [chunks, heads * dim] log decay over a whole chunk
   float* attn_part = nullptr;                // split partials of the per-token attention
-  int max_segs = 0, max_chunks = 0, attn_splits_cap = 1;
-  size_t inputs_cap = 0;
+  int max_segs = 0, max_chunks = 0;
+  int tile_positions = 0;                    // positions of an attention tile that suit every layer (0: no tiles)
   std::map<int, LayeredPlans> plans;         // by rows bucket
   std::map<int, TcGemmPlan> head_plans;      // by wanted-rows bucket
   std::map<int, LayeredGraph> graphs;        // by number of decoded sequences

@@ -1,0 +1,135 @@
+// Public entry points of the layered models' mechanisms.
+#include "layered_ops.h"
+
+namespace hb {
+
+static SpanAttention span_of(const hb_span_attention_args* p) {
+  SpanAttention a;
+  a.q = p->q; a.ld_q = p->ld_q; a.out = p->out; a.ld_out = p->ld_out;
+  a.kc = p->k_cache; a.vc = p->v_cache;
+  a.tables = p->block_tables; a.max_blocks = p->max_blocks; a.num_blocks = p->num_blocks;
+  a.row_seg = p->row_segment; a.pos = p->positions;
+  a.heads = p->heads; a.kv_heads = p->kv_heads; a.dim = p->dim; a.vdim = p->vdim;
+  a.window = p->window; a.keep_first = p->keep_first; a.scale = p->scale;
+  return a;
+}
+
+static int check_span(const hb_span_attention_args* p) {
+  HB_CHECK_ARG(p && p->k_cache && p->v_cache, "span attention: null argument");
+  HB_CHECK_ARG(p->heads > 0 && p->kv_heads > 0 && p->heads % p->kv_heads == 0 && p->dim > 0 && p->vdim > 0,
+               "span attention: bad sizes");
+  HB_CHECK_ARG(p->window >= 0 && p->keep_first >= 0 && p->num_blocks > 0, "span attention: bad window or pool");
+  return HB_OK;
+}
+
+static Recurrence recurrence_of(const hb_linear_recurrence_args* p) {
+  Recurrence a;
+  a.p = p->p; a.ld = p->ld;
+  a.off_q = p->off_q; a.off_k = p->off_k; a.off_v = p->off_v; a.off_a1 = p->off_a1;
+  a.heads = p->heads; a.dim = p->dim; a.vdim = p->vdim;
+  a.q_scale = p->q_scale; a.silu_qkv = p->silu_qkv;
+  a.decay = p->decay; a.a2 = p->a2; a.a2_bias = p->a2_bias;
+  a.rank = p->decay ? 0 : p->rank;
+  a.inv_tau = p->decay ? 1.f : (float)(1.0 / p->tau);
+  a.state = p->state; a.o = p->o; a.ld_o = p->ld_o;
+  a.segs = (const SegInfo*)p->segments;
+  return a;
+}
+
+}  // namespace hb
+
+extern "C" {
+
+int hb_span_attention_tile_positions(const hb_span_attention_args* a, hb_dtype dtype) {
+  int rc = hb::check_span(a);
+  return rc ? rc : hb::span_attention_tile_positions(hb::span_of(a), dtype);
+}
+
+int hb_span_attention(void* stream, const hb_span_attention_args* p, const int32_t* tiles, int n_tiles, const int32_t* rows,
+                      int n_rows, int n_splits, float* workspace, hb_dtype dtype) {
+  int rc = hb::check_span(p);
+  if (rc) return rc;
+  HB_CHECK_ARG(p->q && p->out && p->block_tables && p->row_segment && p->positions && p->max_blocks > 0,
+               "hb_span_attention: null argument");
+  HB_CHECK_ARG((tiles || n_tiles == 0) && (rows || n_rows == 0) && n_tiles >= 0 && n_rows >= 0, "hb_span_attention: bad lists");
+  HB_CHECK_ARG(n_splits >= 1 && n_splits <= 64 && (n_splits == 1 || workspace), "hb_span_attention: bad splits");
+  const hb::SpanAttention a = hb::span_of(p);
+  auto st = (cudaStream_t)stream;
+  if (n_tiles) {
+    HB_CHECK_ARG(hb::span_attention_tile_positions(a, dtype) > 0, "hb_span_attention: these sizes do not go as tiles");
+    if ((rc = hb::span_attention_tiles(st, a, (const hb::RowRange*)tiles, n_tiles))) return rc;
+  }
+  if (hb::span_attention_tokens_supported(a, dtype)) return hb::span_attention_tokens(st, a, rows, n_rows, n_splits, workspace);
+  return hb::span_attention_rows(st, a, rows, n_rows, dtype);
+}
+
+int hb_span_kv_write(void* stream, const hb_span_attention_args* p, const void* k, const void* v, int64_t ld,
+                     const int64_t* slots, int64_t rows, hb_dtype dtype) {
+  int rc = hb::check_span(p);
+  if (rc) return rc;
+  HB_CHECK_ARG(k && v && slots && rows >= 0, "hb_span_kv_write: null argument");
+  return rows ? hb::span_kv_write((cudaStream_t)stream, hb::span_of(p), k, v, ld, slots, rows, dtype) : HB_OK;
+}
+
+int hb_linear_recurrence_chunked(const hb_linear_recurrence_args* a, hb_dtype dtype) {
+  HB_CHECK_ARG(a, "hb_linear_recurrence_chunked: null argument");
+  return hb::recurrence_chunks_supported(hb::recurrence_of(a), dtype) ? 1 : 0;
+}
+
+int hb_linear_recurrence(void* stream, const hb_linear_recurrence_args* p, const int32_t* list, int n_list,
+                         const int32_t* chunks, int n_chunks, const int32_t* long_segments, int n_long, float* cum,
+                         float* chunk_state, hb_dtype dtype) {
+  HB_CHECK_ARG(p && p->p && p->state && p->o && p->segments, "hb_linear_recurrence: null argument");
+  HB_CHECK_ARG(p->heads > 0 && p->dim > 0 && p->vdim > 0, "hb_linear_recurrence: bad sizes");
+  HB_CHECK_ARG(p->decay || (p->a2 && p->a2_bias && p->rank > 0 && p->tau > 0.f), "hb_linear_recurrence: no decay");
+  const hb::Recurrence a = hb::recurrence_of(p);
+  auto st = (cudaStream_t)stream;
+  int rc = hb::recurrence_tokens(st, a, list, n_list, dtype);
+  if (rc || n_chunks == 0) return rc;
+  HB_CHECK_ARG(chunks && long_segments && n_long > 0 && chunk_state && (p->decay || cum), "hb_linear_recurrence: bad chunk lists");
+  HB_CHECK_ARG(hb::recurrence_chunks_supported(a, dtype), "hb_linear_recurrence: these sizes do not go in chunks");
+  hb::RecurrenceChunks c;
+  c.chunks = (const hb::RowRange*)chunks; c.n_chunks = n_chunks;
+  c.segs = (const hb::RowRange*)long_segments; c.n_segs = n_long;
+  c.cum = cum; c.state = chunk_state;
+  int64_t launches = 0;
+  return hb::recurrence_chunks(st, a, c, &launches);
+}
+
+int hb_streams_embed(void* stream, float* x, void* h, const void* embed, const void* pos_table, const uint32_t* ids,
+                     const int32_t* positions, const float* in, const float* norm, int64_t rows, int streams, int64_t width,
+                     int64_t ld_h, int64_t vocab, int64_t max_positions, float eps, hb_dtype dtype) {
+  HB_CHECK_ARG(x && h && embed && pos_table && ids && positions && in && norm, "hb_streams_embed: null argument");
+  HB_CHECK_ARG(rows >= 0 && streams > 0 && width > 0 && vocab > 0 && max_positions > 0, "hb_streams_embed: bad shape");
+  if (rows == 0) return HB_OK;
+  return hb::streams_embed((cudaStream_t)stream, x, h, embed, pos_table, ids, positions, in, norm, rows, streams, width, ld_h,
+                           vocab, max_positions, eps, dtype);
+}
+
+int hb_streams_mix(void* stream, float* x, void* h, const float* y, const float* y2, int64_t ld_y, const float* mix,
+                   const float* out, const float* next_in, const float* next_norm, const float* w1, const float* w2,
+                   int64_t rows, int streams, int64_t width, int64_t ld_h, float eps, hb_dtype dtype) {
+  HB_CHECK_ARG(x && y && mix && out && (!next_norm || (next_in && h)) && (!y2 || (w1 && w2)), "hb_streams_mix: null argument");
+  HB_CHECK_ARG(rows >= 0 && width > 0, "hb_streams_mix: bad shape");
+  if (rows == 0) return HB_OK;
+  hb::StreamMix m;
+  m.mix = mix; m.out = out; m.next_in = next_in; m.next_norm = next_norm; m.w1 = w1; m.w2 = w2;
+  return hb::streams_mix((cudaStream_t)stream, x, h, y, y2, ld_y, m, rows, streams, width, ld_h, eps, dtype);
+}
+
+int hb_streams_final(void* stream, void* h, const float* x, const int32_t* want, const float* norm, int64_t n_want,
+                     int streams, int64_t width, int64_t ld_h, float eps, hb_dtype dtype) {
+  HB_CHECK_ARG(h && x && want && norm && streams > 0 && width > 0, "hb_streams_final: bad argument");
+  return hb::streams_final((cudaStream_t)stream, h, x, want, norm, n_want, streams, width, ld_h, eps, dtype);
+}
+
+int hb_gated_group_norm(void* stream, void* out, int64_t ld_out, const float* o, int64_t ld_o, const void* gate,
+                        int64_t ld_gate, const float* weight, int64_t rows, int groups, int size, int gate_silu, float eps,
+                        hb_dtype dtype) {
+  HB_CHECK_ARG(out && o && gate && weight && groups > 0 && size > 0 && rows >= 0, "hb_gated_group_norm: bad argument");
+  if (rows == 0) return HB_OK;
+  return hb::gated_group_norm((cudaStream_t)stream, out, ld_out, o, ld_o, gate, ld_gate, weight, rows, groups, size,
+                              gate_silu != 0, eps, dtype);
+}
+
+}  // extern "C"

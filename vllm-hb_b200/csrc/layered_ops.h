@@ -67,6 +67,15 @@ int span_kv_write(cudaStream_t st, const SpanAttention& a, const void* k, const 
 // One CTA per (row of `row_list`, kv head): any dtype and any sizes.
 int span_attention_rows(cudaStream_t st, const SpanAttention& a, const int32_t* row_list, int n_rows, hb_dtype dtype);
 
+// Tensor-core forms (attention_span_mma.cu): prompt portions as tiles of up to
+// span_attention_tile_positions() consecutive positions (0: these sizes are not taken) and decoded
+// tokens as single rows, their keys split over n_splits CTAs when the rows alone leave SMs idle
+// (`part`: n_rows * heads * n_splits * (vdim + 2) floats).
+int span_attention_tile_positions(const SpanAttention& a, hb_dtype dtype);
+bool span_attention_tokens_supported(const SpanAttention& a, hb_dtype dtype);
+int span_attention_tiles(cudaStream_t st, const SpanAttention& a, const RowRange* tiles, int n_tiles);
+int span_attention_tokens(cudaStream_t st, const SpanAttention& a, const int32_t* rows, int n_rows, int n_splits, float* part);
+
 // ------------------------------------------------------------ linear recurrence (recurrence.cu)
 struct Recurrence {
   const void* p = nullptr;     // projection rows: q, k, v (and the low-rank decay input) at offsets
@@ -88,5 +97,20 @@ struct Recurrence {
 // Token by token, state in and out of HBM once per segment where it fits the registers:
 // decoded tokens and short portions.  `list` holds segment numbers.
 int recurrence_tokens(cudaStream_t st, const Recurrence& a, const int32_t* list, int n_list, hb_dtype dtype);
+
+// Prompt portions in chunks of kRecChunk tokens on tensor cores (recurrence_chunk.cu, bf16
+// projections): every chunk's own contribution to the state, a scan over the chunks of a segment,
+// every chunk's outputs.  Chunks of a segment are neighbours in `chunks`.
+constexpr int kRecChunk = 64;
+struct RecurrenceChunks {
+  const RowRange* chunks = nullptr;   // device
+  int n_chunks = 0;
+  const RowRange* segs = nullptr;     // longer segments: seg, first chunk (row0), number of chunks (n)
+  int n_segs = 0;
+  float* cum = nullptr;               // [rows, heads * dim] running log2 decay inside a chunk
+  float* state = nullptr;             // [n_chunks, heads, dim, vdim]
+};
+bool recurrence_chunks_supported(const Recurrence& a, hb_dtype dtype);
+int recurrence_chunks(cudaStream_t st, const Recurrence& a, const RecurrenceChunks& c, int64_t* launches);
 
 }  // namespace hb

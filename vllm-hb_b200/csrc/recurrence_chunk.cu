@@ -1,0 +1,443 @@
+// Chunked form of the linear recurrence (see recurrence.cu) for prompt portions.
+//
+// With b_i the running sum of log2 decays inside a chunk of C = 64 tokens (per key channel, fp32),
+//   o_i   = (q_i 2^b_i)^T S_0 + sum_{j <= i} [sum_d q_i[d] k_j[d] 2^(b_i[d] - b_j[d])] v_j
+//   S_end = diag(2^b_end) S_0 + sum_j (k_j 2^(b_end - b_j)) v_j^T
+// where S_0 is the state before the chunk.  All exponents that are formed are <= 0: keys are
+// scaled to the end of their own 16-token block, queries from there on, and inside a block the
+// difference b_i - b_j is formed per pair, so that any decay (0 and 1 included) is safe.
+//
+// Products run on tensor cores with both operands as pairs of bf16 numbers (hi + lo), which keeps
+// fp32-like precision; sums, decays and states are fp32.
+//
+//   decay   running log2 decays of a chunk (low-rank decay only)
+//   state   per (chunk, head, 64 state columns): the chunk's own contribution to the state
+//   scan    per element of the state: over the chunks of a segment, contribution -> state before
+//   output  per (chunk, head): scores, outputs
+#include <algorithm>
+
+#include "layered_ops.h"
+#include "mma_sync.cuh"
+#include "tc_core.cuh"
+
+namespace hb {
+
+namespace {
+constexpr int kC = kRecChunk;
+constexpr int kT = 128;        // threads: four warps of 16 tokens
+constexpr int kVT = 64;        // state columns of a tile
+constexpr int kVS = kVT + 8;   // padded row of a bf16 tile
+constexpr float kLog2e = 1.4426950408889634f;
+using bf16 = __nv_bfloat16;
+
+__device__ __forceinline__ float rec_silu(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float log2_sigmoid(float z) { return (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * kLog2e; }
+__device__ __forceinline__ float ld_proj(const Recurrence& a, int64_t row, int col) {
+  return __bfloat162float(((const bf16*)a.p)[row * a.ld + col]);
+}
+// log2 of a constant decay to the power n (n = 0: exactly 0, also for decay 0)
+__device__ __forceinline__ float log2_pow(float log2_decay, int n) { return n == 0 ? 0.f : log2_decay * (float)n; }
+__device__ __forceinline__ int pad16d(int n) { return (n + 15) / 16 * 16; }
+__device__ __forceinline__ void put_split(bf16* hi, bf16* lo, float x) {
+  const bf16 h = __float2bfloat16_rn(x);
+  *hi = h;
+  *lo = __float2bfloat16_rn(x - __bfloat162float(h));
+}
+}  // namespace
+
+__global__ void __launch_bounds__(256)
+recurrence_decay_kernel(const Recurrence a, const RowRange* __restrict__ chunks, float* __restrict__ cum) {
+  extern __shared__ float s_t[];  // [64][rank]
+  pdl_trigger();
+  pdl_grid_wait();
+  const RowRange ch = chunks[blockIdx.x];
+  for (int i = threadIdx.x; i < ch.n * a.rank; i += blockDim.x)
+    s_t[i] = ld_proj(a, ch.row0 + i / a.rank, a.off_a1 + i % a.rank);
+  __syncthreads();
+  const int hd = a.heads * a.dim, c = blockIdx.y * blockDim.x + threadIdx.x;
+  if (c >= hd) return;
+  const float* w = a.a2 + (int64_t)c * a.rank;
+  const float bias = a.a2_bias[c];
+  float b = 0.f;
+  if (a.rank == 16) {
+    float wr[16];
+#pragma unroll
+    for (int r = 0; r < 16; ++r) wr[r] = w[r];
+    for (int i = 0; i < ch.n; ++i) {
+      float z = bias;
+#pragma unroll
+      for (int r = 0; r < 16; ++r) z = fmaf(wr[r], s_t[i * 16 + r], z);
+      b = fmaf(log2_sigmoid(z), a.inv_tau, b);
+      cum[(int64_t)(ch.row0 + i) * hd + c] = b;
+    }
+  } else {
+    for (int i = 0; i < ch.n; ++i) {
+      float z = bias;
+      for (int r = 0; r < a.rank; ++r) z = fmaf(w[r], s_t[i * a.rank + r], z);
+      b = fmaf(log2_sigmoid(z), a.inv_tau, b);
+      cum[(int64_t)(ch.row0 + i) * hd + c] = b;
+    }
+  }
+}
+
+// Value tile [64 tokens][64 columns] as hi/lo pairs; rows and columns outside are zero.
+__device__ __forceinline__ void load_values(const Recurrence& a, const RowRange& ch, int h, int v0, bf16* hi, bf16* lo) {
+  for (int i = threadIdx.x; i < kC * kVT; i += kT) {
+    const int j = i / kVT, c = i % kVT;
+    float v = 0.f;
+    if (j < ch.n && v0 + c < a.vdim) {
+      v = ld_proj(a, ch.row0 + j, a.off_v + h * a.vdim + v0 + c);
+      if (a.silu_qkv) v = rec_silu(v);
+    }
+    put_split(hi + j * kVS + c, lo + j * kVS + c, v);
+  }
+}
+
+__global__ void __launch_bounds__(kT)
+recurrence_state_kernel(const Recurrence a, const RowRange* __restrict__ chunks, const float* __restrict__ cum,
+                        float* __restrict__ out) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  const int D = a.dim, DP = pad16d(D), KS = DP + 8, h = blockIdx.y, v0 = blockIdx.z * kVT;
+  bf16* k_hi = (bf16*)smem;
+  bf16* k_lo = k_hi + kC * KS;
+  bf16* v_hi = k_lo + kC * KS;
+  bf16* v_lo = v_hi + kC * kVS;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  pdl_grid_wait();
+  const RowRange ch = chunks[blockIdx.x];
+  const int hd = a.heads * D;
+  const float ld2 = a.decay ? log2f(a.decay[h]) : 0.f;
+  for (int i = tid; i < kC * DP; i += kT) {
+    const int j = i / DP, d = i % DP;
+    float k = 0.f;
+    if (j < ch.n && d < D) {
+      k = ld_proj(a, ch.row0 + j, a.off_k + h * D + d);
+      if (a.silu_qkv) k = rec_silu(k);
+      const float e = a.decay ? log2_pow(ld2, ch.n - 1 - j)
+                              : cum[(int64_t)(ch.row0 + ch.n - 1) * hd + h * D + d] - cum[(int64_t)(ch.row0 + j) * hd + h * D + d];
+      k *= exp2f(e);
+    }
+    put_split(k_hi + j * KS + d, k_lo + j * KS + d, k);
+  }
+  load_values(a, ch, h, v0, v_hi, v_lo);
+  __syncthreads();
+  float* o = out + ((int64_t)blockIdx.x * a.heads + h) * D * a.vdim + v0;
+  // A = (scaled keys)^T: stored [token][channel], read transposed.  Matrices of the x4 load: channels
+  // 0-7 / 8-15 of tokens 0-7, then of tokens 8-15.
+  const uint32_t ah = smem_u32(k_hi + ((lane & 7) + (lane >> 4) * 8) * KS + ((lane >> 3) & 1) * 8);
+  const uint32_t al = smem_u32(k_lo + ((lane & 7) + (lane >> 4) * 8) * KS + ((lane >> 3) & 1) * 8);
+  const uint32_t bh = smem_u32(v_hi + (lane & 15) * kVS + (lane >> 4) * 8);
+  const uint32_t bl = smem_u32(v_lo + (lane & 15) * kVS + (lane >> 4) * 8);
+  for (int mt = warp; mt < DP / 16; mt += kT / 32) {
+    float acc[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+#pragma unroll
+    for (int ks = 0; ks < kC / 16; ++ks) {
+      uint32_t hi[4], lo[4];
+      ldsm_x4_trans(ah + (ks * 16 * KS + mt * 16) * 2, hi[0], hi[1], hi[2], hi[3]);
+      ldsm_x4_trans(al + (ks * 16 * KS + mt * 16) * 2, lo[0], lo[1], lo[2], lo[3]);
+#pragma unroll
+      for (int nv = 0; nv < 4; ++nv) {
+        uint32_t b[4], c[4];
+        ldsm_x4_trans(bh + (ks * 16 * kVS + nv * 16) * 2, b[0], b[1], b[2], b[3]);
+        ldsm_x4_trans(bl + (ks * 16 * kVS + nv * 16) * 2, c[0], c[1], c[2], c[3]);
+        mma_split(acc[2 * nv], hi, lo, b[0], b[1], c[0], c[1]);
+        mma_split(acc[2 * nv + 1], hi, lo, b[2], b[3], c[2], c[3]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int d = mt * 16 + g + (e >> 1) * 8, c = i * 8 + 2 * t + (e & 1);
+        if (d < D && v0 + c < a.vdim) o[(int64_t)d * a.vdim + c] = acc[i][e];
+      }
+  }
+}
+
+// One thread per VEC neighbouring state elements.
+template <int VEC>
+__global__ void __launch_bounds__(256)
+recurrence_scan_kernel(const Recurrence a, const RowRange* __restrict__ segs, const RowRange* __restrict__ chunks,
+                       const float* __restrict__ cum, float* __restrict__ chunk_state) {
+  pdl_grid_wait();
+  const int64_t per_head = (int64_t)a.dim * a.vdim;
+  const int64_t i = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+  if (i >= per_head) return;
+  const int h = blockIdx.y, d = (int)(i / a.vdim), hd = a.heads * a.dim;
+  const RowRange sg = segs[blockIdx.z];
+  const SegInfo info = a.segs[sg.seg];
+  float* state = a.state + ((int64_t)info.slot * a.heads + h) * per_head + i;
+  const float ld2 = a.decay ? log2f(a.decay[h]) : 0.f;
+  float s[VEC];
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) s[j] = info.pos0 > 0 ? state[j] : 0.f;  // a new sequence starts from zero
+  for (int c = 0; c < sg.n; ++c) {
+    float* u = chunk_state + ((int64_t)(sg.row0 + c) * a.heads + h) * per_head + i;
+    const RowRange ch = chunks[sg.row0 + c];
+    const float f = exp2f(a.decay ? log2_pow(ld2, ch.n) : cum[(int64_t)(ch.row0 + ch.n - 1) * hd + h * a.dim + d]);
+    float v[VEC];
+    if (VEC == 4) {
+      const float4 x = *reinterpret_cast<const float4*>(u);
+      v[0] = x.x; v[1 % VEC] = x.y; v[2 % VEC] = x.z; v[3 % VEC] = x.w;
+      *reinterpret_cast<float4*>(u) = make_float4(s[0], s[1 % VEC], s[2 % VEC], s[3 % VEC]);
+    } else {
+      v[0] = *u;
+      *u = s[0];
+    }
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) s[j] = fmaf(f, s[j], v[j]);
+  }
+  pdl_trigger();
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) state[j] = s[j];
+}
+
+// LR: low-rank decay (q and k are exact bf16, decays per channel); else a constant decay per head.
+template <bool LR>
+__global__ void __launch_bounds__(kT)
+recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks, const float* __restrict__ cum,
+                         const float* __restrict__ chunk_state) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  const int D = a.dim, DP = pad16d(D), KS = DP + 8, BS = DP + 4, h = blockIdx.y;
+  // LR: q | b | k | scaled k (hi, lo);  constant: q (hi, lo) | k (hi, lo).  The keys' part is reused by
+  // the value and state tiles of the second phase.
+  bf16* q_hi = (bf16*)smem;                       // [64][KS]
+  bf16* q_lo = q_hi + kC * KS;                    // constant decay only
+  float* s_b = (float*)(q_hi + kC * KS);          // LR only: [64][BS]
+  uint8_t* keys = LR ? (uint8_t*)(s_b + kC * BS) : (uint8_t*)(q_lo + kC * KS);
+  bf16* k_raw = (bf16*)keys;                      // LR only
+  bf16* k_hi = LR ? k_raw + kC * KS : (bf16*)keys;
+  bf16* k_lo = k_hi + kC * KS;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  pdl_grid_wait();
+  const RowRange ch = chunks[blockIdx.x];
+  const int hd = a.heads * D;
+  const float ld2 = LR ? 0.f : log2f(a.decay[h]);
+  if (LR) {
+    for (int i = tid; i < kC * DP; i += kT) {
+      const int j = i / DP, d = i % DP;
+      // tokens past the end keep the last decay: every exponent stays <= 0
+      s_b[j * BS + d] = d < D ? cum[(int64_t)(ch.row0 + min(j, ch.n - 1)) * hd + h * D + d] : 0.f;
+    }
+    __syncthreads();
+  }
+  for (int i = tid; i < kC * DP; i += kT) {
+    const int j = i / DP, d = i % DP;
+    float q = 0.f, k = 0.f;
+    if (j < ch.n && d < D) {
+      q = ld_proj(a, ch.row0 + j, a.off_q + h * D + d);
+      k = ld_proj(a, ch.row0 + j, a.off_k + h * D + d);
+      if (a.silu_qkv) { q = rec_silu(q); k = rec_silu(k); }
+    }
+    if (LR) {
+      q_hi[j * KS + d] = __float2bfloat16_rn(q);   // exact; the scale is applied to the results
+      k_raw[j * KS + d] = __float2bfloat16_rn(k);
+      put_split(k_hi + j * KS + d, k_lo + j * KS + d, k * exp2f(s_b[(j | 15) * BS + d] - s_b[j * BS + d]));
+    } else {
+      put_split(q_hi + j * KS + d, q_lo + j * KS + d, q);
+      put_split(k_hi + j * KS + d, k_lo + j * KS + d, k);
+    }
+  }
+  __syncthreads();
+
+  // ---- scores of this warp's 16 tokens with all tokens up to them: s[n] = keys 8n .. 8n+7
+  float s[8][4];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+  const int i0 = warp * 16 + g, i1 = i0 + 8;
+  const uint32_t kh = smem_u32(k_hi + ((lane & 7) + (lane >> 4) * 8) * KS + ((lane >> 3) & 1) * 8);
+  const uint32_t kl = smem_u32(k_lo + ((lane & 7) + (lane >> 4) * 8) * KS + ((lane >> 3) & 1) * 8);
+  const uint32_t qh = smem_u32(q_hi + (warp * 16 + (lane & 15)) * KS + (lane >> 4) * 8);
+  const uint32_t ql = smem_u32(q_lo + (warp * 16 + (lane & 15)) * KS + (lane >> 4) * 8);
+  // query fragment of one 16-channel step, scaled by 2^(b_i - e) with e the reference of the key
+  // block (ref < 0: the start of the chunk, e = 0)
+  auto q_frag = [&](int ks, int ref, uint32_t (&hi)[4], uint32_t (&lo)[4]) {
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int d = ks * 16 + half * 8 + 2 * t;
+      const float e0 = ref < 0 ? 0.f : s_b[ref * BS + d], e1 = ref < 0 ? 0.f : s_b[ref * BS + d + 1];
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int i = r ? i1 : i0;
+        const __nv_bfloat162 q2 = *reinterpret_cast<const __nv_bfloat162*>(q_hi + i * KS + d);
+        split_bf16(__low2float(q2) * exp2f(s_b[i * BS + d] - e0), __high2float(q2) * exp2f(s_b[i * BS + d + 1] - e1),
+                   hi[half * 2 + r], lo[half * 2 + r]);
+      }
+    }
+  };
+#pragma unroll
+  for (int nb = 0; nb < 4; ++nb) {   // blocks of 16 keys
+    if (LR ? nb < warp : nb <= warp) {
+      for (int ks = 0; ks < DP / 16; ++ks) {
+        uint32_t hi[4], lo[4], b[4], c[4];
+        if (LR) {
+          q_frag(ks, nb * 16 + 15, hi, lo);
+        } else {
+          ldsm_x4(qh + ks * 32, hi[0], hi[1], hi[2], hi[3]);
+          ldsm_x4(ql + ks * 32, lo[0], lo[1], lo[2], lo[3]);
+        }
+        ldsm_x4(kh + (nb * 16 * KS + ks * 16) * 2, b[0], b[1], b[2], b[3]);
+        ldsm_x4(kl + (nb * 16 * KS + ks * 16) * 2, c[0], c[1], c[2], c[3]);
+        mma_split(s[2 * nb], hi, lo, b[0], b[1], c[0], c[1]);
+        mma_split(s[2 * nb + 1], hi, lo, b[2], b[3], c[2], c[3]);
+      }
+    }
+    if (LR && nb == warp) {
+      // inside the block the decay differs per pair: fp32 on CUDA cores.  Keys 8-15 of the block never
+      // meet queries 0-7.
+      float p[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) p[e] = 0.f;
+      const int j0 = warp * 16 + 2 * t;
+      for (int d = 0; d < D; ++d) {
+        const float b0 = s_b[i0 * BS + d], b1 = s_b[i1 * BS + d];
+        const float q0 = __bfloat162float(q_hi[i0 * KS + d]), q1 = __bfloat162float(q_hi[i1 * KS + d]);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float kj = __bfloat162float(k_raw[(j0 + e) * KS + d]), bj = s_b[(j0 + e) * BS + d];
+          const float kj8 = __bfloat162float(k_raw[(j0 + 8 + e) * KS + d]), bj8 = s_b[(j0 + 8 + e) * BS + d];
+          p[e] = fmaf(q0 * kj, exp2f(fminf(b0 - bj, 0.f)), p[e]);
+          p[2 + e] = fmaf(q1 * kj, exp2f(fminf(b1 - bj, 0.f)), p[2 + e]);
+          p[6 + e] = fmaf(q1 * kj8, exp2f(fminf(b1 - bj8, 0.f)), p[6 + e]);
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { s[2 * nb][e] = p[e]; s[2 * nb + 1][e] = p[4 + e]; }
+    }
+  }
+#pragma unroll
+  for (int n = 0; n < 8; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int i = e < 2 ? i0 : i1, j = n * 8 + 2 * t + (e & 1);
+      if (j > i) s[n][e] = 0.f;
+      else if (!LR) s[n][e] *= exp2f(log2_pow(ld2, i - j));
+    }
+  __syncthreads();  // keys are done with: their memory holds the tiles of phase two
+
+  bf16* v_hi = (bf16*)keys;            // [64][kVS] values
+  bf16* v_lo = v_hi + kC * kVS;
+  bf16* t_hi = v_lo + kC * kVS;        // [64][kVS] 64 channels of the state before the chunk
+  bf16* t_lo = t_hi + kC * kVS;
+  const uint32_t vh = smem_u32(v_hi + (lane & 15) * kVS + (lane >> 4) * 8), vl = smem_u32(v_lo + (lane & 15) * kVS + (lane >> 4) * 8);
+  const uint32_t th = smem_u32(t_hi + (lane & 15) * kVS + (lane >> 4) * 8), tl = smem_u32(t_lo + (lane & 15) * kVS + (lane >> 4) * 8);
+  const float f0 = LR ? 1.f : exp2f(log2_pow(ld2, i0 + 1)), f1 = LR ? 1.f : exp2f(log2_pow(ld2, i1 + 1));
+  const float* st = chunk_state + ((int64_t)blockIdx.x * a.heads + h) * D * a.vdim;
+  const bool live = warp * 16 < ch.n;
+  for (int v0 = 0; v0 < a.vdim; v0 += kVT) {
+    float o[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    for (int d0 = 0; d0 < DP; d0 += 64) {
+      for (int i = tid; i < 64 * kVT; i += kT) {
+        const int d = d0 + i / kVT, c = i % kVT;
+        const float x = d < D && v0 + c < a.vdim ? st[(int64_t)d * a.vdim + v0 + c] : 0.f;
+        put_split(t_hi + i / kVT * kVS + c, t_lo + i / kVT * kVS + c, x);
+      }
+      if (d0 == 0) load_values(a, ch, h, v0, v_hi, v_lo);
+      __syncthreads();
+      if (live) {
+        const int n_ks = min(4, (DP - d0) / 16);
+        for (int ks = 0; ks < n_ks; ++ks) {
+          uint32_t hi[4], lo[4];
+          if (LR) {
+            q_frag(d0 / 16 + ks, -1, hi, lo);
+          } else {
+            ldsm_x4(qh + (d0 / 16 + ks) * 32, hi[0], hi[1], hi[2], hi[3]);
+            ldsm_x4(ql + (d0 / 16 + ks) * 32, lo[0], lo[1], lo[2], lo[3]);
+          }
+#pragma unroll
+          for (int nv = 0; nv < 4; ++nv) {
+            uint32_t b[4], c[4];
+            ldsm_x4_trans(th + (ks * 16 * kVS + nv * 16) * 2, b[0], b[1], b[2], b[3]);
+            ldsm_x4_trans(tl + (ks * 16 * kVS + nv * 16) * 2, c[0], c[1], c[2], c[3]);
+            mma_split(o[2 * nv], hi, lo, b[0], b[1], c[0], c[1]);
+            mma_split(o[2 * nv + 1], hi, lo, b[2], b[3], c[2], c[3]);
+          }
+        }
+      }
+      if (d0 + 64 < DP) __syncthreads();  // the state tile is refilled
+    }
+    if (live) {
+      if (!LR) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) { o[i][0] *= f0; o[i][1] *= f0; o[i][2] *= f1; o[i][3] *= f1; }
+      }
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk) {
+        if (kk <= warp) {
+          uint32_t hi[4], lo[4];
+          split_bf16(s[2 * kk][0], s[2 * kk][1], hi[0], lo[0]);
+          split_bf16(s[2 * kk][2], s[2 * kk][3], hi[1], lo[1]);
+          split_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1], hi[2], lo[2]);
+          split_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3], hi[3], lo[3]);
+#pragma unroll
+          for (int nv = 0; nv < 4; ++nv) {
+            uint32_t b[4], c[4];
+            ldsm_x4_trans(vh + (kk * 16 * kVS + nv * 16) * 2, b[0], b[1], b[2], b[3]);
+            ldsm_x4_trans(vl + (kk * 16 * kVS + nv * 16) * 2, c[0], c[1], c[2], c[3]);
+            mma_split(o[2 * nv], hi, lo, b[0], b[1], c[0], c[1]);
+            mma_split(o[2 * nv + 1], hi, lo, b[2], b[3], c[2], c[3]);
+          }
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int r = e < 2 ? i0 : i1, c = i * 8 + 2 * t + (e & 1);
+          if (r < ch.n && v0 + c < a.vdim)
+            a.o[(int64_t)(ch.row0 + r) * a.ld_o + (int64_t)h * a.vdim + v0 + c] = o[i][e] * a.q_scale;
+        }
+    }
+    __syncthreads();
+  }
+  pdl_trigger();
+}
+
+static int pad16h(int n) { return (n + 15) / 16 * 16; }
+static size_t state_smem(const Recurrence& a) { return (size_t)2 * kC * (pad16h(a.dim) + 8 + kVS) * 2; }
+static size_t output_smem(const Recurrence& a) {
+  const size_t ks = (size_t)kC * (pad16h(a.dim) + 8) * 2, tiles = (size_t)4 * kC * kVS * 2;
+  return a.decay ? 2 * ks + std::max(2 * ks, tiles)
+                 : ks + (size_t)kC * (pad16h(a.dim) + 4) * 4 + std::max(3 * ks, tiles);
+}
+
+bool recurrence_chunks_supported(const Recurrence& a, hb_dtype dtype) {
+  static const bool off = [] { const char* e = getenv("HB_RECURRENCE"); return e && e[0] == 't'; }();
+  return !off && dtype == HB_BF16 && output_smem(a) <= 224 * 1024 && state_smem(a) <= 224 * 1024 &&
+         (size_t)kC * a.rank * 4 <= 48 * 1024;
+}
+
+int recurrence_chunks(cudaStream_t st, const Recurrence& a, const RecurrenceChunks& c, int64_t* launches) {
+  if (c.n_chunks == 0) return HB_OK;
+  const unsigned nc = (unsigned)c.n_chunks, H = (unsigned)a.heads;
+  auto opt_in = [](auto* k, size_t smem) -> int {
+    if (smem > 48 * 1024) HB_CUDA_CHECK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024));
+    return HB_OK;
+  };
+  int rc;
+  if (!a.decay) {
+    HB_CUDA_CHECK(launch_pdl(recurrence_decay_kernel, dim3(nc, (unsigned)((a.heads * a.dim + 255) / 256)), dim3(256),
+                             (size_t)kC * a.rank * 4, st, a, c.chunks, c.cum));
+    ++*launches;
+  }
+  const size_t ss = state_smem(a), os = output_smem(a);
+  if ((rc = opt_in(recurrence_state_kernel, ss))) return rc;
+  HB_CUDA_CHECK(launch_pdl(recurrence_state_kernel, dim3(nc, H, (unsigned)((a.vdim + kVT - 1) / kVT)), dim3(kT), ss, st, a,
+                           c.chunks, (const float*)c.cum, c.state));
+  const int64_t per_head = (int64_t)a.dim * a.vdim;
+  const int vec = a.vdim % 4 == 0 ? 4 : 1;
+  auto* scan = vec == 4 ? recurrence_scan_kernel<4> : recurrence_scan_kernel<1>;
+  HB_CUDA_CHECK(launch_pdl(scan, dim3((unsigned)((per_head / vec + 255) / 256), H, (unsigned)c.n_segs), dim3(256), 0, st, a,
+                           c.segs, c.chunks, (const float*)c.cum, c.state));
+  auto* out = a.decay ? recurrence_output_kernel<false> : recurrence_output_kernel<true>;
+  if ((rc = opt_in(out, os))) return rc;
+  HB_CUDA_CHECK(launch_pdl(out, dim3(nc, H), dim3(kT), os, st, a, c.chunks, (const float*)c.cum, (const float*)c.state));
+  *launches += 3;
+  return HB_OK;
+}
+
+}  // namespace hb
