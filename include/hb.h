@@ -651,6 +651,9 @@ int hb_kv_swap_blocks(hb_engine* e, const int64_t* pairs, size_t n_pairs, int to
 #define HB_PROFILE_KINDS 11
 int hb_engine_profile_step(hb_engine* e, hb_seq* const* seqs, size_t B,
                            const uint32_t* last_tokens, uint32_t* next_tokens, float* ms_by_kind);
+/* The same for every step while on (hb_step, hb_forward, ...): the times of the last step. */
+int hb_engine_set_profiling(hb_engine* e, int on);
+int hb_engine_profile_ms(const hb_engine* e, float* ms_by_kind);
 /* Algorithmic bytes all GEMM launches of one decode step move for batch B on this rank
  * (weights + activations in + results out). */
 double hb_engine_gemm_bytes(const hb_engine* e, int64_t B);

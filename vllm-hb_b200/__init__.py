@@ -201,6 +201,8 @@ _SIGS = {
     "hb_step": (_i, [_vp, _vp, _sz, _vp, _vp]),
     "hb_engine_sample": (_i, [_vp, _sz, _vp, _f, _f, _vp]),
     "hb_engine_num_free_state_slots": (_i, [_vp]),
+    "hb_engine_set_profiling": (_i, [_vp, _i]),
+    "hb_engine_profile_ms": (_i, [_vp, _vp]),
     "hb_engine_free": (_i, [_vp]),
     "hb_engine_num_layers": (_i64, [_vp]),
     "hb_engine_vocab_size": (_i64, [_vp]),
@@ -830,9 +832,10 @@ class Sequence_:
 class Engine:
     """Engine (src/engine/loader.rs:66-339) for the TP Llama path."""
 
-    def __init__(self, handle: int, world: Optional[TpWorld]):
+    def __init__(self, handle: int, world: Optional[TpWorld], max_batch: int):
         self.handle = handle
         self.world = world
+        self.max_batch = max_batch  # rows of one step
 
     @staticmethod
     def _config(model_path: Optional[str], max_seq_len: int, bf16: bool, tp: int, num_kv_blocks: int,
@@ -850,7 +853,7 @@ class Engine:
                           force_f32, max_seqs)
         h = C.c_void_p()
         check(lib.hb_engine_load(C.byref(cfg), world.handle if world else None, C.byref(h)))
-        return cls(h.value, world)
+        return cls(h.value, world, max_batch)
 
     @classmethod
     def create_random_config(cls, config: dict, *, seed: int = 1, std: float = 0.02, max_seq_len: int = 2048,
@@ -862,7 +865,7 @@ class Engine:
         cfg = cls._config(None, max_seq_len, bf16, 1, num_kv_blocks, max_batch, force_f32, max_seqs)
         h = C.c_void_p()
         check(lib.hb_engine_create_random_config(json.dumps(config).encode(), C.byref(cfg), seed, std, C.byref(h)))
-        return cls(h.value, None)
+        return cls(h.value, None, max_batch)
 
     @classmethod
     def create_random(cls, shape: dict, *, seed: int = 1, std: float = 0.02, norm_ones: bool = True,
@@ -878,7 +881,7 @@ class Engine:
         h = C.c_void_p()
         check(lib.hb_engine_create_random(C.byref(sh), C.byref(cfg), world.handle if world else None,
                                           seed, std, int(norm_ones), C.byref(h)))
-        return cls(h.value, world)
+        return cls(h.value, world, max_batch)
 
     def num_layers(self) -> int:
         return lib.hb_engine_num_layers(self.handle)
@@ -952,6 +955,15 @@ class Engine:
         out = np.empty(len(s), dtype=np.uint32)
         check(lib.hb_engine_sample(self.handle, len(s), s.ctypes.data, float(temperature), float(top_p), out.ctypes.data))
         return out
+
+    def set_profiling(self, on: bool) -> None:
+        """Steps that follow record the device time of every kind of kernel (profile_ms)."""
+        check(lib.hb_engine_set_profiling(self.handle, int(on)))
+
+    def profile_ms(self) -> dict:
+        ms = np.zeros(len(self.PROFILE_KINDS), dtype=np.float32)
+        check(lib.hb_engine_profile_ms(self.handle, ms.ctypes.data))
+        return dict(zip(self.PROFILE_KINDS, ms.tolist()))
 
     def num_free_state_slots(self) -> int:
         return lib.hb_engine_num_free_state_slots(self.handle)

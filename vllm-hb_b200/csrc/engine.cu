@@ -1462,6 +1462,18 @@ int hb_engine_profile_step(hb_engine* e, hb_seq* const* seqs, size_t B, const ui
   return HB_OK;
 }
 
+int hb_engine_set_profiling(hb_engine* e, int on) {
+  HB_CHECK_ARG(e, "hb_engine_set_profiling: null engine");
+  e->profiling = on != 0;
+  return HB_OK;
+}
+
+int hb_engine_profile_ms(const hb_engine* e, float* ms_by_kind) {
+  HB_CHECK_ARG(e && ms_by_kind, "hb_engine_profile_ms: null argument");
+  for (int c = 0; c < HB_PROFILE_KINDS; ++c) ms_by_kind[c] = e->prof_ms[c];
+  return HB_OK;
+}
+
 double hb_engine_gemm_bytes(const hb_engine* e, int64_t B) { return e ? e->family->gemm_bytes(e, B) : -1.0; }
 
 int hb_forward(hb_engine* e, hb_seq* s, const uint32_t* ids, size_t n, size_t seq_pos,

@@ -49,7 +49,11 @@ class _Live:
 
 class Scheduler:
     def __init__(self, engine, *, max_live: int = 64, step_tokens: int = 256):
-        self.engine, self.max_live, self.step_tokens = engine, max_live, step_tokens
+        # a step is one batch of the engine, and every live request may hold a state slot
+        slots = engine.num_free_state_slots()
+        self.engine = engine
+        self.max_live = min(max_live, slots) if slots > 0 else max_live
+        self.step_tokens = min(step_tokens, engine.max_batch)
         self.waiting: deque[Request] = deque()
         self.live: list[_Live] = []
         self.done: dict[str, list] = {}
