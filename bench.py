@@ -561,6 +561,39 @@ def run_gpu_arm(args, rank: int, world: int, local_rank: int) -> None:
         raise SystemExit("tensor-parallel parity check failed: " + json.dumps(parity))
 
 
+# --------------------------------------------------------------------- layered models
+def run_latarax(args) -> None:
+    """Prefill and decode of the Latarax design beside the Llama family at equal size (one GPU)."""
+    import torch
+
+    import __graft_entry__ as entry
+
+    hb = entry.load_package()
+    from vllm_hb_b200 import bench_layered
+
+    torch.cuda.set_device(0)
+    peak, kind = measured_peaks()
+    tflops = 1590.0
+    try:
+        tflops = float(json.loads((ROOT / "MEASURED_PEAKS.json").read_text())["bf16_tflops"])
+    except Exception:
+        pass
+    sampler = ClockSampler(0)
+    sampler.start()
+    sampler.begin_region()
+    report = bench_layered.run(hb, peak, tflops, args.steps, args.warmup, args.size)
+    clocks = sampler.stop()
+    launches = report.pop("gpu_launches")
+    first = report[next(reversed(report))]["latarax"]["decode batch 64"]
+    print(json.dumps({"metric": METRIC, "value": first["tok_s"], "unit": UNIT, "n_gpus": 1, "steps": args.steps,
+                      "warmup": args.warmup, "ms_per_step": first["ms"], "higher_is_better": True, "scaling": "weak",
+                      "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+                      "config": {"workload": "latarax and llama family at equal size, decode batch 64 of the last size",
+                                 "parallelism": "tp1", "l2": "inputs larger than L2 (weights read once per step)",
+                                 "peaks": f"of {kind}"},
+                      "gpu_launches": int(launches), "clocks": clocks, "sizes": report}), flush=True)
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -579,8 +612,10 @@ def main() -> None:
     ap.add_argument("--skip-checks", action="store_true",
                     help="N > 1: skip the untimed parity checks, the single-GPU base point and the row-parallel points")
     ap.add_argument("--tp1-layers", type=int, default=8, help="layers of the single-GPU base point of the N > 1 shape")
-    ap.add_argument("--workload", default="auto", choices=["auto", "mixtral"],
-                    help="auto: Llama-3.1-8B shape on one GPU, 70B shape on several; mixtral: Mixtral-8x7B shape")
+    ap.add_argument("--workload", default="auto", choices=["auto", "mixtral", "latarax"],
+                    help="auto: Llama-3.1-8B shape on one GPU, 70B shape on several; mixtral: Mixtral-8x7B shape; "
+                         "latarax: that design beside the Llama family at equal size, one GPU")
+    ap.add_argument("--size", default="", help="latarax: only the sizes whose name contains this text")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
@@ -593,6 +628,9 @@ def main() -> None:
         if args.gpus != 1 or world != 1:
             raise SystemExit(f"--gpus {args.gpus} needs torchrun with {args.gpus} ranks (WORLD_SIZE={world})")
     args.warmup = max(args.warmup, 3)
+    if args.workload == "latarax":
+        run_latarax(args)
+        return
     run_gpu_arm(args, rank, world, local_rank)
 
 

@@ -1,0 +1,206 @@
+"""Latarax beside the Llama family at equal width, feed-forward, depth and vocabulary.
+
+`python bench.py --workload latarax` runs it on one GPU: prefill of one long prompt and of several
+shorter ones, decode at several batch sizes, random weights.  For every kind of kernel it reports
+the time of a profiled step and the fraction of the roofline (the larger of bytes / measured HBM
+bandwidth and FLOPs / measured bf16 throughput, over the time).
+"""
+from __future__ import annotations
+
+import numpy as np
+
+VOCAB = 32000
+
+
+def gla(heads, dim, vdim, ff):
+    return {"type": "gla", "mixer": dict(heads=heads, dim=dim, vdim=vdim, tau=16.0), "mlp": {"kind": "dense", "ff": ff}}
+
+
+def parallel(heads, kv, dim, window, keep, rec_heads, ff):
+    decay = [1.0 - 2.0 ** (-3.0 - 5.0 * i / max(1, rec_heads - 1)) for i in range(rec_heads)]
+    return {"type": "parallel",
+            "mixer": {"left": dict(heads=heads, kv_heads=kv, dim=dim, vdim=dim, scale=dim ** -0.5,
+                                   mask=dict(size=window, keep_first=keep)),
+                      "right": dict(heads=rec_heads, dim=128, vdim=128, decay=decay)},
+            "mlp": {"kind": "dense", "ff": ff}}
+
+
+def sizes() -> list[dict]:
+    """Layers of about 1.3B- and 8B-parameter models; half of them gla, half parallel."""
+    out = []
+    for width, ff, layers in ((2048, 5632, 12), (4096, 14336, 8)):
+        heads = width // 128
+        pattern = [gla(heads, 64, 128, ff), parallel(heads, heads // 4, 128, 1024, 16, heads // 2, ff)]
+        out.append({
+            "name": f"width {width}, ff {ff}, {layers} layers",
+            "latarax": {"architecture": "Latarax", "width": width, "vocab": VOCAB, "streams": 4, "max_positions": 8192,
+                        "norm": {"eps": 1e-6}, "layers": [pattern[i % 2] for i in range(layers)]},
+            "llama": dict(hidden_size=width, intermediate_size=ff, num_hidden_layers=layers, num_attention_heads=heads,
+                          num_key_value_heads=heads // 4, vocab_size=VOCAB, rms_norm_eps=1e-6, rope_theta=500000.0)})
+    return out
+
+
+# ------------------------------------------------------------------------- work per kind
+def keys_seen(pos: np.ndarray, window: int, keep: int) -> float:
+    lo = np.maximum(0, pos - window + 1) if window else np.zeros_like(pos)
+    return float(np.sum(np.minimum(keep, lo) + pos - lo + 1))
+
+
+def work(shape: dict, family: str, positions: list[np.ndarray], wanted: int) -> dict:
+    """{kind: (bytes, flops)} of one step; positions[i] are the positions of segment i's rows."""
+    rows = float(sum(len(p) for p in positions))
+    w: dict = {}
+
+    def add(kind, nbytes, flops=0.0):
+        b, f = w.get(kind, (0.0, 0.0))
+        w[kind] = (b + nbytes, f + flops)
+
+    def gemm(kind, n, k, m=rows, n_out=None, out=2):
+        add(kind, 2.0 * n * k + 2.0 * m * k + out * m * (n_out or n), 2.0 * m * n * k)
+
+    def attention(heads, kv, dim, vdim, window, keep):
+        seen = sum(keys_seen(p, window, keep) for p in positions)
+        # every key a segment reads is counted once per segment (decode: once per row)
+        span = sum((min(p[-1] + 1, len(p) - 1 + window + min(keep, max(0, p[0] - window + 1))) if window else p[-1] + 1)
+                   for p in positions)
+        add("attention", 2.0 * kv * (dim + vdim) * span + 2.0 * rows * heads * (dim + vdim), 2.0 * heads * (dim + vdim) * seen)
+
+    if family == "llama":
+        H, I, hq, kv = (shape[k] for k in ("hidden_size", "intermediate_size", "num_attention_heads", "num_key_value_heads"))
+        for _ in range(shape["num_hidden_layers"]):
+            gemm("gemm_qkv", (hq + 2 * kv) * 128, H)
+            attention(hq, kv, 128, 128, 0, 0)
+            gemm("gemm_o_proj", H, hq * 128)
+            gemm("gemm_gate_up", 2 * I, H, n_out=I)
+            gemm("gemm_down", H, I)
+        gemm("gemm_lm_head", shape["vocab_size"], H, m=rows, out=4)  # this family computes every row's logits
+        return w
+    H, S = shape["width"], shape["streams"]
+    for layer in shape["layers"]:
+        m, I = layer["mixer"], layer["mlp"]["ff"]
+        recs = []
+        if layer["type"] == "gla":
+            q, v = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            gemm("gemm_qkv", 2 * q + 2 * v + 16, H)
+            recs.append(m)
+        else:
+            a, r = m["left"], m["right"]
+            recs.append(r)
+            q, v = r["heads"] * r["dim"], r["heads"] * r["vdim"]
+            kvw = a["kv_heads"] * (a["dim"] + a["vdim"])
+            gemm("gemm_qkv", a["heads"] * a["dim"] + kvw + 2 * q + 2 * v, H)
+            add("rope_kv", 4.0 * rows * kvw)
+            attention(a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["mask"]["size"], a["mask"]["keep_first"])
+            gemm("gemm_o_proj", H, a["heads"] * a["vdim"], out=4)
+        for r in recs:
+            hd, hv, st = r["heads"] * r["dim"], r["heads"] * r["vdim"], r["heads"] * r["dim"] * r["vdim"]
+            # state in and out once per segment; q, k, v in, o out; the recurrence itself is 6 flops per
+            # state element and token (chunked forms do more, which is not counted)
+            add("recurrence", 8.0 * st * len(positions) + rows * (2.0 * (2 * hd + hv) + 4.0 * hv), 6.0 * st * rows)
+            add("norm", rows * hv * (4.0 + 2.0 + 2.0))
+            gemm("gemm_o_proj", H, hv, out=4)
+        for two in (layer["type"] != "gla", False):
+            add("norm", rows * H * (8.0 * S + (8.0 if two else 4.0) + 2.0))
+        gemm("gemm_gate_up", 2 * I, H, n_out=I)
+        gemm("gemm_down", H, I, out=4)
+    add("norm", wanted * H * (4.0 * S + 2.0))
+    gemm("gemm_lm_head", shape["vocab"], H, m=wanted, out=4)
+    return w
+
+
+def kinds(ms: dict, w: dict, hbm_gbs: float, tflops: float) -> dict:
+    out = {}
+    for kind, (nbytes, flops) in w.items():
+        t = ms.get(kind, 0.0)
+        if t > 0:
+            ideal = max(nbytes / (hbm_gbs * 1e9), flops / (tflops * 1e12)) * 1e3
+            out[kind] = {"ms": round(t, 4), "roofline": round(ideal / t, 3)}
+    out["other"] = {"ms": round(sum(v for k, v in ms.items() if k not in w), 4)}
+    return out
+
+
+# ------------------------------------------------------------------------------ timing
+def prefill(eng, prompts, rows: int, steps: int, warmup: int):
+    """ms of one pass over the prompts: portions of up to `rows` tokens a step, all prompts together."""
+    per = max(1, rows // len(prompts))
+
+    def run(profile=False):
+        seqs = [eng.create_kv_cache() for _ in prompts]
+        total, ms, at, n = 0.0, {}, 0, len(prompts[0])
+        eng.set_profiling(profile)
+        while at < n:
+            c = min(per, n - at)
+            last = at + c == n
+            eng.step([(s, p[at:at + c], [c - 1] if last else []) for s, p in zip(seqs, prompts)], logits=False)
+            total += eng.last_step_ms()
+            if profile:
+                ms = {k: ms.get(k, 0.0) + v for k, v in eng.profile_ms().items()}
+            at += c
+        eng.set_profiling(False)
+        for s in seqs:
+            s.free()
+        return total, ms
+
+    for _ in range(warmup):
+        run()
+    t = min(run()[0] for _ in range(steps))
+    return t, run(profile=True)[1]
+
+
+def decode(eng, batch: int, ctx: int, steps: int, warmup: int, rows: int):
+    rng = np.random.default_rng(1)
+    seqs = [eng.create_kv_cache() for _ in range(batch)]
+    for s in seqs:
+        p = rng.integers(0, VOCAB, ctx)
+        for at in range(0, ctx, rows):
+            eng.step([(s, p[at:at + rows], [])], logits=False)
+    nxt = np.zeros(batch, dtype=np.uint32)
+    for _ in range(warmup):
+        eng.decode_batch(seqs, nxt.copy(), next_tokens=nxt)
+    ms = 0.0
+    for _ in range(steps):
+        eng.decode_batch(seqs, nxt.copy(), next_tokens=nxt)
+        ms += eng.last_step_ms()
+    _, prof = eng.profile_step(seqs, nxt.copy())
+    launches = eng.last_step_launches()
+    prof.pop("gemm", None)
+    for s in seqs:
+        s.free()
+    return ms / steps, prof, launches
+
+
+def run(hb, hbm_gbs: float, tflops: float, steps: int, warmup: int, only: str = "") -> dict:
+    rows, ctx = 2048, 1536
+    report = {}
+    launches = 0
+    for size in sizes():
+        if only and only not in size["name"]:
+            continue
+        entry = report[size["name"]] = {}
+        for family in ("latarax", "llama"):
+            shape = size[family]
+            kw = dict(max_seq_len=4224, max_batch=rows, max_seqs=128, num_kv_blocks=128 * 128)
+            eng = hb.Engine.create_random_config(shape, **kw) if family == "latarax" else \
+                hb.Engine.create_random(shape, **{k: v for k, v in kw.items() if k != "max_seqs"})
+            res = entry[family] = {"parameters": eng.param_count()}
+            rng = np.random.default_rng(0)
+            for label, n, length in (("prefill 1 x 4096", 1, 4096), ("prefill 8 x 512", 8, 512)):
+                prompts = rng.integers(0, VOCAB, (n, length))
+                ms, prof = prefill(eng, prompts, rows, 3, 2)
+                per = max(1, rows // n)
+                total: dict = {}
+                for at in range(0, length, per):
+                    w = work(shape, family, [np.arange(at, min(at + per, length))] * n, n if at + per >= length else 0)
+                    for k, (b, f) in w.items():
+                        total[k] = (total.get(k, (0, 0))[0] + b, total.get(k, (0, 0))[1] + f)
+                res[label] = {"tok_s": round(n * length / ms * 1e3), "ms": round(ms, 3),
+                              "kinds": kinds(prof, total, hbm_gbs, tflops)}
+            for batch in (1, 16, 64, 128):
+                ms, prof, n_launch = decode(eng, batch, ctx, steps, warmup, rows)
+                launches += n_launch * steps
+                w = work(shape, family, [np.arange(ctx + warmup + steps, ctx + warmup + steps + 1)] * batch, batch)
+                res[f"decode batch {batch}"] = {"tok_s": round(batch / ms * 1e3), "ms": round(ms, 4), "launches": n_launch,
+                                                "kinds": kinds(prof, w, hbm_gbs, tflops)}
+            eng.close()
+    report["gpu_launches"] = launches
+    return report

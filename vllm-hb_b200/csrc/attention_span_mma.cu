@@ -48,6 +48,22 @@ __device__ __forceinline__ BlockRuns block_runs(int first_pos, int last_pos, int
 __device__ __forceinline__ bool visible(int key, int pos, int window, int keep_first) {
   return key <= pos && (window <= 0 || pos - key < window || key < keep_first);
 }
+// A warp copies a 16-row block of `w` 16-byte vectors a row into rows of `stride` bytes; (j, c) is the
+// lane's first (row, vector), stepped without divisions.
+struct BlockCopy {
+  int w, j, c, dj, dc;
+  __device__ __forceinline__ BlockCopy(int width, int lane) : w(width / 8), j(lane / w), c(lane % w), dj(32 / w), dc(32 % w) {}
+  __device__ __forceinline__ void operator()(uint32_t dst, int stride, const __nv_bfloat16* src, int64_t src_row) const {
+    int jj = j, cc = c;
+#pragma unroll 4
+    while (jj < kBS) {
+      cp_async_16(dst + jj * stride + cc * 16, src + jj * src_row + cc * 8);
+      jj += dj;
+      cc += dc;
+      if (cc >= w) { cc -= w; ++jj; }
+    }
+  }
+};
 }  // namespace
 
 // NV: 16-column pairs of n-tiles, i.e. the value slice is at most 16 * NV wide.
@@ -80,22 +96,16 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
     if (m < n_rows) v = *reinterpret_cast<const uint4*>(q + (int64_t)(tile.row0 + m / R) * a.ld_q + (m % R) * D + c);
     *reinterpret_cast<uint4*>(s_q + m * KS + c) = v;
   }
-  auto load = [&](int step) {
+  const BlockCopy copy_k(D, lane), copy_v(VW, lane);
+  auto load = [&](int step) {  // every warp one block of 16 keys
     const int s = step % stages;
-    const uint32_t dk = smem_u32(s_k + s * kKeys * KS), dv = smem_u32(s_v + s * kKeys * VS);
-    const int kc = D / 8, vc = VW / 8;
-    for (int i = tid; i < kKeys * (kc + vc); i += kThreads) {
-      const bool is_k = i < kKeys * kc;
-      const int w = is_k ? kc : vc, e = is_k ? i : i - kKeys * kc, j = e / w, c = e % w * 8;
-      const int vb = step * (kKeys / kBS) + j / kBS;
-      // past the last block: any block will do, its keys are masked (positions beyond the row's)
-      const int lb = runs.block(min(vb, runs.n - 1));
-      int64_t phys = lb < a.max_blocks ? table[lb] : 0;
-      if (phys < 0 || phys >= a.num_blocks) phys = 0;  // never outside the pool
-      const int64_t slot = (phys * a.kv_heads + kvh) * kBS + j % kBS;
-      if (is_k) cp_async_16(dk + (j * KS + c) * 2, (const __nv_bfloat16*)a.kc + slot * D + c);
-      else cp_async_16(dv + (j * VS + c) * 2, (const __nv_bfloat16*)a.vc + slot * a.vdim + v0 + c);
-    }
+    // past the last block: any block will do, its keys are masked (positions beyond the row's)
+    const int lb = runs.block(min(step * kWarps + warp, runs.n - 1));
+    int64_t phys = lb < a.max_blocks ? table[lb] : 0;
+    if (phys < 0 || phys >= a.num_blocks) phys = 0;  // never outside the pool
+    const int64_t slot = (phys * a.kv_heads + kvh) * kBS;
+    copy_k(smem_u32(s_k + (s * kKeys + warp * kBS) * KS), KS * 2, (const __nv_bfloat16*)a.kc + slot * D, D);
+    copy_v(smem_u32(s_v + (s * kKeys + warp * kBS) * VS), VS * 2, (const __nv_bfloat16*)a.vc + slot * a.vdim + v0, a.vdim);
     cp_async_commit();
   };
   load(0);
@@ -244,21 +254,14 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
     tab = lb < a.max_blocks ? table[lb] : 0;
     if (tab < 0 || tab >= a.num_blocks) tab = 0;  // never outside the pool
   };
+  const BlockCopy copy_k(D, lane), copy_v(VW, lane);
   auto load = [&](int i) {
     if (i < n_w) {
       if (i >= tab_base + 32) load_tab(i);
       const int64_t slot = ((int64_t)__shfl_sync(0xffffffffu, tab, i - tab_base) * a.kv_heads + kvh) * kBS;
       const uint32_t dst = smem_u32(ring + i % kRing * stage_elems);
-      const __nv_bfloat16* k = (const __nv_bfloat16*)a.kc + slot * D;
-      const __nv_bfloat16* v = (const __nv_bfloat16*)a.vc + slot * a.vdim + v0;
-      for (int e = lane; e < kBS * (D / 8); e += 32) {
-        const int j = e / (D / 8), c = e % (D / 8) * 8;
-        cp_async_16(dst + (j * KS + c) * 2, k + j * D + c);
-      }
-      for (int e = lane; e < kBS * (VW / 8); e += 32) {
-        const int j = e / (VW / 8), c = e % (VW / 8) * 8;
-        cp_async_16(dst + (kBS * KS + j * VS + c) * 2, v + (int64_t)j * a.vdim + c);
-      }
+      copy_k(dst, KS * 2, (const __nv_bfloat16*)a.kc + slot * D, D);
+      copy_v(dst + kBS * KS * 2, VS * 2, (const __nv_bfloat16*)a.vc + slot * a.vdim + v0, a.vdim);
     }
     cp_async_commit();
   };

@@ -26,7 +26,7 @@ __device__ __forceinline__ float low_rank_log_decay(const Recurrence& a, const f
 // DG-th state row, so its part of the state never meets another thread's; only the output needs
 // a sum over the row groups.  RPT > 0: the thread's rows stay in registers for the whole segment.
 template <typename T, int VEC, int RPT>
-__global__ void __launch_bounds__(kRecThreads)
+__global__ void __launch_bounds__(kRecThreads, RPT == 4 ? 5 : RPT == 8 ? 4 : 1)
 recurrence_tokens_kernel(const Recurrence a, const int32_t* __restrict__ list) {
   constexpr int LANES = kRecCols / VEC, DG = kRecThreads / LANES;
   extern __shared__ float sm[];
@@ -152,6 +152,7 @@ int recurrence_tokens(cudaStream_t st, const Recurrence& a, const int32_t* list,
   }
   if (dtype == HB_BF16) {
     if (!vec) return launch(recurrence_tokens_kernel<__nv_bfloat16, 1, 0>);
+    if (a.dim <= 64) return launch(recurrence_tokens_kernel<__nv_bfloat16, 4, 4>);
     return a.dim <= 128 ? launch(recurrence_tokens_kernel<__nv_bfloat16, 4, 8>) : launch(recurrence_tokens_kernel<__nv_bfloat16, 4, 0>);
   }
   return fail(HB_ERR_UNSUPPORTED_DTYPE, "recurrence runs in bf16 or f32");

@@ -38,10 +38,55 @@ __device__ __forceinline__ float ld_proj(const Recurrence& a, int64_t row, int c
 // log2 of a constant decay to the power n (n = 0: exactly 0, also for decay 0)
 __device__ __forceinline__ float log2_pow(float log2_decay, int n) { return n == 0 ? 0.f : log2_decay * (float)n; }
 __device__ __forceinline__ int pad16d(int n) { return (n + 15) / 16 * 16; }
-__device__ __forceinline__ void put_split(bf16* hi, bf16* lo, float x) {
-  const bf16 h = __float2bfloat16_rn(x);
-  *hi = h;
-  *lo = __float2bfloat16_rn(x - __bfloat162float(h));
+// Eight neighbouring columns of a projection row (16 bytes where they are aligned); columns from
+// `valid` on are zero.
+__device__ __forceinline__ void ld_proj8(float (&f)[8], const Recurrence& a, int64_t row, int col, int valid) {
+  const bf16* p = (const bf16*)a.p + row * a.ld + col;
+  if (valid >= 8 && (reinterpret_cast<uintptr_t>(p) & 15) == 0) {
+    const uint4 v = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const __nv_bfloat162 b = *reinterpret_cast<const __nv_bfloat162*>(&w[i]);
+      f[2 * i] = __low2float(b);
+      f[2 * i + 1] = __high2float(b);
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) f[i] = i < valid ? __bfloat162float(p[i]) : 0.f;
+  }
+}
+// hi/lo pairs of eight values to 16-byte aligned shared memory
+__device__ __forceinline__ void put_split8(bf16* hi, bf16* lo, const float (&f)[8]) {
+  uint32_t h[4], l[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) split_bf16(f[2 * i], f[2 * i + 1], h[i], l[i]);
+  *reinterpret_cast<uint4*>(hi) = make_uint4(h[0], h[1], h[2], h[3]);
+  *reinterpret_cast<uint4*>(lo) = make_uint4(l[0], l[1], l[2], l[3]);
+}
+__device__ __forceinline__ void put8(bf16* dst, const float (&f)[8]) {
+  *reinterpret_cast<uint4*>(dst) = make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
+}
+// Calls f(token, first channel) for every group of eight channels of a [64][DP] tile, spread over the
+// CTA's threads without divisions in the loop.
+template <typename F>
+__device__ __forceinline__ void for_groups(int DP, F f) {
+  const int w = DP / 8, dj = kT / w, dc = kT % w;
+  int j = threadIdx.x / w, c = threadIdx.x % w;
+  while (j < kC) {
+    f(j, c * 8);
+    j += dj;
+    c += dc;
+    if (c >= w) { c -= w; ++j; }
+  }
+}
+// Two neighbouring outputs of an accumulator row
+__device__ __forceinline__ void put_pair(float* p, float x, float y, int valid) {
+  if (valid >= 2 && (reinterpret_cast<uintptr_t>(p) & 7) == 0) *reinterpret_cast<float2*>(p) = make_float2(x, y);
+  else {
+    if (valid >= 1) p[0] = x;
+    if (valid >= 2) p[1] = y;
+  }
 }
 }  // namespace
 
@@ -82,14 +127,16 @@ recurrence_decay_kernel(const Recurrence a, const RowRange* __restrict__ chunks,
 
 // Value tile [64 tokens][64 columns] as hi/lo pairs; rows and columns outside are zero.
 __device__ __forceinline__ void load_values(const Recurrence& a, const RowRange& ch, int h, int v0, bf16* hi, bf16* lo) {
-  for (int i = threadIdx.x; i < kC * kVT; i += kT) {
-    const int j = i / kVT, c = i % kVT;
-    float v = 0.f;
-    if (j < ch.n && v0 + c < a.vdim) {
-      v = ld_proj(a, ch.row0 + j, a.off_v + h * a.vdim + v0 + c);
-      if (a.silu_qkv) v = rec_silu(v);
+#pragma unroll 4
+  for (int i = threadIdx.x; i < kC * kVT / 8; i += kT) {
+    const int j = i / (kVT / 8), c = i % (kVT / 8) * 8;
+    float v[8];
+    ld_proj8(v, a, ch.row0 + min(j, ch.n - 1), a.off_v + h * a.vdim + v0 + c, j < ch.n ? a.vdim - v0 - c : 0);
+    if (a.silu_qkv) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] = rec_silu(v[e]);
     }
-    put_split(hi + j * kVS + c, lo + j * kVS + c, v);
+    put_split8(hi + j * kVS + c, lo + j * kVS + c, v);
   }
 }
 
@@ -107,18 +154,22 @@ recurrence_state_kernel(const Recurrence a, const RowRange* __restrict__ chunks,
   const RowRange ch = chunks[blockIdx.x];
   const int hd = a.heads * D;
   const float ld2 = a.decay ? log2f(a.decay[h]) : 0.f;
-  for (int i = tid; i < kC * DP; i += kT) {
-    const int j = i / DP, d = i % DP;
-    float k = 0.f;
-    if (j < ch.n && d < D) {
-      k = ld_proj(a, ch.row0 + j, a.off_k + h * D + d);
-      if (a.silu_qkv) k = rec_silu(k);
-      const float e = a.decay ? log2_pow(ld2, ch.n - 1 - j)
-                              : cum[(int64_t)(ch.row0 + ch.n - 1) * hd + h * D + d] - cum[(int64_t)(ch.row0 + j) * hd + h * D + d];
-      k *= exp2f(e);
+  for_groups(DP, [&](int j, int d) {
+    float k[8];
+    const bool live = j < ch.n;
+    ld_proj8(k, a, ch.row0 + min(j, ch.n - 1), a.off_k + h * D + d, live ? D - d : 0);
+    if (live) {
+      const float f = a.decay ? exp2f(log2_pow(ld2, ch.n - 1 - j)) : 1.f;
+      const float* end = cum + (int64_t)(ch.row0 + ch.n - 1) * hd + h * D + d;
+      const float* own = cum + (int64_t)(ch.row0 + j) * hd + h * D + d;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        if (a.silu_qkv) k[e] = rec_silu(k[e]);
+        k[e] *= a.decay ? f : (d + e < D ? exp2f(end[e] - own[e]) : 0.f);
+      }
     }
-    put_split(k_hi + j * KS + d, k_lo + j * KS + d, k);
-  }
+    put_split8(k_hi + j * KS + d, k_lo + j * KS + d, k);
+  });
   load_values(a, ch, h, v0, v_hi, v_lo);
   __syncthreads();
   float* o = out + ((int64_t)blockIdx.x * a.heads + h) * D * a.vdim + v0;
@@ -149,9 +200,9 @@ recurrence_state_kernel(const Recurrence a, const RowRange* __restrict__ chunks,
 #pragma unroll
     for (int i = 0; i < 8; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int d = mt * 16 + g + (e >> 1) * 8, c = i * 8 + 2 * t + (e & 1);
-        if (d < D && v0 + c < a.vdim) o[(int64_t)d * a.vdim + c] = acc[i][e];
+      for (int r = 0; r < 2; ++r) {
+        const int d = mt * 16 + g + r * 8, c = i * 8 + 2 * t;
+        if (d < D) put_pair(o + (int64_t)d * a.vdim + c, acc[i][2 * r], acc[i][2 * r + 1], a.vdim - v0 - c);
       }
   }
 }
@@ -173,21 +224,36 @@ recurrence_scan_kernel(const Recurrence a, const RowRange* __restrict__ segs, co
   float s[VEC];
 #pragma unroll
   for (int j = 0; j < VEC; ++j) s[j] = info.pos0 > 0 ? state[j] : 0.f;  // a new sequence starts from zero
-  for (int c = 0; c < sg.n; ++c) {
-    float* u = chunk_state + ((int64_t)(sg.row0 + c) * a.heads + h) * per_head + i;
-    const RowRange ch = chunks[sg.row0 + c];
-    const float f = exp2f(a.decay ? log2_pow(ld2, ch.n) : cum[(int64_t)(ch.row0 + ch.n - 1) * hd + h * a.dim + d]);
-    float v[VEC];
-    if (VEC == 4) {
-      const float4 x = *reinterpret_cast<const float4*>(u);
-      v[0] = x.x; v[1 % VEC] = x.y; v[2 % VEC] = x.z; v[3 % VEC] = x.w;
-      *reinterpret_cast<float4*>(u) = make_float4(s[0], s[1 % VEC], s[2 % VEC], s[3 % VEC]);
-    } else {
-      v[0] = *u;
-      *u = s[0];
+  constexpr int AHEAD = 4;  // chunks fetched together
+  const int64_t stride = (int64_t)a.heads * per_head;
+  float* u = chunk_state + ((int64_t)sg.row0 * a.heads + h) * per_head + i;
+  for (int c0 = 0; c0 < sg.n; c0 += AHEAD) {
+    float v[AHEAD][VEC], f[AHEAD];
+#pragma unroll
+    for (int c = 0; c < AHEAD; ++c) {
+      f[c] = 0.f;
+      if (c0 + c < sg.n) {
+        const RowRange ch = chunks[sg.row0 + c0 + c];
+        f[c] = a.decay ? log2_pow(ld2, ch.n) : cum[(int64_t)(ch.row0 + ch.n - 1) * hd + h * a.dim + d];
+        if (VEC == 4) {
+          const float4 x = *reinterpret_cast<const float4*>(u + c * stride);
+          v[c][0] = x.x; v[c][1 % VEC] = x.y; v[c][2 % VEC] = x.z; v[c][3 % VEC] = x.w;
+        } else {
+          v[c][0] = u[c * stride];
+        }
+      }
     }
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) s[j] = fmaf(f, s[j], v[j]);
+    for (int c = 0; c < AHEAD; ++c) {
+      if (c0 + c < sg.n) {
+        if (VEC == 4) *reinterpret_cast<float4*>(u + c * stride) = make_float4(s[0], s[1 % VEC], s[2 % VEC], s[3 % VEC]);
+        else u[c * stride] = s[0];
+        const float k = exp2f(f[c]);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) s[j] = fmaf(k, s[j], v[c][j]);
+      }
+    }
+    u += AHEAD * stride;
   }
   pdl_trigger();
 #pragma unroll
@@ -216,30 +282,36 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
   const int hd = a.heads * D;
   const float ld2 = LR ? 0.f : log2f(a.decay[h]);
   if (LR) {
-    for (int i = tid; i < kC * DP; i += kT) {
-      const int j = i / DP, d = i % DP;
+    for_groups(DP, [&](int j, int d) {
       // tokens past the end keep the last decay: every exponent stays <= 0
-      s_b[j * BS + d] = d < D ? cum[(int64_t)(ch.row0 + min(j, ch.n - 1)) * hd + h * D + d] : 0.f;
-    }
+      const float* c = cum + (int64_t)(ch.row0 + min(j, ch.n - 1)) * hd + h * D + d;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) s_b[j * BS + d + e] = d + e < D ? c[e] : 0.f;
+    });
     __syncthreads();
   }
-  for (int i = tid; i < kC * DP; i += kT) {
-    const int j = i / DP, d = i % DP;
-    float q = 0.f, k = 0.f;
-    if (j < ch.n && d < D) {
-      q = ld_proj(a, ch.row0 + j, a.off_q + h * D + d);
-      k = ld_proj(a, ch.row0 + j, a.off_k + h * D + d);
-      if (a.silu_qkv) { q = rec_silu(q); k = rec_silu(k); }
+  for_groups(DP, [&](int j, int d) {
+    float q[8], k[8];
+    const int valid = j < ch.n ? D - d : 0;
+    const int64_t row = ch.row0 + min(j, ch.n - 1);
+    ld_proj8(q, a, row, a.off_q + h * D + d, valid);
+    ld_proj8(k, a, row, a.off_k + h * D + d, valid);
+    if (a.silu_qkv) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) { q[e] = rec_silu(q[e]); k[e] = rec_silu(k[e]); }
     }
     if (LR) {
-      q_hi[j * KS + d] = __float2bfloat16_rn(q);   // exact; the scale is applied to the results
-      k_raw[j * KS + d] = __float2bfloat16_rn(k);
-      put_split(k_hi + j * KS + d, k_lo + j * KS + d, k * exp2f(s_b[(j | 15) * BS + d] - s_b[j * BS + d]));
+      put8(q_hi + j * KS + d, q);   // exact; the scale is applied to the results
+      put8(k_raw + j * KS + d, k);
+      const float *end = s_b + (j | 15) * BS + d, *own = s_b + j * BS + d;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) k[e] *= exp2f(end[e] - own[e]);
+      put_split8(k_hi + j * KS + d, k_lo + j * KS + d, k);
     } else {
-      put_split(q_hi + j * KS + d, q_lo + j * KS + d, q);
-      put_split(k_hi + j * KS + d, k_lo + j * KS + d, k);
+      put_split8(q_hi + j * KS + d, q_lo + j * KS + d, q);
+      put_split8(k_hi + j * KS + d, k_lo + j * KS + d, k);
     }
-  }
+  });
   __syncthreads();
 
   // ---- scores of this warp's 16 tokens with all tokens up to them: s[n] = keys 8n .. 8n+7
@@ -291,16 +363,25 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
 #pragma unroll
       for (int e = 0; e < 8; ++e) p[e] = 0.f;
       const int j0 = warp * 16 + 2 * t;
-      for (int d = 0; d < D; ++d) {
-        const float b0 = s_b[i0 * BS + d], b1 = s_b[i1 * BS + d];
-        const float q0 = __bfloat162float(q_hi[i0 * KS + d]), q1 = __bfloat162float(q_hi[i1 * KS + d]);
+      auto bf2 = [](const bf16* p2) {
+        const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(p2);
+        return make_float2(__low2float(v), __high2float(v));
+      };
+      auto fl2 = [](const float* p2) { return *reinterpret_cast<const float2*>(p2); };
+      auto pair = [](float& acc, float2 q, float2 k, float2 bi, float2 bj) {
+        acc = fmaf(q.x * k.x, exp2f(fminf(bi.x - bj.x, 0.f)), acc);
+        acc = fmaf(q.y * k.y, exp2f(fminf(bi.y - bj.y, 0.f)), acc);
+      };
+      for (int d = 0; d < D; d += 2) {  // channels past D are zero
+        const float2 b0 = fl2(s_b + i0 * BS + d), b1 = fl2(s_b + i1 * BS + d);
+        const float2 q0 = bf2(q_hi + i0 * KS + d), q1 = bf2(q_hi + i1 * KS + d);
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const float kj = __bfloat162float(k_raw[(j0 + e) * KS + d]), bj = s_b[(j0 + e) * BS + d];
-          const float kj8 = __bfloat162float(k_raw[(j0 + 8 + e) * KS + d]), bj8 = s_b[(j0 + 8 + e) * BS + d];
-          p[e] = fmaf(q0 * kj, exp2f(fminf(b0 - bj, 0.f)), p[e]);
-          p[2 + e] = fmaf(q1 * kj, exp2f(fminf(b1 - bj, 0.f)), p[2 + e]);
-          p[6 + e] = fmaf(q1 * kj8, exp2f(fminf(b1 - bj8, 0.f)), p[6 + e]);
+          const float2 kj = bf2(k_raw + (j0 + e) * KS + d), bj = fl2(s_b + (j0 + e) * BS + d);
+          const float2 kj8 = bf2(k_raw + (j0 + 8 + e) * KS + d), bj8 = fl2(s_b + (j0 + 8 + e) * BS + d);
+          pair(p[e], q0, kj, b0, bj);
+          pair(p[2 + e], q1, kj, b1, bj);
+          pair(p[6 + e], q1, kj8, b1, bj8);
         }
       }
 #pragma unroll
@@ -331,10 +412,21 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
 #pragma unroll
     for (int i = 0; i < 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     for (int d0 = 0; d0 < DP; d0 += 64) {
-      for (int i = tid; i < 64 * kVT; i += kT) {
-        const int d = d0 + i / kVT, c = i % kVT;
-        const float x = d < D && v0 + c < a.vdim ? st[(int64_t)d * a.vdim + v0 + c] : 0.f;
-        put_split(t_hi + i / kVT * kVS + c, t_lo + i / kVT * kVS + c, x);
+      const bool aligned = a.vdim % 4 == 0;
+#pragma unroll 4
+      for (int i = tid; i < 64 * kVT / 8; i += kT) {
+        const int r = i / (kVT / 8), d = d0 + r, c = i % (kVT / 8) * 8;
+        const float* src = st + (int64_t)d * a.vdim + v0 + c;
+        float f[8];
+        if (aligned && d < D && v0 + c + 8 <= a.vdim) {
+          const float4 x = *reinterpret_cast<const float4*>(src), y = *reinterpret_cast<const float4*>(src + 4);
+          f[0] = x.x; f[1] = x.y; f[2] = x.z; f[3] = x.w;
+          f[4] = y.x; f[5] = y.y; f[6] = y.z; f[7] = y.w;
+        } else {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) f[e] = d < D && v0 + c + e < a.vdim ? src[e] : 0.f;
+        }
+        put_split8(t_hi + r * kVS + c, t_lo + r * kVS + c, f);
       }
       if (d0 == 0) load_values(a, ch, h, v0, v_hi, v_lo);
       __syncthreads();
@@ -386,10 +478,11 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
 #pragma unroll
       for (int i = 0; i < 8; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int r = e < 2 ? i0 : i1, c = i * 8 + 2 * t + (e & 1);
-          if (r < ch.n && v0 + c < a.vdim)
-            a.o[(int64_t)(ch.row0 + r) * a.ld_o + (int64_t)h * a.vdim + v0 + c] = o[i][e] * a.q_scale;
+        for (int e = 0; e < 2; ++e) {
+          const int r = e ? i1 : i0, c = i * 8 + 2 * t;
+          if (r < ch.n)
+            put_pair(a.o + (int64_t)(ch.row0 + r) * a.ld_o + (int64_t)h * a.vdim + v0 + c, o[i][2 * e] * a.q_scale,
+                     o[i][2 * e + 1] * a.q_scale, a.vdim - v0 - c);
         }
     }
     __syncthreads();
