@@ -288,7 +288,7 @@ def test_recurrence_remembers_a_far_token(hb, cuda):
 # ------------------------------------------------------------------- streams and gated norms
 @pytest.mark.parametrize("dtype", ["bf16", "f32"])
 @pytest.mark.parametrize("streams", [1, 2, 3, 4, 5, 11])
-@pytest.mark.parametrize("width", [64, 101, 1000])
+@pytest.mark.parametrize("width", [64, 101, 1000, 13000])
 def test_streams(hb, cuda, dtype, streams, width):
     import torch
 

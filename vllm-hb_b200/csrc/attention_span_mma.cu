@@ -5,9 +5,9 @@
 //
 //   tiles  (prompt portions): CTA = 64 rows = up to 64 / R consecutive positions of one segment x
 //          the R query heads of a kv head; four warps of 16 rows share every 64-key tile.
-//   tokens (decoded tokens): CTA = one row and kv head, the R <= 16 query heads padded to 16 MMA
-//          rows; each of four warps streams every fourth 16-key block through a ring of its own
-//          and the warps' (m, l, O) meet in shared memory.
+//   tokens (decoded tokens): CTA = one row and kv head with its R <= 16 query heads; each of four
+//          warps streams every fourth 16-key block through a ring of its own and the warps'
+//          (m, l, O) meet in shared memory.
 //
 // Both read only the 16-key blocks that some row of the CTA sees: those of the first kept tokens
 // and those from the earliest window on.  Rows of shared memory are padded by 8 elements, so that
@@ -47,6 +47,10 @@ __device__ __forceinline__ BlockRuns block_runs(int first_pos, int last_pos, int
 }
 __device__ __forceinline__ bool visible(int key, int pos, int window, int keep_first) {
   return key <= pos && (window <= 0 || pos - key < window || key < keep_first);
+}
+// Every key of the block that starts at `key` is visible from all positions first .. last.
+__device__ __forceinline__ bool all_visible(int key, int first, int last, int window, int keep_first) {
+  return key + kBS - 1 <= first && (window <= 0 || last - key < window || key + kBS <= keep_first);
 }
 // A warp copies a 16-row block of `w` 16-byte vectors a row into rows of `stride` bytes; (j, c) is the
 // lane's first (row, vector), stepped without divisions.
@@ -118,6 +122,9 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
   for (int i = 0; i < 2 * NV; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
   const float sc = a.scale * 1.4426950408889634f;  // scores in units of log2
+  const bool sc_ok = sc > 0.f;
+  const float es = sc_ok ? sc : 1.f;               // what the exponential still multiplies by
+  const int warp_first = first_pos + warp * 16 / R, warp_last = min(first_pos + (warp * 16 + 15) / R, last_pos);
   const uint32_t q_addr = smem_u32(s_q + (warp * 16 + (lane & 15)) * KS + (lane >> 4) * 8);
 
   for (int step = 0; step < n_steps; ++step) {
@@ -147,32 +154,46 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
           mma_bf16_16816(s[2 * nk + 1], qa, b2, b3);
         }
       }
+      // scores stay unscaled: sc > 0 is applied inside the exponential (sc <= 0: scaled here)
+      bool full = sc_ok;
+#pragma unroll
+      for (int b = 0; b < 4; ++b) {
+        const int vb = step * (kKeys / kBS) + b;
+        full = full && vb < runs.n && all_visible(runs.block(vb) * kBS, warp_first, warp_last, a.window, a.keep_first);
+      }
+      if (!full) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const int vb = step * (kKeys / kBS) + i / 2;
+          const int key = vb < runs.n ? runs.block(vb) * kBS + (i & 1) * 8 + 2 * t : INT_MAX - 1;
+#pragma unroll
+          for (int c = 0; c < 2; ++c) {
+            s[i][c] = visible(key + c, p0, a.window, a.keep_first) ? (sc_ok ? s[i][c] : s[i][c] * sc) : -INFINITY;
+            s[i][2 + c] = visible(key + c, p1, a.window, a.keep_first) ? (sc_ok ? s[i][2 + c] : s[i][2 + c] * sc) : -INFINITY;
+          }
+        }
+      }
       float x0 = -INFINITY, x1 = -INFINITY;
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
-        const int vb = step * (kKeys / kBS) + i / 2;
-        const int key = vb < runs.n ? runs.block(vb) * kBS + (i & 1) * 8 + 2 * t : INT_MAX - 1;
-#pragma unroll
-        for (int c = 0; c < 2; ++c) {
-          s[i][c] = visible(key + c, p0, a.window, a.keep_first) ? s[i][c] * sc : -INFINITY;
-          s[i][2 + c] = visible(key + c, p1, a.window, a.keep_first) ? s[i][2 + c] * sc : -INFINITY;
-          x0 = fmaxf(x0, s[i][c]);
-          x1 = fmaxf(x1, s[i][2 + c]);
-        }
+        x0 = fmaxf(x0, fmaxf(s[i][0], s[i][1]));
+        x1 = fmaxf(x1, fmaxf(s[i][2], s[i][3]));
       }
       x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 1)); x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 2));
       x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 1)); x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
       const float n0 = fmaxf(m0, x0), n1 = fmaxf(m1, x1);
       const float e0 = n0 == -INFINITY ? 0.f : n0, e1 = n1 == -INFINITY ? 0.f : n1;  // nothing visible yet
-      const float al0 = exp2f(m0 - e0), al1 = exp2f(m1 - e1);
-      m0 = n0; m1 = n1;
-      l0 *= al0; l1 *= al1;
+      if (__any_sync(0xffffffffu, n0 != m0 || n1 != m1)) {
+        const float al0 = ex2((m0 - e0) * es), al1 = ex2((m1 - e1) * es);
+        m0 = n0; m1 = n1;
+        l0 *= al0; l1 *= al1;
 #pragma unroll
-      for (int i = 0; i < 2 * NV; ++i) { o[i][0] *= al0; o[i][1] *= al0; o[i][2] *= al1; o[i][3] *= al1; }
+        for (int i = 0; i < 2 * NV; ++i) { o[i][0] *= al0; o[i][1] *= al0; o[i][2] *= al1; o[i][3] *= al1; }
+      }
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
-        s[i][0] = exp2f(s[i][0] - e0); s[i][1] = exp2f(s[i][1] - e0);
-        s[i][2] = exp2f(s[i][2] - e1); s[i][3] = exp2f(s[i][3] - e1);
+        s[i][0] = ex2((s[i][0] - e0) * es); s[i][1] = ex2((s[i][1] - e0) * es);
+        s[i][2] = ex2((s[i][2] - e1) * es); s[i][3] = ex2((s[i][3] - e1) * es);
         l0 += s[i][0] + s[i][1];
         l1 += s[i][2] + s[i][3];
       }
@@ -219,7 +240,11 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
 }
 
 // n_splits > 1: every CTA takes its share of the row's blocks and writes (m, l, O) partials.
-template <int NV>
+//
+// The products are turned over, so that the few query heads are the narrow MMA side:
+// S^T[16 keys, 8 NT heads] = K Q^T and O^T[values, heads] += V^T P^T (P transposed in registers).
+// MT: 16-column tiles of the value slice, NT: groups of 8 query heads.
+template <int MT, int NT>
 __global__ void __launch_bounds__(kThreads)
 span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, int n_splits, float* __restrict__ part) {
   extern __shared__ __align__(16) uint8_t smem[];
@@ -231,12 +256,13 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
   const int stage_elems = kBS * (KS + VS);
   __nv_bfloat16* s_q = (__nv_bfloat16*)smem;                                  // [16][KS]
   __nv_bfloat16* ring = s_q + 16 * KS + (size_t)warp * kRing * stage_elems;   // [kRing][K 16 x KS | V 16 x VS]
-  for (int s = 0; s < kRing; ++s) {
-    for (int i = lane; i < kBS; i += 32) {
-      for (int c = D; c < KS; c += 8) *reinterpret_cast<uint4*>(ring + s * stage_elems + i * KS + c) = make_uint4(0, 0, 0, 0);
-      for (int c = VW; c < VS; c += 8)
-        *reinterpret_cast<uint4*>(ring + s * stage_elems + kBS * KS + i * VS + c) = make_uint4(0, 0, 0, 0);
-    }
+  if (D % 16 || VW % 16) {  // padding columns stay zero
+    for (int s = 0; s < kRing; ++s)
+      for (int i = lane; i < kBS; i += 32) {
+        for (int c = D; c < DP; c += 8) *reinterpret_cast<uint4*>(ring + s * stage_elems + i * KS + c) = make_uint4(0, 0, 0, 0);
+        for (int c = VW; c < VP; c += 8)
+          *reinterpret_cast<uint4*>(ring + s * stage_elems + kBS * KS + i * VS + c) = make_uint4(0, 0, 0, 0);
+      }
   }
   pdl_grid_wait();
   const int64_t row = rows[blockIdx.x];
@@ -255,15 +281,18 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
     if (tab < 0 || tab >= a.num_blocks) tab = 0;  // never outside the pool
   };
   const BlockCopy copy_k(D, lane), copy_v(VW, lane);
+  const uint32_t ring_u = smem_u32(ring);
+  int stage_in = 0;  // stage the next load fills
   auto load = [&](int i) {
     if (i < n_w) {
       if (i >= tab_base + 32) load_tab(i);
       const int64_t slot = ((int64_t)__shfl_sync(0xffffffffu, tab, i - tab_base) * a.kv_heads + kvh) * kBS;
-      const uint32_t dst = smem_u32(ring + i % kRing * stage_elems);
+      const uint32_t dst = ring_u + stage_in * stage_elems * 2;
       copy_k(dst, KS * 2, (const __nv_bfloat16*)a.kc + slot * D, D);
       copy_v(dst + kBS * KS * 2, VS * 2, (const __nv_bfloat16*)a.vc + slot * a.vdim + v0, a.vdim);
     }
     cp_async_commit();
+    stage_in = stage_in + 1 == kRing ? 0 : stage_in + 1;
   };
   load_tab(0);
   for (int i = 0; i < kRing - 1; ++i) load(i);
@@ -275,114 +304,138 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
     *reinterpret_cast<uint4*>(s_q + m * KS + c) = v;
   }
   __syncthreads();
-  float o[2 * NV][4];
+  float o[NT][MT][4], m[NT][2], l[NT][2];  // heads 8n + 2t, 8n + 2t + 1; o: value columns gi, gi + 8 of a tile
 #pragma unroll
-  for (int i = 0; i < 2 * NV; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
-  const float sc = a.scale * 1.4426950408889634f;
-  const uint32_t q_addr = smem_u32(s_q + (lane & 15) * KS + (lane >> 4) * 8);
+  for (int n = 0; n < NT; ++n) {
+#pragma unroll
+    for (int i = 0; i < MT; ++i) o[n][i][0] = o[n][i][1] = o[n][i][2] = o[n][i][3] = 0.f;
+    m[n][0] = m[n][1] = -INFINITY;
+    l[n][0] = l[n][1] = 0.f;
+  }
+  const float sc = a.scale * 1.4426950408889634f;  // scores in units of log2
+  const uint32_t q_addr = smem_u32(s_q + (lane & 7) * KS + (lane >> 3) * 8);  // B fragments of two 16-channel steps
+  const uint32_t k_off = (uint32_t)(((lane & 15) * KS + (lane >> 4) * 8) * 2);
+  const uint32_t v_off = (uint32_t)((kBS * KS + ((lane & 7) + (lane >> 4) * 8) * VS + ((lane >> 3) & 1) * 8) * 2);
+  int stage = 0;
   for (int i = 0; i < n_w; ++i) {
     load(i + kRing - 1);
     cp_async_wait<kRing - 1>();
     __syncwarp();
-    const __nv_bfloat16* kt = ring + i % kRing * stage_elems;
-    const __nv_bfloat16* vt = kt + kBS * KS;
-    float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-    const uint32_t k_addr = smem_u32(kt + ((lane & 7) + (lane >> 4) * 8) * KS + ((lane >> 3) & 1) * 8);
-    for (int ks = 0; ks < DP / 16; ++ks) {
-      uint32_t qa[4], b0, b1, b2, b3;
-      ldsm_x4(q_addr + ks * 32, qa[0], qa[1], qa[2], qa[3]);
-      ldsm_x4(k_addr + ks * 32, b0, b1, b2, b3);
-      mma_bf16_16816(s[0], qa, b0, b1);
-      mma_bf16_16816(s[1], qa, b2, b3);
+    const uint32_t base = ring_u + stage * stage_elems * 2;
+    stage = stage + 1 == kRing ? 0 : stage + 1;
+    float s[NT][2][4];  // two partial sums, so that neighbouring steps do not wait for each other
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[n][0][e] = s[n][1][e] = 0.f;
+#pragma unroll 4
+    for (int ks = 0; ks < DP / 16; ks += 2) {
+      uint32_t k0[4], k1[4];
+      ldsm_x4(base + k_off + ks * 32, k0[0], k0[1], k0[2], k0[3]);
+      const bool two = ks + 1 < DP / 16;
+      if (two) ldsm_x4(base + k_off + ks * 32 + 32, k1[0], k1[1], k1[2], k1[3]);
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        uint32_t b0, b1, b2, b3;
+        // (a lone last step also reads the 16 elements behind it, into the ring at most: unused)
+        ldsm_x4(q_addr + (n * 8 * KS + ks * 16) * 2, b0, b1, b2, b3);
+        mma_bf16_16816(s[n][0], k0, b0, b1);
+        if (two) mma_bf16_16816(s[n][1], k1, b2, b3);
+      }
     }
     const int key0 = runs.block(s_lo + warp + kWarps * i) * kBS;
-    float x0 = -INFINITY, x1 = -INFINITY;
+    const bool full = all_visible(key0, pos, pos, a.window, a.keep_first);
+    const bool see0 = full || visible(key0 + gi, pos, a.window, a.keep_first);
+    const bool see1 = full || visible(key0 + gi + 8, pos, a.window, a.keep_first);
+    uint32_t ph[NT][2], plo[NT][2];
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
+    for (int n = 0; n < NT; ++n) {
+      float p[4];
 #pragma unroll
-      for (int c = 0; c < 2; ++c) {
-        const bool vis = visible(key0 + n * 8 + 2 * t + c, pos, a.window, a.keep_first);
-        s[n][c] = vis ? s[n][c] * sc : -INFINITY;
-        s[n][2 + c] = vis ? s[n][2 + c] * sc : -INFINITY;
-        x0 = fmaxf(x0, s[n][c]);
-        x1 = fmaxf(x1, s[n][2 + c]);
+      for (int e = 0; e < 4; ++e) p[e] = (e < 2 ? see0 : see1) ? (s[n][0][e] + s[n][1][e]) * sc : -INFINITY;
+      float x0 = fmaxf(p[0], p[2]), x1 = fmaxf(p[1], p[3]);
+#pragma unroll
+      for (int w = 4; w < 32; w <<= 1) {
+        x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, w));
+        x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, w));
       }
-    x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 1)); x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 2));
-    x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 1)); x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
-    const float n0 = fmaxf(m0, x0), n1 = fmaxf(m1, x1);
-    const float e0 = n0 == -INFINITY ? 0.f : n0, e1 = n1 == -INFINITY ? 0.f : n1;
-    const float al0 = exp2f(m0 - e0), al1 = exp2f(m1 - e1);
-    m0 = n0; m1 = n1;
-    l0 *= al0; l1 *= al1;
+      const float n0 = fmaxf(m[n][0], x0), n1 = fmaxf(m[n][1], x1);
+      const float e0 = n0 == -INFINITY ? 0.f : n0, e1 = n1 == -INFINITY ? 0.f : n1;
+      if (__any_sync(0xffffffffu, n0 != m[n][0] || n1 != m[n][1])) {
+        const float al0 = ex2(m[n][0] - e0), al1 = ex2(m[n][1] - e1);
+        m[n][0] = n0; m[n][1] = n1;
+        l[n][0] *= al0; l[n][1] *= al1;
 #pragma unroll
-    for (int n = 0; n < 2 * NV; ++n) { o[n][0] *= al0; o[n][1] *= al0; o[n][2] *= al1; o[n][3] *= al1; }
-#pragma unroll
-    for (int n = 0; n < 2; ++n) {
-      s[n][0] = exp2f(s[n][0] - e0); s[n][1] = exp2f(s[n][1] - e0);
-      s[n][2] = exp2f(s[n][2] - e1); s[n][3] = exp2f(s[n][3] - e1);
-      l0 += s[n][0] + s[n][1];
-      l1 += s[n][2] + s[n][3];
+        for (int k = 0; k < MT; ++k) { o[n][k][0] *= al0; o[n][k][1] *= al1; o[n][k][2] *= al0; o[n][k][3] *= al1; }
+      }
+      p[0] = ex2(p[0] - e0); p[1] = ex2(p[1] - e1);
+      p[2] = ex2(p[2] - e0); p[3] = ex2(p[3] - e1);
+      l[n][0] += p[0] + p[2];
+      l[n][1] += p[1] + p[3];
+      uint32_t h0, g0, h1, g1;
+      split_bf16(p[0], p[1], h0, g0);
+      split_bf16(p[2], p[3], h1, g1);
+      ph[n][0] = transpose_8x8(h0); ph[n][1] = transpose_8x8(h1);
+      plo[n][0] = transpose_8x8(g0); plo[n][1] = transpose_8x8(g1);
     }
-    uint32_t hi[4], lo[4];
-    split_bf16(s[0][0], s[0][1], hi[0], lo[0]);
-    split_bf16(s[0][2], s[0][3], hi[1], lo[1]);
-    split_bf16(s[1][0], s[1][1], hi[2], lo[2]);
-    split_bf16(s[1][2], s[1][3], hi[3], lo[3]);
-    const uint32_t v_addr = smem_u32(vt + (lane & 15) * VS + (lane >> 4) * 8);
 #pragma unroll
-    for (int nv = 0; nv < NV; ++nv) {
-      if (nv * 16 < VP) {
-        uint32_t b0, b1, b2, b3;
-        ldsm_x4_trans(v_addr + nv * 32, b0, b1, b2, b3);
-        mma_bf16_16816(o[2 * nv], hi, b0, b1);
-        mma_bf16_16816(o[2 * nv + 1], hi, b2, b3);
-        mma_bf16_16816(o[2 * nv], lo, b0, b1);
-        mma_bf16_16816(o[2 * nv + 1], lo, b2, b3);
+    for (int k = 0; k < MT; ++k) {
+      if (k * 16 < VP) {
+        uint32_t va[4];
+        ldsm_x4_trans(base + v_off + k * 32, va[0], va[1], va[2], va[3]);
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+          mma_bf16_16816(o[n][k], va, ph[n][0], ph[n][1]);
+          mma_bf16_16816(o[n][k], va, plo[n][0], plo[n][1]);
+        }
       }
     }
     __syncwarp();  // the stage is refilled by the next iteration's load
   }
   cp_async_wait<0>();
   pdl_trigger();
-  l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
-  l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
   // the warps' results meet in shared memory (the rings are idle now)
   __syncthreads();
   const int OS = VP + 2;
   float* s_o = (float*)(s_q + 16 * KS);          // [kWarps][R][OS]
   float* s_ml = s_o + (size_t)kWarps * R * OS;   // [kWarps][R][2]
-  auto put = [&](int m, float mm, float ll, int half) {
-    if (m >= R) return;
-    float* dst = s_o + ((size_t)warp * R + m) * OS;
 #pragma unroll
-    for (int n = 0; n < 2 * NV; ++n)
-      if (n * 8 < VP) *reinterpret_cast<float2*>(dst + n * 8 + 2 * t) = make_float2(o[n][half], o[n][half + 1]);
-    if (t == 0) { s_ml[(warp * R + m) * 2] = mm; s_ml[(warp * R + m) * 2 + 1] = ll; }
-  };
-  put(gi, m0, l0, 0);
-  put(gi + 8, m1, l1, 2);
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+      float ll = l[n][c];
+#pragma unroll
+      for (int w = 4; w < 32; w <<= 1) ll += __shfl_xor_sync(0xffffffffu, ll, w);
+      const int head = n * 8 + 2 * t + c;
+      if (head < R) {
+        float* dst = s_o + ((size_t)warp * R + head) * OS;
+#pragma unroll
+        for (int k = 0; k < MT; ++k)
+          if (k * 16 < VP) { dst[k * 16 + gi] = o[n][k][c]; dst[k * 16 + gi + 8] = o[n][k][2 + c]; }
+        if (gi == 0) { s_ml[(warp * R + head) * 2] = m[n][c]; s_ml[(warp * R + head) * 2 + 1] = ll; }
+      }
+    }
   __syncthreads();
-  for (int i = tid; i < R * VW; i += kThreads) {
-    const int m = i / VW, c = i % VW;
-    float mx = -INFINITY, l = 0.f, acc = 0.f;
+  for (int h = warp; h < R; h += kWarps) {
+    float mx = -INFINITY, ls = 0.f, f[kWarps];
 #pragma unroll
-    for (int w = 0; w < kWarps; ++w) mx = fmaxf(mx, s_ml[(w * R + m) * 2]);
+    for (int w = 0; w < kWarps; ++w) mx = fmaxf(mx, s_ml[(w * R + h) * 2]);
 #pragma unroll
     for (int w = 0; w < kWarps; ++w) {
-      const float mw = s_ml[(w * R + m) * 2];
-      const float f = mw == -INFINITY ? 0.f : exp2f(mw - mx);
-      l = fmaf(f, s_ml[(w * R + m) * 2 + 1], l);
-      acc = fmaf(f, s_o[((size_t)w * R + m) * OS + c], acc);
+      const float mw = s_ml[(w * R + h) * 2];
+      f[w] = mw == -INFINITY ? 0.f : ex2(mw - mx);
+      ls = fmaf(f[w], s_ml[(w * R + h) * 2 + 1], ls);
     }
-    const int64_t head = (int64_t)kvh * R + m;
-    if (n_splits == 1) {
-      ((__nv_bfloat16*)a.out)[row * a.ld_out + head * a.vdim + v0 + c] = __float2bfloat16_rn(acc / l);
-    } else {
-      float* p = part + (((int64_t)blockIdx.x * a.heads + head) * n_splits + split) * (a.vdim + 2);
-      p[v0 + c] = acc;
-      if (c == 0 && v0 == 0) { p[a.vdim] = mx; p[a.vdim + 1] = l; }
+    const int64_t head = (int64_t)kvh * R + h;
+    float* p = n_splits > 1 ? part + (((int64_t)blockIdx.x * a.heads + head) * n_splits + split) * (a.vdim + 2) : nullptr;
+    for (int c = lane; c < VW; c += 32) {
+      float acc = 0.f;
+#pragma unroll
+      for (int w = 0; w < kWarps; ++w) acc = fmaf(f[w], s_o[((size_t)w * R + h) * OS + c], acc);
+      if (n_splits == 1) ((__nv_bfloat16*)a.out)[row * a.ld_out + head * a.vdim + v0 + c] = __float2bfloat16_rn(acc / ls);
+      else p[v0 + c] = acc;
     }
+    if (n_splits > 1 && lane == 0 && v0 == 0) { p[a.vdim] = mx; p[a.vdim + 1] = ls; }
   }
 }
 
@@ -398,13 +451,13 @@ span_attention_merge_kernel(const SpanAttention a, const int32_t* __restrict__ r
   for (int s = 0; s < n_splits; ++s) mx = fmaxf(mx, p[s * (a.vdim + 2) + a.vdim]);
   for (int s = 0; s < n_splits; ++s) {
     const float m = p[s * (a.vdim + 2) + a.vdim];
-    if (m != -INFINITY) l = fmaf(exp2f(m - mx), p[s * (a.vdim + 2) + a.vdim + 1], l);
+    if (m != -INFINITY) l = fmaf(ex2(m - mx), p[s * (a.vdim + 2) + a.vdim + 1], l);
   }
   for (int c = threadIdx.x; c < a.vdim; c += kThreads) {
     float acc = 0.f;
     for (int s = 0; s < n_splits; ++s) {
       const float m = p[s * (a.vdim + 2) + a.vdim];
-      if (m != -INFINITY) acc = fmaf(exp2f(m - mx), p[s * (a.vdim + 2) + c], acc);
+      if (m != -INFINITY) acc = fmaf(ex2(m - mx), p[s * (a.vdim + 2) + c], acc);
     }
     ((__nv_bfloat16*)a.out)[row * a.ld_out + (int64_t)head * a.vdim + c] = __float2bfloat16_rn(acc / l);
   }
@@ -475,10 +528,10 @@ int span_attention_tokens(cudaStream_t st, const SpanAttention& a, const int32_t
   };
   const int vw = std::min(a.vdim, kSlice);
   int rc;
-  if (vw <= 64) rc = launch(span_attention_tokens_kernel<4>);
-  else if (vw <= 128) rc = launch(span_attention_tokens_kernel<8>);
-  else if (vw <= 192) rc = launch(span_attention_tokens_kernel<12>);
-  else rc = launch(span_attention_tokens_kernel<16>);
+  const bool wide = a.heads / a.kv_heads > 8;
+  if (vw <= 64) rc = wide ? launch(span_attention_tokens_kernel<4, 2>) : launch(span_attention_tokens_kernel<4, 1>);
+  else if (vw <= 128) rc = wide ? launch(span_attention_tokens_kernel<8, 2>) : launch(span_attention_tokens_kernel<8, 1>);
+  else rc = wide ? launch(span_attention_tokens_kernel<16, 2>) : launch(span_attention_tokens_kernel<16, 1>);
   if (rc || n_splits == 1) return rc;
   HB_CUDA_CHECK(launch_pdl(span_attention_merge_kernel, dim3((unsigned)n_rows, (unsigned)a.heads), dim3(kThreads), 0, st, a, rows,
                            n_splits, (const float*)part));

@@ -45,6 +45,19 @@ __device__ __forceinline__ void mma_split(float (&d)[4], const uint32_t (&ahi)[4
   mma_bf16_16816(d, ahi, bl0, bl1);
 }
 
+// 2^x in one instruction (ex2.approx, about 2 ulp)
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// Transposes an 8x8 matrix of 16-bit elements held one row of pairs per four lanes.
+__device__ __forceinline__ uint32_t transpose_8x8(uint32_t v) {
+  uint32_t r;
+  asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
+  return r;
+}
+
 __device__ __forceinline__ void cp_async_16(uint32_t dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
 }

@@ -7,38 +7,36 @@
 namespace hb {
 
 constexpr int kRecThreads = 256;
-constexpr int kRecCols = 64;  // state columns of a CTA
-
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 // log(sigmoid(z)) without cancellation on either side
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
-// log of the decay of key channel c = head * dim + d, from the row's low-rank input s_t
+// log of the decay of key channel c = head * dim + d, from the row's low-rank input t
 template <typename T>
-__device__ __forceinline__ float low_rank_log_decay(const Recurrence& a, const float* s_t, int c) {
+__device__ __forceinline__ float low_rank_log_decay(const Recurrence& a, const T* t, int c) {
   float z = a.a2_bias[c];
   const float* w = a.a2 + (int64_t)c * a.rank;
-  for (int r = 0; r < a.rank; ++r) z = fmaf(w[r], s_t[r], z);
+#pragma unroll 8
+  for (int r = 0; r < a.rank; ++r) z = fmaf(w[r], to_f32<T>(t[r]), z);
   return log_sigmoid(z) * a.inv_tau;
 }
 
-// CTA = (segment, head, 64 state columns).  A thread owns VEC neighbouring columns of every
+// CTA = (segment, head, COLS state columns).  A thread owns VEC neighbouring columns of every
 // DG-th state row, so its part of the state never meets another thread's; only the output needs
 // a sum over the row groups.  RPT > 0: the thread's rows stay in registers for the whole segment.
-template <typename T, int VEC, int RPT>
-__global__ void __launch_bounds__(kRecThreads, RPT == 4 ? 5 : RPT == 8 ? 4 : 1)
+template <typename T, int COLS, int VEC, int RPT>
+__global__ void __launch_bounds__(kRecThreads, RPT > 0 ? 4 : 1)
 recurrence_tokens_kernel(const Recurrence a, const int32_t* __restrict__ list) {
-  constexpr int LANES = kRecCols / VEC, DG = kRecThreads / LANES;
+  constexpr int LANES = COLS / VEC, DG = kRecThreads / LANES;
   extern __shared__ float sm[];
   const int D = a.dim, VD = a.vdim;
   float* s_q = sm;               // [D]
   float* s_k = s_q + D;          // [D]
   float* s_a = s_k + D;          // [D]
-  float* s_t = s_a + D;          // [rank]
-  __shared__ float s_v[kRecCols];
-  __shared__ float s_o[DG][kRecCols];
+  __shared__ float s_v[COLS];
+  __shared__ float s_o[DG][COLS];
   const int tid = threadIdx.x, col = tid % LANES * VEC, dg = tid / LANES, h = blockIdx.y;
-  const int v0 = blockIdx.z * kRecCols;
+  const int v0 = blockIdx.z * COLS;
   pdl_grid_wait();
   const SegInfo seg = a.segs[list[blockIdx.x]];
   float* state = a.state + ((int64_t)seg.slot * a.heads + h) * D * VD + v0 + col;
@@ -68,20 +66,21 @@ recurrence_tokens_kernel(const Recurrence a, const int32_t* __restrict__ list) {
   for (int t = 0; t < seg.n; ++t) {
     const int64_t row = seg.row0 + t;
     const T* p = (const T*)a.p + row * a.ld;
-    if (!a.decay) {
-      for (int i = tid; i < a.rank; i += kRecThreads) s_t[i] = to_f32<T>(p[a.off_a1 + i]);
-      __syncthreads();
-    }
-    for (int d = tid; d < D; d += kRecThreads) {
-      float q = to_f32<T>(p[a.off_q + h * D + d]), k = to_f32<T>(p[a.off_k + h * D + d]);
-      if (a.silu_qkv) { q = silu_f(q); k = silu_f(k); }
-      s_q[d] = q * a.q_scale;
-      s_k[d] = k;
-      s_a[d] = a.decay ? a.decay[h] : expf(low_rank_log_decay<T>(a, s_t, h * D + d));
-    }
-    for (int i = tid; i < kRecCols; i += kRecThreads) {
-      float v = v0 + i < VD ? to_f32<T>(p[a.off_v + h * VD + v0 + i]) : 0.f;
-      s_v[i] = a.silu_qkv ? silu_f(v) : v;
+    // every kind of input has threads of its own: decays, then q and k, then v
+    for (int i = tid; i < 2 * D + COLS; i += kRecThreads) {
+      if (i < D) {
+        s_a[i] = a.decay ? a.decay[h] : expf(low_rank_log_decay<T>(a, p + a.off_a1, h * D + i));
+      } else if (i < 2 * D) {
+        const int d = i - D;
+        float q = to_f32<T>(p[a.off_q + h * D + d]), k = to_f32<T>(p[a.off_k + h * D + d]);
+        if (a.silu_qkv) { q = silu_f(q); k = silu_f(k); }
+        s_q[d] = q * a.q_scale;
+        s_k[d] = k;
+      } else {
+        const int c = i - 2 * D;
+        const float v = v0 + c < VD ? to_f32<T>(p[a.off_v + h * VD + v0 + c]) : 0.f;
+        s_v[c] = a.silu_qkv ? silu_f(v) : v;
+      }
     }
     __syncthreads();
     float vv[VEC], acc[VEC];
@@ -119,7 +118,7 @@ recurrence_tokens_kernel(const Recurrence a, const int32_t* __restrict__ list) {
 #pragma unroll
     for (int j = 0; j < VEC; ++j) s_o[dg][col + j] = acc[j];
     __syncthreads();
-    for (int i = tid; i < kRecCols; i += kRecThreads) {
+    for (int i = tid; i < COLS; i += kRecThreads) {
       float o = 0.f;
 #pragma unroll
       for (int g = 0; g < DG; ++g) o += s_o[g][i];
@@ -139,21 +138,23 @@ recurrence_tokens_kernel(const Recurrence a, const int32_t* __restrict__ list) {
 
 int recurrence_tokens(cudaStream_t st, const Recurrence& a, const int32_t* list, int n_list, hb_dtype dtype) {
   if (n_list == 0) return HB_OK;
-  const dim3 grid((unsigned)n_list, (unsigned)a.heads, (unsigned)((a.vdim + kRecCols - 1) / kRecCols));
-  const size_t smem = ((size_t)3 * a.dim + a.rank) * sizeof(float);
-  auto launch = [&](auto* kernel) -> int {
+  const size_t smem = (size_t)3 * a.dim * sizeof(float);
+  auto launch = [&](auto* kernel, int cols) -> int {
+    const dim3 grid((unsigned)n_list, (unsigned)a.heads, (unsigned)((a.vdim + cols - 1) / cols));
     HB_CUDA_CHECK(launch_pdl(kernel, grid, dim3(kRecThreads), smem, st, a, list));
     return HB_OK;
   };
+  // about 32 KB of state per CTA in registers: enough loads in flight to stream it
   const bool vec = a.vdim % 4 == 0;
   if (dtype == HB_F32) {
-    if (!vec) return launch(recurrence_tokens_kernel<float, 1, 0>);
-    return a.dim <= 128 ? launch(recurrence_tokens_kernel<float, 4, 8>) : launch(recurrence_tokens_kernel<float, 4, 0>);
+    if (!vec) return launch(recurrence_tokens_kernel<float, 64, 1, 0>, 64);
+    return a.dim <= 128 ? launch(recurrence_tokens_kernel<float, 64, 4, 8>, 64) : launch(recurrence_tokens_kernel<float, 64, 4, 0>, 64);
   }
   if (dtype == HB_BF16) {
-    if (!vec) return launch(recurrence_tokens_kernel<__nv_bfloat16, 1, 0>);
-    if (a.dim <= 64) return launch(recurrence_tokens_kernel<__nv_bfloat16, 4, 4>);
-    return a.dim <= 128 ? launch(recurrence_tokens_kernel<__nv_bfloat16, 4, 8>) : launch(recurrence_tokens_kernel<__nv_bfloat16, 4, 0>);
+    if (!vec) return launch(recurrence_tokens_kernel<__nv_bfloat16, 64, 1, 0>, 64);
+    if (a.dim <= 64 && a.vdim > 64) return launch(recurrence_tokens_kernel<__nv_bfloat16, 128, 4, 8>, 128);
+    return a.dim <= 128 ? launch(recurrence_tokens_kernel<__nv_bfloat16, 64, 4, 8>, 64)
+                        : launch(recurrence_tokens_kernel<__nv_bfloat16, 64, 4, 0>, 64);
   }
   return fail(HB_ERR_UNSUPPORTED_DTYPE, "recurrence runs in bf16 or f32");
 }

@@ -8,6 +8,8 @@
 namespace hb {
 
 constexpr int kStreamThreads = 256;
+constexpr int kWideThreads = 512;   // few rows (decoding): more loads in flight per row
+constexpr int kFewRows = 592;
 
 template <typename T, int VEC>
 __device__ __forceinline__ void load_vec(float (&f)[VEC], const T* p);
@@ -84,20 +86,20 @@ streams_embed_kernel(float* __restrict__ x, T* __restrict__ h, const T* __restri
 }
 
 template <typename T, int VEC, int NS, bool TWO>
-__global__ void __launch_bounds__(kStreamThreads)
+__global__ void __launch_bounds__(NS <= 4 ? kWideThreads : kStreamThreads)
 streams_mix_kernel(float* __restrict__ x, T* __restrict__ h, const float* __restrict__ y, const float* __restrict__ y2,
                    int64_t ld_y, StreamMix m, int S, int64_t W, int64_t ld_h, float eps) {
   pdl_trigger();
   extern __shared__ float s_u[];  // [W] the next sublayer's input before its norm
   __shared__ float red[33];
   __shared__ float s_mix[NS][NS], s_out[NS], s_in[NS];
-  const int tid = threadIdx.x;
+  const int tid = threadIdx.x, threads = blockDim.x;
   // mixing weights are parameters: they may be read before the producing kernel has finished
-  for (int i = tid; i < NS * NS; i += kStreamThreads) {
+  for (int i = tid; i < NS * NS; i += threads) {
     const int a = i / NS, b = i % NS;
     s_mix[a][b] = (a < S && b < S) ? m.mix[a * S + b] : 0.f;
   }
-  for (int i = tid; i < NS; i += kStreamThreads) {
+  for (int i = tid; i < NS; i += threads) {
     s_out[i] = i < S ? m.out[i] : 0.f;
     s_in[i] = (i < S && m.next_norm) ? m.next_in[i] : 0.f;
   }
@@ -108,7 +110,7 @@ streams_mix_kernel(float* __restrict__ x, T* __restrict__ h, const float* __rest
   float r1 = 0.f, r2 = 0.f;
   if (TWO) {
     float a1 = 0.f, a2 = 0.f;
-    for (int64_t i = (int64_t)tid * VEC; i < W; i += kStreamThreads * VEC) {
+    for (int64_t i = (int64_t)tid * VEC; i < W; i += threads * VEC) {
       float f[VEC], g[VEC];
       load_vec<float, VEC>(f, yr + i);
       load_vec<float, VEC>(g, y2r + i);
@@ -125,7 +127,7 @@ streams_mix_kernel(float* __restrict__ x, T* __restrict__ h, const float* __rest
   }
   float* xr = x + row * S * W;
   float ss = 0.f;
-  for (int64_t i = (int64_t)tid * VEC; i < W; i += kStreamThreads * VEC) {
+  for (int64_t i = (int64_t)tid * VEC; i < W; i += threads * VEC) {
     float xs[NS][VEC], f[VEC];
 #pragma unroll
     for (int s = 0; s < NS; ++s) {
@@ -168,7 +170,7 @@ streams_mix_kernel(float* __restrict__ x, T* __restrict__ h, const float* __rest
   }
   if (!m.next_norm) return;
   const float r = inv_rms(block_sum(ss, red), W, eps);
-  for (int64_t i = (int64_t)tid * VEC; i < W; i += kStreamThreads * VEC) {
+  for (int64_t i = (int64_t)tid * VEC; i < W; i += threads * VEC) {
     float u[VEC], w[VEC];
     load_vec<float, VEC>(u, s_u + i);  // written by this thread
     load_vec<float, VEC>(w, m.next_norm + i);
@@ -214,7 +216,7 @@ streams_final_kernel(T* __restrict__ h, const float* __restrict__ x, const int32
 
 // Groups of up to a warp's worth of work are normed by one warp each; a single wide group by the
 // whole CTA.
-template <typename T, bool WARP>
+template <typename T, bool WARP, int VEC>
 __global__ void __launch_bounds__(kStreamThreads)
 gated_group_norm_kernel(T* __restrict__ out, int64_t ld_out, const float* __restrict__ o, int64_t ld_o,
                         const T* __restrict__ gate, int64_t ld_gate, const float* __restrict__ weight, int groups, int size,
@@ -223,22 +225,36 @@ gated_group_norm_kernel(T* __restrict__ out, int64_t ld_out, const float* __rest
   pdl_grid_wait();
   __shared__ float red[33];
   const int64_t row = blockIdx.x;
-  const float* orow = o + row * ld_o;
-  const T* grow = gate + row * ld_gate;
-  T* outr = out + row * ld_out;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int first = WARP ? blockIdx.y * (kStreamThreads / 32) + warp : blockIdx.y;
-  const int lane_i = WARP ? lane : (int)threadIdx.x, step = WARP ? 32 : kStreamThreads;
-  if (WARP && first >= groups) return;
-  const float* og = orow + (int64_t)first * size;
+  const int group = WARP ? blockIdx.y * (kStreamThreads / 32) + warp : blockIdx.y;
+  const int first = (WARP ? lane : (int)threadIdx.x) * VEC, step = (WARP ? 32 : kStreamThreads) * VEC;
+  if (WARP && group >= groups) return;
+  const int64_t at = (int64_t)group * size;
+  const float* og = o + row * ld_o + at;
+  const T* gg = gate + row * ld_gate + at;
+  T* dst = out + row * ld_out + at;
   float ss = 0.f;
-  for (int i = lane_i; i < size; i += step) ss = fmaf(og[i], og[i], ss);
+#pragma unroll 4
+  for (int i = first; i < size; i += step) {
+    float f[VEC];
+    load_vec<float, VEC>(f, og + i);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) ss = fmaf(f[j], f[j], ss);
+  }
   ss = WARP ? warp_sum(ss) : block_sum(ss, red);
   const float r = inv_rms(ss, size, eps);
-  for (int i = lane_i; i < size; i += step) {
-    const float g = to_f32<T>(grow[(int64_t)first * size + i]);
-    const float sg = 1.f / (1.f + expf(-g));
-    outr[(int64_t)first * size + i] = from_f32<T>(og[i] * r * weight[i] * (gate_silu ? g * sg : sg));
+#pragma unroll 2
+  for (int i = first; i < size; i += step) {
+    float f[VEC], g[VEC], w[VEC];
+    load_vec<float, VEC>(f, og + i);
+    load_vec<T, VEC>(g, gg + i);
+    load_vec<float, VEC>(w, weight + i);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+      const float sg = 1.f / (1.f + expf(-g[j]));
+      f[j] = f[j] * r * w[j] * (gate_silu ? g[j] * sg : sg);
+    }
+    store_vec<T, VEC>(dst + i, f);
   }
 }
 
@@ -261,10 +277,21 @@ int streams_embed(cudaStream_t st, float* x, void* h, const void* embed, const v
   return HB_OK;
 }
 
+// The row's sublayer input waits for its norm in shared memory; rows above 48 KB need the opt-in.
+template <typename K>
+static int row_smem(K kernel, int64_t width) {
+  if (width * 4 > 200 * 1024) return fail(HB_ERR_INVALID_ARG, "a width of %lld is not supported", (long long)width);
+  if (width * 4 > 47 * 1024) HB_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+  return HB_OK;
+}
+
 template <typename T, int VEC, int NS, bool TWO>
 static int launch_mix(cudaStream_t st, float* x, void* h, const float* y, const float* y2, int64_t ld_y, const StreamMix& m,
                       int64_t rows, int streams, int64_t width, int64_t ld_h, float eps) {
-  HB_CUDA_CHECK(launch_pdl(streams_mix_kernel<T, VEC, NS, TWO>, dim3((unsigned)rows), dim3(kStreamThreads),
+  const int threads = NS <= 4 && rows <= kFewRows && width >= kWideThreads * VEC ? kWideThreads : kStreamThreads;
+  const int rc = row_smem(streams_mix_kernel<T, VEC, NS, TWO>, width);
+  if (rc) return rc;
+  HB_CUDA_CHECK(launch_pdl(streams_mix_kernel<T, VEC, NS, TWO>, dim3((unsigned)rows), dim3((unsigned)threads),
                            (size_t)width * 4, st, x, (T*)h, y, y2, ld_y, m, streams, width, ld_h, eps));
   return HB_OK;
 }
@@ -296,6 +323,8 @@ int streams_final(cudaStream_t st, void* h, const float* x, const int32_t* want,
   if (n_want == 0) return HB_OK;
   HB_DISPATCH_LAYERED(dtype, T, {
     auto* k = width % 4 == 0 ? streams_final_kernel<T, 4> : streams_final_kernel<T, 1>;
+    const int rc = row_smem(k, width);
+    if (rc) return rc;
     HB_CUDA_CHECK(launch_pdl(k, dim3((unsigned)n_want), dim3(kStreamThreads), (size_t)width * 4, st, (T*)h, x, want, norm,
                              streams, width, ld_h, eps));
   });
@@ -308,7 +337,11 @@ int gated_group_norm(cudaStream_t st, void* out, int64_t ld_out, const float* o,
   const bool warp = groups > 1 && size <= 1024;
   const unsigned gy = warp ? (unsigned)((groups + kStreamThreads / 32 - 1) / (kStreamThreads / 32)) : (unsigned)groups;
   HB_DISPATCH_LAYERED(dtype, T, {
-    auto* k = warp ? gated_group_norm_kernel<T, true> : gated_group_norm_kernel<T, false>;
+    const uintptr_t bits = (uintptr_t)o | (uintptr_t)weight | ((uintptr_t)gate * (16 / (4 * sizeof(T)))) |
+                           ((uintptr_t)out * (16 / (4 * sizeof(T))));
+    const bool vec = (bits & 15) == 0 && size % 4 == 0 && ld_o % 4 == 0 && ld_gate % 4 == 0 && ld_out % 4 == 0;
+    auto* k = vec ? (warp ? gated_group_norm_kernel<T, true, 4> : gated_group_norm_kernel<T, false, 4>)
+                  : (warp ? gated_group_norm_kernel<T, true, 1> : gated_group_norm_kernel<T, false, 1>);
     HB_CUDA_CHECK(launch_pdl(k, dim3((unsigned)rows, gy), dim3(kStreamThreads), 0, st, (T*)out, ld_out, o, ld_o,
                              (const T*)gate, ld_gate, weight, groups, size, gate_silu ? 1 : 0, eps));
   });
