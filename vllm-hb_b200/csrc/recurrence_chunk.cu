@@ -159,13 +159,13 @@ recurrence_state_kernel(const Recurrence a, const RowRange* __restrict__ chunks,
     const bool live = j < ch.n;
     ld_proj8(k, a, ch.row0 + min(j, ch.n - 1), a.off_k + h * D + d, live ? D - d : 0);
     if (live) {
-      const float f = a.decay ? exp2f(log2_pow(ld2, ch.n - 1 - j)) : 1.f;
+      const float f = a.decay ? ex2(log2_pow(ld2, ch.n - 1 - j)) : 1.f;
       const float* end = cum + (int64_t)(ch.row0 + ch.n - 1) * hd + h * D + d;
       const float* own = cum + (int64_t)(ch.row0 + j) * hd + h * D + d;
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
         if (a.silu_qkv) k[e] = rec_silu(k[e]);
-        k[e] *= a.decay ? f : (d + e < D ? exp2f(end[e] - own[e]) : 0.f);
+        k[e] *= a.decay ? f : (d + e < D ? ex2(end[e] - own[e]) : 0.f);
       }
     }
     put_split8(k_hi + j * KS + d, k_lo + j * KS + d, k);
@@ -248,7 +248,7 @@ recurrence_scan_kernel(const Recurrence a, const RowRange* __restrict__ segs, co
       if (c0 + c < sg.n) {
         if (VEC == 4) *reinterpret_cast<float4*>(u + c * stride) = make_float4(s[0], s[1 % VEC], s[2 % VEC], s[3 % VEC]);
         else u[c * stride] = s[0];
-        const float k = exp2f(f[c]);
+        const float k = ex2(f[c]);
 #pragma unroll
         for (int j = 0; j < VEC; ++j) s[j] = fmaf(k, s[j], v[c][j]);
       }
@@ -305,7 +305,7 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
       put8(k_raw + j * KS + d, k);
       const float *end = s_b + (j | 15) * BS + d, *own = s_b + j * BS + d;
 #pragma unroll
-      for (int e = 0; e < 8; ++e) k[e] *= exp2f(end[e] - own[e]);
+      for (int e = 0; e < 8; ++e) k[e] *= ex2(end[e] - own[e]);
       put_split8(k_hi + j * KS + d, k_lo + j * KS + d, k);
     } else {
       put_split8(q_hi + j * KS + d, q_lo + j * KS + d, q);
@@ -334,7 +334,7 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
       for (int r = 0; r < 2; ++r) {
         const int i = r ? i1 : i0;
         const __nv_bfloat162 q2 = *reinterpret_cast<const __nv_bfloat162*>(q_hi + i * KS + d);
-        split_bf16(__low2float(q2) * exp2f(s_b[i * BS + d] - e0), __high2float(q2) * exp2f(s_b[i * BS + d + 1] - e1),
+        split_bf16(__low2float(q2) * ex2(s_b[i * BS + d] - e0), __high2float(q2) * ex2(s_b[i * BS + d + 1] - e1),
                    hi[half * 2 + r], lo[half * 2 + r]);
       }
     }
@@ -357,7 +357,8 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
       }
     }
     if (LR && nb == warp) {
-      // inside the block the decay differs per pair: fp32 on CUDA cores.  Keys 8-15 of the block never
+      // inside the block the decay differs per pair: fp32 on CUDA cores (pairs with j > i are dropped
+      // below, whatever their exponential is).  Keys 8-15 of the block never
       // meet queries 0-7.
       float p[8];
 #pragma unroll
@@ -369,8 +370,8 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
       };
       auto fl2 = [](const float* p2) { return *reinterpret_cast<const float2*>(p2); };
       auto pair = [](float& acc, float2 q, float2 k, float2 bi, float2 bj) {
-        acc = fmaf(q.x * k.x, exp2f(fminf(bi.x - bj.x, 0.f)), acc);
-        acc = fmaf(q.y * k.y, exp2f(fminf(bi.y - bj.y, 0.f)), acc);
+        acc = fmaf(q.x * k.x, ex2(bi.x - bj.x), acc);
+        acc = fmaf(q.y * k.y, ex2(bi.y - bj.y), acc);
       };
       for (int d = 0; d < D; d += 2) {  // channels past D are zero
         const float2 b0 = fl2(s_b + i0 * BS + d), b1 = fl2(s_b + i1 * BS + d);
@@ -394,7 +395,7 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
     for (int e = 0; e < 4; ++e) {
       const int i = e < 2 ? i0 : i1, j = n * 8 + 2 * t + (e & 1);
       if (j > i) s[n][e] = 0.f;
-      else if (!LR) s[n][e] *= exp2f(log2_pow(ld2, i - j));
+      else if (!LR) s[n][e] *= ex2(log2_pow(ld2, i - j));
     }
   __syncthreads();  // keys are done with: their memory holds the tiles of phase two
 
@@ -404,7 +405,7 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
   bf16* t_lo = t_hi + kC * kVS;
   const uint32_t vh = smem_u32(v_hi + (lane & 15) * kVS + (lane >> 4) * 8), vl = smem_u32(v_lo + (lane & 15) * kVS + (lane >> 4) * 8);
   const uint32_t th = smem_u32(t_hi + (lane & 15) * kVS + (lane >> 4) * 8), tl = smem_u32(t_lo + (lane & 15) * kVS + (lane >> 4) * 8);
-  const float f0 = LR ? 1.f : exp2f(log2_pow(ld2, i0 + 1)), f1 = LR ? 1.f : exp2f(log2_pow(ld2, i1 + 1));
+  const float f0 = LR ? 1.f : ex2(log2_pow(ld2, i0 + 1)), f1 = LR ? 1.f : ex2(log2_pow(ld2, i1 + 1));
   const float* st = chunk_state + ((int64_t)blockIdx.x * a.heads + h) * D * a.vdim;
   const bool live = warp * 16 < ch.n;
   for (int v0 = 0; v0 < a.vdim; v0 += kVT) {
