@@ -40,6 +40,9 @@ CONFIGS = {
     "one": (model(64, 48, 1, [par(1, 1, 32, 8, 0.5, (1, 1), 1, 32, 32, [0.8], 64), gla(1, 32, 64, 1.0, 64)]), 1),
     "wide": (model(128, 200, 4, [par(8, 1, 128, 256, 0.09, (70, 20), 2, 128, 72, [0.6, 0.999], 264), gla(2, 136, 80, 16.0, 128),
                                  par(2, 2, 64, 320, 0.12, None, 4, 16, 16, [0.99, 0.9, 0.7, 0.1], 40)]), 8),
+    # split-K plans whose last K chunk and last feature tile are ragged
+    "broad": (model(520, 1001, 3, [par(6, 2, 48, 80, 0.15, (64, 16), 3, 40, 56, [0.9, 0.99, 0.5], 1100),
+                                   gla(5, 40, 104, 8.0, 1100)]), 12),
     "many": (model(72, 56, 6, [gla(2, 16, 16, 2.0, 40), gla(2, 16, 16, 3.0, 40),
                                par(20, 1, 8, 16, 0.4, (40, 3), 1, 8, 8, [0.95], 40)]), 3),
 }
@@ -106,7 +109,7 @@ def test_whole_prompt(hb, cuda, models, name, dtype):
     eng = load(hb, models[name][2], dtype)
     assert eng.num_layers() == len(models[name][0]["layers"]) and eng.hidden_size() == models[name][0]["width"]
     assert eng.param_count() == sum(v.size for v in models[name][1].values())
-    for n in (1, 2, 17, 230):
+    for n in (1, 2, 17, 301):
         toks = prompt(models, name, n, n)
         seq = eng.create_kv_cache()
         check(feed(eng, seq, toks, [n]), expected(models, name, toks), dtype, n)
