@@ -232,7 +232,13 @@ int hb_sample(void* stream, uint32_t* tokens, float* probs_workspace, const floa
  * one sequence.  Ranges are int32 quadruples in device memory. */
 
 /* Paged attention whose queries at position p see the keys j <= p with p - j < window
- * (window 0: all) or j < keep_first; keys and values may differ in width.
+ * (window 0: all) or j < keep_first, or with chunk > 0 those of their own chunk
+ * (p / chunk == j / chunk); keys and values may differ in width.  Optional (NULL / 0: none):
+ * dist_bias [heads, dist_len] is added to the scaled score by distance (the last entry also beyond
+ * it); sink [heads] is the score of one more softmax member without a value; gate: the output is
+ * multiplied by sigmoid(gate), row r, head h at gate + r*ld_gate + h*vdim (`dtype`);
+ * key_scale [num_blocks*16]: the K pool holds the values too (v_cache unused, vdim == dim) and a key
+ * is its value times the scale of its slot.
  * q row r, head h at q + r*ld_q + h*dim; out likewise with vdim; K pool [num_blocks, kv_heads, 16,
  * dim], V pool [num_blocks, kv_heads, 16, vdim]; softmax(scale * q.k) v, scores and weights in fp32.
  * tiles {segment, first row, rows, -}: up to hb_span_attention_tile_positions() consecutive
@@ -250,6 +256,13 @@ typedef struct hb_span_attention_args {
   const int32_t* positions;
   int heads, kv_heads, dim, vdim, window, keep_first;
   float scale;
+  int chunk;
+  const float* key_scale;
+  const float* dist_bias;
+  int dist_len;
+  const float* sink;
+  const void* gate;
+  int64_t ld_gate;
 } hb_span_attention_args;
 int hb_span_attention_tile_positions(const hb_span_attention_args* a, hb_dtype dtype);
 int hb_span_attention(void* stream, const hb_span_attention_args* a, const int32_t* tiles, int n_tiles, const int32_t* rows,
@@ -257,6 +270,58 @@ int hb_span_attention(void* stream, const hb_span_attention_args* a, const int32
 /* K and V rows (stride ld elements) to their slots (block*16 + offset; negative: skipped). */
 int hb_span_kv_write(void* stream, const hb_span_attention_args* a, const void* k, const void* v, int64_t ld,
                      const int64_t* slots, int64_t rows, hb_dtype dtype);
+
+/* From projection rows (queries, keys, values at column offsets of p) to queries in their place and
+ * keys and values in their slots: biases [heads*dim], [kv_heads*dim] added; then either RMS norms
+ * over all query and all key rows (weights q_norm, k_norm) or a rotation of the first 2*pairs
+ * channels of every head, channel 2i with 2i+1, by position * rotation[i].  With key_scale the K pool
+ * takes the keys before their norm, key_scale[slot] the factor of the norm, and the queries are
+ * multiplied by k_norm (hb_span_attention's key_scale).  fp32 inside. */
+typedef struct hb_attention_prep_args {
+  void* p;
+  int64_t ld;
+  int off_q, off_k, off_v, heads, kv_heads, dim, vdim;
+  const int32_t* positions;
+  const int64_t* slots; /* block*16 + offset; negative: skipped */
+  void *k_cache, *v_cache;
+  int64_t num_blocks;
+  const float *q_bias, *k_bias, *q_norm, *k_norm;
+  float eps;
+  const double* rotation;
+  int pairs;
+  float* key_scale;
+} hb_attention_prep_args;
+int hb_attention_prepare(void* stream, const hb_attention_prep_args* a, int64_t rows, hb_dtype dtype);
+
+/* Mixture of experts, every expert on its own rows only.
+ * hb_moe_route_top: logits h . router^T + bias [experts] in fp32, the `top` largest per row (ids,
+ * the lower expert among equals), the softmax over them (weight), each choice's rank among the rows
+ * of its expert, and batch tiles of m_pad places: expert e has tiles from place first[e] on,
+ * tile_group[i] is the expert of tile i (-1: no such tile).  max_tiles >= min(experts, n) + n / m_pad
+ * for n = rows * top.  count [experts + 1] is zero before and after.
+ * hb_moe_gather: row r of h (stride ld) to place[r,k] = first + rank in x.
+ * hb_gemm_grouped: Y[r] = X[r] . W[group of r]^T with [N, K] weights per group, on the sorted rows
+ * (X, Y: max_tiles*m_pad rows; bf16 with K % 8 == 0 and m_pad % 16 == 0 on tensor cores); gated:
+ * the N rows are [gate | up] and Y = act(gate, up), N/2 wide (bf16 only). */
+typedef struct hb_moe_routing {
+  int experts, top, m_pad, max_tiles;
+  int32_t *ids, *rank, *place; /* [rows, top] */
+  float* weight;               /* [rows, top] */
+  int32_t *count, *first, *tile_group;
+} hb_moe_routing;
+int hb_moe_route_top(void* stream, const hb_moe_routing* m, const void* h, int64_t ld_h, const void* router,
+                     const float* bias, int64_t rows, int64_t width, hb_dtype dtype);
+int hb_moe_gather(void* stream, const hb_moe_routing* m, void* x, const void* h, int64_t ld, int64_t rows, hb_dtype dtype);
+/* g clipped from above, u to both sides at `limit`: g * sigmoid(slope * (g + cubic * g^3)) * (u + shift).
+ * SiLU: 1, 0, INFINITY, 0; gelu in its tanh form: 2 sqrt(2/pi), 0.044715, INFINITY, 0. */
+typedef struct hb_gated_act_spec {
+  float slope, cubic, limit, shift;
+} hb_gated_act_spec;
+int hb_gated_act(void* stream, void* out, const void* gate_up, int64_t M, int64_t inter, const hb_gated_act_spec* act,
+                 hb_dtype dtype);
+int hb_gemm_grouped(void* stream, void* Y, const void* X, const void* W, int groups, int64_t N, int64_t K, int m_pad,
+                    int max_tiles, int likely_tiles, const int32_t* tile_group, int out_f32,
+                    const hb_gated_act_spec* gated, hb_dtype dtype);
 
 /* S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per head, state and outputs fp32.
  * p holds q, k (heads*dim), v (heads*vdim) and, for a low-rank decay, rank columns, at the given
@@ -298,6 +363,21 @@ int hb_streams_embed(void* stream, float* x, void* h, const void* embed, const v
 int hb_streams_mix(void* stream, float* x, void* h, const float* y, const float* y2, int64_t ld_y, const float* mix,
                    const float* out, const float* next_in, const float* next_norm, const float* w1, const float* w2,
                    int64_t rows, int streams, int64_t width, int64_t ld_h, float eps, hb_dtype dtype);
+/* hb_streams_mix with everything it can do: norm weights apply as norm_offset + norm; without y2, y may
+ * be NULL, and bias [width] and the outputs of a mixture's experts are added to it:
+ * sum_k expert_weight[r,k] * expert_y[expert_place[r,k]] (rows of `dtype`, stride ld_y). */
+typedef struct hb_stream_mix_args {
+  const float *mix, *out, *next_in, *next_norm, *w1, *w2;
+  float norm_offset;
+  const float* bias;
+  const void* expert_y;
+  const int32_t* expert_place;
+  const float* expert_weight;
+  int top;
+} hb_stream_mix_args;
+int hb_streams_mix_ex(void* stream, float* x, void* h, const float* y, const float* y2, int64_t ld_y,
+                      const hb_stream_mix_args* m, int64_t rows, int streams, int64_t width, int64_t ld_h, float eps,
+                      hb_dtype dtype);
 int hb_streams_final(void* stream, void* h, const float* x, const int32_t* want, const float* norm, int64_t n_want,
                      int streams, int64_t width, int64_t ld_h, float eps, hb_dtype dtype);
 /* out[r, g*size + i] = o / rms over group g * weight[i] * act(gate); the weight [size] is shared by the
@@ -647,8 +727,9 @@ int hb_kv_swap_blocks(hb_engine* e, const int64_t* pairs, size_t n_pairs, int to
  * 0 QKV projection, 1 decode attention, 2 RoPE + KV write, 3 (add +) RMSNorm, 4 embedding /
  * argmax / SwiGLU gate, 5 all-reduce, 6 o_proj, 7 gate|up projection, 8 down_proj,
  * 9 lm_head (6 and 8 include the fused all-reduce + residual + norm when that kernel
- * runs), 10 linear recurrence.  The step counts like any other decode step. */
-#define HB_PROFILE_KINDS 11
+ * runs), 10 linear recurrence, 11 routing to experts, 12 / 13 the experts' gate|up and down
+ * projections.  The step counts like any other decode step. */
+#define HB_PROFILE_KINDS 14
 int hb_engine_profile_step(hb_engine* e, hb_seq* const* seqs, size_t B,
                            const uint32_t* last_tokens, uint32_t* next_tokens, float* ms_by_kind);
 /* The same for every step while on (hb_step, hb_forward, ...): the times of the last step. */

@@ -102,6 +102,42 @@ class SpanAttentionArgs(C.Structure):
         ("max_blocks", C.c_int64), ("num_blocks", C.c_int64), ("row_segment", C.c_void_p), ("positions", C.c_void_p),
         ("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("window", C.c_int),
         ("keep_first", C.c_int), ("scale", C.c_float),
+        ("chunk", C.c_int), ("key_scale", C.c_void_p), ("dist_bias", C.c_void_p), ("dist_len", C.c_int),
+        ("sink", C.c_void_p), ("gate", C.c_void_p), ("ld_gate", C.c_int64),
+    ]
+
+
+class AttentionPrepArgs(C.Structure):
+    """hb_attention_prep_args: biases, norms or rotation of queries and keys, and the K/V write."""
+    _fields_ = [
+        ("p", C.c_void_p), ("ld", C.c_int64), ("off_q", C.c_int), ("off_k", C.c_int), ("off_v", C.c_int),
+        ("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("positions", C.c_void_p),
+        ("slots", C.c_void_p), ("k_cache", C.c_void_p), ("v_cache", C.c_void_p), ("num_blocks", C.c_int64),
+        ("q_bias", C.c_void_p), ("k_bias", C.c_void_p), ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("eps", C.c_float),
+        ("rotation", C.c_void_p), ("pairs", C.c_int), ("key_scale", C.c_void_p),
+    ]
+
+
+class MoeRouting(C.Structure):
+    """hb_moe_routing: what a router decided and where the rows of the experts lie."""
+    _fields_ = [
+        ("experts", C.c_int), ("top", C.c_int), ("m_pad", C.c_int), ("max_tiles", C.c_int), ("ids", C.c_void_p),
+        ("rank", C.c_void_p), ("place", C.c_void_p), ("weight", C.c_void_p), ("count", C.c_void_p), ("first", C.c_void_p),
+        ("tile_group", C.c_void_p),
+    ]
+
+
+class GatedActSpec(C.Structure):
+    """hb_gated_act_spec: g * sigmoid(slope * (g + cubic * g^3)) * (u + shift), clipped at limit."""
+    _fields_ = [("slope", C.c_float), ("cubic", C.c_float), ("limit", C.c_float), ("shift", C.c_float)]
+
+
+class StreamMixArgs(C.Structure):
+    """hb_stream_mix_args: how a sublayer's output goes back into the residual streams."""
+    _fields_ = [
+        ("mix", C.c_void_p), ("out", C.c_void_p), ("next_in", C.c_void_p), ("next_norm", C.c_void_p), ("w1", C.c_void_p),
+        ("w2", C.c_void_p), ("norm_offset", C.c_float), ("bias", C.c_void_p), ("expert_y", C.c_void_p),
+        ("expert_place", C.c_void_p), ("expert_weight", C.c_void_p), ("top", C.c_int),
     ]
 
 
@@ -141,6 +177,12 @@ _SIGS = {
     "hb_linear_recurrence": (_i, [_vp, _vp, _vp, _i, _vp, _i, _vp, _i, _vp, _vp, _i]),
     "hb_streams_embed": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i, _i64, _i64, _i64, _i64, _f, _i]),
     "hb_streams_mix": (_i, [_vp, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i, _i64, _i64, _f, _i]),
+    "hb_streams_mix_ex": (_i, [_vp, _vp, _vp, _vp, _vp, _i64, _vp, _i64, _i, _i64, _i64, _f, _i]),
+    "hb_attention_prepare": (_i, [_vp, _vp, _i64, _i]),
+    "hb_moe_route_top": (_i, [_vp, _vp, _vp, _i64, _vp, _vp, _i64, _i64, _i]),
+    "hb_moe_gather": (_i, [_vp, _vp, _vp, _vp, _i64, _i64, _i]),
+    "hb_gated_act": (_i, [_vp, _vp, _vp, _i64, _i64, _vp, _i]),
+    "hb_gemm_grouped": (_i, [_vp, _vp, _vp, _vp, _i, _i64, _i64, _i, _i, _i, _vp, _i, _vp, _i]),
     "hb_streams_final": (_i, [_vp, _vp, _vp, _vp, _vp, _i64, _i, _i64, _i64, _f, _i]),
     "hb_gated_group_norm": (_i, [_vp, _vp, _i64, _vp, _i64, _vp, _i64, _vp, _i64, _i, _i, _i, _f, _i]),
     "hb_gemm_workspace_bytes": (_sz, [_i64, _i64, _i64, _i]),
@@ -1017,7 +1059,8 @@ class Engine:
         check(lib.hb_kv_swap_blocks(self.handle, p.ctypes.data if len(p) else None, len(p), 1 if to_cpu else 0))
 
     PROFILE_KINDS = ("gemm_qkv", "attention", "rope_kv", "norm", "other", "all_reduce",
-                     "gemm_o_proj", "gemm_gate_up", "gemm_down", "gemm_lm_head", "recurrence")
+                     "gemm_o_proj", "gemm_gate_up", "gemm_down", "gemm_lm_head", "recurrence",
+                     "routing", "experts_gate_up", "experts_down")
 
     def profile_step(self, seqs: Sequence[Sequence_], last_tokens: np.ndarray) -> tuple[np.ndarray, dict]:
         """One eager decode step with per-kernel-kind device times (ms)."""

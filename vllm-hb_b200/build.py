@@ -41,7 +41,7 @@ def _sources() -> list[Path]:
 
 
 def _headers_mtime() -> float:
-    hs = list(CSRC.glob("*.h")) + list((HERE.parent / "include").glob("*.h"))
+    hs = list(CSRC.glob("*.h")) + list(CSRC.glob("*.cuh")) + list((HERE.parent / "include").glob("*.h"))
     return max(h.stat().st_mtime for h in hs)
 
 

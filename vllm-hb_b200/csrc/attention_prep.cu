@@ -1,0 +1,201 @@
+// From a layer's projection rows to queries in place and keys and values in their slots: biases,
+// norms over whole projections, rotation of channel pairs, all in fp32, one CTA per row.
+#include "layered_ops.h"
+
+namespace hb {
+
+constexpr int kPrepThreads = 256;
+
+// Elements in runs of V (1: any sizes; 8 bf16 or 4 fp32 numbers: 16-byte accesses).
+template <typename T, int V>
+struct Run {
+  static __device__ __forceinline__ void load(float (&f)[V], const T* p) {
+    if constexpr (V == 1) {
+      f[0] = to_f32<T>(*p);
+    } else {
+      Vec16<T> v;
+      v.load(p);
+      v.unpack(f);
+    }
+  }
+  static __device__ __forceinline__ void store(T* p, const float (&f)[V]) {
+    if constexpr (V == 1) {
+      *p = from_f32<T>(f[0]);
+    } else {
+      Vec16<T> v;
+      v.pack(f);
+      v.store(p);
+    }
+  }
+};
+
+// Where element d of kv head g of a row's key (value) lies in its pool.
+__device__ __forceinline__ int64_t pool_at(int64_t slot, int G, int g, int width, int d) {
+  return ((slot / HB_BLOCK_SIZE * G + g) * HB_BLOCK_SIZE + slot % HB_BLOCK_SIZE) * width + d;
+}
+
+// Rotation of channel pairs.  V > 1: runs of V channels (widths and the number of rotated channels
+// are multiples of V); V == 1: pair by pair.
+template <typename T, int V>
+__global__ void __launch_bounds__(kPrepThreads) attention_rotate_kernel(const AttentionPrep a) {
+  pdl_trigger();
+  extern __shared__ float s_cs[];  // [pairs] cosines, [pairs] sines
+  pdl_grid_wait();
+  const int64_t row = blockIdx.x, slot = a.slots[row];
+  const int tid = threadIdx.x, P = a.pairs, D = a.dim;
+  const bool keep = slot >= 0 && slot < a.num_blocks * HB_BLOCK_SIZE;
+  // the angle less its whole turns in fp64: far positions keep the accuracy of near ones
+  const double pos = (double)a.pos[row], turn = 6.283185307179586;
+  for (int i = tid; i < P; i += kPrepThreads) {
+    const double angle = pos * a.rotation[i];
+    sincosf((float)(angle - turn * rint(angle * (1.0 / turn))), s_cs + P + i, s_cs + i);
+  }
+  __syncthreads();
+  T* pr = (T*)a.p + row * a.ld;
+  constexpr int W = V == 1 ? 2 : V;           // channels a thread turns at a time
+  const int per = (D + W - 1) / W, total = (a.heads + a.kv_heads) * per;
+  for (int i = tid; i < total; i += kPrepThreads) {
+    const int head = i / per, d = i % per * W;
+    const bool query = head < a.heads;
+    const int g = query ? head : head - a.heads, off = query ? a.off_q : a.off_k;
+    const float* bias = query ? a.q_bias : a.k_bias;
+    T* src = pr + off + g * D + d;
+    float f[W];
+    if constexpr (V == 1) {
+      f[0] = to_f32<T>(src[0]);
+      f[1] = d + 1 < D ? to_f32<T>(src[1]) : 0.f;
+    } else {
+      Run<T, V>::load(f, src);
+    }
+    if (bias)
+#pragma unroll
+      for (int j = 0; j < W; ++j)
+        if (d + j < D) f[j] += bias[g * D + d + j];
+    if (d / 2 < P) {
+#pragma unroll
+      for (int j = 0; j < W; j += 2) {
+        const float c = s_cs[d / 2 + j / 2], s = s_cs[P + d / 2 + j / 2], u = f[j], v = f[j + 1];
+        f[j] = u * c - v * s;
+        f[j + 1] = v * c + u * s;
+      }
+    }
+    if (!query && !keep) continue;
+    T* dst = query ? src : (T*)a.kc + pool_at(slot, a.kv_heads, g, D, d);
+    if constexpr (V == 1) {
+      dst[0] = from_f32<T>(f[0]);
+      if (d + 1 < D) dst[1] = from_f32<T>(f[1]);
+    } else {
+      Run<T, V>::store(dst, f);
+    }
+  }
+  if (!keep) return;
+  const int vper = a.vdim / V;
+  for (int i = tid; i < a.kv_heads * vper; i += kPrepThreads) {
+    const int g = i / vper, d = i % vper * V;
+    float f[V];
+    Run<T, V>::load(f, pr + a.off_v + g * a.vdim + d);
+    Run<T, V>::store((T*)a.vc + pool_at(slot, a.kv_heads, g, a.vdim, d), f);
+  }
+}
+
+// RMS norms over all query rows and all key rows of a position.
+template <typename T, int V>
+__global__ void __launch_bounds__(kPrepThreads) attention_norm_kernel(const AttentionPrep a) {
+  pdl_trigger();
+  pdl_grid_wait();
+  __shared__ float red[33];
+  const int64_t row = blockIdx.x, slot = a.slots[row];
+  const int tid = threadIdx.x, D = a.dim, nq = a.heads * D, nk = a.kv_heads * D, rep = a.heads / a.kv_heads;
+  const bool keep = slot >= 0 && slot < a.num_blocks * HB_BLOCK_SIZE, tied = a.key_scale != nullptr;
+  T* q = (T*)a.p + row * a.ld + a.off_q;
+  const T* k = (const T*)a.p + row * a.ld + a.off_k;
+  auto load = [&](float (&f)[V], const T* src, const float* bias, int i) {
+    Run<T, V>::load(f, src + i);
+    if (bias)
+#pragma unroll
+      for (int j = 0; j < V; ++j) f[j] += bias[i + j];
+  };
+  float sq = 0.f, sk = 0.f, f[V];
+  for (int i = tid * V; i < nq; i += kPrepThreads * V) {
+    load(f, q, a.q_bias, i);
+#pragma unroll
+    for (int j = 0; j < V; ++j) sq = fmaf(f[j], f[j], sq);
+  }
+  for (int i = tid * V; i < nk; i += kPrepThreads * V) {
+    load(f, k, a.k_bias, i);
+#pragma unroll
+    for (int j = 0; j < V; ++j) sk = fmaf(f[j], f[j], sk);
+  }
+  const float rq = 1.f / sqrtf(block_sum(sq, red) / (float)nq + a.eps);
+  const float rk = 1.f / sqrtf(block_sum(sk, red) / (float)nk + a.eps);
+  for (int i = tid * V; i < nq; i += kPrepThreads * V) {
+    load(f, q, a.q_bias, i);
+    const int at = tied ? i / (rep * D) * D + i % D : 0;  // the key channel this query channel meets
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      f[j] *= rq * a.q_norm[i + j];
+      if (tied) f[j] *= a.k_norm[at + j];
+    }
+    Run<T, V>::store(q + i, f);
+  }
+  if (!keep) return;
+  for (int i = tid * V; i < nk; i += kPrepThreads * V) {
+    load(f, k, a.k_bias, i);
+    if (!tied)
+#pragma unroll
+      for (int j = 0; j < V; ++j) f[j] *= rk * a.k_norm[i + j];
+    Run<T, V>::store((T*)a.kc + pool_at(slot, a.kv_heads, i / D, D, i % D), f);
+  }
+  if (tied) {
+    if (tid == 0) a.key_scale[slot] = rk;
+    return;
+  }
+  const int nv = a.kv_heads * a.vdim;
+  for (int i = tid * V; i < nv; i += kPrepThreads * V) {
+    Run<T, V>::load(f, (const T*)a.p + row * a.ld + a.off_v + i);
+    Run<T, V>::store((T*)a.vc + pool_at(slot, a.kv_heads, i / a.vdim, a.vdim, i % a.vdim), f);
+  }
+}
+
+int attention_prepare(cudaStream_t st, const AttentionPrep& a, int64_t rows, hb_dtype dtype) {
+  if (rows == 0) return HB_OK;
+  const bool norm = a.q_norm || a.k_norm;
+  if (norm && (!a.q_norm || !a.k_norm || a.pairs))
+    return fail(HB_ERR_INVALID_ARG, "attention_prepare: norms come for queries and keys, and without a rotation");
+  if (a.key_scale && (!norm || a.vdim != a.dim))
+    return fail(HB_ERR_INVALID_ARG, "attention_prepare: keys that are the values have a norm and their width");
+  if (2 * a.pairs > a.dim || a.pairs > 5000) return fail(HB_ERR_INVALID_ARG, "attention_prepare: %d pairs of %d channels", a.pairs, a.dim);
+  const int es = (int)dtype_size(dtype), n = 16 / es;
+  auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  const bool vec = a.dim % n == 0 && a.vdim % n == 0 && (2 * a.pairs) % n == 0 && a.off_q % n == 0 && a.off_k % n == 0 &&
+                   a.off_v % n == 0 && a.ld % n == 0 && al(a.p) && al(a.kc) && al(a.vc);
+  const dim3 grid((unsigned)rows), block(kPrepThreads);
+  const size_t smem = (size_t)a.pairs * 2 * sizeof(float);
+  auto launch = [&](auto* rotate, auto* normed) -> int {
+    if (norm) HB_CUDA_CHECK(launch_pdl(normed, grid, block, 0, st, a));
+    else HB_CUDA_CHECK(launch_pdl(rotate, grid, block, smem, st, a));
+    return HB_OK;
+  };
+  if (dtype == HB_F32)
+    return vec ? launch(attention_rotate_kernel<float, 4>, attention_norm_kernel<float, 4>)
+               : launch(attention_rotate_kernel<float, 1>, attention_norm_kernel<float, 1>);
+  if (dtype == HB_BF16)
+    return vec ? launch(attention_rotate_kernel<__nv_bfloat16, 8>, attention_norm_kernel<__nv_bfloat16, 8>)
+               : launch(attention_rotate_kernel<__nv_bfloat16, 1>, attention_norm_kernel<__nv_bfloat16, 1>);
+  return fail(HB_ERR_UNSUPPORTED_DTYPE, "attention_prepare runs in bf16 or f32");
+}
+
+__global__ void expand_distance_bias_kernel(float* __restrict__ out, const float* __restrict__ rel,
+                                            const int32_t* __restrict__ bucket, int heads, int dist_len) {
+  const int d = blockIdx.x * blockDim.x + threadIdx.x;
+  if (d < dist_len) out[(int64_t)blockIdx.y * dist_len + d] = rel[(int64_t)bucket[d] * heads + blockIdx.y];
+}
+
+int expand_distance_bias(cudaStream_t st, float* out, const float* rel, const int32_t* bucket, int heads, int dist_len) {
+  expand_distance_bias_kernel<<<dim3((unsigned)((dist_len + 255) / 256), (unsigned)heads), 256, 0, st>>>(out, rel, bucket, heads,
+                                                                                                    dist_len);
+  HB_LAUNCH_CHECK();
+  return HB_OK;
+}
+
+}  // namespace hb

@@ -1,8 +1,9 @@
-// Paged attention over a span of positions: the last `window` of them (or all) and the first
-// `keep_first`, with keys and values of any (different) widths.
+// Paged attention over a span of positions: the last `window` of them (or all), or those of the
+// position's own chunk, and the first `keep_first`; keys and values of any (different) widths, a
+// bias by distance, a sink, a gate on the outputs.
 //
 // The visible keys of a query at position p are two runs, [0, keep) and [lo, p] with
-// lo = max(0, p - window + 1) and keep = min(keep_first, lo); only their blocks are read.
+// lo = SpanAttention::first_seen(p) and keep = min(keep_first, lo); only their blocks are read.
 #include <climits>
 
 #include "layered_ops.h"
@@ -63,10 +64,13 @@ span_attention_rows_kernel(const SpanAttention a, const int32_t* __restrict__ ro
   float* s_l = s_m + R;               // [R] running sum
   float* s_a = s_l + R;               // [R] rescale of this tile
   __shared__ int64_t s_key[kSpanTile];  // (block * kv_heads + head) * 16 + offset of the tile's keys
+  __shared__ float s_ks[kSpanTile];     // scale of the keys
+  __shared__ int s_dist[kSpanTile];     // their distance, up to the last of the bias table
+  const T* values = (const T*)(a.key_scale ? a.kc : a.vc);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = blockIdx.y;
   const int64_t row = row_list[blockIdx.x];
   const int pos = a.pos[row];
-  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int lo = a.first_seen(pos);
   const int keep = min(a.keep_first, lo);
   const int n_keys = keep + (pos - lo + 1);
   const int32_t* table = a.tables + (int64_t)a.row_seg[row] * a.max_blocks;
@@ -82,6 +86,8 @@ span_attention_rows_kernel(const SpanAttention a, const int32_t* __restrict__ ro
       int64_t blk = j / HB_BLOCK_SIZE < a.max_blocks ? table[j / HB_BLOCK_SIZE] : 0;
       if (blk < 0 || blk >= a.num_blocks) blk = 0;  // never outside the pool
       s_key[i] = (blk * a.kv_heads + g) * HB_BLOCK_SIZE + j % HB_BLOCK_SIZE;
+      s_ks[i] = a.key_scale ? a.key_scale[blk * HB_BLOCK_SIZE + j % HB_BLOCK_SIZE] : 1.f;
+      s_dist[i] = min(pos - j, a.dist_len - 1);
     }
     __syncthreads();
     for (int i = warp; i < nt; i += kSpanWarps) {
@@ -90,7 +96,8 @@ span_attention_rows_kernel(const SpanAttention a, const int32_t* __restrict__ ro
         float s = 0.f;
         for (int d = lane; d < D; d += 32) s = fmaf(s_q[h * D + d], to_f32<T>(kr[d]), s);
         s = warp_sum(s);
-        if (lane == 0) s_p[h * kSpanTile + i] = s;
+        if (lane == 0)
+          s_p[h * kSpanTile + i] = fmaf(s, s_ks[i], a.dist_bias ? a.dist_bias[(int64_t)(g * R + h) * a.dist_len + s_dist[i]] : 0.f);
       }
     }
     __syncthreads();
@@ -118,14 +125,27 @@ span_attention_rows_kernel(const SpanAttention a, const int32_t* __restrict__ ro
     for (int d = tid; d < VD; d += kSpanThreads) {
       for (int h = 0; h < R; ++h) s_acc[h * VD + d] *= s_a[h];
       for (int i = 0; i < nt; ++i) {
-        const float v = to_f32<T>(((const T*)a.vc)[s_key[i] * VD + d]);
+        const float v = to_f32<T>(values[s_key[i] * VD + d]);
         for (int h = 0; h < R; ++h) s_acc[h * VD + d] = fmaf(s_p[h * kSpanTile + i], v, s_acc[h * VD + d]);
       }
     }
   }
   __syncthreads();
+  if (a.sink)  // one more member of the softmax, without a value
+    for (int h = tid; h < R; h += kSpanThreads) {
+      const float k = a.sink[g * R + h], top = fmaxf(s_m[h], k), f = expf(s_m[h] - top);
+      s_a[h] = f;
+      s_l[h] = fmaf(s_l[h], f, expf(k - top));
+    }
+  __syncthreads();
   T* out = (T*)a.out + row * a.ld_out + (int64_t)g * R * VD;
-  for (int i = tid; i < R * VD; i += kSpanThreads) out[i] = from_f32<T>(s_acc[i] / s_l[i / VD]);
+  const T* gate = a.gate ? (const T*)a.gate + row * a.ld_gate + (int64_t)g * R * VD : nullptr;
+  for (int i = tid; i < R * VD; i += kSpanThreads) {
+    float o = s_acc[i] / s_l[i / VD];
+    if (a.sink) o *= s_a[i / VD];
+    if (gate) o /= 1.f + expf(-to_f32<T>(gate[i]));
+    out[i] = from_f32<T>(o);
+  }
 }
 
 int span_attention_rows(cudaStream_t st, const SpanAttention& a, const int32_t* row_list, int n_rows, hb_dtype dtype) {

@@ -1,7 +1,8 @@
 // Span attention (see attention_span.cu) on tensor cores: bf16, key and value widths that are
 // multiples of 8.  S = Q K^T with bf16 operands and fp32 accumulation, softmax in fp32, and
 // O += P V with P as a pair of bf16 numbers (P = hi + lo), so that the weights keep fp32-like
-// precision.
+// precision.  Kernels instantiated with EXT also take a bias by distance and keys that are their
+// values times a scale: K and V are then one tile of shared memory, read once.
 //
 //   tiles  (prompt portions): CTA = 64 rows = up to 64 / R consecutive positions of one segment x
 //          the R query heads of a kv head; four warps of 16 rows share every 64-key tile.
@@ -37,20 +38,27 @@ struct BlockRuns {
   int na, b0, n;
   __device__ __forceinline__ int block(int i) const { return i < na ? i : b0 + (i - na); }
 };
-__device__ __forceinline__ BlockRuns block_runs(int first_pos, int last_pos, int window, int keep_first) {
+__device__ __forceinline__ BlockRuns block_runs(int first_pos, int last_pos, const SpanAttention& a) {
   BlockRuns r;
-  const int lo = window > 0 ? max(0, first_pos - window + 1) : 0;
+  const int lo = a.first_seen(first_pos);
   r.b0 = lo / kBS;
-  r.na = min((min(keep_first, lo) + kBS - 1) / kBS, r.b0);
+  r.na = min((min(a.keep_first, lo) + kBS - 1) / kBS, r.b0);
   r.n = r.na + last_pos / kBS - r.b0 + 1;
   return r;
 }
-__device__ __forceinline__ bool visible(int key, int pos, int window, int keep_first) {
-  return key <= pos && (window <= 0 || pos - key < window || key < keep_first);
+// lo: first_seen() of the position
+__device__ __forceinline__ bool visible(int key, int pos, int lo, int keep_first) {
+  return key <= pos && (key >= lo || key < keep_first);
 }
-// Every key of the block that starts at `key` is visible from all positions first .. last.
-__device__ __forceinline__ bool all_visible(int key, int first, int last, int window, int keep_first) {
-  return key + kBS - 1 <= first && (window <= 0 || last - key < window || key + kBS <= keep_first);
+// Every key of the block that starts at `key` is visible from all positions of a range: `first` is
+// the earliest, `lo` what the latest of them sees first (it grows with the position).
+__device__ __forceinline__ bool all_visible(int key, int first, int lo, int keep_first) {
+  return key + kBS - 1 <= first && (key >= lo || key + kBS <= keep_first);
+}
+constexpr float kLog2e = 1.4426950408889634f;
+__device__ __forceinline__ float sigmoid_of(uint32_t bits16) {
+  const float z = __uint_as_float(bits16 << 16);  // a bf16 number
+  return __fdividef(1.f, 1.f + __expf(-z));
 }
 // A warp copies a 16-row block of `w` 16-byte vectors a row into rows of `stride` bytes; (j, c) is the
 // lane's first (row, vector), stepped without divisions.
@@ -71,25 +79,28 @@ struct BlockCopy {
 }  // namespace
 
 // NV: 16-column pairs of n-tiles, i.e. the value slice is at most 16 * NV wide.
-template <int NV>
+template <int NV, bool EXT>
 __global__ void __launch_bounds__(kThreads)
 span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ tiles, int stages) {
   extern __shared__ __align__(16) uint8_t smem[];
   const int R = a.heads / a.kv_heads, D = a.dim, DP = pad16(D), KS = DP + 8;
-  const int v0 = blockIdx.z * kSlice, VW = min(kSlice, a.vdim - v0), VP = pad16(VW), VS = VP + 8;
+  const bool tied = EXT && a.key_scale != nullptr;      // one tile is keys and values
+  const int v0 = blockIdx.z * kSlice, VW = min(kSlice, a.vdim - v0), VP = pad16(VW), VS = tied ? KS : VP + 8;
   __nv_bfloat16* s_q = (__nv_bfloat16*)smem;           // [64][KS]
   __nv_bfloat16* s_k = s_q + kRows * KS;               // [stages][64][KS]
-  __nv_bfloat16* s_v = s_k + stages * kKeys * KS;      // [stages][64][VS]
+  __nv_bfloat16* s_v = tied ? s_k : s_k + stages * kKeys * KS;               // [stages][64][VS]
+  float* s_ks = (float*)(s_k + stages * kKeys * KS);   // tied: [stages][64] scales of the keys
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gi = lane >> 2, t = lane & 3, kvh = blockIdx.y;
   // padding columns stay zero
   for (int i = tid; i < (kRows + stages * kKeys) * KS / 8; i += kThreads)
     if (i % (KS / 8) * 8 >= D) reinterpret_cast<uint4*>(s_q)[i] = make_uint4(0, 0, 0, 0);
-  for (int i = tid; i < stages * kKeys * VS / 8; i += kThreads)
-    if (i % (VS / 8) * 8 >= VW) reinterpret_cast<uint4*>(s_v)[i] = make_uint4(0, 0, 0, 0);
+  if (!tied)
+    for (int i = tid; i < stages * kKeys * VS / 8; i += kThreads)
+      if (i % (VS / 8) * 8 >= VW) reinterpret_cast<uint4*>(s_v)[i] = make_uint4(0, 0, 0, 0);
   pdl_grid_wait();
   const RowRange tile = tiles[blockIdx.x];
   const int first_pos = a.pos[tile.row0], last_pos = first_pos + tile.n - 1;
-  const BlockRuns runs = block_runs(first_pos, last_pos, a.window, a.keep_first);
+  const BlockRuns runs = block_runs(first_pos, last_pos, a);
   const int32_t* table = a.tables + (int64_t)tile.seg * a.max_blocks;
   const int n_rows = tile.n * R, n_steps = (runs.n + kKeys / kBS - 1) / (kKeys / kBS);
 
@@ -109,22 +120,33 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
     if (phys < 0 || phys >= a.num_blocks) phys = 0;  // never outside the pool
     const int64_t slot = (phys * a.kv_heads + kvh) * kBS;
     copy_k(smem_u32(s_k + (s * kKeys + warp * kBS) * KS), KS * 2, (const __nv_bfloat16*)a.kc + slot * D, D);
-    copy_v(smem_u32(s_v + (s * kKeys + warp * kBS) * VS), VS * 2, (const __nv_bfloat16*)a.vc + slot * a.vdim + v0, a.vdim);
+    if (!tied) copy_v(smem_u32(s_v + (s * kKeys + warp * kBS) * VS), VS * 2, (const __nv_bfloat16*)a.vc + slot * a.vdim + v0, a.vdim);
+    else if (lane < 4) cp_async_16(smem_u32(s_ks + s * kKeys + warp * kBS + lane * 4), a.key_scale + phys * kBS + lane * 4);
     cp_async_commit();
   };
   load(0);
 
   const int r0 = warp * 16 + gi, r1 = r0 + 8;
   const int p0 = first_pos + r0 / R, p1 = first_pos + r1 / R;
+  const int lo0 = a.first_seen(p0), lo1 = a.first_seen(p1);
   const bool live = warp * 16 < n_rows;  // warps without rows only help to load
   float o[2 * NV][4];
 #pragma unroll
   for (int i = 0; i < 2 * NV; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
-  const float sc = a.scale * 1.4426950408889634f;  // scores in units of log2
-  const bool sc_ok = sc > 0.f;
+  const float sc = a.scale * kLog2e;               // scores in units of log2
+  const bool sc_ok = !EXT && sc > 0.f;
   const float es = sc_ok ? sc : 1.f;               // what the exponential still multiplies by
   const int warp_first = first_pos + warp * 16 / R, warp_last = min(first_pos + (warp * 16 + 15) / R, last_pos);
+  const int warp_lo = a.first_seen(warp_last);
+  const float *bias0 = nullptr, *bias1 = nullptr;  // of the rows' heads, by distance
+  float far0 = 0.f, far1 = 0.f;                    // from distance dist_len - 1 on, in units of log2
+  if (EXT && a.dist_bias) {
+    bias0 = a.dist_bias + (int64_t)(kvh * R + r0 % R) * a.dist_len;
+    bias1 = a.dist_bias + (int64_t)(kvh * R + r1 % R) * a.dist_len;
+    far0 = __ldg(bias0 + a.dist_len - 1) * kLog2e;
+    far1 = __ldg(bias1 + a.dist_len - 1) * kLog2e;
+  }
   const uint32_t q_addr = smem_u32(s_q + (warp * 16 + (lane & 15)) * KS + (lane >> 4) * 8);
 
   for (int step = 0; step < n_steps; ++step) {
@@ -155,11 +177,37 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
         }
       }
       // scores stay unscaled: sc > 0 is applied inside the exponential (sc <= 0: scaled here)
-      bool full = sc_ok;
+      bool full = sc_ok || EXT;
+      int last_key = 0;
 #pragma unroll
       for (int b = 0; b < 4; ++b) {
         const int vb = step * (kKeys / kBS) + b;
-        full = full && vb < runs.n && all_visible(runs.block(vb) * kBS, warp_first, warp_last, a.window, a.keep_first);
+        full = full && vb < runs.n && all_visible(runs.block(vb) * kBS, warp_first, warp_lo, a.keep_first);
+        last_key = max(last_key, vb < runs.n ? runs.block(vb) * kBS + kBS - 1 : INT_MAX / 2);
+      }
+      if (EXT) {
+        // scale per key and bias by distance; from the table's last distance on the bias is one number
+        const bool far = !bias0 || warp_first - last_key >= a.dist_len - 1;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          float2 f = make_float2(sc, sc);
+          if (tied) {
+            f = *reinterpret_cast<const float2*>(s_ks + step % stages * kKeys + i * 8 + 2 * t);
+            f.x *= sc;
+            f.y *= sc;
+          }
+          if (far) {
+            s[i][0] = fmaf(s[i][0], f.x, far0); s[i][1] = fmaf(s[i][1], f.y, far0);
+            s[i][2] = fmaf(s[i][2], f.x, far1); s[i][3] = fmaf(s[i][3], f.y, far1);
+          } else {
+            const int vb = step * (kKeys / kBS) + i / 2, top = a.dist_len - 1;
+            const int key = (vb < runs.n ? runs.block(vb) * kBS : 0) + (i & 1) * 8 + 2 * t;
+            s[i][0] = fmaf(s[i][0], f.x, __ldg(bias0 + min(max(p0 - key, 0), top)) * kLog2e);
+            s[i][1] = fmaf(s[i][1], f.y, __ldg(bias0 + min(max(p0 - key - 1, 0), top)) * kLog2e);
+            s[i][2] = fmaf(s[i][2], f.x, __ldg(bias1 + min(max(p1 - key, 0), top)) * kLog2e);
+            s[i][3] = fmaf(s[i][3], f.y, __ldg(bias1 + min(max(p1 - key - 1, 0), top)) * kLog2e);
+          }
+        }
       }
       if (!full) {
 #pragma unroll
@@ -168,8 +216,9 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
           const int key = vb < runs.n ? runs.block(vb) * kBS + (i & 1) * 8 + 2 * t : INT_MAX - 1;
 #pragma unroll
           for (int c = 0; c < 2; ++c) {
-            s[i][c] = visible(key + c, p0, a.window, a.keep_first) ? (sc_ok ? s[i][c] : s[i][c] * sc) : -INFINITY;
-            s[i][2 + c] = visible(key + c, p1, a.window, a.keep_first) ? (sc_ok ? s[i][2 + c] : s[i][2 + c] * sc) : -INFINITY;
+            const bool scaled = EXT || sc_ok;
+            s[i][c] = visible(key + c, p0, lo0, a.keep_first) ? (scaled ? s[i][c] : s[i][c] * sc) : -INFINITY;
+            s[i][2 + c] = visible(key + c, p1, lo1, a.keep_first) ? (scaled ? s[i][2 + c] : s[i][2 + c] * sc) : -INFINITY;
           }
         }
       }
@@ -197,7 +246,7 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
         l0 += s[i][0] + s[i][1];
         l1 += s[i][2] + s[i][3];
       }
-      const uint32_t v_addr = smem_u32(vt + (lane & 15) * VS + (lane >> 4) * 8);
+      const uint32_t v_addr = smem_u32(vt + (lane & 15) * VS + (lane >> 4) * 8 + (tied ? v0 : 0));
 #pragma unroll
       for (int kk = 0; kk < 4; ++kk) {
         uint32_t hi[4], lo[4];
@@ -225,7 +274,19 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
   if (!live) return;
   l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
-  const float i0 = 1.f / l0, i1 = 1.f / l1;
+  float i0 = 1.f / l0, i1 = 1.f / l1;
+  if (a.sink) {  // one more member of the softmax, without a value
+    const float k0 = a.sink[kvh * R + r0 % R] * kLog2e, k1 = a.sink[kvh * R + r1 % R] * kLog2e;
+    const float t0 = fmaxf(m0 * es, k0), t1 = fmaxf(m1 * es, k1), f0 = ex2(m0 * es - t0), f1 = ex2(m1 * es - t1);
+    i0 = f0 / fmaf(l0, f0, ex2(k0 - t0));
+    i1 = f1 / fmaf(l1, f1, ex2(k1 - t1));
+  }
+  const __nv_bfloat16 *g0 = nullptr, *g1 = nullptr;
+  if (a.gate) {
+    const __nv_bfloat16* gate = (const __nv_bfloat16*)a.gate + (int64_t)kvh * R * a.vdim + v0;
+    g0 = gate + (int64_t)(tile.row0 + r0 / R) * a.ld_gate + (r0 % R) * a.vdim;
+    g1 = gate + (int64_t)(tile.row0 + r1 / R) * a.ld_gate + (r1 % R) * a.vdim;
+  }
   __nv_bfloat16* out = (__nv_bfloat16*)a.out + (int64_t)kvh * R * a.vdim + v0;
   __nv_bfloat16* w0 = out + (int64_t)(tile.row0 + r0 / R) * a.ld_out + (r0 % R) * a.vdim;
   __nv_bfloat16* w1 = out + (int64_t)(tile.row0 + r1 / R) * a.ld_out + (r1 % R) * a.vdim;
@@ -233,8 +294,15 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
   for (int i = 0; i < 2 * NV; ++i) {
     const int c = i * 8 + 2 * t;
     if (c < VW) {
-      if (r0 < n_rows) *reinterpret_cast<uint32_t*>(w0 + c) = pack_bf16(o[i][0] * i0, o[i][1] * i0);
-      if (r1 < n_rows) *reinterpret_cast<uint32_t*>(w1 + c) = pack_bf16(o[i][2] * i1, o[i][3] * i1);
+      float x[4] = {o[i][0] * i0, o[i][1] * i0, o[i][2] * i1, o[i][3] * i1};
+      if (a.gate) {
+        const uint32_t z0 = r0 < n_rows ? *reinterpret_cast<const uint32_t*>(g0 + c) : 0u;
+        const uint32_t z1 = r1 < n_rows ? *reinterpret_cast<const uint32_t*>(g1 + c) : 0u;
+        x[0] *= sigmoid_of(z0 & 0xffffu); x[1] *= sigmoid_of(z0 >> 16);
+        x[2] *= sigmoid_of(z1 & 0xffffu); x[3] *= sigmoid_of(z1 >> 16);
+      }
+      if (r0 < n_rows) *reinterpret_cast<uint32_t*>(w0 + c) = pack_bf16(x[0], x[1]);
+      if (r1 < n_rows) *reinterpret_cast<uint32_t*>(w1 + c) = pack_bf16(x[2], x[3]);
     }
   }
 }
@@ -244,23 +312,24 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
 // The products are turned over, so that the few query heads are the narrow MMA side:
 // S^T[16 keys, 8 NT heads] = K Q^T and O^T[values, heads] += V^T P^T (P transposed in registers).
 // MT: 16-column tiles of the value slice, NT: groups of 8 query heads.
-template <int MT, int NT>
+template <int MT, int NT, bool EXT>
 __global__ void __launch_bounds__(kThreads)
 span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, int n_splits, float* __restrict__ part) {
   extern __shared__ __align__(16) uint8_t smem[];
   const int R = a.heads / a.kv_heads, D = a.dim, DP = pad16(D), KS = DP + 8;
   const int slices = (a.vdim + kSlice - 1) / kSlice;
+  const bool tied = EXT && a.key_scale != nullptr;  // one tile is keys and values; their scales lie behind it
   const int v0 = (int)(blockIdx.z % slices) * kSlice, VW = min(kSlice, a.vdim - v0), VP = pad16(VW), VS = VP + 8;
   const int split = blockIdx.z / slices;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gi = lane >> 2, t = lane & 3, kvh = blockIdx.y;
-  const int stage_elems = kBS * (KS + VS);
+  const int stage_elems = tied ? kBS * (KS + 2) : kBS * (KS + VS);
   __nv_bfloat16* s_q = (__nv_bfloat16*)smem;                                  // [16][KS]
   __nv_bfloat16* ring = s_q + 16 * KS + (size_t)warp * kRing * stage_elems;   // [kRing][K 16 x KS | V 16 x VS]
   if (D % 16 || VW % 16) {  // padding columns stay zero
     for (int s = 0; s < kRing; ++s)
       for (int i = lane; i < kBS; i += 32) {
         for (int c = D; c < DP; c += 8) *reinterpret_cast<uint4*>(ring + s * stage_elems + i * KS + c) = make_uint4(0, 0, 0, 0);
-        for (int c = VW; c < VP; c += 8)
+        for (int c = VW; c < VP && !tied; c += 8)
           *reinterpret_cast<uint4*>(ring + s * stage_elems + kBS * KS + i * VS + c) = make_uint4(0, 0, 0, 0);
       }
   }
@@ -268,7 +337,8 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
   const int64_t row = rows[blockIdx.x];
   const int pos = a.pos[row];
   const int32_t* table = a.tables + (int64_t)a.row_seg[row] * a.max_blocks;
-  const BlockRuns runs = block_runs(pos, pos, a.window, a.keep_first);
+  const int lo = a.first_seen(pos);
+  const BlockRuns runs = block_runs(pos, pos, a);
   const int per = (runs.n + n_splits - 1) / n_splits, s_lo = split * per, s_hi = min(runs.n, s_lo + per);
   const int n_w = s_hi - s_lo > warp ? (s_hi - s_lo - warp + kWarps - 1) / kWarps : 0;  // this warp's blocks
 
@@ -286,10 +356,11 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
   auto load = [&](int i) {
     if (i < n_w) {
       if (i >= tab_base + 32) load_tab(i);
-      const int64_t slot = ((int64_t)__shfl_sync(0xffffffffu, tab, i - tab_base) * a.kv_heads + kvh) * kBS;
+      const int64_t phys = __shfl_sync(0xffffffffu, tab, i - tab_base), slot = (phys * a.kv_heads + kvh) * kBS;
       const uint32_t dst = ring_u + stage_in * stage_elems * 2;
       copy_k(dst, KS * 2, (const __nv_bfloat16*)a.kc + slot * D, D);
-      copy_v(dst + kBS * KS * 2, VS * 2, (const __nv_bfloat16*)a.vc + slot * a.vdim + v0, a.vdim);
+      if (!tied) copy_v(dst + kBS * KS * 2, VS * 2, (const __nv_bfloat16*)a.vc + slot * a.vdim + v0, a.vdim);
+      else if (lane < 4) cp_async_16(dst + kBS * KS * 2 + lane * 16, a.key_scale + phys * kBS + lane * 4);
     }
     cp_async_commit();
     stage_in = stage_in + 1 == kRing ? 0 : stage_in + 1;
@@ -312,16 +383,26 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
     m[n][0] = m[n][1] = -INFINITY;
     l[n][0] = l[n][1] = 0.f;
   }
-  const float sc = a.scale * 1.4426950408889634f;  // scores in units of log2
+  const float sc = a.scale * kLog2e;  // scores in units of log2
+  float far[NT][2];                   // bias from distance dist_len - 1 on
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+      const int head = min(n * 8 + 2 * t + c, R - 1);
+      far[n][c] = EXT && a.dist_bias ? __ldg(a.dist_bias + (int64_t)(kvh * R + head + 1) * a.dist_len - 1) * kLog2e : 0.f;
+    }
   const uint32_t q_addr = smem_u32(s_q + (lane & 7) * KS + (lane >> 3) * 8);  // B fragments of two 16-channel steps
   const uint32_t k_off = (uint32_t)(((lane & 15) * KS + (lane >> 4) * 8) * 2);
-  const uint32_t v_off = (uint32_t)((kBS * KS + ((lane & 7) + (lane >> 4) * 8) * VS + ((lane >> 3) & 1) * 8) * 2);
+  const uint32_t v_off = (uint32_t)(((tied ? v0 : kBS * KS) + ((lane & 7) + (lane >> 4) * 8) * (tied ? KS : VS) +
+                                     ((lane >> 3) & 1) * 8) * 2);
   int stage = 0;
   for (int i = 0; i < n_w; ++i) {
     load(i + kRing - 1);
     cp_async_wait<kRing - 1>();
     __syncwarp();
     const uint32_t base = ring_u + stage * stage_elems * 2;
+    const __nv_bfloat16* stage_ptr = ring + stage * stage_elems;
     stage = stage + 1 == kRing ? 0 : stage + 1;
     float s[NT][2][4];  // two partial sums, so that neighbouring steps do not wait for each other
 #pragma unroll
@@ -344,15 +425,32 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
       }
     }
     const int key0 = runs.block(s_lo + warp + kWarps * i) * kBS;
-    const bool full = all_visible(key0, pos, pos, a.window, a.keep_first);
-    const bool see0 = full || visible(key0 + gi, pos, a.window, a.keep_first);
-    const bool see1 = full || visible(key0 + gi + 8, pos, a.window, a.keep_first);
+    const bool full = all_visible(key0, pos, lo, a.keep_first);
+    const bool see0 = full || visible(key0 + gi, pos, lo, a.keep_first);
+    const bool see1 = full || visible(key0 + gi + 8, pos, lo, a.keep_first);
+    float f0 = sc, f1 = sc;  // scales of keys gi and gi + 8
+    if (tied) {
+      const float* ks = reinterpret_cast<const float*>(stage_ptr + kBS * KS);
+      f0 *= ks[gi];
+      f1 *= ks[gi + 8];
+    }
+    const bool near = EXT && a.dist_bias && pos - (key0 + kBS - 1) < a.dist_len - 1;
+    const int d0 = near ? min(max(pos - key0 - gi, 0), a.dist_len - 1) : 0;
+    const int d1 = near ? min(max(pos - key0 - gi - 8, 0), a.dist_len - 1) : 0;
     uint32_t ph[NT][2], plo[NT][2];
 #pragma unroll
     for (int n = 0; n < NT; ++n) {
       float p[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) p[e] = (e < 2 ? see0 : see1) ? (s[n][0][e] + s[n][1][e]) * sc : -INFINITY;
+      for (int e = 0; e < 4; ++e) {
+        float b = far[n][e & 1];
+        if (near) {
+          const int head = min(n * 8 + 2 * t + (e & 1), R - 1);
+          b = __ldg(a.dist_bias + (int64_t)(kvh * R + head) * a.dist_len + (e < 2 ? d0 : d1)) * kLog2e;
+        }
+        const float x = s[n][0][e] + s[n][1][e];
+        p[e] = (e < 2 ? see0 : see1) ? (EXT ? fmaf(x, e < 2 ? f0 : f1, b) : x * sc) : -INFINITY;
+      }
       float x0 = fmaxf(p[0], p[2]), x1 = fmaxf(p[1], p[3]);
 #pragma unroll
       for (int w = 4; w < 32; w <<= 1) {
@@ -427,13 +525,23 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
       ls = fmaf(f[w], s_ml[(w * R + h) * 2 + 1], ls);
     }
     const int64_t head = (int64_t)kvh * R + h;
+    float inv = 1.f / ls;
+    if (a.sink && n_splits == 1) {
+      const float k = a.sink[head] * kLog2e, top = fmaxf(mx, k), f = ex2(mx - top);
+      inv = f / fmaf(ls, f, ex2(k - top));
+    }
     float* p = n_splits > 1 ? part + (((int64_t)blockIdx.x * a.heads + head) * n_splits + split) * (a.vdim + 2) : nullptr;
     for (int c = lane; c < VW; c += 32) {
       float acc = 0.f;
 #pragma unroll
       for (int w = 0; w < kWarps; ++w) acc = fmaf(f[w], s_o[((size_t)w * R + h) * OS + c], acc);
-      if (n_splits == 1) ((__nv_bfloat16*)a.out)[row * a.ld_out + head * a.vdim + v0 + c] = __float2bfloat16_rn(acc / ls);
-      else p[v0 + c] = acc;
+      if (n_splits == 1) {
+        acc *= inv;
+        if (a.gate) acc *= sigmoid_of(((const uint16_t*)a.gate)[row * a.ld_gate + head * a.vdim + v0 + c]);
+        ((__nv_bfloat16*)a.out)[row * a.ld_out + head * a.vdim + v0 + c] = __float2bfloat16_rn(acc);
+      } else {
+        p[v0 + c] = acc;
+      }
     }
     if (n_splits > 1 && lane == 0 && v0 == 0) { p[a.vdim] = mx; p[a.vdim + 1] = ls; }
   }
@@ -447,8 +555,10 @@ span_attention_merge_kernel(const SpanAttention a, const int32_t* __restrict__ r
   const int64_t row = rows[blockIdx.x];
   const int head = blockIdx.y;
   const float* p = part + ((int64_t)blockIdx.x * a.heads + head) * n_splits * (a.vdim + 2);
-  float mx = -INFINITY, l = 0.f;
+  float mx = a.sink ? a.sink[head] * kLog2e : -INFINITY, l = 0.f;
+  const float k = mx;
   for (int s = 0; s < n_splits; ++s) mx = fmaxf(mx, p[s * (a.vdim + 2) + a.vdim]);
+  if (a.sink) l = ex2(k - mx);
   for (int s = 0; s < n_splits; ++s) {
     const float m = p[s * (a.vdim + 2) + a.vdim];
     if (m != -INFINITY) l = fmaf(ex2(m - mx), p[s * (a.vdim + 2) + a.vdim + 1], l);
@@ -459,17 +569,19 @@ span_attention_merge_kernel(const SpanAttention a, const int32_t* __restrict__ r
       const float m = p[s * (a.vdim + 2) + a.vdim];
       if (m != -INFINITY) acc = fmaf(ex2(m - mx), p[s * (a.vdim + 2) + c], acc);
     }
-    ((__nv_bfloat16*)a.out)[row * a.ld_out + (int64_t)head * a.vdim + c] = __float2bfloat16_rn(acc / l);
+    acc /= l;
+    if (a.gate) acc *= sigmoid_of(((const uint16_t*)a.gate)[row * a.ld_gate + (int64_t)head * a.vdim + c]);
+    ((__nv_bfloat16*)a.out)[row * a.ld_out + (int64_t)head * a.vdim + c] = __float2bfloat16_rn(acc);
   }
 }
 
 static size_t tiles_smem(const SpanAttention& a, int stages) {
   const int KS = pad16(a.dim) + 8, VS = pad16(std::min(a.vdim, kSlice)) + 8;
-  return (size_t)(kRows * KS + stages * kKeys * (KS + VS)) * 2;
+  return (size_t)(kRows * KS + stages * kKeys * (KS + (a.key_scale ? 2 : VS))) * 2;
 }
 static size_t tokens_smem(const SpanAttention& a) {
   const int R = a.heads / a.kv_heads, KS = pad16(a.dim) + 8, VP = pad16(std::min(a.vdim, kSlice)), VS = VP + 8;
-  const size_t ring = (size_t)kWarps * kRing * kBS * (KS + VS) * 2;
+  const size_t ring = (size_t)kWarps * kRing * kBS * (KS + (a.key_scale ? 2 : VS)) * 2;
   const size_t merge = (size_t)kWarps * R * (VP + 4) * sizeof(float);
   return (size_t)16 * KS * 2 + std::max(ring, merge);
 }
@@ -479,7 +591,8 @@ static bool span_mma_ok(const SpanAttention& a, hb_dtype dtype) {
   auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   static const bool simt = [] { const char* e = getenv("HB_ATTN"); return e && e[0] == 's'; }();
   return !simt && dtype == HB_BF16 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ld_q % 8 == 0 && a.ld_out % 2 == 0 && al(a.q) &&
-         al(a.out);
+         al(a.out) && (!a.gate || (a.ld_gate % 2 == 0 && (reinterpret_cast<uintptr_t>(a.gate) & 3) == 0)) &&
+         (!a.key_scale || (a.dim == a.vdim && al(a.key_scale)));
 }
 
 int span_attention_tile_positions(const SpanAttention& a, hb_dtype dtype) {
@@ -509,10 +622,13 @@ int span_attention_tiles(cudaStream_t st, const SpanAttention& a, const RowRange
     return HB_OK;
   };
   const int vw = std::min(a.vdim, kSlice);
-  if (vw <= 64) return launch(span_attention_tiles_kernel<4>);
-  if (vw <= 128) return launch(span_attention_tiles_kernel<8>);
-  if (vw <= 192) return launch(span_attention_tiles_kernel<12>);
-  return launch(span_attention_tiles_kernel<16>);
+  const bool ext = a.key_scale || a.dist_bias;
+#define HB_TILES(NV) return ext ? launch(span_attention_tiles_kernel<NV, true>) : launch(span_attention_tiles_kernel<NV, false>)
+  if (vw <= 64) HB_TILES(4);
+  if (vw <= 128) HB_TILES(8);
+  if (vw <= 192) HB_TILES(12);
+  HB_TILES(16);
+#undef HB_TILES
 }
 
 int span_attention_tokens(cudaStream_t st, const SpanAttention& a, const int32_t* rows, int n_rows, int n_splits, float* part) {
@@ -529,9 +645,14 @@ int span_attention_tokens(cudaStream_t st, const SpanAttention& a, const int32_t
   const int vw = std::min(a.vdim, kSlice);
   int rc;
   const bool wide = a.heads / a.kv_heads > 8;
-  if (vw <= 64) rc = wide ? launch(span_attention_tokens_kernel<4, 2>) : launch(span_attention_tokens_kernel<4, 1>);
-  else if (vw <= 128) rc = wide ? launch(span_attention_tokens_kernel<8, 2>) : launch(span_attention_tokens_kernel<8, 1>);
-  else rc = wide ? launch(span_attention_tokens_kernel<16, 2>) : launch(span_attention_tokens_kernel<16, 1>);
+  const bool ext = a.key_scale || a.dist_bias;
+#define HB_TOKENS(MT)                                                                                                        \
+  rc = ext ? (wide ? launch(span_attention_tokens_kernel<MT, 2, true>) : launch(span_attention_tokens_kernel<MT, 1, true>)) \
+           : (wide ? launch(span_attention_tokens_kernel<MT, 2, false>) : launch(span_attention_tokens_kernel<MT, 1, false>))
+  if (vw <= 64) HB_TOKENS(4);
+  else if (vw <= 128) HB_TOKENS(8);
+  else HB_TOKENS(16);
+#undef HB_TOKENS
   if (rc || n_splits == 1) return rc;
   HB_CUDA_CHECK(launch_pdl(span_attention_merge_kernel, dim3((unsigned)n_rows, (unsigned)a.heads), dim3(kThreads), 0, st, a, rows,
                            n_splits, (const float*)part));

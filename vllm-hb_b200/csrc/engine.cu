@@ -1311,7 +1311,7 @@ int hb_kv_copy_blocks(hb_engine* e, const int64_t* pairs, size_t n_pairs) {
     HB_CUDA_CHECK(cudaMemcpyAsync(e->d_pairs, pairs + 2 * done, n * 2 * sizeof(int64_t), cudaMemcpyHostToDevice, e->stream));
     for (size_t l = 0; l < e->kc.size(); ++l) {
       int rc = hb::kv_copy_blocks(e->stream, e->kc[l], e->vc[l], e->d_pairs, (int64_t)n, (int64_t)e->k_block_bytes[l],
-                                  e->num_blocks);
+                                  (int64_t)e->v_block_bytes[l], e->num_blocks);
       if (rc) return rc;
     }
     HB_CUDA_CHECK(cudaStreamSynchronize(e->stream));  // `pairs` and d_pairs may be reused

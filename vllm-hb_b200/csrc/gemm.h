@@ -3,6 +3,8 @@
 
 #include <cuda.h>
 
+#include <cmath>
+
 #include "common.h"
 
 namespace hb {
@@ -11,10 +13,34 @@ namespace hb {
 int gemm_simt(cudaStream_t st, void* Y, const void* X, const void* W, int64_t M, int64_t N,
               int64_t K, hb_dtype dtype, bool out_f32);
 
+// Gated activation of a feed-forward: with g clipped from above and u to both sides at `limit`,
+//   act(g, u) = g * sigmoid(slope * (g + cubic * g^3)) * (u + shift).
+// The defaults are SiLU; gelu in its tanh form is slope = 2 sqrt(2 / pi), cubic = 0.044715, because
+// (1 + tanh(z)) / 2 = sigmoid(2 z).
+struct GatedAct {
+  float slope = 1.f, cubic = 0.f, limit = INFINITY, shift = 0.f;
+  bool silu() const { return slope == 1.f && cubic == 0.f && limit == INFINITY && shift == 0.f; }
+};
+// out[m, i] = act(gate_up[m, i], gate_up[m, inter + i]); rows of out have stride inter.
+int gated_act(cudaStream_t st, void* out, const void* gate_up, int64_t M, int64_t inter, const GatedAct& act, hb_dtype dtype);
+
+// Rows of a GEMM sorted by group (mixture of experts): every batch tile of `m_pad` rows belongs to
+// one group, whose weights start at row group * (weight rows of one group); tile_group[i] < 0: no
+// such tile.  The number of tiles is only known on the device; `max_tiles` bounds it, `likely_tiles`
+// steers the split of K.
+struct TcGroups {
+  int groups = 0;
+  int m_pad = 0;
+  int max_tiles = 0, likely_tiles = 0;
+};
+// CUDA-core form: Y[r] = X[r] . W[group of r]^T, tiles of m_pad rows (a multiple of 8).
+int gemm_simt_grouped(cudaStream_t st, void* Y, const void* X, const void* W, int64_t N, int64_t K, hb_dtype dtype, bool out_f32,
+                      const TcGroups& groups, const int32_t* tile_group);
+
 // What the tensor-core kernel does with the finished fp32 tile.
 enum TcEpilogue : int {
   kEpiStore = 0,     // Y = acc (bf16, or f32 when out_f32)
-  kEpiSwiGLU = 1,    // W rows are [gate tile | up tile] pairs: Y = silu(gate) * up, N_out = N/2
+  kEpiSwiGLU = 1,    // W rows are [gate tile | up tile] pairs: Y = act(gate, up) (GatedAct), N_out = N/2
   kEpiResidual = 2,  // deferred RMSNorm producer (cluster plans only), see TcNormLink
   kEpiPush = 3,      // row-parallel partial pushed into the reducing ranks' staging, see TcNormLink
 };
@@ -92,6 +118,9 @@ struct TcGemmPlan {
   int tmem_cols = 0;
   size_t smem_bytes = 0;
   int epilogue = kEpiStore;
+  GatedAct act;          // kEpiSwiGLU
+  int groups = 0;        // > 0: TcGroups form; rows of the batch operand are sorted by group
+  int group_rows = 0;    // weight rows of one group
   bool out_f32 = false;
   bool tma_store = false;  // output rows are 16-byte multiples: bulk tensor stores
   // scratch layout inside the caller's workspace
@@ -103,7 +132,9 @@ struct TcGemmPlan {
 bool gemm_tc_supported(int64_t M, int64_t N, int64_t K, hb_dtype dtype);
 // X and W must be 16-byte aligned device pointers; they are baked into the plan.
 int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int64_t N, int64_t K,
-                 int epilogue, bool out_f32, int device, int force_splits = 0);
+                 int epilogue, bool out_f32, int device, int force_splits = 0, const TcGroups* groups = nullptr);
+// groups: W holds the [N, K] matrices of all groups one after another, M is the row capacity of the
+// sorted batch operand; gemm_tc_run then needs tile_group (device, max_tiles entries).
 // Y row stride ldy in elements.  workspace: plan.workspace_bytes(), zeroed once.
 // err_flag (device int, may be null) is set non-zero when a bounded wait ran out.
 // True when `plan` can carry the RoPE + KV-write epilogue of TcNormLink.
@@ -113,6 +144,6 @@ bool gemm_tc_rope_epilogue_ok(const TcGemmPlan& plan);
 // the plan cannot push.
 int gemm_tc_push_row_block(const TcGemmPlan& plan);
 int gemm_tc_run(const TcGemmPlan& plan, cudaStream_t st, void* Y, int64_t ldy, void* workspace,
-                int* err_flag, const TcNormLink* link = nullptr);
+                int* err_flag, const TcNormLink* link = nullptr, const int32_t* tile_group = nullptr);
 
 }  // namespace hb

@@ -12,16 +12,20 @@ namespace hb {
 constexpr int kSimtWarps = 8;
 constexpr int kMB = 8;
 
+// tile_group (may be null): rows m belong to group tile_group[m / m_pad], whose weights are the
+// group-th [N, K] matrix of W; rows of a negative group are skipped (m_pad is a multiple of kMB).
 template <typename T, typename OutT, bool VEC>
 __global__ void __launch_bounds__(kSimtWarps * 32)
 gemm_simt_kernel(OutT* __restrict__ Y, const T* __restrict__ X, const T* __restrict__ W, int64_t M,
-                 int64_t N, int64_t K, int64_t ldy) {
+                 int64_t N, int64_t K, int64_t ldy, const int32_t* __restrict__ tile_group, int m_pad) {
   constexpr int NV = Vec16<T>::N;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int64_t n = (int64_t)blockIdx.x * kSimtWarps + warp;
   const int64_t m0 = (int64_t)blockIdx.y * kMB;
   if (n >= N) return;
-  const T* wr = W + n * K;
+  const int group = tile_group ? tile_group[m0 / m_pad] : 0;
+  if (group < 0) return;
+  const T* wr = W + ((int64_t)group * N + n) * K;
   float acc[kMB];
 #pragma unroll
   for (int i = 0; i < kMB; ++i) acc[i] = 0.f;
@@ -60,15 +64,15 @@ gemm_simt_kernel(OutT* __restrict__ Y, const T* __restrict__ X, const T* __restr
 
 template <typename T, typename OutT>
 static int launch_simt(cudaStream_t st, OutT* Y, const T* X, const T* W, int64_t M, int64_t N,
-                       int64_t K, int64_t ldy) {
+                       int64_t K, int64_t ldy, const int32_t* tile_group = nullptr, int m_pad = 1) {
   constexpr int NV = Vec16<T>::N;
   const bool vec = K % NV == 0 && (reinterpret_cast<uintptr_t>(X) & 15) == 0 &&
                    (reinterpret_cast<uintptr_t>(W) & 15) == 0;
   dim3 grid((unsigned)((N + kSimtWarps - 1) / kSimtWarps), (unsigned)((M + kMB - 1) / kMB));
   if (vec)
-    gemm_simt_kernel<T, OutT, true><<<grid, kSimtWarps * 32, 0, st>>>(Y, X, W, M, N, K, ldy);
+    gemm_simt_kernel<T, OutT, true><<<grid, kSimtWarps * 32, 0, st>>>(Y, X, W, M, N, K, ldy, tile_group, m_pad);
   else
-    gemm_simt_kernel<T, OutT, false><<<grid, kSimtWarps * 32, 0, st>>>(Y, X, W, M, N, K, ldy);
+    gemm_simt_kernel<T, OutT, false><<<grid, kSimtWarps * 32, 0, st>>>(Y, X, W, M, N, K, ldy, tile_group, m_pad);
   HB_LAUNCH_CHECK();
   return HB_OK;
 }
@@ -80,6 +84,20 @@ int gemm_simt(cudaStream_t st, void* Y, const void* X, const void* W, int64_t M,
     if (out_f32)
       return (launch_simt<T, float>(st, (float*)Y, (const T*)X, (const T*)W, M, N, K, N));
     return (launch_simt<T, T>(st, (T*)Y, (const T*)X, (const T*)W, M, N, K, N));
+  });
+  return HB_OK;
+}
+
+int gemm_simt_grouped(cudaStream_t st, void* Y, const void* X, const void* W, int64_t N, int64_t K, hb_dtype dtype, bool out_f32,
+                      const TcGroups& groups, const int32_t* tile_group) {
+  if (groups.m_pad % kMB || groups.m_pad < 1)
+    return fail(HB_ERR_INVALID_ARG, "gemm_simt_grouped: tiles of %d rows", groups.m_pad);
+  const int64_t M = (int64_t)groups.max_tiles * groups.m_pad;
+  if (M == 0 || N == 0) return HB_OK;
+  HB_DISPATCH_DTYPE(dtype, T, {
+    if (out_f32)
+      return (launch_simt<T, float>(st, (float*)Y, (const T*)X, (const T*)W, M, N, K, N, tile_group, groups.m_pad));
+    return (launch_simt<T, T>(st, (T*)Y, (const T*)X, (const T*)W, M, N, K, N, tile_group, groups.m_pad));
   });
   return HB_OK;
 }

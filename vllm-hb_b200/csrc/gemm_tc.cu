@@ -48,6 +48,10 @@ struct TcParams {
   int epilogue, out_f32;
   int64_t ldy;
   int up_row_offset;        // SwiGLU: first row of the up projection inside W
+  GatedAct act;             // activation of the pair; act_silu: the plain one
+  int act_silu;
+  const int32_t* tile_group;  // TcGroups: group of every batch tile (negative: no such tile)
+  int group_rows;             // weight rows of one group
   int cluster;              // split-K partners form a thread-block cluster of `splits` CTAs
   int tma_store;            // the output leaves through bulk tensor stores (tm_y is valid)
   // Deferred RMSNorm (see TcNormLink in gemm.h).  Producer (epilogue kEpiResidual, cluster
@@ -152,6 +156,16 @@ __device__ __forceinline__ void push_tile(const TcParams& p, const uint8_t* stag
     peer_st_release(&reinterpret_cast<CommFlags*>(p.push_peer[q])->tflag[(row_block * R + me) * T + ti], seq + 1);
 }
 
+// Gated activation of one output element (fast divide and exponential, as silu_f).
+__device__ __forceinline__ float gated_f(float g, float u, const TcParams& p) {
+  if (p.act_silu) return silu_f(g) * u;
+  g = fminf(g, p.act.limit);
+  u = fminf(fmaxf(u, -p.act.limit), p.act.limit);
+  const float z = p.act.slope * fmaf(p.act.cubic * g * g, g, g);
+  // far below zero the gate is zero (the fast divide wants a denominator below 2^126)
+  return z < -80.f ? 0.f : __fdividef(g, 1.f + __expf(-z)) * (u + p.act.shift);
+}
+
 // ----------------------------------------------------------------------- kernel
 __global__ void __launch_bounds__(kTcThreads, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x,
@@ -181,6 +195,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
   const int tile = blockIdx.x / p.splits;
   const int split = p.cluster ? (int)cluster_ctarank() : blockIdx.x % p.splits;
   const int m_tile = blockIdx.y;
+  int w_row = tile * kTileN;  // first weight row of the tile
+  if (p.tile_group) {
+    // rows sorted by group: the previous kernels say whose weights this batch tile meets
+    pdl_wait();
+    const int group = p.tile_group[m_tile];
+    if (group < 0) return;  // uniform over the grid row, so over every cluster
+    w_row += group * p.group_rows;
+  }
   const int base_c = p.k_chunks / p.splits, rem_c = p.k_chunks % p.splits;
   const int kc0 = split * base_c + min(split, rem_c);
   const int n_kc = base_c + (split < rem_c ? 1 : 0);
@@ -291,8 +313,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
         const uint32_t sa = smem_base + i * stage_bytes;
         mbar_expect_tx(full, stage_bytes);
         const int kx = (kc0 + i) * kTileK;
-        load_w(sa, kx, tile * kTileN, full);
-        if (swiglu) load_w(sa + a_bytes, kx, p.up_row_offset + tile * kTileN, full);
+        load_w(sa, kx, w_row, full);
+        if (swiglu) load_w(sa + a_bytes, kx, p.up_row_offset + w_row, full);
       }
       // (Requesting further chunks into L2 at this point was measured harmful: -2 % to -7 % per
       // decode step after HBM-bound kernels, no gain after an NVLink exchange.  Requesting the
@@ -316,8 +338,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
         const uint32_t sa = smem_base + s * stage_bytes;
         mbar_expect_tx(full, stage_bytes);
         const int kx = (kc0 + i) * kTileK;
-        load_w(sa, kx, tile * kTileN, full);
-        if (swiglu) load_w(sa + a_bytes, kx, p.up_row_offset + tile * kTileN, full);
+        load_w(sa, kx, w_row, full);
+        if (swiglu) load_w(sa + a_bytes, kx, p.up_row_offset + w_row, full);
         tma_load_2d(sa + a_bytes * n_acc, &tm_x, kx, m_tile * p.m_pad, full);
         armed = i + 1;
       }
@@ -505,7 +527,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           }
         }
 #pragma unroll
-        for (int j = 0; j < 16; ++j) g[j] = swiglu ? silu_f(g[j]) * u[j] : g[j];
+        for (int j = 0; j < 16; ++j) g[j] = swiglu ? gated_f(g[j], u[j], p) : g[j];
         if (p.post_scale) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) g[j] *= s_pscale[c0 + j];
@@ -653,7 +675,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
             for (int j = 0; j < 16; ++j) u[j] *= s_rscale[g * 16 + j];
           }
 #pragma unroll
-          for (int j = 0; j < 16; ++j) v[j] = silu_f(v[j]) * u[j];
+          for (int j = 0; j < 16; ++j) v[j] = gated_f(v[j], u[j], p);
         }
         if (p.post_scale) {
 #pragma unroll
@@ -693,7 +715,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           float u[16];
           tmem_ld16(t_lane + p.m_pad + c0, u);
 #pragma unroll
-          for (int j = 0; j < 16; ++j) v[j] = silu_f(v[j]) * u[j];
+          for (int j = 0; j < 16; ++j) v[j] = gated_f(v[j], u[j], p);
         }
         if (n_glob < p.N) {
 #pragma unroll
@@ -750,7 +772,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           for (int j = 0; j < 8; ++j) {
             const int m = m0 + j;
             if (m < m_lim && n_glob < p.N) {
-              const float r = swiglu ? silu_f(g[j]) * u[j] : g[j];
+              const float r = swiglu ? gated_f(g[j], u[j], p) : g[j];
               if (p.out_f32) ((float*)p.Y)[(int64_t)(m_base + m) * p.ldy + n_glob] = r;
               else ((__nv_bfloat16*)p.Y)[(int64_t)(m_base + m) * p.ldy + n_glob] = __float2bfloat16_rn(r);
             }
@@ -868,8 +890,7 @@ static int pick_cluster_splits(int units, int k_chunks, int sm_count) {
 }
 
 int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int64_t N, int64_t K,
-                 int epilogue, bool out_f32, int device, int force_splits) {
-
+                 int epilogue, bool out_f32, int device, int force_splits, const TcGroups* groups) {
   if (!gemm_tc_supported(M, N, K, HB_BF16))
     return fail(HB_ERR_INVALID_ARG, "gemm_tc: unsupported shape M=%lld N=%lld K=%lld", (long long)M,
                 (long long)N, (long long)K);
@@ -885,6 +906,11 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
   pl.M = M; pl.K = K;
   pl.epilogue = epilogue;
   pl.out_f32 = out_f32;
+  pl.groups = groups ? groups->groups : 0;
+  pl.group_rows = groups ? (int)N : 0;
+  if (groups && (groups->groups < 1 || groups->m_pad < 16 || groups->m_pad > 128 || groups->m_pad % 16 || groups->max_tiles < 1 ||
+                 groups->likely_tiles < 1 || (int64_t)groups->max_tiles * groups->m_pad > M || epilogue > kEpiSwiGLU))
+    return fail(HB_ERR_INVALID_ARG, "gemm_tc: bad groups");
   const int n_acc = epilogue == kEpiSwiGLU ? 2 : 1;
   if (epilogue == kEpiSwiGLU && N % 2) return fail(HB_ERR_INVALID_ARG, "gemm_tc: SwiGLU needs even N");
   const int64_t n_rows = epilogue == kEpiSwiGLU ? N / 2 : N;  // output features
@@ -899,19 +925,20 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
   const int k_chunks = (int)((K + kTileK - 1) / kTileK);
   const bool want_cluster = true;  // split-K partners reduce on chip; global scratch only where a cluster cannot form
   const bool tuned = want_cluster && force_splits <= 0;
+  if (groups) pl.m_pad = groups->m_pad;
   // Few weights under a wide batch (o_proj and q|k|v at high tensor-parallel degrees): the
   // split-K exchange moves 128 x m_pad fp32 per CTA through the SM-to-SM network, which at
   // m_pad = 128 costs more than the matrix takes to stream.  Two batch tiles of 64 rows read
   // the weight tile twice (the second time from L2) and need no, or a smaller, exchange
   // (measured: 8192 x 1024 at M = 128 15.4 -> 11.1 us, 1280 x 8192 19.0 -> 16.4 us).
   bool m_split = false;
-  if (tuned && n_acc == 1 && pl.m_pad >= 128 && (int64_t)pl.n_tiles * k_chunks <= 2048 &&
+  if (tuned && !groups && n_acc == 1 && pl.m_pad >= 128 && (int64_t)pl.n_tiles * k_chunks <= 2048 &&
       (epilogue == kEpiStore || epilogue == kEpiPush)) {
     pl.m_pad = 64;
     m_split = true;
   }
-  pl.m_tiles = (int)((M + pl.m_pad - 1) / pl.m_pad);
-  const int units = pl.n_tiles * pl.m_tiles;
+  pl.m_tiles = groups ? groups->max_tiles : (int)((M + pl.m_pad - 1) / pl.m_pad);
+  const int units = pl.n_tiles * (groups ? groups->likely_tiles : pl.m_tiles);
   const int acc_cols = pl.m_pad * n_acc;
   pl.tmem_cols = acc_cols <= 32 ? 32 : acc_cols <= 64 ? 64 : acc_cols <= 128 ? 128 : acc_cols <= 256 ? 256 : 512;
   const size_t stage = (size_t)kTileN * kTileK * 2 * n_acc + (size_t)pl.m_pad * kTileK * 2;
@@ -1014,7 +1041,7 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
   // The tile counters sit in a block of FIXED size at the start of the workspace, so
   // that plans of different shapes sharing one workspace never see each other's
   // partials where they expect zeroed counters.
-  if (!pl.cluster && (size_t)units * sizeof(int) > kCounterBlockBytes) pl.splits = 1;
+  if (!pl.cluster && ((size_t)units * sizeof(int) > kCounterBlockBytes || groups)) pl.splits = 1;
   pl.ws_partials_bytes = (pl.splits > 1 && !pl.cluster) ? (size_t)units * pl.splits * n_acc * pl.m_pad * kTileN * sizeof(float) : 0;
   pl.ws_counters_bytes = (pl.splits > 1 && !pl.cluster) ? kCounterBlockBytes : 0;
   // opt in to the large dynamic shared memory window once per device (here, not at
@@ -1032,7 +1059,7 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
       dev_done[cur] = true;
     }
   }
-  rc = encode_map(&pl.tm_w, W, N, K, kTileN);
+  rc = encode_map(&pl.tm_w, W, groups ? N * groups->groups : N, K, kTileN);
   if (rc) return rc;
   rc = encode_map(&pl.tm_x, X, M, K, pl.m_pad);
   return rc;
@@ -1053,12 +1080,13 @@ bool gemm_tc_rope_epilogue_ok(const TcGemmPlan& pl) {
 }
 
 int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, void* workspace,
-                int* err_flag, const TcNormLink* link) {
+                int* err_flag, const TcNormLink* link, const int32_t* tile_group) {
+  if ((pl.groups > 0) != (tile_group != nullptr) || (tile_group && link))
+    return fail(HB_ERR_INVALID_ARG, "gemm_tc: grouped plans (and no others) run with a list of tile groups and without a link");
   if (pl.splits > 1 && !pl.cluster && !workspace)
     return fail(HB_ERR_INVALID_ARG, "gemm_tc: split-K plan needs a workspace of %zu bytes",
                 pl.workspace_bytes());
-  TcParams p;
-  memset(&p, 0, sizeof(p));
+  TcParams p{};
 #ifdef HB_TC_TRACE
   static std::atomic<int> launch_no{0};
   p.trace_id = launch_no.fetch_add(1) % kLaunchRing;
@@ -1070,6 +1098,10 @@ int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, voi
   p.epilogue = pl.epilogue; p.out_f32 = pl.out_f32 ? 1 : 0;
   p.ldy = ldy;
   p.up_row_offset = (int)pl.N;
+  p.act = pl.act;
+  p.act_silu = pl.act.silu() ? 1 : 0;
+  p.tile_group = tile_group;
+  p.group_rows = pl.group_rows;
   p.Y = Y;
   // counters first (16-byte aligned block), partials after
   p.counters = (int*)workspace;

@@ -6,12 +6,9 @@
 #include <climits>
 #include <cmath>
 
-#include "json.h"
-#include "layered.h"
+#include "design_reader.h"
 
 namespace hb {
-
-static int64_t int_of(const Json* j, const char* key) { return j ? (int64_t)j->number_or(key, 0) : 0; }
 
 bool is_latarax(const Json& config) { return config.string_or("architecture", "") == "Latarax"; }
 
@@ -23,13 +20,6 @@ static int read_window(const Json* mask, AttentionSpec* a) {
   a->window = (int)(size > INT_MAX / 2 ? 0 : size);
   a->keep_first = (int)(keep > INT_MAX / 2 ? INT_MAX / 2 : keep);
   return HB_OK;
-}
-
-static void place(ProjPart* p, std::string tensor, int64_t rows, int64_t* offset) {
-  p->tensor = std::move(tensor);
-  p->rows = rows;
-  p->offset = *offset;
-  *offset = (*offset + rows + 7) / 8 * 8;
 }
 
 static int read_gla(const Json* m, const std::string& t, MixerSpec* out) {
@@ -106,6 +96,7 @@ static int read_parallel(const Json* m, const std::string& t, MixerSpec* out) {
 
 int read_latarax(const Json& config, LayeredSpec* out) {
   out->design = "Latarax";
+  out->norm_offset = 1.f;
   out->width = int_of(&config, "width");
   out->vocab = int_of(&config, "vocab");
   out->max_positions = int_of(&config, "max_positions");
@@ -137,18 +128,18 @@ int read_latarax(const Json& config, LayeredSpec* out) {
     const Json* mlp = j.get("mlp");
     if (mlp && mlp->kind == Json::Obj) {
       const std::string kind = mlp->string_or("kind", "dense");
-      l.ff = int_of(mlp, "ff");
-      if (kind != "dense" || l.ff < 1) return fail(HB_ERR_INVALID_ARG, "config.json: layer %zu has a bad feed-forward", i);
+      l.ffn.ff = int_of(mlp, "ff");
+      if (kind != "dense" || l.ffn.ff < 1) return fail(HB_ERR_INVALID_ARG, "config.json: layer %zu has a bad feed-forward", i);
       l.norm2 = l.prefix + "norm2";
-      l.gate = l.prefix + "mlp.gate";
-      l.up = l.prefix + "mlp.up";
-      l.down = l.prefix + "mlp.down";
+      l.ffn.gate = l.prefix + "mlp.gate";
+      l.ffn.up = l.prefix + "mlp.up";
+      l.ffn.down = l.prefix + "mlp.down";
     }
     if (mixed) {
       l.hc1_in = l.prefix + "hc1.in";
       l.hc1_out = l.prefix + "hc1.out";
       l.hc1_mix = l.prefix + "hc1.mix";
-      if (l.ff) {
+      if (l.ffn.ff) {
         l.hc2_in = l.prefix + "hc2.in";
         l.hc2_out = l.prefix + "hc2.out";
         l.hc2_mix = l.prefix + "hc2.mix";

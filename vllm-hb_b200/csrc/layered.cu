@@ -1,5 +1,6 @@
 // The layered family: weights, pools and the step of models described by a LayeredSpec.
 #include <algorithm>
+#include <cmath>
 #include <cstring>
 
 #include "engine.h"
@@ -16,13 +17,26 @@ static int64_t pad8(int64_t n) { return (n + 7) / 8 * 8; }
 static int64_t pad_to(int64_t n, int64_t m) { return (n + m - 1) / m * m; }
 
 // ------------------------------------------------------------------------------- load
-static bool layered_serves(const Json& config) { return is_latarax(config); }
+// The designs of this family: which config.json a reader takes, and the reader.
+struct LayeredDesign {
+  bool (*serves)(const Json&);
+  int (*read)(const Json&, LayeredSpec*);
+};
+static const LayeredDesign kDesigns[] = {{is_latarax, read_latarax}, {is_biberax, read_biberax}};
+
+static const LayeredDesign* design_of(const Json& config) {
+  for (const LayeredDesign& d : kDesigns)
+    if (d.serves(config)) return &d;
+  return nullptr;
+}
+
+static bool layered_serves(const Json& config) { return design_of(config) != nullptr; }
 
 static int layered_configure(hb_engine* e, const Json& config) {
   if (e->ws > 1) return fail(HB_ERR_INVALID_ARG, "this design runs on one rank");
   if (e->dtype == HB_F16) return fail(HB_ERR_UNSUPPORTED_DTYPE, "this design runs in bf16 or f32, not f16");
   e->lm.reset(new LayeredModel);
-  int rc = read_latarax(config, &e->lm->spec);
+  int rc = design_of(config)->read(config, &e->lm->spec);
   if (rc) return rc;
   const LayeredSpec& s = e->lm->spec;
   if (s.streams < 1 || s.streams > kMaxStreams)
@@ -59,6 +73,9 @@ struct Loader {
     int rc = alloc(lin, pad8(n), k);
     return rc ? rc : part(*lin, name, 0, n, k);
   }
+  int vector(float** dst, const std::string& name, int64_t n, float neutral) {  // none where the design names none
+    return name.empty() ? HB_OK : small(dst, name, 1, n, neutral);
+  }
   // fp32 vector or small matrix; generated weights take `neutral` (mix: the identity)
   int small(float** dst, const std::string& name, int64_t rows, int64_t cols, float neutral, bool identity = false) {
     int rc = dev_alloc(e, (void**)dst, (size_t)rows * cols * 4);
@@ -93,7 +110,66 @@ struct Loader {
       if ((rc = small(&q->out, out, 1, S, 1.f))) return rc;
       if ((rc = small(&q->mix, mix, S, S, 0.f, true))) return rc;
     }
-    return small(&q->norm, norm, 1, m->spec.width, 0.f);
+    return small(&q->norm, norm, 1, m->spec.width, 1.f - m->spec.norm_offset);
+  }
+  int attention(LayeredLayer* l, const MixerSpec& mx) {
+    const AttentionSpec& a = mx.attn;
+    const int64_t q = (int64_t)a.heads * a.dim, k = (int64_t)a.kv_heads * a.dim;
+    int rc;
+    if ((rc = linear(&l->attn_o, mx.attn_o, m->spec.width, (int64_t)a.heads * a.vdim))) return rc;
+    if ((rc = vector(&l->q_bias, mx.attn_q_bias, q, 0.f))) return rc;
+    if ((rc = vector(&l->k_bias, mx.attn_k_bias, k, 0.f))) return rc;
+    if ((rc = vector(&l->o_bias, mx.attn_o_bias, m->spec.width, 0.f))) return rc;
+    if ((rc = vector(&l->q_norm, mx.attn_q_norm, q, 1.f))) return rc;
+    if ((rc = vector(&l->k_norm, mx.attn_k_norm, k, 1.f))) return rc;
+    if ((rc = vector(&l->sink, mx.attn_sink, a.heads, 0.f))) return rc;
+    if (a.unit_sink) {
+      if ((rc = dev_alloc(e, (void**)&l->sink, (size_t)a.heads * 4, true))) return rc;
+    }
+    if (!mx.attn_rel.empty()) {
+      const std::vector<int64_t> shape = src.shape(mx.attn_rel);
+      if (!src.generated() && (shape.size() != 2 || shape[0] < 1 || shape[0] > (1 << 20)))
+        return fail(HB_ERR_IO, "Weight not found: %s", mx.attn_rel.c_str());
+      l->buckets = src.generated() ? 32 : (int)shape[0];  // the number of buckets is the tensor's own
+      if ((rc = small(&l->rel, mx.attn_rel, l->buckets, a.heads, 0.f))) return rc;
+    }
+    if (!a.rotation.empty()) {
+      if ((rc = dev_alloc(e, (void**)&l->rotation, a.rotation.size() * 8))) return rc;
+      HB_CUDA_CHECK(cudaMemcpyAsync(l->rotation, a.rotation.data(), a.rotation.size() * 8, cudaMemcpyHostToDevice, e->stream));
+      HB_CUDA_CHECK(cudaStreamSynchronize(e->stream));
+    }
+    return HB_OK;
+  }
+  int gated(LayeredLinear* gate_up, LayeredLinear* down, int64_t* ffp, const FeedForwardSpec& f) {
+    const int64_t W = m->spec.width;
+    int rc;
+    *ffp = pad8(f.ff);
+    if ((rc = alloc(gate_up, 2 * *ffp, W))) return rc;
+    if ((rc = part(*gate_up, f.gate, 0, f.ff, W))) return rc;
+    if ((rc = part(*gate_up, f.up, *ffp, f.ff, W))) return rc;
+    return linear(down, f.down, W, f.ff);
+  }
+  int experts(LayeredExperts* x, const ExpertsSpec& s) {
+    const int64_t W = m->spec.width, E = s.experts;
+    int rc;
+    x->ffp = pad8(s.ff);
+    LayeredLinear all_up, all_down;
+    if ((rc = alloc(&all_up, E * 2 * x->ffp, W)) || (rc = alloc(&all_down, E * pad8(W), s.ff))) return rc;
+    for (int64_t i = 0; i < E; ++i) {
+      const std::string t = s.prefix + std::to_string(i) + ".";
+      if ((rc = part(all_up, t + "gate", i * 2 * x->ffp, s.ff, W))) return rc;
+      if ((rc = part(all_up, t + "up", (i * 2 + 1) * x->ffp, s.ff, W))) return rc;
+      if ((rc = part(all_down, t + "down", i * pad8(W), W, s.ff))) return rc;
+    }
+    x->gate_up = all_up;
+    x->gate_up.N = 2 * x->ffp;
+    x->down = all_down;
+    x->down.N = pad8(W);
+    if ((rc = dev_alloc(e, &x->router, (size_t)E * W * e->es))) return rc;
+    if ((rc = src.fetch_all(s.router, E, W, x->router, e->dtype))) return rc;
+    e->named[s.router] = {x->router, E, W};
+    m->params += E * W;
+    return small(&x->router_bias, s.router_bias, 1, E, 0.f);
   }
 };
 }  // namespace
@@ -108,13 +184,16 @@ static int layered_load(hb_engine* e, TensorSource& src) {
   if ((rc = dev_alloc(e, &m->embed, (size_t)s.vocab * W * e->es))) return rc;
   if ((rc = src.fetch_all(s.embed, s.vocab, W, m->embed, e->dtype))) return rc;
   e->named[s.embed] = {m->embed, s.vocab, W};
-  if ((rc = dev_alloc(e, &m->pos, (size_t)s.max_positions * W * e->es))) return rc;
-  if ((rc = src.fetch_all(s.pos, s.max_positions, W, m->pos, e->dtype))) return rc;
-  e->named[s.pos] = {m->pos, s.max_positions, W};
-  m->params += (s.vocab + s.max_positions) * W;
+  m->params += s.vocab * W;
+  if (!s.pos.empty()) {
+    if ((rc = dev_alloc(e, &m->pos, (size_t)s.max_positions * W * e->es))) return rc;
+    if ((rc = src.fetch_all(s.pos, s.max_positions, W, m->pos, e->dtype))) return rc;
+    e->named[s.pos] = {m->pos, s.max_positions, W};
+    m->params += s.max_positions * W;
+  }
   if ((rc = ld.alloc(&m->head, s.vocab, W))) return rc;
   if ((rc = ld.part(m->head, s.head, 0, s.vocab, W))) return rc;
-  if ((rc = ld.small(&m->final_norm, s.final_norm, 1, W, 0.f))) return rc;
+  if ((rc = ld.small(&m->final_norm, s.final_norm, 1, W, 1.f - s.norm_offset))) return rc;
   m->layers.resize(s.layers.size());
   for (size_t i = 0; i < s.layers.size(); ++i) {
     LayerSpec& sp = s.layers[i];
@@ -128,15 +207,13 @@ static int layered_load(hb_engine* e, TensorSource& src) {
       if (mx.rec.rank < 1) return fail(HB_ERR_IO, "%s is empty", mx.ra1.tensor.c_str());
     }
     int64_t n = 0;
-    const ProjPart* parts[] = {&mx.aq, &mx.ak, &mx.av, &mx.rq, &mx.rk, &mx.rv, &mx.rg, &mx.ra1};
+    const ProjPart* parts[] = {&mx.aq, &mx.ak, &mx.av, &mx.ag, &mx.rq, &mx.rk, &mx.rv, &mx.rg, &mx.ra1};
     for (const ProjPart* p : parts)
       if (p->rows) n = std::max(n, p->offset + p->rows);
     if ((rc = ld.alloc(&l.proj, pad8(n), W))) return rc;
     for (const ProjPart* p : parts)
       if (p->rows && (rc = ld.part(l.proj, p->tensor, p->offset, p->rows, W))) return rc;
-    if (mx.has_attn) {
-      if ((rc = ld.linear(&l.attn_o, mx.attn_o, W, (int64_t)mx.attn.heads * mx.attn.vdim))) return rc;
-    }
+    if (mx.has_attn && (rc = ld.attention(&l, mx))) return rc;
     if (mx.has_rec) {
       const RecurrenceSpec& r = mx.rec;
       const int64_t hd = (int64_t)r.heads * r.dim, hv = (int64_t)r.heads * r.vdim;
@@ -158,12 +235,9 @@ static int layered_load(hb_engine* e, TensorSource& src) {
       if ((rc = ld.small(&l.rec_out_norm, mx.rec_out_norm, 1, W, 1.f))) return rc;
     }
     if ((rc = ld.sublayer(&l.sub1, sp.hc1_in, sp.hc1_out, sp.hc1_mix, sp.norm1))) return rc;
-    if (sp.ff) {
-      l.ffp = pad8(sp.ff);
-      if ((rc = ld.alloc(&l.gate_up, 2 * l.ffp, W))) return rc;
-      if ((rc = ld.part(l.gate_up, sp.gate, 0, sp.ff, W))) return rc;
-      if ((rc = ld.part(l.gate_up, sp.up, l.ffp, sp.ff, W))) return rc;
-      if ((rc = ld.linear(&l.down, sp.down, W, sp.ff))) return rc;
+    if (sp.ffn.ff && (rc = ld.gated(&l.gate_up, &l.down, &l.ffp, sp.ffn))) return rc;
+    if (sp.moe.experts && (rc = ld.experts(&l.moe, sp.moe))) return rc;
+    if (sp.has_ffn()) {
       if ((rc = ld.sublayer(&l.sub2, sp.hc2_in, sp.hc2_out, sp.hc2_mix, sp.norm2))) return rc;
     }
   }
@@ -216,8 +290,92 @@ static SpanAttention span_args(const hb_engine* e, size_t i, const LayeredStep& 
   a.row_seg = (const int32_t*)(e->d_inputs + s.off_row_seg);
   a.pos = (const int32_t*)(e->d_inputs + s.off_pos);
   a.heads = as.heads; a.kv_heads = as.kv_heads; a.dim = as.dim; a.vdim = as.vdim;
-  a.window = as.window; a.keep_first = as.keep_first; a.scale = as.scale;
+  a.window = as.window; a.keep_first = as.keep_first; a.chunk = as.chunk; a.scale = as.scale;
+  if (as.values_are_keys) {  // the second pool holds the keys' scales
+    a.key_scale = (const float*)a.vc;
+    a.vc = nullptr;
+  }
+  a.dist_bias = l.dist_bias; a.dist_len = l.dist_len;
+  a.sink = l.sink;
+  if (mx.ag.rows) {
+    a.gate = (const uint8_t*)m->proj + mx.ag.offset * e->es;
+    a.ld_gate = l.proj.N;
+  }
   return a;
+}
+
+// Queries in place, keys and values to their slots; false: the design only needs the K/V write.
+static bool prep_args(const hb_engine* e, size_t i, const LayeredStep& s, AttentionPrep* p) {
+  const LayeredModel* m = e->lm.get();
+  const MixerSpec& mx = m->spec.layers[i].mixer;
+  const LayeredLayer& l = m->layers[i];
+  const AttentionSpec& as = mx.attn;
+  if (!l.rotation && !l.q_norm && !l.q_bias) return false;
+  p->p = m->proj; p->ld = l.proj.N;
+  p->off_q = (int)mx.aq.offset; p->off_k = (int)mx.ak.offset; p->off_v = (int)mx.av.offset;
+  p->heads = as.heads; p->kv_heads = as.kv_heads; p->dim = as.dim; p->vdim = as.vdim;
+  p->pos = (const int32_t*)(e->d_inputs + s.off_pos);
+  p->slots = (const int64_t*)(e->d_inputs + s.off_slots);
+  p->kc = e->kc[l.kv_pool]; p->vc = e->vc[l.kv_pool]; p->num_blocks = e->num_blocks;
+  p->q_bias = l.q_bias; p->k_bias = l.k_bias; p->q_norm = l.q_norm; p->k_norm = l.k_norm;
+  p->eps = m->spec.eps;
+  p->rotation = l.rotation; p->pairs = (int)as.rotation.size();
+  if (as.values_are_keys) p->key_scale = (float*)p->vc;
+  return true;
+}
+
+// Row of the bias table for distance n: exact below half of the buckets, logarithmic above.
+static int distance_bucket(int64_t n, int buckets, double far) {
+  const int half = buckets / 2;
+  if (n < half) return (int)n;
+  if (half == 0 || far <= half) return buckets - 1;
+  const double x = std::log((double)n / half) / std::log(far / half) * (buckets - half);
+  return x >= buckets - half ? buckets - 1 : std::min(buckets - 1, half + (int)std::floor(x));
+}
+
+// The bias by distance, up to where it no longer changes (or no sequence reaches).
+static int build_distance_bias(hb_engine* e, LayeredLayer* l, const AttentionSpec& a, int64_t max_seq) {
+  std::vector<int32_t> bucket;
+  for (int64_t n = 0; n < max_seq; ++n) {
+    bucket.push_back(distance_bucket(n, l->buckets, a.bias_far));
+    if (bucket.back() == l->buckets - 1) break;
+  }
+  l->dist_len = (int)bucket.size();
+  int32_t* d = nullptr;
+  int rc;
+  if ((rc = dev_alloc(e, (void**)&l->dist_bias, (size_t)a.heads * l->dist_len * 4))) return rc;
+  HB_CUDA_CHECK(cudaMalloc((void**)&d, bucket.size() * 4));
+  rc = cudaMemcpyAsync(d, bucket.data(), bucket.size() * 4, cudaMemcpyHostToDevice, e->stream) == cudaSuccess
+           ? expand_distance_bias(e->stream, l->dist_bias, l->rel, d, a.heads, l->dist_len)
+           : fail(HB_ERR_CUDA, "upload of the distance buckets failed");
+  const cudaError_t ce = cudaStreamSynchronize(e->stream);
+  cudaFree(d);
+  if (rc) return rc;
+  HB_CUDA_CHECK(ce);
+  return HB_OK;
+}
+
+// Batch tiles of a mixture for `rows` rows of a step: tiles of about the rows an expert gets.
+static TcGroups moe_groups(const ExpertsSpec& x, int rows, bool tc) {
+  TcGroups g;
+  const int64_t n = (int64_t)rows * x.top;
+  g.groups = x.experts;
+  g.m_pad = tc ? (int)std::min<int64_t>(128, pad_to((n * 3 / 2 + x.experts - 1) / x.experts, 16)) : 16;
+  g.max_tiles = (int)(std::min<int64_t>(x.experts, n) + n / g.m_pad);
+  // experts that some row of a random batch chooses, and their tiles
+  const double active = x.experts * (1.0 - std::pow(1.0 - 1.0 / x.experts, (double)n));
+  const double tiles = active * std::max(1.0, std::ceil((double)n / std::max(1.0, active) / g.m_pad));
+  g.likely_tiles = (int)std::max<int64_t>(1, std::min<int64_t>((int64_t)tiles, g.max_tiles));
+  return g;
+}
+
+static MoeRouting moe_args(const LayeredModel* m, const ExpertsSpec& x, const TcGroups& g) {
+  MoeRouting r;
+  r.experts = x.experts; r.top = x.top;
+  r.m_pad = g.m_pad; r.max_tiles = g.max_tiles;
+  r.ids = m->moe_ids; r.rank = m->moe_rank; r.place = m->moe_place; r.weight = m->moe_weight;
+  r.count = m->moe_count; r.first = m->moe_first; r.tile_group = m->moe_tiles;
+  return r;
 }
 
 // Prompt portions as tiles, decoded tokens as rows; sizes the tensor-core kernels do not take go
@@ -239,7 +397,8 @@ static int issue_attention(hb_engine* e, const SpanAttention& a, const LayeredSt
   ++e->last_launches;
   if (!span_attention_tokens_supported(a, e->dtype)) return span_attention_rows(st, a, rows, s.n_token_rows, e->dtype);
   // the longest span a row can have decides the split: it is the same in every replay of a graph
-  const int64_t longest = a.window > 0 ? (int64_t)a.window + a.keep_first : a.max_blocks * HB_BLOCK_SIZE;
+  const int64_t span = a.chunk > 0 ? a.chunk : a.window;
+  const int64_t longest = span > 0 ? span + a.keep_first : a.max_blocks * HB_BLOCK_SIZE;
   const int64_t blocks = std::min<int64_t>(longest / HB_BLOCK_SIZE + 2, a.max_blocks), units = (int64_t)s.n_token_rows * a.kv_heads;
   int64_t splits = units < kSplitUnits / 2 ? std::min((kSplitUnits + units - 1) / units, (blocks + 15) / 16) : 1;
   splits = std::max<int64_t>(1, std::min<int64_t>(splits, 16));
@@ -269,7 +428,7 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   int rc;
   e->max_batch = cfg->max_batch > 0 ? cfg->max_batch : 256;
   int64_t max_seq = cfg->max_seq_len > 0 ? (int64_t)cfg->max_seq_len : 2048;
-  max_seq = std::min(max_seq, s.max_positions);
+  if (s.max_positions > 0) max_seq = std::min(max_seq, s.max_positions);
   e->max_blocks_per_seq = (max_seq + HB_BLOCK_SIZE - 1) / HB_BLOCK_SIZE;
   m->max_segs = std::min(e->max_batch, cfg->max_seqs > 0 ? cfg->max_seqs : e->max_batch);
   e->num_blocks = cfg->num_kv_blocks > 0 ? cfg->num_kv_blocks : e->max_blocks_per_seq * m->max_segs;
@@ -278,6 +437,7 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   m->row_cap = R;
   m->max_chunks = e->max_batch / kRecChunk + std::min(m->max_segs, e->max_batch / (kShortSegment + 1)) + 1;
   int64_t max_attn = 0, max_rec = 0, max_o = 0, max_ffp = 0, max_cum = 0, max_state = 0, max_part = 0;
+  int64_t max_experts = 0, max_top = 0, max_eff = 0, max_tiles = 0;
   for (size_t i = 0; i < s.layers.size(); ++i) {
     LayeredLayer& l = m->layers[i];
     const MixerSpec& mx = s.layers[i].mixer;
@@ -286,7 +446,9 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
     if (mx.has_attn) {
       const AttentionSpec& a = mx.attn;
       l.kv_pool = (int)e->kc.size();
-      const size_t kb = (size_t)a.kv_heads * HB_BLOCK_SIZE * a.dim * es, vb = (size_t)a.kv_heads * HB_BLOCK_SIZE * a.vdim * es;
+      const size_t kb = (size_t)a.kv_heads * HB_BLOCK_SIZE * a.dim * es;
+      // values that are the keys: the second pool holds one scale per token
+      const size_t vb = a.values_are_keys ? (size_t)HB_BLOCK_SIZE * 4 : (size_t)a.kv_heads * HB_BLOCK_SIZE * a.vdim * es;
       void *k = nullptr, *v = nullptr;
       // unwritten slots may be fetched (and masked): keep them finite
       if ((rc = dev_alloc(e, &k, kb * e->num_blocks, true))) return rc;
@@ -297,6 +459,18 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
       e->v_block_bytes.push_back(vb);
       max_attn = std::max(max_attn, l.attn_o.K);
       max_part = std::max(max_part, (int64_t)kSplitUnits * 2 * (a.heads / a.kv_heads) * (a.vdim + 2));
+      if (l.rel && (rc = build_distance_bias(e, &l, a, e->max_blocks_per_seq * HB_BLOCK_SIZE))) return rc;
+    }
+    if (const ExpertsSpec& x = s.layers[i].moe; x.experts) {
+      if (x.experts > kMoeMaxExperts) return fail(HB_ERR_INVALID_ARG, "%d experts (at most %d)", x.experts, kMoeMaxExperts);
+      max_experts = std::max<int64_t>(max_experts, x.experts);
+      max_top = std::max<int64_t>(max_top, x.top);
+      max_eff = std::max(max_eff, l.moe.ffp);
+      for (int64_t M = 16; M <= R; M += 16) {
+        const TcGroups g = moe_groups(x, (int)M, e->use_tc);
+        max_tiles = std::max<int64_t>(max_tiles, g.max_tiles);
+        m->moe_places = std::max<int64_t>(m->moe_places, (int64_t)g.max_tiles * g.m_pad);
+      }
     }
     if (mx.has_rec) {
       const RecurrenceSpec& r = mx.rec;
@@ -331,11 +505,26 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   if ((rc = dev_alloc(e, (void**)&m->y2, (size_t)R * m->Hp * 4, true))) return rc;
   if (!e->use_tc && (rc = dev_alloc(e, &m->gu, (size_t)R * 2 * max_ffp * es, true))) return rc;
   if ((rc = dev_alloc(e, &m->act, (size_t)R * max_ffp * es, true))) return rc;
+  if (max_experts) {
+    const size_t picks = (size_t)R * max_top * 4;
+    if ((rc = dev_alloc(e, &m->moe_x, (size_t)m->moe_places * m->Hp * es, true))) return rc;
+    if ((rc = dev_alloc(e, &m->moe_act, (size_t)m->moe_places * max_eff * es, true))) return rc;
+    if ((rc = dev_alloc(e, &m->moe_y, (size_t)m->moe_places * m->Hp * es, true))) return rc;
+    if (!e->use_tc && (rc = dev_alloc(e, &m->moe_gu, (size_t)m->moe_places * 2 * max_eff * es, true))) return rc;
+    if ((rc = dev_alloc(e, (void**)&m->moe_ids, picks, true))) return rc;
+    if ((rc = dev_alloc(e, (void**)&m->moe_rank, picks, true))) return rc;
+    if ((rc = dev_alloc(e, (void**)&m->moe_place, picks, true))) return rc;
+    if ((rc = dev_alloc(e, (void**)&m->moe_weight, picks, true))) return rc;
+    if ((rc = dev_alloc(e, (void**)&m->moe_count, (size_t)(max_experts + 1) * 4, true))) return rc;
+    if ((rc = dev_alloc(e, (void**)&m->moe_first, (size_t)max_experts * 4, true))) return rc;
+    if ((rc = dev_alloc(e, (void**)&m->moe_tiles, (size_t)max_tiles * 4, true))) return rc;
+  }
   if ((rc = dev_alloc(e, &m->hf, (size_t)LR * m->Hp * es, true))) return rc;
   if ((rc = dev_alloc(e, (void**)&e->d_logits, (size_t)LR * s.vocab * 4))) return rc;
   if ((rc = dev_alloc(e, (void**)&e->d_next, (size_t)LR * 4, true))) return rc;
   HB_CUDA_CHECK(cudaMallocHost((void**)&e->h_next, (size_t)LR * 4));
   if ((rc = dev_alloc(e, (void**)&e->d_err, 16, true))) return rc;
+  if ((rc = dev_alloc(e, (void**)&e->d_pairs, (size_t)kPairCap * 2 * sizeof(int64_t)))) return rc;
   // the largest step: every list at its longest
   LayeredStep cap;
   cap.rows = e->max_batch;
@@ -361,7 +550,7 @@ static int layered_plans(hb_engine* e, int rows, LayeredPlans** out) {
   if (it != m->plans.end()) { *out = &it->second; return HB_OK; }
   LayeredPlans p;
   const size_t L = m->layers.size();
-  p.proj.resize(L); p.attn_o.resize(L); p.rec_o.resize(L); p.gate_up.resize(L); p.down.resize(L);
+  for (auto* v : {&p.proj, &p.attn_o, &p.rec_o, &p.gate_up, &p.down, &p.moe_gate_up, &p.moe_down}) v->resize(L);
   size_t ws = 0;
   int rc;
   auto plan = [&](TcGemmPlan* pl, const void* X, const LayeredLinear& w, int epi, bool f32) -> int {
@@ -376,7 +565,17 @@ static int layered_plans(hb_engine* e, int rows, LayeredPlans** out) {
     if ((rc = plan(&p.attn_o[i], m->attn, l.attn_o, kEpiStore, true))) return rc;
     if ((rc = plan(&p.rec_o[i], m->rec, l.rec_o, kEpiStore, true))) return rc;
     if ((rc = plan(&p.gate_up[i], m->h, l.gate_up, kEpiSwiGLU, false))) return rc;
+    p.gate_up[i].act = m->spec.layers[i].ffn.act;
     if ((rc = plan(&p.down[i], m->act, l.down, kEpiStore, true))) return rc;
+    const ExpertsSpec& x = m->spec.layers[i].moe;
+    if (!x.experts) continue;
+    const TcGroups g = moe_groups(x, M, true);
+    if ((int64_t)g.max_tiles * g.m_pad > m->moe_places) return fail(HB_ERR_INVALID_ARG, "experts of %d rows need more places", M);
+    if ((rc = gemm_tc_plan(&p.moe_gate_up[i], m->moe_x, l.moe.gate_up.w, m->moe_places, l.moe.gate_up.N, l.moe.gate_up.K,
+                           kEpiSwiGLU, false, e->device, 0, &g))) return rc;
+    p.moe_gate_up[i].act = x.act;
+    if ((rc = gemm_tc_plan(&p.moe_down[i], m->moe_act, l.moe.down.w, m->moe_places, l.moe.down.N, l.moe.down.K, kEpiStore, false,
+                           e->device, 0, &g))) return rc;
   }
   if ((rc = ensure_gemm_workspace(e, ws))) return rc;
   *out = &m->plans.emplace(M, std::move(p)).first->second;
@@ -491,11 +690,36 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
     return gemm_simt(st, Y, X, w.w, rows, w.N, w.K, e->dtype, f32);
   };
   const LayeredPlans* pl = s.plans;
+  auto grouped = [&](const std::vector<TcGemmPlan>* plans, size_t i, void* Y, const void* X, const LayeredLinear& w,
+                     const TcGroups& g) -> int {
+    ++e->last_launches;
+    if (e->use_tc) return gemm_tc_run((*plans)[i], st, Y, (*plans)[i].N, e->d_gemm_ws, e->d_err, nullptr, m->moe_tiles);
+    return gemm_simt_grouped(st, Y, X, w.w, w.N, w.K, e->dtype, false, g, m->moe_tiles);
+  };
+  // the experts' outputs of every row, side by side in moe_y
+  auto experts = [&](size_t i, const ExpertsSpec& x, const LayeredExperts& w) -> int {
+    const TcGroups g = moe_groups(x, e->use_tc ? row_bucket((int)rows) : (int)rows, e->use_tc);
+    const MoeRouting r = moe_args(m, x, g);
+    prof_mark(e, kCatRouting);
+    if ((rc = moe_route_top(st, r, m->h, m->Hp, w.router, w.router_bias, rows, W, e->dtype))) return rc;
+    if ((rc = moe_gather(st, r, m->moe_x, m->h, m->Hp, rows, e->dtype))) return rc;
+    e->last_launches += 2;
+    prof_mark(e, kCatExpertsUp);
+    if (e->use_tc) {
+      if ((rc = grouped(&pl->moe_gate_up, i, m->moe_act, m->moe_x, w.gate_up, g))) return rc;
+    } else {
+      if ((rc = grouped(nullptr, i, m->moe_gu, m->moe_x, w.gate_up, g))) return rc;
+      if ((rc = gated_act(st, m->moe_act, m->moe_gu, (int64_t)g.max_tiles * g.m_pad, w.ffp, x.act, e->dtype))) return rc;
+      ++e->last_launches;
+    }
+    prof_mark(e, kCatExpertsDown);
+    return grouped(pl ? &pl->moe_down : nullptr, i, m->moe_y, m->moe_act, w.down, g);
+  };
   auto at = [&](void* p, int64_t elements) { return (void*)((uint8_t*)p + (size_t)elements * es); };
 
   prof_mark(e, kCatOther);
-  if ((rc = streams_embed(st, m->x, m->h, m->embed, m->pos, ids, pos, m->layers[0].sub1.in, m->layers[0].sub1.norm, rows, S, W,
-                          m->Hp, sp.vocab, sp.max_positions, sp.eps, e->dtype))) return rc;
+  if ((rc = streams_embed(st, m->x, m->h, m->embed, m->pos, ids, pos, m->layers[0].sub1.in, m->layers[0].sub1.norm, sp.norm_offset,
+                          rows, S, W, m->Hp, sp.vocab, sp.max_positions, sp.eps, e->dtype))) return rc;
   ++e->last_launches;
   for (size_t i = 0; i < m->layers.size(); ++i) {
     LayeredLayer& l = m->layers[i];
@@ -508,7 +732,10 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
     if (mx.has_attn) {
       const SpanAttention a = span_args(e, i, s);
       prof_mark(e, kCatRopeKv);
-      if ((rc = span_kv_write(st, a, at(m->proj, mx.ak.offset), at(m->proj, mx.av.offset), ldp, slots, rows, e->dtype))) return rc;
+      AttentionPrep prep;
+      if (prep_args(e, i, s, &prep)) rc = attention_prepare(st, prep, rows, e->dtype);
+      else rc = span_kv_write(st, a, at(m->proj, mx.ak.offset), at(m->proj, mx.av.offset), ldp, slots, rows, e->dtype);
+      if (rc) return rc;
       prof_mark(e, kCatAttention);
       if ((rc = issue_attention(e, a, s))) return rc;
       prof_mark(e, kCatGemmO);
@@ -536,36 +763,44 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
       ++e->last_launches;  // the gated norm
     }
     const bool both = mx.has_attn && mx.has_rec;
-    const SublayerMix* next = lsp.ff ? &l.sub2 : (i + 1 < m->layers.size() ? &m->layers[i + 1].sub1 : nullptr);
-    auto boundary = [&](const SublayerMix& q, bool two) -> int {
-      StreamMix sm;
+    const SublayerMix* next = lsp.has_ffn() ? &l.sub2 : (i + 1 < m->layers.size() ? &m->layers[i + 1].sub1 : nullptr);
+    auto boundary = [&](const SublayerMix& q, const float* y, bool two, StreamMix sm) -> int {
       sm.mix = q.mix; sm.out = q.out;
       sm.next_in = next ? next->in : nullptr;
       sm.next_norm = next ? next->norm : nullptr;
       sm.w1 = l.attn_out_norm; sm.w2 = l.rec_out_norm;
+      sm.norm_offset = sp.norm_offset;
       ++e->last_launches;
       prof_mark(e, kCatNorm);
-      return streams_mix(st, m->x, m->h, m->y1, two ? m->y2 : nullptr, m->Hp, sm, rows, S, W, m->Hp, sp.eps, e->dtype);
+      return streams_mix(st, m->x, m->h, y, two ? m->y2 : nullptr, m->Hp, sm, rows, S, W, m->Hp, sp.eps, e->dtype);
     };
-    if ((rc = boundary(l.sub1, both))) return rc;
-    if (lsp.ff) {
+    StreamMix mixed{};
+    mixed.bias = l.o_bias;
+    if ((rc = boundary(l.sub1, m->y1, both, mixed))) return rc;
+    if (!lsp.has_ffn()) continue;
+    next = i + 1 < m->layers.size() ? &m->layers[i + 1].sub1 : nullptr;
+    StreamMix fed{};
+    if (lsp.moe.experts) {
+      if ((rc = experts(i, lsp.moe, l.moe))) return rc;
+      fed.expert_y = m->moe_y; fed.expert_place = m->moe_place; fed.expert_weight = m->moe_weight; fed.top = lsp.moe.top;
+    }
+    if (lsp.ffn.ff) {
       prof_mark(e, kCatGemmGateUp);
       if (e->use_tc) {
         if ((rc = gemm(&pl->gate_up, i, m->act, m->h, l.gate_up, false))) return rc;
       } else {
         if ((rc = gemm(nullptr, i, m->gu, m->h, l.gate_up, false))) return rc;
-        if ((rc = hb_silu_mul(st, m->act, m->gu, rows, l.ffp, e->dtype))) return rc;
+        if ((rc = gated_act(st, m->act, m->gu, rows, l.ffp, lsp.ffn.act, e->dtype))) return rc;
         ++e->last_launches;
       }
       prof_mark(e, kCatGemmDown);
       if ((rc = gemm(pl ? &pl->down : nullptr, i, m->y1, m->act, l.down, true))) return rc;
-      next = i + 1 < m->layers.size() ? &m->layers[i + 1].sub1 : nullptr;
-      if ((rc = boundary(l.sub2, false))) return rc;
     }
+    if ((rc = boundary(l.sub2, lsp.ffn.ff ? m->y1 : nullptr, false, fed))) return rc;
   }
   if (s.want) {
     prof_mark(e, kCatNorm);
-    if ((rc = streams_final(st, m->hf, m->x, (const int32_t*)(in + s.off_want), m->final_norm, s.want, S, W, m->Hp, sp.eps,
+    if ((rc = streams_final(st, m->hf, m->x, (const int32_t*)(in + s.off_want), m->final_norm, sp.norm_offset, s.want, S, W, m->Hp, sp.eps,
                             e->dtype))) return rc;
     prof_mark(e, kCatGemmLmHead);
     if (e->use_tc) rc = gemm_tc_run(*s.head_plan, st, e->d_logits, sp.vocab, e->d_gemm_ws, e->d_err);
@@ -591,15 +826,20 @@ static double layered_step_bytes(const hb_engine* e, const int32_t* ctx_lens, in
     const MixerSpec& mx = s.layers[i].mixer;
     if (mx.has_attn) {
       const AttentionSpec& a = mx.attn;
+      const double per_key = a.values_are_keys ? a.kv_heads * a.dim * es + 4.0 : a.kv_heads * (a.dim + a.vdim) * es;
       for (int64_t k = 0; k < n_seqs; ++k) {
         const int64_t ctx = ctx_lens ? ctx_lens[k] : 0;
         int64_t seen = ctx;
-        if (a.window > 0) seen = std::min<int64_t>(ctx, (int64_t)a.window + std::min<int64_t>(a.keep_first, std::max<int64_t>(0, ctx - a.window)));
-        w += ((double)seen + 1.0) * a.kv_heads * (a.dim + a.vdim) * es;
+        if (a.chunk > 0) seen = ctx % a.chunk;
+        else if (a.window > 0) seen = std::min<int64_t>(ctx, (int64_t)a.window + std::min<int64_t>(a.keep_first, std::max<int64_t>(0, ctx - a.window)));
+        w += ((double)seen + 1.0) * per_key;
       }
     }
     if (mx.has_rec) w += n * 2.0 * mx.rec.heads * mx.rec.dim * mx.rec.vdim * 4.0;
-    w += n * (s.layers[i].ff ? 2.0 : 1.0) * 2.0 * s.streams * s.width * 4.0;
+    w += n * (s.layers[i].has_ffn() ? 2.0 : 1.0) * 2.0 * s.streams * s.width * 4.0;
+    if (const ExpertsSpec& x = s.layers[i].moe; x.experts)  // the experts a random batch chooses
+      w += x.experts * (1.0 - std::pow(1.0 - 1.0 / x.experts, n * x.top)) *
+               ((double)l.moe.gate_up.N * l.moe.gate_up.K + (double)l.moe.down.N * l.moe.down.K) * es + (double)x.experts * s.width * es;
   }
   return w;
 }
@@ -611,9 +851,17 @@ static double layered_gemm_bytes(const hb_engine* e, int64_t rows) {
     return q.w ? ((double)q.N * q.K + b * q.K) * es + b * n_out * out_es : 0.0;
   };
   double t = lin(m->head, (double)m->head.N, 4.0);
-  for (const LayeredLayer& l : m->layers)
+  for (size_t i = 0; i < m->layers.size(); ++i) {
+    const LayeredLayer& l = m->layers[i];
     t += lin(l.proj, (double)l.proj.N, es) + lin(l.attn_o, (double)l.attn_o.N, 4.0) + lin(l.rec_o, (double)l.rec_o.N, 4.0) +
          lin(l.gate_up, (double)l.ffp, es) + lin(l.down, (double)l.down.N, 4.0);
+    if (const ExpertsSpec& x = m->spec.layers[i].moe; x.experts) {
+      const double picks = b * x.top, active = x.experts * (1.0 - std::pow(1.0 - 1.0 / x.experts, picks));
+      const LayeredExperts& w = l.moe;
+      t += active * ((double)w.gate_up.N * w.gate_up.K + (double)w.down.N * w.down.K) * es +
+           picks * ((double)w.gate_up.K + 2.0 * w.ffp + (double)w.down.N) * es;
+    }
+  }
   return t;
 }
 

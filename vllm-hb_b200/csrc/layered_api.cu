@@ -1,4 +1,5 @@
 // Public entry points of the layered models' mechanisms.
+#include "gemm.h"
 #include "layered_ops.h"
 
 namespace hb {
@@ -10,15 +11,19 @@ static SpanAttention span_of(const hb_span_attention_args* p) {
   a.tables = p->block_tables; a.max_blocks = p->max_blocks; a.num_blocks = p->num_blocks;
   a.row_seg = p->row_segment; a.pos = p->positions;
   a.heads = p->heads; a.kv_heads = p->kv_heads; a.dim = p->dim; a.vdim = p->vdim;
-  a.window = p->window; a.keep_first = p->keep_first; a.scale = p->scale;
+  a.window = p->window; a.keep_first = p->keep_first; a.chunk = p->chunk; a.scale = p->scale;
+  a.key_scale = p->key_scale; a.dist_bias = p->dist_bias; a.dist_len = p->dist_len; a.sink = p->sink;
+  a.gate = p->gate; a.ld_gate = p->ld_gate;
   return a;
 }
 
 static int check_span(const hb_span_attention_args* p) {
-  HB_CHECK_ARG(p && p->k_cache && p->v_cache, "span attention: null argument");
+  HB_CHECK_ARG(p && p->k_cache && (p->v_cache || p->key_scale), "span attention: null argument");
   HB_CHECK_ARG(p->heads > 0 && p->kv_heads > 0 && p->heads % p->kv_heads == 0 && p->dim > 0 && p->vdim > 0,
                "span attention: bad sizes");
-  HB_CHECK_ARG(p->window >= 0 && p->keep_first >= 0 && p->num_blocks > 0, "span attention: bad window or pool");
+  HB_CHECK_ARG(p->window >= 0 && p->keep_first >= 0 && p->chunk >= 0 && p->num_blocks > 0, "span attention: bad window or pool");
+  HB_CHECK_ARG(!p->key_scale || p->dim == p->vdim, "span attention: keys that are the values have their width");
+  HB_CHECK_ARG(!p->dist_bias || p->dist_len > 0, "span attention: an empty bias table");
   return HB_OK;
 }
 
@@ -67,7 +72,7 @@ int hb_span_kv_write(void* stream, const hb_span_attention_args* p, const void* 
                      const int64_t* slots, int64_t rows, hb_dtype dtype) {
   int rc = hb::check_span(p);
   if (rc) return rc;
-  HB_CHECK_ARG(k && v && slots && rows >= 0, "hb_span_kv_write: null argument");
+  HB_CHECK_ARG(k && v && slots && rows >= 0 && p->v_cache, "hb_span_kv_write: null argument");
   return rows ? hb::span_kv_write((cudaStream_t)stream, hb::span_of(p), k, v, ld, slots, rows, dtype) : HB_OK;
 }
 
@@ -102,7 +107,7 @@ int hb_streams_embed(void* stream, float* x, void* h, const void* embed, const v
   HB_CHECK_ARG(x && h && embed && pos_table && ids && positions && in && norm, "hb_streams_embed: null argument");
   HB_CHECK_ARG(rows >= 0 && streams > 0 && width > 0 && vocab > 0 && max_positions > 0, "hb_streams_embed: bad shape");
   if (rows == 0) return HB_OK;
-  return hb::streams_embed((cudaStream_t)stream, x, h, embed, pos_table, ids, positions, in, norm, rows, streams, width, ld_h,
+  return hb::streams_embed((cudaStream_t)stream, x, h, embed, pos_table, ids, positions, in, norm, 1.f, rows, streams, width, ld_h,
                            vocab, max_positions, eps, dtype);
 }
 
@@ -117,10 +122,97 @@ int hb_streams_mix(void* stream, float* x, void* h, const float* y, const float*
   return hb::streams_mix((cudaStream_t)stream, x, h, y, y2, ld_y, m, rows, streams, width, ld_h, eps, dtype);
 }
 
+int hb_streams_mix_ex(void* stream, float* x, void* h, const float* y, const float* y2, int64_t ld_y,
+                      const hb_stream_mix_args* a, int64_t rows, int streams, int64_t width, int64_t ld_h, float eps,
+                      hb_dtype dtype) {
+  HB_CHECK_ARG(x && a && a->mix && a->out && (!a->next_norm || (a->next_in && h)), "hb_streams_mix_ex: null argument");
+  HB_CHECK_ARG(!y2 || (y && a->w1 && a->w2 && !a->bias && !a->top), "hb_streams_mix_ex: bad second branch");
+  HB_CHECK_ARG(rows >= 0 && width > 0 && a->top >= 0 && (!a->top || (a->expert_y && a->expert_place && a->expert_weight)),
+               "hb_streams_mix_ex: bad shape");
+  if (rows == 0) return HB_OK;
+  hb::StreamMix m;
+  m.mix = a->mix; m.out = a->out; m.next_in = a->next_in; m.next_norm = a->next_norm; m.w1 = a->w1; m.w2 = a->w2;
+  m.norm_offset = a->norm_offset; m.bias = a->bias;
+  m.expert_y = a->expert_y; m.expert_place = a->expert_place; m.expert_weight = a->expert_weight; m.top = a->top;
+  return hb::streams_mix((cudaStream_t)stream, x, h, y, y2, ld_y, m, rows, streams, width, ld_h, eps, dtype);
+}
+
+int hb_attention_prepare(void* stream, const hb_attention_prep_args* p, int64_t rows, hb_dtype dtype) {
+  HB_CHECK_ARG(p && p->p && p->positions && p->slots && p->k_cache && (p->v_cache || p->key_scale) && rows >= 0,
+               "hb_attention_prepare: null argument");
+  HB_CHECK_ARG(p->heads > 0 && p->kv_heads > 0 && p->heads % p->kv_heads == 0 && p->dim > 0 && p->vdim > 0 && p->num_blocks > 0 &&
+               p->pairs >= 0 && (p->pairs == 0 || p->rotation), "hb_attention_prepare: bad sizes");
+  hb::AttentionPrep a;
+  a.p = p->p; a.ld = p->ld;
+  a.off_q = p->off_q; a.off_k = p->off_k; a.off_v = p->off_v;
+  a.heads = p->heads; a.kv_heads = p->kv_heads; a.dim = p->dim; a.vdim = p->vdim;
+  a.pos = p->positions; a.slots = p->slots; a.kc = p->k_cache; a.vc = p->v_cache; a.num_blocks = p->num_blocks;
+  a.q_bias = p->q_bias; a.k_bias = p->k_bias; a.q_norm = p->q_norm; a.k_norm = p->k_norm; a.eps = p->eps;
+  a.rotation = p->rotation; a.pairs = p->pairs; a.key_scale = p->key_scale;
+  return hb::attention_prepare((cudaStream_t)stream, a, rows, dtype);
+}
+
+static hb::MoeRouting routing_of(const hb_moe_routing* p) {
+  hb::MoeRouting m;
+  m.experts = p->experts; m.top = p->top; m.m_pad = p->m_pad; m.max_tiles = p->max_tiles;
+  m.ids = p->ids; m.rank = p->rank; m.place = p->place; m.weight = p->weight;
+  m.count = p->count; m.first = p->first; m.tile_group = p->tile_group;
+  return m;
+}
+
+int hb_moe_route_top(void* stream, const hb_moe_routing* m, const void* h, int64_t ld_h, const void* router,
+                     const float* bias, int64_t rows, int64_t width, hb_dtype dtype) {
+  HB_CHECK_ARG(m && h && router && bias && m->ids && m->rank && m->weight && m->count && m->first && m->tile_group,
+               "hb_moe_route_top: null argument");
+  HB_CHECK_ARG(rows >= 0 && width > 0 && m->m_pad > 0 &&
+               m->max_tiles >= (rows * m->top < m->experts ? rows * m->top : m->experts) + rows * m->top / m->m_pad,
+               "hb_moe_route_top: bad shape");
+  return hb::moe_route_top((cudaStream_t)stream, routing_of(m), h, ld_h, router, bias, rows, width, dtype);
+}
+
+int hb_moe_gather(void* stream, const hb_moe_routing* m, void* x, const void* h, int64_t ld, int64_t rows, hb_dtype dtype) {
+  HB_CHECK_ARG(m && x && h && m->ids && m->rank && m->place && m->first && ld > 0 && rows >= 0, "hb_moe_gather: null argument");
+  return hb::moe_gather((cudaStream_t)stream, routing_of(m), x, h, ld, rows, dtype);
+}
+
+static hb::GatedAct act_of(const hb_gated_act_spec* p) {
+  hb::GatedAct a;
+  a.slope = p->slope; a.cubic = p->cubic; a.limit = p->limit; a.shift = p->shift;
+  return a;
+}
+
+int hb_gated_act(void* stream, void* out, const void* gate_up, int64_t M, int64_t inter, const hb_gated_act_spec* act,
+                 hb_dtype dtype) {
+  HB_CHECK_ARG(out && gate_up && act && M >= 0 && inter > 0, "hb_gated_act: bad argument");
+  return hb::gated_act((cudaStream_t)stream, out, gate_up, M, inter, act_of(act), dtype);
+}
+
+int hb_gemm_grouped(void* stream, void* Y, const void* X, const void* W, int groups, int64_t N, int64_t K, int m_pad,
+                    int max_tiles, int likely_tiles, const int32_t* tile_group, int out_f32,
+                    const hb_gated_act_spec* gated, hb_dtype dtype) {
+  HB_CHECK_ARG(Y && X && W && tile_group && groups > 0 && N > 0 && K > 0 && m_pad > 0 && max_tiles > 0 && likely_tiles > 0,
+               "hb_gemm_grouped: bad argument");
+  hb::TcGroups g;
+  g.groups = groups; g.m_pad = m_pad; g.max_tiles = max_tiles; g.likely_tiles = likely_tiles;
+  const int64_t M = (int64_t)max_tiles * m_pad;
+  auto st = (cudaStream_t)stream;
+  if (hb::gemm_tc_supported(M, N, K, dtype) && m_pad % 16 == 0) {
+    int dev = 0;
+    HB_CUDA_CHECK(cudaGetDevice(&dev));
+    hb::TcGemmPlan plan;
+    int rc = hb::gemm_tc_plan(&plan, X, W, M, N, K, gated ? hb::kEpiSwiGLU : hb::kEpiStore, out_f32 != 0, dev, 0, &g);
+    if (rc) return rc;
+    if (gated) plan.act = act_of(gated);
+    return hb::gemm_tc_run(plan, st, Y, plan.N, nullptr, nullptr, nullptr, tile_group);
+  }
+  HB_CHECK_ARG(!gated, "hb_gemm_grouped: the gated form runs on tensor cores (bf16, K %% 8 == 0)");
+  return hb::gemm_simt_grouped(st, Y, X, W, N, K, dtype, out_f32 != 0, g, tile_group);
+}
+
 int hb_streams_final(void* stream, void* h, const float* x, const int32_t* want, const float* norm, int64_t n_want,
                      int streams, int64_t width, int64_t ld_h, float eps, hb_dtype dtype) {
   HB_CHECK_ARG(h && x && want && norm && streams > 0 && width > 0, "hb_streams_final: bad argument");
-  return hb::streams_final((cudaStream_t)stream, h, x, want, norm, n_want, streams, width, ld_h, eps, dtype);
+  return hb::streams_final((cudaStream_t)stream, h, x, want, norm, 1.f, n_want, streams, width, ld_h, eps, dtype);
 }
 
 int hb_gated_group_norm(void* stream, void* out, int64_t ld_out, const float* o, int64_t ld_o, const void* gate,

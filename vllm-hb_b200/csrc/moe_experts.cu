@@ -1,0 +1,212 @@
+// Mixture of experts with a router bias and top-k routing, each expert run on its own rows only.
+//
+//   route   logits, the top experts of every row and their weights; every (row, expert) draws a rank
+//           among the expert's rows; the last CTA turns the counts into batch tiles
+//   gather  rows to the places of their experts (tiles of m_pad places that belong to one expert)
+//   (two grouped GEMMs, gemm_tc.cu / gemm_simt.cu; the weighted sum is part of streams_mix)
+//
+// The order of the rows inside an expert depends on timing; no result does, because rows do not
+// meet before the weighted sum, which runs in the order of the router.
+#include <algorithm>
+
+#include "gemm.h"
+#include "layered_ops.h"
+
+namespace hb {
+
+constexpr int kRouteThreads = 256;
+constexpr int kRouteWarps = kRouteThreads / 32;
+
+// RB rows per CTA share every router row they read.
+template <typename T, int RB>
+__global__ void __launch_bounds__(kRouteThreads)
+moe_route_top_kernel(const MoeRouting m, const T* __restrict__ h, int64_t ld_h, const T* __restrict__ router,
+                     const float* __restrict__ bias, int64_t rows, int64_t width) {
+  pdl_trigger();
+  extern __shared__ float s_logit[];  // [RB][experts]
+  __shared__ int s_last;
+  pdl_grid_wait();
+  constexpr int N = Vec16<T>::N;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, E = m.experts;
+  const int64_t row0 = (int64_t)blockIdx.x * RB;
+  const int nr = (int)min((int64_t)RB, rows - row0);
+  const bool vec = width % N == 0 && ld_h % N == 0;
+  for (int e = warp; e < E; e += kRouteWarps) {
+    const T* w = router + (int64_t)e * width;
+    float acc[RB];
+#pragma unroll
+    for (int r = 0; r < RB; ++r) acc[r] = 0.f;
+    if (vec) {
+#pragma unroll 4
+      for (int64_t v = lane; v < width / N; v += 32) {
+        Vec16<T> a, b;
+        b.load(w + v * N);
+        float fa[N], fb[N];
+        b.unpack(fb);
+#pragma unroll
+        for (int r = 0; r < RB; ++r) {
+          if (r < nr) {
+            a.load(h + (row0 + r) * ld_h + v * N);
+            a.unpack(fa);
+#pragma unroll
+            for (int j = 0; j < N; ++j) acc[r] = fmaf(fa[j], fb[j], acc[r]);
+          }
+        }
+      }
+    } else {
+      for (int64_t i = lane; i < width; i += 32) {
+        const float b = to_f32<T>(w[i]);
+#pragma unroll
+        for (int r = 0; r < RB; ++r)
+          if (r < nr) acc[r] = fmaf(to_f32<T>(h[(row0 + r) * ld_h + i]), b, acc[r]);
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < RB; ++r) {
+      const float s = warp_sum(acc[r]);
+      if (lane == 0) s_logit[r * E + e] = s + bias[e];
+    }
+  }
+  __syncthreads();
+  // one warp per row: the largest logit `top` times, the lower expert among equals
+  for (int r = warp; r < nr; r += kRouteWarps) {
+    float* z = s_logit + r * E;
+    const int64_t at = (row0 + r) * m.top;
+    float first = 0.f, sum = 0.f;
+    for (int k = 0; k < m.top; ++k) {
+      float best = -INFINITY;
+      int who = E;
+      for (int e = lane; e < E; e += 32)
+        if (z[e] > best || who == E) {
+          if (!isnan(z[e])) { best = z[e]; who = e; }
+        }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float b = __shfl_xor_sync(0xffffffffu, best, o);
+        const int w = __shfl_xor_sync(0xffffffffu, who, o);
+        if (w < E && (who == E || b > best || (b == best && w < who))) { best = b; who = w; }
+      }
+      const int e = min(who, E - 1);  // a row of NaNs still names an expert
+      if (k == 0) first = best;
+      const float p = expf(best - first);
+      sum += p;
+      if (lane == 0) {
+        z[e] = __int_as_float(0x7fc00000);  // taken
+        m.ids[at + k] = e;
+        m.weight[at + k] = p;
+        m.rank[at + k] = atomicAdd(m.count + e, 1);
+      }
+      __syncwarp();
+    }
+    for (int k = lane; k < m.top; k += 32) m.weight[at + k] /= sum;
+  }
+  // the last CTA: every expert's tiles
+  __threadfence();
+  __syncthreads();
+  if (threadIdx.x == 0) s_last = atomicAdd(m.count + E, 1) == (int)gridDim.x - 1;
+  __syncthreads();
+  if (!s_last || warp != 0) return;
+  __threadfence();
+  int tile = 0;  // tiles of the experts before this group of 32
+  for (int e0 = 0; e0 < E; e0 += 32) {
+    const int e = e0 + lane;
+    const int n = e < E ? (__ldcg(m.count + e) + m.m_pad - 1) / m.m_pad : 0;
+    int incl = n;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, incl, o);
+      if (lane >= o) incl += v;
+    }
+    const int at = tile + incl - n;
+    if (e < E) {
+      m.first[e] = at * m.m_pad;
+      m.count[e] = 0;
+      for (int i = 0; i < n && at + i < m.max_tiles; ++i) m.tile_group[at + i] = e;
+    }
+    tile += __shfl_sync(0xffffffffu, incl, 31);
+  }
+  for (int i = tile + lane; i < m.max_tiles; i += 32) m.tile_group[i] = -1;
+  if (lane == 0) m.count[E] = 0;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kRouteThreads)
+moe_gather_kernel(const MoeRouting m, T* __restrict__ x, const T* __restrict__ h, int64_t ld) {
+  pdl_trigger();
+  extern __shared__ int32_t s_place[];  // [top]
+  pdl_grid_wait();
+  constexpr int N = Vec16<T>::N;
+  const int64_t row = blockIdx.x, places = (int64_t)m.max_tiles * m.m_pad;
+  for (int k = threadIdx.x; k < m.top; k += kRouteThreads) {
+    const int64_t at = row * m.top + k;
+    const int p = m.first[m.ids[at]] + m.rank[at];
+    s_place[k] = p < places ? p : 0;  // never outside the buffer
+    m.place[at] = s_place[k];
+  }
+  __syncthreads();
+  for (int64_t v = threadIdx.x; v < ld / N; v += kRouteThreads) {
+    Vec16<T> a;
+    a.load(h + row * ld + v * N);
+    for (int k = 0; k < m.top; ++k) a.store(x + (int64_t)s_place[k] * ld + v * N);
+  }
+}
+
+int moe_route_top(cudaStream_t st, const MoeRouting& m, const void* h, int64_t ld_h, const void* router, const float* bias,
+                  int64_t rows, int64_t width, hb_dtype dtype) {
+  if (rows == 0) return HB_OK;
+  if (m.experts < 1 || m.experts > kMoeMaxExperts || m.top < 1 || m.top > m.experts || m.m_pad < 1)
+    return fail(HB_ERR_INVALID_ARG, "moe_route_top: %d of %d experts (at most %d)", m.top, m.experts, kMoeMaxExperts);
+  auto launch = [&](auto* k, int rb, auto* t) -> int {
+    using T = std::remove_pointer_t<decltype(t)>;
+    HB_CUDA_CHECK(launch_pdl(k, dim3((unsigned)((rows + rb - 1) / rb)), dim3(kRouteThreads),
+                             (size_t)rb * m.experts * sizeof(float), st, m, (const T*)h, ld_h, (const T*)router, bias, rows, width));
+    return HB_OK;
+  };
+  const bool few = rows <= 512;
+  if (dtype == HB_F32)
+    return few ? launch(moe_route_top_kernel<float, 1>, 1, (float*)nullptr) : launch(moe_route_top_kernel<float, 8>, 8, (float*)nullptr);
+  if (dtype == HB_BF16)
+    return few ? launch(moe_route_top_kernel<__nv_bfloat16, 1>, 1, (__nv_bfloat16*)nullptr)
+               : launch(moe_route_top_kernel<__nv_bfloat16, 8>, 8, (__nv_bfloat16*)nullptr);
+  return fail(HB_ERR_UNSUPPORTED_DTYPE, "moe_route_top runs in bf16 or f32");
+}
+
+int moe_gather(cudaStream_t st, const MoeRouting& m, void* x, const void* h, int64_t ld, int64_t rows, hb_dtype dtype) {
+  if (rows == 0) return HB_OK;
+  const int n = (int)(16 / dtype_size(dtype));
+  if (ld % n || (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(h) & 15))
+    return fail(HB_ERR_INVALID_ARG, "moe_gather: rows must be multiples of 16 bytes");
+  const size_t smem = (size_t)m.top * sizeof(int32_t);
+  if (dtype == HB_F32)
+    HB_CUDA_CHECK(launch_pdl(moe_gather_kernel<float>, dim3((unsigned)rows), dim3(kRouteThreads), smem, st, m, (float*)x,
+                             (const float*)h, ld));
+  else if (dtype == HB_BF16)
+    HB_CUDA_CHECK(launch_pdl(moe_gather_kernel<__nv_bfloat16>, dim3((unsigned)rows), dim3(kRouteThreads), smem, st, m,
+                             (__nv_bfloat16*)x, (const __nv_bfloat16*)h, ld));
+  else
+    return fail(HB_ERR_UNSUPPORTED_DTYPE, "moe_gather runs in bf16 or f32");
+  return HB_OK;
+}
+
+// ------------------------------------------------------------------- gated activation
+template <typename T>
+__global__ void gated_act_kernel(T* __restrict__ out, const T* __restrict__ gu, int64_t inter, GatedAct act) {
+  pdl_trigger();
+  pdl_grid_wait();
+  const int64_t row = blockIdx.x;
+  for (int64_t i = threadIdx.x; i < inter; i += blockDim.x) {
+    const float g = fminf(to_f32<T>(gu[row * 2 * inter + i]), act.limit);
+    const float u = fminf(fmaxf(to_f32<T>(gu[row * 2 * inter + inter + i]), -act.limit), act.limit);
+    out[row * inter + i] = from_f32<T>(g / (1.f + expf(-act.slope * (g + act.cubic * g * g * g))) * (u + act.shift));
+  }
+}
+
+int gated_act(cudaStream_t st, void* out, const void* gate_up, int64_t M, int64_t inter, const GatedAct& act, hb_dtype dtype) {
+  if (M == 0) return HB_OK;
+  HB_DISPATCH_DTYPE(dtype, T, {
+    HB_CUDA_CHECK(launch_pdl(gated_act_kernel<T>, dim3((unsigned)M), dim3(256), 0, st, (T*)out, (const T*)gate_up, inter, act));
+  });
+  return HB_OK;
+}
+
+}  // namespace hb

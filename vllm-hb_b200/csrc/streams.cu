@@ -48,8 +48,8 @@ template <typename T, int VEC>
 __global__ void __launch_bounds__(kStreamThreads)
 streams_embed_kernel(float* __restrict__ x, T* __restrict__ h, const T* __restrict__ embed, const T* __restrict__ pos_table,
                      const uint32_t* __restrict__ ids, const int32_t* __restrict__ pos, const float* __restrict__ in,
-                     const float* __restrict__ norm, int S, int64_t W, int64_t ld_h, int64_t vocab, int64_t max_positions,
-                     float eps) {
+                     const float* __restrict__ norm, float norm_offset, int S, int64_t W, int64_t ld_h, int64_t vocab,
+                     int64_t max_positions, float eps) {
   pdl_trigger();
   pdl_grid_wait();
   __shared__ float red[33];
@@ -57,7 +57,7 @@ streams_embed_kernel(float* __restrict__ x, T* __restrict__ h, const T* __restri
   const int64_t id = min((int64_t)ids[row], vocab - 1);                       // never outside the tables
   const int64_t p = max((int64_t)0, min((int64_t)pos[row], max_positions - 1));
   const T* er = embed + id * W;
-  const T* pr = pos_table + p * W;
+  const T* pr = pos_table ? pos_table + p * W : nullptr;
   float* xr = x + row * S * W;
   float in_sum = 0.f;
   for (int s = 0; s < S; ++s) in_sum += in[s];
@@ -65,10 +65,10 @@ streams_embed_kernel(float* __restrict__ x, T* __restrict__ h, const T* __restri
   for (int64_t i = (int64_t)threadIdx.x * VEC; i < W; i += kStreamThreads * VEC) {
     float a[VEC], b[VEC];
     load_vec<T, VEC>(a, er + i);
-    load_vec<T, VEC>(b, pr + i);
+    if (pr) load_vec<T, VEC>(b, pr + i);
 #pragma unroll
     for (int j = 0; j < VEC; ++j) {
-      a[j] += b[j];
+      if (pr) a[j] += b[j];
       const float u = in_sum * a[j];
       ss = fmaf(u, u, ss);
     }
@@ -80,7 +80,7 @@ streams_embed_kernel(float* __restrict__ x, T* __restrict__ h, const T* __restri
     load_vec<float, VEC>(a, xr + i);  // written by this thread
     load_vec<float, VEC>(w, norm + i);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) a[j] = in_sum * a[j] * r * (1.f + w[j]);
+    for (int j = 0; j < VEC; ++j) a[j] = in_sum * a[j] * r * (norm_offset + w[j]);
     store_vec<T, VEC>(h + row * ld_h + i, a);
   }
 }
@@ -105,7 +105,7 @@ streams_mix_kernel(float* __restrict__ x, T* __restrict__ h, const float* __rest
   }
   pdl_grid_wait();
   const int64_t row = blockIdx.x;
-  const float* yr = y + row * ld_y;
+  const float* yr = y ? y + row * ld_y : nullptr;
   const float* y2r = TWO ? y2 + row * ld_y : nullptr;
   float r1 = 0.f, r2 = 0.f;
   if (TWO) {
@@ -137,7 +137,30 @@ streams_mix_kernel(float* __restrict__ x, T* __restrict__ h, const float* __rest
         for (int j = 0; j < VEC; ++j) xs[s][j] = 0.f;
       }
     }
-    load_vec<float, VEC>(f, yr + i);
+    if (TWO || yr) {
+      load_vec<float, VEC>(f, yr + i);
+    } else {
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) f[j] = 0.f;
+    }
+    if (!TWO && m.bias) {
+      float b[VEC];
+      load_vec<float, VEC>(b, m.bias + i);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) f[j] += b[j];
+    }
+    if (!TWO && m.top) {
+      const int32_t* place = m.expert_place + row * m.top;
+      const float* weight = m.expert_weight + row * m.top;
+#pragma unroll 4
+      for (int k = 0; k < m.top; ++k) {
+        float e[VEC];
+        load_vec<T, VEC>(e, (const T*)m.expert_y + (int64_t)place[k] * ld_y + i);
+        const float w = weight[k];
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) f[j] = fmaf(w, e[j], f[j]);
+      }
+    }
     if (TWO) {
       float g[VEC], w1[VEC], w2[VEC];
       load_vec<float, VEC>(g, y2r + i);
@@ -175,7 +198,7 @@ streams_mix_kernel(float* __restrict__ x, T* __restrict__ h, const float* __rest
     load_vec<float, VEC>(u, s_u + i);  // written by this thread
     load_vec<float, VEC>(w, m.next_norm + i);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) u[j] = u[j] * r * (1.f + w[j]);
+    for (int j = 0; j < VEC; ++j) u[j] = u[j] * r * (m.norm_offset + w[j]);
     store_vec<T, VEC>(h + row * ld_h + i, u);
   }
 }
@@ -183,7 +206,7 @@ streams_mix_kernel(float* __restrict__ x, T* __restrict__ h, const float* __rest
 template <typename T, int VEC>
 __global__ void __launch_bounds__(kStreamThreads)
 streams_final_kernel(T* __restrict__ h, const float* __restrict__ x, const int32_t* __restrict__ want,
-                     const float* __restrict__ norm, int S, int64_t W, int64_t ld_h, float eps) {
+                     const float* __restrict__ norm, float norm_offset, int S, int64_t W, int64_t ld_h, float eps) {
   pdl_trigger();
   pdl_grid_wait();
   extern __shared__ float s_u[];
@@ -209,7 +232,7 @@ streams_final_kernel(T* __restrict__ h, const float* __restrict__ x, const int32
     load_vec<float, VEC>(u, s_u + i);
     load_vec<float, VEC>(w, norm + i);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) u[j] = u[j] * r * (1.f + w[j]);
+    for (int j = 0; j < VEC; ++j) u[j] = u[j] * r * (norm_offset + w[j]);
     store_vec<T, VEC>(h + (int64_t)blockIdx.x * ld_h + i, u);
   }
 }
@@ -267,12 +290,12 @@ gated_group_norm_kernel(T* __restrict__ out, int64_t ld_out, const float* __rest
   }
 
 int streams_embed(cudaStream_t st, float* x, void* h, const void* embed, const void* pos_table, const uint32_t* ids,
-                  const int32_t* pos, const float* in, const float* norm, int64_t rows, int streams, int64_t width,
-                  int64_t ld_h, int64_t vocab, int64_t max_positions, float eps, hb_dtype dtype) {
+                  const int32_t* pos, const float* in, const float* norm, float norm_offset, int64_t rows, int streams,
+                  int64_t width, int64_t ld_h, int64_t vocab, int64_t max_positions, float eps, hb_dtype dtype) {
   HB_DISPATCH_LAYERED(dtype, T, {
     auto* k = width % 4 == 0 ? streams_embed_kernel<T, 4> : streams_embed_kernel<T, 1>;
     HB_CUDA_CHECK(launch_pdl(k, dim3((unsigned)rows), dim3(kStreamThreads), 0, st, x, (T*)h, (const T*)embed,
-                             (const T*)pos_table, ids, pos, in, norm, streams, width, ld_h, vocab, max_positions, eps));
+                             (const T*)pos_table, ids, pos, in, norm, norm_offset, streams, width, ld_h, vocab, max_positions, eps));
   });
   return HB_OK;
 }
@@ -318,15 +341,15 @@ int streams_mix(cudaStream_t st, float* x, void* h, const float* y, const float*
   return HB_OK;
 }
 
-int streams_final(cudaStream_t st, void* h, const float* x, const int32_t* want, const float* norm, int64_t n_want,
-                  int streams, int64_t width, int64_t ld_h, float eps, hb_dtype dtype) {
+int streams_final(cudaStream_t st, void* h, const float* x, const int32_t* want, const float* norm, float norm_offset,
+                  int64_t n_want, int streams, int64_t width, int64_t ld_h, float eps, hb_dtype dtype) {
   if (n_want == 0) return HB_OK;
   HB_DISPATCH_LAYERED(dtype, T, {
     auto* k = width % 4 == 0 ? streams_final_kernel<T, 4> : streams_final_kernel<T, 1>;
     const int rc = row_smem(k, width);
     if (rc) return rc;
     HB_CUDA_CHECK(launch_pdl(k, dim3((unsigned)n_want), dim3(kStreamThreads), (size_t)width * 4, st, (T*)h, x, want, norm,
-                             streams, width, ld_h, eps));
+                             norm_offset, streams, width, ld_h, eps));
   });
   return HB_OK;
 }
