@@ -142,6 +142,15 @@ def route(h, w_router, bias, top):
     return chosen, e / e.sum(axis=1, keepdims=True)
 
 
+def route_margin(h, w_router, bias, top):
+    """How far the last chosen logit of every token lies above the first one left out, in units of
+    the spread of the logits (infinite when nothing is left out)."""
+    z = np.sort(h @ w_router.T + bias, axis=1)[:, ::-1]
+    if z.shape[1] == top:
+        return np.full(len(z), np.inf)
+    return (z[:, top - 1] - z[:, top]) / np.maximum(z.std(axis=1), 1e-9)
+
+
 def moe_ffn(h, w, mlp):
     chosen, weight = route(h, w["router"], w["router.b"], mlp["router"]["top"])
     y = np.zeros_like(h)
@@ -154,7 +163,7 @@ def moe_ffn(h, w, mlp):
 
 
 # ------------------------------------------------------------------------------ the model
-def forward(config: dict, weights: dict, tokens, layers_out: list | None = None):
+def forward(config: dict, weights: dict, tokens, layers_out: list | None = None, margins_out: list | None = None):
     """Logits [n, vocab] of one sequence from its first token."""
     eps = config["norm"]["eps"]
     x = weights["embed"][np.asarray(tokens, dtype=np.int64)]
@@ -167,6 +176,8 @@ def forward(config: dict, weights: dict, tokens, layers_out: list | None = None)
         mlp = layer.get("mlp")
         if mlp:
             h = rms_norm(x, w["norm2"], eps)
+            if margins_out is not None and mlp["kind"] == "moe":
+                margins_out.append(route_margin(h, w["mlp.router"], w["mlp.router.b"], mlp["router"]["top"]))
             x = x + (dense_ffn(h, sub(w, "mlp.")) if mlp["kind"] == "dense" else moe_ffn(h, sub(w, "mlp."), mlp))
         if layers_out is not None:
             layers_out.append(x.copy())
@@ -208,6 +219,23 @@ def tensor_shapes(config: dict, buckets: int = 12) -> dict:
     out["final.norm"] = (W,)
     out["head"] = (V, W)
     return out
+
+
+def steady_routers(config: dict, weights: dict, channels: int = 6) -> dict:
+    """The same model with routers that read only the last `channels` of the width, which the
+    embedding sets and no layer writes to: rounding inside the layers then hardly moves a logit, and a
+    16-bit run chooses the experts an exact one does (close calls apart)."""
+    w = {k: v.copy() for k, v in weights.items()}
+    rng = np.random.default_rng(7)
+    w["embed"][:, -channels:] = rng.choice([-3.0, -2.0, -1.0, 1.0, 2.0, 3.0], w["embed"][:, -channels:].shape)
+    for name, a in w.items():
+        leaf = name.rsplit(".", 1)[-1]
+        if name.endswith(".router"):
+            a[:, :-channels] = 0.0
+            a[:, -channels:] = round_bf16((a[:, -channels:] * (a.shape[1] / channels) ** 0.5).astype(np.float32))
+        elif leaf in ("o", "down") or name.endswith(".o.b"):
+            a[-channels:] = 0.0
+    return w
 
 
 def random_weights(config: dict, seed: int = 0, buckets: int = 12) -> dict:
