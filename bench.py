@@ -562,8 +562,8 @@ def run_gpu_arm(args, rank: int, world: int, local_rank: int) -> None:
 
 
 # --------------------------------------------------------------------- layered models
-def run_latarax(args) -> None:
-    """Prefill and decode of the Latarax design beside the Llama family at equal size (one GPU)."""
+def run_layered(args) -> None:
+    """Prefill and decode of a layered design beside the Llama family at equal size (one GPU)."""
     import torch
 
     import __graft_entry__ as entry
@@ -581,14 +581,14 @@ def run_latarax(args) -> None:
     sampler = ClockSampler(0)
     sampler.start()
     sampler.begin_region()
-    report = bench_layered.run(hb, peak, tflops, args.steps, args.warmup, args.size)
+    report = bench_layered.run(hb, peak, tflops, args.steps, args.warmup, args.workload, args.size)
     clocks = sampler.stop()
     launches = report.pop("gpu_launches")
-    first = report[next(reversed(report))]["latarax"]["decode batch 64"]
+    first = report[next(reversed(report))][args.workload]["decode batch 64"]
     print(json.dumps({"metric": METRIC, "value": first["tok_s"], "unit": UNIT, "n_gpus": 1, "steps": args.steps,
                       "warmup": args.warmup, "ms_per_step": first["ms"], "higher_is_better": True, "scaling": "weak",
                       "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
-                      "config": {"workload": "latarax and llama family at equal size, decode batch 64 of the last size",
+                      "config": {"workload": f"{args.workload} and llama family at equal size, decode batch 64 of the last size",
                                  "parallelism": "tp1", "l2": "inputs larger than L2 (weights read once per step)",
                                  "peaks": f"of {kind}"},
                       "gpu_launches": int(launches), "clocks": clocks, "sizes": report}), flush=True)
@@ -612,10 +612,10 @@ def main() -> None:
     ap.add_argument("--skip-checks", action="store_true",
                     help="N > 1: skip the untimed parity checks, the single-GPU base point and the row-parallel points")
     ap.add_argument("--tp1-layers", type=int, default=8, help="layers of the single-GPU base point of the N > 1 shape")
-    ap.add_argument("--workload", default="auto", choices=["auto", "mixtral", "latarax"],
+    ap.add_argument("--workload", default="auto", choices=["auto", "mixtral", "latarax", "biberax"],
                     help="auto: Llama-3.1-8B shape on one GPU, 70B shape on several; mixtral: Mixtral-8x7B shape; "
-                         "latarax: that design beside the Llama family at equal size, one GPU")
-    ap.add_argument("--size", default="", help="latarax: only the sizes whose name contains this text")
+                         "latarax, biberax: that design beside the Llama family at equal size, one GPU")
+    ap.add_argument("--size", default="", help="latarax, biberax: only the sizes whose name contains this text")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
@@ -628,8 +628,8 @@ def main() -> None:
         if args.gpus != 1 or world != 1:
             raise SystemExit(f"--gpus {args.gpus} needs torchrun with {args.gpus} ranks (WORLD_SIZE={world})")
     args.warmup = max(args.warmup, 3)
-    if args.workload == "latarax":
-        run_latarax(args)
+    if args.workload in ("latarax", "biberax"):
+        run_layered(args)
         return
     run_gpu_arm(args, rank, world, local_rank)
 

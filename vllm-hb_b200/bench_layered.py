@@ -1,9 +1,10 @@
-"""Latarax beside the Llama family at equal width, feed-forward, depth and vocabulary.
+"""Models described layer by layer beside the Llama family (and, for a mixture of experts, its
+Mixtral form) at equal width, feed-forward, depth and vocabulary.
 
-`python bench.py --workload latarax` runs it on one GPU: prefill of one long prompt and of several
-shorter ones, decode at several batch sizes, random weights.  For every kind of kernel it reports
-the time of a profiled step and the fraction of the roofline (the larger of bytes / measured HBM
-bandwidth and FLOPs / measured bf16 throughput, over the time).
+`python bench.py --workload latarax` or `biberax` runs it on one GPU: prefill of one long prompt and
+of several shorter ones, decode at several batch sizes, random weights and tokens.  For every kind of
+kernel it reports the time of a profiled step and the fraction of the roofline (the larger of bytes /
+measured HBM bandwidth and FLOPs / measured bf16 throughput, over the time).
 """
 from __future__ import annotations
 
@@ -25,8 +26,32 @@ def parallel(heads, kv, dim, window, keep, rec_heads, ff):
             "mlp": {"kind": "dense", "ff": ff}}
 
 
-def sizes() -> list[dict]:
-    """Layers of about 1.3B- and 8B-parameter models; half of them gla, half parallel."""
+def biberax_layers(heads, chunk, far, dense_ff, experts, top, ff, shared, layers):
+    """Chunked and distance-biased attention in turn; a dense feed-forward first, experts after it."""
+    sizes = dict(heads=heads, kv_heads=heads // 4, dim=128, vdim=128, scale=128 ** -0.5)
+    rot = dict(base=500000.0, dims=128, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192))
+    mixers = [("attention", dict(sizes, mask=dict(size=chunk), rot=rot)), ("attention_2", dict(sizes, bias_max=far))]
+    moe = {"kind": "moe", "expert": dict(ff=ff, limit=7.0), "router": dict(experts=experts, top=top),
+           "shared": dict(ff=shared, limit=7.0)}
+    return [{"type": mixers[i % 2][0], "mixer": mixers[i % 2][1], "mlp": {"kind": "dense", "ff": dense_ff} if i == 0 else moe}
+            for i in range(layers)]
+
+
+def sizes(design: str) -> list[dict]:
+    """Layers of about 1.3B- and 8B-parameter models (dense ones; a mixture has more)."""
+    if design == "biberax":
+        out = []
+        for width, dense_ff, experts, top, ff, shared, layers in ((2048, 5632, 16, 4, 1408, 1408, 12),
+                                                                  (4096, 14336, 8, 2, 7168, 7168, 8)):
+            heads = width // 128
+            llama = dict(hidden_size=width, intermediate_size=dense_ff, num_hidden_layers=layers, num_attention_heads=heads,
+                         num_key_value_heads=heads // 4, vocab_size=VOCAB, rms_norm_eps=1e-6, rope_theta=500000.0)
+            out.append({"name": f"width {width}, {top} of {experts} experts of {ff}, {layers} layers",
+                        "biberax": {"architecture": "Biberax", "width": width, "vocab": VOCAB, "norm": {"eps": 1e-6},
+                                    "layers": biberax_layers(heads, 1024, 1024, dense_ff, experts, top, ff, shared, layers)},
+                        "llama": llama,
+                        "mixtral": dict(llama, intermediate_size=ff, num_local_experts=experts, num_experts_per_tok=top)})
+        return out
     out = []
     for width, ff, layers in ((2048, 5632, 12), (4096, 14336, 8)):
         heads = width // 128
@@ -58,22 +83,60 @@ def work(shape: dict, family: str, positions: list[np.ndarray], wanted: int) -> 
     def gemm(kind, n, k, m=rows, n_out=None, out=2):
         add(kind, 2.0 * n * k + 2.0 * m * k + out * m * (n_out or n), 2.0 * m * n * k)
 
-    def attention(heads, kv, dim, vdim, window, keep):
+    def attention(heads, kv, dim, vdim, window, keep, chunk=0, tied=False, gated=False):
+        if chunk:
+            seen = sum(float(np.sum(p % chunk + 1)) for p in positions)
+            span = sum(float(p[-1] - p[0] // chunk * chunk + 1) for p in positions)
+            add("attention", 2.0 * kv * (dim + vdim) * span + 2.0 * rows * heads * (dim + vdim * (2 if gated else 1)),
+                2.0 * heads * (dim + vdim) * seen)
+            return
+        if tied:  # one read serves as keys and values
+            seen, span = sum(keys_seen(p, 0, 0) for p in positions), sum(float(p[-1] + 1) for p in positions)
+            add("attention", (2.0 * kv * dim + 4.0) * span + 2.0 * rows * heads * (dim + vdim * (2 if gated else 1)),
+                2.0 * heads * (dim + vdim) * seen)
+            return
         seen = sum(keys_seen(p, window, keep) for p in positions)
         # every key a segment reads is counted once per segment (decode: once per row)
         span = sum((min(p[-1] + 1, len(p) - 1 + window + min(keep, max(0, p[0] - window + 1))) if window else p[-1] + 1)
                    for p in positions)
         add("attention", 2.0 * kv * (dim + vdim) * span + 2.0 * rows * heads * (dim + vdim), 2.0 * heads * (dim + vdim) * seen)
 
-    if family == "llama":
+    if family in ("llama", "mixtral"):
         H, I, hq, kv = (shape[k] for k in ("hidden_size", "intermediate_size", "num_attention_heads", "num_key_value_heads"))
         for _ in range(shape["num_hidden_layers"]):
             gemm("gemm_qkv", (hq + 2 * kv) * 128, H)
             attention(hq, kv, 128, 128, 0, 0)
             gemm("gemm_o_proj", H, hq * 128)
-            gemm("gemm_gate_up", 2 * I, H, n_out=I)
-            gemm("gemm_down", H, I)
+            E = shape.get("num_local_experts", 1)  # every expert runs on every token
+            gemm("gemm_gate_up", 2 * E * I, H, n_out=E * I)
+            gemm("gemm_down", H, E * I)
         gemm("gemm_lm_head", shape["vocab_size"], H, m=rows, out=4)  # this family computes every row's logits
+        return w
+    if family == "biberax":
+        H = shape["width"]
+        for layer in shape["layers"]:
+            m, f = layer["mixer"], layer["mlp"]
+            tied = layer["type"] == "attention_2"
+            q, k, v = m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["heads"] * m["vdim"]
+            kv = k if tied else k + m["kv_heads"] * m["vdim"]
+            gemm("gemm_qkv", q + kv + v, H)
+            add("rope_kv", 4.0 * rows * (q + kv))
+            attention(m["heads"], m["kv_heads"], m["dim"], m["vdim"], 0, 0, m.get("mask", {}).get("size", 0), tied, True)
+            gemm("gemm_o_proj", H, v, out=4)
+            add("norm", 2 * rows * H * 14.0)
+            I = f["ff"] if f["kind"] == "dense" else f["shared"]["ff"]
+            gemm("gemm_gate_up", 2 * I, H, n_out=I)
+            gemm("gemm_down", H, I, out=4)
+            if f["kind"] == "moe":
+                E, top, F = f["router"]["experts"], f["router"]["top"], f["expert"]["ff"]
+                picks = rows * top
+                active = E * (1.0 - (1.0 - top / E) ** rows)
+                add("routing", 2.0 * E * H + 2.0 * rows * H * (1 + top))
+                add("experts_gate_up", 4.0 * active * F * H + 2.0 * picks * (H + F), 4.0 * picks * F * H)
+                add("experts_down", 2.0 * active * F * H + 2.0 * picks * (H + F), 2.0 * picks * F * H)
+                add("norm", 2.0 * picks * H)
+        add("norm", wanted * H * 6.0)
+        gemm("gemm_lm_head", shape["vocab"], H, m=wanted, out=4)
         return w
     H, S = shape["width"], shape["streams"]
     for layer in shape["layers"]:
@@ -155,13 +218,14 @@ def decode(eng, batch: int, ctx: int, steps: int, warmup: int, rows: int):
         for at in range(0, ctx, rows):
             eng.step([(s, p[at:at + rows], [])], logits=False)
     nxt = np.zeros(batch, dtype=np.uint32)
+    draw = lambda: rng.integers(0, VOCAB, batch).astype(np.uint32)  # what greedy random weights repeat is no workload
     for _ in range(warmup):
-        eng.decode_batch(seqs, nxt.copy(), next_tokens=nxt)
+        eng.decode_batch(seqs, draw(), next_tokens=nxt)
     ms = 0.0
     for _ in range(steps):
-        eng.decode_batch(seqs, nxt.copy(), next_tokens=nxt)
+        eng.decode_batch(seqs, draw(), next_tokens=nxt)
         ms += eng.last_step_ms()
-    _, prof = eng.profile_step(seqs, nxt.copy())
+    _, prof = eng.profile_step(seqs, draw())
     launches = eng.last_step_launches()
     prof.pop("gemm", None)
     for s in seqs:
@@ -169,18 +233,21 @@ def decode(eng, batch: int, ctx: int, steps: int, warmup: int, rows: int):
     return ms / steps, prof, launches
 
 
-def run(hb, hbm_gbs: float, tflops: float, steps: int, warmup: int, only: str = "") -> dict:
+def run(hb, hbm_gbs: float, tflops: float, steps: int, warmup: int, design: str = "latarax", only: str = "",
+        batches=(1, 16, 64, 128)) -> dict:
     rows, ctx = 2048, 1536
     report = {}
     launches = 0
-    for size in sizes():
+    for size in sizes(design):
         if only and only not in size["name"]:
             continue
         entry = report[size["name"]] = {}
-        for family in ("latarax", "llama"):
-            shape = size[family]
+        for family in (design, "llama", "mixtral"):
+            shape = size.get(family)
+            if not shape:
+                continue
             kw = dict(max_seq_len=4224, max_batch=rows, max_seqs=128, num_kv_blocks=128 * 128)
-            eng = hb.Engine.create_random_config(shape, **kw) if family == "latarax" else \
+            eng = hb.Engine.create_random_config(shape, **kw) if family == design else \
                 hb.Engine.create_random(shape, **{k: v for k, v in kw.items() if k != "max_seqs"})
             res = entry[family] = {"parameters": eng.param_count()}
             rng = np.random.default_rng(0)
@@ -195,7 +262,7 @@ def run(hb, hbm_gbs: float, tflops: float, steps: int, warmup: int, only: str = 
                         total[k] = (total.get(k, (0, 0))[0] + b, total.get(k, (0, 0))[1] + f)
                 res[label] = {"tok_s": round(n * length / ms * 1e3), "ms": round(ms, 3),
                               "kinds": kinds(prof, total, hbm_gbs, tflops)}
-            for batch in (1, 16, 64, 128):
+            for batch in batches:
                 ms, prof, n_launch = decode(eng, batch, ctx, steps, warmup, rows)
                 launches += n_launch * steps
                 w = work(shape, family, [np.arange(ctx + warmup + steps, ctx + warmup + steps + 1)] * batch, batch)
