@@ -299,15 +299,18 @@ int hb_attention_prepare(void* stream, const hb_attention_prep_args* a, int64_t 
  * of its expert, and batch tiles of m_pad places: expert e has tiles from place first[e] on,
  * tile_group[i] is the expert of tile i (-1: no such tile).  max_tiles >= min(experts, n) + n / m_pad
  * for n = rows * top.  count [experts + 1] is zero before and after.
+ * With `shared` every row has one pick more: group number `experts`, weight 1, tiles after all
+ * others (ceil(rows / m_pad) of them, counted in max_tiles).
  * hb_moe_gather: row r of h (stride ld) to place[r,k] = first + rank in x.
  * hb_gemm_grouped: Y[r] = X[r] . W[group of r]^T with [N, K] weights per group, on the sorted rows
- * (X, Y: max_tiles*m_pad rows; bf16 with K % 8 == 0 and m_pad % 16 == 0 on tensor cores); gated:
- * the N rows are [gate | up] and Y = act(gate, up), N/2 wide (bf16 only). */
+ * (X, Y: max_tiles*m_pad rows of strides ldx, ldy; bf16 with K % 8 == 0 and m_pad % 16 == 0 on tensor
+ * cores); gated: the N rows are [gate | up] and Y = act(gate, up), N/2 wide (bf16 only). */
 typedef struct hb_moe_routing {
   int experts, top, m_pad, max_tiles;
-  int32_t *ids, *rank, *place; /* [rows, top] */
-  float* weight;               /* [rows, top] */
-  int32_t *count, *first, *tile_group;
+  int32_t *ids, *rank, *place; /* [rows, top + shared] */
+  float* weight;               /* [rows, top + shared] */
+  int32_t *count, *first, *tile_group; /* [experts + 1], [experts + shared], [max_tiles] */
+  int shared;
 } hb_moe_routing;
 int hb_moe_route_top(void* stream, const hb_moe_routing* m, const void* h, int64_t ld_h, const void* router,
                      const float* bias, int64_t rows, int64_t width, hb_dtype dtype);
@@ -319,9 +322,21 @@ typedef struct hb_gated_act_spec {
 } hb_gated_act_spec;
 int hb_gated_act(void* stream, void* out, const void* gate_up, int64_t M, int64_t inter, const hb_gated_act_spec* act,
                  hb_dtype dtype);
-int hb_gemm_grouped(void* stream, void* Y, const void* X, const void* W, int groups, int64_t N, int64_t K, int m_pad,
-                    int max_tiles, int likely_tiles, const int32_t* tile_group, int out_f32,
-                    const hb_gated_act_spec* gated, hb_dtype dtype);
+typedef struct hb_grouped_gemm {
+  int groups;
+  int64_t N, K;
+  int m_pad, max_tiles, likely_tiles; /* likely_tiles steers the split of K */
+  const int32_t* tile_group;
+  int64_t ldx, ldy;
+  int gated, out_f32;
+  hb_gated_act_spec act;
+  const void* shared_w; /* NULL: none; else [shared_n, shared_k], the matrix of group number `groups` */
+  int64_t shared_n, shared_k;
+  hb_gated_act_spec shared_act;
+} hb_grouped_gemm;
+int hb_gemm_grouped(void* stream, void* Y, const void* X, const void* W, const hb_grouped_gemm* g, hb_dtype dtype);
+/* hb_gated_act on the rows of such a product whose gated is 0: rows of gate_up have stride ld_gu. */
+int hb_gated_act_grouped(void* stream, void* out, const void* gate_up, int64_t ld_gu, const hb_grouped_gemm* g, hb_dtype dtype);
 
 /* S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per head, state and outputs fp32.
  * p holds q, k (heads*dim), v (heads*vdim) and, for a low-rank decay, rank columns, at the given

@@ -304,7 +304,7 @@ def test_gated_activations(hb, cuda, slope, cubic, limit, shift, dtype):
 class Experts:
     """A whole mixture: routing, sorted rows, two grouped products, the weighted sum."""
 
-    def __init__(self, hb, rows, width, experts, top, ff, dtype, m_pad, limit=1.4, seed=0, skew=0.0):
+    def __init__(self, hb, rows, width, experts, top, ff, dtype, m_pad, limit=1.4, seed=0, skew=0.0, shared_ff=0):
         import torch
 
         rng = np.random.default_rng(seed)
@@ -325,32 +325,47 @@ class Experts:
             up[e, :ff, :width] = self.w[f"e{e}.gate"]
             up[e, ffp:ffp + ff, :width] = self.w[f"e{e}.up"]
             down[e, :width, :ff] = self.w[f"e{e}.down"]
-        n = rows * top
-        tiles = min(experts, n) + n // m_pad
+        n, picks = rows * top, top + (1 if shared_ff else 0)
+        tiles = min(experts, n) + n // m_pad + (-(-rows // m_pad) if shared_ff else 0)
+        sfp = (shared_ff + 7) // 8 * 8
+        s_up, s_down = np.zeros((2 * sfp, self.ld)), np.zeros((self.ld, sfp))
+        if shared_ff:
+            for name, shape in (("gate", (shared_ff, width)), ("up", (shared_ff, width)), ("down", (width, shared_ff))):
+                self.w["shared." + name] = rounded(1.5 * rng.standard_normal(shape) * shape[1] ** -0.5, dtype)
+            s_up[:shared_ff, :width], s_up[sfp:sfp + shared_ff, :width] = self.w["shared.gate"], self.w["shared.up"]
+            s_down[:width, :shared_ff] = self.w["shared.down"]
+        wide = max(ffp, sfp)
         z32 = lambda *s: torch.zeros(s, device="cuda", dtype=torch.int32)
-        self.ids, self.rank, self.place = z32(rows, top), z32(rows, top), z32(rows, top)
-        self.weight = torch.zeros((rows, top), device="cuda")
-        self.count, self.first, self.tiles = z32(experts + 1), z32(experts), z32(tiles)
+        self.ids, self.rank, self.place = z32(rows, picks), z32(rows, picks), z32(rows, picks)
+        self.weight = torch.zeros((rows, picks), device="cuda")
+        self.count, self.first, self.tiles = z32(experts + 1), z32(experts + 1), z32(tiles)
         r = hb.MoeRouting(experts, top, m_pad, tiles, *(t.data_ptr() for t in (self.ids, self.rank, self.place, self.weight,
-                                                                              self.count, self.first, self.tiles)))
+                                                                              self.count, self.first, self.tiles)),
+                          1 if shared_ff else 0)
         th, tr, tb = put(self.h, dtype), put(self.router, dtype), put(self.bias)
-        tu, td = put(up, dtype), put(down, dtype)
+        tu, td, tsu, tsd = put(up, dtype), put(down, dtype), put(s_up, dtype), put(s_down, dtype)
         x = put(np.zeros((tiles * m_pad, self.ld)), dtype)
-        act, y = put(np.zeros((tiles * m_pad, ffp)), dtype), put(np.zeros((tiles * m_pad, self.ld)), dtype)
-        spec = hb.GatedActSpec(1.702, 0.0, limit, 1.0)
+        act, y = put(np.zeros((tiles * m_pad, wide)), dtype), put(np.zeros((tiles * m_pad, self.ld)), dtype)
+        self.shared_limit = 0.6
+        spec, spec2 = hb.GatedActSpec(1.702, 0.0, limit, 1.0), hb.GatedActSpec(1.702, 0.0, self.shared_limit, 1.0)
         for _ in range(2):  # the second run finds the counters as the first one left them
             hb.check(hb.lib.hb_moe_route_top(None, C.byref(r), th.data_ptr(), self.ld, tr.data_ptr(), tb.data_ptr(), rows, width,
                                              dt(hb, dtype)))
             hb.check(hb.lib.hb_moe_gather(None, C.byref(r), x.data_ptr(), th.data_ptr(), self.ld, rows, dt(hb, dtype)))
-        args = (experts, 2 * ffp, self.ld, m_pad, tiles, max(1, tiles // 2), self.tiles.data_ptr(), 0)
+        likely = max(1, tiles // 2)
+        gu_gemm = hb.GroupedGemm(experts, 2 * ffp, self.ld, m_pad, tiles, likely, self.tiles.data_ptr(), self.ld, wide, 1, 0, spec,
+                                 tsu.data_ptr() if shared_ff else None, 2 * sfp, self.ld if shared_ff else 0, spec2)
+        down_gemm = hb.GroupedGemm(experts, self.ld, ffp, m_pad, tiles, likely, self.tiles.data_ptr(), wide, self.ld, 0, 0, spec,
+                                   tsd.data_ptr() if shared_ff else None, self.ld if shared_ff else 0, sfp, spec2)
         if dtype == "bf16":
-            hb.check(hb.lib.hb_gemm_grouped(None, act.data_ptr(), x.data_ptr(), tu.data_ptr(), *args, C.byref(spec), dt(hb, dtype)))
+            hb.check(hb.lib.hb_gemm_grouped(None, act.data_ptr(), x.data_ptr(), tu.data_ptr(), C.byref(gu_gemm), dt(hb, dtype)))
         else:
-            gu = put(np.zeros((tiles * m_pad, 2 * ffp)), dtype)
-            hb.check(hb.lib.hb_gemm_grouped(None, gu.data_ptr(), x.data_ptr(), tu.data_ptr(), *args, None, dt(hb, dtype)))
-            hb.check(hb.lib.hb_gated_act(None, act.data_ptr(), gu.data_ptr(), tiles * m_pad, ffp, C.byref(spec), dt(hb, dtype)))
-        hb.check(hb.lib.hb_gemm_grouped(None, y.data_ptr(), act.data_ptr(), td.data_ptr(), experts, self.ld, ffp, m_pad, tiles,
-                                        max(1, tiles // 2), self.tiles.data_ptr(), 0, None, dt(hb, dtype)))
+            gu = put(np.zeros((tiles * m_pad, 2 * wide)), dtype)
+            gu_gemm.gated, gu_gemm.ldy = 0, 2 * wide
+            hb.check(hb.lib.hb_gemm_grouped(None, gu.data_ptr(), x.data_ptr(), tu.data_ptr(), C.byref(gu_gemm), dt(hb, dtype)))
+            gu_gemm.ldy = wide
+            hb.check(hb.lib.hb_gated_act_grouped(None, act.data_ptr(), gu.data_ptr(), 2 * wide, C.byref(gu_gemm), dt(hb, dtype)))
+        hb.check(hb.lib.hb_gemm_grouped(None, y.data_ptr(), act.data_ptr(), td.data_ptr(), C.byref(down_gemm), dt(hb, dtype)))
         # the weighted sum goes into a plain residual stream together with a shared output and a bias
         self.x0, self.shared, self.o_bias = rng.standard_normal((rows, width)), rng.standard_normal((rows, self.ld)), \
             rng.standard_normal(width)
@@ -358,7 +373,7 @@ class Experts:
         tx, ts, to, tn, one = put(self.x0), put(self.shared), put(self.o_bias), put(self.norm), put(np.ones(1))
         out = put(np.zeros((rows, self.ld)), dtype)
         m = hb.StreamMixArgs(one.data_ptr(), one.data_ptr(), one.data_ptr(), tn.data_ptr(), None, None, 0.0, to.data_ptr(),
-                             y.data_ptr(), self.place.data_ptr(), self.weight.data_ptr(), top)
+                             y.data_ptr(), self.place.data_ptr(), self.weight.data_ptr(), picks)
         hb.check(hb.lib.hb_streams_mix_ex(None, tx.data_ptr(), out.data_ptr(), ts.data_ptr(), None, self.ld, C.byref(m), rows, 1,
                                           width, self.ld, 1e-5, dt(hb, dtype)))
         torch.cuda.synchronize()
@@ -371,19 +386,25 @@ class Experts:
         chosen, weight = R.route(h, self.router, self.bias, self.top)
         clear = R.route_margin(h, self.router, self.bias, self.top) > 1e-4
         assert clear.mean() > 0.9
-        ids, place = self.ids.cpu().numpy(), self.place.cpu().numpy()
+        ids, place, weights = self.ids.cpu().numpy(), self.place.cpu().numpy(), back(self.weight)
+        tiles = self.tiles.cpu().numpy()
+        # every place once, in a tile of its own expert
+        assert len(np.unique(place)) == place.size and np.array_equal(tiles[place // self.m_pad], ids)
+        used = sum(-(-int((ids == e).sum()) // self.m_pad) for e in range(self.experts + 1))
+        assert (tiles[:used] >= 0).all() and (tiles[used:] == -1).all()
+        if ids.shape[1] > self.top:
+            assert (ids[:, self.top] == self.experts).all() and (weights[:, self.top] == 1.0).all()
+        ids, weights = ids[:, :self.top], weights[:, :self.top]
         assert np.array_equal(np.sort(ids[clear]), np.sort(chosen[clear]))
         same = (ids == chosen).all(axis=1)
-        np.testing.assert_allclose(back(self.weight)[same], weight[same], atol=2e-5)
+        np.testing.assert_allclose(weights[same], weight[same], atol=2e-5)
         assert not self.count.cpu().numpy().any()
-        # every place once, in a tile of its own expert
-        tiles = self.tiles.cpu().numpy()
-        assert len(np.unique(place)) == place.size and np.array_equal(tiles[place // self.m_pad], ids)
-        assert (tiles >= 0).sum() == sum(-(-int((ids == e).sum()) // self.m_pad) for e in range(self.experts))
         want = self.x0 + self.shared[:, :self.width] + self.o_bias
         for t in range(self.rows):
             for e, p in zip(chosen[t], weight[t]):
                 want[t] += p * R.clamped_expert(h[t:t + 1], R.sub(self.w, f"e{e}."), self.limit)[0]
+        if "shared.up" in self.w:
+            want += R.clamped_expert(h, R.sub(self.w, "shared."), self.shared_limit)
         limit = 5e-3 if self.dtype == "bf16" else 2e-6
         assert rms_err(self.x1[clear], want[clear]) < limit
         assert rms_err(self.normed[clear], R.rms_norm(want, self.norm, 1e-5)[clear]) < 2 * limit
@@ -396,9 +417,12 @@ MOE = [  # rows, width, experts, top, ff, m_pad
 
 
 @pytest.mark.parametrize("rows,width,experts,top,ff,m_pad", MOE)
+@pytest.mark.parametrize("shared", ["no", "narrower", "wider"])
 @pytest.mark.parametrize("dtype", ["bf16", "f32"])
-def test_mixture_of_experts(hb, cuda, rows, width, experts, top, ff, m_pad, dtype):
-    Experts(hb, rows, width, experts, top, ff, dtype, m_pad, seed=rows).check()
+def test_mixture_of_experts(hb, cuda, rows, width, experts, top, ff, m_pad, shared, dtype):
+    """shared: one more expert that every row passes through, of another width and limit."""
+    shared_ff = {"no": 0, "narrower": max(3, ff // 3), "wider": 2 * ff + 70}[shared]
+    Experts(hb, rows, width, experts, top, ff, dtype, m_pad, seed=rows, shared_ff=shared_ff).check()
 
 
 @pytest.mark.parametrize("dtype", ["bf16", "f32"])

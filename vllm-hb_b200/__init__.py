@@ -123,13 +123,23 @@ class MoeRouting(C.Structure):
     _fields_ = [
         ("experts", C.c_int), ("top", C.c_int), ("m_pad", C.c_int), ("max_tiles", C.c_int), ("ids", C.c_void_p),
         ("rank", C.c_void_p), ("place", C.c_void_p), ("weight", C.c_void_p), ("count", C.c_void_p), ("first", C.c_void_p),
-        ("tile_group", C.c_void_p),
+        ("tile_group", C.c_void_p), ("shared", C.c_int),
     ]
 
 
 class GatedActSpec(C.Structure):
     """hb_gated_act_spec: g * sigmoid(slope * (g + cubic * g^3)) * (u + shift), clipped at limit."""
     _fields_ = [("slope", C.c_float), ("cubic", C.c_float), ("limit", C.c_float), ("shift", C.c_float)]
+
+
+class GroupedGemm(C.Structure):
+    """hb_grouped_gemm: a matrix product over rows sorted by group, every group with its own weights."""
+    _fields_ = [
+        ("groups", C.c_int), ("N", C.c_int64), ("K", C.c_int64), ("m_pad", C.c_int), ("max_tiles", C.c_int),
+        ("likely_tiles", C.c_int), ("tile_group", C.c_void_p), ("ldx", C.c_int64), ("ldy", C.c_int64), ("gated", C.c_int),
+        ("out_f32", C.c_int), ("act", GatedActSpec), ("shared_w", C.c_void_p), ("shared_n", C.c_int64), ("shared_k", C.c_int64),
+        ("shared_act", GatedActSpec),
+    ]
 
 
 class StreamMixArgs(C.Structure):
@@ -182,7 +192,8 @@ _SIGS = {
     "hb_moe_route_top": (_i, [_vp, _vp, _vp, _i64, _vp, _vp, _i64, _i64, _i]),
     "hb_moe_gather": (_i, [_vp, _vp, _vp, _vp, _i64, _i64, _i]),
     "hb_gated_act": (_i, [_vp, _vp, _vp, _i64, _i64, _vp, _i]),
-    "hb_gemm_grouped": (_i, [_vp, _vp, _vp, _vp, _i, _i64, _i64, _i, _i, _i, _vp, _i, _vp, _i]),
+    "hb_gemm_grouped": (_i, [_vp, _vp, _vp, _vp, _vp, _i]),
+    "hb_gated_act_grouped": (_i, [_vp, _vp, _vp, _i64, _vp, _i]),
     "hb_streams_final": (_i, [_vp, _vp, _vp, _vp, _vp, _i64, _i, _i64, _i64, _f, _i]),
     "hb_gated_group_norm": (_i, [_vp, _vp, _i64, _vp, _i64, _vp, _i64, _vp, _i64, _i, _i, _i, _f, _i]),
     "hb_gemm_workspace_bytes": (_sz, [_i64, _i64, _i64, _i]),

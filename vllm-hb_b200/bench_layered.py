@@ -124,17 +124,20 @@ def work(shape: dict, family: str, positions: list[np.ndarray], wanted: int) -> 
             attention(m["heads"], m["kv_heads"], m["dim"], m["vdim"], 0, 0, m.get("mask", {}).get("size", 0), tied, True)
             gemm("gemm_o_proj", H, v, out=4)
             add("norm", 2 * rows * H * 14.0)
-            I = f["ff"] if f["kind"] == "dense" else f["shared"]["ff"]
-            gemm("gemm_gate_up", 2 * I, H, n_out=I)
-            gemm("gemm_down", H, I, out=4)
-            if f["kind"] == "moe":
+            if f["kind"] == "dense":
+                gemm("gemm_gate_up", 2 * f["ff"], H, n_out=f["ff"])
+                gemm("gemm_down", H, f["ff"], out=4)
+            else:  # the experts' products, the shared one among them
+                S = f["shared"]["ff"]
+                gemm("experts_gate_up", 2 * S, H, n_out=S)
+                gemm("experts_down", H, S)
                 E, top, F = f["router"]["experts"], f["router"]["top"], f["expert"]["ff"]
                 picks = rows * top
                 active = E * (1.0 - (1.0 - top / E) ** rows)
-                add("routing", 2.0 * E * H + 2.0 * rows * H * (1 + top))
+                add("routing", 2.0 * E * H + 2.0 * rows * H * (2 + top))
                 add("experts_gate_up", 4.0 * active * F * H + 2.0 * picks * (H + F), 4.0 * picks * F * H)
                 add("experts_down", 2.0 * active * F * H + 2.0 * picks * (H + F), 2.0 * picks * F * H)
-                add("norm", 2.0 * picks * H)
+                add("norm", (2.0 * picks + 2.0 * rows) * H)
         add("norm", wanted * H * 6.0)
         gemm("gemm_lm_head", shape["vocab"], H, m=wanted, out=4)
         return w

@@ -44,6 +44,14 @@ __global__ void __launch_bounds__(kPrepThreads) attention_rotate_kernel(const At
   const int64_t row = blockIdx.x, slot = a.slots[row];
   const int tid = threadIdx.x, P = a.pairs, D = a.dim;
   const bool keep = slot >= 0 && slot < a.num_blocks * HB_BLOCK_SIZE;
+  T* pr = (T*)a.p + row * a.ld;
+  constexpr int W = V == 1 ? 2 : V;           // channels a thread turns at a time
+  const int per = (D + W - 1) / W, total = (a.heads + a.kv_heads) * per;
+  // channels i of head i / per: queries first, then keys
+  auto source = [&](int i) { return pr + (i < a.heads * per ? a.off_q : a.off_k - a.heads * D) + i / per * D + i % per * W; };
+  Vec16<T> ahead;  // the first run of every thread is on its way while the angles are formed
+  if constexpr (V > 1)
+    if (tid < total) ahead.load(source(tid));
   // the angle less its whole turns in fp64: far positions keep the accuracy of near ones
   const double pos = (double)a.pos[row], turn = 6.283185307179586;
   for (int i = tid; i < P; i += kPrepThreads) {
@@ -51,21 +59,19 @@ __global__ void __launch_bounds__(kPrepThreads) attention_rotate_kernel(const At
     sincosf((float)(angle - turn * rint(angle * (1.0 / turn))), s_cs + P + i, s_cs + i);
   }
   __syncthreads();
-  T* pr = (T*)a.p + row * a.ld;
-  constexpr int W = V == 1 ? 2 : V;           // channels a thread turns at a time
-  const int per = (D + W - 1) / W, total = (a.heads + a.kv_heads) * per;
   for (int i = tid; i < total; i += kPrepThreads) {
     const int head = i / per, d = i % per * W;
     const bool query = head < a.heads;
-    const int g = query ? head : head - a.heads, off = query ? a.off_q : a.off_k;
+    const int g = query ? head : head - a.heads;
     const float* bias = query ? a.q_bias : a.k_bias;
-    T* src = pr + off + g * D + d;
+    T* src = source(i);
     float f[W];
     if constexpr (V == 1) {
       f[0] = to_f32<T>(src[0]);
       f[1] = d + 1 < D ? to_f32<T>(src[1]) : 0.f;
     } else {
-      Run<T, V>::load(f, src);
+      if (i >= kPrepThreads) ahead.load(src);
+      ahead.unpack(f);
     }
     if (bias)
 #pragma unroll
@@ -98,60 +104,97 @@ __global__ void __launch_bounds__(kPrepThreads) attention_rotate_kernel(const At
   }
 }
 
-// RMS norms over all query rows and all key rows of a position.
+// RMS norms over all query rows and all key rows of a position.  A thread keeps its first kHeld runs
+// of queries and its first run of keys in registers between the sums and the results.
+constexpr int kHeld = 2;
 template <typename T, int V>
 __global__ void __launch_bounds__(kPrepThreads) attention_norm_kernel(const AttentionPrep a) {
   pdl_trigger();
   pdl_grid_wait();
-  __shared__ float red[33];
+  __shared__ float red[2][33];
   const int64_t row = blockIdx.x, slot = a.slots[row];
   const int tid = threadIdx.x, D = a.dim, nq = a.heads * D, nk = a.kv_heads * D, rep = a.heads / a.kv_heads;
   const bool keep = slot >= 0 && slot < a.num_blocks * HB_BLOCK_SIZE, tied = a.key_scale != nullptr;
   T* q = (T*)a.p + row * a.ld + a.off_q;
   const T* k = (const T*)a.p + row * a.ld + a.off_k;
+  constexpr int step = kPrepThreads * V;
   auto load = [&](float (&f)[V], const T* src, const float* bias, int i) {
     Run<T, V>::load(f, src + i);
     if (bias)
 #pragma unroll
       for (int j = 0; j < V; ++j) f[j] += bias[i + j];
   };
-  float sq = 0.f, sk = 0.f, f[V];
-  for (int i = tid * V; i < nq; i += kPrepThreads * V) {
-    load(f, q, a.q_bias, i);
+  auto squares = [&](const float (&f)[V], float s) {
 #pragma unroll
-    for (int j = 0; j < V; ++j) sq = fmaf(f[j], f[j], sq);
+    for (int j = 0; j < V; ++j) s = fmaf(f[j], f[j], s);
+    return s;
+  };
+  float sq = 0.f, sk = 0.f, f[V], held[kHeld][V], key[V];
+#pragma unroll
+  for (int n = 0; n < kHeld; ++n)
+    if (tid * V + n * step < nq) load(held[n], q, a.q_bias, tid * V + n * step);
+  if (tid * V < nk) load(key, k, a.k_bias, tid * V);
+#pragma unroll
+  for (int n = 0; n < kHeld; ++n)
+    if (tid * V + n * step < nq) sq = squares(held[n], sq);
+  if (tid * V < nk) sk = squares(key, sk);
+  for (int i = tid * V + kHeld * step; i < nq; i += step) {
+    load(f, q, a.q_bias, i);
+    sq = squares(f, sq);
   }
-  for (int i = tid * V; i < nk; i += kPrepThreads * V) {
+  for (int i = tid * V + step; i < nk; i += step) {
     load(f, k, a.k_bias, i);
-#pragma unroll
-    for (int j = 0; j < V; ++j) sk = fmaf(f[j], f[j], sk);
+    sk = squares(f, sk);
   }
-  const float rq = 1.f / sqrtf(block_sum(sq, red) / (float)nq + a.eps);
-  const float rk = 1.f / sqrtf(block_sum(sk, red) / (float)nk + a.eps);
-  for (int i = tid * V; i < nq; i += kPrepThreads * V) {
-    load(f, q, a.q_bias, i);
+  // both sums behind one barrier
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if ((tid & 31) == 0) {
+    red[0][tid >> 5] = sq;
+    red[1][tid >> 5] = sk;
+  }
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int w = 0; w < kPrepThreads / 32; ++w) {
+    sq += red[0][w];
+    sk += red[1][w];
+  }
+  const float rq = 1.f / sqrtf(sq / (float)nq + a.eps), rk = 1.f / sqrtf(sk / (float)nk + a.eps);
+  auto query = [&](float (&v)[V], int i) {
     const int at = tied ? i / (rep * D) * D + i % D : 0;  // the key channel this query channel meets
 #pragma unroll
     for (int j = 0; j < V; ++j) {
-      f[j] *= rq * a.q_norm[i + j];
-      if (tied) f[j] *= a.k_norm[at + j];
+      v[j] *= rq * a.q_norm[i + j];
+      if (tied) v[j] *= a.k_norm[at + j];
     }
-    Run<T, V>::store(q + i, f);
-  }
-  if (!keep) return;
-  for (int i = tid * V; i < nk; i += kPrepThreads * V) {
-    load(f, k, a.k_bias, i);
+    Run<T, V>::store(q + i, v);
+  };
+  auto keyed = [&](float (&v)[V], int i) {
     if (!tied)
 #pragma unroll
-      for (int j = 0; j < V; ++j) f[j] *= rk * a.k_norm[i + j];
-    Run<T, V>::store((T*)a.kc + pool_at(slot, a.kv_heads, i / D, D, i % D), f);
+      for (int j = 0; j < V; ++j) v[j] *= rk * a.k_norm[i + j];
+    Run<T, V>::store((T*)a.kc + pool_at(slot, a.kv_heads, i / D, D, i % D), v);
+  };
+#pragma unroll
+  for (int n = 0; n < kHeld; ++n)
+    if (tid * V + n * step < nq) query(held[n], tid * V + n * step);
+  for (int i = tid * V + kHeld * step; i < nq; i += step) {
+    load(f, q, a.q_bias, i);
+    query(f, i);
+  }
+  if (!keep) return;
+  if (tid * V < nk) keyed(key, tid * V);
+  for (int i = tid * V + step; i < nk; i += step) {
+    load(f, k, a.k_bias, i);
+    keyed(f, i);
   }
   if (tied) {
     if (tid == 0) a.key_scale[slot] = rk;
     return;
   }
   const int nv = a.kv_heads * a.vdim;
-  for (int i = tid * V; i < nv; i += kPrepThreads * V) {
+  for (int i = tid * V; i < nv; i += step) {
     Run<T, V>::load(f, (const T*)a.p + row * a.ld + a.off_v + i);
     Run<T, V>::store((T*)a.vc + pool_at(slot, a.kv_heads, i / a.vdim, a.vdim, i % a.vdim), f);
   }

@@ -30,6 +30,7 @@ constexpr int kKeys = 64;      // keys of a tile step
 constexpr int kBS = HB_BLOCK_SIZE;
 constexpr int kSlice = 256;    // widest value slice
 constexpr int kRing = 3;       // 16-key stages of a warp (token kernel)
+constexpr int kMaxCluster = 8; // splits of a row that sum up in a cluster
 
 __host__ __device__ constexpr int pad16(int n) { return (n + 15) / 16 * 16; }
 
@@ -307,20 +308,22 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
   }
 }
 
-// n_splits > 1: every CTA takes its share of the row's blocks and writes (m, l, O) partials.
+// n_splits > 1: every CTA takes its share of the row's blocks.  The CTAs of a row and kv head form a
+// thread-block cluster (`clustered`) and sum up through each other's shared memory, or, more than
+// fit one, write (m, l, O) partials that a second kernel sums up.
 //
 // The products are turned over, so that the few query heads are the narrow MMA side:
 // S^T[16 keys, 8 NT heads] = K Q^T and O^T[values, heads] += V^T P^T (P transposed in registers).
 // MT: 16-column tiles of the value slice, NT: groups of 8 query heads.
 template <int MT, int NT, bool EXT>
 __global__ void __launch_bounds__(kThreads)
-span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, int n_splits, float* __restrict__ part) {
+span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, int n_splits, int clustered,
+                             float* __restrict__ part) {
   extern __shared__ __align__(16) uint8_t smem[];
   const int R = a.heads / a.kv_heads, D = a.dim, DP = pad16(D), KS = DP + 8;
-  const int slices = (a.vdim + kSlice - 1) / kSlice;
   const bool tied = EXT && a.key_scale != nullptr;  // one tile is keys and values; their scales lie behind it
-  const int v0 = (int)(blockIdx.z % slices) * kSlice, VW = min(kSlice, a.vdim - v0), VP = pad16(VW), VS = VP + 8;
-  const int split = blockIdx.z / slices;
+  const int v0 = (int)(blockIdx.z / n_splits) * kSlice, VW = min(kSlice, a.vdim - v0), VP = pad16(VW), VS = VP + 8;
+  const int split = blockIdx.z % n_splits;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gi = lane >> 2, t = lane & 3, kvh = blockIdx.y;
   const int stage_elems = tied ? kBS * (KS + 2) : kBS * (KS + VS);
   __nv_bfloat16* s_q = (__nv_bfloat16*)smem;                                  // [16][KS]
@@ -530,7 +533,7 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
       const float k = a.sink[head] * kLog2e, top = fmaxf(mx, k), f = ex2(mx - top);
       inv = f / fmaf(ls, f, ex2(k - top));
     }
-    float* p = n_splits > 1 ? part + (((int64_t)blockIdx.x * a.heads + head) * n_splits + split) * (a.vdim + 2) : nullptr;
+    float* p = n_splits > 1 && !clustered ? part + (((int64_t)blockIdx.x * a.heads + head) * n_splits + split) * (a.vdim + 2) : nullptr;
     for (int c = lane; c < VW; c += 32) {
       float acc = 0.f;
 #pragma unroll
@@ -539,12 +542,47 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
         acc *= inv;
         if (a.gate) acc *= sigmoid_of(((const uint16_t*)a.gate)[row * a.ld_gate + head * a.vdim + v0 + c]);
         ((__nv_bfloat16*)a.out)[row * a.ld_out + head * a.vdim + v0 + c] = __float2bfloat16_rn(acc);
+      } else if (clustered) {
+        s_o[(size_t)h * OS + c] = acc;  // the place of warp 0, read by this lane above
       } else {
         p[v0 + c] = acc;
       }
     }
-    if (n_splits > 1 && lane == 0 && v0 == 0) { p[a.vdim] = mx; p[a.vdim + 1] = ls; }
+    if (clustered) {
+      __syncwarp();
+      if (lane == 0) { s_ml[h * 2] = mx; s_ml[h * 2 + 1] = ls; }
+    } else if (n_splits > 1 && lane == 0 && v0 == 0) {
+      p[a.vdim] = mx;
+      p[a.vdim + 1] = ls;
+    }
   }
+  if (!clustered) return;
+  cluster_sync_all();
+  const uint32_t o_addr = smem_u32(s_o), ml_addr = smem_u32(s_ml);
+  for (int i = split * kThreads + tid; i < R * VW; i += n_splits * kThreads) {
+    const int h = i / VW, c = i % VW;
+    const int64_t head = (int64_t)kvh * R + h;
+    const float k = a.sink ? a.sink[head] * kLog2e : -INFINITY;
+    float mx = k, ls = 0.f, acc = 0.f, mw[kMaxCluster];
+#pragma unroll
+    for (int s = 0; s < kMaxCluster; ++s) {
+      mw[s] = s < n_splits ? ld_cluster_f32(cluster_map(ml_addr + h * 8, s)) : -INFINITY;
+      mx = fmaxf(mx, mw[s]);
+    }
+    if (a.sink) ls = ex2(k - mx);
+#pragma unroll
+    for (int s = 0; s < kMaxCluster; ++s) {
+      if (s < n_splits) {
+        const float f = mw[s] == -INFINITY ? 0.f : ex2(mw[s] - mx);
+        ls = fmaf(f, ld_cluster_f32(cluster_map(ml_addr + h * 8 + 4, s)), ls);
+        acc = fmaf(f, ld_cluster_f32(cluster_map(o_addr + (uint32_t)(h * OS + c) * 4, s)), acc);
+      }
+    }
+    acc /= ls;
+    if (a.gate) acc *= sigmoid_of(((const uint16_t*)a.gate)[row * a.ld_gate + head * a.vdim + v0 + c]);
+    ((__nv_bfloat16*)a.out)[row * a.ld_out + head * a.vdim + v0 + c] = __float2bfloat16_rn(acc);
+  }
+  cluster_sync_all();  // nobody leaves while a partner still reads its shared memory
 }
 
 // Sum of a row's split partials, weighted by their maxima.
@@ -635,11 +673,30 @@ int span_attention_tokens(cudaStream_t st, const SpanAttention& a, const int32_t
   if (n_rows == 0) return HB_OK;
   const size_t smem = tokens_smem(a);
   const int slices = (a.vdim + kSlice - 1) / kSlice;
+  const bool clustered = n_splits > 1 && n_splits <= kMaxCluster;
   const dim3 grid((unsigned)n_rows, (unsigned)a.kv_heads, (unsigned)(slices * n_splits));
   auto launch = [&](auto* k) -> int {
     int rc = opt_in(k, smem);
     if (rc) return rc;
-    HB_CUDA_CHECK(launch_pdl(k, grid, dim3(kThreads), smem, st, a, rows, n_splits, part));
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = dim3(kThreads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute attr[2];
+    int n = 0;
+    if (pdl_enabled()) {
+      attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+      attr[n++].val.programmaticStreamSerializationAllowed = 1;
+    }
+    if (clustered) {
+      attr[n].id = cudaLaunchAttributeClusterDimension;
+      attr[n].val.clusterDim.x = attr[n].val.clusterDim.y = 1;
+      attr[n++].val.clusterDim.z = (unsigned)n_splits;
+    }
+    cfg.attrs = attr;
+    cfg.numAttrs = n;
+    HB_CUDA_CHECK(cudaLaunchKernelEx(&cfg, k, a, rows, n_splits, clustered ? 1 : 0, part));
     return HB_OK;
   };
   const int vw = std::min(a.vdim, kSlice);
@@ -653,7 +710,7 @@ int span_attention_tokens(cudaStream_t st, const SpanAttention& a, const int32_t
   else if (vw <= 128) HB_TOKENS(8);
   else HB_TOKENS(16);
 #undef HB_TOKENS
-  if (rc || n_splits == 1) return rc;
+  if (rc || n_splits == 1 || clustered) return rc;
   HB_CUDA_CHECK(launch_pdl(span_attention_merge_kernel, dim3((unsigned)n_rows, (unsigned)a.heads), dim3(kThreads), 0, st, a, rows,
                            n_splits, (const float*)part));
   return HB_OK;

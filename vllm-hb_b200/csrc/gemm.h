@@ -27,15 +27,25 @@ int gated_act(cudaStream_t st, void* out, const void* gate_up, int64_t M, int64_
 // Rows of a GEMM sorted by group (mixture of experts): every batch tile of `m_pad` rows belongs to
 // one group, whose weights start at row group * (weight rows of one group); tile_group[i] < 0: no
 // such tile.  The number of tiles is only known on the device; `max_tiles` bounds it, `likely_tiles`
-// steers the split of K.
+// steers the split of K.  One further group, number `groups`, may have a [shared_n, shared_k] matrix
+// and an activation of its own (the expert every token passes through); rows of X and Y have
+// strides of ldx and ldy elements, so that groups of different K and N share them.
 struct TcGroups {
   int groups = 0;
   int m_pad = 0;
   int max_tiles = 0, likely_tiles = 0;
+  const void* shared_w = nullptr;
+  int64_t shared_n = 0, shared_k = 0;
+  GatedAct shared_act;
+  int64_t ldx = 0, ldy = 0;  // 0: K, N
 };
 // CUDA-core form: Y[r] = X[r] . W[group of r]^T, tiles of m_pad rows (a multiple of 8).
 int gemm_simt_grouped(cudaStream_t st, void* Y, const void* X, const void* W, int64_t N, int64_t K, hb_dtype dtype, bool out_f32,
                       const TcGroups& groups, const int32_t* tile_group);
+// gated_act over the rows of such a GEMM: gate | up rows of stride ld_gu, out rows of stride ld_out;
+// inter and act of the groups, and of the further one.
+int gated_act_grouped(cudaStream_t st, void* out, int64_t ld_out, const void* gate_up, int64_t ld_gu, int64_t inter,
+                      const GatedAct& act, hb_dtype dtype, const TcGroups& groups, const int32_t* tile_group);
 
 // What the tensor-core kernel does with the finished fp32 tile.
 enum TcEpilogue : int {
@@ -121,6 +131,10 @@ struct TcGemmPlan {
   GatedAct act;          // kEpiSwiGLU
   int groups = 0;        // > 0: TcGroups form; rows of the batch operand are sorted by group
   int group_rows = 0;    // weight rows of one group
+  CUtensorMap tm_w2;     // further group: its weights, features, K and activation
+  int64_t N2 = 0, K2 = 0;
+  GatedAct act2;
+  int64_t ldx = 0, ldy = 0;
   bool out_f32 = false;
   bool tma_store = false;  // output rows are 16-byte multiples: bulk tensor stores
   // scratch layout inside the caller's workspace

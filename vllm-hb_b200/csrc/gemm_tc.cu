@@ -52,6 +52,9 @@ struct TcParams {
   int act_silu;
   const int32_t* tile_group;  // TcGroups: group of every batch tile (negative: no such tile)
   int group_rows;             // weight rows of one group
+  int further;                // number of the further group (tm_h holds its weights), -1: none
+  int n_tiles2, k_chunks2, up_row_offset2, act_silu2;
+  GatedAct act2;
   int cluster;              // split-K partners form a thread-block cluster of `splits` CTAs
   int tma_store;            // the output leaves through bulk tensor stores (tm_y is valid)
   // Deferred RMSNorm (see TcNormLink in gemm.h).  Producer (epilogue kEpiResidual, cluster
@@ -157,13 +160,13 @@ __device__ __forceinline__ void push_tile(const TcParams& p, const uint8_t* stag
 }
 
 // Gated activation of one output element (fast divide and exponential, as silu_f).
-__device__ __forceinline__ float gated_f(float g, float u, const TcParams& p) {
-  if (p.act_silu) return silu_f(g) * u;
-  g = fminf(g, p.act.limit);
-  u = fminf(fmaxf(u, -p.act.limit), p.act.limit);
-  const float z = p.act.slope * fmaf(p.act.cubic * g * g, g, g);
+__device__ __forceinline__ float gated_f(float g, float u, bool silu, const GatedAct& act) {
+  if (silu) return silu_f(g) * u;
+  g = fminf(g, act.limit);
+  u = fminf(fmaxf(u, -act.limit), act.limit);
+  const float z = act.slope * fmaf(act.cubic * g * g, g, g);
   // far below zero the gate is zero (the fast divide wants a denominator below 2^126)
-  return z < -80.f ? 0.f : __fdividef(g, 1.f + __expf(-z)) * (u + p.act.shift);
+  return z < -80.f ? 0.f : __fdividef(g, 1.f + __expf(-z)) * (u + act.shift);
 }
 
 // ----------------------------------------------------------------------- kernel
@@ -196,14 +199,28 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
   const int split = p.cluster ? (int)cluster_ctarank() : blockIdx.x % p.splits;
   const int m_tile = blockIdx.y;
   int w_row = tile * kTileN;  // first weight row of the tile
+  const CUtensorMap* w_map = &tm_w;
+  int k_chunks = p.k_chunks, up_row_offset = p.up_row_offset;
+  bool act_silu = p.act_silu != 0;
+  GatedAct act = p.act;
   if (p.tile_group) {
     // rows sorted by group: the previous kernels say whose weights this batch tile meets
     pdl_wait();
     const int group = p.tile_group[m_tile];
-    if (group < 0) return;  // uniform over the grid row, so over every cluster
-    w_row += group * p.group_rows;
+    const bool further = group == p.further;
+    // uniform over the CTAs of a tile, so over every cluster
+    if (group < 0 || tile >= (further ? p.n_tiles2 : p.n_tiles)) return;
+    if (further) {
+      w_map = &tm_h;
+      k_chunks = p.k_chunks2;
+      up_row_offset = p.up_row_offset2;
+      act_silu = p.act_silu2 != 0;
+      act = p.act2;
+    } else {
+      w_row += group * p.group_rows;
+    }
   }
-  const int base_c = p.k_chunks / p.splits, rem_c = p.k_chunks % p.splits;
+  const int base_c = k_chunks / p.splits, rem_c = k_chunks % p.splits;
   const int kc0 = split * base_c + min(split, rem_c);
   const int n_kc = base_c + (split < rem_c ? 1 : 0);
 
@@ -303,7 +320,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
       // every weight byte is read once per launch: it may leave L2 first (measured +1 % on the
       // 8B decode step against the default policy)
       auto load_w = [&](uint32_t dst, int kx, int row, uint32_t bar) {
-        tma_load_2d_hint(dst, &tm_w, kx, row, bar, w_policy);
+        tma_load_2d_hint(dst, w_map, kx, row, bar, w_policy);
       };
       // Weights never depend on the previous kernel: the first stages' weight slabs are
       // requested before waiting for it; activations only afterwards.
@@ -314,7 +331,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
         mbar_expect_tx(full, stage_bytes);
         const int kx = (kc0 + i) * kTileK;
         load_w(sa, kx, w_row, full);
-        if (swiglu) load_w(sa + a_bytes, kx, p.up_row_offset + w_row, full);
+        if (swiglu) load_w(sa + a_bytes, kx, up_row_offset + w_row, full);
       }
       // (Requesting further chunks into L2 at this point was measured harmful: -2 % to -7 % per
       // decode step after HBM-bound kernels, no gain after an NVLink exchange.  Requesting the
@@ -339,7 +356,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
         mbar_expect_tx(full, stage_bytes);
         const int kx = (kc0 + i) * kTileK;
         load_w(sa, kx, w_row, full);
-        if (swiglu) load_w(sa + a_bytes, kx, p.up_row_offset + w_row, full);
+        if (swiglu) load_w(sa + a_bytes, kx, up_row_offset + w_row, full);
         tma_load_2d(sa + a_bytes * n_acc, &tm_x, kx, m_tile * p.m_pad, full);
         armed = i + 1;
       }
@@ -527,7 +544,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           }
         }
 #pragma unroll
-        for (int j = 0; j < 16; ++j) g[j] = swiglu ? gated_f(g[j], u[j], p) : g[j];
+        for (int j = 0; j < 16; ++j) g[j] = swiglu ? gated_f(g[j], u[j], act_silu, act) : g[j];
         if (p.post_scale) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) g[j] *= s_pscale[c0 + j];
@@ -675,7 +692,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
             for (int j = 0; j < 16; ++j) u[j] *= s_rscale[g * 16 + j];
           }
 #pragma unroll
-          for (int j = 0; j < 16; ++j) v[j] = gated_f(v[j], u[j], p);
+          for (int j = 0; j < 16; ++j) v[j] = gated_f(v[j], u[j], act_silu, act);
         }
         if (p.post_scale) {
 #pragma unroll
@@ -715,7 +732,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           float u[16];
           tmem_ld16(t_lane + p.m_pad + c0, u);
 #pragma unroll
-          for (int j = 0; j < 16; ++j) v[j] = gated_f(v[j], u[j], p);
+          for (int j = 0; j < 16; ++j) v[j] = gated_f(v[j], u[j], act_silu, act);
         }
         if (n_glob < p.N) {
 #pragma unroll
@@ -772,7 +789,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           for (int j = 0; j < 8; ++j) {
             const int m = m0 + j;
             if (m < m_lim && n_glob < p.N) {
-              const float r = swiglu ? gated_f(g[j], u[j], p) : g[j];
+              const float r = swiglu ? gated_f(g[j], u[j], act_silu, act) : g[j];
               if (p.out_f32) ((float*)p.Y)[(int64_t)(m_base + m) * p.ldy + n_glob] = r;
               else ((__nv_bfloat16*)p.Y)[(int64_t)(m_base + m) * p.ldy + n_glob] = __float2bfloat16_rn(r);
             }
@@ -909,7 +926,9 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
   pl.groups = groups ? groups->groups : 0;
   pl.group_rows = groups ? (int)N : 0;
   if (groups && (groups->groups < 1 || groups->m_pad < 16 || groups->m_pad > 128 || groups->m_pad % 16 || groups->max_tiles < 1 ||
-                 groups->likely_tiles < 1 || (int64_t)groups->max_tiles * groups->m_pad > M || epilogue > kEpiSwiGLU))
+                 groups->likely_tiles < 1 || (int64_t)groups->max_tiles * groups->m_pad > M || epilogue > kEpiSwiGLU ||
+                 (groups->ldx && (groups->ldx < K || groups->ldx % 8)) || (groups->shared_w && (groups->shared_k % 8 ||
+                 groups->shared_n < 1 || groups->shared_k < 8 || groups->ldx < std::max(K, groups->shared_k)))))
     return fail(HB_ERR_INVALID_ARG, "gemm_tc: bad groups");
   const int n_acc = epilogue == kEpiSwiGLU ? 2 : 1;
   if (epilogue == kEpiSwiGLU && N % 2) return fail(HB_ERR_INVALID_ARG, "gemm_tc: SwiGLU needs even N");
@@ -922,7 +941,17 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
   const int64_t m_eff = std::min<int64_t>(M, m_cap);
   pl.m_pad = (int)std::max<int64_t>(16, (m_eff + 15) / 16 * 16);
   pl.n_tiles = (int)((n_rows + kTileN - 1) / kTileN);
-  const int k_chunks = (int)((K + kTileK - 1) / kTileK);
+  int k_chunks = (int)((K + kTileK - 1) / kTileK);
+  if (groups) {
+    pl.ldx = groups->ldx ? groups->ldx : K;
+    pl.ldy = groups->ldy ? groups->ldy : n_rows;
+    if (groups->shared_w) {
+      pl.N2 = epilogue == kEpiSwiGLU ? groups->shared_n / 2 : groups->shared_n;
+      pl.K2 = groups->shared_k;
+      pl.act2 = groups->shared_act;
+      k_chunks = std::min(k_chunks, (int)((pl.K2 + kTileK - 1) / kTileK));  // what the split of K can count on
+    }
+  }
   const bool want_cluster = true;  // split-K partners reduce on chip; global scratch only where a cluster cannot form
   const bool tuned = want_cluster && force_splits <= 0;
   if (groups) pl.m_pad = groups->m_pad;
@@ -1061,7 +1090,8 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
   }
   rc = encode_map(&pl.tm_w, W, groups ? N * groups->groups : N, K, kTileN);
   if (rc) return rc;
-  rc = encode_map(&pl.tm_x, X, M, K, pl.m_pad);
+  rc = encode_map(&pl.tm_x, X, M, groups ? pl.ldx : K, pl.m_pad);
+  if (!rc && pl.N2) rc = encode_map(&pl.tm_w2, groups->shared_w, groups->shared_n, pl.K2, kTileN);
   return rc;
 }
 
@@ -1102,6 +1132,12 @@ int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, voi
   p.act_silu = pl.act.silu() ? 1 : 0;
   p.tile_group = tile_group;
   p.group_rows = pl.group_rows;
+  p.further = pl.N2 ? pl.groups : -1;
+  p.n_tiles2 = (int)((pl.N2 + kTileN - 1) / kTileN);
+  p.k_chunks2 = (int)((pl.K2 + kTileK - 1) / kTileK);
+  p.up_row_offset2 = (int)pl.N2;
+  p.act2 = pl.act2;
+  p.act_silu2 = pl.act2.silu() ? 1 : 0;
   p.Y = Y;
   // counters first (16-byte aligned block), partials after
   p.counters = (int*)workspace;
@@ -1133,11 +1169,15 @@ int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, voi
   }
   if (p.tma_store && !push) {
     const int box_rows = pl.cluster ? pl.m_pad / pl.splits : 16;
-    int rc = encode_out_map(&tm_y, Y, pl.M, pl.N, ldy, pl.out_f32, box_rows);
+    // groups of different widths share the rows: columns between one's width and the next
+    // multiple of 128 may be written, and every reader of them multiplies them by zero
+    int rc = encode_out_map(&tm_y, Y, pl.M, pl.groups ? std::min(ldy, std::max(pl.N, pl.N2)) : pl.N, ldy, pl.out_f32, box_rows);
     if (rc) return rc;
   }
   CUtensorMap tm_h;
   memset(&tm_h, 0, sizeof(tm_h));
+  if (pl.groups && !p.tma_store) return fail(HB_ERR_INVALID_ARG, "gemm_tc: grouped plans need output rows of 16-byte multiples");
+  if (pl.N2) tm_h = pl.tm_w2;
   if (pl.epilogue == kEpiResidual) {
     if (!pl.cluster || !p.tma_store || pl.out_f32 || !link || !link->resid || !link->norm_w || !link->rowsq_out)
       return fail(HB_ERR_INVALID_ARG, "gemm_tc: the residual epilogue needs a cluster plan, bf16 output and a norm link");
@@ -1184,7 +1224,7 @@ int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, voi
     p.rs_inv_n = 1.0f / link->n;
     p.rs_eps = link->eps;
   }
-  dim3 grid((unsigned)(pl.n_tiles * pl.splits), (unsigned)pl.m_tiles);
+  dim3 grid((unsigned)(std::max(pl.n_tiles, p.n_tiles2) * pl.splits), (unsigned)pl.m_tiles);
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = grid;
   cfg.blockDim = dim3(kTcThreads);

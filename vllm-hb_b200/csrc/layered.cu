@@ -149,7 +149,7 @@ struct Loader {
     if ((rc = part(*gate_up, f.up, *ffp, f.ff, W))) return rc;
     return linear(down, f.down, W, f.ff);
   }
-  int experts(LayeredExperts* x, const ExpertsSpec& s) {
+  int experts(LayeredExperts* x, const ExpertsSpec& s, const FeedForwardSpec& shared) {
     const int64_t W = m->spec.width, E = s.experts;
     int rc;
     x->ffp = pad8(s.ff);
@@ -169,6 +169,7 @@ struct Loader {
     if ((rc = src.fetch_all(s.router, E, W, x->router, e->dtype))) return rc;
     e->named[s.router] = {x->router, E, W};
     m->params += E * W;
+    if (shared.ff && (rc = gated(&x->shared_gate_up, &x->shared_down, &x->shared_ffp, shared))) return rc;
     return small(&x->router_bias, s.router_bias, 1, E, 0.f);
   }
 };
@@ -235,8 +236,9 @@ static int layered_load(hb_engine* e, TensorSource& src) {
       if ((rc = ld.small(&l.rec_out_norm, mx.rec_out_norm, 1, W, 1.f))) return rc;
     }
     if ((rc = ld.sublayer(&l.sub1, sp.hc1_in, sp.hc1_out, sp.hc1_mix, sp.norm1))) return rc;
-    if (sp.ffn.ff && (rc = ld.gated(&l.gate_up, &l.down, &l.ffp, sp.ffn))) return rc;
-    if (sp.moe.experts && (rc = ld.experts(&l.moe, sp.moe))) return rc;
+    if (sp.moe.experts) rc = ld.experts(&l.moe, sp.moe, sp.ffn);
+    else if (sp.ffn.ff) rc = ld.gated(&l.gate_up, &l.down, &l.ffp, sp.ffn);
+    if (rc) return rc;
     if (sp.has_ffn()) {
       if ((rc = ld.sublayer(&l.sub2, sp.hc2_in, sp.hc2_out, sp.hc2_mix, sp.norm2))) return rc;
     }
@@ -356,7 +358,7 @@ static int build_distance_bias(hb_engine* e, LayeredLayer* l, const AttentionSpe
 }
 
 // Batch tiles of a mixture for `rows` rows of a step: tiles of about the rows an expert gets.
-static TcGroups moe_groups(const ExpertsSpec& x, int rows, bool tc) {
+static TcGroups moe_groups(const ExpertsSpec& x, bool shared, int rows, bool tc) {
   TcGroups g;
   const int64_t n = (int64_t)rows * x.top;
   g.groups = x.experts;
@@ -366,12 +368,31 @@ static TcGroups moe_groups(const ExpertsSpec& x, int rows, bool tc) {
   const double active = x.experts * (1.0 - std::pow(1.0 - 1.0 / x.experts, (double)n));
   const double tiles = active * std::max(1.0, std::ceil((double)n / std::max(1.0, active) / g.m_pad));
   g.likely_tiles = (int)std::max<int64_t>(1, std::min<int64_t>((int64_t)tiles, g.max_tiles));
+  if (shared) {
+    const int more = (rows + g.m_pad - 1) / g.m_pad;
+    g.max_tiles += more;
+    g.likely_tiles += more;
+  }
+  return g;
+}
+// The two products of a mixture: gate | up into rows of activations, and from there back to the width.
+static TcGroups up_groups(TcGroups g, const LayeredExperts& w, const GatedAct& shared_act) {
+  g.ldx = w.gate_up.K; g.ldy = w.ld();
+  if (w.shared_ffp) {
+    g.shared_w = w.shared_gate_up.w; g.shared_n = w.shared_gate_up.N; g.shared_k = w.shared_gate_up.K;
+    g.shared_act = shared_act;
+  }
+  return g;
+}
+static TcGroups down_groups(TcGroups g, const LayeredExperts& w) {
+  g.ldx = w.ld(); g.ldy = w.down.N;
+  if (w.shared_ffp) { g.shared_w = w.shared_down.w; g.shared_n = w.shared_down.N; g.shared_k = w.shared_down.K; }
   return g;
 }
 
-static MoeRouting moe_args(const LayeredModel* m, const ExpertsSpec& x, const TcGroups& g) {
+static MoeRouting moe_args(const LayeredModel* m, const ExpertsSpec& x, bool shared, const TcGroups& g) {
   MoeRouting r;
-  r.experts = x.experts; r.top = x.top;
+  r.experts = x.experts; r.top = x.top; r.shared = shared ? 1 : 0;
   r.m_pad = g.m_pad; r.max_tiles = g.max_tiles;
   r.ids = m->moe_ids; r.rank = m->moe_rank; r.place = m->moe_place; r.weight = m->moe_weight;
   r.count = m->moe_count; r.first = m->moe_first; r.tile_group = m->moe_tiles;
@@ -402,7 +423,7 @@ static int issue_attention(hb_engine* e, const SpanAttention& a, const LayeredSt
   const int64_t blocks = std::min<int64_t>(longest / HB_BLOCK_SIZE + 2, a.max_blocks), units = (int64_t)s.n_token_rows * a.kv_heads;
   int64_t splits = units < kSplitUnits / 2 ? std::min((kSplitUnits + units - 1) / units, (blocks + 15) / 16) : 1;
   splits = std::max<int64_t>(1, std::min<int64_t>(splits, 16));
-  if (splits > 1) ++e->last_launches;
+  if (splits > 8) ++e->last_launches;  // more than a cluster sums up
   return span_attention_tokens(st, a, rows, s.n_token_rows, (int)splits, m->attn_part);
 }
 
@@ -464,10 +485,10 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
     if (const ExpertsSpec& x = s.layers[i].moe; x.experts) {
       if (x.experts > kMoeMaxExperts) return fail(HB_ERR_INVALID_ARG, "%d experts (at most %d)", x.experts, kMoeMaxExperts);
       max_experts = std::max<int64_t>(max_experts, x.experts);
-      max_top = std::max<int64_t>(max_top, x.top);
-      max_eff = std::max(max_eff, l.moe.ffp);
-      for (int64_t M = 16; M <= R; M += 16) {
-        const TcGroups g = moe_groups(x, (int)M, e->use_tc);
+      max_top = std::max<int64_t>(max_top, x.top + 1);
+      max_eff = std::max(max_eff, l.moe.ld());
+      for (int64_t M = 1; M <= R; M = M < 16 ? M * 2 : M + 16) {
+        const TcGroups g = moe_groups(x, l.moe.shared_ffp > 0, (int)M, e->use_tc);
         max_tiles = std::max<int64_t>(max_tiles, g.max_tiles);
         m->moe_places = std::max<int64_t>(m->moe_places, (int64_t)g.max_tiles * g.m_pad);
       }
@@ -516,7 +537,7 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
     if ((rc = dev_alloc(e, (void**)&m->moe_place, picks, true))) return rc;
     if ((rc = dev_alloc(e, (void**)&m->moe_weight, picks, true))) return rc;
     if ((rc = dev_alloc(e, (void**)&m->moe_count, (size_t)(max_experts + 1) * 4, true))) return rc;
-    if ((rc = dev_alloc(e, (void**)&m->moe_first, (size_t)max_experts * 4, true))) return rc;
+    if ((rc = dev_alloc(e, (void**)&m->moe_first, (size_t)(max_experts + 1) * 4, true))) return rc;
     if ((rc = dev_alloc(e, (void**)&m->moe_tiles, (size_t)max_tiles * 4, true))) return rc;
   }
   if ((rc = dev_alloc(e, &m->hf, (size_t)LR * m->Hp * es, true))) return rc;
@@ -541,7 +562,14 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
 // ------------------------------------------------------------------------------- step
 // Matrix products are planned for a bucket of rows, so that steps of similar size share plans;
 // the rows above the step's own are scratch.
-static int row_bucket(int rows) { return (int)(rows <= 256 ? pad_to(rows, 16) : pad_to(rows, 128)); }
+static int row_bucket(int rows) {
+  if (rows <= 16) {  // few rows choose few experts: how many decides how their products are cut
+    int b = 1;
+    while (b < rows) b *= 2;
+    return b;
+  }
+  return (int)(rows <= 256 ? pad_to(rows, 16) : pad_to(rows, 128));
+}
 
 static int layered_plans(hb_engine* e, int rows, LayeredPlans** out) {
   LayeredModel* m = e->lm.get();
@@ -569,13 +597,14 @@ static int layered_plans(hb_engine* e, int rows, LayeredPlans** out) {
     if ((rc = plan(&p.down[i], m->act, l.down, kEpiStore, true))) return rc;
     const ExpertsSpec& x = m->spec.layers[i].moe;
     if (!x.experts) continue;
-    const TcGroups g = moe_groups(x, M, true);
+    const TcGroups g = moe_groups(x, l.moe.shared_ffp > 0, M, true);
+    const TcGroups up = up_groups(g, l.moe, m->spec.layers[i].ffn.act), down = down_groups(g, l.moe);
     if ((int64_t)g.max_tiles * g.m_pad > m->moe_places) return fail(HB_ERR_INVALID_ARG, "experts of %d rows need more places", M);
     if ((rc = gemm_tc_plan(&p.moe_gate_up[i], m->moe_x, l.moe.gate_up.w, m->moe_places, l.moe.gate_up.N, l.moe.gate_up.K,
-                           kEpiSwiGLU, false, e->device, 0, &g))) return rc;
+                           kEpiSwiGLU, false, e->device, 0, &up))) return rc;
     p.moe_gate_up[i].act = x.act;
     if ((rc = gemm_tc_plan(&p.moe_down[i], m->moe_act, l.moe.down.w, m->moe_places, l.moe.down.N, l.moe.down.K, kEpiStore, false,
-                           e->device, 0, &g))) return rc;
+                           e->device, 0, &down))) return rc;
   }
   if ((rc = ensure_gemm_workspace(e, ws))) return rc;
   *out = &m->plans.emplace(M, std::move(p)).first->second;
@@ -693,27 +722,31 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
   auto grouped = [&](const std::vector<TcGemmPlan>* plans, size_t i, void* Y, const void* X, const LayeredLinear& w,
                      const TcGroups& g) -> int {
     ++e->last_launches;
-    if (e->use_tc) return gemm_tc_run((*plans)[i], st, Y, (*plans)[i].N, e->d_gemm_ws, e->d_err, nullptr, m->moe_tiles);
+    if (e->use_tc) return gemm_tc_run((*plans)[i], st, Y, (*plans)[i].ldy, e->d_gemm_ws, e->d_err, nullptr, m->moe_tiles);
     return gemm_simt_grouped(st, Y, X, w.w, w.N, w.K, e->dtype, false, g, m->moe_tiles);
   };
   // the experts' outputs of every row, side by side in moe_y
-  auto experts = [&](size_t i, const ExpertsSpec& x, const LayeredExperts& w) -> int {
-    const TcGroups g = moe_groups(x, e->use_tc ? row_bucket((int)rows) : (int)rows, e->use_tc);
-    const MoeRouting r = moe_args(m, x, g);
+  auto experts = [&](size_t i, const ExpertsSpec& x, const LayeredExperts& w, const GatedAct& shared_act) -> int {
+    const bool shared = w.shared_ffp > 0;
+    const TcGroups g = moe_groups(x, shared, e->use_tc ? row_bucket((int)rows) : (int)rows, e->use_tc);
+    const TcGroups up = up_groups(g, w, shared_act), down = down_groups(g, w);
+    const MoeRouting r = moe_args(m, x, shared, g);
     prof_mark(e, kCatRouting);
     if ((rc = moe_route_top(st, r, m->h, m->Hp, w.router, w.router_bias, rows, W, e->dtype))) return rc;
     if ((rc = moe_gather(st, r, m->moe_x, m->h, m->Hp, rows, e->dtype))) return rc;
     e->last_launches += 2;
     prof_mark(e, kCatExpertsUp);
     if (e->use_tc) {
-      if ((rc = grouped(&pl->moe_gate_up, i, m->moe_act, m->moe_x, w.gate_up, g))) return rc;
+      if ((rc = grouped(&pl->moe_gate_up, i, m->moe_act, m->moe_x, w.gate_up, up))) return rc;
     } else {
-      if ((rc = grouped(nullptr, i, m->moe_gu, m->moe_x, w.gate_up, g))) return rc;
-      if ((rc = gated_act(st, m->moe_act, m->moe_gu, (int64_t)g.max_tiles * g.m_pad, w.ffp, x.act, e->dtype))) return rc;
+      TcGroups raw = up;
+      raw.ldy = 2 * w.ld();
+      if ((rc = grouped(nullptr, i, m->moe_gu, m->moe_x, w.gate_up, raw))) return rc;
+      if ((rc = gated_act_grouped(st, m->moe_act, w.ld(), m->moe_gu, 2 * w.ld(), w.ffp, x.act, e->dtype, up, m->moe_tiles))) return rc;
       ++e->last_launches;
     }
     prof_mark(e, kCatExpertsDown);
-    return grouped(pl ? &pl->moe_down : nullptr, i, m->moe_y, m->moe_act, w.down, g);
+    return grouped(pl ? &pl->moe_down : nullptr, i, m->moe_y, m->moe_act, w.down, down);
   };
   auto at = [&](void* p, int64_t elements) { return (void*)((uint8_t*)p + (size_t)elements * es); };
 
@@ -781,10 +814,10 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
     next = i + 1 < m->layers.size() ? &m->layers[i + 1].sub1 : nullptr;
     StreamMix fed{};
     if (lsp.moe.experts) {
-      if ((rc = experts(i, lsp.moe, l.moe))) return rc;
-      fed.expert_y = m->moe_y; fed.expert_place = m->moe_place; fed.expert_weight = m->moe_weight; fed.top = lsp.moe.top;
-    }
-    if (lsp.ffn.ff) {
+      if ((rc = experts(i, lsp.moe, l.moe, lsp.ffn.act))) return rc;
+      fed.expert_y = m->moe_y; fed.expert_place = m->moe_place; fed.expert_weight = m->moe_weight;
+      fed.top = lsp.moe.top + (l.moe.shared_ffp ? 1 : 0);
+    } else {
       prof_mark(e, kCatGemmGateUp);
       if (e->use_tc) {
         if ((rc = gemm(&pl->gate_up, i, m->act, m->h, l.gate_up, false))) return rc;
@@ -796,7 +829,7 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
       prof_mark(e, kCatGemmDown);
       if ((rc = gemm(pl ? &pl->down : nullptr, i, m->y1, m->act, l.down, true))) return rc;
     }
-    if ((rc = boundary(l.sub2, lsp.ffn.ff ? m->y1 : nullptr, false, fed))) return rc;
+    if ((rc = boundary(l.sub2, lsp.moe.experts ? nullptr : m->y1, false, fed))) return rc;
   }
   if (s.want) {
     prof_mark(e, kCatNorm);
@@ -839,7 +872,9 @@ static double layered_step_bytes(const hb_engine* e, const int32_t* ctx_lens, in
     w += n * (s.layers[i].has_ffn() ? 2.0 : 1.0) * 2.0 * s.streams * s.width * 4.0;
     if (const ExpertsSpec& x = s.layers[i].moe; x.experts)  // the experts a random batch chooses
       w += x.experts * (1.0 - std::pow(1.0 - 1.0 / x.experts, n * x.top)) *
-               ((double)l.moe.gate_up.N * l.moe.gate_up.K + (double)l.moe.down.N * l.moe.down.K) * es + (double)x.experts * s.width * es;
+               ((double)l.moe.gate_up.N * l.moe.gate_up.K + (double)l.moe.down.N * l.moe.down.K) * es +
+           ((double)x.experts * s.width + (double)l.moe.shared_gate_up.N * l.moe.shared_gate_up.K +
+            (double)l.moe.shared_down.N * l.moe.shared_down.K) * es;
   }
   return w;
 }
@@ -859,7 +894,8 @@ static double layered_gemm_bytes(const hb_engine* e, int64_t rows) {
       const double picks = b * x.top, active = x.experts * (1.0 - std::pow(1.0 - 1.0 / x.experts, picks));
       const LayeredExperts& w = l.moe;
       t += active * ((double)w.gate_up.N * w.gate_up.K + (double)w.down.N * w.down.K) * es +
-           picks * ((double)w.gate_up.K + 2.0 * w.ffp + (double)w.down.N) * es;
+           picks * ((double)w.gate_up.K + 2.0 * w.ffp + (double)w.down.N) * es +
+           lin(w.shared_gate_up, (double)w.shared_ffp, es) + lin(w.shared_down, (double)w.shared_down.N, es);
     }
   }
   return t;

@@ -93,7 +93,7 @@ struct LayerSpec {
   MixerSpec mixer;
   std::string norm1, norm2;
   std::string hc1_in, hc1_out, hc1_mix, hc2_in, hc2_out, hc2_mix;  // empty: one plain residual stream
-  FeedForwardSpec ffn;                       // the layer's feed-forward, or the shared expert beside `moe`
+  FeedForwardSpec ffn;                       // the layer's feed-forward, or what every token takes beside `moe`
   ExpertsSpec moe;
   bool has_ffn() const { return ffn.ff > 0 || moe.experts > 0; }
 };
@@ -127,9 +127,11 @@ struct SublayerMix {        // how a sublayer's output goes back into the stream
   float* norm = nullptr;    // [width]
 };
 
-struct LayeredExperts {     // experts' matrices one after another
+struct LayeredExperts {     // experts' matrices one after another; the expert every token passes through
   LayeredLinear gate_up, down;   // one expert's [2 * ffp, K] and [N, ffp]
-  int64_t ffp = 0;
+  LayeredLinear shared_gate_up, shared_down;
+  int64_t ffp = 0, shared_ffp = 0;
+  int64_t ld() const { return ffp > shared_ffp ? ffp : shared_ffp; }  // row stride of the activations
   void* router = nullptr;        // [experts, width] engine dtype
   float* router_bias = nullptr;  // [experts]
 };
@@ -202,8 +204,8 @@ struct LayeredModel {
   // mixture of experts: what the router decided, the rows of every expert side by side
   void *moe_x = nullptr, *moe_act = nullptr, *moe_y = nullptr;  // [places, Hp], [places, ffp], [places, Hp]
   void* moe_gu = nullptr;                    // fp32 engines: gate | up before the activation
-  int32_t *moe_ids = nullptr, *moe_rank = nullptr, *moe_place = nullptr;  // [rows, top]
-  float* moe_weight = nullptr;               // [rows, top]
+  int32_t *moe_ids = nullptr, *moe_rank = nullptr, *moe_place = nullptr;  // [rows, picks]
+  float* moe_weight = nullptr;               // [rows, picks]
   int64_t moe_places = 0;
   int32_t *moe_count = nullptr, *moe_first = nullptr, *moe_tiles = nullptr;
   int max_segs = 0, max_chunks = 0;

@@ -154,7 +154,7 @@ int hb_attention_prepare(void* stream, const hb_attention_prep_args* p, int64_t 
 
 static hb::MoeRouting routing_of(const hb_moe_routing* p) {
   hb::MoeRouting m;
-  m.experts = p->experts; m.top = p->top; m.m_pad = p->m_pad; m.max_tiles = p->max_tiles;
+  m.experts = p->experts; m.top = p->top; m.shared = p->shared ? 1 : 0; m.m_pad = p->m_pad; m.max_tiles = p->max_tiles;
   m.ids = p->ids; m.rank = p->rank; m.place = p->place; m.weight = p->weight;
   m.count = p->count; m.first = p->first; m.tile_group = p->tile_group;
   return m;
@@ -165,7 +165,8 @@ int hb_moe_route_top(void* stream, const hb_moe_routing* m, const void* h, int64
   HB_CHECK_ARG(m && h && router && bias && m->ids && m->rank && m->weight && m->count && m->first && m->tile_group,
                "hb_moe_route_top: null argument");
   HB_CHECK_ARG(rows >= 0 && width > 0 && m->m_pad > 0 &&
-               m->max_tiles >= (rows * m->top < m->experts ? rows * m->top : m->experts) + rows * m->top / m->m_pad,
+               m->max_tiles >= (rows * m->top < m->experts ? rows * m->top : m->experts) + rows * m->top / m->m_pad +
+                                   (m->shared ? (rows + m->m_pad - 1) / m->m_pad : 0),
                "hb_moe_route_top: bad shape");
   return hb::moe_route_top((cudaStream_t)stream, routing_of(m), h, ld_h, router, bias, rows, width, dtype);
 }
@@ -187,26 +188,50 @@ int hb_gated_act(void* stream, void* out, const void* gate_up, int64_t M, int64_
   return hb::gated_act((cudaStream_t)stream, out, gate_up, M, inter, act_of(act), dtype);
 }
 
-int hb_gemm_grouped(void* stream, void* Y, const void* X, const void* W, int groups, int64_t N, int64_t K, int m_pad,
-                    int max_tiles, int likely_tiles, const int32_t* tile_group, int out_f32,
-                    const hb_gated_act_spec* gated, hb_dtype dtype) {
-  HB_CHECK_ARG(Y && X && W && tile_group && groups > 0 && N > 0 && K > 0 && m_pad > 0 && max_tiles > 0 && likely_tiles > 0,
-               "hb_gemm_grouped: bad argument");
+static hb::TcGroups groups_of(const hb_grouped_gemm* p) {
   hb::TcGroups g;
-  g.groups = groups; g.m_pad = m_pad; g.max_tiles = max_tiles; g.likely_tiles = likely_tiles;
-  const int64_t M = (int64_t)max_tiles * m_pad;
+  g.groups = p->groups; g.m_pad = p->m_pad; g.max_tiles = p->max_tiles; g.likely_tiles = p->likely_tiles;
+  g.ldx = p->ldx; g.ldy = p->ldy;
+  g.shared_w = p->shared_w; g.shared_n = p->shared_n; g.shared_k = p->shared_k;
+  if (p->shared_w) g.shared_act = act_of(&p->shared_act);
+  return g;
+}
+
+static int check_grouped(const hb_grouped_gemm* p) {
+  HB_CHECK_ARG(p && p->tile_group && p->groups > 0 && p->N > 0 && p->K > 0 && p->m_pad > 0 && p->max_tiles > 0 &&
+               p->likely_tiles > 0 && p->ldx >= p->K && (!p->shared_w || (p->shared_n > 0 && p->shared_k > 0 && p->ldx >= p->shared_k)),
+               "grouped gemm: bad argument");
+  return HB_OK;
+}
+
+int hb_gemm_grouped(void* stream, void* Y, const void* X, const void* W, const hb_grouped_gemm* p, hb_dtype dtype) {
+  int rc = check_grouped(p);
+  if (rc) return rc;
+  const int64_t wide = p->shared_n > p->N ? p->shared_n : p->N;
+  HB_CHECK_ARG(Y && X && W && p->ldy >= (p->gated ? wide / 2 : wide), "hb_gemm_grouped: bad output");
+  const hb::TcGroups g = groups_of(p);
+  const int64_t M = (int64_t)p->max_tiles * p->m_pad;
   auto st = (cudaStream_t)stream;
-  if (hb::gemm_tc_supported(M, N, K, dtype) && m_pad % 16 == 0) {
+  if (hb::gemm_tc_supported(M, p->N, p->K, dtype) && p->m_pad % 16 == 0) {
     int dev = 0;
     HB_CUDA_CHECK(cudaGetDevice(&dev));
     hb::TcGemmPlan plan;
-    int rc = hb::gemm_tc_plan(&plan, X, W, M, N, K, gated ? hb::kEpiSwiGLU : hb::kEpiStore, out_f32 != 0, dev, 0, &g);
+    rc = hb::gemm_tc_plan(&plan, X, W, M, p->N, p->K, p->gated ? hb::kEpiSwiGLU : hb::kEpiStore, p->out_f32 != 0, dev, 0, &g);
     if (rc) return rc;
-    if (gated) plan.act = act_of(gated);
-    return hb::gemm_tc_run(plan, st, Y, plan.N, nullptr, nullptr, nullptr, tile_group);
+    if (p->gated) plan.act = act_of(&p->act);
+    return hb::gemm_tc_run(plan, st, Y, p->ldy, nullptr, nullptr, nullptr, p->tile_group);
   }
-  HB_CHECK_ARG(!gated, "hb_gemm_grouped: the gated form runs on tensor cores (bf16, K %% 8 == 0)");
-  return hb::gemm_simt_grouped(st, Y, X, W, N, K, dtype, out_f32 != 0, g, tile_group);
+  HB_CHECK_ARG(!p->gated, "hb_gemm_grouped: the gated form runs on tensor cores (bf16, K %% 8 == 0)");
+  return hb::gemm_simt_grouped(st, Y, X, W, p->N, p->K, dtype, p->out_f32 != 0, g, p->tile_group);
+}
+
+int hb_gated_act_grouped(void* stream, void* out, const void* gate_up, int64_t ld_gu, const hb_grouped_gemm* p, hb_dtype dtype) {
+  int rc = check_grouped(p);
+  if (rc) return rc;
+  HB_CHECK_ARG(out && gate_up && ld_gu >= p->N && ld_gu >= p->shared_n && p->ldy >= p->N / 2 && p->ldy >= p->shared_n / 2,
+               "hb_gated_act_grouped: bad argument");
+  return hb::gated_act_grouped((cudaStream_t)stream, out, p->ldy, gate_up, ld_gu, p->N / 2, act_of(&p->act), dtype, groups_of(p),
+                               p->tile_group);
 }
 
 int hb_streams_final(void* stream, void* h, const float* x, const int32_t* want, const float* norm, int64_t n_want,

@@ -131,12 +131,14 @@ int expand_distance_bias(cudaStream_t st, float* out, const float* rel, const in
 constexpr int kMoeMaxExperts = 1024;
 struct MoeRouting {
   int experts = 0, top = 0;
+  int shared = 0;                      // 1: every row also goes to the further group (TcGroups), with weight 1
   int m_pad = 0, max_tiles = 0;        // TcGroups
-  int32_t *ids = nullptr, *rank = nullptr, *place = nullptr;  // [rows, top]
-  float* weight = nullptr;             // [rows, top]
+  int32_t *ids = nullptr, *rank = nullptr, *place = nullptr;  // [rows, picks()]
+  float* weight = nullptr;             // [rows, picks()]
   int32_t* count = nullptr;            // [experts + 1], zero between calls
-  int32_t* first = nullptr;            // [experts] first place of an expert
+  int32_t* first = nullptr;            // [experts + shared] first place of an expert
   int32_t* tile_group = nullptr;       // [max_tiles]
+  __host__ __device__ __forceinline__ int picks() const { return top + shared; }
 };
 // Router logits h . router^T + bias in fp32; the `top` largest per row (the lower expert among
 // equals), their softmax as weights, every chosen (row, expert) a rank among the expert's rows, and

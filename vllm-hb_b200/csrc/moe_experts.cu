@@ -71,8 +71,10 @@ moe_route_top_kernel(const MoeRouting m, const T* __restrict__ h, int64_t ld_h, 
   // one warp per row: the largest logit `top` times, the lower expert among equals
   for (int r = warp; r < nr; r += kRouteWarps) {
     float* z = s_logit + r * E;
-    const int64_t at = (row0 + r) * m.top;
+    const int64_t at = (row0 + r) * m.picks();
     float first = 0.f, sum = 0.f;
+    int mine = 0;        // lane k keeps choice k (of every 32) and its unscaled weight
+    float mine_p = 0.f;
     for (int k = 0; k < m.top; ++k) {
       float best = -INFINITY;
       int who = E;
@@ -90,15 +92,28 @@ moe_route_top_kernel(const MoeRouting m, const T* __restrict__ h, int64_t ld_h, 
       if (k == 0) first = best;
       const float p = expf(best - first);
       sum += p;
-      if (lane == 0) {
-        z[e] = __int_as_float(0x7fc00000);  // taken
-        m.ids[at + k] = e;
-        m.weight[at + k] = p;
-        m.rank[at + k] = atomicAdd(m.count + e, 1);
+      if (lane == 0) z[e] = __int_as_float(0x7fc00000);  // taken
+      if (lane == (k & 31)) {
+        mine = e;
+        mine_p = p;
       }
       __syncwarp();
+      if ((k & 31) == 31 || k == m.top - 1) {
+        const int at_k = (k & ~31) + lane;
+        if (at_k <= k) {
+          m.ids[at + at_k] = mine;
+          m.weight[at + at_k] = mine_p;
+          m.rank[at + at_k] = atomicAdd(m.count + mine, 1);
+        }
+      }
     }
-    for (int k = lane; k < m.top; k += 32) m.weight[at + k] /= sum;
+    __syncwarp();
+    for (int k = lane; k < m.top; k += 32) m.weight[at + k] /= sum;  // written by this lane
+    if (m.shared && lane == 0) {
+      m.ids[at + m.top] = E;
+      m.weight[at + m.top] = 1.f;
+      m.rank[at + m.top] = (int)(row0 + r);
+    }
   }
   // the last CTA: every expert's tiles
   __threadfence();
@@ -125,6 +140,12 @@ moe_route_top_kernel(const MoeRouting m, const T* __restrict__ h, int64_t ld_h, 
     }
     tile += __shfl_sync(0xffffffffu, incl, 31);
   }
+  if (m.shared) {
+    const int n = (int)((rows + m.m_pad - 1) / m.m_pad);
+    if (lane == 0) m.first[E] = tile * m.m_pad;
+    for (int i = lane; i < n && tile + i < m.max_tiles; i += 32) m.tile_group[tile + i] = E;
+    tile += n;
+  }
   for (int i = tile + lane; i < m.max_tiles; i += 32) m.tile_group[i] = -1;
   if (lane == 0) m.count[E] = 0;
 }
@@ -133,21 +154,24 @@ template <typename T>
 __global__ void __launch_bounds__(kRouteThreads)
 moe_gather_kernel(const MoeRouting m, T* __restrict__ x, const T* __restrict__ h, int64_t ld) {
   pdl_trigger();
-  extern __shared__ int32_t s_place[];  // [top]
+  extern __shared__ int32_t s_place[];  // [picks]
   pdl_grid_wait();
   constexpr int N = Vec16<T>::N;
   const int64_t row = blockIdx.x, places = (int64_t)m.max_tiles * m.m_pad;
-  for (int k = threadIdx.x; k < m.top; k += kRouteThreads) {
-    const int64_t at = row * m.top + k;
+  const int picks = m.picks();
+  Vec16<T> a;
+  int64_t v = threadIdx.x;
+  if (v < ld / N) a.load(h + row * ld + v * N);  // on its way while the places are looked up
+  for (int k = threadIdx.x; k < picks; k += kRouteThreads) {
+    const int64_t at = row * picks + k;
     const int p = m.first[m.ids[at]] + m.rank[at];
     s_place[k] = p < places ? p : 0;  // never outside the buffer
     m.place[at] = s_place[k];
   }
   __syncthreads();
-  for (int64_t v = threadIdx.x; v < ld / N; v += kRouteThreads) {
-    Vec16<T> a;
-    a.load(h + row * ld + v * N);
-    for (int k = 0; k < m.top; ++k) a.store(x + (int64_t)s_place[k] * ld + v * N);
+  for (; v < ld / N; v += kRouteThreads) {
+    if (v >= kRouteThreads) a.load(h + row * ld + v * N);
+    for (int k = 0; k < picks; ++k) a.store(x + (int64_t)s_place[k] * ld + v * N);
   }
 }
 
@@ -162,12 +186,12 @@ int moe_route_top(cudaStream_t st, const MoeRouting& m, const void* h, int64_t l
                              (size_t)rb * m.experts * sizeof(float), st, m, (const T*)h, ld_h, (const T*)router, bias, rows, width));
     return HB_OK;
   };
-  const bool few = rows <= 512;
+  const bool few = rows <= 296;
   if (dtype == HB_F32)
-    return few ? launch(moe_route_top_kernel<float, 1>, 1, (float*)nullptr) : launch(moe_route_top_kernel<float, 8>, 8, (float*)nullptr);
+    return few ? launch(moe_route_top_kernel<float, 1>, 1, (float*)nullptr) : launch(moe_route_top_kernel<float, 4>, 4, (float*)nullptr);
   if (dtype == HB_BF16)
     return few ? launch(moe_route_top_kernel<__nv_bfloat16, 1>, 1, (__nv_bfloat16*)nullptr)
-               : launch(moe_route_top_kernel<__nv_bfloat16, 8>, 8, (__nv_bfloat16*)nullptr);
+               : launch(moe_route_top_kernel<__nv_bfloat16, 4>, 4, (__nv_bfloat16*)nullptr);
   return fail(HB_ERR_UNSUPPORTED_DTYPE, "moe_route_top runs in bf16 or f32");
 }
 
@@ -176,7 +200,7 @@ int moe_gather(cudaStream_t st, const MoeRouting& m, void* x, const void* h, int
   const int n = (int)(16 / dtype_size(dtype));
   if (ld % n || (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(h) & 15))
     return fail(HB_ERR_INVALID_ARG, "moe_gather: rows must be multiples of 16 bytes");
-  const size_t smem = (size_t)m.top * sizeof(int32_t);
+  const size_t smem = (size_t)m.picks() * sizeof(int32_t);
   if (dtype == HB_F32)
     HB_CUDA_CHECK(launch_pdl(moe_gather_kernel<float>, dim3((unsigned)rows), dim3(kRouteThreads), smem, st, m, (float*)x,
                              (const float*)h, ld));
@@ -189,22 +213,46 @@ int moe_gather(cudaStream_t st, const MoeRouting& m, void* x, const void* h, int
 }
 
 // ------------------------------------------------------------------- gated activation
+// tile_group (may be null): rows of negative groups are skipped, those of group `further` have inter2
+// and act2.
 template <typename T>
-__global__ void gated_act_kernel(T* __restrict__ out, const T* __restrict__ gu, int64_t inter, GatedAct act) {
+__global__ void gated_act_kernel(T* __restrict__ out, int64_t ld_out, const T* __restrict__ gu, int64_t ld_gu, int64_t inter,
+                                 GatedAct act, const int32_t* __restrict__ tile_group, int m_pad, int further, int64_t inter2,
+                                 GatedAct act2) {
   pdl_trigger();
   pdl_grid_wait();
   const int64_t row = blockIdx.x;
+  if (tile_group) {
+    const int group = tile_group[row / m_pad];
+    if (group < 0) return;
+    if (group == further) {
+      inter = inter2;
+      act = act2;
+    }
+  }
   for (int64_t i = threadIdx.x; i < inter; i += blockDim.x) {
-    const float g = fminf(to_f32<T>(gu[row * 2 * inter + i]), act.limit);
-    const float u = fminf(fmaxf(to_f32<T>(gu[row * 2 * inter + inter + i]), -act.limit), act.limit);
-    out[row * inter + i] = from_f32<T>(g / (1.f + expf(-act.slope * (g + act.cubic * g * g * g))) * (u + act.shift));
+    const float g = fminf(to_f32<T>(gu[row * ld_gu + i]), act.limit);
+    const float u = fminf(fmaxf(to_f32<T>(gu[row * ld_gu + inter + i]), -act.limit), act.limit);
+    out[row * ld_out + i] = from_f32<T>(g / (1.f + expf(-act.slope * (g + act.cubic * g * g * g))) * (u + act.shift));
   }
 }
 
 int gated_act(cudaStream_t st, void* out, const void* gate_up, int64_t M, int64_t inter, const GatedAct& act, hb_dtype dtype) {
   if (M == 0) return HB_OK;
   HB_DISPATCH_DTYPE(dtype, T, {
-    HB_CUDA_CHECK(launch_pdl(gated_act_kernel<T>, dim3((unsigned)M), dim3(256), 0, st, (T*)out, (const T*)gate_up, inter, act));
+    HB_CUDA_CHECK(launch_pdl(gated_act_kernel<T>, dim3((unsigned)M), dim3(256), 0, st, (T*)out, inter, (const T*)gate_up, 2 * inter,
+                             inter, act, nullptr, 1, -1, 0, act));
+  });
+  return HB_OK;
+}
+
+int gated_act_grouped(cudaStream_t st, void* out, int64_t ld_out, const void* gate_up, int64_t ld_gu, int64_t inter,
+                      const GatedAct& act, hb_dtype dtype, const TcGroups& g, const int32_t* tile_group) {
+  const int64_t rows = (int64_t)g.max_tiles * g.m_pad;
+  if (rows == 0) return HB_OK;
+  HB_DISPATCH_DTYPE(dtype, T, {
+    HB_CUDA_CHECK(launch_pdl(gated_act_kernel<T>, dim3((unsigned)rows), dim3(256), 0, st, (T*)out, ld_out, (const T*)gate_up,
+                             ld_gu, inter, act, tile_group, g.m_pad, g.shared_w ? g.groups : -1, g.shared_n / 2, g.shared_act));
   });
   return HB_OK;
 }

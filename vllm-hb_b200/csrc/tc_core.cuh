@@ -164,6 +164,11 @@ __device__ __forceinline__ void st_cluster_v4(uint32_t caddr, float a, float b, 
   asm volatile("st.shared::cluster.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(caddr), "f"(a), "f"(b), "f"(c), "f"(d)
                : "memory");
 }
+__device__ __forceinline__ float ld_cluster_f32(uint32_t caddr) {
+  float v;
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(caddr) : "memory");
+  return v;
+}
 // 16-byte store into a partner CTA's shared memory that reports its bytes to an mbarrier of
 // THAT CTA (both addresses already mapped into the partner's window): the receiver waits on
 // its own barrier and needs no cluster-wide barrier or fence to see the data.
