@@ -638,6 +638,9 @@ int span_attention_tile_positions(const SpanAttention& a, hb_dtype dtype) {
   if (!span_mma_ok(a, dtype) || R > kRows || tiles_smem(a, 1) > kSmemCap) return 0;
   return kRows / R;
 }
+int span_attention_tokens_slots(const SpanAttention& a) {
+  return 148 * (int)std::max<size_t>(1, std::min<size_t>(8, (size_t)227 * 1024 / (tokens_smem(a) + 1024)));
+}
 bool span_attention_tokens_supported(const SpanAttention& a, hb_dtype dtype) {
   return span_mma_ok(a, dtype) && a.heads / a.kv_heads <= 16 && tokens_smem(a) <= kSmemCap;
 }

@@ -194,10 +194,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
   TC_TRACE(tid == 0, 0);
   TC_LAUNCH_TRACE(0);
 
-  // work unit: blockIdx.x = tile * splits + split, blockIdx.y = batch tile
-  const int tile = blockIdx.x / p.splits;
+  // work unit: blockIdx.x = batch tile * splits + split, blockIdx.y = output tile: the batch tiles that
+  // meet the same weights run side by side, so weights leave HBM once and L2 serves the others
+  const int tile = blockIdx.y;
   const int split = p.cluster ? (int)cluster_ctarank() : blockIdx.x % p.splits;
-  const int m_tile = blockIdx.y;
+  const int m_tile = blockIdx.x / p.splits;
   int w_row = tile * kTileN;  // first weight row of the tile
   const CUtensorMap* w_map = &tm_w;
   int k_chunks = p.k_chunks, up_row_offset = p.up_row_offset;
@@ -208,7 +209,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
     pdl_wait();
     const int group = p.tile_group[m_tile];
     const bool further = group == p.further;
-    // uniform over the CTAs of a tile, so over every cluster
+    // uniform over the CTAs of a unit, so over every cluster
     if (group < 0 || tile >= (further ? p.n_tiles2 : p.n_tiles)) return;
     if (further) {
       w_map = &tm_h;
@@ -273,7 +274,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
     // deferred norm: scale of every batch row of this tile column, from the row sums the
     // producing GEMM left per 128-feature tile (fixed summation order)
     for (int i = tid - 64; i < p.m_pad; i += 64) {
-      const int m = blockIdx.y * p.m_pad + i;
+      const int m = m_tile * p.m_pad + i;
       float sc = 1.f;
       if (m < p.M) {
         // rows are padded to a multiple of four entries that stay zero: 128-bit loads,
@@ -306,9 +307,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
     }
   }
   if (warp >= 2 && p.post_scale) {
-    const int grp = (blockIdx.x / p.splits) / p.post_tiles_per_group;
+    const int grp = tile / p.post_tiles_per_group;
     for (int i = tid - 64; i < p.m_pad; i += 64) {
-      const int m = blockIdx.y * p.m_pad + i;
+      const int m = m_tile * p.m_pad + i;
       s_pscale[i] = m < p.M ? __ldcg(p.post_scale + (int64_t)m * p.post_groups + grp) : 0.f;
     }
   }
@@ -1224,7 +1225,7 @@ int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, voi
     p.rs_inv_n = 1.0f / link->n;
     p.rs_eps = link->eps;
   }
-  dim3 grid((unsigned)(std::max(pl.n_tiles, p.n_tiles2) * pl.splits), (unsigned)pl.m_tiles);
+  dim3 grid((unsigned)(pl.m_tiles * pl.splits), (unsigned)std::max(pl.n_tiles, p.n_tiles2));
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = grid;
   cfg.blockDim = dim3(kTcThreads);

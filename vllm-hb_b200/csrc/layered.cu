@@ -275,8 +275,8 @@ static size_t layered_layout(const hb_engine* e, LayeredStep* s) {
 
 // Segments of up to this many tokens go through the recurrence token by token.
 constexpr int kShortSegment = 8;
-// Decoded tokens: with fewer (row, kv head) units than this the keys are split over several CTAs.
-constexpr int kSplitUnits = 296;
+// Decoded tokens: with fewer (row, kv head) units than this the keys may be split over several CTAs.
+constexpr int kSplitUnits = 592;
 
 static SpanAttention span_args(const hb_engine* e, size_t i, const LayeredStep& s) {
   const LayeredModel* m = e->lm.get();
@@ -421,8 +421,10 @@ static int issue_attention(hb_engine* e, const SpanAttention& a, const LayeredSt
   const int64_t span = a.chunk > 0 ? a.chunk : a.window;
   const int64_t longest = span > 0 ? span + a.keep_first : a.max_blocks * HB_BLOCK_SIZE;
   const int64_t blocks = std::min<int64_t>(longest / HB_BLOCK_SIZE + 2, a.max_blocks), units = (int64_t)s.n_token_rows * a.kv_heads;
-  int64_t splits = units < kSplitUnits / 2 ? std::min((kSplitUnits + units - 1) / units, (blocks + 15) / 16) : 1;
+  // as many as are resident at once, every one with some blocks for each of its warps
+  int64_t splits = std::min<int64_t>(std::min(kSplitUnits, span_attention_tokens_slots(a)) / units, (blocks + 7) / 8);
   splits = std::max<int64_t>(1, std::min<int64_t>(splits, 16));
+  if (splits > 8 && blocks < 1024) splits = 8;  // what a cluster sums up
   if (splits > 8) ++e->last_launches;  // more than a cluster sums up
   return span_attention_tokens(st, a, rows, s.n_token_rows, (int)splits, m->attn_part);
 }

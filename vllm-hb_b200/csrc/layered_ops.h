@@ -97,6 +97,8 @@ int span_attention_rows(cudaStream_t st, const SpanAttention& a, const int32_t* 
 // tokens as single rows, their keys split over n_splits CTAs when the rows alone leave SMs idle
 // (`part`: n_rows * heads * n_splits * (vdim + 2) floats).
 int span_attention_tile_positions(const SpanAttention& a, hb_dtype dtype);
+// CTAs of the per-token kernel that are resident at once.
+int span_attention_tokens_slots(const SpanAttention& a);
 bool span_attention_tokens_supported(const SpanAttention& a, hb_dtype dtype);
 int span_attention_tiles(cudaStream_t st, const SpanAttention& a, const RowRange* tiles, int n_tiles);
 int span_attention_tokens(cudaStream_t st, const SpanAttention& a, const int32_t* rows, int n_rows, int n_splits, float* part);
