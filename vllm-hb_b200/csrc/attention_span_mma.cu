@@ -67,6 +67,12 @@ struct BlockCopy {
   int w, j, c, dj, dc;
   __device__ __forceinline__ BlockCopy(int width, int lane) : w(width / 8), j(lane / w), c(lane % w), dj(32 / w), dc(32 % w) {}
   __device__ __forceinline__ void operator()(uint32_t dst, int stride, const __nv_bfloat16* src, int64_t src_row) const {
+    if (dc == 0 && dj > 0) {  // whole rows at a time: a lane stays in its column
+      dst += j * stride + c * 16;
+      src += j * src_row + c * 8;
+      for (int jj = j; jj < kBS; jj += dj, dst += dj * stride, src += dj * src_row) cp_async_16(dst, src);
+      return;
+    }
     int jj = j, cc = c;
 #pragma unroll 4
     while (jj < kBS) {
@@ -79,14 +85,15 @@ struct BlockCopy {
 };
 }  // namespace
 
-// NV: 16-column pairs of n-tiles, i.e. the value slice is at most 16 * NV wide.
-template <int NV, bool EXT>
+// NV: 16-column pairs of n-tiles, i.e. the value slice is at most 16 * NV wide.  FIX: keys and values
+// are 16 * NV wide exactly, known to the compiler.
+template <int NV, bool EXT, bool FIX>
 __global__ void __launch_bounds__(kThreads)
 span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ tiles, int stages) {
   extern __shared__ __align__(16) uint8_t smem[];
-  const int R = a.heads / a.kv_heads, D = a.dim, DP = pad16(D), KS = DP + 8;
+  const int R = a.heads / a.kv_heads, D = FIX ? 16 * NV : a.dim, DP = pad16(D), KS = DP + 8;
   const bool tied = EXT && a.key_scale != nullptr;      // one tile is keys and values
-  const int v0 = blockIdx.z * kSlice, VW = min(kSlice, a.vdim - v0), VP = pad16(VW), VS = tied ? KS : VP + 8;
+  const int v0 = FIX ? 0 : blockIdx.z * kSlice, VW = FIX ? 16 * NV : min(kSlice, a.vdim - v0), VP = pad16(VW), VS = tied ? KS : VP + 8;
   __nv_bfloat16* s_q = (__nv_bfloat16*)smem;           // [64][KS]
   __nv_bfloat16* s_k = s_q + kRows * KS;               // [stages][64][KS]
   __nv_bfloat16* s_v = tied ? s_k : s_k + stages * kKeys * KS;               // [stages][64][VS]
@@ -166,6 +173,7 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
       for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
       // lanes 0-7 / 8-15 / 16-23 / 24-31 address keys 0-7 k-low, 0-7 k-high, 8-15 k-low, 8-15 k-high
       const uint32_t k_addr = smem_u32(kt + ((lane & 7) + (lane >> 4) * 8) * KS + ((lane >> 3) & 1) * 8);
+#pragma unroll(FIX ? NV : 1)
       for (int ks = 0; ks < DP / 16; ++ks) {
         uint32_t qa[4];
         ldsm_x4(q_addr + ks * 32, qa[0], qa[1], qa[2], qa[3]);
@@ -315,14 +323,15 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
 // The products are turned over, so that the few query heads are the narrow MMA side:
 // S^T[16 keys, 8 NT heads] = K Q^T and O^T[values, heads] += V^T P^T (P transposed in registers).
 // MT: 16-column tiles of the value slice, NT: groups of 8 query heads.
-template <int MT, int NT, bool EXT>
+// FIX: keys and values are 16 * MT wide exactly, known to the compiler.
+template <int MT, int NT, bool EXT, bool FIX>
 __global__ void __launch_bounds__(kThreads)
 span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, int n_splits, int clustered,
                              float* __restrict__ part) {
   extern __shared__ __align__(16) uint8_t smem[];
-  const int R = a.heads / a.kv_heads, D = a.dim, DP = pad16(D), KS = DP + 8;
+  const int R = a.heads / a.kv_heads, D = FIX ? 16 * MT : a.dim, DP = pad16(D), KS = DP + 8;
   const bool tied = EXT && a.key_scale != nullptr;  // one tile is keys and values; their scales lie behind it
-  const int v0 = (int)(blockIdx.z / n_splits) * kSlice, VW = min(kSlice, a.vdim - v0), VP = pad16(VW), VS = VP + 8;
+  const int v0 = FIX ? 0 : (int)(blockIdx.z / n_splits) * kSlice, VW = FIX ? 16 * MT : min(kSlice, a.vdim - v0), VP = pad16(VW), VS = VP + 8;
   const int split = blockIdx.z % n_splits;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gi = lane >> 2, t = lane & 3, kvh = blockIdx.y;
   const int stage_elems = tied ? kBS * (KS + 2) : kBS * (KS + VS);
@@ -412,7 +421,7 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
     for (int n = 0; n < NT; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) s[n][0][e] = s[n][1][e] = 0.f;
-#pragma unroll 4
+#pragma unroll(FIX ? (MT + 1) / 2 : 4)
     for (int ks = 0; ks < DP / 16; ks += 2) {
       uint32_t k0[4], k1[4];
       ldsm_x4(base + k_off + ks * 32, k0[0], k0[1], k0[2], k0[3]);
@@ -664,7 +673,10 @@ int span_attention_tiles(cudaStream_t st, const SpanAttention& a, const RowRange
   };
   const int vw = std::min(a.vdim, kSlice);
   const bool ext = a.key_scale || a.dist_bias;
-#define HB_TILES(NV) return ext ? launch(span_attention_tiles_kernel<NV, true>) : launch(span_attention_tiles_kernel<NV, false>)
+#define HB_TILES(NV)                                                                                          \
+  return a.dim == 16 * NV && a.vdim == 16 * NV                                                                \
+             ? (ext ? launch(span_attention_tiles_kernel<NV, true, true>) : launch(span_attention_tiles_kernel<NV, false, true>)) \
+             : (ext ? launch(span_attention_tiles_kernel<NV, true, false>) : launch(span_attention_tiles_kernel<NV, false, false>))
   if (vw <= 64) HB_TILES(4);
   if (vw <= 128) HB_TILES(8);
   if (vw <= 192) HB_TILES(12);
@@ -706,13 +718,19 @@ int span_attention_tokens(cudaStream_t st, const SpanAttention& a, const int32_t
   int rc;
   const bool wide = a.heads / a.kv_heads > 8;
   const bool ext = a.key_scale || a.dist_bias;
-#define HB_TOKENS(MT)                                                                                                        \
-  rc = ext ? (wide ? launch(span_attention_tokens_kernel<MT, 2, true>) : launch(span_attention_tokens_kernel<MT, 1, true>)) \
-           : (wide ? launch(span_attention_tokens_kernel<MT, 2, false>) : launch(span_attention_tokens_kernel<MT, 1, false>))
+#define HB_TOKENS_OF(MT, FIX)                                                                                      \
+  rc = ext ? (wide ? launch(span_attention_tokens_kernel<MT, 2, true, FIX>) : launch(span_attention_tokens_kernel<MT, 1, true, FIX>)) \
+           : (wide ? launch(span_attention_tokens_kernel<MT, 2, false, FIX>) : launch(span_attention_tokens_kernel<MT, 1, false, FIX>))
+#define HB_TOKENS(MT)                                            \
+  do {                                                           \
+    if (a.dim == 16 * MT && a.vdim == 16 * MT) HB_TOKENS_OF(MT, true); \
+    else HB_TOKENS_OF(MT, false);                                \
+  } while (0)
   if (vw <= 64) HB_TOKENS(4);
   else if (vw <= 128) HB_TOKENS(8);
   else HB_TOKENS(16);
 #undef HB_TOKENS
+#undef HB_TOKENS_OF
   if (rc || n_splits == 1 || clustered) return rc;
   HB_CUDA_CHECK(launch_pdl(span_attention_merge_kernel, dim3((unsigned)n_rows, (unsigned)a.heads), dim3(kThreads), 0, st, a, rows,
                            n_splits, (const float*)part));
