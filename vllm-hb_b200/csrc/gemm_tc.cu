@@ -1004,6 +1004,16 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
     pl.splits = sp;
   } else {
     pl.splits = pick_cluster_splits(units, k_chunks, di.sm_count);
+    if (groups && n_acc == 1 && pl.splits == 1 && units < 2 * slots) {
+      // A little more than a wave of long units would leave most SMs idle for the rest: cut K where
+      // that fills the last wave better than the exchange costs (4096 x 7168, 8 experts, 256 picks:
+      // 155 -> 125 us; short K and wide tiles lose).
+      double best = 0;
+      for (int sp = 1; sp <= 4 && k_chunks / sp >= 16; sp *= 2) {
+        const double waves = (double)units * sp / slots, score = waves / std::ceil(waves) * (1.0 - 0.04 * sp);
+        if (score > best) { best = score; pl.splits = sp; }
+      }
+    }
   }
   // (Partner counts that are not powers of two, with shares of the batch rows that differ by
   // four rows, were built and measured to cover more SMs where 28 tiles x 4 partners leave 36 of
