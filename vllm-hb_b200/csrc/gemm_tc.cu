@@ -48,12 +48,12 @@ struct TcParams {
   int epilogue, out_f32;
   int64_t ldy;
   int up_row_offset;        // SwiGLU: first row of the up projection inside W
-  GatedAct act;             // activation of the pair; act_silu: the plain one
-  int act_silu;
+  GatedAct act;             // activation of the pair (GENERAL)
+  int m_fast;               // the batch tiles are the fast dimension of the grid
   const int32_t* tile_group;  // TcGroups: group of every batch tile (negative: no such tile)
   int group_rows;             // weight rows of one group
   int further;                // number of the further group (tm_h holds its weights), -1: none
-  int n_tiles2, k_chunks2, up_row_offset2, act_silu2;
+  int n_tiles2, k_chunks2, up_row_offset2;
   GatedAct act2;
   int cluster;              // split-K partners form a thread-block cluster of `splits` CTAs
   int tma_store;            // the output leaves through bulk tensor stores (tm_y is valid)
@@ -160,8 +160,9 @@ __device__ __forceinline__ void push_tile(const TcParams& p, const uint8_t* stag
 }
 
 // Gated activation of one output element (fast divide and exponential, as silu_f).
-__device__ __forceinline__ float gated_f(float g, float u, bool silu, const GatedAct& act) {
-  if (silu) return silu_f(g) * u;
+template <bool GENERAL>
+__device__ __forceinline__ float gated_f(float g, float u, const GatedAct& act) {
+  if (!GENERAL) return silu_f(g) * u;
   g = fminf(g, act.limit);
   u = fminf(fmaxf(u, -act.limit), act.limit);
   const float z = act.slope * fmaf(act.cubic * g * g, g, g);
@@ -170,6 +171,10 @@ __device__ __forceinline__ float gated_f(float g, float u, bool silu, const Gate
 }
 
 // ----------------------------------------------------------------------- kernel
+// GROUPS: rows sorted by group (TcGroups).  GENERAL: any GatedAct, else SiLU.  The instance without
+// either is the one decode steps of dense models run: whatever it does not need costs it registers
+// and time (2 % of an 8B step).
+template <bool GROUPS, bool GENERAL>
 __global__ void __launch_bounds__(kTcThreads, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x,
                const __grid_constant__ CUtensorMap tm_y, const __grid_constant__ CUtensorMap tm_h,
@@ -194,17 +199,19 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
   TC_TRACE(tid == 0, 0);
   TC_LAUNCH_TRACE(0);
 
-  // work unit: blockIdx.x = batch tile * splits + split, blockIdx.y = output tile: the batch tiles that
-  // meet the same weights run side by side, so weights leave HBM once and L2 serves the others
-  const int tile = blockIdx.y;
+  // work unit: blockIdx.x = output tile * splits + split for one batch tile.  With several (m_fast)
+  // blockIdx.x = batch tile * splits + split, blockIdx.y = output tile: the batch tiles that meet the
+  // same weights run side by side, so weights leave HBM once and L2 serves the others.
+  const bool m_fast = GROUPS || p.m_fast;
+  const int unit = blockIdx.x / p.splits;
+  const int tile = m_fast ? (int)blockIdx.y : unit;
   const int split = p.cluster ? (int)cluster_ctarank() : blockIdx.x % p.splits;
-  const int m_tile = blockIdx.x / p.splits;
+  const int m_tile = m_fast ? unit : (int)blockIdx.y;
   int w_row = tile * kTileN;  // first weight row of the tile
   const CUtensorMap* w_map = &tm_w;
   int k_chunks = p.k_chunks, up_row_offset = p.up_row_offset;
-  bool act_silu = p.act_silu != 0;
   GatedAct act = p.act;
-  if (p.tile_group) {
+  if (GROUPS) {
     // rows sorted by group: the previous kernels say whose weights this batch tile meets
     pdl_wait();
     const int group = p.tile_group[m_tile];
@@ -215,7 +222,6 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
       w_map = &tm_h;
       k_chunks = p.k_chunks2;
       up_row_offset = p.up_row_offset2;
-      act_silu = p.act_silu2 != 0;
       act = p.act2;
     } else {
       w_row += group * p.group_rows;
@@ -545,7 +551,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           }
         }
 #pragma unroll
-        for (int j = 0; j < 16; ++j) g[j] = swiglu ? gated_f(g[j], u[j], act_silu, act) : g[j];
+        for (int j = 0; j < 16; ++j) g[j] = swiglu ? gated_f<GENERAL>(g[j], u[j], act) : g[j];
         if (p.post_scale) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) g[j] *= s_pscale[c0 + j];
@@ -693,7 +699,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
             for (int j = 0; j < 16; ++j) u[j] *= s_rscale[g * 16 + j];
           }
 #pragma unroll
-          for (int j = 0; j < 16; ++j) v[j] = gated_f(v[j], u[j], act_silu, act);
+          for (int j = 0; j < 16; ++j) v[j] = gated_f<GENERAL>(v[j], u[j], act);
         }
         if (p.post_scale) {
 #pragma unroll
@@ -733,7 +739,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           float u[16];
           tmem_ld16(t_lane + p.m_pad + c0, u);
 #pragma unroll
-          for (int j = 0; j < 16; ++j) v[j] = gated_f(v[j], u[j], act_silu, act);
+          for (int j = 0; j < 16; ++j) v[j] = gated_f<GENERAL>(v[j], u[j], act);
         }
         if (n_glob < p.N) {
 #pragma unroll
@@ -790,7 +796,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           for (int j = 0; j < 8; ++j) {
             const int m = m0 + j;
             if (m < m_lim && n_glob < p.N) {
-              const float r = swiglu ? gated_f(g[j], u[j], act_silu, act) : g[j];
+              const float r = swiglu ? gated_f<GENERAL>(g[j], u[j], act) : g[j];
               if (p.out_f32) ((float*)p.Y)[(int64_t)(m_base + m) * p.ldy + n_glob] = r;
               else ((__nv_bfloat16*)p.Y)[(int64_t)(m_base + m) * p.ldy + n_glob] = __float2bfloat16_rn(r);
             }
@@ -1094,8 +1100,8 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
     std::lock_guard<std::mutex> lock(mu);
     if (cur >= 0 && cur < 64 && !dev_done[cur]) {
       // 227 KiB per CTA minus the kernel's static shared memory (barriers, flags, row scales)
-      HB_CUDA_CHECK(cudaFuncSetAttribute(gemm_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         224 * 1024));
+      for (auto* k : {gemm_tc_kernel<false, false>, gemm_tc_kernel<false, true>, gemm_tc_kernel<true, true>})
+        HB_CUDA_CHECK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024));
       dev_done[cur] = true;
     }
   }
@@ -1140,7 +1146,7 @@ int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, voi
   p.ldy = ldy;
   p.up_row_offset = (int)pl.N;
   p.act = pl.act;
-  p.act_silu = pl.act.silu() ? 1 : 0;
+  p.m_fast = pl.groups || pl.m_tiles > 1 ? 1 : 0;
   p.tile_group = tile_group;
   p.group_rows = pl.group_rows;
   p.further = pl.N2 ? pl.groups : -1;
@@ -1148,7 +1154,6 @@ int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, voi
   p.k_chunks2 = (int)((pl.K2 + kTileK - 1) / kTileK);
   p.up_row_offset2 = (int)pl.N2;
   p.act2 = pl.act2;
-  p.act_silu2 = pl.act2.silu() ? 1 : 0;
   p.Y = Y;
   // counters first (16-byte aligned block), partials after
   p.counters = (int*)workspace;
@@ -1235,7 +1240,8 @@ int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, voi
     p.rs_inv_n = 1.0f / link->n;
     p.rs_eps = link->eps;
   }
-  dim3 grid((unsigned)(pl.m_tiles * pl.splits), (unsigned)std::max(pl.n_tiles, p.n_tiles2));
+  const unsigned n_tiles = (unsigned)std::max(pl.n_tiles, p.n_tiles2), m_tiles = (unsigned)pl.m_tiles;
+  const dim3 grid((p.m_fast ? m_tiles : n_tiles) * (unsigned)pl.splits, p.m_fast ? n_tiles : m_tiles);
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = grid;
   cfg.blockDim = dim3(kTcThreads);
@@ -1258,7 +1264,9 @@ int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, voi
   }
   cfg.attrs = attr;
   cfg.numAttrs = na;
-  HB_CUDA_CHECK(cudaLaunchKernelEx(&cfg, gemm_tc_kernel, pl.tm_w, pl.tm_x, tm_y, tm_h, p));
+  auto* kernel = pl.groups ? gemm_tc_kernel<true, true>
+                           : pl.act.silu() ? gemm_tc_kernel<false, false> : gemm_tc_kernel<false, true>;
+  HB_CUDA_CHECK(cudaLaunchKernelEx(&cfg, kernel, pl.tm_w, pl.tm_x, tm_y, tm_h, p));
   return HB_OK;
 }
 
