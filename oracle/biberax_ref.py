@@ -144,11 +144,11 @@ def route(h, w_router, bias, top):
 
 def route_margin(h, w_router, bias, top):
     """How far the last chosen logit of every token lies above the first one left out, in units of
-    the spread of the logits (infinite when nothing is left out)."""
+    the spread of all logits (infinite when nothing is left out)."""
     z = np.sort(h @ w_router.T + bias, axis=1)[:, ::-1]
     if z.shape[1] == top:
         return np.full(len(z), np.inf)
-    return (z[:, top - 1] - z[:, top]) / np.maximum(z.std(axis=1), 1e-9)
+    return (z[:, top - 1] - z[:, top]) / max(float(z.std()), 1e-9)
 
 
 def moe_ffn(h, w, mlp):

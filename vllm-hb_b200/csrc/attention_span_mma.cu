@@ -106,7 +106,7 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
     for (int i = tid; i < stages * kKeys * VS / 8; i += kThreads)
       if (i % (VS / 8) * 8 >= VW) reinterpret_cast<uint4*>(s_v)[i] = make_uint4(0, 0, 0, 0);
   pdl_grid_wait();
-  const RowRange tile = tiles[blockIdx.x];
+  const RowRange tile = tiles[gridDim.x - 1 - blockIdx.x];  // later positions see more: they go first
   const int first_pos = a.pos[tile.row0], last_pos = first_pos + tile.n - 1;
   const BlockRuns runs = block_runs(first_pos, last_pos, a);
   const int32_t* table = a.tables + (int64_t)tile.seg * a.max_blocks;
@@ -648,7 +648,8 @@ int span_attention_tile_positions(const SpanAttention& a, hb_dtype dtype) {
   return kRows / R;
 }
 int span_attention_tokens_slots(const SpanAttention& a) {
-  return 148 * (int)std::max<size_t>(1, std::min<size_t>(8, (size_t)227 * 1024 / (tokens_smem(a) + 1024)));
+  constexpr int kSms = 148;
+  return kSms * (int)std::max<size_t>(1, std::min<size_t>(8, (size_t)227 * 1024 / (tokens_smem(a) + 1024)));
 }
 bool span_attention_tokens_supported(const SpanAttention& a, hb_dtype dtype) {
   return span_mma_ok(a, dtype) && a.heads / a.kv_heads <= 16 && tokens_smem(a) <= kSmemCap;
