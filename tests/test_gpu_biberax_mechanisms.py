@@ -88,7 +88,7 @@ class Paged:
     def forms(self):
         """Every way the kernels can be asked for the same rows."""
         yield "rows", self.run(rows=np.arange(self.n))
-        for splits in (2, 5):
+        for splits in (2, 5, 8, 12):
             yield f"{splits} splits", self.run(rows=np.arange(self.n), splits=splits)
         tp = self.tile_positions()
         for size in sorted({tp, max(1, tp // 2 - 1), min(2, tp)} if tp else ()):
