@@ -236,9 +236,11 @@ int hb_sample(void* stream, uint32_t* tokens, float* probs_workspace, const floa
  * (p / chunk == j / chunk); keys and values may differ in width.  Optional (NULL / 0: none):
  * dist_bias [heads, dist_len] is added to the scaled score by distance (the last entry also beyond
  * it); sink [heads] is the score of one more softmax member without a value; gate: the output is
- * multiplied by sigmoid(gate), row r, head h at gate + r*ld_gate + h*vdim (`dtype`);
- * key_scale [num_blocks*16]: the K pool holds the values too (v_cache unused, vdim == dim) and a key
- * is its value times the scale of its slot.
+ * multiplied by sigmoid(gate), row r, head h at gate + r*ld_gate + h*vdim (`dtype`); softcap: a scaled
+ * score s becomes softcap * tanh(s / softcap) (before the bias).
+ * v_cache NULL: the values are the first vdim channels of the keys; with key_scale [num_blocks*16] (and
+ * vdim == dim, v_cache unused) the K pool holds the values and a key is its value times the scale of its
+ * slot.
  * q row r, head h at q + r*ld_q + h*dim; out likewise with vdim; K pool [num_blocks, kv_heads, 16,
  * dim], V pool [num_blocks, kv_heads, 16, vdim]; softmax(scale * q.k) v, scores and weights in fp32.
  * tiles {segment, first row, rows, -}: up to hb_span_attention_tile_positions() consecutive
@@ -263,6 +265,7 @@ typedef struct hb_span_attention_args {
   const float* sink;
   const void* gate;
   int64_t ld_gate;
+  float softcap;
 } hb_span_attention_args;
 int hb_span_attention_tile_positions(const hb_span_attention_args* a, hb_dtype dtype);
 int hb_span_attention(void* stream, const hb_span_attention_args* a, const int32_t* tiles, int n_tiles, const int32_t* rows,
@@ -274,7 +277,8 @@ int hb_span_kv_write(void* stream, const hb_span_attention_args* a, const void* 
 /* From projection rows (queries, keys, values at column offsets of p) to queries in their place and
  * keys and values in their slots: biases [heads*dim], [kv_heads*dim] added; then either RMS norms
  * over all query and all key rows (weights q_norm, k_norm) or a rotation of the first 2*pairs
- * channels of every head, channel 2i with 2i+1, by position * rotation[i].  With key_scale the K pool
+ * channels of every head, channel 2i with 2i+1 (halves: channel i with i+pairs), by position *
+ * rotation[i], times rotation_gain (0: 1).  k_cache NULL: queries only.  With key_scale the K pool
  * takes the keys before their norm, key_scale[slot] the factor of the norm, and the queries are
  * multiplied by k_norm (hb_span_attention's key_scale).  fp32 inside. */
 typedef struct hb_attention_prep_args {
@@ -290,15 +294,48 @@ typedef struct hb_attention_prep_args {
   const double* rotation;
   int pairs;
   float* key_scale;
+  int halves;
+  float rotation_gain;
 } hb_attention_prep_args;
 int hb_attention_prepare(void* stream, const hb_attention_prep_args* a, int64_t rows, hb_dtype dtype);
 
+/* Attention over a latent that all heads share (hb_span_attention with kv_heads 1, dim = rank+rot_dim,
+ * vdim = rank and no V pool).  Row r of p holds at off_q the heads' queries [dim | rot_dim] and at off_c
+ * [latent of rank | key part of rot_dim].  The latent is RMS-normed (weight norm [rank]), the key part
+ * rotated (channel i with i+pairs), both go to the row's slot of k_cache [num_blocks, 16, rank+rot_dim];
+ * the queries' rotated parts go to q, head h at q + r*ld_q + h*(rank+rot_dim) + rank.  fp32 inside. */
+typedef struct hb_latent_prep_args {
+  const void* p;
+  int64_t ld;
+  int off_q, off_c, heads, dim, rot_dim, rank;
+  void* q;
+  int64_t ld_q;
+  const int32_t* positions;
+  const int64_t* slots;
+  void* k_cache;
+  int64_t num_blocks;
+  const float* norm;
+  float eps;
+  const double* rotation;
+  int pairs;
+  float rotation_gain;
+} hb_latent_prep_args;
+int hb_latent_prepare(void* stream, const hb_latent_prep_args* a, int64_t rows, hb_dtype dtype);
+/* One product per head: Y_h[M, N] = X_h . W_h^T with the heads' [N, K] matrices one after another in W,
+ * X_h = X + h*x_step (rows of ldx elements) and Y_h = Y + h*y_step (rows of ldy).  bf16 with K, N and all
+ * strides multiples of 8 on tensor cores. */
+int hb_gemm_heads(void* stream, void* Y, const void* X, const void* W, int64_t M, int64_t N, int64_t K, int heads, int64_t ldx,
+                  int64_t x_step, int64_t ldy, int64_t y_step, hb_dtype dtype);
+
 /* Mixture of experts, every expert on its own rows only.
- * hb_moe_route_top: logits h . router^T + bias [experts] in fp32, the `top` largest per row (ids,
+ * hb_moe_route_top: logits h . router^T + bias [experts] (NULL: none) in fp32, the `top` largest per row (ids,
  * the lower expert among equals), the softmax over them (weight), each choice's rank among the rows
  * of its expert, and batch tiles of m_pad places: expert e has tiles from place first[e] on,
  * tile_group[i] is the expert of tile i (-1: no such tile).  max_tiles >= min(experts, n) + n / m_pad
  * for n = rows * top.  count [experts + 1] is zero before and after.
+ * sigmoid: scores sigmoid(logit), the chosen ones over their sum as weights; groups > 1: only experts of
+ * the `keep` best of that many equal groups of neighbours are chosen, a group counting the sum of its
+ * two largest scores.
  * With `shared` every row has one pick more: group number `experts`, weight 1, tiles after all
  * others (ceil(rows / m_pad) of them, counted in max_tiles).
  * hb_moe_gather: row r of h (stride ld) to place[r,k] = first + rank in x.
@@ -311,6 +348,7 @@ typedef struct hb_moe_routing {
   float* weight;               /* [rows, top + shared] */
   int32_t *count, *first, *tile_group; /* [experts + 1], [experts + shared], [max_tiles] */
   int shared;
+  int sigmoid, groups, keep; /* groups 0: one */
 } hb_moe_routing;
 int hb_moe_route_top(void* stream, const hb_moe_routing* m, const void* h, int64_t ld_h, const void* router,
                      const float* bias, int64_t rows, int64_t width, hb_dtype dtype);
@@ -342,6 +380,10 @@ int hb_gated_act_grouped(void* stream, void* out, const void* gate_up, int64_t l
  * p holds q, k (heads*dim), v (heads*vdim) and, for a low-rank decay, rank columns, at the given
  * column offsets; q is scaled by q_scale, q, k and v pass through SiLU when silu_qkv.  Decay:
  * `decay` [heads], or (decay NULL) sigmoid(a2 . p[off_a1..] + a2_bias)^(1/tau) per key channel.
+ * Or (dt not NULL; row r, head h at dt + r*ld_dt + h, `dtype`) a selective state space: a step t =
+ * softplus(dt + dt_bias) per token and head, decay exp(-exp(a_log) t), keys scaled by t, and skip * v
+ * added to the output (dt_bias, a_log, skip [heads]); cum then takes rows*2*heads floats.  qk_heads > 0:
+ * q and k have that many heads, each serving heads / qk_heads neighbours.
  * segments {first row, rows, first position, state slot}: position 0 starts from a zero state.
  * `list`: segments that go token by token; `chunks` {segment, first row, rows <= 64, index} and
  * `long_segments` {segment, first chunk, chunks, -}: segments that go in chunks on tensor cores
@@ -360,11 +402,33 @@ typedef struct hb_linear_recurrence_args {
   float* o;     /* row r, head h at o + r*ld_o + h*vdim */
   int64_t ld_o;
   const int32_t* segments;
+  const void* dt;
+  int64_t ld_dt;
+  const float *dt_bias, *a_log, *skip;
+  int qk_heads;
 } hb_linear_recurrence_args;
 int hb_linear_recurrence_chunked(const hb_linear_recurrence_args* a, hb_dtype dtype);
 int hb_linear_recurrence(void* stream, const hb_linear_recurrence_args* a, const int32_t* list, int n_list,
                          const int32_t* chunks, int n_chunks, const int32_t* long_segments, int n_long, float* cum,
                          float* chunk_state, hb_dtype dtype);
+
+/* Causal convolution per channel: out = SiLU(bias + sum_j w[j] x[t - (taps-1) + j]) over the tokens of a
+ * sequence, zeros before its start; w [taps, channels] (taps <= 65).  Row r, channel c of the input at
+ * p + r*ld + off + c, of the output at out + r*ld_out + c.  The last taps-1 inputs of a sequence stay in
+ * its slot of state [slots, taps-1, channels] (`dtype`); position 0 starts from zeros.  Every segment is
+ * either in `list` (at most 64 tokens) or cut into `chunks` of 64 tokens. */
+typedef struct hb_short_conv_args {
+  const void* p;
+  int64_t ld;
+  int off, channels, taps;
+  const float *w, *bias;
+  void* out;
+  int64_t ld_out;
+  void* state;
+  const int32_t* segments;
+} hb_short_conv_args;
+int hb_short_conv(void* stream, const hb_short_conv_args* a, const int32_t* list, int n_list, const int32_t* chunks, int n_chunks,
+                  hb_dtype dtype);
 
 /* Several residual streams x [rows, streams, width] in fp32.
  * hb_streams_embed: every stream = embed[ids] + pos_table[positions]; h = rms(sum_s in[s] x_s) *
@@ -396,9 +460,10 @@ int hb_streams_mix_ex(void* stream, float* x, void* h, const float* y, const flo
 int hb_streams_final(void* stream, void* h, const float* x, const int32_t* want, const float* norm, int64_t n_want,
                      int streams, int64_t width, int64_t ld_h, float eps, hb_dtype dtype);
 /* out[r, g*size + i] = o / rms over group g * weight[i] * act(gate); the weight [size] is shared by the
- * groups; act: SiLU, or sigmoid when gate_silu is 0. */
+ * groups; act: SiLU with bit 0 of gate_mode, else sigmoid.  Bit 1: the product o * act(gate) is what is
+ * normed, and weight is [groups*size]. */
 int hb_gated_group_norm(void* stream, void* out, int64_t ld_out, const float* o, int64_t ld_o, const void* gate,
-                        int64_t ld_gate, const float* weight, int64_t rows, int groups, int size, int gate_silu, float eps,
+                        int64_t ld_gate, const float* weight, int64_t rows, int groups, int size, int gate_mode, float eps,
                         hb_dtype dtype);
 
 /* --------------------------------------------------------------- comm surface */
@@ -743,8 +808,8 @@ int hb_kv_swap_blocks(hb_engine* e, const int64_t* pairs, size_t n_pairs, int to
  * argmax / SwiGLU gate, 5 all-reduce, 6 o_proj, 7 gate|up projection, 8 down_proj,
  * 9 lm_head (6 and 8 include the fused all-reduce + residual + norm when that kernel
  * runs), 10 linear recurrence, 11 routing to experts, 12 / 13 the experts' gate|up and down
- * projections.  The step counts like any other decode step. */
-#define HB_PROFILE_KINDS 14
+ * projections, 14 latent attention's products per head, 15 convolutions.  The step counts like any other decode step. */
+#define HB_PROFILE_KINDS 16
 int hb_engine_profile_step(hb_engine* e, hb_seq* const* seqs, size_t B,
                            const uint32_t* last_tokens, uint32_t* next_tokens, float* ms_by_kind);
 /* The same for every step while on (hb_step, hb_forward, ...): the times of the last step. */

@@ -103,7 +103,7 @@ class SpanAttentionArgs(C.Structure):
         ("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("window", C.c_int),
         ("keep_first", C.c_int), ("scale", C.c_float),
         ("chunk", C.c_int), ("key_scale", C.c_void_p), ("dist_bias", C.c_void_p), ("dist_len", C.c_int),
-        ("sink", C.c_void_p), ("gate", C.c_void_p), ("ld_gate", C.c_int64),
+        ("sink", C.c_void_p), ("gate", C.c_void_p), ("ld_gate", C.c_int64), ("softcap", C.c_float),
     ]
 
 
@@ -114,7 +114,25 @@ class AttentionPrepArgs(C.Structure):
         ("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("positions", C.c_void_p),
         ("slots", C.c_void_p), ("k_cache", C.c_void_p), ("v_cache", C.c_void_p), ("num_blocks", C.c_int64),
         ("q_bias", C.c_void_p), ("k_bias", C.c_void_p), ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("eps", C.c_float),
-        ("rotation", C.c_void_p), ("pairs", C.c_int), ("key_scale", C.c_void_p),
+        ("rotation", C.c_void_p), ("pairs", C.c_int), ("key_scale", C.c_void_p), ("halves", C.c_int), ("rotation_gain", C.c_float),
+    ]
+
+
+class LatentPrepArgs(C.Structure):
+    """hb_latent_prep_args: a normed latent and a rotated key part to the cache, rotated parts of queries."""
+    _fields_ = [
+        ("p", C.c_void_p), ("ld", C.c_int64), ("off_q", C.c_int), ("off_c", C.c_int), ("heads", C.c_int), ("dim", C.c_int),
+        ("rot_dim", C.c_int), ("rank", C.c_int), ("q", C.c_void_p), ("ld_q", C.c_int64), ("positions", C.c_void_p),
+        ("slots", C.c_void_p), ("k_cache", C.c_void_p), ("num_blocks", C.c_int64), ("norm", C.c_void_p), ("eps", C.c_float),
+        ("rotation", C.c_void_p), ("pairs", C.c_int), ("rotation_gain", C.c_float),
+    ]
+
+
+class ShortConvArgs(C.Structure):
+    """hb_short_conv_args: causal convolution per channel with its state."""
+    _fields_ = [
+        ("p", C.c_void_p), ("ld", C.c_int64), ("off", C.c_int), ("channels", C.c_int), ("taps", C.c_int), ("w", C.c_void_p),
+        ("bias", C.c_void_p), ("out", C.c_void_p), ("ld_out", C.c_int64), ("state", C.c_void_p), ("segments", C.c_void_p),
     ]
 
 
@@ -123,7 +141,7 @@ class MoeRouting(C.Structure):
     _fields_ = [
         ("experts", C.c_int), ("top", C.c_int), ("m_pad", C.c_int), ("max_tiles", C.c_int), ("ids", C.c_void_p),
         ("rank", C.c_void_p), ("place", C.c_void_p), ("weight", C.c_void_p), ("count", C.c_void_p), ("first", C.c_void_p),
-        ("tile_group", C.c_void_p), ("shared", C.c_int),
+        ("tile_group", C.c_void_p), ("shared", C.c_int), ("sigmoid", C.c_int), ("groups", C.c_int), ("keep", C.c_int),
     ]
 
 
@@ -158,6 +176,8 @@ class LinearRecurrenceArgs(C.Structure):
         ("off_a1", C.c_int), ("heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("q_scale", C.c_float),
         ("silu_qkv", C.c_int), ("decay", C.c_void_p), ("a2", C.c_void_p), ("a2_bias", C.c_void_p), ("rank", C.c_int),
         ("tau", C.c_float), ("state", C.c_void_p), ("o", C.c_void_p), ("ld_o", C.c_int64), ("segments", C.c_void_p),
+        ("dt", C.c_void_p), ("ld_dt", C.c_int64), ("dt_bias", C.c_void_p), ("a_log", C.c_void_p), ("skip", C.c_void_p),
+        ("qk_heads", C.c_int),
     ]
 
 
@@ -189,6 +209,9 @@ _SIGS = {
     "hb_streams_mix": (_i, [_vp, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i, _i64, _i64, _f, _i]),
     "hb_streams_mix_ex": (_i, [_vp, _vp, _vp, _vp, _vp, _i64, _vp, _i64, _i, _i64, _i64, _f, _i]),
     "hb_attention_prepare": (_i, [_vp, _vp, _i64, _i]),
+    "hb_latent_prepare": (_i, [_vp, _vp, _i64, _i]),
+    "hb_gemm_heads": (_i, [_vp, _vp, _vp, _vp, _i64, _i64, _i64, _i, _i64, _i64, _i64, _i64, _i]),
+    "hb_short_conv": (_i, [_vp, _vp, _vp, _i, _vp, _i, _i]),
     "hb_moe_route_top": (_i, [_vp, _vp, _vp, _i64, _vp, _vp, _i64, _i64, _i]),
     "hb_moe_gather": (_i, [_vp, _vp, _vp, _vp, _i64, _i64, _i]),
     "hb_gated_act": (_i, [_vp, _vp, _vp, _i64, _i64, _vp, _i]),
@@ -1071,7 +1094,7 @@ class Engine:
 
     PROFILE_KINDS = ("gemm_qkv", "attention", "rope_kv", "norm", "other", "all_reduce",
                      "gemm_o_proj", "gemm_gate_up", "gemm_down", "gemm_lm_head", "recurrence",
-                     "routing", "experts_gate_up", "experts_down")
+                     "routing", "experts_gate_up", "experts_down", "latent", "convolution")
 
     def profile_step(self, seqs: Sequence[Sequence_], last_tokens: np.ndarray) -> tuple[np.ndarray, dict]:
         """One eager decode step with per-kernel-kind device times (ms)."""

@@ -1,40 +1,22 @@
 // From a layer's projection rows to queries in place and keys and values in their slots: biases,
 // norms over whole projections, rotation of channel pairs, all in fp32, one CTA per row.
 #include "layered_ops.h"
+#include "prep_core.cuh"
 
 namespace hb {
 
-constexpr int kPrepThreads = 256;
-
-// Elements in runs of V (1: any sizes; 8 bf16 or 4 fp32 numbers: 16-byte accesses).
 template <typename T, int V>
-struct Run {
-  static __device__ __forceinline__ void load(float (&f)[V], const T* p) {
-    if constexpr (V == 1) {
-      f[0] = to_f32<T>(*p);
-    } else {
-      Vec16<T> v;
-      v.load(p);
-      v.unpack(f);
-    }
+__device__ __forceinline__ void copy_values(const AttentionPrep& a, const T* pr, int64_t slot) {
+  const int vper = a.vdim / V;
+  for (int i = threadIdx.x; i < a.kv_heads * vper; i += kPrepThreads) {
+    const int g = i / vper, d = i % vper * V;
+    float f[V];
+    Run<T, V>::load(f, pr + a.off_v + g * a.vdim + d);
+    Run<T, V>::store((T*)a.vc + pool_at(slot, a.kv_heads, g, a.vdim, d), f);
   }
-  static __device__ __forceinline__ void store(T* p, const float (&f)[V]) {
-    if constexpr (V == 1) {
-      *p = from_f32<T>(f[0]);
-    } else {
-      Vec16<T> v;
-      v.pack(f);
-      v.store(p);
-    }
-  }
-};
-
-// Where element d of kv head g of a row's key (value) lies in its pool.
-__device__ __forceinline__ int64_t pool_at(int64_t slot, int G, int g, int width, int d) {
-  return ((slot / HB_BLOCK_SIZE * G + g) * HB_BLOCK_SIZE + slot % HB_BLOCK_SIZE) * width + d;
 }
 
-// Rotation of channel pairs.  V > 1: runs of V channels (widths and the number of rotated channels
+// Rotation of neighbouring channels.  V > 1: runs of V channels (widths and the number of rotated channels
 // are multiples of V); V == 1: pair by pair.
 template <typename T, int V>
 __global__ void __launch_bounds__(kPrepThreads) attention_rotate_kernel(const AttentionPrep a) {
@@ -43,21 +25,16 @@ __global__ void __launch_bounds__(kPrepThreads) attention_rotate_kernel(const At
   pdl_grid_wait();
   const int64_t row = blockIdx.x, slot = a.slots[row];
   const int tid = threadIdx.x, P = a.pairs, D = a.dim;
-  const bool keep = slot >= 0 && slot < a.num_blocks * HB_BLOCK_SIZE;
+  const bool keep = a.kc && slot >= 0 && slot < a.num_blocks * HB_BLOCK_SIZE;
   T* pr = (T*)a.p + row * a.ld;
   constexpr int W = V == 1 ? 2 : V;           // channels a thread turns at a time
-  const int per = (D + W - 1) / W, total = (a.heads + a.kv_heads) * per;
+  const int per = (D + W - 1) / W, total = (a.heads + (a.kc ? a.kv_heads : 0)) * per;
   // channels i of head i / per: queries first, then keys
   auto source = [&](int i) { return pr + (i < a.heads * per ? a.off_q : a.off_k - a.heads * D) + i / per * D + i % per * W; };
   Vec16<T> ahead;  // the first run of every thread is on its way while the angles are formed
   if constexpr (V > 1)
     if (tid < total) ahead.load(source(tid));
-  // the angle less its whole turns in fp64: far positions keep the accuracy of near ones
-  const double pos = (double)a.pos[row], turn = 6.283185307179586;
-  for (int i = tid; i < P; i += kPrepThreads) {
-    const double angle = pos * a.rotation[i];
-    sincosf((float)(angle - turn * rint(angle * (1.0 / turn))), s_cs + P + i, s_cs + i);
-  }
+  angles_of(s_cs, a.rotation, P, a.pos[row], a.rotation_gain);
   __syncthreads();
   for (int i = tid; i < total; i += kPrepThreads) {
     const int head = i / per, d = i % per * W;
@@ -94,14 +71,58 @@ __global__ void __launch_bounds__(kPrepThreads) attention_rotate_kernel(const At
       Run<T, V>::store(dst, f);
     }
   }
-  if (!keep) return;
-  const int vper = a.vdim / V;
-  for (int i = tid; i < a.kv_heads * vper; i += kPrepThreads) {
-    const int g = i / vper, d = i % vper * V;
-    float f[V];
-    Run<T, V>::load(f, pr + a.off_v + g * a.vdim + d);
-    Run<T, V>::store((T*)a.vc + pool_at(slot, a.kv_heads, g, a.vdim, d), f);
+  if (keep) copy_values<T, V>(a, pr, slot);
+}
+
+// Channel i turned with channel i + pairs.  A thread takes V pairs, or V channels behind the pairs, at
+// a time (V > 1: widths and the number of pairs are multiples of V).
+template <typename T, int V>
+__global__ void __launch_bounds__(kPrepThreads) attention_rotate_halves_kernel(const AttentionPrep a) {
+  pdl_trigger();
+  extern __shared__ float s_cs[];  // [pairs] cosines, [pairs] sines
+  pdl_grid_wait();
+  const int64_t row = blockIdx.x, slot = a.slots[row];
+  const int tid = threadIdx.x, P = a.pairs, D = a.dim;
+  const bool keep = a.kc && slot >= 0 && slot < a.num_blocks * HB_BLOCK_SIZE;
+  T* pr = (T*)a.p + row * a.ld;
+  const int turned = P / V, per = turned + (D - 2 * P) / V, total = (a.heads + (keep ? a.kv_heads : 0)) * per;
+  auto channel = [&](int u) { return u < turned ? u * V : P + u * V; };  // first channel of unit u of a head
+  auto source = [&](int i) { return pr + (i < a.heads * per ? a.off_q : a.off_k - a.heads * D) + i / per * D + channel(i % per); };
+  float f[V], g[V];
+  auto load = [&](int i) {
+    const T* src = source(i);
+    Run<T, V>::load(f, src);
+    if (i % per < turned) Run<T, V>::load(g, src + P);
+  };
+  if (tid < total) load(tid);  // on its way while the angles are formed
+  angles_of(s_cs, a.rotation, P, a.pos[row], a.rotation_gain);
+  __syncthreads();
+  for (int i = tid; i < total; i += kPrepThreads) {
+    if (i >= kPrepThreads) load(i);
+    const int head = i / per, u = i % per, d = channel(u);
+    const bool query = head < a.heads, pair = u < turned;
+    const int h = query ? head : head - a.heads;
+    const float* bias = query ? a.q_bias : a.k_bias;
+    if (bias)
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        f[j] += bias[h * D + d + j];
+        if (pair) g[j] += bias[h * D + d + P + j];
+      }
+    if (pair) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        float x, y;
+        rope_rotate(f[j], g[j], s_cs[d + j], s_cs[P + d + j], &x, &y);
+        f[j] = x;
+        g[j] = y;
+      }
+    }
+    T* dst = query ? source(i) : (T*)a.kc + pool_at(slot, a.kv_heads, h, D, d);
+    Run<T, V>::store(dst, f);
+    if (pair) Run<T, V>::store(dst + P, g);
   }
+  if (keep) copy_values<T, V>(a, pr, slot);
 }
 
 // RMS norms over all query rows and all key rows of a position.  A thread keeps its first kHeld runs
@@ -207,24 +228,29 @@ int attention_prepare(cudaStream_t st, const AttentionPrep& a, int64_t rows, hb_
     return fail(HB_ERR_INVALID_ARG, "attention_prepare: norms come for queries and keys, and without a rotation");
   if (a.key_scale && (!norm || a.vdim != a.dim))
     return fail(HB_ERR_INVALID_ARG, "attention_prepare: keys that are the values have a norm and their width");
+  if (!a.kc && norm)
+    return fail(HB_ERR_INVALID_ARG, "attention_prepare: queries without keys are only rotated");
   if (2 * a.pairs > a.dim || a.pairs > 5000) return fail(HB_ERR_INVALID_ARG, "attention_prepare: %d pairs of %d channels", a.pairs, a.dim);
   const int es = (int)dtype_size(dtype), n = 16 / es;
   auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-  const bool vec = a.dim % n == 0 && a.vdim % n == 0 && (2 * a.pairs) % n == 0 && a.off_q % n == 0 && a.off_k % n == 0 &&
+  const bool vec = a.dim % n == 0 && a.vdim % n == 0 && (a.halves ? a.pairs : 2 * a.pairs) % n == 0 && a.off_q % n == 0 && a.off_k % n == 0 &&
                    a.off_v % n == 0 && a.ld % n == 0 && al(a.p) && al(a.kc) && al(a.vc);
   const dim3 grid((unsigned)rows), block(kPrepThreads);
   const size_t smem = (size_t)a.pairs * 2 * sizeof(float);
-  auto launch = [&](auto* rotate, auto* normed) -> int {
+  auto launch = [&](auto* rotate, auto* halves, auto* normed) -> int {
+    if (a.halves) rotate = halves;
     if (norm) HB_CUDA_CHECK(launch_pdl(normed, grid, block, 0, st, a));
     else HB_CUDA_CHECK(launch_pdl(rotate, grid, block, smem, st, a));
     return HB_OK;
   };
   if (dtype == HB_F32)
-    return vec ? launch(attention_rotate_kernel<float, 4>, attention_norm_kernel<float, 4>)
-               : launch(attention_rotate_kernel<float, 1>, attention_norm_kernel<float, 1>);
+    return vec ? launch(attention_rotate_kernel<float, 4>, attention_rotate_halves_kernel<float, 4>, attention_norm_kernel<float, 4>)
+               : launch(attention_rotate_kernel<float, 1>, attention_rotate_halves_kernel<float, 1>, attention_norm_kernel<float, 1>);
   if (dtype == HB_BF16)
-    return vec ? launch(attention_rotate_kernel<__nv_bfloat16, 8>, attention_norm_kernel<__nv_bfloat16, 8>)
-               : launch(attention_rotate_kernel<__nv_bfloat16, 1>, attention_norm_kernel<__nv_bfloat16, 1>);
+    return vec ? launch(attention_rotate_kernel<__nv_bfloat16, 8>, attention_rotate_halves_kernel<__nv_bfloat16, 8>,
+                         attention_norm_kernel<__nv_bfloat16, 8>)
+               : launch(attention_rotate_kernel<__nv_bfloat16, 1>, attention_rotate_halves_kernel<__nv_bfloat16, 1>,
+                         attention_norm_kernel<__nv_bfloat16, 1>);
   return fail(HB_ERR_UNSUPPORTED_DTYPE, "attention_prepare runs in bf16 or f32");
 }
 

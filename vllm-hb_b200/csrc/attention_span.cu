@@ -4,6 +4,7 @@
 //
 // The visible keys of a query at position p are two runs, [0, keep) and [lo, p] with
 // lo = SpanAttention::first_seen(p) and keep = min(keep_first, lo); only their blocks are read.
+#include <algorithm>
 #include <climits>
 
 #include "layered_ops.h"
@@ -49,14 +50,15 @@ int span_kv_write(cudaStream_t st, const SpanAttention& a, const void* k, const 
   return HB_OK;
 }
 
-// One CTA per (row, kv head): scores and running softmax of all query heads of the group in
+// One CTA per (row, kv head, slice of its query heads): scores and running softmax of all query heads of the group in
 // fp32 on CUDA cores.  The kernel for fp32 models and for sizes the tensor-core kernels do not take.
 template <typename T>
 __global__ void __launch_bounds__(kSpanThreads)
 span_attention_rows_kernel(const SpanAttention a, const int32_t* __restrict__ row_list) {
   pdl_grid_wait();
   extern __shared__ float sm[];
-  const int R = a.heads / a.kv_heads, D = a.dim, VD = a.vdim;
+  const HeadSlice hs(a, blockIdx.y);
+  const int R = hs.n, D = a.dim, VD = a.vdim;
   float* s_q = sm;                    // [R][D]
   float* s_p = s_q + R * D;           // [R][kSpanTile]
   float* s_acc = s_p + R * kSpanTile; // [R][VD]
@@ -66,15 +68,16 @@ span_attention_rows_kernel(const SpanAttention a, const int32_t* __restrict__ ro
   __shared__ int64_t s_key[kSpanTile];  // (block * kv_heads + head) * 16 + offset of the tile's keys
   __shared__ float s_ks[kSpanTile];     // scale of the keys
   __shared__ int s_dist[kSpanTile];     // their distance, up to the last of the bias table
-  const T* values = (const T*)(a.key_scale ? a.kc : a.vc);
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = blockIdx.y;
+  const T* values = (const T*)(a.vc ? a.vc : a.kc);
+  const int ld_v = a.vc ? VD : D;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = hs.kvh;
   const int64_t row = row_list[blockIdx.x];
   const int pos = a.pos[row];
   const int lo = a.first_seen(pos);
   const int keep = min(a.keep_first, lo);
   const int n_keys = keep + (pos - lo + 1);
   const int32_t* table = a.tables + (int64_t)a.row_seg[row] * a.max_blocks;
-  const T* q = (const T*)a.q + row * a.ld_q + (int64_t)g * R * D;
+  const T* q = (const T*)a.q + row * a.ld_q + (int64_t)hs.first * D;
   for (int i = tid; i < R * D; i += kSpanThreads) s_q[i] = to_f32<T>(q[i]) * a.scale;
   for (int i = tid; i < R * VD; i += kSpanThreads) s_acc[i] = 0.f;
   for (int i = tid; i < R; i += kSpanThreads) { s_m[i] = -INFINITY; s_l[i] = 0.f; }
@@ -96,8 +99,11 @@ span_attention_rows_kernel(const SpanAttention a, const int32_t* __restrict__ ro
         float s = 0.f;
         for (int d = lane; d < D; d += 32) s = fmaf(s_q[h * D + d], to_f32<T>(kr[d]), s);
         s = warp_sum(s);
-        if (lane == 0)
-          s_p[h * kSpanTile + i] = fmaf(s, s_ks[i], a.dist_bias ? a.dist_bias[(int64_t)(g * R + h) * a.dist_len + s_dist[i]] : 0.f);
+        if (lane == 0) {
+          s *= s_ks[i];
+          if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+          s_p[h * kSpanTile + i] = s + (a.dist_bias ? a.dist_bias[(int64_t)(hs.first + h) * a.dist_len + s_dist[i]] : 0.f);
+        }
       }
     }
     __syncthreads();
@@ -125,7 +131,7 @@ span_attention_rows_kernel(const SpanAttention a, const int32_t* __restrict__ ro
     for (int d = tid; d < VD; d += kSpanThreads) {
       for (int h = 0; h < R; ++h) s_acc[h * VD + d] *= s_a[h];
       for (int i = 0; i < nt; ++i) {
-        const float v = to_f32<T>(values[s_key[i] * VD + d]);
+        const float v = to_f32<T>(values[s_key[i] * ld_v + d]);
         for (int h = 0; h < R; ++h) s_acc[h * VD + d] = fmaf(s_p[h * kSpanTile + i], v, s_acc[h * VD + d]);
       }
     }
@@ -133,13 +139,13 @@ span_attention_rows_kernel(const SpanAttention a, const int32_t* __restrict__ ro
   __syncthreads();
   if (a.sink)  // one more member of the softmax, without a value
     for (int h = tid; h < R; h += kSpanThreads) {
-      const float k = a.sink[g * R + h], top = fmaxf(s_m[h], k), f = expf(s_m[h] - top);
+      const float k = a.sink[hs.first + h], top = fmaxf(s_m[h], k), f = expf(s_m[h] - top);
       s_a[h] = f;
       s_l[h] = fmaf(s_l[h], f, expf(k - top));
     }
   __syncthreads();
-  T* out = (T*)a.out + row * a.ld_out + (int64_t)g * R * VD;
-  const T* gate = a.gate ? (const T*)a.gate + row * a.ld_gate + (int64_t)g * R * VD : nullptr;
+  T* out = (T*)a.out + row * a.ld_out + (int64_t)hs.first * VD;
+  const T* gate = a.gate ? (const T*)a.gate + row * a.ld_gate + (int64_t)hs.first * VD : nullptr;
   for (int i = tid; i < R * VD; i += kSpanThreads) {
     float o = s_acc[i] / s_l[i / VD];
     if (a.sink) o *= s_a[i / VD];
@@ -148,16 +154,19 @@ span_attention_rows_kernel(const SpanAttention a, const int32_t* __restrict__ ro
   }
 }
 
-int span_attention_rows(cudaStream_t st, const SpanAttention& a, const int32_t* row_list, int n_rows, hb_dtype dtype) {
+int span_attention_rows(cudaStream_t st, const SpanAttention& args, const int32_t* row_list, int n_rows, hb_dtype dtype) {
   if (n_rows == 0) return HB_OK;
-  const int R = a.heads / a.kv_heads;
-  const size_t smem = (size_t)R * (a.dim + kSpanTile + a.vdim + 3) * sizeof(float);
+  SpanAttention a = args;
+  const size_t per_head = (size_t)(a.dim + kSpanTile + a.vdim + 3) * sizeof(float);
+  a.cut(std::max(1, (int)(100 * 1024 / per_head)));
+  const size_t smem = a.slice * per_head;
   if (smem > 200 * 1024)
-    return fail(HB_ERR_INVALID_ARG, "attention: %d query heads of %d + %d per kv head do not fit shared memory", R, a.dim, a.vdim);
+    return fail(HB_ERR_INVALID_ARG, "attention: a head of %d + %d channels does not fit shared memory", a.dim, a.vdim);
   auto launch = [&](auto* kernel) -> int {
     if (smem > 48 * 1024)
       HB_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    HB_CUDA_CHECK(launch_pdl(kernel, dim3((unsigned)n_rows, (unsigned)a.kv_heads), dim3(kSpanThreads), smem, st, a, row_list));
+    HB_CUDA_CHECK(launch_pdl(kernel, dim3((unsigned)n_rows, (unsigned)(a.kv_heads * a.slices())), dim3(kSpanThreads), smem,
+                             st, a, row_list));
     return HB_OK;
   };
   if (dtype == HB_F32) return launch(span_attention_rows_kernel<float>);

@@ -1,8 +1,8 @@
 // Span attention (see attention_span.cu) on tensor cores: bf16, key and value widths that are
 // multiples of 8.  S = Q K^T with bf16 operands and fp32 accumulation, softmax in fp32, and
 // O += P V with P as a pair of bf16 numbers (P = hi + lo), so that the weights keep fp32-like
-// precision.  Kernels instantiated with EXT also take a bias by distance and keys that are their
-// values times a scale: K and V are then one tile of shared memory, read once.
+// precision.  Kernels instantiated with EXT also take a bias by distance, a cap on the scores, and keys
+// that are or contain their values: K and V are then one tile of shared memory, read once.
 //
 //   tiles  (prompt portions): CTA = 64 rows = up to 64 / R consecutive positions of one segment x
 //          the R query heads of a kv head; four warps of 16 rows share every 64-key tile.
@@ -57,6 +57,8 @@ __device__ __forceinline__ bool all_visible(int key, int first, int lo, int keep
   return key + kBS - 1 <= first && (key >= lo || key + kBS <= keep_first);
 }
 constexpr float kLog2e = 1.4426950408889634f;
+// cap * tanh(s / cap) for a score and a cap in units of log2, tanh(y) = 1 - 2 / (1 + e^(2y)); k = 2 / softcap
+__device__ __forceinline__ float capped(float s, float cap, float k) { return cap - __fdividef(2.f * cap, 1.f + ex2(s * k)); }
 __device__ __forceinline__ float sigmoid_of(uint32_t bits16) {
   const float z = __uint_as_float(bits16 << 16);  // a bf16 number
   return __fdividef(1.f, 1.f + __expf(-z));
@@ -91,14 +93,15 @@ template <int NV, bool EXT, bool FIX>
 __global__ void __launch_bounds__(kThreads)
 span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ tiles, int stages) {
   extern __shared__ __align__(16) uint8_t smem[];
-  const int R = a.heads / a.kv_heads, D = FIX ? 16 * NV : a.dim, DP = pad16(D), KS = DP + 8;
-  const bool tied = EXT && a.key_scale != nullptr;      // one tile is keys and values
+  const HeadSlice hs(a, blockIdx.y);
+  const int R = hs.n, D = FIX ? 16 * NV : a.dim, DP = pad16(D), KS = DP + 8;
+  const bool tied = EXT && !a.vc;                       // one tile is keys and values
   const int v0 = FIX ? 0 : blockIdx.z * kSlice, VW = FIX ? 16 * NV : min(kSlice, a.vdim - v0), VP = pad16(VW), VS = tied ? KS : VP + 8;
   __nv_bfloat16* s_q = (__nv_bfloat16*)smem;           // [64][KS]
   __nv_bfloat16* s_k = s_q + kRows * KS;               // [stages][64][KS]
   __nv_bfloat16* s_v = tied ? s_k : s_k + stages * kKeys * KS;               // [stages][64][VS]
   float* s_ks = (float*)(s_k + stages * kKeys * KS);   // tied: [stages][64] scales of the keys
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gi = lane >> 2, t = lane & 3, kvh = blockIdx.y;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gi = lane >> 2, t = lane & 3, kvh = hs.kvh;
   // padding columns stay zero
   for (int i = tid; i < (kRows + stages * kKeys) * KS / 8; i += kThreads)
     if (i % (KS / 8) * 8 >= D) reinterpret_cast<uint4*>(s_q)[i] = make_uint4(0, 0, 0, 0);
@@ -112,7 +115,7 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
   const int32_t* table = a.tables + (int64_t)tile.seg * a.max_blocks;
   const int n_rows = tile.n * R, n_steps = (runs.n + kKeys / kBS - 1) / (kKeys / kBS);
 
-  const __nv_bfloat16* q = (const __nv_bfloat16*)a.q + (int64_t)kvh * R * D;
+  const __nv_bfloat16* q = (const __nv_bfloat16*)a.q + (int64_t)hs.first * D;
   for (int i = tid; i < kRows * (D / 8); i += kThreads) {
     const int m = i / (D / 8), c = i % (D / 8) * 8;
     uint4 v = make_uint4(0, 0, 0, 0);
@@ -129,7 +132,7 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
     const int64_t slot = (phys * a.kv_heads + kvh) * kBS;
     copy_k(smem_u32(s_k + (s * kKeys + warp * kBS) * KS), KS * 2, (const __nv_bfloat16*)a.kc + slot * D, D);
     if (!tied) copy_v(smem_u32(s_v + (s * kKeys + warp * kBS) * VS), VS * 2, (const __nv_bfloat16*)a.vc + slot * a.vdim + v0, a.vdim);
-    else if (lane < 4) cp_async_16(smem_u32(s_ks + s * kKeys + warp * kBS + lane * 4), a.key_scale + phys * kBS + lane * 4);
+    else if (a.key_scale && lane < 4) cp_async_16(smem_u32(s_ks + s * kKeys + warp * kBS + lane * 4), a.key_scale + phys * kBS + lane * 4);
     cp_async_commit();
   };
   load(0);
@@ -147,11 +150,12 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
   const float es = sc_ok ? sc : 1.f;               // what the exponential still multiplies by
   const int warp_first = first_pos + warp * 16 / R, warp_last = min(first_pos + (warp * 16 + 15) / R, last_pos);
   const int warp_lo = a.first_seen(warp_last);
+  const float cap = EXT ? a.softcap * kLog2e : 0.f, cap_k = cap > 0.f ? 2.f / a.softcap : 0.f;
   const float *bias0 = nullptr, *bias1 = nullptr;  // of the rows' heads, by distance
   float far0 = 0.f, far1 = 0.f;                    // from distance dist_len - 1 on, in units of log2
   if (EXT && a.dist_bias) {
-    bias0 = a.dist_bias + (int64_t)(kvh * R + r0 % R) * a.dist_len;
-    bias1 = a.dist_bias + (int64_t)(kvh * R + r1 % R) * a.dist_len;
+    bias0 = a.dist_bias + (int64_t)(hs.first + r0 % R) * a.dist_len;
+    bias1 = a.dist_bias + (int64_t)(hs.first + r1 % R) * a.dist_len;
     far0 = __ldg(bias0 + a.dist_len - 1) * kLog2e;
     far1 = __ldg(bias1 + a.dist_len - 1) * kLog2e;
   }
@@ -200,10 +204,15 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
           float2 f = make_float2(sc, sc);
-          if (tied) {
+          if (a.key_scale) {
             f = *reinterpret_cast<const float2*>(s_ks + step % stages * kKeys + i * 8 + 2 * t);
             f.x *= sc;
             f.y *= sc;
+          }
+          if (cap > 0.f) {
+            s[i][0] = capped(s[i][0] * f.x, cap, cap_k); s[i][1] = capped(s[i][1] * f.y, cap, cap_k);
+            s[i][2] = capped(s[i][2] * f.x, cap, cap_k); s[i][3] = capped(s[i][3] * f.y, cap, cap_k);
+            f = make_float2(1.f, 1.f);
           }
           if (far) {
             s[i][0] = fmaf(s[i][0], f.x, far0); s[i][1] = fmaf(s[i][1], f.y, far0);
@@ -285,18 +294,18 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
   float i0 = 1.f / l0, i1 = 1.f / l1;
   if (a.sink) {  // one more member of the softmax, without a value
-    const float k0 = a.sink[kvh * R + r0 % R] * kLog2e, k1 = a.sink[kvh * R + r1 % R] * kLog2e;
+    const float k0 = a.sink[hs.first + r0 % R] * kLog2e, k1 = a.sink[hs.first + r1 % R] * kLog2e;
     const float t0 = fmaxf(m0 * es, k0), t1 = fmaxf(m1 * es, k1), f0 = ex2(m0 * es - t0), f1 = ex2(m1 * es - t1);
     i0 = f0 / fmaf(l0, f0, ex2(k0 - t0));
     i1 = f1 / fmaf(l1, f1, ex2(k1 - t1));
   }
   const __nv_bfloat16 *g0 = nullptr, *g1 = nullptr;
   if (a.gate) {
-    const __nv_bfloat16* gate = (const __nv_bfloat16*)a.gate + (int64_t)kvh * R * a.vdim + v0;
+    const __nv_bfloat16* gate = (const __nv_bfloat16*)a.gate + (int64_t)hs.first * a.vdim + v0;
     g0 = gate + (int64_t)(tile.row0 + r0 / R) * a.ld_gate + (r0 % R) * a.vdim;
     g1 = gate + (int64_t)(tile.row0 + r1 / R) * a.ld_gate + (r1 % R) * a.vdim;
   }
-  __nv_bfloat16* out = (__nv_bfloat16*)a.out + (int64_t)kvh * R * a.vdim + v0;
+  __nv_bfloat16* out = (__nv_bfloat16*)a.out + (int64_t)hs.first * a.vdim + v0;
   __nv_bfloat16* w0 = out + (int64_t)(tile.row0 + r0 / R) * a.ld_out + (r0 % R) * a.vdim;
   __nv_bfloat16* w1 = out + (int64_t)(tile.row0 + r1 / R) * a.ld_out + (r1 % R) * a.vdim;
 #pragma unroll
@@ -329,11 +338,12 @@ __global__ void __launch_bounds__(kThreads)
 span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, int n_splits, int clustered,
                              float* __restrict__ part) {
   extern __shared__ __align__(16) uint8_t smem[];
-  const int R = a.heads / a.kv_heads, D = FIX ? 16 * MT : a.dim, DP = pad16(D), KS = DP + 8;
-  const bool tied = EXT && a.key_scale != nullptr;  // one tile is keys and values; their scales lie behind it
+  const HeadSlice hs(a, blockIdx.y);
+  const int R = hs.n, D = FIX ? 16 * MT : a.dim, DP = pad16(D), KS = DP + 8;
+  const bool tied = EXT && !a.vc;                   // one tile is keys and values; their scales lie behind it
   const int v0 = FIX ? 0 : (int)(blockIdx.z / n_splits) * kSlice, VW = FIX ? 16 * MT : min(kSlice, a.vdim - v0), VP = pad16(VW), VS = VP + 8;
   const int split = blockIdx.z % n_splits;
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gi = lane >> 2, t = lane & 3, kvh = blockIdx.y;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gi = lane >> 2, t = lane & 3, kvh = hs.kvh;
   const int stage_elems = tied ? kBS * (KS + 2) : kBS * (KS + VS);
   __nv_bfloat16* s_q = (__nv_bfloat16*)smem;                                  // [16][KS]
   __nv_bfloat16* ring = s_q + 16 * KS + (size_t)warp * kRing * stage_elems;   // [kRing][K 16 x KS | V 16 x VS]
@@ -372,14 +382,14 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
       const uint32_t dst = ring_u + stage_in * stage_elems * 2;
       copy_k(dst, KS * 2, (const __nv_bfloat16*)a.kc + slot * D, D);
       if (!tied) copy_v(dst + kBS * KS * 2, VS * 2, (const __nv_bfloat16*)a.vc + slot * a.vdim + v0, a.vdim);
-      else if (lane < 4) cp_async_16(dst + kBS * KS * 2 + lane * 16, a.key_scale + phys * kBS + lane * 4);
+      else if (a.key_scale && lane < 4) cp_async_16(dst + kBS * KS * 2 + lane * 16, a.key_scale + phys * kBS + lane * 4);
     }
     cp_async_commit();
     stage_in = stage_in + 1 == kRing ? 0 : stage_in + 1;
   };
   load_tab(0);
   for (int i = 0; i < kRing - 1; ++i) load(i);
-  const __nv_bfloat16* q = (const __nv_bfloat16*)a.q + row * a.ld_q + (int64_t)kvh * R * D;
+  const __nv_bfloat16* q = (const __nv_bfloat16*)a.q + row * a.ld_q + (int64_t)hs.first * D;
   for (int i = tid; i < 16 * (KS / 8); i += kThreads) {
     const int m = i / (KS / 8), c = i % (KS / 8) * 8;
     uint4 v = make_uint4(0, 0, 0, 0);
@@ -396,13 +406,14 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
     l[n][0] = l[n][1] = 0.f;
   }
   const float sc = a.scale * kLog2e;  // scores in units of log2
+  const float cap = EXT ? a.softcap * kLog2e : 0.f, cap_k = cap > 0.f ? 2.f / a.softcap : 0.f;
   float far[NT][2];                   // bias from distance dist_len - 1 on
 #pragma unroll
   for (int n = 0; n < NT; ++n)
 #pragma unroll
     for (int c = 0; c < 2; ++c) {
       const int head = min(n * 8 + 2 * t + c, R - 1);
-      far[n][c] = EXT && a.dist_bias ? __ldg(a.dist_bias + (int64_t)(kvh * R + head + 1) * a.dist_len - 1) * kLog2e : 0.f;
+      far[n][c] = EXT && a.dist_bias ? __ldg(a.dist_bias + (int64_t)(hs.first + head + 1) * a.dist_len - 1) * kLog2e : 0.f;
     }
   const uint32_t q_addr = smem_u32(s_q + (lane & 7) * KS + (lane >> 3) * 8);  // B fragments of two 16-channel steps
   const uint32_t k_off = (uint32_t)(((lane & 15) * KS + (lane >> 4) * 8) * 2);
@@ -441,7 +452,7 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
     const bool see0 = full || visible(key0 + gi, pos, lo, a.keep_first);
     const bool see1 = full || visible(key0 + gi + 8, pos, lo, a.keep_first);
     float f0 = sc, f1 = sc;  // scales of keys gi and gi + 8
-    if (tied) {
+    if (EXT && a.key_scale) {
       const float* ks = reinterpret_cast<const float*>(stage_ptr + kBS * KS);
       f0 *= ks[gi];
       f1 *= ks[gi + 8];
@@ -458,10 +469,14 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
         float b = far[n][e & 1];
         if (near) {
           const int head = min(n * 8 + 2 * t + (e & 1), R - 1);
-          b = __ldg(a.dist_bias + (int64_t)(kvh * R + head) * a.dist_len + (e < 2 ? d0 : d1)) * kLog2e;
+          b = __ldg(a.dist_bias + (int64_t)(hs.first + head) * a.dist_len + (e < 2 ? d0 : d1)) * kLog2e;
         }
-        const float x = s[n][0][e] + s[n][1][e];
-        p[e] = (e < 2 ? see0 : see1) ? (EXT ? fmaf(x, e < 2 ? f0 : f1, b) : x * sc) : -INFINITY;
+        float x = s[n][0][e] + s[n][1][e];
+        if (EXT) {
+          x *= e < 2 ? f0 : f1;
+          if (cap > 0.f) x = capped(x, cap, cap_k);
+        }
+        p[e] = (e < 2 ? see0 : see1) ? (EXT ? x + b : x * sc) : -INFINITY;
       }
       float x0 = fmaxf(p[0], p[2]), x1 = fmaxf(p[1], p[3]);
 #pragma unroll
@@ -536,7 +551,7 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
       f[w] = mw == -INFINITY ? 0.f : ex2(mw - mx);
       ls = fmaf(f[w], s_ml[(w * R + h) * 2 + 1], ls);
     }
-    const int64_t head = (int64_t)kvh * R + h;
+    const int64_t head = hs.first + h;
     float inv = 1.f / ls;
     if (a.sink && n_splits == 1) {
       const float k = a.sink[head] * kLog2e, top = fmaxf(mx, k), f = ex2(mx - top);
@@ -570,7 +585,7 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
   const uint32_t o_addr = smem_u32(s_o), ml_addr = smem_u32(s_ml);
   for (int i = split * kThreads + tid; i < R * VW; i += n_splits * kThreads) {
     const int h = i / VW, c = i % VW;
-    const int64_t head = (int64_t)kvh * R + h;
+    const int64_t head = hs.first + h;
     const float k = a.sink ? a.sink[head] * kLog2e : -INFINITY;
     float mx = k, ls = 0.f, acc = 0.f, mw[kMaxCluster];
 #pragma unroll
@@ -622,13 +637,19 @@ span_attention_merge_kernel(const SpanAttention a, const int32_t* __restrict__ r
   }
 }
 
+static SpanAttention sliced(const SpanAttention& args, int most) {
+  SpanAttention a = args;
+  a.cut(most);
+  return a;
+}
+static bool is_ext(const SpanAttention& a) { return !a.vc || a.dist_bias || a.softcap > 0.f; }
 static size_t tiles_smem(const SpanAttention& a, int stages) {
   const int KS = pad16(a.dim) + 8, VS = pad16(std::min(a.vdim, kSlice)) + 8;
-  return (size_t)(kRows * KS + stages * kKeys * (KS + (a.key_scale ? 2 : VS))) * 2;
+  return (size_t)(kRows * KS + stages * kKeys * (KS + (a.vc ? VS : 2))) * 2;
 }
 static size_t tokens_smem(const SpanAttention& a) {
-  const int R = a.heads / a.kv_heads, KS = pad16(a.dim) + 8, VP = pad16(std::min(a.vdim, kSlice)), VS = VP + 8;
-  const size_t ring = (size_t)kWarps * kRing * kBS * (KS + (a.key_scale ? 2 : VS)) * 2;
+  const int R = sliced(a, 16).slice, KS = pad16(a.dim) + 8, VP = pad16(std::min(a.vdim, kSlice)), VS = VP + 8;
+  const size_t ring = (size_t)kWarps * kRing * kBS * (KS + (a.vc ? VS : 2)) * 2;
   const size_t merge = (size_t)kWarps * R * (VP + 4) * sizeof(float);
   return (size_t)16 * KS * 2 + std::max(ring, merge);
 }
@@ -639,20 +660,19 @@ static bool span_mma_ok(const SpanAttention& a, hb_dtype dtype) {
   static const bool simt = [] { const char* e = getenv("HB_ATTN"); return e && e[0] == 's'; }();
   return !simt && dtype == HB_BF16 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ld_q % 8 == 0 && a.ld_out % 2 == 0 && al(a.q) &&
          al(a.out) && (!a.gate || (a.ld_gate % 2 == 0 && (reinterpret_cast<uintptr_t>(a.gate) & 3) == 0)) &&
-         (!a.key_scale || (a.dim == a.vdim && al(a.key_scale)));
+         (a.vc || a.vdim <= a.dim) && (!a.key_scale || (a.dim == a.vdim && !a.vc && al(a.key_scale)));
 }
 
 int span_attention_tile_positions(const SpanAttention& a, hb_dtype dtype) {
-  const int R = a.heads / a.kv_heads;
-  if (!span_mma_ok(a, dtype) || R > kRows || tiles_smem(a, 1) > kSmemCap) return 0;
-  return kRows / R;
+  if (!span_mma_ok(a, dtype) || tiles_smem(a, 1) > kSmemCap) return 0;
+  return kRows / sliced(a, kRows).slice;
 }
 int span_attention_tokens_slots(const SpanAttention& a) {
   constexpr int kSms = 148;
   return kSms * (int)std::max<size_t>(1, std::min<size_t>(8, (size_t)227 * 1024 / (tokens_smem(a) + 1024)));
 }
 bool span_attention_tokens_supported(const SpanAttention& a, hb_dtype dtype) {
-  return span_mma_ok(a, dtype) && a.heads / a.kv_heads <= 16 && tokens_smem(a) <= kSmemCap;
+  return span_mma_ok(a, dtype) && tokens_smem(a) <= kSmemCap;
 }
 
 template <typename K>
@@ -661,11 +681,14 @@ static int opt_in(K kernel, size_t smem) {
   return HB_OK;
 }
 
-int span_attention_tiles(cudaStream_t st, const SpanAttention& a, const RowRange* tiles, int n_tiles) {
+int span_attention_token_units(const SpanAttention& a) { return a.kv_heads * sliced(a, 16).slices(); }
+
+int span_attention_tiles(cudaStream_t st, const SpanAttention& args, const RowRange* tiles, int n_tiles) {
   if (n_tiles == 0) return HB_OK;
+  const SpanAttention a = sliced(args, kRows);
   const int stages = tiles_smem(a, 2) <= kSmemCap ? 2 : 1;
   const size_t smem = tiles_smem(a, stages);
-  const dim3 grid((unsigned)n_tiles, (unsigned)a.kv_heads, (unsigned)((a.vdim + kSlice - 1) / kSlice));
+  const dim3 grid((unsigned)n_tiles, (unsigned)(a.kv_heads * a.slices()), (unsigned)((a.vdim + kSlice - 1) / kSlice));
   auto launch = [&](auto* k) -> int {
     int rc = opt_in(k, smem);
     if (rc) return rc;
@@ -673,7 +696,7 @@ int span_attention_tiles(cudaStream_t st, const SpanAttention& a, const RowRange
     return HB_OK;
   };
   const int vw = std::min(a.vdim, kSlice);
-  const bool ext = a.key_scale || a.dist_bias;
+  const bool ext = is_ext(a);
 #define HB_TILES(NV)                                                                                          \
   return a.dim == 16 * NV && a.vdim == 16 * NV                                                                \
              ? (ext ? launch(span_attention_tiles_kernel<NV, true, true>) : launch(span_attention_tiles_kernel<NV, false, true>)) \
@@ -685,12 +708,13 @@ int span_attention_tiles(cudaStream_t st, const SpanAttention& a, const RowRange
 #undef HB_TILES
 }
 
-int span_attention_tokens(cudaStream_t st, const SpanAttention& a, const int32_t* rows, int n_rows, int n_splits, float* part) {
+int span_attention_tokens(cudaStream_t st, const SpanAttention& args, const int32_t* rows, int n_rows, int n_splits, float* part) {
   if (n_rows == 0) return HB_OK;
+  const SpanAttention a = sliced(args, 16);
   const size_t smem = tokens_smem(a);
   const int slices = (a.vdim + kSlice - 1) / kSlice;
   const bool clustered = n_splits > 1 && n_splits <= kMaxCluster;
-  const dim3 grid((unsigned)n_rows, (unsigned)a.kv_heads, (unsigned)(slices * n_splits));
+  const dim3 grid((unsigned)n_rows, (unsigned)(a.kv_heads * a.slices()), (unsigned)(slices * n_splits));
   auto launch = [&](auto* k) -> int {
     int rc = opt_in(k, smem);
     if (rc) return rc;
@@ -717,8 +741,8 @@ int span_attention_tokens(cudaStream_t st, const SpanAttention& a, const int32_t
   };
   const int vw = std::min(a.vdim, kSlice);
   int rc;
-  const bool wide = a.heads / a.kv_heads > 8;
-  const bool ext = a.key_scale || a.dist_bias;
+  const bool wide = a.slice > 8;
+  const bool ext = is_ext(a);
 #define HB_TOKENS_OF(MT, FIX)                                                                                      \
   rc = ext ? (wide ? launch(span_attention_tokens_kernel<MT, 2, true, FIX>) : launch(span_attention_tokens_kernel<MT, 1, true, FIX>)) \
            : (wide ? launch(span_attention_tokens_kernel<MT, 2, false, FIX>) : launch(span_attention_tokens_kernel<MT, 1, false, FIX>))

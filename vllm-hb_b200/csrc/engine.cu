@@ -1350,6 +1350,7 @@ int hb_kv_swap_blocks(hb_engine* e, const int64_t* pairs, size_t n_pairs, int to
     for (size_t l = 0; l < e->kc.size(); ++l)
       for (int kv = 0; kv < 2; ++kv) {
         const size_t block_bytes = kv ? e->v_block_bytes[l] : e->k_block_bytes[l];
+        if (!block_bytes) continue;  // a layer of one pool
         uint8_t* dev = (uint8_t*)(kv ? e->vc[l] : e->kc[l]) + (size_t)g * block_bytes;
         if (to_cpu) HB_CUDA_CHECK(cudaMemcpyAsync(host, dev, block_bytes, cudaMemcpyDeviceToHost, e->stream));
         else HB_CUDA_CHECK(cudaMemcpyAsync(dev, host, block_bytes, cudaMemcpyHostToDevice, e->stream));

@@ -202,7 +202,7 @@ namespace hb {
 // kCatGemm is the QKV projection; the other projections have kinds of their own
 enum ProfCat { kCatGemm = 0, kCatAttention = 1, kCatRopeKv = 2, kCatNorm = 3, kCatOther = 4, kCatComm = 5,
                kCatGemmO = 6, kCatGemmGateUp = 7, kCatGemmDown = 8, kCatGemmLmHead = 9, kCatRecurrence = 10,
-               kCatRouting = 11, kCatExpertsUp = 12, kCatExpertsDown = 13, kNumCats = 14 };
+               kCatRouting = 11, kCatExpertsUp = 12, kCatExpertsDown = 13, kCatLatent = 14, kCatConv = 15, kNumCats = 16 };
 
 // While profiling, every call opens a timed segment of kind `cat` on the stream.
 void prof_mark(hb_engine* e, int cat);

@@ -21,8 +21,10 @@ struct GatedAct {
   float slope = 1.f, cubic = 0.f, limit = INFINITY, shift = 0.f;
   bool silu() const { return slope == 1.f && cubic == 0.f && limit == INFINITY && shift == 0.f; }
 };
-// out[m, i] = act(gate_up[m, i], gate_up[m, inter + i]); rows of out have stride inter.
-int gated_act(cudaStream_t st, void* out, const void* gate_up, int64_t M, int64_t inter, const GatedAct& act, hb_dtype dtype);
+// out[m, i] = act(gate_up[m, i] + gate_bias[i], gate_up[m, inter + i] + up_bias[i]); rows of out have
+// stride inter, the biases may be null.
+int gated_act(cudaStream_t st, void* out, const void* gate_up, int64_t M, int64_t inter, const GatedAct& act, hb_dtype dtype,
+              const float* gate_bias = nullptr, const float* up_bias = nullptr);
 
 // Rows of a GEMM sorted by group (mixture of experts): every batch tile of `m_pad` rows belongs to
 // one group, whose weights start at row group * (weight rows of one group); tile_group[i] < 0: no
@@ -42,7 +44,19 @@ struct TcGroups {
 // CUDA-core form: Y[r] = X[r] . W[group of r]^T, tiles of m_pad rows (a multiple of 8).
 int gemm_simt_grouped(cudaStream_t st, void* Y, const void* X, const void* W, int64_t N, int64_t K, hb_dtype dtype, bool out_f32,
                       const TcGroups& groups, const int32_t* tile_group);
-// gated_act over the rows of such a GEMM: gate | up rows of stride ld_gu, out rows of stride ld_out;
+// Independent products side by side, one per head: Y_h = X_h . W_h^T with the [N, K] matrices of all
+// heads one after another in W, X_h = X + h * x_step (rows of ldx elements) and Y_h = Y + h * y_step
+// (rows of ldy elements, y_step >= N).
+struct TcHeads {
+  int heads = 0;
+  int64_t ldx = 0, x_step = 0, ldy = 0, y_step = 0;
+};
+// CUDA-core form.
+int gemm_simt_heads(cudaStream_t st, void* Y, const void* X, const void* W, int64_t M, int64_t N, int64_t K, hb_dtype dtype,
+                    bool out_f32, const TcHeads& heads);
+// Sizes and steps that gemm_tc_plan takes with heads (bf16).
+bool gemm_tc_heads_supported(int64_t N, int64_t K, bool out_f32, const TcHeads& heads);
+// gated_act over the rows of a grouped GEMM: gate | up rows of stride ld_gu, out rows of stride ld_out;
 // inter and act of the groups, and of the further one.
 int gated_act_grouped(cudaStream_t st, void* out, int64_t ld_out, const void* gate_up, int64_t ld_gu, int64_t inter,
                       const GatedAct& act, hb_dtype dtype, const TcGroups& groups, const int32_t* tile_group);
@@ -129,8 +143,10 @@ struct TcGemmPlan {
   size_t smem_bytes = 0;
   int epilogue = kEpiStore;
   GatedAct act;          // kEpiSwiGLU
+  const float *gate_bias = nullptr, *up_bias = nullptr;  // kEpiSwiGLU: [N], added before the activation
+  TcHeads heads;         // heads > 0: TcHeads form
   int groups = 0;        // > 0: TcGroups form; rows of the batch operand are sorted by group
-  int group_rows = 0;    // weight rows of one group
+  int group_rows = 0;    // weight rows of one group (or head)
   CUtensorMap tm_w2;     // further group: its weights, features, K and activation
   int64_t N2 = 0, K2 = 0;
   GatedAct act2;
@@ -146,7 +162,8 @@ struct TcGemmPlan {
 bool gemm_tc_supported(int64_t M, int64_t N, int64_t K, hb_dtype dtype);
 // X and W must be 16-byte aligned device pointers; they are baked into the plan.
 int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int64_t N, int64_t K,
-                 int epilogue, bool out_f32, int device, int force_splits = 0, const TcGroups* groups = nullptr);
+                 int epilogue, bool out_f32, int device, int force_splits = 0, const TcGroups* groups = nullptr,
+                 const TcHeads* heads = nullptr);
 // groups: W holds the [N, K] matrices of all groups one after another, M is the row capacity of the
 // sorted batch operand; gemm_tc_run then needs tile_group (device, max_tiles entries).
 // Y row stride ldy in elements.  workspace: plan.workspace_bytes(), zeroed once.

@@ -20,6 +20,8 @@ struct SimtGroups {
   int m_pad = 1, further = -1;
   const void* w2 = nullptr;
   int64_t n2 = 0, k2 = 0;
+  int heads = 0;  // TcHeads: blockIdx.z is the head
+  int64_t x_step = 0, y_step = 0;
 };
 template <typename T, typename OutT, bool VEC>
 __global__ void __launch_bounds__(kSimtWarps * 32)
@@ -30,6 +32,11 @@ gemm_simt_kernel(OutT* __restrict__ Y, const T* __restrict__ X, const T* __restr
   const int64_t n = (int64_t)blockIdx.x * kSimtWarps + warp;
   const int64_t m0 = (int64_t)blockIdx.y * kMB;
   const T* wr = W + n * K;
+  if (g.heads) {
+    wr += (int64_t)blockIdx.z * N * K;
+    X += (int64_t)blockIdx.z * g.x_step;
+    Y += (int64_t)blockIdx.z * g.y_step;
+  }
   if (g.tile_group) {
     const int group = g.tile_group[m0 / g.m_pad];
     if (group < 0) return;
@@ -81,10 +88,11 @@ template <typename T, typename OutT>
 static int launch_simt(cudaStream_t st, OutT* Y, const T* X, const T* W, int64_t M, int64_t N,
                        int64_t K, int64_t ldx, int64_t ldy, const SimtGroups& g = SimtGroups()) {
   constexpr int NV = Vec16<T>::N;
-  const bool vec = K % NV == 0 && ldx % NV == 0 && g.k2 % NV == 0 && (reinterpret_cast<uintptr_t>(g.w2) & 15) == 0 && (reinterpret_cast<uintptr_t>(X) & 15) == 0 &&
+  const bool vec = K % NV == 0 && ldx % NV == 0 && g.k2 % NV == 0 && g.x_step % NV == 0 && (reinterpret_cast<uintptr_t>(g.w2) & 15) == 0 && (reinterpret_cast<uintptr_t>(X) & 15) == 0 &&
                    (reinterpret_cast<uintptr_t>(W) & 15) == 0;
   const int64_t widest = N > g.n2 ? N : g.n2;
-  dim3 grid((unsigned)((widest + kSimtWarps - 1) / kSimtWarps), (unsigned)((M + kMB - 1) / kMB));
+  dim3 grid((unsigned)((widest + kSimtWarps - 1) / kSimtWarps), (unsigned)((M + kMB - 1) / kMB),
+            (unsigned)(g.heads ? g.heads : 1));
   if (vec)
     gemm_simt_kernel<T, OutT, true><<<grid, kSimtWarps * 32, 0, st>>>(Y, X, W, M, N, K, ldx, ldy, g);
   else
@@ -100,6 +108,20 @@ int gemm_simt(cudaStream_t st, void* Y, const void* X, const void* W, int64_t M,
     if (out_f32)
       return (launch_simt<T, float>(st, (float*)Y, (const T*)X, (const T*)W, M, N, K, K, N));
     return (launch_simt<T, T>(st, (T*)Y, (const T*)X, (const T*)W, M, N, K, K, N));
+  });
+  return HB_OK;
+}
+
+int gemm_simt_heads(cudaStream_t st, void* Y, const void* X, const void* W, int64_t M, int64_t N, int64_t K, hb_dtype dtype,
+                    bool out_f32, const TcHeads& heads) {
+  if (heads.heads < 1 || heads.heads > 65535) return fail(HB_ERR_INVALID_ARG, "gemm_simt_heads: %d heads", heads.heads);
+  if (M == 0 || N == 0) return HB_OK;
+  SimtGroups g;
+  g.heads = heads.heads; g.x_step = heads.x_step; g.y_step = heads.y_step;
+  HB_DISPATCH_DTYPE(dtype, T, {
+    if (out_f32)
+      return (launch_simt<T, float>(st, (float*)Y, (const T*)X, (const T*)W, M, N, K, heads.ldx, heads.ldy, g));
+    return (launch_simt<T, T>(st, (T*)Y, (const T*)X, (const T*)W, M, N, K, heads.ldx, heads.ldy, g));
   });
   return HB_OK;
 }

@@ -55,6 +55,7 @@ struct TcParams {
   int further;                // number of the further group (tm_h holds its weights), -1: none
   int n_tiles2, k_chunks2, up_row_offset2;
   GatedAct act2;
+  const float *gate_bias, *up_bias;  // SwiGLU: added to the pair before its activation (may be null)
   int cluster;              // split-K partners form a thread-block cluster of `splits` CTAs
   int tma_store;            // the output leaves through bulk tensor stores (tm_y is valid)
   // Deferred RMSNorm (see TcNormLink in gemm.h).  Producer (epilogue kEpiResidual, cluster
@@ -171,10 +172,11 @@ __device__ __forceinline__ float gated_f(float g, float u, const GatedAct& act) 
 }
 
 // ----------------------------------------------------------------------- kernel
-// GROUPS: rows sorted by group (TcGroups).  GENERAL: any GatedAct, else SiLU.  The instance without
-// either is the one decode steps of dense models run: whatever it does not need costs it registers
-// and time (2 % of an 8B step).
-template <bool GROUPS, bool GENERAL>
+// GROUPS: rows sorted by group (TcGroups).  GENERAL: any GatedAct and biases of the pair, else SiLU.
+// HEADS: blockIdx.z counts independent products (TcHeads).  The instance without any of them is the
+// one decode steps of dense models run: whatever it does not need costs it registers and time (2 % of
+// an 8B step).
+template <bool GROUPS, bool GENERAL, bool HEADS>
 __global__ void __launch_bounds__(kTcThreads, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x,
                const __grid_constant__ CUtensorMap tm_y, const __grid_constant__ CUtensorMap tm_h,
@@ -207,7 +209,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
   const int tile = m_fast ? (int)blockIdx.y : unit;
   const int split = p.cluster ? (int)cluster_ctarank() : blockIdx.x % p.splits;
   const int m_tile = m_fast ? unit : (int)blockIdx.y;
-  int w_row = tile * kTileN;  // first weight row of the tile
+  const int head = HEADS ? (int)blockIdx.z : 0;
+  int w_row = tile * kTileN + (HEADS ? head * p.group_rows : 0);  // first weight row of the tile
   const CUtensorMap* w_map = &tm_w;
   int k_chunks = p.k_chunks, up_row_offset = p.up_row_offset;
   GatedAct act = p.act;
@@ -329,6 +332,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
       auto load_w = [&](uint32_t dst, int kx, int row, uint32_t bar) {
         tma_load_2d_hint(dst, w_map, kx, row, bar, w_policy);
       };
+      auto load_x = [&](uint32_t dst, int kx, uint32_t bar) {
+        if (HEADS) tma_load_3d(dst, &tm_x, kx, m_tile * p.m_pad, head, bar);
+        else tma_load_2d(dst, &tm_x, kx, m_tile * p.m_pad, bar);
+      };
       // Weights never depend on the previous kernel: the first stages' weight slabs are
       // requested before waiting for it; activations only afterwards.
       const int pre = min(p.stages, n_kc);
@@ -350,8 +357,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
       pdl_wait();
       TC_LAUNCH_TRACE(3);
       for (int i = 0; i < pre; ++i) {
-        tma_load_2d(smem_base + i * stage_bytes + a_bytes * n_acc, &tm_x, (kc0 + i) * kTileK, m_tile * p.m_pad,
-                    smem_u32(&s_full[i]));
+        load_x(smem_base + i * stage_bytes + a_bytes * n_acc, (kc0 + i) * kTileK, smem_u32(&s_full[i]));
       }
       armed = pre;
       for (int i = pre; i < n_kc; ++i) {
@@ -364,7 +370,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
         const int kx = (kc0 + i) * kTileK;
         load_w(sa, kx, w_row, full);
         if (swiglu) load_w(sa + a_bytes, kx, up_row_offset + w_row, full);
-        tma_load_2d(sa + a_bytes * n_acc, &tm_x, kx, m_tile * p.m_pad, full);
+        load_x(sa + a_bytes * n_acc, kx, full);
         armed = i + 1;
       }
       if (s_abort) {
@@ -433,6 +439,17 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
   tc_fence_after();
   const bool ok_all = s_abort == 0;
   TC_TRACE(tid == 0, 4);
+  auto store_tile = [&](uint32_t src, int m) {
+    if (HEADS) tma_store_3d(&tm_y, src, tile * kTileN, m, head);
+    else tma_store_2d(&tm_y, src, tile * kTileN, m);
+  };
+  // biases of this thread's output feature
+  constexpr bool BIAS = GENERAL && !GROUPS;
+  float gate_b = 0.f, up_b = 0.f;
+  if (BIAS && swiglu && n_glob < p.N) {
+    if (p.gate_bias) gate_b = __ldg(p.gate_bias + n_glob);
+    if (p.up_bias) up_b = __ldg(p.up_bias + n_glob);
+  }
 
   // Output tiles are staged in the (now idle) pipeline buffers as [batch row][128
   // features] and leave through bulk tensor stores: one instruction per box instead of
@@ -551,7 +568,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           }
         }
 #pragma unroll
-        for (int j = 0; j < 16; ++j) g[j] = swiglu ? gated_f<GENERAL>(g[j], u[j], act) : g[j];
+        for (int j = 0; j < 16; ++j) g[j] = swiglu ? gated_f<GENERAL>(g[j] + gate_b, u[j] + up_b, act) : g[j];
         if (p.post_scale) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) g[j] *= s_pscale[c0 + j];
@@ -663,7 +680,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
       }
     }
     if (tail_ok && store_y && tid == 0 && m_base + split * CW < p.M) {
-      tma_store_2d(&tm_y, smem_base + out_off, tile * kTileN, m_base + split * CW);
+      store_tile(smem_base + out_off, m_base + split * CW);
       if (residual) tma_store_2d(&tm_h, smem_base + h_off, tile * kTileN, m_base + split * CW);
       tma_store_commit();
       tma_store_wait_read();
@@ -699,7 +716,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
             for (int j = 0; j < 16; ++j) u[j] *= s_rscale[g * 16 + j];
           }
 #pragma unroll
-          for (int j = 0; j < 16; ++j) v[j] = gated_f<GENERAL>(v[j], u[j], act);
+          for (int j = 0; j < 16; ++j) v[j] = gated_f<GENERAL>(v[j] + gate_b, u[j] + up_b, act);
         }
         if (p.post_scale) {
 #pragma unroll
@@ -725,7 +742,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
       } else if (tid == 0) {
         for (int g = g0; g < g1; ++g)
           if (m_base + g * 16 < p.M)
-            tma_store_2d(&tm_y, smem_base + (uint32_t)(g - g0) * grp_bytes, tile * kTileN, m_base + g * 16);
+            store_tile(smem_base + (uint32_t)(g - g0) * grp_bytes, m_base + g * 16);
         tma_store_commit();
       }
     }
@@ -739,7 +756,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           float u[16];
           tmem_ld16(t_lane + p.m_pad + c0, u);
 #pragma unroll
-          for (int j = 0; j < 16; ++j) v[j] = gated_f<GENERAL>(v[j], u[j], act);
+          for (int j = 0; j < 16; ++j) v[j] = gated_f<GENERAL>(v[j] + gate_b, u[j] + up_b, act);
         }
         if (n_glob < p.N) {
 #pragma unroll
@@ -796,7 +813,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           for (int j = 0; j < 8; ++j) {
             const int m = m0 + j;
             if (m < m_lim && n_glob < p.N) {
-              const float r = swiglu ? gated_f<GENERAL>(g[j], u[j], act) : g[j];
+              const float r = swiglu ? gated_f<GENERAL>(g[j] + gate_b, u[j] + up_b, act) : g[j];
               if (p.out_f32) ((float*)p.Y)[(int64_t)(m_base + m) * p.ldy + n_glob] = r;
               else ((__nv_bfloat16*)p.Y)[(int64_t)(m_base + m) * p.ldy + n_glob] = __float2bfloat16_rn(r);
             }
@@ -853,14 +870,16 @@ static EncodeTiledFn get_encode() {
 }
 
 // 2-D bf16 row-major [rows, cols] tensor, box [box_rows, 64 cols], 128-byte swizzle.
-static int encode_map(CUtensorMap* tm, const void* ptr, int64_t rows, int64_t cols, int box_rows) {
+// heads > 0: that many such tensors `step` elements apart, rows of ld elements.
+static int encode_map(CUtensorMap* tm, const void* ptr, int64_t rows, int64_t cols, int box_rows, int heads = 0, int64_t ld = 0,
+                      int64_t step = 0) {
   EncodeTiledFn enc = get_encode();
   if (!enc) return fail(HB_ERR_CUDA, "cuTensorMapEncodeTiled entry point not available");
-  cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
-  cuuint64_t strides[1] = {(cuuint64_t)cols * 2};
-  cuuint32_t box[2] = {(cuuint32_t)kTileK, (cuuint32_t)box_rows};
-  cuuint32_t estr[2] = {1, 1};
-  CUresult r = enc(tm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), dims, strides,
+  cuuint64_t dims[3] = {(cuuint64_t)cols, (cuuint64_t)rows, (cuuint64_t)heads};
+  cuuint64_t strides[2] = {(cuuint64_t)(heads ? ld : cols) * 2, (cuuint64_t)step * 2};
+  cuuint32_t box[3] = {(cuuint32_t)kTileK, (cuuint32_t)box_rows, 1};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = enc(tm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, heads ? 3 : 2, const_cast<void*>(ptr), dims, strides,
                    box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
                    CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
   if (r != CUDA_SUCCESS) return fail(HB_ERR_CUDA, "cuTensorMapEncodeTiled failed with code %d", (int)r);
@@ -869,16 +888,17 @@ static int encode_map(CUtensorMap* tm, const void* ptr, int64_t rows, int64_t co
 
 // Output map: [rows, cols] elements of elt bytes, row stride ld elements, box
 // [box_rows, 128 cols], no swizzle (the kernel stages rows of 128 features densely).
+// heads > 0: that many such tensors `step` elements apart.
 static int encode_out_map(CUtensorMap* tm, void* ptr, int64_t rows, int64_t cols, int64_t ld, bool f32,
-                          int box_rows) {
+                          int box_rows, int heads = 0, int64_t step = 0) {
   EncodeTiledFn enc = get_encode();
   if (!enc) return fail(HB_ERR_CUDA, "cuTensorMapEncodeTiled entry point not available");
   const cuuint64_t elt = f32 ? 4 : 2;
-  cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
-  cuuint64_t strides[1] = {(cuuint64_t)ld * elt};
-  cuuint32_t box[2] = {(cuuint32_t)kTileN, (cuuint32_t)box_rows};
-  cuuint32_t estr[2] = {1, 1};
-  CUresult r = enc(tm, f32 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT32 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, ptr, dims,
+  cuuint64_t dims[3] = {(cuuint64_t)cols, (cuuint64_t)rows, (cuuint64_t)heads};
+  cuuint64_t strides[2] = {(cuuint64_t)ld * elt, (cuuint64_t)step * elt};
+  cuuint32_t box[3] = {(cuuint32_t)kTileN, (cuuint32_t)box_rows, 1};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = enc(tm, f32 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT32 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, heads ? 3 : 2, ptr, dims,
                    strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_NONE,
                    CU_TENSOR_MAP_L2_PROMOTION_NONE, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
   if (r != CUDA_SUCCESS) return fail(HB_ERR_CUDA, "cuTensorMapEncodeTiled (output) failed with code %d", (int)r);
@@ -890,6 +910,13 @@ bool gemm_tc_supported(int64_t M, int64_t N, int64_t K, hb_dtype dtype) {
   // (rows must be 16-byte multiples)
   return dtype == HB_BF16 && M >= 1 && N >= 1 && K >= 8 && K % 8 == 0 &&
          N < (1ll << 30) && M < (1ll << 30);
+}
+
+bool gemm_tc_heads_supported(int64_t N, int64_t K, bool out_f32, const TcHeads& h) {
+  const int64_t elt = out_f32 ? 4 : 2;
+  return h.heads >= 1 && h.heads <= 65535 && K % 8 == 0 && h.ldx % 8 == 0 && h.x_step % 8 == 0 && h.ldx >= K && h.x_step >= K &&
+         (N * elt) % 16 == 0 && (h.ldy * elt) % 16 == 0 && (h.y_step * elt) % 16 == 0 && h.y_step >= N &&
+         (int64_t)h.heads * N < (1ll << 30);
 }
 
 static int pick_splits(int units, int k_chunks, int slots) {
@@ -914,7 +941,7 @@ static int pick_cluster_splits(int units, int k_chunks, int sm_count) {
 }
 
 int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int64_t N, int64_t K,
-                 int epilogue, bool out_f32, int device, int force_splits, const TcGroups* groups) {
+                 int epilogue, bool out_f32, int device, int force_splits, const TcGroups* groups, const TcHeads* heads) {
   if (!gemm_tc_supported(M, N, K, HB_BF16))
     return fail(HB_ERR_INVALID_ARG, "gemm_tc: unsupported shape M=%lld N=%lld K=%lld", (long long)M,
                 (long long)N, (long long)K);
@@ -937,6 +964,12 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
                  (groups->ldx && (groups->ldx < K || groups->ldx % 8)) || (groups->shared_w && (groups->shared_k % 8 ||
                  groups->shared_n < 1 || groups->shared_k < 8 || groups->ldx < std::max(K, groups->shared_k)))))
     return fail(HB_ERR_INVALID_ARG, "gemm_tc: bad groups");
+  if (heads) {
+    if (groups || epilogue != kEpiStore || !gemm_tc_heads_supported(N, K, out_f32, *heads))
+      return fail(HB_ERR_INVALID_ARG, "gemm_tc: bad heads");
+    pl.heads = *heads;
+    pl.group_rows = (int)N;
+  }
   const int n_acc = epilogue == kEpiSwiGLU ? 2 : 1;
   if (epilogue == kEpiSwiGLU && N % 2) return fail(HB_ERR_INVALID_ARG, "gemm_tc: SwiGLU needs even N");
   const int64_t n_rows = epilogue == kEpiSwiGLU ? N / 2 : N;  // output features
@@ -968,13 +1001,13 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
   // the weight tile twice (the second time from L2) and need no, or a smaller, exchange
   // (measured: 8192 x 1024 at M = 128 15.4 -> 11.1 us, 1280 x 8192 19.0 -> 16.4 us).
   bool m_split = false;
-  if (tuned && !groups && n_acc == 1 && pl.m_pad >= 128 && (int64_t)pl.n_tiles * k_chunks <= 2048 &&
+  if (tuned && !groups && !heads && n_acc == 1 && pl.m_pad >= 128 && (int64_t)pl.n_tiles * k_chunks <= 2048 &&
       (epilogue == kEpiStore || epilogue == kEpiPush)) {
     pl.m_pad = 64;
     m_split = true;
   }
   pl.m_tiles = groups ? groups->max_tiles : (int)((M + pl.m_pad - 1) / pl.m_pad);
-  const int units = pl.n_tiles * (groups ? groups->likely_tiles : pl.m_tiles);
+  const int units = pl.n_tiles * (groups ? groups->likely_tiles : pl.m_tiles) * (heads ? heads->heads : 1);
   const int acc_cols = pl.m_pad * n_acc;
   pl.tmem_cols = acc_cols <= 32 ? 32 : acc_cols <= 64 ? 64 : acc_cols <= 128 ? 128 : acc_cols <= 256 ? 256 : 512;
   const size_t stage = (size_t)kTileN * kTileK * 2 * n_acc + (size_t)pl.m_pad * kTileK * 2;
@@ -1087,7 +1120,7 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
   // The tile counters sit in a block of FIXED size at the start of the workspace, so
   // that plans of different shapes sharing one workspace never see each other's
   // partials where they expect zeroed counters.
-  if (!pl.cluster && ((size_t)units * sizeof(int) > kCounterBlockBytes || groups)) pl.splits = 1;
+  if (!pl.cluster && ((size_t)units * sizeof(int) > kCounterBlockBytes || groups || heads)) pl.splits = 1;
   pl.ws_partials_bytes = (pl.splits > 1 && !pl.cluster) ? (size_t)units * pl.splits * n_acc * pl.m_pad * kTileN * sizeof(float) : 0;
   pl.ws_counters_bytes = (pl.splits > 1 && !pl.cluster) ? kCounterBlockBytes : 0;
   // opt in to the large dynamic shared memory window once per device (here, not at
@@ -1100,13 +1133,15 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
     std::lock_guard<std::mutex> lock(mu);
     if (cur >= 0 && cur < 64 && !dev_done[cur]) {
       // 227 KiB per CTA minus the kernel's static shared memory (barriers, flags, row scales)
-      for (auto* k : {gemm_tc_kernel<false, false>, gemm_tc_kernel<false, true>, gemm_tc_kernel<true, true>})
+      for (auto* k : {gemm_tc_kernel<false, false, false>, gemm_tc_kernel<false, true, false>, gemm_tc_kernel<true, true, false>,
+                      gemm_tc_kernel<false, false, true>})
         HB_CUDA_CHECK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024));
       dev_done[cur] = true;
     }
   }
-  rc = encode_map(&pl.tm_w, W, groups ? N * groups->groups : N, K, kTileN);
+  rc = encode_map(&pl.tm_w, W, groups ? N * groups->groups : heads ? N * heads->heads : N, K, kTileN);
   if (rc) return rc;
+  if (heads) return encode_map(&pl.tm_x, X, M, K, pl.m_pad, heads->heads, heads->ldx, heads->x_step);
   rc = encode_map(&pl.tm_x, X, M, groups ? pl.ldx : K, pl.m_pad);
   if (!rc && pl.N2) rc = encode_map(&pl.tm_w2, groups->shared_w, groups->shared_n, pl.K2, kTileN);
   return rc;
@@ -1154,6 +1189,8 @@ int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, voi
   p.k_chunks2 = (int)((pl.K2 + kTileK - 1) / kTileK);
   p.up_row_offset2 = (int)pl.N2;
   p.act2 = pl.act2;
+  p.gate_bias = pl.gate_bias;
+  p.up_bias = pl.up_bias;
   p.Y = Y;
   // counters first (16-byte aligned block), partials after
   p.counters = (int*)workspace;
@@ -1187,11 +1224,14 @@ int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, voi
     const int box_rows = pl.cluster ? pl.m_pad / pl.splits : 16;
     // groups of different widths share the rows: columns between one's width and the next
     // multiple of 128 may be written, and every reader of them multiplies them by zero
-    int rc = encode_out_map(&tm_y, Y, pl.M, pl.groups ? std::min(ldy, std::max(pl.N, pl.N2)) : pl.N, ldy, pl.out_f32, box_rows);
+    int rc = encode_out_map(&tm_y, Y, pl.M, pl.groups ? std::min(ldy, std::max(pl.N, pl.N2)) : pl.N, ldy, pl.out_f32, box_rows,
+                            pl.heads.heads, pl.heads.y_step);
     if (rc) return rc;
   }
   CUtensorMap tm_h;
   memset(&tm_h, 0, sizeof(tm_h));
+  if (pl.heads.heads && (!p.tma_store || link || ldy != pl.heads.ldy))
+    return fail(HB_ERR_INVALID_ARG, "gemm_tc: products of heads need the output rows they were planned for and no link");
   if (pl.groups && !p.tma_store) return fail(HB_ERR_INVALID_ARG, "gemm_tc: grouped plans need output rows of 16-byte multiples");
   if (pl.N2) tm_h = pl.tm_w2;
   if (pl.epilogue == kEpiResidual) {
@@ -1241,7 +1281,8 @@ int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, voi
     p.rs_eps = link->eps;
   }
   const unsigned n_tiles = (unsigned)std::max(pl.n_tiles, p.n_tiles2), m_tiles = (unsigned)pl.m_tiles;
-  const dim3 grid((p.m_fast ? m_tiles : n_tiles) * (unsigned)pl.splits, p.m_fast ? n_tiles : m_tiles);
+  const dim3 grid((p.m_fast ? m_tiles : n_tiles) * (unsigned)pl.splits, p.m_fast ? n_tiles : m_tiles,
+                  (unsigned)std::max(1, pl.heads.heads));
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = grid;
   cfg.blockDim = dim3(kTcThreads);
@@ -1264,8 +1305,10 @@ int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, voi
   }
   cfg.attrs = attr;
   cfg.numAttrs = na;
-  auto* kernel = pl.groups ? gemm_tc_kernel<true, true>
-                           : pl.act.silu() ? gemm_tc_kernel<false, false> : gemm_tc_kernel<false, true>;
+  const bool general = !pl.act.silu() || pl.gate_bias || pl.up_bias;
+  auto* kernel = pl.groups ? gemm_tc_kernel<true, true, false>
+                 : pl.heads.heads ? gemm_tc_kernel<false, false, true>
+                 : general ? gemm_tc_kernel<false, true, false> : gemm_tc_kernel<false, false, false>;
   HB_CUDA_CHECK(cudaLaunchKernelEx(&cfg, kernel, pl.tm_w, pl.tm_x, tm_y, tm_h, p));
   return HB_OK;
 }

@@ -22,7 +22,7 @@ struct LayeredDesign {
   bool (*serves)(const Json&);
   int (*read)(const Json&, LayeredSpec*);
 };
-static const LayeredDesign kDesigns[] = {{is_latarax, read_latarax}, {is_biberax, read_biberax}};
+static const LayeredDesign kDesigns[] = {{is_latarax, read_latarax}, {is_biberax, read_biberax}, {is_badolix, read_badolix}};
 
 static const LayeredDesign* design_of(const Json& config) {
   for (const LayeredDesign& d : kDesigns)
@@ -69,6 +69,12 @@ struct Loader {
     lin->K = pad8(k);
     return dev_alloc(e, &lin->w, (size_t)n * lin->K * e->es, true);
   }
+  int part(const LayeredLinear& lin, const ProjPart& p) {
+    if (!p.of) return part(lin, p.tensor, p.offset, p.rows, m->spec.width);
+    uint8_t* dst = (uint8_t*)lin.w + (size_t)p.offset * lin.K * e->es;
+    m->params += p.rows * m->spec.width;
+    return src.fetch(p.tensor, p.of, m->spec.width, p.first, p.rows, 0, m->spec.width, dst, e->dtype, lin.K);
+  }
   int linear(LayeredLinear* lin, const std::string& name, int64_t n, int64_t k) {
     int rc = alloc(lin, pad8(n), k);
     return rc ? rc : part(*lin, name, 0, n, k);
@@ -99,11 +105,10 @@ struct Loader {
                const std::string& norm) {
     const int S = m->spec.streams;
     int rc;
-    if (in.empty()) {  // one plain stream: x += y
-      const std::vector<float> one(1, 1.f);
+    if (in.empty()) {  // one plain stream: x += mult * y
       for (float** p : {&q->in, &q->out, &q->mix}) {
         if ((rc = dev_alloc(e, (void**)p, 4))) return rc;
-        if ((rc = upload(*p, one))) return rc;
+        if ((rc = upload(*p, std::vector<float>(1, p == &q->out ? m->spec.residual_mult : 1.f)))) return rc;
       }
     } else {
       if ((rc = small(&q->in, in, 1, S, 1.f / S))) return rc;
@@ -133,12 +138,65 @@ struct Loader {
       l->buckets = src.generated() ? 32 : (int)shape[0];  // the number of buckets is the tensor's own
       if ((rc = small(&l->rel, mx.attn_rel, l->buckets, a.heads, 0.f))) return rc;
     }
+    if (a.rank && (rc = latent(l, mx))) return rc;
     if (!a.rotation.empty()) {
       if ((rc = dev_alloc(e, (void**)&l->rotation, a.rotation.size() * 8))) return rc;
       HB_CUDA_CHECK(cudaMemcpyAsync(l->rotation, a.rotation.data(), a.rotation.size() * 8, cudaMemcpyHostToDevice, e->stream));
       HB_CUDA_CHECK(cudaStreamSynchronize(e->stream));
     }
     return HB_OK;
+  }
+  int latent(LayeredLayer* l, const MixerSpec& mx) {
+    const AttentionSpec& a = mx.attn;
+    const int64_t H = a.heads, C = a.rank;
+    const size_t uk = (size_t)H * a.dim * C * e->es;
+    int rc;
+    if ((rc = vector(&l->latent_norm, mx.attn_latent_norm, C, 1.f))) return rc;
+    if ((rc = dev_alloc(e, &l->uk_t, uk)) || (rc = dev_alloc(e, &l->uv, (size_t)H * a.vdim * C * e->es))) return rc;
+    if ((rc = src.fetch_all(mx.attn_uv, H * a.vdim, C, l->uv, e->dtype))) return rc;
+    e->named[mx.attn_uv] = {l->uv, H * a.vdim, C};
+    m->params += H * (a.dim + a.vdim) * C;
+    void* rows = nullptr;
+    HB_CUDA_CHECK(cudaMalloc(&rows, uk));
+    rc = src.fetch_all(mx.attn_uk, H * a.dim, C, rows, e->dtype);
+    if (!rc) rc = transpose_matrices(e->stream, l->uk_t, rows, H, a.dim, C, e->es);
+    const cudaError_t ce = cudaStreamSynchronize(e->stream);
+    cudaFree(rows);
+    if (rc) return rc;
+    HB_CUDA_CHECK(ce);
+    return HB_OK;
+  }
+  // convolution weights [channels, taps] as [taps, channels], steps, decays
+  int state_space(LayeredLayer* l, const MixerSpec& mx) {
+    const RecurrenceSpec& r = mx.rec;
+    const int64_t n = r.conv_channels();
+    int rc;
+    if ((rc = dev_alloc(e, (void**)&l->conv_w, (size_t)n * r.conv_taps * 4))) return rc;
+    m->params += n * r.conv_taps;
+    float* rows = nullptr;
+    HB_CUDA_CHECK(cudaMalloc((void**)&rows, (size_t)n * r.conv_taps * 4));
+    rc = src.fetch_all(mx.rec_conv, n, r.conv_taps, rows, HB_F32);
+    if (!rc) rc = transpose_matrices(e->stream, l->conv_w, rows, 1, n, r.conv_taps, 4);
+    const cudaError_t ce = cudaStreamSynchronize(e->stream);
+    cudaFree(rows);
+    if (rc) return rc;
+    HB_CUDA_CHECK(ce);
+    if ((rc = vector(&l->conv_b, mx.rec_conv_bias, n, 0.f))) return rc;
+    if ((rc = vector(&l->dt_bias, mx.rec_dt_bias, r.heads, 0.f))) return rc;
+    if ((rc = vector(&l->a_log, mx.rec_a_log, r.heads, 0.f))) return rc;
+    return vector(&l->skip, mx.rec_skip, r.heads, 1.f);
+  }
+  // biases of a dense feed-forward, as long as the padded rows they meet
+  int biases(LayeredLayer* l, const FeedForwardSpec& f) {
+    int rc = vector(&l->down_b, f.down_bias, m->spec.width, 0.f);
+    for (auto b : {std::make_pair(&l->gate_b, &f.gate_bias), std::make_pair(&l->up_b, &f.up_bias)}) {
+      if (rc || b.second->empty()) continue;
+      if ((rc = dev_alloc(e, (void**)b.first, (size_t)l->ffp * 4, true))) return rc;
+      e->named[*b.second] = {*b.first, 1, f.ff, 0, HB_F32};
+      m->params += f.ff;
+      if (!src.generated()) rc = src.fetch_all(*b.second, 1, f.ff, *b.first, HB_F32);
+    }
+    return rc;
   }
   int gated(LayeredLinear* gate_up, LayeredLinear* down, int64_t* ffp, const FeedForwardSpec& f) {
     const int64_t W = m->spec.width;
@@ -170,7 +228,7 @@ struct Loader {
     e->named[s.router] = {x->router, E, W};
     m->params += E * W;
     if (shared.ff && (rc = gated(&x->shared_gate_up, &x->shared_down, &x->shared_ffp, shared))) return rc;
-    return small(&x->router_bias, s.router_bias, 1, E, 0.f);
+    return vector(&x->router_bias, s.router_bias, E, 0.f);
   }
 };
 }  // namespace
@@ -192,8 +250,17 @@ static int layered_load(hb_engine* e, TensorSource& src) {
     e->named[s.pos] = {m->pos, s.max_positions, W};
     m->params += s.max_positions * W;
   }
-  if ((rc = ld.alloc(&m->head, s.vocab, W))) return rc;
-  if ((rc = ld.part(m->head, s.head, 0, s.vocab, W))) return rc;
+  if (!s.head.empty()) {
+    if ((rc = ld.alloc(&m->head, s.vocab, W))) return rc;
+    if ((rc = ld.part(m->head, s.head, 0, s.vocab, W))) return rc;
+  } else if (W % 8 == 0) {  // the embedding table itself
+    m->head.w = m->embed;
+    m->head.N = s.vocab;
+    m->head.K = W;
+  } else {
+    if ((rc = ld.alloc(&m->head, s.vocab, W))) return rc;
+    if ((rc = src.fetch_all(s.embed, s.vocab, W, m->head.w, e->dtype, m->head.K))) return rc;
+  }
   if ((rc = ld.small(&m->final_norm, s.final_norm, 1, W, 1.f - s.norm_offset))) return rc;
   m->layers.resize(s.layers.size());
   for (size_t i = 0; i < s.layers.size(); ++i) {
@@ -208,19 +275,21 @@ static int layered_load(hb_engine* e, TensorSource& src) {
       if (mx.rec.rank < 1) return fail(HB_ERR_IO, "%s is empty", mx.ra1.tensor.c_str());
     }
     int64_t n = 0;
-    const ProjPart* parts[] = {&mx.aq, &mx.ak, &mx.av, &mx.ag, &mx.rq, &mx.rk, &mx.rv, &mx.rg, &mx.ra1};
+    const ProjPart* parts[] = {&mx.aq, &mx.ak, &mx.av, &mx.ag, &mx.rq, &mx.rk, &mx.rv, &mx.rg, &mx.ra1, &mx.rx, &mx.rdt};
     for (const ProjPart* p : parts)
       if (p->rows) n = std::max(n, p->offset + p->rows);
     if ((rc = ld.alloc(&l.proj, pad8(n), W))) return rc;
     for (const ProjPart* p : parts)
-      if (p->rows && (rc = ld.part(l.proj, p->tensor, p->offset, p->rows, W))) return rc;
+      if (p->rows && (rc = ld.part(l.proj, *p))) return rc;
     if (mx.has_attn && (rc = ld.attention(&l, mx))) return rc;
     if (mx.has_rec) {
       const RecurrenceSpec& r = mx.rec;
       const int64_t hd = (int64_t)r.heads * r.dim, hv = (int64_t)r.heads * r.vdim;
       if ((rc = ld.linear(&l.rec_o, mx.rec_o, W, hv))) return rc;
       if ((rc = ld.small(&l.rec_norm, mx.rec_norm, 1, r.norm_per_head ? r.vdim : hv, 1.f))) return rc;
-      if (r.low_rank_decay) {
+      if (r.per_token_decay) {
+        if ((rc = ld.state_space(&l, mx))) return rc;
+      } else if (r.low_rank_decay) {
         if ((rc = dev_alloc(e, (void**)&l.a2, (size_t)hd * r.rank * 4))) return rc;
         if ((rc = src.fetch_all(mx.rec_a2, hd, r.rank, l.a2, HB_F32))) return rc;
         e->named[mx.rec_a2] = {l.a2, hd, r.rank, 0, HB_F32};
@@ -238,6 +307,7 @@ static int layered_load(hb_engine* e, TensorSource& src) {
     if ((rc = ld.sublayer(&l.sub1, sp.hc1_in, sp.hc1_out, sp.hc1_mix, sp.norm1))) return rc;
     if (sp.moe.experts) rc = ld.experts(&l.moe, sp.moe, sp.ffn);
     else if (sp.ffn.ff) rc = ld.gated(&l.gate_up, &l.down, &l.ffp, sp.ffn);
+    if (!rc && sp.ffn.ff && !sp.moe.experts) rc = ld.biases(&l, sp.ffn);
     if (rc) return rc;
     if (sp.has_ffn()) {
       if ((rc = ld.sublayer(&l.sub2, sp.hc2_in, sp.hc2_out, sp.hc2_mix, sp.norm2))) return rc;
@@ -267,7 +337,7 @@ static size_t layered_layout(const hb_engine* e, LayeredStep* s) {
   s->off_short = l.take((size_t)s->segs * 4);
   s->off_long = l.take((size_t)s->n_long * sizeof(RowRange));
   s->off_chunk = l.take((size_t)s->n_chunks * sizeof(RowRange));
-  s->off_tile = l.take((size_t)s->n_tiles * sizeof(RowRange));
+  for (int k = 0; k < kTileKinds; ++k) s->off_tile[k] = l.take((size_t)s->n_tiles[k] * sizeof(RowRange));
   s->off_row_list = l.take((size_t)s->rows * 4);
   s->off_tables = l.take((size_t)s->segs * e->max_blocks_per_seq * 4);
   return l.bytes;
@@ -291,8 +361,13 @@ static SpanAttention span_args(const hb_engine* e, size_t i, const LayeredStep& 
   a.max_blocks = e->max_blocks_per_seq; a.num_blocks = e->num_blocks;
   a.row_seg = (const int32_t*)(e->d_inputs + s.off_row_seg);
   a.pos = (const int32_t*)(e->d_inputs + s.off_pos);
-  a.heads = as.heads; a.kv_heads = as.kv_heads; a.dim = as.dim; a.vdim = as.vdim;
-  a.window = as.window; a.keep_first = as.keep_first; a.chunk = as.chunk; a.scale = as.scale;
+  a.heads = as.heads; a.kv_heads = as.cached_heads(); a.dim = as.key_width(); a.vdim = as.value_width();
+  a.window = as.window; a.keep_first = as.keep_first; a.chunk = as.chunk; a.scale = as.scale; a.softcap = as.softcap;
+  if (as.rank) {
+    a.q = m->latent_q; a.ld_q = (int64_t)as.heads * a.dim;
+    a.out = m->latent_o; a.ld_out = (int64_t)as.heads * a.vdim;
+    a.vc = nullptr;
+  }
   if (as.values_are_keys) {  // the second pool holds the keys' scales
     a.key_scale = (const float*)a.vc;
     a.vc = nullptr;
@@ -304,6 +379,40 @@ static SpanAttention span_args(const hb_engine* e, size_t i, const LayeredStep& 
     a.ld_gate = l.proj.N;
   }
   return a;
+}
+
+static LatentPrep latent_args(const hb_engine* e, size_t i, const LayeredStep& s) {
+  const LayeredModel* m = e->lm.get();
+  const MixerSpec& mx = m->spec.layers[i].mixer;
+  const LayeredLayer& l = m->layers[i];
+  const AttentionSpec& as = mx.attn;
+  LatentPrep p;
+  p.p = m->proj; p.ld = l.proj.N; p.off_q = (int)mx.aq.offset; p.off_c = (int)mx.ak.offset;
+  p.heads = as.heads; p.dim = as.dim; p.rot_dim = as.rot_dim; p.rank = as.rank;
+  p.q = m->latent_q; p.ld_q = (int64_t)as.heads * as.key_width();
+  p.pos = (const int32_t*)(e->d_inputs + s.off_pos);
+  p.slots = (const int64_t*)(e->d_inputs + s.off_slots);
+  p.kc = e->kc[l.kv_pool]; p.num_blocks = e->num_blocks;
+  p.norm = l.latent_norm; p.eps = m->spec.eps;
+  p.rotation = l.rotation; p.pairs = (int)as.rotation.size(); p.rotation_gain = as.rotation_gain;
+  return p;
+}
+
+// The products of latent attention, head by head: W_uk^T on the queries' first parts, W_uv on what the
+// heads gathered from the latents.
+static TcHeads latent_q_heads(const LayeredLayer& l, const AttentionSpec& a) {
+  TcHeads h;
+  h.heads = a.heads;
+  h.ldx = l.proj.N; h.x_step = a.dim + a.rot_dim;
+  h.ldy = (int64_t)a.heads * a.key_width(); h.y_step = a.key_width();
+  return h;
+}
+static TcHeads latent_v_heads(const LayeredLayer& l, const AttentionSpec& a) {
+  TcHeads h;
+  h.heads = a.heads;
+  h.ldx = (int64_t)a.heads * a.rank; h.x_step = a.rank;
+  h.ldy = l.attn_o.K; h.y_step = a.vdim;
+  return h;
 }
 
 // Queries in place, keys and values to their slots; false: the design only needs the K/V write.
@@ -322,6 +431,8 @@ static bool prep_args(const hb_engine* e, size_t i, const LayeredStep& s, Attent
   p->q_bias = l.q_bias; p->k_bias = l.k_bias; p->q_norm = l.q_norm; p->k_norm = l.k_norm;
   p->eps = m->spec.eps;
   p->rotation = l.rotation; p->pairs = (int)as.rotation.size();
+  p->halves = as.rotation_halves ? 1 : 0; p->rotation_gain = as.rotation_gain;
+  if (as.kv_from >= 0) p->kc = p->vc = nullptr;  // that layer has written them
   if (as.values_are_keys) p->key_scale = (float*)p->vc;
   return true;
 }
@@ -393,6 +504,7 @@ static TcGroups down_groups(TcGroups g, const LayeredExperts& w) {
 static MoeRouting moe_args(const LayeredModel* m, const ExpertsSpec& x, bool shared, const TcGroups& g) {
   MoeRouting r;
   r.experts = x.experts; r.top = x.top; r.shared = shared ? 1 : 0;
+  r.sigmoid = x.sigmoid ? 1 : 0; r.groups = x.groups; r.keep = x.keep;
   r.m_pad = g.m_pad; r.max_tiles = g.max_tiles;
   r.ids = m->moe_ids; r.rank = m->moe_rank; r.place = m->moe_place; r.weight = m->moe_weight;
   r.count = m->moe_count; r.first = m->moe_first; r.tile_group = m->moe_tiles;
@@ -401,18 +513,18 @@ static MoeRouting moe_args(const LayeredModel* m, const ExpertsSpec& x, bool sha
 
 // Prompt portions as tiles, decoded tokens as rows; sizes the tensor-core kernels do not take go
 // row by row.
-static int issue_attention(hb_engine* e, const SpanAttention& a, const LayeredStep& s) {
+static int issue_attention(hb_engine* e, const SpanAttention& a, int kind, const LayeredStep& s) {
   LayeredModel* m = e->lm.get();
   cudaStream_t st = e->stream;
   const int32_t* rows = (const int32_t*)(e->d_inputs + s.off_row_list);
   int rc;
-  if (!m->tile_positions || span_attention_tile_positions(a, e->dtype) < m->tile_positions) {
+  if (kind < 0) {
     ++e->last_launches;
     return span_attention_rows(st, a, rows, s.rows, e->dtype);
   }
-  if (s.n_tiles) {
+  if (s.n_tiles[kind]) {
     ++e->last_launches;
-    if ((rc = span_attention_tiles(st, a, (const RowRange*)(e->d_inputs + s.off_tile), s.n_tiles))) return rc;
+    if ((rc = span_attention_tiles(st, a, (const RowRange*)(e->d_inputs + s.off_tile[kind]), s.n_tiles[kind]))) return rc;
   }
   if (!s.n_token_rows) return HB_OK;
   ++e->last_launches;
@@ -420,7 +532,7 @@ static int issue_attention(hb_engine* e, const SpanAttention& a, const LayeredSt
   // the longest span a row can have decides the split: it is the same in every replay of a graph
   const int64_t span = a.chunk > 0 ? a.chunk : a.window;
   const int64_t longest = span > 0 ? span + a.keep_first : a.max_blocks * HB_BLOCK_SIZE;
-  const int64_t blocks = std::min<int64_t>(longest / HB_BLOCK_SIZE + 2, a.max_blocks), units = (int64_t)s.n_token_rows * a.kv_heads;
+  const int64_t blocks = std::min<int64_t>(longest / HB_BLOCK_SIZE + 2, a.max_blocks), units = (int64_t)s.n_token_rows * span_attention_token_units(a);
   // as many as are resident at once, every one with some blocks for each of its warps
   int64_t splits = std::min<int64_t>(std::min(kSplitUnits, span_attention_tokens_slots(a)) / units, (blocks + 7) / 8);
   splits = std::max<int64_t>(1, std::min<int64_t>(splits, 16));
@@ -460,7 +572,7 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   m->row_cap = R;
   m->max_chunks = e->max_batch / kRecChunk + std::min(m->max_segs, e->max_batch / (kShortSegment + 1)) + 1;
   int64_t max_attn = 0, max_rec = 0, max_o = 0, max_ffp = 0, max_cum = 0, max_state = 0, max_part = 0;
-  int64_t max_experts = 0, max_top = 0, max_eff = 0, max_tiles = 0;
+  int64_t max_experts = 0, max_top = 0, max_eff = 0, max_tiles = 0, max_conv = 0, max_latent_q = 0, max_latent_o = 0;
   for (size_t i = 0; i < s.layers.size(); ++i) {
     LayeredLayer& l = m->layers[i];
     const MixerSpec& mx = s.layers[i].mixer;
@@ -468,20 +580,30 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
     max_ffp = std::max(max_ffp, l.ffp);
     if (mx.has_attn) {
       const AttentionSpec& a = mx.attn;
-      l.kv_pool = (int)e->kc.size();
-      const size_t kb = (size_t)a.kv_heads * HB_BLOCK_SIZE * a.dim * es;
-      // values that are the keys: the second pool holds one scale per token
-      const size_t vb = a.values_are_keys ? (size_t)HB_BLOCK_SIZE * 4 : (size_t)a.kv_heads * HB_BLOCK_SIZE * a.vdim * es;
-      void *k = nullptr, *v = nullptr;
-      // unwritten slots may be fetched (and masked): keep them finite
-      if ((rc = dev_alloc(e, &k, kb * e->num_blocks, true))) return rc;
-      if ((rc = dev_alloc(e, &v, vb * e->num_blocks, true))) return rc;
-      e->kc.push_back(k);
-      e->vc.push_back(v);
-      e->k_block_bytes.push_back(kb);
-      e->v_block_bytes.push_back(vb);
+      if (a.kv_from >= 0) {
+        l.kv_pool = m->layers[a.kv_from].kv_pool;
+      } else {
+        l.kv_pool = (int)e->kc.size();
+        const size_t kb = (size_t)a.cached_heads() * HB_BLOCK_SIZE * a.key_width() * es;
+        // values that are the keys: the second pool holds one scale per token; a latent: nothing
+        const size_t vb = a.values_are_keys ? (size_t)HB_BLOCK_SIZE * 4 : (size_t)(a.kv_heads * HB_BLOCK_SIZE * a.value_pool_width()) * es;
+        void *k = nullptr, *v = nullptr;
+        // unwritten slots may be fetched (and masked): keep them finite
+        if ((rc = dev_alloc(e, &k, kb * e->num_blocks, true))) return rc;
+        if (vb && (rc = dev_alloc(e, &v, vb * e->num_blocks, true))) return rc;
+        e->kc.push_back(k);
+        e->vc.push_back(v);
+        e->k_block_bytes.push_back(kb);
+        e->v_block_bytes.push_back(vb);
+      }
       max_attn = std::max(max_attn, l.attn_o.K);
-      max_part = std::max(max_part, (int64_t)kSplitUnits * 2 * (a.heads / a.kv_heads) * (a.vdim + 2));
+      max_part = std::max(max_part, (int64_t)kSplitUnits * 2 * (a.heads / a.cached_heads()) * (a.value_width() + 2));
+      if (a.rank) {
+        max_latent_q = std::max(max_latent_q, (int64_t)a.heads * a.key_width());
+        max_latent_o = std::max(max_latent_o, (int64_t)a.heads * a.rank);
+        l.latent_tc = e->use_tc && gemm_tc_heads_supported(a.rank, a.dim, false, latent_q_heads(l, a)) &&
+                      gemm_tc_heads_supported(a.vdim, a.rank, false, latent_v_heads(l, a));
+      }
       if (l.rel && (rc = build_distance_bias(e, &l, a, e->max_blocks_per_seq * HB_BLOCK_SIZE))) return rc;
     }
     if (const ExpertsSpec& x = s.layers[i].moe; x.experts) {
@@ -502,6 +624,12 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
       max_rec = std::max(max_rec, l.rec_o.K);
       max_o = std::max(max_o, (int64_t)r.heads * r.vdim);
       if (r.low_rank_decay) max_cum = std::max(max_cum, (int64_t)r.heads * r.dim);
+      if (r.per_token_decay) {
+        max_cum = std::max(max_cum, 2 * (int64_t)r.heads);
+        max_conv = std::max(max_conv, pad8(r.conv_channels()));
+        if (r.conv_taps > 1 &&
+            (rc = dev_alloc(e, &l.conv_state, (size_t)m->max_segs * (r.conv_taps - 1) * r.conv_channels() * es, true))) return rc;
+      }
       max_state = std::max(max_state, (int64_t)r.heads * r.dim * r.vdim);
     }
   }
@@ -514,6 +642,9 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   if ((rc = dev_alloc(e, &m->attn, (size_t)R * max_attn * es, true))) return rc;
   if ((rc = dev_alloc(e, &m->rec, (size_t)R * max_rec * es, true))) return rc;
   if ((rc = dev_alloc(e, (void**)&m->o, (size_t)R * max_o * 4, true))) return rc;
+  if (max_conv && (rc = dev_alloc(e, &m->conv, (size_t)R * max_conv * es, true))) return rc;
+  if (max_latent_q && (rc = dev_alloc(e, &m->latent_q, (size_t)R * max_latent_q * es, true))) return rc;
+  if (max_latent_o && (rc = dev_alloc(e, &m->latent_o, (size_t)R * max_latent_o * es, true))) return rc;
   if (e->use_tc) {
     if ((rc = dev_alloc(e, (void**)&m->cum, (size_t)R * max_cum * 4))) return rc;
     if ((rc = dev_alloc(e, (void**)&m->chunk_state, (size_t)m->max_chunks * max_state * 4))) return rc;
@@ -522,7 +653,16 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   for (size_t i = 0; i < s.layers.size(); ++i)
     if (s.layers[i].mixer.has_attn) {
       const int tp = span_attention_tile_positions(span_args(e, i, LayeredStep()), e->dtype);
-      if (tp > 0) m->tile_positions = m->tile_positions ? std::min(m->tile_positions, tp) : tp;
+      std::vector<int>& sizes = m->tile_sizes;
+      auto at = std::find(sizes.begin(), sizes.end(), tp);
+      if (tp < 1) continue;
+      if (at == sizes.end() && (int)sizes.size() < kTileKinds) at = sizes.insert(sizes.end(), tp);
+      if (at == sizes.end()) {  // as many sizes as there are lists: the largest that is small enough
+        for (auto k = sizes.begin(); k != sizes.end(); ++k)
+          if (*k < tp && (at == sizes.end() || *k > *at)) at = k;
+        if (at == sizes.end()) continue;
+      }
+      m->layers[i].tile_kind = (int)(at - sizes.begin());
     }
   if ((rc = dev_alloc(e, (void**)&m->y1, (size_t)R * m->Hp * 4, true))) return rc;
   if ((rc = dev_alloc(e, (void**)&m->y2, (size_t)R * m->Hp * 4, true))) return rc;
@@ -554,7 +694,7 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   cap.want = e->max_batch;
   cap.segs = cap.n_long = m->max_segs;
   cap.n_chunks = m->max_chunks;
-  cap.n_tiles = e->max_batch + m->max_segs;
+  for (size_t k = 0; k < m->tile_sizes.size(); ++k) cap.n_tiles[k] = e->max_batch / m->tile_sizes[k] + m->max_segs;
   e->inputs_bytes = layered_layout(e, &cap);
   if ((rc = dev_alloc(e, (void**)&e->d_inputs, e->inputs_bytes, true))) return rc;
   HB_CUDA_CHECK(cudaMallocHost((void**)&e->h_inputs, e->inputs_bytes));
@@ -580,7 +720,7 @@ static int layered_plans(hb_engine* e, int rows, LayeredPlans** out) {
   if (it != m->plans.end()) { *out = &it->second; return HB_OK; }
   LayeredPlans p;
   const size_t L = m->layers.size();
-  for (auto* v : {&p.proj, &p.attn_o, &p.rec_o, &p.gate_up, &p.down, &p.moe_gate_up, &p.moe_down}) v->resize(L);
+  for (auto* v : {&p.proj, &p.latent_q, &p.latent_v, &p.attn_o, &p.rec_o, &p.gate_up, &p.down, &p.moe_gate_up, &p.moe_down}) v->resize(L);
   size_t ws = 0;
   int rc;
   auto plan = [&](TcGemmPlan* pl, const void* X, const LayeredLinear& w, int epi, bool f32) -> int {
@@ -592,10 +732,20 @@ static int layered_plans(hb_engine* e, int rows, LayeredPlans** out) {
   for (size_t i = 0; i < L; ++i) {
     LayeredLayer& l = m->layers[i];
     if ((rc = plan(&p.proj[i], m->h, l.proj, kEpiStore, false))) return rc;
+    if (l.latent_tc) {
+      const MixerSpec& mx = m->spec.layers[i].mixer;
+      const AttentionSpec& a = mx.attn;
+      const TcHeads q = latent_q_heads(l, a), v = latent_v_heads(l, a);
+      const void* X = (const uint8_t*)m->proj + mx.aq.offset * e->es;
+      if ((rc = gemm_tc_plan(&p.latent_q[i], X, l.uk_t, M, a.rank, a.dim, kEpiStore, false, e->device, 0, nullptr, &q))) return rc;
+      if ((rc = gemm_tc_plan(&p.latent_v[i], m->latent_o, l.uv, M, a.vdim, a.rank, kEpiStore, false, e->device, 0, nullptr, &v))) return rc;
+      ws = std::max(ws, std::max(p.latent_q[i].workspace_bytes(), p.latent_v[i].workspace_bytes()));
+    }
     if ((rc = plan(&p.attn_o[i], m->attn, l.attn_o, kEpiStore, true))) return rc;
     if ((rc = plan(&p.rec_o[i], m->rec, l.rec_o, kEpiStore, true))) return rc;
     if ((rc = plan(&p.gate_up[i], m->h, l.gate_up, kEpiSwiGLU, false))) return rc;
     p.gate_up[i].act = m->spec.layers[i].ffn.act;
+    p.gate_up[i].gate_bias = l.gate_b; p.gate_up[i].up_bias = l.up_b;
     if ((rc = plan(&p.down[i], m->act, l.down, kEpiStore, true))) return rc;
     const ExpertsSpec& x = m->spec.layers[i].moe;
     if (!x.experts) continue;
@@ -639,7 +789,8 @@ static int layered_prepare(hb_engine* e, const StepBatch& batch, StepExec* x) {
     if (t.n <= kShortSegment) ++s.n_short;
     else { ++s.n_long; s.n_chunks += (t.n + kRecChunk - 1) / kRecChunk; }
     if (t.n == 1) ++s.n_token_rows;
-    else if (m->tile_positions) s.n_tiles += (t.n + m->tile_positions - 1) / m->tile_positions;
+    else
+      for (size_t k = 0; k < m->tile_sizes.size(); ++k) s.n_tiles[k] += (t.n + m->tile_sizes[k] - 1) / m->tile_sizes[k];
   }
   x->rows = batch.rows;
   x->logits_compact = true;
@@ -654,9 +805,8 @@ static int layered_prepare(hb_engine* e, const StepBatch& batch, StepExec* x) {
   int32_t* shorts = (int32_t*)(in + s.off_short);
   RowRange* longs = (RowRange*)(in + s.off_long);
   RowRange* chunks = (RowRange*)(in + s.off_chunk);
-  RowRange* tiles = (RowRange*)(in + s.off_tile);
   int32_t* row_list = (int32_t*)(in + s.off_row_list);
-  int at_short = 0, at_long = s.n_short, n_long = 0, n_chunks = 0, n_tiles = 0, at_token = 0, at_row = s.n_token_rows;
+  int at_short = 0, at_long = s.n_short, n_long = 0, n_chunks = 0, n_tiles[kTileKinds] = {0}, at_token = 0, at_row = s.n_token_rows;
   int32_t* tables = (int32_t*)(in + s.off_tables);
   for (int g = 0; g < s.segs; ++g) {
     const StepSeg& t = batch.segs[g];
@@ -670,9 +820,11 @@ static int layered_prepare(hb_engine* e, const StepBatch& batch, StepExec* x) {
       for (int i = 0; i < t.n; i += kRecChunk)
         chunks[n_chunks++] = {g, t.row0 + i, std::min(kRecChunk, t.n - i), l.n++};
     }
-    if (t.n > 1 && m->tile_positions)
-      for (int i = 0; i < t.n; i += m->tile_positions)
-        tiles[n_tiles++] = {g, t.row0 + i, std::min(m->tile_positions, t.n - i), i / m->tile_positions};
+    for (size_t k = 0; t.n > 1 && k < m->tile_sizes.size(); ++k) {
+      RowRange* tiles = (RowRange*)(in + s.off_tile[k]);
+      const int size = m->tile_sizes[k];
+      for (int i = 0; i < t.n; i += size) tiles[n_tiles[k]++] = {g, t.row0 + i, std::min(size, t.n - i), i / size};
+    }
     for (int i = 0; i < t.n; ++i) {
       const int64_t p = t.pos0 + i;
       ids[t.row0 + i] = t.tokens[i];
@@ -754,7 +906,7 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
 
   prof_mark(e, kCatOther);
   if ((rc = streams_embed(st, m->x, m->h, m->embed, m->pos, ids, pos, m->layers[0].sub1.in, m->layers[0].sub1.norm, sp.norm_offset,
-                          rows, S, W, m->Hp, sp.vocab, sp.max_positions, sp.eps, e->dtype))) return rc;
+                          rows, S, W, m->Hp, sp.vocab, sp.max_positions, sp.eps, e->dtype, sp.embed_scale))) return rc;
   ++e->last_launches;
   for (size_t i = 0; i < m->layers.size(); ++i) {
     LayeredLayer& l = m->layers[i];
@@ -766,13 +918,28 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
     float* y = m->y1;
     if (mx.has_attn) {
       const SpanAttention a = span_args(e, i, s);
+      const AttentionSpec& as = mx.attn;
+      // one product per head of latent attention
+      auto heads = [&](const std::vector<TcGemmPlan>* plans, void* Y, const void* X, const void* w, int64_t N, int64_t K,
+                       const TcHeads& h) -> int {
+        ++e->last_launches;
+        prof_mark(e, kCatLatent);
+        if (l.latent_tc) return gemm_tc_run((*plans)[i], st, Y, h.ldy, e->d_gemm_ws, e->d_err);
+        return gemm_simt_heads(st, Y, X, w, rows, N, K, e->dtype, false, h);
+      };
+      if (as.rank && (rc = heads(pl ? &pl->latent_q : nullptr, m->latent_q, at(m->proj, mx.aq.offset), l.uk_t, as.rank, as.dim,
+                                 latent_q_heads(l, as)))) return rc;
       prof_mark(e, kCatRopeKv);
       AttentionPrep prep;
-      if (prep_args(e, i, s, &prep)) rc = attention_prepare(st, prep, rows, e->dtype);
+      if (as.rank) rc = latent_prepare(st, latent_args(e, i, s), rows, e->dtype);
+      else if (as.kv_from >= 0 && !l.rotation && !l.q_bias) rc = HB_OK;  // queries as projected, keys of another layer
+      else if (prep_args(e, i, s, &prep)) rc = attention_prepare(st, prep, rows, e->dtype);
       else rc = span_kv_write(st, a, at(m->proj, mx.ak.offset), at(m->proj, mx.av.offset), ldp, slots, rows, e->dtype);
       if (rc) return rc;
       prof_mark(e, kCatAttention);
-      if ((rc = issue_attention(e, a, s))) return rc;
+      if ((rc = issue_attention(e, a, l.tile_kind, s))) return rc;
+      if (as.rank && (rc = heads(pl ? &pl->latent_v : nullptr, m->attn, m->latent_o, l.uv, as.vdim, as.rank, latent_v_heads(l, as))))
+        return rc;
       prof_mark(e, kCatGemmO);
       if ((rc = gemm(pl ? &pl->attn_o : nullptr, i, y, m->attn, l.attn_o, true))) return rc;
       ++e->last_launches;  // the K/V write
@@ -786,13 +953,32 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
       r.heads = rs.heads; r.dim = rs.dim; r.vdim = rs.vdim;
       r.q_scale = rs.q_scale; r.silu_qkv = rs.silu_qkv ? 1 : 0;
       r.decay = l.decay; r.a2 = l.a2; r.a2_bias = l.a2_bias; r.rank = rs.rank; r.inv_tau = (float)(1.0 / rs.tau);
+      r.qk_heads = rs.qk_heads;
+      if (rs.per_token_decay) {
+        ShortConv c;
+        c.p = m->proj; c.ld = ldp; c.off = (int)mx.rx.offset; c.channels = (int)rs.conv_channels(); c.taps = rs.conv_taps;
+        c.w = l.conv_w; c.bias = l.conv_b; c.out = m->conv; c.ld_out = pad8(rs.conv_channels());
+        c.state = l.conv_state; c.segs = seg;
+        prof_mark(e, kCatConv);
+        if ((rc = short_conv(st, c, (const int32_t*)(in + s.off_short), s.n_short, (const RowRange*)(in + s.off_chunk), s.n_chunks,
+                             e->dtype))) return rc;
+        ++e->last_launches;
+        r.p = m->conv; r.ld = c.ld_out;
+        r.off_v = 0; r.off_k = rs.heads * rs.vdim; r.off_q = r.off_k + rs.qk_heads * rs.dim;
+        r.dt = at(m->proj, mx.rdt.offset); r.ld_dt = ldp;
+        r.dt_bias = l.dt_bias; r.a_log = l.a_log; r.skip = l.skip;
+      }
       r.state = l.state; r.o = m->o; r.ld_o = (int64_t)rs.heads * rs.vdim; r.segs = seg;
       prof_mark(e, kCatRecurrence);
       if ((rc = issue_recurrence(e, r, s))) return rc;
       prof_mark(e, kCatNorm);
-      const int groups = rs.norm_per_head ? rs.heads : 1, size = rs.norm_per_head ? rs.vdim : rs.heads * rs.vdim;
-      if ((rc = gated_group_norm(st, m->rec, l.rec_o.K, m->o, r.ld_o, at(m->proj, mx.rg.offset), ldp, l.rec_norm, rows, groups,
-                                 size, rs.gate_silu, sp.eps, e->dtype))) return rc;
+      GroupNorm n;
+      n.groups = rs.norm_per_head ? rs.heads : std::max(1, rs.gated_norm_groups);
+      n.size = rs.heads * rs.vdim / n.groups;
+      n.gate_silu = rs.gate_silu; n.gate_first = n.own_weights = rs.gated_norm_groups > 0;
+      n.eps = sp.eps;
+      if ((rc = gated_group_norm(st, m->rec, l.rec_o.K, m->o, r.ld_o, at(m->proj, mx.rg.offset), ldp, l.rec_norm, rows, n, e->dtype)))
+        return rc;
       prof_mark(e, kCatGemmO);
       if ((rc = gemm(pl ? &pl->rec_o : nullptr, i, y, m->rec, l.rec_o, true))) return rc;
       ++e->last_launches;  // the gated norm
@@ -825,18 +1011,19 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
         if ((rc = gemm(&pl->gate_up, i, m->act, m->h, l.gate_up, false))) return rc;
       } else {
         if ((rc = gemm(nullptr, i, m->gu, m->h, l.gate_up, false))) return rc;
-        if ((rc = gated_act(st, m->act, m->gu, rows, l.ffp, lsp.ffn.act, e->dtype))) return rc;
+        if ((rc = gated_act(st, m->act, m->gu, rows, l.ffp, lsp.ffn.act, e->dtype, l.gate_b, l.up_b))) return rc;
         ++e->last_launches;
       }
       prof_mark(e, kCatGemmDown);
       if ((rc = gemm(pl ? &pl->down : nullptr, i, m->y1, m->act, l.down, true))) return rc;
     }
+    fed.bias = l.down_b;
     if ((rc = boundary(l.sub2, lsp.moe.experts ? nullptr : m->y1, false, fed))) return rc;
   }
   if (s.want) {
     prof_mark(e, kCatNorm);
     if ((rc = streams_final(st, m->hf, m->x, (const int32_t*)(in + s.off_want), m->final_norm, sp.norm_offset, s.want, S, W, m->Hp, sp.eps,
-                            e->dtype))) return rc;
+                            e->dtype, sp.logit_scale))) return rc;
     prof_mark(e, kCatGemmLmHead);
     if (e->use_tc) rc = gemm_tc_run(*s.head_plan, st, e->d_logits, sp.vocab, e->d_gemm_ws, e->d_err);
     else rc = gemm_simt(st, e->d_logits, m->hf, m->head.w, s.want, m->head.N, m->head.K, e->dtype, true);
@@ -861,7 +1048,8 @@ static double layered_step_bytes(const hb_engine* e, const int32_t* ctx_lens, in
     const MixerSpec& mx = s.layers[i].mixer;
     if (mx.has_attn) {
       const AttentionSpec& a = mx.attn;
-      const double per_key = a.values_are_keys ? a.kv_heads * a.dim * es + 4.0 : a.kv_heads * (a.dim + a.vdim) * es;
+      const double per_key = a.rank ? a.key_width() * es : a.values_are_keys ? a.kv_heads * a.dim * es + 4.0 : a.kv_heads * (a.dim + a.vdim) * es;
+      if (a.rank) w += (double)a.heads * (a.dim + a.vdim) * a.rank * es;
       for (int64_t k = 0; k < n_seqs; ++k) {
         const int64_t ctx = ctx_lens ? ctx_lens[k] : 0;
         int64_t seen = ctx;
@@ -870,6 +1058,7 @@ static double layered_step_bytes(const hb_engine* e, const int32_t* ctx_lens, in
         w += ((double)seen + 1.0) * per_key;
       }
     }
+    if (mx.has_rec && mx.rec.per_token_decay) w += n * 2.0 * (mx.rec.conv_taps - 1) * mx.rec.conv_channels() * es;
     if (mx.has_rec) w += n * 2.0 * mx.rec.heads * mx.rec.dim * mx.rec.vdim * 4.0;
     w += n * (s.layers[i].has_ffn() ? 2.0 : 1.0) * 2.0 * s.streams * s.width * 4.0;
     if (const ExpertsSpec& x = s.layers[i].moe; x.experts)  // the experts a random batch chooses
@@ -887,11 +1076,14 @@ static double layered_gemm_bytes(const hb_engine* e, int64_t rows) {
   auto lin = [&](const LayeredLinear& q, double n_out, double out_es) {
     return q.w ? ((double)q.N * q.K + b * q.K) * es + b * n_out * out_es : 0.0;
   };
+  auto latent = [&](const AttentionSpec& a) {
+    return a.heads * ((double)(a.dim + a.vdim) * a.rank + b * (a.dim + 2.0 * a.rank + a.vdim)) * es;
+  };
   double t = lin(m->head, (double)m->head.N, 4.0);
   for (size_t i = 0; i < m->layers.size(); ++i) {
     const LayeredLayer& l = m->layers[i];
     t += lin(l.proj, (double)l.proj.N, es) + lin(l.attn_o, (double)l.attn_o.N, 4.0) + lin(l.rec_o, (double)l.rec_o.N, 4.0) +
-         lin(l.gate_up, (double)l.ffp, es) + lin(l.down, (double)l.down.N, 4.0);
+         (m->spec.layers[i].mixer.attn.rank ? latent(m->spec.layers[i].mixer.attn) : 0.0) + lin(l.gate_up, (double)l.ffp, es) + lin(l.down, (double)l.down.N, 4.0);
     if (const ExpertsSpec& x = m->spec.layers[i].moe; x.experts) {
       const double picks = b * x.top, active = x.experts * (1.0 - std::pow(1.0 - 1.0 / x.experts, picks));
       const LayeredExperts& w = l.moe;

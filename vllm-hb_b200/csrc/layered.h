@@ -1,7 +1,7 @@
 // Models described layer by layer: every layer has a mixer (attention, a gated linear
 // recurrence, or both side by side) and possibly a feed-forward (one gated layer, or a mixture of
 // them), over one or several residual streams held in fp32.  The mechanisms and their constants are
-// data (LayeredSpec); a design's reader (latarax.cc, biberax.cc) turns its config.json and tensor
+// data (LayeredSpec); a design's reader (latarax.cc, biberax.cc, badolix.cc) turns its config.json and tensor
 // names into it.
 #pragma once
 
@@ -25,9 +25,24 @@ struct AttentionSpec {
   int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
   float scale = 1.f;
   int window = 0, keep_first = 0, chunk = 0;
-  // interleaved rotation of the first 2 * rotation.size() channels of queries and keys; the
-  // angle of pair i is position * rotation[i]
+  float softcap = 0.f;              // scores s become softcap * tanh(s / softcap) (0: they stay)
+  // rotation of the first 2 * rotation.size() channels of queries and keys, channel 2i with 2i + 1 or
+  // (halves) channel i with i + rotation.size(); the angle of pair i is position * rotation[i], and sines
+  // and cosines are multiplied by rotation_gain
   std::vector<double> rotation;
+  bool rotation_halves = false;
+  float rotation_gain = 1.f;
+  int kv_from = -1;                 // the layer whose keys and values are used (-1: the layer's own)
+  // Latent attention (rank > 0): keys and values of all heads are products of one normed latent of
+  // `rank` channels; a query head is [dim | rot_dim], its second part and one key part of rot_dim
+  // channels that all heads share are rotated.  The cache holds [latent | rotated key part], and the
+  // attention runs over the latent itself (as keys and as values, with the heads' matrices applied to
+  // queries and outputs).
+  int rank = 0, rot_dim = 0;
+  int cached_heads() const { return rank ? 1 : kv_heads; }
+  int key_width() const { return rank ? rank + rot_dim : dim; }
+  int value_width() const { return rank ? rank : vdim; }
+  int64_t value_pool_width() const { return rank || values_are_keys ? 0 : vdim; }
   bool values_are_keys = false;     // the values are the keys as projected (before their norm)
   bool unit_sink = false;           // the softmax denominator has one more member of score 0
   // learned bias by distance: row bucket(i - j) of a [buckets, heads] table; the lower half of the
@@ -40,11 +55,16 @@ struct FeedForwardSpec {
   int64_t ff = 0;                   // 0: none
   GatedAct act;
   std::string gate, up, down;
+  std::string gate_bias, up_bias, down_bias;  // empty: none
 };
 
-// `top` of the experts run for every token, weighted by the softmax over their router logits.
+// `top` of the experts run for every token, weighted by the softmax over their router logits, or
+// (sigmoid) by their sigmoid scores over the scores' sum, chosen among the best `keep` of `groups`
+// equal groups of neighbours.
 struct ExpertsSpec {
   int experts = 0, top = 0;         // 0: no mixture
+  bool sigmoid = false;
+  int groups = 1, keep = 1;
   int64_t ff = 0;
   GatedAct act;
   std::string router, router_bias;
@@ -54,6 +74,12 @@ struct ExpertsSpec {
 // S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per head, fp32 state of [dim, vdim].
 struct RecurrenceSpec {
   int heads = 0, dim = 0, vdim = 0;
+  int qk_heads = 0;                 // heads of q and k, each serving heads / qk_heads neighbours (0: one each)
+  // Selective state space: v, k and q pass through a causal convolution of conv_taps taps and SiLU; a
+  // step softplus(dt + bias) per token and head gives the decay exp(-exp(a_log) step) and scales the
+  // key, and the output gets skip * v
+  bool per_token_decay = false;
+  int conv_taps = 0;
   float q_scale = 1.f;
   bool silu_qkv = false;            // q, k and v pass through SiLU
   // decay: a constant per head, or sigmoid(W2 (W1 h) + bias)^(1/tau) per key channel
@@ -65,6 +91,8 @@ struct RecurrenceSpec {
   // [heads * vdim]) and multiplied by a gate
   bool norm_per_head = false;
   bool gate_silu = false;           // gate activation: SiLU, else sigmoid
+  int gated_norm_groups = 0;        // > 0: the gate comes first, then the norm in that many equal parts
+  int64_t conv_channels() const { return (int64_t)heads * vdim + 2 * (int64_t)qk_heads * dim; }
 };
 
 // Rows of the layer's input projection that come from one checkpoint tensor.
@@ -72,6 +100,7 @@ struct ProjPart {
   std::string tensor;
   int64_t rows = 0;
   int64_t offset = 0;  // first column of the projection's output (a multiple of 8)
+  int64_t first = 0, of = 0;  // of > 0: the rows from `first` on of a tensor of `of` rows
 };
 
 struct MixerSpec {
@@ -81,6 +110,9 @@ struct MixerSpec {
   // tensors: projections that read h, concatenated into one matrix
   ProjPart aq, ak, av, ag;                   // attention (ag: gate of the heads' outputs)
   ProjPart rq, rk, rv, rg, ra1;              // recurrence (ra1: low-rank decay)
+  ProjPart rx, rdt;                          // selective state space: [v | k | q] before the convolution, steps
+  std::string rec_conv, rec_conv_bias, rec_dt_bias, rec_a_log, rec_skip;
+  std::string attn_latent_norm, attn_uk, attn_uv;  // latent attention (ak: [latent | shared key part])
   std::string attn_o, rec_o, rec_norm, rec_a2, rec_a2_bias;
   // attention, empty where the design has none: biases of the projections, norms over the whole
   // query and key projections, distance bias table, learned sinks [heads]
@@ -104,7 +136,8 @@ struct LayeredSpec {
   int streams = 1;
   float eps = 1e-6f;
   float norm_offset = 0.f;                   // of norm1, norm2, final norm: 0 stored as they apply, 1 around zero
-  std::string embed, pos, final_norm, head;  // pos empty: no learned positions
+  float embed_scale = 1.f, residual_mult = 1.f, logit_scale = 1.f;  // residual_mult: of designs with one plain stream
+  std::string embed, pos, final_norm, head;  // pos empty: no learned positions; head empty: the embedding table
   std::vector<LayerSpec> layers;
 };
 
@@ -113,6 +146,8 @@ bool is_latarax(const Json& config);
 int read_latarax(const Json& config, LayeredSpec* out);
 bool is_biberax(const Json& config);
 int read_biberax(const Json& config, LayeredSpec* out);
+bool is_badolix(const Json& config);
+int read_badolix(const Json& config, LayeredSpec* out);
 
 // ---------------------------------------------------------------------------- weights
 struct LayeredLinear {
@@ -147,15 +182,25 @@ struct LayeredLayer {
   float *q_bias = nullptr, *k_bias = nullptr, *o_bias = nullptr, *q_norm = nullptr, *k_norm = nullptr, *sink = nullptr;
   float *rel = nullptr, *dist_bias = nullptr;  // [buckets, heads]; the same by distance, [heads, dist_len]
   int dist_len = 0, buckets = 0;
+  // latent attention: per head W_uk^T [rank, dim] and W_uv [vdim, rank]; whether the tensor-core kernel
+  // takes these products
+  void *uk_t = nullptr, *uv = nullptr;
+  float* latent_norm = nullptr;
+  bool latent_tc = false;
+  // selective state space
+  float *conv_w = nullptr, *conv_b = nullptr, *dt_bias = nullptr, *a_log = nullptr, *skip = nullptr;
+  void* conv_state = nullptr;                // [slots, taps - 1, channels] engine dtype
+  float *gate_b = nullptr, *up_b = nullptr, *down_b = nullptr;  // biases of a dense feed-forward
   LayeredExperts moe;
   int kv_pool = -1;                          // index into hb_engine::kc / vc
+  int tile_kind = -1;                        // index into LayeredModel::tile_sizes (-1: row by row)
   float* state = nullptr;                    // [slots, heads, dim, vdim]
   SublayerMix sub1, sub2;
 };
 
 // Plans of all matrix products for one bucket of batch rows.
 struct LayeredPlans {
-  std::vector<TcGemmPlan> proj, attn_o, rec_o, gate_up, down, moe_gate_up, moe_down;
+  std::vector<TcGemmPlan> proj, latent_q, latent_v, attn_o, rec_o, gate_up, down, moe_gate_up, moe_down;
 };
 
 struct LayeredGraph {
@@ -163,17 +208,19 @@ struct LayeredGraph {
   int64_t launches = 0;
 };
 
+constexpr int kTileKinds = 4;  // different sizes of attention tiles in one model
+
 // Where a step's inputs lie in the (pinned and device) input block, and what it contains.
 struct LayeredStep {
   int rows = 0, segs = 0, want = 0;
   int n_short = 0;        // segments the token-by-token recurrence kernel takes
   int n_chunks = 0;       // chunks of the longer segments (chunked recurrence kernels)
   int n_long = 0;         // longer segments
-  int n_tiles = 0;        // query tiles of the tiled attention kernel
+  int n_tiles[kTileKinds] = {0};  // query tiles of the tiled attention kernel, by tile size
   int n_token_rows = 0;   // rows that are single decoded tokens (first in the list of rows)
   bool decode = false;    // every segment is one token
   size_t off_ids = 0, off_pos = 0, off_slots = 0, off_row_seg = 0, off_want = 0, off_seg = 0, off_short = 0,
-         off_long = 0, off_chunk = 0, off_tile = 0, off_row_list = 0, off_tables = 0;
+         off_long = 0, off_chunk = 0, off_tile[kTileKinds] = {0}, off_row_list = 0, off_tables = 0;
   LayeredPlans* plans = nullptr;
   TcGemmPlan* head_plan = nullptr;
 };
@@ -195,6 +242,8 @@ struct LayeredModel {
   void* proj = nullptr;                      // [rows, max_proj]
   void *attn = nullptr, *rec = nullptr;      // branch outputs before their output projection
   float* o = nullptr;                        // [rows, heads * vdim] recurrence outputs
+  void* conv = nullptr;                      // [rows, channels] after the convolution
+  void *latent_q = nullptr, *latent_o = nullptr;  // [rows, heads * (rank + rot_dim)], [rows, heads * rank]
   float *y1 = nullptr, *y2 = nullptr;        // [rows, Hp] sublayer outputs
   void *gu = nullptr, *act = nullptr;        // feed-forward
   void* hf = nullptr;                        // [logits rows, Hp] final normed rows
@@ -209,7 +258,7 @@ struct LayeredModel {
   int64_t moe_places = 0;
   int32_t *moe_count = nullptr, *moe_first = nullptr, *moe_tiles = nullptr;
   int max_segs = 0, max_chunks = 0;
-  int tile_positions = 0;                    // positions of an attention tile that suit every layer (0: no tiles)
+  std::vector<int> tile_sizes;               // positions of an attention tile, as the layers need them
   std::map<int, LayeredPlans> plans;         // by rows bucket
   std::map<int, TcGemmPlan> head_plans;      // by wanted-rows bucket
   std::map<int, LayeredGraph> graphs;        // by number of decoded sequences

@@ -14,14 +14,18 @@ static SpanAttention span_of(const hb_span_attention_args* p) {
   a.window = p->window; a.keep_first = p->keep_first; a.chunk = p->chunk; a.scale = p->scale;
   a.key_scale = p->key_scale; a.dist_bias = p->dist_bias; a.dist_len = p->dist_len; a.sink = p->sink;
   a.gate = p->gate; a.ld_gate = p->ld_gate;
+  a.softcap = p->softcap;
+  if (a.key_scale) a.vc = nullptr;
   return a;
 }
 
 static int check_span(const hb_span_attention_args* p) {
-  HB_CHECK_ARG(p && p->k_cache && (p->v_cache || p->key_scale), "span attention: null argument");
+  HB_CHECK_ARG(p && p->k_cache, "span attention: null argument");
   HB_CHECK_ARG(p->heads > 0 && p->kv_heads > 0 && p->heads % p->kv_heads == 0 && p->dim > 0 && p->vdim > 0,
                "span attention: bad sizes");
   HB_CHECK_ARG(p->window >= 0 && p->keep_first >= 0 && p->chunk >= 0 && p->num_blocks > 0, "span attention: bad window or pool");
+  HB_CHECK_ARG(p->v_cache || p->vdim <= p->dim, "span attention: values inside the keys are no wider than they are");
+  HB_CHECK_ARG(p->softcap >= 0.f, "span attention: a negative cap");
   HB_CHECK_ARG(!p->key_scale || p->dim == p->vdim, "span attention: keys that are the values have their width");
   HB_CHECK_ARG(!p->dist_bias || p->dist_len > 0, "span attention: an empty bias table");
   return HB_OK;
@@ -38,6 +42,8 @@ static Recurrence recurrence_of(const hb_linear_recurrence_args* p) {
   a.inv_tau = p->decay ? 1.f : (float)(1.0 / p->tau);
   a.state = p->state; a.o = p->o; a.ld_o = p->ld_o;
   a.segs = (const SegInfo*)p->segments;
+  a.dt = p->dt; a.ld_dt = p->ld_dt; a.dt_bias = p->dt_bias; a.a_log = p->a_log; a.skip = p->skip; a.qk_heads = p->qk_heads;
+  if (a.dt) { a.decay = nullptr; a.rank = 0; a.inv_tau = 1.f; }
   return a;
 }
 
@@ -86,7 +92,8 @@ int hb_linear_recurrence(void* stream, const hb_linear_recurrence_args* p, const
                          float* chunk_state, hb_dtype dtype) {
   HB_CHECK_ARG(p && p->p && p->state && p->o && p->segments, "hb_linear_recurrence: null argument");
   HB_CHECK_ARG(p->heads > 0 && p->dim > 0 && p->vdim > 0, "hb_linear_recurrence: bad sizes");
-  HB_CHECK_ARG(p->decay || (p->a2 && p->a2_bias && p->rank > 0 && p->tau > 0.f), "hb_linear_recurrence: no decay");
+  HB_CHECK_ARG(p->qk_heads >= 0 && (!p->qk_heads || p->heads % p->qk_heads == 0), "hb_linear_recurrence: bad heads of q and k");
+  HB_CHECK_ARG(p->dt ? p->dt_bias && p->a_log : p->decay || (p->a2 && p->a2_bias && p->rank > 0 && p->tau > 0.f), "hb_linear_recurrence: no decay");
   const hb::Recurrence a = hb::recurrence_of(p);
   auto st = (cudaStream_t)stream;
   int rc = hb::recurrence_tokens(st, a, list, n_list, dtype);
@@ -138,7 +145,7 @@ int hb_streams_mix_ex(void* stream, float* x, void* h, const float* y, const flo
 }
 
 int hb_attention_prepare(void* stream, const hb_attention_prep_args* p, int64_t rows, hb_dtype dtype) {
-  HB_CHECK_ARG(p && p->p && p->positions && p->slots && p->k_cache && (p->v_cache || p->key_scale) && rows >= 0,
+  HB_CHECK_ARG(p && p->p && p->positions && p->slots && (!p->k_cache || p->v_cache || p->key_scale) && rows >= 0,
                "hb_attention_prepare: null argument");
   HB_CHECK_ARG(p->heads > 0 && p->kv_heads > 0 && p->heads % p->kv_heads == 0 && p->dim > 0 && p->vdim > 0 && p->num_blocks > 0 &&
                p->pairs >= 0 && (p->pairs == 0 || p->rotation), "hb_attention_prepare: bad sizes");
@@ -149,7 +156,48 @@ int hb_attention_prepare(void* stream, const hb_attention_prep_args* p, int64_t 
   a.pos = p->positions; a.slots = p->slots; a.kc = p->k_cache; a.vc = p->v_cache; a.num_blocks = p->num_blocks;
   a.q_bias = p->q_bias; a.k_bias = p->k_bias; a.q_norm = p->q_norm; a.k_norm = p->k_norm; a.eps = p->eps;
   a.rotation = p->rotation; a.pairs = p->pairs; a.key_scale = p->key_scale;
+  a.halves = p->halves; a.rotation_gain = p->rotation_gain == 0.f ? 1.f : p->rotation_gain;
   return hb::attention_prepare((cudaStream_t)stream, a, rows, dtype);
+}
+
+int hb_latent_prepare(void* stream, const hb_latent_prep_args* p, int64_t rows, hb_dtype dtype) {
+  HB_CHECK_ARG(p && p->p && p->q && p->positions && p->slots && p->k_cache && p->norm && rows >= 0, "hb_latent_prepare: null argument");
+  HB_CHECK_ARG(p->heads > 0 && p->dim > 0 && p->rot_dim >= 0 && p->rank > 0 && p->num_blocks > 0 && p->pairs >= 0 &&
+               (p->pairs == 0 || p->rotation), "hb_latent_prepare: bad sizes");
+  hb::LatentPrep a;
+  a.p = p->p; a.ld = p->ld; a.off_q = p->off_q; a.off_c = p->off_c;
+  a.heads = p->heads; a.dim = p->dim; a.rot_dim = p->rot_dim; a.rank = p->rank;
+  a.q = p->q; a.ld_q = p->ld_q; a.pos = p->positions; a.slots = p->slots; a.kc = p->k_cache; a.num_blocks = p->num_blocks;
+  a.norm = p->norm; a.eps = p->eps; a.rotation = p->rotation; a.pairs = p->pairs;
+  a.rotation_gain = p->rotation_gain == 0.f ? 1.f : p->rotation_gain;
+  return hb::latent_prepare((cudaStream_t)stream, a, rows, dtype);
+}
+
+int hb_gemm_heads(void* stream, void* Y, const void* X, const void* W, int64_t M, int64_t N, int64_t K, int heads, int64_t ldx,
+                  int64_t x_step, int64_t ldy, int64_t y_step, hb_dtype dtype) {
+  HB_CHECK_ARG(Y && X && W && M >= 0 && N > 0 && K > 0 && heads > 0, "hb_gemm_heads: bad argument");
+  hb::TcHeads h;
+  h.heads = heads; h.ldx = ldx; h.x_step = x_step; h.ldy = ldy; h.y_step = y_step;
+  auto st = (cudaStream_t)stream;
+  auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  if (M && hb::gemm_tc_supported(M, N, K, dtype) && hb::gemm_tc_heads_supported(N, K, false, h) && al(X) && al(W) && al(Y)) {
+    int dev = 0;
+    HB_CUDA_CHECK(cudaGetDevice(&dev));
+    hb::TcGemmPlan plan;
+    int rc = hb::gemm_tc_plan(&plan, X, W, M, N, K, hb::kEpiStore, false, dev, 0, nullptr, &h);
+    return rc ? rc : hb::gemm_tc_run(plan, st, Y, ldy, nullptr, nullptr);
+  }
+  return hb::gemm_simt_heads(st, Y, X, W, M, N, K, dtype, false, h);
+}
+
+int hb_short_conv(void* stream, const hb_short_conv_args* p, const int32_t* list, int n_list, const int32_t* chunks, int n_chunks,
+                  hb_dtype dtype) {
+  HB_CHECK_ARG(p && p->p && p->w && p->bias && p->out && p->segments && (p->state || p->taps == 1), "hb_short_conv: null argument");
+  HB_CHECK_ARG(n_list >= 0 && n_chunks >= 0 && (list || !n_list) && (chunks || !n_chunks), "hb_short_conv: bad lists");
+  hb::ShortConv a;
+  a.p = p->p; a.ld = p->ld; a.off = p->off; a.channels = p->channels; a.taps = p->taps; a.w = p->w; a.bias = p->bias;
+  a.out = p->out; a.ld_out = p->ld_out; a.state = p->state; a.segs = (const hb::SegInfo*)p->segments;
+  return hb::short_conv((cudaStream_t)stream, a, list, n_list, (const hb::RowRange*)chunks, n_chunks, dtype);
 }
 
 static hb::MoeRouting routing_of(const hb_moe_routing* p) {
@@ -157,12 +205,14 @@ static hb::MoeRouting routing_of(const hb_moe_routing* p) {
   m.experts = p->experts; m.top = p->top; m.shared = p->shared ? 1 : 0; m.m_pad = p->m_pad; m.max_tiles = p->max_tiles;
   m.ids = p->ids; m.rank = p->rank; m.place = p->place; m.weight = p->weight;
   m.count = p->count; m.first = p->first; m.tile_group = p->tile_group;
+  m.sigmoid = p->sigmoid;
+  if (p->groups) { m.groups = p->groups; m.keep = p->keep; }
   return m;
 }
 
 int hb_moe_route_top(void* stream, const hb_moe_routing* m, const void* h, int64_t ld_h, const void* router,
                      const float* bias, int64_t rows, int64_t width, hb_dtype dtype) {
-  HB_CHECK_ARG(m && h && router && bias && m->ids && m->rank && m->weight && m->count && m->first && m->tile_group,
+  HB_CHECK_ARG(m && h && router && m->ids && m->rank && m->weight && m->count && m->first && m->tile_group,
                "hb_moe_route_top: null argument");
   HB_CHECK_ARG(rows >= 0 && width > 0 && m->m_pad > 0 &&
                m->max_tiles >= (rows * m->top < m->experts ? rows * m->top : m->experts) + rows * m->top / m->m_pad +
@@ -241,12 +291,14 @@ int hb_streams_final(void* stream, void* h, const float* x, const int32_t* want,
 }
 
 int hb_gated_group_norm(void* stream, void* out, int64_t ld_out, const float* o, int64_t ld_o, const void* gate,
-                        int64_t ld_gate, const float* weight, int64_t rows, int groups, int size, int gate_silu, float eps,
+                        int64_t ld_gate, const float* weight, int64_t rows, int groups, int size, int gate_mode, float eps,
                         hb_dtype dtype) {
   HB_CHECK_ARG(out && o && gate && weight && groups > 0 && size > 0 && rows >= 0, "hb_gated_group_norm: bad argument");
   if (rows == 0) return HB_OK;
-  return hb::gated_group_norm((cudaStream_t)stream, out, ld_out, o, ld_o, gate, ld_gate, weight, rows, groups, size,
-                              gate_silu != 0, eps, dtype);
+  hb::GroupNorm n;
+  n.groups = groups; n.size = size; n.gate_silu = (gate_mode & 1) != 0; n.gate_first = n.own_weights = (gate_mode & 2) != 0;
+  n.eps = eps;
+  return hb::gated_group_norm((cudaStream_t)stream, out, ld_out, o, ld_o, gate, ld_gate, weight, rows, n, dtype);
 }
 
 }  // extern "C"

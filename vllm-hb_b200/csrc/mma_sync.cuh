@@ -45,6 +45,12 @@ __device__ __forceinline__ void mma_split(float (&d)[4], const uint32_t (&ahi)[4
   mma_bf16_16816(d, ahi, bl0, bl1);
 }
 
+// d += (ahi + alo) . b
+__device__ __forceinline__ void mma_pair(float (&d)[4], const uint32_t (&ahi)[4], const uint32_t (&alo)[4], uint32_t b0, uint32_t b1) {
+  mma_bf16_16816(d, ahi, b0, b1);
+  mma_bf16_16816(d, alo, b0, b1);
+}
+
 // 2^x in one instruction (ex2.approx, about 2 ulp)
 __device__ __forceinline__ float ex2(float x) {
   float y;

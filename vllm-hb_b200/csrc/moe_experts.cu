@@ -1,4 +1,5 @@
-// Mixture of experts with a router bias and top-k routing, each expert run on its own rows only.
+// Mixture of experts with top-k routing (softmax over the chosen logits, or sigmoid scores with the
+// choice limited to the best groups of experts), each expert run on its own rows only.
 //
 //   route   logits, the top experts of every row and their weights; every (row, expert) draws a rank
 //           among the expert's rows; the last CTA turns the counts into batch tiles
@@ -23,7 +24,7 @@ __global__ void __launch_bounds__(kRouteThreads)
 moe_route_top_kernel(const MoeRouting m, const T* __restrict__ h, int64_t ld_h, const T* __restrict__ router,
                      const float* __restrict__ bias, int64_t rows, int64_t width) {
   pdl_trigger();
-  extern __shared__ float s_logit[];  // [RB][experts]
+  extern __shared__ float s_logit[];  // [RB][experts], then [RB][groups]
   __shared__ int s_last;
   pdl_grid_wait();
   constexpr int N = Vec16<T>::N;
@@ -64,7 +65,10 @@ moe_route_top_kernel(const MoeRouting m, const T* __restrict__ h, int64_t ld_h, 
 #pragma unroll
     for (int r = 0; r < RB; ++r) {
       const float s = warp_sum(acc[r]);
-      if (lane == 0) s_logit[r * E + e] = s + bias[e];
+      if (lane == 0) {
+        const float z = bias ? s + bias[e] : s;
+        s_logit[r * E + e] = m.sigmoid ? 1.f / (1.f + expf(-z)) : z;
+      }
     }
   }
   __syncthreads();
@@ -72,6 +76,28 @@ moe_route_top_kernel(const MoeRouting m, const T* __restrict__ h, int64_t ld_h, 
   for (int r = warp; r < nr; r += kRouteWarps) {
     float* z = s_logit + r * E;
     const int64_t at = (row0 + r) * m.picks();
+    if (m.keep < m.groups) {
+      // groups by the sum of their two largest scores; experts of the others cannot be chosen
+      float* gs = s_logit + RB * E + r * m.groups;
+      const int size = E / m.groups;
+      for (int g = lane; g < m.groups; g += 32) {
+        float a = -INFINITY, b = -INFINITY;
+        for (int e = g * size; e < (g + 1) * size; ++e) {
+          const float v = z[e];
+          if (v > a) { b = a; a = v; }
+          else if (v > b) b = v;
+        }
+        gs[g] = size > 1 ? a + b : a;
+      }
+      __syncwarp();
+      for (int g = lane; g < m.groups; g += 32) {
+        int better = 0;  // groups that go first: larger, or equal and lower
+        for (int o = 0; o < m.groups; ++o) better += gs[o] > gs[g] || (gs[o] == gs[g] && o < g);
+        if (better >= m.keep)
+          for (int e = g * size; e < (g + 1) * size; ++e) z[e] = __int_as_float(0x7fc00000);
+      }
+      __syncwarp();
+    }
     float first = 0.f, sum = 0.f;
     int mine = 0;        // lane k keeps choice k (of every 32) and its unscaled weight
     float mine_p = 0.f;
@@ -90,7 +116,7 @@ moe_route_top_kernel(const MoeRouting m, const T* __restrict__ h, int64_t ld_h, 
       }
       const int e = min(who, E - 1);  // a row of NaNs still names an expert
       if (k == 0) first = best;
-      const float p = expf(best - first);
+      const float p = m.sigmoid ? best : expf(best - first);
       sum += p;
       if (lane == 0) z[e] = __int_as_float(0x7fc00000);  // taken
       if (lane == (k & 31)) {
@@ -108,7 +134,7 @@ moe_route_top_kernel(const MoeRouting m, const T* __restrict__ h, int64_t ld_h, 
       }
     }
     __syncwarp();
-    for (int k = lane; k < m.top; k += 32) m.weight[at + k] /= sum;  // written by this lane
+    for (int k = lane; k < m.top; k += 32) m.weight[at + k] /= m.sigmoid ? sum + 1e-20f : sum;  // written by this lane
     if (m.shared && lane == 0) {
       m.ids[at + m.top] = E;
       m.weight[at + m.top] = 1.f;
@@ -180,10 +206,12 @@ int moe_route_top(cudaStream_t st, const MoeRouting& m, const void* h, int64_t l
   if (rows == 0) return HB_OK;
   if (m.experts < 1 || m.experts > kMoeMaxExperts || m.top < 1 || m.top > m.experts || m.m_pad < 1)
     return fail(HB_ERR_INVALID_ARG, "moe_route_top: %d of %d experts (at most %d)", m.top, m.experts, kMoeMaxExperts);
+  if (m.groups < 1 || m.experts % m.groups || m.keep < 1 || m.keep > m.groups || m.top > m.experts / m.groups * m.keep)
+    return fail(HB_ERR_INVALID_ARG, "moe_route_top: %d of %d groups of %d experts, top %d", m.keep, m.groups, m.experts, m.top);
   auto launch = [&](auto* k, int rb, auto* t) -> int {
     using T = std::remove_pointer_t<decltype(t)>;
     HB_CUDA_CHECK(launch_pdl(k, dim3((unsigned)((rows + rb - 1) / rb)), dim3(kRouteThreads),
-                             (size_t)rb * m.experts * sizeof(float), st, m, (const T*)h, ld_h, (const T*)router, bias, rows, width));
+                             (size_t)rb * (m.experts + m.groups) * sizeof(float), st, m, (const T*)h, ld_h, (const T*)router, bias, rows, width));
     return HB_OK;
   };
   const bool few = rows <= 296;
@@ -218,7 +246,7 @@ int moe_gather(cudaStream_t st, const MoeRouting& m, void* x, const void* h, int
 template <typename T>
 __global__ void gated_act_kernel(T* __restrict__ out, int64_t ld_out, const T* __restrict__ gu, int64_t ld_gu, int64_t inter,
                                  GatedAct act, const int32_t* __restrict__ tile_group, int m_pad, int further, int64_t inter2,
-                                 GatedAct act2) {
+                                 GatedAct act2, const float* __restrict__ gate_bias, const float* __restrict__ up_bias) {
   pdl_trigger();
   pdl_grid_wait();
   const int64_t row = blockIdx.x;
@@ -231,17 +259,19 @@ __global__ void gated_act_kernel(T* __restrict__ out, int64_t ld_out, const T* _
     }
   }
   for (int64_t i = threadIdx.x; i < inter; i += blockDim.x) {
-    const float g = fminf(to_f32<T>(gu[row * ld_gu + i]), act.limit);
-    const float u = fminf(fmaxf(to_f32<T>(gu[row * ld_gu + inter + i]), -act.limit), act.limit);
+    const float gb = gate_bias ? gate_bias[i] : 0.f, ub = up_bias ? up_bias[i] : 0.f;
+    const float g = fminf(to_f32<T>(gu[row * ld_gu + i]) + gb, act.limit);
+    const float u = fminf(fmaxf(to_f32<T>(gu[row * ld_gu + inter + i]) + ub, -act.limit), act.limit);
     out[row * ld_out + i] = from_f32<T>(g / (1.f + expf(-act.slope * (g + act.cubic * g * g * g))) * (u + act.shift));
   }
 }
 
-int gated_act(cudaStream_t st, void* out, const void* gate_up, int64_t M, int64_t inter, const GatedAct& act, hb_dtype dtype) {
+int gated_act(cudaStream_t st, void* out, const void* gate_up, int64_t M, int64_t inter, const GatedAct& act, hb_dtype dtype,
+              const float* gate_bias, const float* up_bias) {
   if (M == 0) return HB_OK;
   HB_DISPATCH_DTYPE(dtype, T, {
     HB_CUDA_CHECK(launch_pdl(gated_act_kernel<T>, dim3((unsigned)M), dim3(256), 0, st, (T*)out, inter, (const T*)gate_up, 2 * inter,
-                             inter, act, nullptr, 1, -1, 0, act));
+                             inter, act, nullptr, 1, -1, 0, act, gate_bias, up_bias));
   });
   return HB_OK;
 }
@@ -252,7 +282,8 @@ int gated_act_grouped(cudaStream_t st, void* out, int64_t ld_out, const void* ga
   if (rows == 0) return HB_OK;
   HB_DISPATCH_DTYPE(dtype, T, {
     HB_CUDA_CHECK(launch_pdl(gated_act_kernel<T>, dim3((unsigned)rows), dim3(256), 0, st, (T*)out, ld_out, (const T*)gate_up,
-                             ld_gu, inter, act, tile_group, g.m_pad, g.shared_w ? g.groups : -1, g.shared_n / 2, g.shared_act));
+                             ld_gu, inter, act, tile_group, g.m_pad, g.shared_w ? g.groups : -1, g.shared_n / 2, g.shared_act,
+                             nullptr, nullptr));
   });
   return HB_OK;
 }

@@ -1,7 +1,8 @@
 // Gated linear recurrences with a matrix state per head:
 //   S_t = diag(a_t) S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t        (S fp32 [dim, vdim])
 // The decay a_t is a constant per head or, per key channel, sigmoid(z)^(1/tau) with z from a
-// low-rank projection; q, k and v may pass through SiLU and q carries a scale.
+// low-rank projection, or follows a step per token (selective state space), which also scales the key;
+// q, k and v may pass through SiLU and q carries a scale.
 #include "layered_ops.h"
 
 namespace hb {
@@ -19,6 +20,13 @@ __device__ __forceinline__ float low_rank_log_decay(const Recurrence& a, const T
 #pragma unroll 8
   for (int r = 0; r < a.rank; ++r) z = fmaf(w[r], to_f32<T>(t[r]), z);
   return log_sigmoid(z) * a.inv_tau;
+}
+
+// step of a row and head
+template <typename T>
+__device__ __forceinline__ float step_of(const Recurrence& a, int64_t row, int h) {
+  const float z = to_f32<T>(((const T*)a.dt)[row * a.ld_dt + h]) + a.dt_bias[h];
+  return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
 }
 
 // CTA = (segment, head, COLS state columns).  A thread owns VEC neighbouring columns of every
@@ -69,13 +77,14 @@ recurrence_tokens_kernel(const Recurrence a, const int32_t* __restrict__ list) {
     // every kind of input has threads of its own: decays, then q and k, then v
     for (int i = tid; i < 2 * D + COLS; i += kRecThreads) {
       if (i < D) {
-        s_a[i] = a.decay ? a.decay[h] : expf(low_rank_log_decay<T>(a, p + a.off_a1, h * D + i));
+        if (a.dt) s_a[i] = expf(-expf(a.a_log[h]) * step_of<T>(a, row, h));
+        else s_a[i] = a.decay ? a.decay[h] : expf(low_rank_log_decay<T>(a, p + a.off_a1, h * D + i));
       } else if (i < 2 * D) {
         const int d = i - D;
-        float q = to_f32<T>(p[a.off_q + h * D + d]), k = to_f32<T>(p[a.off_k + h * D + d]);
+        float q = to_f32<T>(p[a.off_q + a.qk(h) * D + d]), k = to_f32<T>(p[a.off_k + a.qk(h) * D + d]);
         if (a.silu_qkv) { q = silu_f(q); k = silu_f(k); }
         s_q[d] = q * a.q_scale;
-        s_k[d] = k;
+        s_k[d] = a.dt ? k * step_of<T>(a, row, h) : k;
       } else {
         const int c = i - 2 * D;
         const float v = v0 + c < VD ? to_f32<T>(p[a.off_v + h * VD + v0 + c]) : 0.f;
@@ -122,6 +131,7 @@ recurrence_tokens_kernel(const Recurrence a, const int32_t* __restrict__ list) {
       float o = 0.f;
 #pragma unroll
       for (int g = 0; g < DG; ++g) o += s_o[g][i];
+      if (a.skip) o = fmaf(a.skip[h], s_v[i], o);
       if (v0 + i < VD) a.o[row * a.ld_o + (int64_t)h * VD + v0 + i] = o;
     }
     __syncthreads();

@@ -10,7 +10,10 @@
 // Products run on tensor cores with both operands as pairs of bf16 numbers (hi + lo), which keeps
 // fp32-like precision; sums, decays and states are fp32.
 //
-//   decay   running log2 decays of a chunk (low-rank decay only)
+// With a decay per token and head (selective state space) b_i is one number per token, so scores are
+// q_i . k_j * 2^(b_i - b_j) * step_j; q, k and v are exact bf16 numbers and need no second half.
+//
+//   decay   running log2 decays of a chunk (low-rank decay), also steps (decay per token)
 //   state   per (chunk, head, 64 state columns): the chunk's own contribution to the state
 //   scan    per element of the state: over the chunks of a segment, contribution -> state before
 //   output  per (chunk, head): scores, outputs
@@ -29,6 +32,7 @@ constexpr int kVT = 64;        // state columns of a tile
 constexpr int kVS = kVT + 8;   // padded row of a bf16 tile
 constexpr float kLog2e = 1.4426950408889634f;
 using bf16 = __nv_bfloat16;
+enum Decay { kConstant, kLowRank, kPerToken };
 
 __device__ __forceinline__ float rec_silu(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float log2_sigmoid(float z) { return (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * kLog2e; }
@@ -125,7 +129,37 @@ recurrence_decay_kernel(const Recurrence a, const RowRange* __restrict__ chunks,
   }
 }
 
-// Value tile [64 tokens][64 columns] as hi/lo pairs; rows and columns outside are zero.
+// Decay per token: CTA = (chunk, 32 heads).
+constexpr int kStepHeads = 32;
+__global__ void __launch_bounds__(256)
+recurrence_step_kernel(const Recurrence a, const RowRange* __restrict__ chunks, float* __restrict__ cum) {
+  __shared__ float s_t[kC][kStepHeads + 1];
+  pdl_trigger();
+  pdl_grid_wait();
+  const RowRange ch = chunks[blockIdx.x];
+  const int h0 = blockIdx.y * kStepHeads, n = min(kStepHeads, a.heads - h0), x = threadIdx.x % kStepHeads;
+  const float bias = x < n ? a.dt_bias[h0 + x] : 0.f;
+#pragma unroll 4
+  for (int i = threadIdx.x / kStepHeads; i < ch.n; i += 256 / kStepHeads) {
+    if (x >= n) continue;
+    const float z = __bfloat162float(((const bf16*)a.dt)[(int64_t)(ch.row0 + i) * a.ld_dt + h0 + x]) + bias;
+    const float t = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+    s_t[i][x] = t;
+    cum[((int64_t)(ch.row0 + i) * 2 + 1) * a.heads + h0 + x] = t;
+  }
+  __syncthreads();
+  if ((int)threadIdx.x >= n) return;
+  const float rate = -expf(a.a_log[h0 + threadIdx.x]) * kLog2e;
+  float b = 0.f;
+  for (int i = 0; i < ch.n; ++i) {
+    b = fmaf(rate, s_t[i][threadIdx.x], b);
+    cum[(int64_t)(ch.row0 + i) * 2 * a.heads + h0 + threadIdx.x] = b;
+  }
+}
+
+// Value tile [64 tokens][64 columns] as hi/lo pairs (EXACT: as they are); rows and columns outside are
+// zero.
+template <bool EXACT>
 __device__ __forceinline__ void load_values(const Recurrence& a, const RowRange& ch, int h, int v0, bf16* hi, bf16* lo) {
 #pragma unroll 4
   for (int i = threadIdx.x; i < kC * kVT / 8; i += kT) {
@@ -136,10 +170,12 @@ __device__ __forceinline__ void load_values(const Recurrence& a, const RowRange&
 #pragma unroll
       for (int e = 0; e < 8; ++e) v[e] = rec_silu(v[e]);
     }
-    put_split8(hi + j * kVS + c, lo + j * kVS + c, v);
+    if (EXACT) put8(hi + j * kVS + c, v);
+    else put_split8(hi + j * kVS + c, lo + j * kVS + c, v);
   }
 }
 
+template <int MODE>
 __global__ void __launch_bounds__(kT)
 recurrence_state_kernel(const Recurrence a, const RowRange* __restrict__ chunks, const float* __restrict__ cum,
                         float* __restrict__ out) {
@@ -148,29 +184,37 @@ recurrence_state_kernel(const Recurrence a, const RowRange* __restrict__ chunks,
   bf16* k_hi = (bf16*)smem;
   bf16* k_lo = k_hi + kC * KS;
   bf16* v_hi = k_lo + kC * KS;
-  bf16* v_lo = v_hi + kC * kVS;
+  bf16* v_lo = v_hi + kC * kVS;                   // not with a decay per token
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
   pdl_grid_wait();
   const RowRange ch = chunks[blockIdx.x];
-  const int hd = a.heads * D;
-  const float ld2 = a.decay ? log2f(a.decay[h]) : 0.f;
+  const int hd = a.heads * D, hk = a.qk(h);
+  const float ld2 = MODE == kConstant ? log2f(a.decay[h]) : 0.f;
+  __shared__ float s_f[kC];                       // decay per token: factors of the keys
+  if (MODE == kPerToken) {
+    if (tid < ch.n) {
+      const float* own = cum + (int64_t)(ch.row0 + tid) * 2 * a.heads + h;
+      s_f[tid] = own[a.heads] * ex2(cum[(int64_t)(ch.row0 + ch.n - 1) * 2 * a.heads + h] - own[0]);
+    }
+    __syncthreads();
+  }
   for_groups(DP, [&](int j, int d) {
     float k[8];
     const bool live = j < ch.n;
-    ld_proj8(k, a, ch.row0 + min(j, ch.n - 1), a.off_k + h * D + d, live ? D - d : 0);
+    ld_proj8(k, a, ch.row0 + min(j, ch.n - 1), a.off_k + hk * D + d, live ? D - d : 0);
     if (live) {
-      const float f = a.decay ? ex2(log2_pow(ld2, ch.n - 1 - j)) : 1.f;
+      const float f = MODE == kConstant ? ex2(log2_pow(ld2, ch.n - 1 - j)) : MODE == kPerToken ? s_f[j] : 1.f;
       const float* end = cum + (int64_t)(ch.row0 + ch.n - 1) * hd + h * D + d;
       const float* own = cum + (int64_t)(ch.row0 + j) * hd + h * D + d;
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
         if (a.silu_qkv) k[e] = rec_silu(k[e]);
-        k[e] *= a.decay ? f : (d + e < D ? ex2(end[e] - own[e]) : 0.f);
+        k[e] *= MODE != kLowRank ? f : (d + e < D ? ex2(end[e] - own[e]) : 0.f);
       }
     }
     put_split8(k_hi + j * KS + d, k_lo + j * KS + d, k);
   });
-  load_values(a, ch, h, v0, v_hi, v_lo);
+  load_values<MODE == kPerToken>(a, ch, h, v0, v_hi, v_lo);
   __syncthreads();
   float* o = out + ((int64_t)blockIdx.x * a.heads + h) * D * a.vdim + v0;
   // A = (scaled keys)^T: stored [token][channel], read transposed.  Matrices of the x4 load: channels
@@ -192,6 +236,11 @@ recurrence_state_kernel(const Recurrence a, const RowRange* __restrict__ chunks,
       for (int nv = 0; nv < 4; ++nv) {
         uint32_t b[4], c[4];
         ldsm_x4_trans(bh + (ks * 16 * kVS + nv * 16) * 2, b[0], b[1], b[2], b[3]);
+        if (MODE == kPerToken) {
+          mma_pair(acc[2 * nv], hi, lo, b[0], b[1]);
+          mma_pair(acc[2 * nv + 1], hi, lo, b[2], b[3]);
+          continue;
+        }
         ldsm_x4_trans(bl + (ks * 16 * kVS + nv * 16) * 2, c[0], c[1], c[2], c[3]);
         mma_split(acc[2 * nv], hi, lo, b[0], b[1], c[0], c[1]);
         mma_split(acc[2 * nv + 1], hi, lo, b[2], b[3], c[2], c[3]);
@@ -208,7 +257,7 @@ recurrence_state_kernel(const Recurrence a, const RowRange* __restrict__ chunks,
 }
 
 // One thread per VEC neighbouring state elements.
-template <int VEC>
+template <int VEC, int MODE>
 __global__ void __launch_bounds__(256)
 recurrence_scan_kernel(const Recurrence a, const RowRange* __restrict__ segs, const RowRange* __restrict__ chunks,
                        const float* __restrict__ cum, float* __restrict__ chunk_state) {
@@ -220,7 +269,7 @@ recurrence_scan_kernel(const Recurrence a, const RowRange* __restrict__ segs, co
   const RowRange sg = segs[blockIdx.z];
   const SegInfo info = a.segs[sg.seg];
   float* state = a.state + ((int64_t)info.slot * a.heads + h) * per_head + i;
-  const float ld2 = a.decay ? log2f(a.decay[h]) : 0.f;
+  const float ld2 = MODE == kConstant ? log2f(a.decay[h]) : 0.f;
   float s[VEC];
 #pragma unroll
   for (int j = 0; j < VEC; ++j) s[j] = info.pos0 > 0 ? state[j] : 0.f;  // a new sequence starts from zero
@@ -234,7 +283,8 @@ recurrence_scan_kernel(const Recurrence a, const RowRange* __restrict__ segs, co
       f[c] = 0.f;
       if (c0 + c < sg.n) {
         const RowRange ch = chunks[sg.row0 + c0 + c];
-        f[c] = a.decay ? log2_pow(ld2, ch.n) : cum[(int64_t)(ch.row0 + ch.n - 1) * hd + h * a.dim + d];
+        const int64_t end = ch.row0 + ch.n - 1;
+        f[c] = MODE == kConstant ? log2_pow(ld2, ch.n) : MODE == kPerToken ? cum[end * 2 * a.heads + h] : cum[end * hd + h * a.dim + d];
         if (VEC == 4) {
           const float4 x = *reinterpret_cast<const float4*>(u + c * stride);
           v[c][0] = x.x; v[c][1 % VEC] = x.y; v[c][2 % VEC] = x.z; v[c][3 % VEC] = x.w;
@@ -260,19 +310,21 @@ recurrence_scan_kernel(const Recurrence a, const RowRange* __restrict__ segs, co
   for (int j = 0; j < VEC; ++j) state[j] = s[j];
 }
 
-// LR: low-rank decay (q and k are exact bf16, decays per channel); else a constant decay per head.
-template <bool LR>
+template <int MODE>
 __global__ void __launch_bounds__(kT)
 recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks, const float* __restrict__ cum,
                          const float* __restrict__ chunk_state) {
   extern __shared__ __align__(16) uint8_t smem[];
-  const int D = a.dim, DP = pad16d(D), KS = DP + 8, BS = DP + 4, h = blockIdx.y;
-  // LR: q | b | k | scaled k (hi, lo);  constant: q (hi, lo) | k (hi, lo).  The keys' part is reused by
-  // the value and state tiles of the second phase.
+  // LR: q and k are exact bf16, decays per channel
+  constexpr bool LR = MODE == kLowRank, TOKEN = MODE == kPerToken;
+  const int D = a.dim, DP = pad16d(D), KS = DP + 8, BS = DP + 4, h = blockIdx.y, hk = a.qk(h);
+  // low rank: q | b | k | scaled k (hi, lo);  constant: q (hi, lo) | k (hi, lo);  per token: q | k.  The
+  // keys' part is reused by the value and state tiles of the second phase.
   bf16* q_hi = (bf16*)smem;                       // [64][KS]
   bf16* q_lo = q_hi + kC * KS;                    // constant decay only
   float* s_b = (float*)(q_hi + kC * KS);          // LR only: [64][BS]
-  uint8_t* keys = LR ? (uint8_t*)(s_b + kC * BS) : (uint8_t*)(q_lo + kC * KS);
+  uint8_t* keys = LR ? (uint8_t*)(s_b + kC * BS) : TOKEN ? (uint8_t*)(q_hi + kC * KS) : (uint8_t*)(q_lo + kC * KS);
+  __shared__ float s_cum[kC], s_step[kC];         // decay per token
   bf16* k_raw = (bf16*)keys;                      // LR only
   bf16* k_hi = LR ? k_raw + kC * KS : (bf16*)keys;
   bf16* k_lo = k_hi + kC * KS;
@@ -280,7 +332,12 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
   pdl_grid_wait();
   const RowRange ch = chunks[blockIdx.x];
   const int hd = a.heads * D;
-  const float ld2 = LR ? 0.f : log2f(a.decay[h]);
+  const float ld2 = MODE == kConstant ? log2f(a.decay[h]) : 0.f;
+  if (TOKEN && tid < kC) {  // tokens past the end keep the last decay
+    const float* own = cum + (int64_t)(ch.row0 + min(tid, ch.n - 1)) * 2 * a.heads + h;
+    s_cum[tid] = own[0];
+    s_step[tid] = own[a.heads];
+  }
   if (LR) {
     for_groups(DP, [&](int j, int d) {
       // tokens past the end keep the last decay: every exponent stays <= 0
@@ -294,8 +351,8 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
     float q[8], k[8];
     const int valid = j < ch.n ? D - d : 0;
     const int64_t row = ch.row0 + min(j, ch.n - 1);
-    ld_proj8(q, a, row, a.off_q + h * D + d, valid);
-    ld_proj8(k, a, row, a.off_k + h * D + d, valid);
+    ld_proj8(q, a, row, a.off_q + hk * D + d, valid);
+    ld_proj8(k, a, row, a.off_k + hk * D + d, valid);
     if (a.silu_qkv) {
 #pragma unroll
       for (int e = 0; e < 8; ++e) { q[e] = rec_silu(q[e]); k[e] = rec_silu(k[e]); }
@@ -307,6 +364,9 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
 #pragma unroll
       for (int e = 0; e < 8; ++e) k[e] *= ex2(end[e] - own[e]);
       put_split8(k_hi + j * KS + d, k_lo + j * KS + d, k);
+    } else if (TOKEN) {
+      put8(q_hi + j * KS + d, q);
+      put8(k_hi + j * KS + d, k);
     } else {
       put_split8(q_hi + j * KS + d, q_lo + j * KS + d, q);
       put_split8(k_hi + j * KS + d, k_lo + j * KS + d, k);
@@ -348,7 +408,13 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
           q_frag(ks, nb * 16 + 15, hi, lo);
         } else {
           ldsm_x4(qh + ks * 32, hi[0], hi[1], hi[2], hi[3]);
-          ldsm_x4(ql + ks * 32, lo[0], lo[1], lo[2], lo[3]);
+          if (!TOKEN) ldsm_x4(ql + ks * 32, lo[0], lo[1], lo[2], lo[3]);
+        }
+        if (TOKEN) {
+          ldsm_x4(kh + (nb * 16 * KS + ks * 16) * 2, b[0], b[1], b[2], b[3]);
+          mma_bf16_16816(s[2 * nb], hi, b[0], b[1]);
+          mma_bf16_16816(s[2 * nb + 1], hi, b[2], b[3]);
+          continue;
         }
         ldsm_x4(kh + (nb * 16 * KS + ks * 16) * 2, b[0], b[1], b[2], b[3]);
         ldsm_x4(kl + (nb * 16 * KS + ks * 16) * 2, c[0], c[1], c[2], c[3]);
@@ -395,17 +461,19 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
     for (int e = 0; e < 4; ++e) {
       const int i = e < 2 ? i0 : i1, j = n * 8 + 2 * t + (e & 1);
       if (j > i) s[n][e] = 0.f;
+      else if (TOKEN) s[n][e] *= ex2(s_cum[i] - s_cum[j]) * s_step[j];
       else if (!LR) s[n][e] *= ex2(log2_pow(ld2, i - j));
     }
   __syncthreads();  // keys are done with: their memory holds the tiles of phase two
 
   bf16* v_hi = (bf16*)keys;            // [64][kVS] values
   bf16* v_lo = v_hi + kC * kVS;
-  bf16* t_hi = v_lo + kC * kVS;        // [64][kVS] 64 channels of the state before the chunk
+  bf16* t_hi = TOKEN ? v_lo : v_lo + kC * kVS;  // [64][kVS] 64 channels of the state before the chunk
   bf16* t_lo = t_hi + kC * kVS;
   const uint32_t vh = smem_u32(v_hi + (lane & 15) * kVS + (lane >> 4) * 8), vl = smem_u32(v_lo + (lane & 15) * kVS + (lane >> 4) * 8);
   const uint32_t th = smem_u32(t_hi + (lane & 15) * kVS + (lane >> 4) * 8), tl = smem_u32(t_lo + (lane & 15) * kVS + (lane >> 4) * 8);
-  const float f0 = LR ? 1.f : ex2(log2_pow(ld2, i0 + 1)), f1 = LR ? 1.f : ex2(log2_pow(ld2, i1 + 1));
+  const float f0 = LR ? 1.f : ex2(TOKEN ? s_cum[i0] : log2_pow(ld2, i0 + 1)), f1 = LR ? 1.f : ex2(TOKEN ? s_cum[i1] : log2_pow(ld2, i1 + 1));
+  const float skip = a.skip ? a.skip[h] : 0.f;
   const float* st = chunk_state + ((int64_t)blockIdx.x * a.heads + h) * D * a.vdim;
   const bool live = warp * 16 < ch.n;
   for (int v0 = 0; v0 < a.vdim; v0 += kVT) {
@@ -429,7 +497,7 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
         }
         put_split8(t_hi + r * kVS + c, t_lo + r * kVS + c, f);
       }
-      if (d0 == 0) load_values(a, ch, h, v0, v_hi, v_lo);
+      if (d0 == 0) load_values<TOKEN>(a, ch, h, v0, v_hi, v_lo);
       __syncthreads();
       if (live) {
         const int n_ks = min(4, (DP - d0) / 16);
@@ -439,13 +507,20 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
             q_frag(d0 / 16 + ks, -1, hi, lo);
           } else {
             ldsm_x4(qh + (d0 / 16 + ks) * 32, hi[0], hi[1], hi[2], hi[3]);
-            ldsm_x4(ql + (d0 / 16 + ks) * 32, lo[0], lo[1], lo[2], lo[3]);
+            if (!TOKEN) ldsm_x4(ql + (d0 / 16 + ks) * 32, lo[0], lo[1], lo[2], lo[3]);
           }
 #pragma unroll
           for (int nv = 0; nv < 4; ++nv) {
             uint32_t b[4], c[4];
             ldsm_x4_trans(th + (ks * 16 * kVS + nv * 16) * 2, b[0], b[1], b[2], b[3]);
             ldsm_x4_trans(tl + (ks * 16 * kVS + nv * 16) * 2, c[0], c[1], c[2], c[3]);
+            if (TOKEN) {
+              mma_bf16_16816(o[2 * nv], hi, b[0], b[1]);
+              mma_bf16_16816(o[2 * nv + 1], hi, b[2], b[3]);
+              mma_bf16_16816(o[2 * nv], hi, c[0], c[1]);
+              mma_bf16_16816(o[2 * nv + 1], hi, c[2], c[3]);
+              continue;
+            }
             mma_split(o[2 * nv], hi, lo, b[0], b[1], c[0], c[1]);
             mma_split(o[2 * nv + 1], hi, lo, b[2], b[3], c[2], c[3]);
           }
@@ -470,6 +545,11 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
           for (int nv = 0; nv < 4; ++nv) {
             uint32_t b[4], c[4];
             ldsm_x4_trans(vh + (kk * 16 * kVS + nv * 16) * 2, b[0], b[1], b[2], b[3]);
+            if (TOKEN) {
+              mma_pair(o[2 * nv], hi, lo, b[0], b[1]);
+              mma_pair(o[2 * nv + 1], hi, lo, b[2], b[3]);
+              continue;
+            }
             ldsm_x4_trans(vl + (kk * 16 * kVS + nv * 16) * 2, c[0], c[1], c[2], c[3]);
             mma_split(o[2 * nv], hi, lo, b[0], b[1], c[0], c[1]);
             mma_split(o[2 * nv + 1], hi, lo, b[2], b[3], c[2], c[3]);
@@ -481,9 +561,15 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int r = e ? i1 : i0, c = i * 8 + 2 * t;
-          if (r < ch.n)
-            put_pair(a.o + (int64_t)(ch.row0 + r) * a.ld_o + (int64_t)h * a.vdim + v0 + c, o[i][2 * e] * a.q_scale,
-                     o[i][2 * e + 1] * a.q_scale, a.vdim - v0 - c);
+          if (r < ch.n) {
+            float x = o[i][2 * e] * a.q_scale, y = o[i][2 * e + 1] * a.q_scale;
+            if (TOKEN) {  // the values' own way around the state
+              const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(v_hi + r * kVS + c);
+              x = fmaf(skip, __low2float(v), x);
+              y = fmaf(skip, __high2float(v), y);
+            }
+            put_pair(a.o + (int64_t)(ch.row0 + r) * a.ld_o + (int64_t)h * a.vdim + v0 + c, x, y, a.vdim - v0 - c);
+          }
         }
     }
     __syncthreads();
@@ -494,14 +580,15 @@ recurrence_output_kernel(const Recurrence a, const RowRange* __restrict__ chunks
 static int pad16h(int n) { return (n + 15) / 16 * 16; }
 static size_t state_smem(const Recurrence& a) { return (size_t)2 * kC * (pad16h(a.dim) + 8 + kVS) * 2; }
 static size_t output_smem(const Recurrence& a) {
-  const size_t ks = (size_t)kC * (pad16h(a.dim) + 8) * 2, tiles = (size_t)4 * kC * kVS * 2;
+  const size_t ks = (size_t)kC * (pad16h(a.dim) + 8) * 2, tiles = (size_t)(a.dt ? 3 : 4) * kC * kVS * 2;
+  if (a.dt) return ks + std::max(ks, tiles);
   return a.decay ? 2 * ks + std::max(2 * ks, tiles)
                  : ks + (size_t)kC * (pad16h(a.dim) + 4) * 4 + std::max(3 * ks, tiles);
 }
 
 bool recurrence_chunks_supported(const Recurrence& a, hb_dtype dtype) {
   static const bool off = [] { const char* e = getenv("HB_RECURRENCE"); return e && e[0] == 't'; }();
-  return !off && dtype == HB_BF16 && output_smem(a) <= 224 * 1024 && state_smem(a) <= 224 * 1024 &&
+  return !off && dtype == HB_BF16 && !(a.dt && (a.silu_qkv || a.q_scale != 1.f)) && !(a.skip && !a.dt) && output_smem(a) <= 224 * 1024 && state_smem(a) <= 224 * 1024 &&
          (size_t)kC * a.rank * 4 <= 48 * 1024;
 }
 
@@ -513,25 +600,35 @@ int recurrence_chunks(cudaStream_t st, const Recurrence& a, const RecurrenceChun
     return HB_OK;
   };
   int rc;
-  if (!a.decay) {
+  if (a.dt) {
+    HB_CUDA_CHECK(launch_pdl(recurrence_step_kernel, dim3(nc, (unsigned)((a.heads + kStepHeads - 1) / kStepHeads)), dim3(256), 0, st,
+                             a, c.chunks, c.cum));
+    ++*launches;
+  } else if (!a.decay) {
     HB_CUDA_CHECK(launch_pdl(recurrence_decay_kernel, dim3(nc, (unsigned)((a.heads * a.dim + 255) / 256)), dim3(256),
                              (size_t)kC * a.rank * 4, st, a, c.chunks, c.cum));
     ++*launches;
   }
   const size_t ss = state_smem(a), os = output_smem(a);
-  if ((rc = opt_in(recurrence_state_kernel, ss))) return rc;
-  HB_CUDA_CHECK(launch_pdl(recurrence_state_kernel, dim3(nc, H, (unsigned)((a.vdim + kVT - 1) / kVT)), dim3(kT), ss, st, a,
-                           c.chunks, (const float*)c.cum, c.state));
   const int64_t per_head = (int64_t)a.dim * a.vdim;
   const int vec = a.vdim % 4 == 0 ? 4 : 1;
-  auto* scan = vec == 4 ? recurrence_scan_kernel<4> : recurrence_scan_kernel<1>;
-  HB_CUDA_CHECK(launch_pdl(scan, dim3((unsigned)((per_head / vec + 255) / 256), H, (unsigned)c.n_segs), dim3(256), 0, st, a,
-                           c.segs, c.chunks, (const float*)c.cum, c.state));
-  auto* out = a.decay ? recurrence_output_kernel<false> : recurrence_output_kernel<true>;
-  if ((rc = opt_in(out, os))) return rc;
-  HB_CUDA_CHECK(launch_pdl(out, dim3(nc, H), dim3(kT), os, st, a, c.chunks, (const float*)c.cum, (const float*)c.state));
-  *launches += 3;
-  return HB_OK;
+  auto run = [&](auto* own, auto* scan, auto* out) -> int {
+    if ((rc = opt_in(own, ss)) || (rc = opt_in(out, os))) return rc;
+    HB_CUDA_CHECK(launch_pdl(own, dim3(nc, H, (unsigned)((a.vdim + kVT - 1) / kVT)), dim3(kT), ss, st, a, c.chunks,
+                             (const float*)c.cum, c.state));
+    HB_CUDA_CHECK(launch_pdl(scan, dim3((unsigned)((per_head / vec + 255) / 256), H, (unsigned)c.n_segs), dim3(256), 0, st, a,
+                             c.segs, c.chunks, (const float*)c.cum, c.state));
+    HB_CUDA_CHECK(launch_pdl(out, dim3(nc, H), dim3(kT), os, st, a, c.chunks, (const float*)c.cum, (const float*)c.state));
+    *launches += 3;
+    return HB_OK;
+  };
+#define HB_RECURRENCE(MODE)                                                                                   \
+  return run(recurrence_state_kernel<MODE>, vec == 4 ? recurrence_scan_kernel<4, MODE> : recurrence_scan_kernel<1, MODE>, \
+             recurrence_output_kernel<MODE>)
+  if (a.dt) HB_RECURRENCE(kPerToken);
+  if (a.decay) HB_RECURRENCE(kConstant);
+  HB_RECURRENCE(kLowRank);
+#undef HB_RECURRENCE
 }
 
 }  // namespace hb

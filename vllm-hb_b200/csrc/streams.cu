@@ -49,7 +49,7 @@ __global__ void __launch_bounds__(kStreamThreads)
 streams_embed_kernel(float* __restrict__ x, T* __restrict__ h, const T* __restrict__ embed, const T* __restrict__ pos_table,
                      const uint32_t* __restrict__ ids, const int32_t* __restrict__ pos, const float* __restrict__ in,
                      const float* __restrict__ norm, float norm_offset, int S, int64_t W, int64_t ld_h, int64_t vocab,
-                     int64_t max_positions, float eps) {
+                     int64_t max_positions, float eps, float embed_scale) {
   pdl_trigger();
   pdl_grid_wait();
   __shared__ float red[33];
@@ -68,6 +68,7 @@ streams_embed_kernel(float* __restrict__ x, T* __restrict__ h, const T* __restri
     if (pr) load_vec<T, VEC>(b, pr + i);
 #pragma unroll
     for (int j = 0; j < VEC; ++j) {
+      a[j] *= embed_scale;
       if (pr) a[j] += b[j];
       const float u = in_sum * a[j];
       ss = fmaf(u, u, ss);
@@ -206,7 +207,7 @@ streams_mix_kernel(float* __restrict__ x, T* __restrict__ h, const float* __rest
 template <typename T, int VEC>
 __global__ void __launch_bounds__(kStreamThreads)
 streams_final_kernel(T* __restrict__ h, const float* __restrict__ x, const int32_t* __restrict__ want,
-                     const float* __restrict__ norm, float norm_offset, int S, int64_t W, int64_t ld_h, float eps) {
+                     const float* __restrict__ norm, float norm_offset, int S, int64_t W, int64_t ld_h, float eps, float scale) {
   pdl_trigger();
   pdl_grid_wait();
   extern __shared__ float s_u[];
@@ -226,7 +227,7 @@ streams_final_kernel(T* __restrict__ h, const float* __restrict__ x, const int32
     for (int j = 0; j < VEC; ++j) ss = fmaf(u[j], u[j], ss);
     store_vec<float, VEC>(s_u + i, u);
   }
-  const float r = inv_rms(block_sum(ss, red), W, eps);
+  const float r = scale * inv_rms(block_sum(ss, red), W, eps);
   for (int64_t i = (int64_t)threadIdx.x * VEC; i < W; i += kStreamThreads * VEC) {
     float u[VEC], w[VEC];
     load_vec<float, VEC>(u, s_u + i);
@@ -242,13 +243,12 @@ streams_final_kernel(T* __restrict__ h, const float* __restrict__ x, const int32
 template <typename T, bool WARP, int VEC>
 __global__ void __launch_bounds__(kStreamThreads)
 gated_group_norm_kernel(T* __restrict__ out, int64_t ld_out, const float* __restrict__ o, int64_t ld_o,
-                        const T* __restrict__ gate, int64_t ld_gate, const float* __restrict__ weight, int groups, int size,
-                        int gate_silu, float eps) {
+                        const T* __restrict__ gate, int64_t ld_gate, const float* __restrict__ weight, const GroupNorm n) {
   pdl_trigger();
   pdl_grid_wait();
   __shared__ float red[33];
   const int64_t row = blockIdx.x;
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, groups = n.groups, size = n.size;
   const int group = WARP ? blockIdx.y * (kStreamThreads / 32) + warp : blockIdx.y;
   const int first = (WARP ? lane : (int)threadIdx.x) * VEC, step = (WARP ? 32 : kStreamThreads) * VEC;
   if (WARP && group >= groups) return;
@@ -256,16 +256,27 @@ gated_group_norm_kernel(T* __restrict__ out, int64_t ld_out, const float* __rest
   const float* og = o + row * ld_o + at;
   const T* gg = gate + row * ld_gate + at;
   T* dst = out + row * ld_out + at;
+  if (n.own_weights) weight += at;
+  auto act = [&](float g) {
+    const float sg = 1.f / (1.f + expf(-g));
+    return n.gate_silu ? g * sg : sg;
+  };
   float ss = 0.f;
 #pragma unroll 4
   for (int i = first; i < size; i += step) {
     float f[VEC];
     load_vec<float, VEC>(f, og + i);
+    if (n.gate_first) {
+      float g[VEC];
+      load_vec<T, VEC>(g, gg + i);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) f[j] *= act(g[j]);
+    }
 #pragma unroll
     for (int j = 0; j < VEC; ++j) ss = fmaf(f[j], f[j], ss);
   }
   ss = WARP ? warp_sum(ss) : block_sum(ss, red);
-  const float r = inv_rms(ss, size, eps);
+  const float r = inv_rms(ss, size, n.eps);
 #pragma unroll 2
   for (int i = first; i < size; i += step) {
     float f[VEC], g[VEC], w[VEC];
@@ -273,10 +284,7 @@ gated_group_norm_kernel(T* __restrict__ out, int64_t ld_out, const float* __rest
     load_vec<T, VEC>(g, gg + i);
     load_vec<float, VEC>(w, weight + i);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) {
-      const float sg = 1.f / (1.f + expf(-g[j]));
-      f[j] = f[j] * r * w[j] * (gate_silu ? g[j] * sg : sg);
-    }
+    for (int j = 0; j < VEC; ++j) f[j] = f[j] * act(g[j]) * r * w[j];
     store_vec<T, VEC>(dst + i, f);
   }
 }
@@ -291,11 +299,12 @@ gated_group_norm_kernel(T* __restrict__ out, int64_t ld_out, const float* __rest
 
 int streams_embed(cudaStream_t st, float* x, void* h, const void* embed, const void* pos_table, const uint32_t* ids,
                   const int32_t* pos, const float* in, const float* norm, float norm_offset, int64_t rows, int streams,
-                  int64_t width, int64_t ld_h, int64_t vocab, int64_t max_positions, float eps, hb_dtype dtype) {
+                  int64_t width, int64_t ld_h, int64_t vocab, int64_t max_positions, float eps, hb_dtype dtype, float embed_scale) {
   HB_DISPATCH_LAYERED(dtype, T, {
     auto* k = width % 4 == 0 ? streams_embed_kernel<T, 4> : streams_embed_kernel<T, 1>;
     HB_CUDA_CHECK(launch_pdl(k, dim3((unsigned)rows), dim3(kStreamThreads), 0, st, x, (T*)h, (const T*)embed,
-                             (const T*)pos_table, ids, pos, in, norm, norm_offset, streams, width, ld_h, vocab, max_positions, eps));
+                             (const T*)pos_table, ids, pos, in, norm, norm_offset, streams, width, ld_h, vocab, max_positions, eps,
+                             embed_scale));
   });
   return HB_OK;
 }
@@ -342,21 +351,21 @@ int streams_mix(cudaStream_t st, float* x, void* h, const float* y, const float*
 }
 
 int streams_final(cudaStream_t st, void* h, const float* x, const int32_t* want, const float* norm, float norm_offset,
-                  int64_t n_want, int streams, int64_t width, int64_t ld_h, float eps, hb_dtype dtype) {
+                  int64_t n_want, int streams, int64_t width, int64_t ld_h, float eps, hb_dtype dtype, float scale) {
   if (n_want == 0) return HB_OK;
   HB_DISPATCH_LAYERED(dtype, T, {
     auto* k = width % 4 == 0 ? streams_final_kernel<T, 4> : streams_final_kernel<T, 1>;
     const int rc = row_smem(k, width);
     if (rc) return rc;
     HB_CUDA_CHECK(launch_pdl(k, dim3((unsigned)n_want), dim3(kStreamThreads), (size_t)width * 4, st, (T*)h, x, want, norm,
-                             norm_offset, streams, width, ld_h, eps));
+                             norm_offset, streams, width, ld_h, eps, scale));
   });
   return HB_OK;
 }
 
 int gated_group_norm(cudaStream_t st, void* out, int64_t ld_out, const float* o, int64_t ld_o, const void* gate,
-                     int64_t ld_gate, const float* weight, int64_t rows, int groups, int size, bool gate_silu, float eps,
-                     hb_dtype dtype) {
+                     int64_t ld_gate, const float* weight, int64_t rows, const GroupNorm& n, hb_dtype dtype) {
+  const int groups = n.groups, size = n.size;
   const bool warp = groups > 1 && size <= 1024;
   const unsigned gy = warp ? (unsigned)((groups + kStreamThreads / 32 - 1) / (kStreamThreads / 32)) : (unsigned)groups;
   HB_DISPATCH_LAYERED(dtype, T, {
@@ -366,7 +375,7 @@ int gated_group_norm(cudaStream_t st, void* out, int64_t ld_out, const float* o,
     auto* k = vec ? (warp ? gated_group_norm_kernel<T, true, 4> : gated_group_norm_kernel<T, false, 4>)
                   : (warp ? gated_group_norm_kernel<T, true, 1> : gated_group_norm_kernel<T, false, 1>);
     HB_CUDA_CHECK(launch_pdl(k, dim3((unsigned)rows, gy), dim3(kStreamThreads), 0, st, (T*)out, ld_out, o, ld_o,
-                             (const T*)gate, ld_gate, weight, groups, size, gate_silu ? 1 : 0, eps));
+                             (const T*)gate, ld_gate, weight, n));
   });
   return HB_OK;
 }
