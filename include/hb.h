@@ -303,9 +303,10 @@ int hb_attention_prepare(void* stream, const hb_attention_prep_args* a, int64_t 
  * vdim = rank and no V pool).  Row r of p holds at off_q the heads' queries [dim | rot_dim] and at off_c
  * [latent of rank | key part of rot_dim].  The latent is RMS-normed (weight norm [rank]), the key part
  * rotated (channel i with i+pairs), both go to the row's slot of k_cache [num_blocks, 16, rank+rot_dim];
- * the queries' rotated parts go to q, head h at q + r*ld_q + h*(rank+rot_dim) + rank.  fp32 inside. */
+ * the queries' rotated parts go back to their place and to q, head h at q + r*ld_q + h*(rank+rot_dim) +
+ * rank.  fp32 inside. */
 typedef struct hb_latent_prep_args {
-  const void* p;
+  void* p;
   int64_t ld;
   int off_q, off_c, heads, dim, rot_dim, rank;
   void* q;

@@ -1,7 +1,7 @@
 """Models described layer by layer beside the Llama family (and, for a mixture of experts, its
 Mixtral form) at equal width, feed-forward, depth and vocabulary.
 
-`python bench.py --workload latarax` or `biberax` runs it on one GPU: prefill of one long prompt and
+`python bench.py --workload latarax`, `biberax` or `badolix` runs it on one GPU: prefill of one long prompt and
 of several shorter ones, decode at several batch sizes, random weights and tokens.  For every kind of
 kernel it reports the time of a profiled step and the fraction of the roofline (the larger of bytes /
 measured HBM bandwidth and FLOPs / measured bf16 throughput, over the time).
@@ -37,8 +37,38 @@ def biberax_layers(heads, chunk, far, dense_ff, experts, top, ff, shared, layers
             for i in range(layers)]
 
 
+def badolix_layers(heads, window, keep, dense_ff, experts, top, ff, layers):
+    """Latent attention, a selective state space, windowed attention and a layer that shares its keys and
+    values, in turn; dense feed-forwards and experts alternate."""
+    rot = dict(base=500000.0, dims=128, scaling=dict(factor=8.0))
+    yarn = dict(base=10000.0, dims=64, scaling=dict(factor=4.0, original=4096, fast=32.0, slow=1.0))
+    attn = dict(heads=heads, kv_heads=heads // 4, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, rot=rot,
+                mask=dict(size=window, keep_first=keep))
+    latent = dict(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, rot=yarn)
+    mamba = dict(heads=4 * heads, vdim=64, state=128, groups=8, conv=4, norm_groups=8)
+    dense = {"kind": "dense", "ff": dense_ff}
+    moe = {"kind": "moe", "expert": dict(ff=ff), "router": dict(experts=experts, top=top, groups=dict(count=4, keep=2))}
+    out = []
+    for i in range(0, layers, 4):
+        out += [{"type": "latent_attention", "mixer": latent, "mlp": dense}, {"type": "mamba2", "mixer": mamba, "mlp": moe},
+                {"type": "attention", "mixer": attn, "mlp": dense}, {"type": "attention", "mixer": dict(attn, kv_from=i + 2), "mlp": moe}]
+    return out
+
+
 def sizes(design: str) -> list[dict]:
     """Layers of about 1.3B- and 8B-parameter models (dense ones; a mixture has more)."""
+    if design == "badolix":  # beside the designs its kernels are shared with or like
+        out = []
+        for small, other in zip(sizes("biberax"), sizes("latarax")):
+            llama, bib = small["llama"], small["biberax"]
+            width, layers, f = llama["hidden_size"], llama["num_hidden_layers"], bib["layers"][1]["mlp"]
+            experts, top, ff = f["router"]["experts"], f["router"]["top"], f["expert"]["ff"]
+            out.append({"name": small["name"],
+                        "badolix": {"architecture": "Badolix", "width": width, "vocab": VOCAB, "norm": {"eps": 1e-6},
+                                    "embedding": {"scale": 1.0}, "residual_mult": 1.0, "logit_scale": 1.0,
+                                    "layers": badolix_layers(width // 128, 1024, 16, llama["intermediate_size"], experts, top, ff, layers)},
+                        "biberax": bib, "latarax": other["latarax"], "llama": llama})
+        return out
     if design == "biberax":
         out = []
         for width, dense_ff, experts, top, ff, shared, layers in ((2048, 5632, 16, 4, 1408, 1408, 12),
@@ -82,6 +112,30 @@ def work(shape: dict, family: str, positions: list[np.ndarray], wanted: int) -> 
 
     def gemm(kind, n, k, m=rows, n_out=None, out=2):
         add(kind, 2.0 * n * k + 2.0 * m * k + out * m * (n_out or n), 2.0 * m * n * k)
+
+    def state_space(m, H):
+        inner, bc, heads = m["heads"] * m["vdim"], 2 * m["groups"] * m["state"], m["heads"]
+        st = heads * m["state"] * m["vdim"]
+        gemm("gemm_qkv", 2 * inner + bc + heads, H)
+        add("convolution", 4.0 * rows * (inner + bc) + 4.0 * len(positions) * (m["conv"] - 1) * (inner + bc))
+        add("recurrence", 8.0 * st * len(positions) + rows * (2.0 * (inner + bc + heads) + 4.0 * inner), 6.0 * st * rows)
+        add("norm", rows * inner * (4.0 + 2.0 + 2.0))
+        gemm("gemm_o_proj", H, inner, out=4)
+
+    def latent(m, H):
+        h, d, r, v, c = (m[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank"))
+        gemm("gemm_qkv", h * (d + r) + c + r, H)
+        add("rope_kv", 4.0 * rows * (h * r + c + r))
+        for p in positions:
+            n, span, seen = len(p), float(p[-1] + 1), keys_seen(p, 0, 0)
+            if n == 1:  # over the latent itself
+                add("attention", 2.0 * (c + r) * span + 2.0 * h * (2 * c + r), 2.0 * h * (2 * c + r) * seen)
+                add("latent", 2.0 * h * (d + v + 2 * c), 2.0 * h * c * (d + v))
+            else:       # keys and values of the heads grown out of the latents
+                add("attention", 2.0 * h * (d + v) * span + 2.0 * r * span + 2.0 * n * h * (d + r + v), 2.0 * h * (d + r + v) * seen)
+                add("latent", 2.0 * span * (c + h * (d + v)), 2.0 * span * h * c * (d + v))
+        add("latent", 2.0 * h * (d + v) * c)
+        gemm("gemm_o_proj", H, h * v, out=4)
 
     def attention(heads, kv, dim, vdim, window, keep, chunk=0, tied=False, gated=False):
         if chunk:
@@ -138,6 +192,36 @@ def work(shape: dict, family: str, positions: list[np.ndarray], wanted: int) -> 
                 add("experts_gate_up", 4.0 * active * F * H + 2.0 * picks * (H + F), 4.0 * picks * F * H)
                 add("experts_down", 2.0 * active * F * H + 2.0 * picks * (H + F), 2.0 * picks * F * H)
                 add("norm", (2.0 * picks + 2.0 * rows) * H)
+        add("norm", wanted * H * 6.0)
+        gemm("gemm_lm_head", shape["vocab"], H, m=wanted, out=4)
+        return w
+    if family == "badolix":
+        H = shape["width"]
+        for layer in shape["layers"]:
+            m, f = layer["mixer"], layer["mlp"]
+            if layer["type"] == "mamba2":
+                state_space(m, H)
+            elif layer["type"] == "latent_attention":
+                latent(m, H)
+            else:
+                q, v = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+                kv = 0 if "kv_from" in m else m["kv_heads"] * (m["dim"] + m["vdim"])
+                gemm("gemm_qkv", q + kv, H)
+                add("rope_kv", 4.0 * rows * (q + kv))
+                attention(m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["mask"]["size"], m["mask"]["keep_first"])
+                gemm("gemm_o_proj", H, v, out=4)
+            add("norm", 2 * rows * H * 14.0)
+            if f["kind"] == "dense":
+                gemm("gemm_gate_up", 2 * f["ff"], H, n_out=f["ff"])
+                gemm("gemm_down", H, f["ff"], out=4)
+            else:
+                E, top, F = f["router"]["experts"], f["router"]["top"], f["expert"]["ff"]
+                picks = rows * top
+                active = E * (1.0 - (1.0 - top / E) ** rows)
+                add("routing", 2.0 * E * H + 2.0 * rows * H * (2 + top))
+                add("experts_gate_up", 4.0 * active * F * H + 2.0 * picks * (H + F), 4.0 * picks * F * H)
+                add("experts_down", 2.0 * active * F * H + 2.0 * picks * (H + F), 2.0 * picks * F * H)
+                add("norm", (2.0 * picks - 2.0 * rows) * H)
         add("norm", wanted * H * 6.0)
         gemm("gemm_lm_head", shape["vocab"], H, m=wanted, out=4)
         return w
@@ -245,12 +329,12 @@ def run(hb, hbm_gbs: float, tflops: float, steps: int, warmup: int, design: str 
         if only and only not in size["name"]:
             continue
         entry = report[size["name"]] = {}
-        for family in (design, "llama", "mixtral"):
+        for family in [design] + [f for f in ("biberax", "latarax", "llama", "mixtral") if f != design]:
             shape = size.get(family)
             if not shape:
                 continue
             kw = dict(max_seq_len=4224, max_batch=rows, max_seqs=128, num_kv_blocks=128 * 128)
-            eng = hb.Engine.create_random_config(shape, **kw) if family == design else \
+            eng = hb.Engine.create_random_config(shape, **kw) if "architecture" in shape else \
                 hb.Engine.create_random(shape, **{k: v for k, v in kw.items() if k != "max_seqs"})
             res = entry[family] = {"parameters": eng.param_count()}
             rng = np.random.default_rng(0)

@@ -17,8 +17,7 @@
 #include <climits>
 
 #include "layered_ops.h"
-#include "mma_sync.cuh"
-#include "tc_core.cuh"
+#include "span_core.cuh"
 
 namespace hb {
 
@@ -27,64 +26,9 @@ constexpr int kThreads = 128;
 constexpr int kWarps = 4;
 constexpr int kRows = 64;      // query rows of a tile
 constexpr int kKeys = 64;      // keys of a tile step
-constexpr int kBS = HB_BLOCK_SIZE;
 constexpr int kSlice = 256;    // widest value slice
 constexpr int kRing = 3;       // 16-key stages of a warp (token kernel)
 constexpr int kMaxCluster = 8; // splits of a row that sum up in a cluster
-
-__host__ __device__ constexpr int pad16(int n) { return (n + 15) / 16 * 16; }
-
-// The blocks a CTA reads: [0, na) of the kept tokens, then [b0, b1].
-struct BlockRuns {
-  int na, b0, n;
-  __device__ __forceinline__ int block(int i) const { return i < na ? i : b0 + (i - na); }
-};
-__device__ __forceinline__ BlockRuns block_runs(int first_pos, int last_pos, const SpanAttention& a) {
-  BlockRuns r;
-  const int lo = a.first_seen(first_pos);
-  r.b0 = lo / kBS;
-  r.na = min((min(a.keep_first, lo) + kBS - 1) / kBS, r.b0);
-  r.n = r.na + last_pos / kBS - r.b0 + 1;
-  return r;
-}
-// lo: first_seen() of the position
-__device__ __forceinline__ bool visible(int key, int pos, int lo, int keep_first) {
-  return key <= pos && (key >= lo || key < keep_first);
-}
-// Every key of the block that starts at `key` is visible from all positions of a range: `first` is
-// the earliest, `lo` what the latest of them sees first (it grows with the position).
-__device__ __forceinline__ bool all_visible(int key, int first, int lo, int keep_first) {
-  return key + kBS - 1 <= first && (key >= lo || key + kBS <= keep_first);
-}
-constexpr float kLog2e = 1.4426950408889634f;
-// cap * tanh(s / cap) for a score and a cap in units of log2, tanh(y) = 1 - 2 / (1 + e^(2y)); k = 2 / softcap
-__device__ __forceinline__ float capped(float s, float cap, float k) { return cap - __fdividef(2.f * cap, 1.f + ex2(s * k)); }
-__device__ __forceinline__ float sigmoid_of(uint32_t bits16) {
-  const float z = __uint_as_float(bits16 << 16);  // a bf16 number
-  return __fdividef(1.f, 1.f + __expf(-z));
-}
-// A warp copies a 16-row block of `w` 16-byte vectors a row into rows of `stride` bytes; (j, c) is the
-// lane's first (row, vector), stepped without divisions.
-struct BlockCopy {
-  int w, j, c, dj, dc;
-  __device__ __forceinline__ BlockCopy(int width, int lane) : w(width / 8), j(lane / w), c(lane % w), dj(32 / w), dc(32 % w) {}
-  __device__ __forceinline__ void operator()(uint32_t dst, int stride, const __nv_bfloat16* src, int64_t src_row) const {
-    if (dc == 0 && dj > 0) {  // whole rows at a time: a lane stays in its column
-      dst += j * stride + c * 16;
-      src += j * src_row + c * 8;
-      for (int jj = j; jj < kBS; jj += dj, dst += dj * stride, src += dj * src_row) cp_async_16(dst, src);
-      return;
-    }
-    int jj = j, cc = c;
-#pragma unroll 4
-    while (jj < kBS) {
-      cp_async_16(dst + jj * stride + cc * 16, src + jj * src_row + cc * 8);
-      jj += dj;
-      cc += dc;
-      if (cc >= w) { cc -= w; ++jj; }
-    }
-  }
-};
 }  // namespace
 
 // NV: 16-column pairs of n-tiles, i.e. the value slice is at most 16 * NV wide.  FIX: keys and values
@@ -112,7 +56,7 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
   const RowRange tile = tiles[gridDim.x - 1 - blockIdx.x];  // later positions see more: they go first
   const int first_pos = a.pos[tile.row0], last_pos = first_pos + tile.n - 1;
   const BlockRuns runs = block_runs(first_pos, last_pos, a);
-  const int32_t* table = a.tables + (int64_t)tile.seg * a.max_blocks;
+  const int32_t* table = a.tables + (a.linear ? (int64_t)tile.seg : (int64_t)tile.seg * a.max_blocks);
   const int n_rows = tile.n * R, n_steps = (runs.n + kKeys / kBS - 1) / (kKeys / kBS);
 
   const __nv_bfloat16* q = (const __nv_bfloat16*)a.q + (int64_t)hs.first * D;
@@ -122,16 +66,20 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
     if (m < n_rows) v = *reinterpret_cast<const uint4*>(q + (int64_t)(tile.row0 + m / R) * a.ld_q + (m % R) * D + c);
     *reinterpret_cast<uint4*>(s_q + m * KS + c) = v;
   }
-  const BlockCopy copy_k(D, lane), copy_v(VW, lane);
+  const int DH = D - a.tail;  // channels of a key that are its head's own
+  const BlockCopy copy_k(DH, lane), copy_v(VW, lane), copy_t(max(a.tail, 8), lane);
   auto load = [&](int step) {  // every warp one block of 16 keys
     const int s = step % stages;
     // past the last block: any block will do, its keys are masked (positions beyond the row's)
     const int lb = runs.block(min(step * kWarps + warp, runs.n - 1));
-    int64_t phys = lb < a.max_blocks ? table[lb] : 0;
+    int64_t phys = lb < a.max_blocks ? (a.linear ? table[0] + lb : table[lb]) : 0;
     if (phys < 0 || phys >= a.num_blocks) phys = 0;  // never outside the pool
-    const int64_t slot = (phys * a.kv_heads + kvh) * kBS;
-    copy_k(smem_u32(s_k + (s * kKeys + warp * kBS) * KS), KS * 2, (const __nv_bfloat16*)a.kc + slot * D, D);
-    if (!tied) copy_v(smem_u32(s_v + (s * kKeys + warp * kBS) * VS), VS * 2, (const __nv_bfloat16*)a.vc + slot * a.vdim + v0, a.vdim);
+    const uint32_t k_dst = smem_u32(s_k + (s * kKeys + warp * kBS) * KS);
+    copy_k(k_dst, KS * 2, (const __nv_bfloat16*)a.kc + phys * a.k_step.block + kvh * a.k_step.head, a.k_step.token);
+    if (a.tail) copy_t(k_dst + DH * 2, KS * 2, (const __nv_bfloat16*)a.kt + phys * kBS * a.ld_kt, a.ld_kt);
+    if (!tied)
+      copy_v(smem_u32(s_v + (s * kKeys + warp * kBS) * VS), VS * 2,
+             (const __nv_bfloat16*)a.vc + phys * a.v_step.block + kvh * a.v_step.head + v0, a.v_step.token);
     else if (a.key_scale && lane < 4) cp_async_16(smem_u32(s_ks + s * kKeys + warp * kBS + lane * 4), a.key_scale + phys * kBS + lane * 4);
     cp_async_commit();
   };
@@ -653,9 +601,7 @@ static size_t tokens_smem(const SpanAttention& a) {
   const size_t merge = (size_t)kWarps * R * (VP + 4) * sizeof(float);
   return (size_t)16 * KS * 2 + std::max(ring, merge);
 }
-constexpr size_t kSmemCap = 224 * 1024;
-
-static bool span_mma_ok(const SpanAttention& a, hb_dtype dtype) {
+bool span_attention_mma_ok(const SpanAttention& a, hb_dtype dtype) {
   auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   static const bool simt = [] { const char* e = getenv("HB_ATTN"); return e && e[0] == 's'; }();
   return !simt && dtype == HB_BF16 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ld_q % 8 == 0 && a.ld_out % 2 == 0 && al(a.q) &&
@@ -664,15 +610,16 @@ static bool span_mma_ok(const SpanAttention& a, hb_dtype dtype) {
 }
 
 int span_attention_tile_positions(const SpanAttention& a, hb_dtype dtype) {
-  if (!span_mma_ok(a, dtype) || tiles_smem(a, 1) > kSmemCap) return 0;
+  if (!span_attention_mma_ok(a, dtype) || tiles_smem(a, 1) > kSmemCap) return 0;
   return kRows / sliced(a, kRows).slice;
 }
 int span_attention_tokens_slots(const SpanAttention& a) {
   constexpr int kSms = 148;
+  if (latent_tokens_supported(a, HB_BF16)) return kSms;
   return kSms * (int)std::max<size_t>(1, std::min<size_t>(8, (size_t)227 * 1024 / (tokens_smem(a) + 1024)));
 }
 bool span_attention_tokens_supported(const SpanAttention& a, hb_dtype dtype) {
-  return span_mma_ok(a, dtype) && tokens_smem(a) <= kSmemCap;
+  return latent_tokens_supported(a, dtype) || (span_attention_mma_ok(a, dtype) && tokens_smem(a) <= kSmemCap);
 }
 
 template <typename K>
@@ -681,11 +628,21 @@ static int opt_in(K kernel, size_t smem) {
   return HB_OK;
 }
 
-int span_attention_token_units(const SpanAttention& a) { return a.kv_heads * sliced(a, 16).slices(); }
+int span_attention_token_units(const SpanAttention& a) {
+  if (latent_tokens_supported(a, HB_BF16)) return latent_tokens_units(a);
+  return a.kv_heads * sliced(a, 16).slices();
+}
 
 int span_attention_tiles(cudaStream_t st, const SpanAttention& args, const RowRange* tiles, int n_tiles) {
   if (n_tiles == 0) return HB_OK;
-  const SpanAttention a = sliced(args, kRows);
+  SpanAttention a = sliced(args, kRows);
+  auto pool = [&](SpanAttention::Steps& s, int width) {
+    if (!s.token) s = {(int64_t)a.kv_heads * kBS * width, (int64_t)kBS * width, width};
+  };
+  pool(a.k_step, a.dim);
+  pool(a.v_step, a.vdim);
+  if (a.tail % 8 || a.k_step.token % 8 || a.v_step.token % 8 || a.k_step.head % 8 || a.v_step.head % 8 || a.ld_kt % 8)
+    return fail(HB_ERR_INVALID_ARG, "span attention: keys and values must lie on 16-byte boundaries");
   const int stages = tiles_smem(a, 2) <= kSmemCap ? 2 : 1;
   const size_t smem = tiles_smem(a, stages);
   const dim3 grid((unsigned)n_tiles, (unsigned)(a.kv_heads * a.slices()), (unsigned)((a.vdim + kSlice - 1) / kSlice));
@@ -710,6 +667,7 @@ int span_attention_tiles(cudaStream_t st, const SpanAttention& args, const RowRa
 
 int span_attention_tokens(cudaStream_t st, const SpanAttention& args, const int32_t* rows, int n_rows, int n_splits, float* part) {
   if (n_rows == 0) return HB_OK;
+  if (latent_tokens_supported(args, HB_BF16)) return latent_tokens(st, args, rows, n_rows, n_splits, part);
   const SpanAttention a = sliced(args, 16);
   const size_t smem = tokens_smem(a);
   const int slices = (a.vdim + kSlice - 1) / kSlice;
@@ -756,9 +714,12 @@ int span_attention_tokens(cudaStream_t st, const SpanAttention& args, const int3
   else HB_TOKENS(16);
 #undef HB_TOKENS
 #undef HB_TOKENS_OF
-  if (rc || n_splits == 1 || clustered) return rc;
+  return rc || n_splits == 1 || clustered ? rc : span_attention_merge(st, a, rows, n_rows, n_splits, part);
+}
+
+int span_attention_merge(cudaStream_t st, const SpanAttention& a, const int32_t* rows, int n_rows, int n_splits, const float* part) {
   HB_CUDA_CHECK(launch_pdl(span_attention_merge_kernel, dim3((unsigned)n_rows, (unsigned)a.heads), dim3(kThreads), 0, st, a, rows,
-                           n_splits, (const float*)part));
+                           n_splits, part));
   return HB_OK;
 }
 

@@ -5,18 +5,17 @@
 
 namespace hb {
 
-constexpr int kConvLanes = 32;                       // threads side by side in the channels
-constexpr int kConvRuns = 8;                         // threads side by side in the tokens
-constexpr int kConvRun = kRecChunk / kConvRuns;      // consecutive tokens of a thread
+constexpr int kConvThreads = 256;
 constexpr int kConvHeld = 4;                         // taps whose inputs stay in registers
 
-// CTA = (segment or chunk of one, kConvLanes * V channels).  The CTA of a segment's first tokens is the
+// CTA = (segment or chunk of one, LANES * V channels); the other threads share its tokens.  The CTA of a segment's first tokens is the
 // only one that reads the old state, and writes the new one at its end.  HELD: at most kConvHeld taps.
-template <typename T, int V, bool HELD>
-__global__ void __launch_bounds__(kConvLanes * kConvRuns)
+template <typename T, int V, bool HELD, int LANES>
+__global__ void __launch_bounds__(kConvThreads)
 short_conv_kernel(const ShortConv a, const int32_t* __restrict__ list, int n_list, const RowRange* __restrict__ chunks) {
   pdl_trigger();
-  const int c = (blockIdx.y * kConvLanes + threadIdx.x % kConvLanes) * V, run = threadIdx.x / kConvLanes;
+  constexpr int kConvRun = kRecChunk / (kConvThreads / LANES);  // consecutive tokens of a thread
+  const int c = (blockIdx.y * LANES + threadIdx.x % LANES) * V, run = threadIdx.x / LANES;
   const bool live = c < a.channels;
   const int back = a.taps - 1;
   float w[HELD ? kConvHeld : 1][V], bias[V];
@@ -105,17 +104,26 @@ int short_conv(cudaStream_t st, const ShortConv& a, const int32_t* list, int n_l
   const int n = (int)(16 / dtype_size(dtype));
   auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   const bool vec = a.channels % n == 0 && a.off % n == 0 && a.ld % n == 0 && a.ld_out % n == 0 && al(a.p) && al(a.out) && al(a.state);
-  auto launch = [&](auto* held, auto* any, int v) -> int {
-    const dim3 grid((unsigned)(n_list + n_chunks), (unsigned)((a.channels + kConvLanes * v - 1) / (kConvLanes * v)));
-    HB_CUDA_CHECK(launch_pdl(a.taps <= kConvHeld ? held : any, grid, dim3(kConvLanes * kConvRuns), 0, st, a, list, n_list, chunks));
+  // whole segments are a few tokens: their CTAs spread over the channels
+  auto launch = [&](auto* wide, auto* narrow, int v) -> int {
+    auto grid = [&](int cta, int lanes) { return dim3((unsigned)cta, (unsigned)((a.channels + lanes * v - 1) / (lanes * v))); };
+    if (n_list) HB_CUDA_CHECK(launch_pdl(wide, grid(n_list, 256), dim3(kConvThreads), 0, st, a, list, n_list, chunks));
+    if (n_chunks) HB_CUDA_CHECK(launch_pdl(narrow, grid(n_chunks, 32), dim3(kConvThreads), 0, st, a, list, 0, chunks));
     return HB_OK;
   };
-  if (dtype == HB_F32)
-    return vec ? launch(short_conv_kernel<float, 4, true>, short_conv_kernel<float, 4, false>, 4)
-               : launch(short_conv_kernel<float, 1, true>, short_conv_kernel<float, 1, false>, 1);
-  if (dtype == HB_BF16)
-    return vec ? launch(short_conv_kernel<__nv_bfloat16, 8, true>, short_conv_kernel<__nv_bfloat16, 8, false>, 8)
-               : launch(short_conv_kernel<__nv_bfloat16, 1, true>, short_conv_kernel<__nv_bfloat16, 1, false>, 1);
+  const bool held = a.taps <= kConvHeld;
+#define HB_CONV(T, V)                                                                                          \
+  return held ? launch(short_conv_kernel<T, V, true, 256>, short_conv_kernel<T, V, true, 32>, V)               \
+              : launch(short_conv_kernel<T, V, false, 256>, short_conv_kernel<T, V, false, 32>, V)
+  if (dtype == HB_F32) {
+    if (vec) HB_CONV(float, 4);
+    HB_CONV(float, 1);
+  }
+  if (dtype == HB_BF16) {
+    if (vec) HB_CONV(__nv_bfloat16, 8);
+    HB_CONV(__nv_bfloat16, 1);
+  }
+#undef HB_CONV
   return fail(HB_ERR_UNSUPPORTED_DTYPE, "short_conv runs in bf16 or f32");
 }
 

@@ -152,19 +152,14 @@ struct Loader {
     const size_t uk = (size_t)H * a.dim * C * e->es;
     int rc;
     if ((rc = vector(&l->latent_norm, mx.attn_latent_norm, C, 1.f))) return rc;
-    if ((rc = dev_alloc(e, &l->uk_t, uk)) || (rc = dev_alloc(e, &l->uv, (size_t)H * a.vdim * C * e->es))) return rc;
+    if ((rc = dev_alloc(e, &l->uk_t, uk)) || (rc = dev_alloc(e, &l->ukv, uk + (size_t)H * a.vdim * C * e->es))) return rc;
+    l->uv = (uint8_t*)l->ukv + uk;
     if ((rc = src.fetch_all(mx.attn_uv, H * a.vdim, C, l->uv, e->dtype))) return rc;
     e->named[mx.attn_uv] = {l->uv, H * a.vdim, C};
     m->params += H * (a.dim + a.vdim) * C;
-    void* rows = nullptr;
-    HB_CUDA_CHECK(cudaMalloc(&rows, uk));
-    rc = src.fetch_all(mx.attn_uk, H * a.dim, C, rows, e->dtype);
-    if (!rc) rc = transpose_matrices(e->stream, l->uk_t, rows, H, a.dim, C, e->es);
-    const cudaError_t ce = cudaStreamSynchronize(e->stream);
-    cudaFree(rows);
-    if (rc) return rc;
-    HB_CUDA_CHECK(ce);
-    return HB_OK;
+    if ((rc = src.fetch_all(mx.attn_uk, H * a.dim, C, l->ukv, e->dtype))) return rc;
+    e->named[mx.attn_uk] = {l->ukv, H * a.dim, C};
+    return transpose_matrices(e->stream, l->uk_t, l->ukv, H, a.dim, C, e->es);
   }
   // convolution weights [channels, taps] as [taps, channels], steps, decays
   int state_space(LayeredLayer* l, const MixerSpec& mx) {
@@ -340,11 +335,17 @@ static size_t layered_layout(const hb_engine* e, LayeredStep* s) {
   for (int k = 0; k < kTileKinds; ++k) s->off_tile[k] = l.take((size_t)s->n_tiles[k] * sizeof(RowRange));
   s->off_row_list = l.take((size_t)s->rows * 4);
   s->off_tables = l.take((size_t)s->segs * e->max_blocks_per_seq * 4);
+  s->off_expand_base = l.take(s->n_expand ? (size_t)s->segs * 4 : 0);
+  s->off_expand_list = l.take((size_t)s->n_expand * 4);
   return l.bytes;
 }
 
 // Segments of up to this many tokens go through the recurrence token by token.
 constexpr int kShortSegment = 8;
+// Latent attention of prompts: keys and values of the heads are grown out of the latents for portions of
+// at least this many tokens (fewer do not pay for it), in at most this much memory.
+constexpr int kExpandTokens = 32;
+constexpr size_t kExpandBytes = (size_t)512 << 20;
 // Decoded tokens: with fewer (row, kv head) units than this the keys may be split over several CTAs.
 constexpr int kSplitUnits = 592;
 
@@ -396,6 +397,32 @@ static LatentPrep latent_args(const hb_engine* e, size_t i, const LayeredStep& s
   p.norm = l.latent_norm; p.eps = m->spec.eps;
   p.rotation = l.rotation; p.pairs = (int)as.rotation.size(); p.rotation_gain = as.rotation_gain;
   return p;
+}
+
+// Attention of expanded segments: every head its own keys [dim | shared part] and values.
+static SpanAttention expanded_args(const hb_engine* e, size_t i, const LayeredStep& s) {
+  const LayeredModel* m = e->lm.get();
+  const MixerSpec& mx = m->spec.layers[i].mixer;
+  const AttentionSpec& as = mx.attn;
+  const LayeredLayer& l = m->layers[i];
+  SpanAttention a = span_args(e, i, s);
+  a.q = (const uint8_t*)m->proj + mx.aq.offset * e->es; a.ld_q = l.proj.N;
+  a.out = m->attn; a.ld_out = l.attn_o.K;
+  a.kv_heads = as.heads; a.dim = as.dim + as.rot_dim; a.vdim = as.vdim;
+  const int64_t row = (int64_t)as.heads * (as.dim + as.vdim);
+  a.kc = m->expand_kv; a.vc = (uint8_t*)m->expand_kv + (size_t)as.heads * as.dim * e->es;
+  a.k_step = {HB_BLOCK_SIZE * row, as.dim, row};
+  a.v_step = {HB_BLOCK_SIZE * row, as.vdim, row};
+  a.linear = 1; a.tables = (const int32_t*)(e->d_inputs + s.off_expand_base); a.num_blocks = m->expand_blocks;
+  a.tail = as.rot_dim; a.kt = (const uint8_t*)m->expand_latent + (size_t)as.rank * e->es; a.ld_kt = as.key_width();
+  return a;
+}
+static TcHeads expand_rows(const AttentionSpec& a) {
+  TcHeads h;
+  h.heads = 1;
+  h.ldx = h.x_step = a.key_width();
+  h.ldy = h.y_step = (int64_t)a.heads * (a.dim + a.vdim);
+  return h;
 }
 
 // The products of latent attention, head by head: W_uk^T on the queries' first parts, W_uv on what the
@@ -534,10 +561,11 @@ static int issue_attention(hb_engine* e, const SpanAttention& a, int kind, const
   const int64_t longest = span > 0 ? span + a.keep_first : a.max_blocks * HB_BLOCK_SIZE;
   const int64_t blocks = std::min<int64_t>(longest / HB_BLOCK_SIZE + 2, a.max_blocks), units = (int64_t)s.n_token_rows * span_attention_token_units(a);
   // as many as are resident at once, every one with some blocks for each of its warps
+  const bool latent = latent_tokens_supported(a, e->dtype);
   int64_t splits = std::min<int64_t>(std::min(kSplitUnits, span_attention_tokens_slots(a)) / units, (blocks + 7) / 8);
-  splits = std::max<int64_t>(1, std::min<int64_t>(splits, 16));
-  if (splits > 8 && blocks < 1024) splits = 8;  // what a cluster sums up
-  if (splits > 8) ++e->last_launches;  // more than a cluster sums up
+  splits = std::max<int64_t>(1, std::min<int64_t>(splits, latent ? 64 : 16));
+  if (splits > 8 && blocks < 1024 && !latent) splits = 8;  // what a cluster sums up
+  if (splits > (latent ? 1 : 8)) ++e->last_launches;  // a kernel sums up
   return span_attention_tokens(st, a, rows, s.n_token_rows, (int)splits, m->attn_part);
 }
 
@@ -556,6 +584,24 @@ static int issue_recurrence(hb_engine* e, const Recurrence& r, const LayeredStep
   return recurrence_chunks(e->stream, r, c, &e->last_launches);
 }
 
+// Index of the kind of tiles a layer takes; where there are as many as there are lists, the one with the
+// most positions that are not too many (-1: none).
+static int tile_kind(LayeredModel* m, int positions, TileKind::Which which) {
+  if (positions < 1) return -1;
+  std::vector<TileKind>& kinds = m->tile_kinds;
+  const TileKind want{positions, which};
+  auto at = std::find(kinds.begin(), kinds.end(), want);
+  if (at != kinds.end()) return (int)(at - kinds.begin());
+  if ((int)kinds.size() < kTileKinds) {
+    kinds.push_back(want);
+    return (int)kinds.size() - 1;
+  }
+  int best = -1;
+  for (size_t k = 0; k < kinds.size(); ++k)
+    if (kinds[k].which == which && kinds[k].positions <= positions && (best < 0 || kinds[k].positions > kinds[best].positions)) best = (int)k;
+  return best;
+}
+
 static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   LayeredModel* m = e->lm.get();
   const LayeredSpec& s = m->spec;
@@ -572,7 +618,8 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   m->row_cap = R;
   m->max_chunks = e->max_batch / kRecChunk + std::min(m->max_segs, e->max_batch / (kShortSegment + 1)) + 1;
   int64_t max_attn = 0, max_rec = 0, max_o = 0, max_ffp = 0, max_cum = 0, max_state = 0, max_part = 0;
-  int64_t max_experts = 0, max_top = 0, max_eff = 0, max_tiles = 0, max_conv = 0, max_latent_q = 0, max_latent_o = 0;
+  int64_t max_experts = 0, max_top = 0, max_eff = 0, max_tiles = 0, max_conv = 0, max_latent_q = 0, max_latent_o = 0, max_expand_row = 0,
+          max_expand_latent = 0;
   for (size_t i = 0; i < s.layers.size(); ++i) {
     LayeredLayer& l = m->layers[i];
     const MixerSpec& mx = s.layers[i].mixer;
@@ -603,6 +650,13 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
         max_latent_o = std::max(max_latent_o, (int64_t)a.heads * a.rank);
         l.latent_tc = e->use_tc && gemm_tc_heads_supported(a.rank, a.dim, false, latent_q_heads(l, a)) &&
                       gemm_tc_heads_supported(a.vdim, a.rank, false, latent_v_heads(l, a));
+        // over the latent a row and key cost more than with a head's own keys and values
+        l.expand = l.latent_tc && gemm_tc_heads_supported(a.heads * (a.dim + a.vdim), a.rank, false, expand_rows(a)) &&
+                   3 * a.rank > a.dim + 2 * a.vdim;
+        if (l.expand) {
+          max_expand_row = std::max(max_expand_row, (int64_t)a.heads * (a.dim + a.vdim));
+          max_expand_latent = std::max(max_expand_latent, (int64_t)a.key_width());
+        }
       }
       if (l.rel && (rc = build_distance_bias(e, &l, a, e->max_blocks_per_seq * HB_BLOCK_SIZE))) return rc;
     }
@@ -642,6 +696,14 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   if ((rc = dev_alloc(e, &m->attn, (size_t)R * max_attn * es, true))) return rc;
   if ((rc = dev_alloc(e, &m->rec, (size_t)R * max_rec * es, true))) return rc;
   if ((rc = dev_alloc(e, (void**)&m->o, (size_t)R * max_o * 4, true))) return rc;
+  if (max_expand_row) {
+    m->expand_blocks = std::min<int64_t>((int64_t)(kExpandBytes / ((size_t)max_expand_row * es * HB_BLOCK_SIZE)),
+                                         std::min(e->num_blocks, e->max_blocks_per_seq * m->max_segs));
+    m->expand_blocks = std::max<int64_t>(8, pad_to(m->expand_blocks, 8));  // whole batch tiles
+    const size_t rows = (size_t)m->expand_blocks * HB_BLOCK_SIZE;
+    if ((rc = dev_alloc(e, &m->expand_kv, rows * max_expand_row * es, true))) return rc;
+    if ((rc = dev_alloc(e, &m->expand_latent, rows * max_expand_latent * es, true))) return rc;
+  }
   if (max_conv && (rc = dev_alloc(e, &m->conv, (size_t)R * max_conv * es, true))) return rc;
   if (max_latent_q && (rc = dev_alloc(e, &m->latent_q, (size_t)R * max_latent_q * es, true))) return rc;
   if (max_latent_o && (rc = dev_alloc(e, &m->latent_o, (size_t)R * max_latent_o * es, true))) return rc;
@@ -652,17 +714,11 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   }
   for (size_t i = 0; i < s.layers.size(); ++i)
     if (s.layers[i].mixer.has_attn) {
+      LayeredLayer& l = m->layers[i];
       const int tp = span_attention_tile_positions(span_args(e, i, LayeredStep()), e->dtype);
-      std::vector<int>& sizes = m->tile_sizes;
-      auto at = std::find(sizes.begin(), sizes.end(), tp);
-      if (tp < 1) continue;
-      if (at == sizes.end() && (int)sizes.size() < kTileKinds) at = sizes.insert(sizes.end(), tp);
-      if (at == sizes.end()) {  // as many sizes as there are lists: the largest that is small enough
-        for (auto k = sizes.begin(); k != sizes.end(); ++k)
-          if (*k < tp && (at == sizes.end() || *k > *at)) at = k;
-        if (at == sizes.end()) continue;
-      }
-      m->layers[i].tile_kind = (int)(at - sizes.begin());
+      if (l.expand) l.expand_kind = tile_kind(m, span_attention_tile_positions(expanded_args(e, i, LayeredStep()), e->dtype), TileKind::kExpanded);
+      l.expand = l.expand_kind >= 0;
+      l.tile_kind = tile_kind(m, tp, l.expand ? TileKind::kNotExpanded : TileKind::kAll);
     }
   if ((rc = dev_alloc(e, (void**)&m->y1, (size_t)R * m->Hp * 4, true))) return rc;
   if ((rc = dev_alloc(e, (void**)&m->y2, (size_t)R * m->Hp * 4, true))) return rc;
@@ -694,7 +750,8 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   cap.want = e->max_batch;
   cap.segs = cap.n_long = m->max_segs;
   cap.n_chunks = m->max_chunks;
-  for (size_t k = 0; k < m->tile_sizes.size(); ++k) cap.n_tiles[k] = e->max_batch / m->tile_sizes[k] + m->max_segs;
+  for (size_t k = 0; k < m->tile_kinds.size(); ++k) cap.n_tiles[k] = e->max_batch / m->tile_kinds[k].positions + m->max_segs;
+  cap.n_expand = (int)m->expand_blocks;
   e->inputs_bytes = layered_layout(e, &cap);
   if ((rc = dev_alloc(e, (void**)&e->d_inputs, e->inputs_bytes, true))) return rc;
   HB_CUDA_CHECK(cudaMallocHost((void**)&e->h_inputs, e->inputs_bytes));
@@ -763,6 +820,27 @@ static int layered_plans(hb_engine* e, int rows, LayeredPlans** out) {
   return HB_OK;
 }
 
+static int layered_expand_plans(hb_engine* e, int blocks, std::vector<TcGemmPlan>** out) {
+  LayeredModel* m = e->lm.get();
+  const int64_t rows = (int64_t)blocks * HB_BLOCK_SIZE, M = std::min<int64_t>(pad_to(rows, rows <= 1024 ? 128 : 512), m->expand_blocks * HB_BLOCK_SIZE);
+  auto it = m->expand_plans.find((int)M);
+  if (it != m->expand_plans.end()) { *out = &it->second; return HB_OK; }
+  std::vector<TcGemmPlan> p(m->layers.size());
+  size_t ws = 0;
+  for (size_t i = 0; i < m->layers.size(); ++i) {
+    if (!m->layers[i].expand) continue;
+    const AttentionSpec& a = m->spec.layers[i].mixer.attn;
+    const TcHeads h = expand_rows(a);
+    const int rc = gemm_tc_plan(&p[i], m->expand_latent, m->layers[i].ukv, M, h.ldy, a.rank, kEpiStore, false, e->device, 0, nullptr, &h);
+    if (rc) return rc;
+    ws = std::max(ws, p[i].workspace_bytes());
+  }
+  const int rc = ensure_gemm_workspace(e, ws);
+  if (rc) return rc;
+  *out = &m->expand_plans.emplace((int)M, std::move(p)).first->second;
+  return HB_OK;
+}
+
 static int layered_head_plan(hb_engine* e, int want, TcGemmPlan** out) {
   LayeredModel* m = e->lm.get();
   const int M = (int)std::min<int64_t>(row_bucket(want), pad_to(e->max_logits_rows, 16));
@@ -789,9 +867,25 @@ static int layered_prepare(hb_engine* e, const StepBatch& batch, StepExec* x) {
     if (t.n <= kShortSegment) ++s.n_short;
     else { ++s.n_long; s.n_chunks += (t.n + kRecChunk - 1) / kRecChunk; }
     if (t.n == 1) ++s.n_token_rows;
-    else
-      for (size_t k = 0; k < m->tile_sizes.size(); ++k) s.n_tiles[k] += (t.n + m->tile_sizes[k] - 1) / m->tile_sizes[k];
   }
+  // expanded segments: as many as the buffers hold
+  std::vector<int32_t> expand_base(batch.segs.size(), -1);
+  s.n_not_expanded = s.rows;
+  for (int g = 0; g < s.segs; ++g) {
+    const StepSeg& t = batch.segs[g];
+    const int64_t blocks = (t.pos0 + t.n - 1) / HB_BLOCK_SIZE + 1;
+    if (t.n >= kExpandTokens && s.n_expand + blocks <= m->expand_blocks) {
+      expand_base[g] = s.n_expand;
+      s.n_expand += (int)blocks;
+      s.n_not_expanded -= t.n;
+    }
+  }
+  auto cut = [&](int g, const TileKind& k) {  // whether a segment is cut into tiles of this kind
+    return batch.segs[g].n > 1 && (k.which == TileKind::kAll || (k.which == TileKind::kExpanded) == (expand_base[g] >= 0));
+  };
+  for (int g = 0; g < s.segs; ++g)
+    for (size_t k = 0; k < m->tile_kinds.size(); ++k)
+      if (cut(g, m->tile_kinds[k])) s.n_tiles[k] += (batch.segs[g].n + m->tile_kinds[k].positions - 1) / m->tile_kinds[k].positions;
   x->rows = batch.rows;
   x->logits_compact = true;
   x->input_bytes = layered_layout(e, &s);
@@ -820,9 +914,10 @@ static int layered_prepare(hb_engine* e, const StepBatch& batch, StepExec* x) {
       for (int i = 0; i < t.n; i += kRecChunk)
         chunks[n_chunks++] = {g, t.row0 + i, std::min(kRecChunk, t.n - i), l.n++};
     }
-    for (size_t k = 0; t.n > 1 && k < m->tile_sizes.size(); ++k) {
+    for (size_t k = 0; k < m->tile_kinds.size(); ++k) {
+      if (!cut(g, m->tile_kinds[k])) continue;
       RowRange* tiles = (RowRange*)(in + s.off_tile[k]);
-      const int size = m->tile_sizes[k];
+      const int size = m->tile_kinds[k].positions;
       for (int i = 0; i < t.n; i += size) tiles[n_tiles[k]++] = {g, t.row0 + i, std::min(size, t.n - i), i / size};
     }
     for (int i = 0; i < t.n; ++i) {
@@ -836,11 +931,14 @@ static int layered_prepare(hb_engine* e, const StepBatch& batch, StepExec* x) {
     const int64_t need = (t.pos0 + t.n - 1) / HB_BLOCK_SIZE + 1;
     int32_t* row = tables + (size_t)g * e->max_blocks_per_seq;
     for (int64_t k = 0; k < need; ++k) row[k] = (int32_t)t.blocks[k];
+    if (s.n_expand) ((int32_t*)(in + s.off_expand_base))[g] = expand_base[g];
+    if (expand_base[g] >= 0) std::copy(row, row + need, (int32_t*)(in + s.off_expand_list) + expand_base[g]);
   }
   std::copy(batch.want.begin(), batch.want.end(), (int32_t*)(in + s.off_want));
   if (e->use_tc) {
     int rc;
     if ((rc = layered_plans(e, s.rows, &s.plans))) return rc;
+    if (s.n_expand && (rc = layered_expand_plans(e, s.n_expand, &s.expand_plans))) return rc;
     if (s.want && (rc = layered_head_plan(e, s.want, &s.head_plan))) return rc;
   }
   // a step of decoded tokens whose logits are all wanted replays from a graph
@@ -927,7 +1025,8 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
         if (l.latent_tc) return gemm_tc_run((*plans)[i], st, Y, h.ldy, e->d_gemm_ws, e->d_err);
         return gemm_simt_heads(st, Y, X, w, rows, N, K, e->dtype, false, h);
       };
-      if (as.rank && (rc = heads(pl ? &pl->latent_q : nullptr, m->latent_q, at(m->proj, mx.aq.offset), l.uk_t, as.rank, as.dim,
+      const bool expand = l.expand && s.n_expand, latent = as.rank && !(expand && s.n_not_expanded == 0);
+      if (latent && (rc = heads(pl ? &pl->latent_q : nullptr, m->latent_q, at(m->proj, mx.aq.offset), l.uk_t, as.rank, as.dim,
                                  latent_q_heads(l, as)))) return rc;
       prof_mark(e, kCatRopeKv);
       AttentionPrep prep;
@@ -937,9 +1036,19 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
       else rc = span_kv_write(st, a, at(m->proj, mx.ak.offset), at(m->proj, mx.av.offset), ldp, slots, rows, e->dtype);
       if (rc) return rc;
       prof_mark(e, kCatAttention);
-      if ((rc = issue_attention(e, a, l.tile_kind, s))) return rc;
-      if (as.rank && (rc = heads(pl ? &pl->latent_v : nullptr, m->attn, m->latent_o, l.uv, as.vdim, as.rank, latent_v_heads(l, as))))
+      if ((!as.rank || latent) && (rc = issue_attention(e, a, l.tile_kind, s))) return rc;
+      if (latent && (rc = heads(pl ? &pl->latent_v : nullptr, m->attn, m->latent_o, l.uv, as.vdim, as.rank, latent_v_heads(l, as))))
         return rc;
+      if (expand) {  // (after the product above, which writes all rows)
+        prof_mark(e, kCatLatent);
+        if ((rc = latent_gather(st, m->expand_latent, e->kc[l.kv_pool], (const int32_t*)(in + s.off_expand_list), s.n_expand,
+                                as.key_width(), e->num_blocks, e->dtype))) return rc;
+        if ((rc = gemm_tc_run((*s.expand_plans)[i], st, m->expand_kv, expand_rows(as).ldy, e->d_gemm_ws, e->d_err))) return rc;
+        prof_mark(e, kCatAttention);
+        if ((rc = span_attention_tiles(st, expanded_args(e, i, s), (const RowRange*)(in + s.off_tile[l.expand_kind]),
+                                       s.n_tiles[l.expand_kind]))) return rc;
+        e->last_launches += 3;
+      }
       prof_mark(e, kCatGemmO);
       if ((rc = gemm(pl ? &pl->attn_o : nullptr, i, y, m->attn, l.attn_o, true))) return rc;
       ++e->last_launches;  // the K/V write
@@ -962,7 +1071,7 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
         prof_mark(e, kCatConv);
         if ((rc = short_conv(st, c, (const int32_t*)(in + s.off_short), s.n_short, (const RowRange*)(in + s.off_chunk), s.n_chunks,
                              e->dtype))) return rc;
-        ++e->last_launches;
+        e->last_launches += (s.n_short ? 1 : 0) + (s.n_chunks ? 1 : 0);
         r.p = m->conv; r.ld = c.ld_out;
         r.off_v = 0; r.off_k = rs.heads * rs.vdim; r.off_q = r.off_k + rs.qk_heads * rs.dim;
         r.dt = at(m->proj, mx.rdt.offset); r.ld_dt = ldp;

@@ -184,7 +184,8 @@ struct LayeredLayer {
   int dist_len = 0, buckets = 0;
   // latent attention: per head W_uk^T [rank, dim] and W_uv [vdim, rank]; whether the tensor-core kernel
   // takes these products
-  void *uk_t = nullptr, *uv = nullptr;
+  void *uk_t = nullptr, *ukv = nullptr, *uv = nullptr;  // ukv [heads * dim | heads * vdim, rank]: W_uk, then W_uv
+  bool expand = false;                       // prompts attend to keys and values of the heads grown out of the latents
   float* latent_norm = nullptr;
   bool latent_tc = false;
   // selective state space
@@ -193,7 +194,7 @@ struct LayeredLayer {
   float *gate_b = nullptr, *up_b = nullptr, *down_b = nullptr;  // biases of a dense feed-forward
   LayeredExperts moe;
   int kv_pool = -1;                          // index into hb_engine::kc / vc
-  int tile_kind = -1;                        // index into LayeredModel::tile_sizes (-1: row by row)
+  int tile_kind = -1, expand_kind = -1;      // indices into LayeredModel::tile_kinds (-1: row by row)
   float* state = nullptr;                    // [slots, heads, dim, vdim]
   SublayerMix sub1, sub2;
 };
@@ -208,7 +209,13 @@ struct LayeredGraph {
   int64_t launches = 0;
 };
 
-constexpr int kTileKinds = 4;  // different sizes of attention tiles in one model
+// Tiles of query positions: how many positions one has, and which segments are cut into them.
+struct TileKind {
+  int positions;
+  enum Which { kAll, kNotExpanded, kExpanded } which;
+  bool operator==(const TileKind& o) const { return positions == o.positions && which == o.which; }
+};
+constexpr int kTileKinds = 6;  // different kinds in one model
 
 // Where a step's inputs lie in the (pinned and device) input block, and what it contains.
 struct LayeredStep {
@@ -217,12 +224,16 @@ struct LayeredStep {
   int n_chunks = 0;       // chunks of the longer segments (chunked recurrence kernels)
   int n_long = 0;         // longer segments
   int n_tiles[kTileKinds] = {0};  // query tiles of the tiled attention kernel, by tile size
+  int n_expand = 0;       // blocks of the contexts whose keys and values are grown out of latents
+  int n_not_expanded = 0; // rows of the other segments
   int n_token_rows = 0;   // rows that are single decoded tokens (first in the list of rows)
   bool decode = false;    // every segment is one token
   size_t off_ids = 0, off_pos = 0, off_slots = 0, off_row_seg = 0, off_want = 0, off_seg = 0, off_short = 0,
-         off_long = 0, off_chunk = 0, off_tile[kTileKinds] = {0}, off_row_list = 0, off_tables = 0;
+         off_long = 0, off_chunk = 0, off_tile[kTileKinds] = {0}, off_row_list = 0, off_tables = 0,
+         off_expand_base = 0, off_expand_list = 0;
   LayeredPlans* plans = nullptr;
   TcGemmPlan* head_plan = nullptr;
+  std::vector<TcGemmPlan>* expand_plans = nullptr;  // by layer
 };
 
 struct LayeredModel {
@@ -258,7 +269,11 @@ struct LayeredModel {
   int64_t moe_places = 0;
   int32_t *moe_count = nullptr, *moe_first = nullptr, *moe_tiles = nullptr;
   int max_segs = 0, max_chunks = 0;
-  std::vector<int> tile_sizes;               // positions of an attention tile, as the layers need them
+  std::vector<TileKind> tile_kinds;          // as the layers need them
+  // contexts of prompts whose latents are expanded: the latents side by side, keys and values of all heads
+  int64_t expand_blocks = 0;                 // capacity
+  void *expand_latent = nullptr, *expand_kv = nullptr;
+  std::map<int, std::vector<TcGemmPlan>> expand_plans;  // by rows bucket
   std::map<int, LayeredPlans> plans;         // by rows bucket
   std::map<int, TcGemmPlan> head_plans;      // by wanted-rows bucket
   std::map<int, LayeredGraph> graphs;        // by number of decoded sequences

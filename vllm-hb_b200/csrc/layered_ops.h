@@ -88,6 +88,16 @@ struct SpanAttention {
   const float* sink = nullptr;
   const void* gate = nullptr;
   int64_t ld_gate = 0;
+  // Where keys and values lie, in elements: token j of a block at block * step.block + head * step.head +
+  // j * step.token (all zero: the pools above).  With `linear` tables holds one number per segment and
+  // its blocks follow one another from there.  The last `tail` channels of every key are one vector per
+  // token for all heads, rows of kt of stride ld_kt numbered like the tokens.  (span_attention_tiles only.)
+  struct Steps {
+    int64_t block = 0, head = 0, token = 0;
+  } k_step, v_step;
+  int linear = 0, tail = 0;
+  const void* kt = nullptr;
+  int64_t ld_kt = 0;
   // first position a query at `pos` sees besides the first keep_first
   __host__ __device__ __forceinline__ int first_seen(int pos) const {
     if (chunk > 0) return pos - pos % chunk;
@@ -128,6 +138,14 @@ int span_attention_tokens_slots(const SpanAttention& a);
 bool span_attention_tokens_supported(const SpanAttention& a, hb_dtype dtype);
 int span_attention_tiles(cudaStream_t st, const SpanAttention& a, const RowRange* tiles, int n_tiles);
 int span_attention_tokens(cudaStream_t st, const SpanAttention& a, const int32_t* rows, int n_rows, int n_splits, float* part);
+// Whether sizes and alignments suit the tensor-core kernels; the sum of a row's split partials.
+bool span_attention_mma_ok(const SpanAttention& a, hb_dtype dtype);
+int span_attention_merge(cudaStream_t st, const SpanAttention& a, const int32_t* rows, int n_rows, int n_splits, const float* part);
+// Per-token kernel for wide values inside the keys (attention_latent.cu); span_attention_tokens takes it
+// where it is supported.
+bool latent_tokens_supported(const SpanAttention& a, hb_dtype dtype);
+int latent_tokens_units(const SpanAttention& a);
+int latent_tokens(cudaStream_t st, const SpanAttention& a, const int32_t* rows, int n_rows, int n_splits, float* part);
 
 // ----------------------------------------------- queries and keys of a step (attention_prep.cu)
 // One pass over projection rows: biases added, RMS norms over all query and all key rows, or a
@@ -157,11 +175,11 @@ struct AttentionPrep {
 // [dim | rot_dim] channels (head h at off_q + h * (dim + rot_dim)) and, from off_c on, the latent of
 // `rank` channels and a key part of rot_dim channels that all heads share.  The latent is RMS-normed
 // (weight norm), the key part rotated, and both go to the token's slot of kc [num_blocks, 16, rank +
-// rot_dim]; the rotated parts of the queries go to q, head h at q + r * ld_q + h * (rank + rot_dim) +
-// rank.  (The other `rank` channels there come from a product of heads: W_uk^T on the first dim
+// rot_dim]; the rotated parts of the queries go back to their place and to q, head h at q + r * ld_q + h *
+// (rank + rot_dim) + rank.  (The other `rank` channels there come from a product of heads: W_uk^T on the first dim
 // channels, so that a query meets the latent itself.)
 struct LatentPrep {
-  const void* p = nullptr;
+  void* p = nullptr;
   int64_t ld = 0;
   int off_q = 0, off_c = 0;
   int heads = 0, dim = 0, rot_dim = 0, rank = 0;
@@ -178,6 +196,9 @@ struct LatentPrep {
   float rotation_gain = 1.f;
 };
 int latent_prepare(cudaStream_t st, const LatentPrep& a, int64_t rows, hb_dtype dtype);
+// Rows of whole contexts side by side: block i of dst (16 rows of `width` elements) is block list[i] of pool.
+int latent_gather(cudaStream_t st, void* dst, const void* pool, const int32_t* list, int n_blocks, int width, int64_t num_blocks,
+                  hb_dtype dtype);
 // dst [n, cols, rows] = src [n, rows, cols] transposed, elements of es bytes (2 or 4).
 int transpose_matrices(cudaStream_t st, void* dst, const void* src, int64_t n, int64_t rows, int64_t cols, size_t es);
 int attention_prepare(cudaStream_t st, const AttentionPrep& a, int64_t rows, hb_dtype dtype);
