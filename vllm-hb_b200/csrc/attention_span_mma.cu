@@ -31,14 +31,15 @@ constexpr int kRing = 3;       // 16-key stages of a warp (token kernel)
 constexpr int kMaxCluster = 8; // splits of a row that sum up in a cluster
 }  // namespace
 
-// NV: 16-column pairs of n-tiles, i.e. the value slice is at most 16 * NV wide.  FIX: keys and values
-// are 16 * NV wide exactly, known to the compiler.
-template <int NV, bool EXT, bool FIX>
+// NV: 16-column pairs of n-tiles, i.e. the value slice is at most 16 * NV wide.  DK > 0: keys are DK and
+// values 16 * NV wide exactly, known to the compiler.
+template <int NV, bool EXT, int DK>
 __global__ void __launch_bounds__(kThreads)
 span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ tiles, int stages) {
   extern __shared__ __align__(16) uint8_t smem[];
   const HeadSlice hs(a, blockIdx.y);
-  const int R = hs.n, D = FIX ? 16 * NV : a.dim, DP = pad16(D), KS = DP + 8;
+  constexpr bool FIX = DK > 0;
+  const int R = hs.n, D = FIX ? DK : a.dim, DP = pad16(D), KS = DP + 8;
   const bool tied = EXT && !a.vc;                       // one tile is keys and values
   const int v0 = FIX ? 0 : blockIdx.z * kSlice, VW = FIX ? 16 * NV : min(kSlice, a.vdim - v0), VP = pad16(VW), VS = tied ? KS : VP + 8;
   __nv_bfloat16* s_q = (__nv_bfloat16*)smem;           // [64][KS]
@@ -125,7 +126,7 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
       for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
       // lanes 0-7 / 8-15 / 16-23 / 24-31 address keys 0-7 k-low, 0-7 k-high, 8-15 k-low, 8-15 k-high
       const uint32_t k_addr = smem_u32(kt + ((lane & 7) + (lane >> 4) * 8) * KS + ((lane >> 3) & 1) * 8);
-#pragma unroll(FIX ? NV : 1)
+#pragma unroll(FIX ? DK / 16 : 1)
       for (int ks = 0; ks < DP / 16; ++ks) {
         uint32_t qa[4];
         ldsm_x4(q_addr + ks * 32, qa[0], qa[1], qa[2], qa[3]);
@@ -656,8 +657,9 @@ int span_attention_tiles(cudaStream_t st, const SpanAttention& args, const RowRa
   const bool ext = is_ext(a);
 #define HB_TILES(NV)                                                                                          \
   return a.dim == 16 * NV && a.vdim == 16 * NV                                                                \
-             ? (ext ? launch(span_attention_tiles_kernel<NV, true, true>) : launch(span_attention_tiles_kernel<NV, false, true>)) \
-             : (ext ? launch(span_attention_tiles_kernel<NV, true, false>) : launch(span_attention_tiles_kernel<NV, false, false>))
+             ? (ext ? launch(span_attention_tiles_kernel<NV, true, 16 * NV>) : launch(span_attention_tiles_kernel<NV, false, 16 * NV>)) \
+             : (ext ? launch(span_attention_tiles_kernel<NV, true, 0>) : launch(span_attention_tiles_kernel<NV, false, 0>))
+  if (a.dim == 192 && a.vdim == 128 && !ext) return launch(span_attention_tiles_kernel<8, false, 192>);  // expanded latents
   if (vw <= 64) HB_TILES(4);
   if (vw <= 128) HB_TILES(8);
   if (vw <= 192) HB_TILES(12);

@@ -450,6 +450,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
     if (p.gate_bias) gate_b = __ldg(p.gate_bias + n_glob);
     if (p.up_bias) up_b = __ldg(p.up_bias + n_glob);
   }
+  auto gated = [&](float g, float u) { return BIAS ? gated_f<GENERAL>(g + gate_b, u + up_b, act) : gated_f<GENERAL>(g, u, act); };
 
   // Output tiles are staged in the (now idle) pipeline buffers as [batch row][128
   // features] and leave through bulk tensor stores: one instruction per box instead of
@@ -568,7 +569,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           }
         }
 #pragma unroll
-        for (int j = 0; j < 16; ++j) g[j] = swiglu ? gated_f<GENERAL>(g[j] + gate_b, u[j] + up_b, act) : g[j];
+        for (int j = 0; j < 16; ++j) g[j] = swiglu ? gated(g[j], u[j]) : g[j];
         if (p.post_scale) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) g[j] *= s_pscale[c0 + j];
@@ -716,7 +717,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
             for (int j = 0; j < 16; ++j) u[j] *= s_rscale[g * 16 + j];
           }
 #pragma unroll
-          for (int j = 0; j < 16; ++j) v[j] = gated_f<GENERAL>(v[j] + gate_b, u[j] + up_b, act);
+          for (int j = 0; j < 16; ++j) v[j] = gated(v[j], u[j]);
         }
         if (p.post_scale) {
 #pragma unroll
@@ -756,7 +757,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           float u[16];
           tmem_ld16(t_lane + p.m_pad + c0, u);
 #pragma unroll
-          for (int j = 0; j < 16; ++j) v[j] = gated_f<GENERAL>(v[j] + gate_b, u[j] + up_b, act);
+          for (int j = 0; j < 16; ++j) v[j] = gated(v[j], u[j]);
         }
         if (n_glob < p.N) {
 #pragma unroll
@@ -813,7 +814,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           for (int j = 0; j < 8; ++j) {
             const int m = m0 + j;
             if (m < m_lim && n_glob < p.N) {
-              const float r = swiglu ? gated_f<GENERAL>(g[j] + gate_b, u[j] + up_b, act) : g[j];
+              const float r = swiglu ? gated(g[j], u[j]) : g[j];
               if (p.out_f32) ((float*)p.Y)[(int64_t)(m_base + m) * p.ldy + n_glob] = r;
               else ((__nv_bfloat16*)p.Y)[(int64_t)(m_base + m) * p.ldy + n_glob] = __float2bfloat16_rn(r);
             }
