@@ -374,6 +374,7 @@ static SpanAttention span_args(const hb_engine* e, size_t i, const LayeredStep& 
     a.vc = nullptr;
   }
   a.dist_bias = l.dist_bias; a.dist_len = l.dist_len;
+  a.err = e->d_err;
   a.sink = l.sink;
   if (mx.ag.rows) {
     a.gate = (const uint8_t*)m->proj + mx.ag.offset * e->es;

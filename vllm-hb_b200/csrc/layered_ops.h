@@ -98,6 +98,7 @@ struct SpanAttention {
   int linear = 0, tail = 0;
   const void* kt = nullptr;
   int64_t ld_kt = 0;
+  int* err = nullptr;          // set to HB_ERR_TIMEOUT when a bounded wait inside a kernel ran out (may be null)
   // first position a query at `pos` sees besides the first keep_first
   __host__ __device__ __forceinline__ int first_seen(int pos) const {
     if (chunk > 0) return pos - pos % chunk;
