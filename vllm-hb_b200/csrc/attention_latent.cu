@@ -107,41 +107,46 @@ int latent_gather(cudaStream_t st, void* dst, const void* pool, const int32_t* l
 }
 
 // Decoded tokens.  CTA = (row, kv head and slice of up to 8 NT query heads, split).  Its warps work on the
-// 64-key tiles of the row side by side:
-//   1 warp    brings the tiles in, one bulk copy per key, `stages` tiles ahead
-//   4 warps   scores S^T[16 keys, 8 heads] = K Q^T of one block each, softmax, weights to shared memory
-//   8 warps   O^T[16 values, 8 heads] += V^T P^T for MT of the value tiles each, one tile behind
-// The weights are pairs of bf16 numbers, in two buffers.  Tiles and buffers change hands through mbarriers;
-// every wait is bounded: when one runs out the CTA goes on without waiting, and *err is set.
-// n_splits > 1: partials (O, m, l) that span_attention_merge sums up.
-constexpr int kLatThreads = 13 * 32;
-constexpr int kLatKeys = 64;
-constexpr int kLatP = kLatKeys + 8;  // padded row of weights
+// 16-key blocks of the row side by side:
+//   4 warps   bring the blocks in, every fourth each, into a ring of `ring` blocks (bulk copies, one per key,
+//             were slower: their issue took longer than the block's arithmetic)
+//   4 warps   scores S^T[16 keys, 8 heads] = K Q^T of every fourth block each, weights to shared memory
+//   8 warps   O^T[16 values, 8 heads] += V^T P^T for MT of the value tiles each, block after block
+// The weights 2^(score - ref) are pairs of bf16 numbers and come with their references: the largest score
+// of the first four blocks, until a warp meets one that lies kLatSlack above its own.  So the warps need no
+// barrier after their first blocks, and the accumulating warps bring blocks of different references
+// together where there are any.  Blocks and weights change hands through mbarriers; every wait
+// is bounded: when one runs out the CTA goes on without waiting, and *err is set.
+// n_splits > 1: partials (O, ref, l) that span_attention_merge sums up.
+constexpr int kLatLoaders = 4, kLatThreads = (kLatLoaders + 4 + 8) * 32;
+constexpr int kLatP = kBS + 8;       // padded row of weights
+constexpr int kLatWeights = 8;       // blocks of weights
+constexpr float kLatSlack = 8.f;
+constexpr int kLatRing = 16;         // most blocks in shared memory
 // most query heads of a CTA (the accumulators of wider values leave registers for fewer)
 static int latent_most_heads(const SpanAttention& a) { return a.vdim > 512 ? 16 : 32; }
-constexpr int kLatStages = 3;        // most tiles in shared memory
 
 template <int MT, int NT>
 __global__ void __launch_bounds__(kLatThreads, 1)
-latent_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, int n_splits, int stages, float* __restrict__ part) {
+latent_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, int n_splits, int ring, float* __restrict__ part) {
   extern __shared__ __align__(16) uint8_t smem[];
   constexpr int HP = NT * 8;
   const HeadSlice hs(a, blockIdx.y);
   const int R = hs.n, D = a.dim, DP = pad16(D), KS = DP + 8, VD = a.vdim, VT = pad16(VD) / 16;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gi = lane >> 2, t = lane & 3, split = blockIdx.z;
   __nv_bfloat16* s_q = (__nv_bfloat16*)smem;                  // [HP][KS]
-  __nv_bfloat16* s_k = s_q + HP * KS;                         // [stages][64][KS]
-  __nv_bfloat16* s_p = s_k + (size_t)stages * kLatKeys * KS;  // [2] hi [HP][kLatP], lo [HP][kLatP]
-  __shared__ float s_max[2][4][HP], s_alpha[2][HP], s_m[HP], s_sum[4][HP];
-  __shared__ __align__(8) uint64_t b_full[kLatStages], b_empty[kLatStages], b_weights[2], b_used[2];
+  __nv_bfloat16* s_k = s_q + HP * KS;                         // [ring][16][KS]
+  __nv_bfloat16* s_p = s_k + (size_t)ring * kBS * KS;         // [kLatWeights] hi [HP][kLatP], lo [HP][kLatP]
+  __shared__ float s_ref[kLatWeights][HP], s_first[4][HP], s_last[4][HP], s_sum[4][HP];
+  __shared__ __align__(8) uint64_t b_full[kLatRing], b_empty[kLatRing], b_weights[kLatWeights], b_used[kLatWeights];
   __shared__ int s_abort;
   if (tid == 0) {
-    for (int s = 0; s < stages; ++s) {
-      mbar_init(smem_u32(&b_full[s]), 1);
-      mbar_init(smem_u32(&b_empty[s]), 12);
+    for (int s = 0; s < ring; ++s) {
+      mbar_init(smem_u32(&b_full[s]), 32);
+      mbar_init(smem_u32(&b_empty[s]), 1 + 8);
     }
-    for (int b = 0; b < 2; ++b) {
-      mbar_init(smem_u32(&b_weights[b]), 4);
+    for (int b = 0; b < kLatWeights; ++b) {
+      mbar_init(smem_u32(&b_weights[b]), 1);
       mbar_init(smem_u32(&b_used[b]), 8);
     }
     s_abort = 0;
@@ -149,94 +154,117 @@ latent_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, in
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
   }
   if (D % 16)  // padding columns stay zero
-    for (int i = tid; i < HP + stages * kLatKeys; i += kLatThreads)
+    for (int i = tid; i < HP + ring * kBS; i += kLatThreads)
       *reinterpret_cast<uint4*>(s_q + i * KS + D) = make_uint4(0, 0, 0, 0);
   __syncthreads();
   pdl_grid_wait();
   const int64_t row = rows[blockIdx.x];
   const int pos = a.pos[row], lo = a.first_seen(pos);
   const BlockRuns runs = block_runs(pos, pos, a);
-  const int n_all = (runs.n + 3) / 4, per = (n_all + n_splits - 1) / n_splits;
-  const int first = split * per, n_tiles = max(0, min(n_all, first + per) - first);
-  float o[MT][NT][4];  // of the eight warps
+  const int per = (runs.n + n_splits - 1) / n_splits;
+  const int first = split * per, n_blocks = max(0, min(runs.n, first + per) - first);
+  float o[MT][NT][4], ref[NT][2], col[NT];  // of the eight warps: sums, references of heads 8n + 2t (+ 1) and 8n + gi
 
-  if (warp == 0) {
+  if (warp < kLatLoaders) {
     const int32_t* table = a.tables + (int64_t)a.row_seg[row] * a.max_blocks;
-    const uint32_t bytes = (uint32_t)D * 2;
-    int issued = 0;
-    for (int i = 0; i < n_tiles; ++i, ++issued) {
-      const int s = i % stages;
-      if (i >= stages && !__all_sync(0xffffffffu, mbar_wait(smem_u32(&b_empty[s]), (uint32_t)(i / stages - 1) & 1u, &s_abort))) break;
-      const uint32_t bar = smem_u32(&b_full[s]);
-      if (lane == 0) mbar_expect_tx(bar, kLatKeys * bytes);
-      __syncwarp();
-#pragma unroll
-      for (int r = lane; r < kLatKeys; r += 32) {
-        // past the last block: any block will do, its keys are masked
-        const int lb = runs.block(min((first + i) * 4 + r / kBS, runs.n - 1));
-        int64_t phys = lb < a.max_blocks ? table[lb] : 0;
-        if (phys < 0 || phys >= a.num_blocks) phys = 0;  // never outside the pool
-        bulk_load(smem_u32(s_k + ((size_t)s * kLatKeys + r) * KS), (const __nv_bfloat16*)a.kc + ((phys * a.kv_heads + hs.kvh) * kBS + r % kBS) * D,
-                  bytes, bar);
+    const BlockCopy copy(D, lane);
+    int tab = 0;
+    for (int j = warp, i = 0; j < n_blocks; j += 4, ++i) {
+      const int s = j % ring;
+      if (i % 32 == 0) {  // block table entries of this warp, 32 at a time, one per lane
+        const int lb = runs.block(min(first + j + 4 * lane, runs.n - 1));
+        tab = lb < a.max_blocks ? table[lb] : 0;
+        if (tab < 0 || tab >= a.num_blocks) tab = 0;  // never outside the pool
       }
+      if (j >= ring && !__all_sync(0xffffffffu, mbar_wait(smem_u32(&b_empty[s]), (uint32_t)(j / ring - 1) & 1u, &s_abort))) break;
+      const int64_t phys = __shfl_sync(0xffffffffu, tab, i % 32);
+      copy(smem_u32(s_k + (size_t)s * kBS * KS), KS * 2,
+           (const __nv_bfloat16*)a.kc + (phys * a.kv_heads + hs.kvh) * kBS * D, D);
+      mbar_arrive_copies(smem_u32(&b_full[s]));
     }
-    if (*(volatile int*)&s_abort)  // let every issued copy land before this CTA's shared memory can be reused
-      for (int i = max(0, issued - stages); i < issued; ++i)
-        for (uint32_t it = 0; it < kSpinLimit && !mbar_try(smem_u32(&b_full[i % stages]), (uint32_t)(i / stages) & 1u); ++it) {
-        }
-    __syncwarp();
+    cp_async_wait<0>();
   } else {
     const __nv_bfloat16* q = (const __nv_bfloat16*)a.q + row * a.ld_q + (int64_t)hs.first * D;
-    for (int i = tid - 32; i < HP * (D / 8); i += kLatThreads - 32) {
+    for (int i = tid - kLatLoaders * 32; i < HP * (D / 8); i += kLatThreads - kLatLoaders * 32) {
       const int m = i / (D / 8), c = i % (D / 8) * 8;
       uint4 v = make_uint4(0, 0, 0, 0);
       if (m < R) v = *reinterpret_cast<const uint4*>(q + m * D + c);
       *reinterpret_cast<uint4*>(s_q + m * KS + c) = v;
     }
-    asm volatile("bar.sync 1, %0;" ::"n"(kLatThreads - 32) : "memory");
+    asm volatile("bar.sync 1, %0;" ::"n"(kLatThreads - kLatLoaders * 32) : "memory");
   }
-  if (warp >= 1 && warp <= 4) {
-    const int blk = warp - 1;
+  if (warp >= kLatLoaders && warp < kLatLoaders + 4) {
+    const int blk = warp - kLatLoaders;
     const float sc = a.scale * kLog2e, cap = a.softcap * kLog2e, cap_k = cap > 0.f ? 2.f / a.softcap : 0.f;
     const uint32_t q_addr = smem_u32(s_q + (lane & 7) * KS + (lane >> 3) * 8);  // B fragments of two 16-channel steps
-    const uint32_t k_off = (uint32_t)((blk * 16 + (lane & 15)) * KS + (lane >> 4) * 8) * 2;
-    float m_run[NT][2], l_run[NT][2];
+    const uint32_t k_off = (uint32_t)((lane & 15) * KS + (lane >> 4) * 8) * 2;
+    float ref[NT][2], l[NT][2];  // of heads 8n + 2t, 8n + 2t + 1
 #pragma unroll
     for (int n = 0; n < NT; ++n) {
-      m_run[n][0] = m_run[n][1] = -INFINITY;
-      l_run[n][0] = l_run[n][1] = 0.f;
+      ref[n][0] = ref[n][1] = -INFINITY;
+      l[n][0] = l[n][1] = 0.f;
     }
-    for (int i = 0; i < n_tiles; ++i) {
-      const int st = i % stages, b = i & 1;
-      mbar_wait(smem_u32(&b_full[st]), (uint32_t)(i / stages) & 1u, &s_abort);
+    auto raise = [&](int n, int c, float to) {
+      l[n][c] *= ref[n][c] == -INFINITY ? 0.f : ex2(ref[n][c] - to);
+      ref[n][c] = to;
+    };
+    auto meet = [&] {  // one reference for the first blocks of all four warps
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+        if (gi == 0) { s_first[blk][n * 8 + 2 * t] = ref[n][0]; s_first[blk][n * 8 + 2 * t + 1] = ref[n][1]; }
+      asm volatile("bar.sync 2, 128;" ::: "memory");
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          const int h = n * 8 + 2 * t + c;
+          ref[n][c] = fmaxf(fmaxf(s_first[0][h], s_first[1][h]), fmaxf(s_first[2][h], s_first[3][h]));
+        }
+    };
+    if (blk >= n_blocks) meet();
+    for (int j = blk; j < n_blocks; j += 4) {
+      const int st = j % ring, b = j % kLatWeights;
+      mbar_wait(smem_u32(&b_full[st]), (uint32_t)(j / ring) & 1u, &s_abort);
       __syncwarp();
-      const uint32_t base = smem_u32(s_k + (size_t)st * kLatKeys * KS);
+      const uint32_t base = smem_u32(s_k + (size_t)st * kBS * KS);
       float s[NT][2][4];  // two partial sums, so that neighbouring steps do not wait for each other
 #pragma unroll
       for (int n = 0; n < NT; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) s[n][0][e] = s[n][1][e] = 0.f;
-#pragma unroll 3
-      for (int ks = 0; ks < DP / 16; ks += 2) {
-        uint32_t k0[4], k1[4];
-        ldsm_x4(base + k_off + ks * 32, k0[0], k0[1], k0[2], k0[3]);
-        const bool two = ks + 1 < DP / 16;
-        if (two) ldsm_x4(base + k_off + ks * 32 + 32, k1[0], k1[1], k1[2], k1[3]);
+      // fragments of two 16-channel steps; the next ones are fetched before the current ones are used
+      uint32_t k[2][2][4], qf[2][NT][4];
+      const int n_ks = (DP / 16 + 1) / 2;
+      auto fetch = [&](uint32_t (&kk)[2][4], uint32_t (&qq)[NT][4], int ks) {
+        // (behind the last step: the padding of the row and the first channels of the next one, unused)
+        ldsm_x4(base + k_off + ks * 64, kk[0][0], kk[0][1], kk[0][2], kk[0][3]);
+        if (2 * ks + 1 < DP / 16) ldsm_x4(base + k_off + ks * 64 + 32, kk[1][0], kk[1][1], kk[1][2], kk[1][3]);
 #pragma unroll
-        for (int n = 0; n < NT; ++n) {
-          uint32_t b0, b1, b2, b3;
-          // (a lone last step also reads the 16 elements behind it: unused)
-          ldsm_x4(q_addr + (n * 8 * KS + ks * 16) * 2, b0, b1, b2, b3);
-          mma_bf16_16816(s[n][0], k0, b0, b1);
-          if (two) mma_bf16_16816(s[n][1], k1, b2, b3);
+        for (int n = 0; n < NT; ++n) ldsm_x4(q_addr + (n * 8 * KS + ks * 32) * 2, qq[n][0], qq[n][1], qq[n][2], qq[n][3]);
+      };
+      auto use = [&](const uint32_t (&kk)[2][4], const uint32_t (&qq)[NT][4], int ks) {
+#pragma unroll
+        for (int n = 0; n < NT; ++n) mma_bf16_16816(s[n][0], kk[0], qq[n][0], qq[n][1]);
+        if (2 * ks + 1 < DP / 16)
+#pragma unroll
+          for (int n = 0; n < NT; ++n) mma_bf16_16816(s[n][1], kk[1], qq[n][2], qq[n][3]);
+      };
+      fetch(k[0], qf[0], 0);
+      for (int ks = 0; ks < n_ks; ks += 2) {
+        if (ks + 1 < n_ks) fetch(k[1], qf[1], ks + 1);
+        use(k[0], qf[0], ks);
+        if (ks + 1 < n_ks) {
+          if (ks + 2 < n_ks) fetch(k[0], qf[0], ks + 2);
+          use(k[1], qf[1], ks + 1);
         }
       }
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(&b_empty[st]));
-      const int vb = (first + i) * 4 + blk, key0 = vb < runs.n ? runs.block(vb) * kBS : -1;
-      const bool full = key0 >= 0 && all_visible(key0, pos, lo, a.keep_first);
-      const bool see0 = full || (key0 >= 0 && visible(key0 + gi, pos, lo, a.keep_first));
-      const bool see1 = full || (key0 >= 0 && visible(key0 + gi + 8, pos, lo, a.keep_first));
+      const int key0 = runs.block(first + j) * kBS;
+      const bool full = all_visible(key0, pos, lo, a.keep_first);
+      const bool see0 = full || visible(key0 + gi, pos, lo, a.keep_first);
+      const bool see1 = full || visible(key0 + gi + 8, pos, lo, a.keep_first);
+      bool above = false;
 #pragma unroll
       for (int n = 0; n < NT; ++n) {
         float (&p)[4] = s[n][0];
@@ -245,42 +273,38 @@ latent_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, in
           float x = (s[n][0][e] + s[n][1][e]) * sc;
           if (cap > 0.f) x = capped(x, cap, cap_k);
           p[e] = (e < 2 ? see0 : see1) ? x : -INFINITY;
+          above = above || p[e] > ref[n][e & 1] + kLatSlack;
         }
-        float x0 = fmaxf(p[0], p[2]), x1 = fmaxf(p[1], p[3]);
-#pragma unroll
-        for (int w = 4; w < 32; w <<= 1) {
-          x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, w));
-          x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, w));
-        }
-        if (gi == 0) { s_max[b][blk][n * 8 + 2 * t] = x0; s_max[b][blk][n * 8 + 2 * t + 1] = x1; }
       }
-      asm volatile("bar.sync 2, 128;" ::: "memory");  // the four blocks' maxima
-      if (i >= 2) mbar_wait(smem_u32(&b_used[b]), (uint32_t)(i / 2 - 1) & 1u, &s_abort);
+      if (__any_sync(0xffffffffu, above)) {
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+          for (int c = 0; c < 2; ++c) {
+            float x = fmaxf(s[n][0][c], s[n][0][2 + c]);
+#pragma unroll
+            for (int w = 4; w < 32; w <<= 1) x = fmaxf(x, __shfl_xor_sync(0xffffffffu, x, w));
+            const float r = fmaxf(ref[n][c], x);
+            if (r > ref[n][c]) raise(n, c, r);
+          }
+      }
+      if (j == blk) meet();
+      if (j >= kLatWeights) mbar_wait(smem_u32(&b_used[b]), (uint32_t)(j / kLatWeights - 1) & 1u, &s_abort);
       __nv_bfloat16* weights = s_p + b * 2 * HP * kLatP;
 #pragma unroll
       for (int n = 0; n < NT; ++n) {
         const int h = n * 8 + 2 * t;
         float (&p)[4] = s[n][0];
-        float top[2];
-#pragma unroll
-        for (int c = 0; c < 2; ++c) {
-          const float x = fmaxf(fmaxf(s_max[b][0][h + c], s_max[b][1][h + c]), fmaxf(s_max[b][2][h + c], s_max[b][3][h + c]));
-          const float m_new = fmaxf(m_run[n][c], x);
-          top[c] = m_new == -INFINITY ? 0.f : m_new;  // nothing visible yet
-          const float al = ex2(m_run[n][c] - top[c]);
-          m_run[n][c] = m_new;
-          l_run[n][c] *= al;
-          if (blk == 0 && gi == 0) s_alpha[b][h + c] = al;
-        }
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          p[e] = ex2(p[e] - top[e & 1]);
-          l_run[n][e & 1] += p[e];
+          p[e] = p[e] == -INFINITY ? 0.f : ex2(p[e] - ref[n][e & 1]);
+          l[n][e & 1] += p[e];
           const __nv_bfloat16 hi = __float2bfloat16_rn(p[e]);
-          __nv_bfloat16* dst = weights + (h + (e & 1)) * kLatP + blk * 16 + gi + (e < 2 ? 0 : 8);
+          __nv_bfloat16* dst = weights + (h + (e & 1)) * kLatP + gi + (e < 2 ? 0 : 8);
           dst[0] = hi;
           dst[HP * kLatP] = __float2bfloat16_rn(p[e] - __bfloat162float(hi));
         }
+        if (gi == 0) { s_ref[b][h] = ref[n][0]; s_ref[b][h + 1] = ref[n][1]; }
       }
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(&b_weights[b]));
@@ -289,67 +313,97 @@ latent_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, in
     for (int n = 0; n < NT; ++n)
 #pragma unroll
       for (int c = 0; c < 2; ++c) {
-        float ll = l_run[n][c];
+        float ll = l[n][c];
 #pragma unroll
         for (int w = 4; w < 32; w <<= 1) ll += __shfl_xor_sync(0xffffffffu, ll, w);
         if (gi == 0) {
           s_sum[blk][n * 8 + 2 * t + c] = ll;
-          if (blk == 0) s_m[n * 8 + 2 * t + c] = m_run[n][c];
+          s_last[blk][n * 8 + 2 * t + c] = ref[n][c];
         }
       }
-  } else if (warp >= 5) {
+  } else if (warp >= kLatLoaders + 4) {
     const uint32_t v_off = (uint32_t)(((lane & 7) + (lane >> 4) * 8) * KS + ((lane >> 3) & 1) * 8) * 2;
 #pragma unroll
     for (int k = 0; k < MT; ++k)
 #pragma unroll
       for (int n = 0; n < NT; ++n) o[k][n][0] = o[k][n][1] = o[k][n][2] = o[k][n][3] = 0.f;
-    for (int i = 0; i < n_tiles; ++i) {
-      const int st = i % stages, b = i & 1;
-      mbar_wait(smem_u32(&b_full[st]), (uint32_t)(i / stages) & 1u, &s_abort);
-      mbar_wait(smem_u32(&b_weights[b]), (uint32_t)(i / 2) & 1u, &s_abort);
+#pragma unroll
+    for (int n = 0; n < NT; ++n) col[n] = ref[n][0] = ref[n][1] = -INFINITY;
+    for (int j = 0; j < n_blocks; ++j) {
+      const int st = j % ring, b = j % kLatWeights;
+      mbar_wait(smem_u32(&b_full[st]), (uint32_t)(j / ring) & 1u, &s_abort);
+      mbar_wait(smem_u32(&b_weights[b]), (uint32_t)(j / kLatWeights) & 1u, &s_abort);
       __syncwarp();
-      const uint32_t base = smem_u32(s_k + (size_t)st * kLatKeys * KS);
+      const uint32_t base = smem_u32(s_k + (size_t)st * kBS * KS);
       const __nv_bfloat16* weights = s_p + b * 2 * HP * kLatP;
+      uint32_t hi[NT][2], low[NT][2];
+      bool moved = false;
 #pragma unroll
       for (int n = 0; n < NT; ++n) {
-        const float a0 = s_alpha[b][n * 8 + 2 * t], a1 = s_alpha[b][n * 8 + 2 * t + 1];
-        if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f))
-#pragma unroll
-          for (int k = 0; k < MT; ++k) { o[k][n][0] *= a0; o[k][n][1] *= a1; o[k][n][2] *= a0; o[k][n][3] *= a1; }
+        const uint32_t* p = reinterpret_cast<const uint32_t*>(weights + (n * 8 + gi) * kLatP + 2 * t);
+        hi[n][0] = p[0]; hi[n][1] = p[4];
+        low[n][0] = p[HP * kLatP / 2]; low[n][1] = p[HP * kLatP / 2 + 4];
+        const float g = s_ref[b][n * 8 + gi];
+        moved = moved || g != col[n];
       }
-#pragma unroll
-      for (int kb = 0; kb < 4; ++kb) {
-        uint32_t hi[NT][2], low[NT][2];
+      if (__any_sync(0xffffffffu, moved)) {
 #pragma unroll
         for (int n = 0; n < NT; ++n) {
-          const uint32_t* p = reinterpret_cast<const uint32_t*>(weights + (n * 8 + gi) * kLatP + kb * 16 + 2 * t);
-          hi[n][0] = p[0]; hi[n][1] = p[4];
-          low[n][0] = p[HP * kLatP / 2]; low[n][1] = p[HP * kLatP / 2 + 4];
-        }
 #pragma unroll
-        for (int k = 0; k < MT; ++k) {
-          const int vt = warp - 5 + 8 * k;
-          if (vt < VT) {
-            uint32_t va[4];
-            ldsm_x4_trans(base + v_off + (kb * 16 * KS + vt * 16) * 2, va[0], va[1], va[2], va[3]);
+          for (int c = 0; c < 2; ++c) {  // the sums so far
+            const float to = fmaxf(ref[n][c], s_ref[b][n * 8 + 2 * t + c]);
+            const float f = ref[n][c] == to ? 1.f : ex2(ref[n][c] - to);
+            ref[n][c] = to;
 #pragma unroll
-            for (int n = 0; n < NT; ++n) mma_bf16_16816(o[k][n], va, hi[n][0], hi[n][1]);
+            for (int k = 0; k < MT; ++k) { o[k][n][c] *= f; o[k][n][2 + c] *= f; }
+          }
+          const float g = s_ref[b][n * 8 + gi], to = fmaxf(col[n], g);
+          const float f = g == to ? 1.f : ex2(g - to);  // the block's weights
+          col[n] = to;
 #pragma unroll
-            for (int n = 0; n < NT; ++n) mma_bf16_16816(o[k][n], va, low[n][0], low[n][1]);
+          for (int x = 0; x < 2; ++x) {
+            const float2 h2 = unpack_bf16(hi[n][x]), l2 = unpack_bf16(low[n][x]);
+            split_bf16((h2.x + l2.x) * f, (h2.y + l2.y) * f, hi[n][x], low[n][x]);
           }
         }
       }
-      __syncwarp();
-      if (lane == 0) {
-        mbar_arrive(smem_u32(&b_empty[st]));
-        mbar_arrive(smem_u32(&b_used[b]));
+      {
+        // two value tiles at a time, the next two fetched before the current ones are used; the low halves of
+        // the weights follow the high ones of both
+        uint32_t va[2][2][4];
+        auto fetch = [&](uint32_t (&v)[2][4], int k) {
+#pragma unroll
+          for (int x = 0; x < 2; ++x) {
+            const int vt = min(warp - kLatLoaders - 4 + 8 * (k + x), VT - 1);  // past the last: unused
+            ldsm_x4_trans(base + v_off + vt * 32, v[x][0], v[x][1], v[x][2], v[x][3]);
+          }
+        };
+        fetch(va[0], 0);
+#pragma unroll
+        for (int k = 0; k < MT; k += 2) {
+          if (k + 2 < MT) fetch(va[(k / 2 + 1) & 1], k + 2);
+          const uint32_t (&v)[2][4] = va[(k / 2) & 1];
+#pragma unroll
+          for (int x = 0; x < 2; ++x)
+#pragma unroll
+            for (int n = 0; n < NT; ++n) mma_bf16_16816(o[k + x][n], v[x], hi[n][0], hi[n][1]);
+#pragma unroll
+          for (int x = 0; x < 2; ++x)
+#pragma unroll
+            for (int n = 0; n < NT; ++n) mma_bf16_16816(o[k + x][n], v[x], low[n][0], low[n][1]);
+        }
+        __syncwarp();
+        if (lane == 0) {
+          mbar_arrive(smem_u32(&b_empty[st]));
+          mbar_arrive(smem_u32(&b_used[b]));
+        }
       }
     }
   }
   pdl_trigger();
   __syncthreads();
   if (tid == 0 && s_abort && a.err) atomicExch(a.err, HB_ERR_TIMEOUT);
-  if (warp < 5) return;
+  if (warp < kLatLoaders + 4) return;
 #pragma unroll
   for (int n = 0; n < NT; ++n)
 #pragma unroll
@@ -357,7 +411,11 @@ latent_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, in
       const int h = n * 8 + 2 * t + c;
       if (h < R) {
         const int64_t head = hs.first + h;
-        const float l = (s_sum[0][h] + s_sum[1][h]) + (s_sum[2][h] + s_sum[3][h]), m = s_m[h];
+        const float m = ref[n][c];
+        float l = 0.f;
+#pragma unroll
+        for (int w = 0; w < 4; ++w)
+          if (s_last[w][h] != -INFINITY) l = fmaf(s_sum[w][h], ex2(s_last[w][h] - m), l);
         float* p = part + (((int64_t)blockIdx.x * a.heads + head) * n_splits + split) * (VD + 2);
         float inv = 1.f / l;
         if (a.sink) {
@@ -368,7 +426,7 @@ latent_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, in
         for (int k = 0; k < MT; ++k)
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
-            const int col = (warp - 5 + 8 * k) * 16 + gi + e * 8;
+            const int col = (warp - kLatLoaders - 4 + 8 * k) * 16 + gi + e * 8;
             if (col >= VD) continue;
             float x = o[k][n][2 * e + c];
             if (n_splits > 1) {
@@ -379,7 +437,7 @@ latent_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, in
               ((__nv_bfloat16*)a.out)[row * a.ld_out + head * VD + col] = __float2bfloat16_rn(x);
             }
           }
-        if (n_splits > 1 && warp == 5 && gi == 0) {
+        if (n_splits > 1 && warp == kLatLoaders + 4 && gi == 0) {
           p[VD] = m;
           p[VD + 1] = l;
         }
@@ -387,9 +445,14 @@ latent_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, in
     }
 }
 
-static size_t latent_tokens_smem(const SpanAttention& a, int heads, int stages) {
-  const size_t KS = pad16(a.dim) + 8;
-  return (heads * KS + (size_t)stages * kLatKeys * KS + (size_t)4 * heads * kLatP) * 2;
+// Blocks the ring may have beside everything else.
+static int latent_ring(const SpanAttention& a, int heads) {
+  const size_t row = (size_t)(pad16(a.dim) + 8) * 2, fixed = heads * row + (size_t)kLatWeights * 2 * heads * kLatP * 2;
+  return fixed < kSmemCap ? (int)std::min<size_t>(kLatRing, (kSmemCap - fixed) / (kBS * row)) : 0;
+}
+static size_t latent_tokens_smem(const SpanAttention& a, int heads) {
+  const size_t row = (size_t)(pad16(a.dim) + 8) * 2;
+  return heads * row + (size_t)kLatWeights * 2 * heads * kLatP * 2 + latent_ring(a, heads) * kBS * row;
 }
 static int latent_heads(const SpanAttention& a) {  // of a slice, padded
   SpanAttention s = a;
@@ -400,7 +463,7 @@ static int latent_heads(const SpanAttention& a) {  // of a slice, padded
 // Narrow latents are left to the kernel of attention_span_mma.cu, whose warps need no barriers.
 bool latent_tokens_supported(const SpanAttention& a, hb_dtype dtype) {
   return span_attention_mma_ok(a, dtype) && !a.vc && !a.key_scale && !a.dist_bias && a.vdim > 128 && a.vdim <= 1024 &&
-         latent_tokens_smem(a, latent_heads(a), 2) <= kSmemCap;
+         latent_ring(a, latent_heads(a)) >= 6;
 }
 
 int latent_tokens_units(const SpanAttention& args) {
@@ -413,12 +476,12 @@ int latent_tokens(cudaStream_t st, const SpanAttention& args, const int32_t* row
   if (n_rows == 0) return HB_OK;
   SpanAttention a = args;
   a.cut(latent_most_heads(a));
-  const int heads = latent_heads(a), stages = latent_tokens_smem(a, heads, kLatStages) <= kSmemCap ? kLatStages : 2;
-  const size_t smem = latent_tokens_smem(a, heads, stages);
+  const int heads = latent_heads(a);
+  const size_t smem = latent_tokens_smem(a, heads);
   auto launch = [&](auto* k) -> int {
     HB_CUDA_CHECK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemCap));
     HB_CUDA_CHECK(launch_pdl(k, dim3((unsigned)n_rows, (unsigned)(a.kv_heads * a.slices()), (unsigned)n_splits), dim3(kLatThreads),
-                             smem, st, a, rows, n_splits, stages, part));
+                             smem, st, a, rows, n_splits, latent_ring(a, heads), part));
     return HB_OK;
   };
   int rc;

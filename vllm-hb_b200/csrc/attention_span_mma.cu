@@ -28,6 +28,7 @@ constexpr int kRows = 64;      // query rows of a tile
 constexpr int kKeys = 64;      // keys of a tile step
 constexpr int kSlice = 256;    // widest value slice
 constexpr int kRing = 3;       // 16-key stages of a warp (token kernel)
+constexpr int kMaxSplits = 64; // of a row
 constexpr int kMaxCluster = 8; // splits of a row that sum up in a cluster
 }  // namespace
 
@@ -563,24 +564,38 @@ __global__ void __launch_bounds__(kThreads)
 span_attention_merge_kernel(const SpanAttention a, const int32_t* __restrict__ rows, int n_splits, const float* __restrict__ part) {
   pdl_trigger();
   pdl_grid_wait();
+  __shared__ float s_f[kMaxSplits], s_scale;
   const int64_t row = rows[blockIdx.x];
-  const int head = blockIdx.y;
-  const float* p = part + ((int64_t)blockIdx.x * a.heads + head) * n_splits * (a.vdim + 2);
-  float mx = a.sink ? a.sink[head] * kLog2e : -INFINITY, l = 0.f;
-  const float k = mx;
-  for (int s = 0; s < n_splits; ++s) mx = fmaxf(mx, p[s * (a.vdim + 2) + a.vdim]);
-  if (a.sink) l = ex2(k - mx);
-  for (int s = 0; s < n_splits; ++s) {
-    const float m = p[s * (a.vdim + 2) + a.vdim];
-    if (m != -INFINITY) l = fmaf(ex2(m - mx), p[s * (a.vdim + 2) + a.vdim + 1], l);
-  }
-  for (int c = threadIdx.x; c < a.vdim; c += kThreads) {
-    float acc = 0.f;
-    for (int s = 0; s < n_splits; ++s) {
-      const float m = p[s * (a.vdim + 2) + a.vdim];
-      if (m != -INFINITY) acc = fmaf(ex2(m - mx), p[s * (a.vdim + 2) + c], acc);
+  const int head = blockIdx.y, tid = threadIdx.x, ld = a.vdim + 2;
+  const float* p = part + ((int64_t)blockIdx.x * a.heads + head) * n_splits * ld;
+  if (tid < 32) {  // the splits' factors, by one warp
+    const float k = a.sink ? a.sink[head] * kLog2e : -INFINITY;
+    float mx = k, l = 0.f, m[kMaxSplits / 32];
+#pragma unroll
+    for (int i = 0; i < kMaxSplits / 32; ++i) {
+      m[i] = tid + 32 * i < n_splits ? p[(tid + 32 * i) * ld + a.vdim] : -INFINITY;
+      mx = fmaxf(mx, m[i]);
     }
-    acc /= l;
+    mx = warp_max(mx);
+#pragma unroll
+    for (int i = 0; i < kMaxSplits / 32; ++i) {
+      if (tid + 32 * i >= n_splits) continue;
+      const float f = m[i] == -INFINITY ? 0.f : ex2(m[i] - mx);
+      s_f[tid + 32 * i] = f;
+      if (f > 0.f) l = fmaf(f, p[(tid + 32 * i) * ld + a.vdim + 1], l);
+    }
+    l = warp_sum(l);
+    if (tid == 0) s_scale = 1.f / (a.sink ? l + ex2(k - mx) : l);
+  }
+  __syncthreads();
+  for (int c = tid; c < a.vdim; c += kThreads) {
+    float acc = 0.f;
+#pragma unroll 8
+    for (int s = 0; s < n_splits; ++s) {
+      const float f = s_f[s];
+      acc = f > 0.f ? fmaf(f, p[s * ld + c], acc) : acc;
+    }
+    acc *= s_scale;
     if (a.gate) acc *= sigmoid_of(((const uint16_t*)a.gate)[row * a.ld_gate + (int64_t)head * a.vdim + c]);
     ((__nv_bfloat16*)a.out)[row * a.ld_out + (int64_t)head * a.vdim + c] = __float2bfloat16_rn(acc);
   }
