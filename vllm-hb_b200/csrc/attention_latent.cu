@@ -123,6 +123,18 @@ constexpr int kLatP = kBS + 8;       // padded row of weights
 constexpr int kLatWeights = 8;       // blocks of weights
 constexpr float kLatSlack = 8.f;
 constexpr int kLatRing = 16;         // most blocks in shared memory
+// Where block j lies in the ring, and the parity of the ring's round, without divisions.
+struct RingPlace {
+  int at;
+  uint32_t parity = 0;
+  __device__ __forceinline__ void step(int by, int ring) {
+    at += by;
+    if (at >= ring) {
+      at -= ring;
+      parity ^= 1u;
+    }
+  }
+};
 // most query heads of a CTA (the accumulators of wider values leave registers for fewer)
 static int latent_most_heads(const SpanAttention& a) { return a.vdim > 512 ? 16 : 32; }
 
@@ -169,14 +181,15 @@ latent_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, in
     const int32_t* table = a.tables + (int64_t)a.row_seg[row] * a.max_blocks;
     const BlockCopy copy(D, lane);
     int tab = 0;
-    for (int j = warp, i = 0; j < n_blocks; j += 4, ++i) {
-      const int s = j % ring;
+    RingPlace place{warp};
+    for (int j = warp, i = 0; j < n_blocks; j += 4, ++i, place.step(4, ring)) {
+      const int s = place.at;
       if (i % 32 == 0) {  // block table entries of this warp, 32 at a time, one per lane
         const int lb = runs.block(min(first + j + 4 * lane, runs.n - 1));
         tab = lb < a.max_blocks ? table[lb] : 0;
         if (tab < 0 || tab >= a.num_blocks) tab = 0;  // never outside the pool
       }
-      if (j >= ring && !__all_sync(0xffffffffu, mbar_wait(smem_u32(&b_empty[s]), (uint32_t)(j / ring - 1) & 1u, &s_abort))) break;
+      if (j >= ring && !__all_sync(0xffffffffu, mbar_wait(smem_u32(&b_empty[s]), place.parity ^ 1u, &s_abort))) break;
       const int64_t phys = __shfl_sync(0xffffffffu, tab, i % 32);
       copy(smem_u32(s_k + (size_t)s * kBS * KS), KS * 2,
            (const __nv_bfloat16*)a.kc + (phys * a.kv_heads + hs.kvh) * kBS * D, D);
@@ -222,9 +235,10 @@ latent_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, in
         }
     };
     if (blk >= n_blocks) meet();
-    for (int j = blk; j < n_blocks; j += 4) {
-      const int st = j % ring, b = j % kLatWeights;
-      mbar_wait(smem_u32(&b_full[st]), (uint32_t)(j / ring) & 1u, &s_abort);
+    RingPlace place{blk};
+    for (int j = blk; j < n_blocks; j += 4, place.step(4, ring)) {
+      const int st = place.at, b = j % kLatWeights;
+      mbar_wait(smem_u32(&b_full[st]), place.parity, &s_abort);
       __syncwarp();
       const uint32_t base = smem_u32(s_k + (size_t)st * kBS * KS);
       float s[NT][2][4];  // two partial sums, so that neighbouring steps do not wait for each other
@@ -329,9 +343,10 @@ latent_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, in
       for (int n = 0; n < NT; ++n) o[k][n][0] = o[k][n][1] = o[k][n][2] = o[k][n][3] = 0.f;
 #pragma unroll
     for (int n = 0; n < NT; ++n) col[n] = ref[n][0] = ref[n][1] = -INFINITY;
-    for (int j = 0; j < n_blocks; ++j) {
-      const int st = j % ring, b = j % kLatWeights;
-      mbar_wait(smem_u32(&b_full[st]), (uint32_t)(j / ring) & 1u, &s_abort);
+    RingPlace place{0};
+    for (int j = 0; j < n_blocks; ++j, place.step(1, ring)) {
+      const int st = place.at, b = j % kLatWeights;
+      mbar_wait(smem_u32(&b_full[st]), place.parity, &s_abort);
       mbar_wait(smem_u32(&b_weights[b]), (uint32_t)(j / kLatWeights) & 1u, &s_abort);
       __syncwarp();
       const uint32_t base = smem_u32(s_k + (size_t)st * kBS * KS);
