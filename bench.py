@@ -614,8 +614,8 @@ def main() -> None:
     ap.add_argument("--tp1-layers", type=int, default=8, help="layers of the single-GPU base point of the N > 1 shape")
     ap.add_argument("--workload", default="auto", choices=["auto", "mixtral", "latarax", "biberax", "badolix"],
                     help="auto: Llama-3.1-8B shape on one GPU, 70B shape on several; mixtral: Mixtral-8x7B shape; "
-                         "latarax, biberax: that design beside the Llama family at equal size, one GPU")
-    ap.add_argument("--size", default="", help="latarax, biberax: only the sizes whose name contains this text")
+                         "latarax, biberax, badolix: that design beside the Llama family at equal size, one GPU")
+    ap.add_argument("--size", default="", help="latarax, biberax, badolix: only the sizes whose name contains this text")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
