@@ -24,6 +24,7 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prepare_kernel(const Late
   const bool keep = slot >= 0 && slot < a.num_blocks * HB_BLOCK_SIZE;
   T* pr = (T*)a.p + row * a.ld;
   const T* latent = pr + a.off_c;
+  T* qr = a.qs ? (T*)a.qs + row * a.ld_qs : pr + a.off_q;
   float f[V], g[V];
   if (tid * V < C) Run<T, V>::load(f, latent + tid * V);  // on its way while the angles are formed
   angles_of(s_cs, a.rotation, P, a.pos[row], a.rotation_gain);
@@ -45,10 +46,47 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prepare_kernel(const Late
     }
   }
   // rotated parts: one per head of the queries, then the key's
+  if (!a.halves) {  // neighbours
+    const int per = (V == 1 ? P : 0) + (V == 1 ? R - 2 * P : R / V);
+    for (int i = tid; i < (a.heads + (keep ? 1 : 0)) * per; i += kPrepThreads) {
+      const int h = i / per, u = i % per;
+      T* src = h < a.heads ? qr + h * QD + a.dim : pr + a.off_c + C;
+      T* dst = (h < a.heads ? (T*)a.q + row * a.ld_q + (int64_t)h * KD : entry) + C;
+      if constexpr (V == 1) {  // a pair, or a channel behind them
+        if (u < P) {
+          float x, y;
+          rope_rotate(to_f32<T>(src[2 * u]), to_f32<T>(src[2 * u + 1]), s_cs[u], s_cs[P + u], &x, &y);
+          dst[2 * u] = from_f32<T>(x);
+          dst[2 * u + 1] = from_f32<T>(y);
+          if (h < a.heads) {
+            src[2 * u] = from_f32<T>(x);
+            src[2 * u + 1] = from_f32<T>(y);
+          }
+        } else {
+          dst[P + u] = src[P + u];
+        }
+      } else {
+        const int d = u * V;
+        Run<T, V>::load(f, src + d);
+        if (d < 2 * P) {
+#pragma unroll
+          for (int j = 0; j < V; j += 2) {
+            float x, y;
+            rope_rotate(f[j], f[j + 1], s_cs[(d + j) / 2], s_cs[P + (d + j) / 2], &x, &y);
+            f[j] = x;
+            f[j + 1] = y;
+          }
+          if (h < a.heads) Run<T, V>::store(src + d, f);
+        }
+        Run<T, V>::store(dst + d, f);
+      }
+    }
+    return;
+  }
   const int turned = P / V, per = turned + (R - 2 * P) / V;
   for (int i = tid; i < (a.heads + (keep ? 1 : 0)) * per; i += kPrepThreads) {
     const int h = i / per, u = i % per, d = u < turned ? u * V : P + u * V;
-    T* src = pr + (h < a.heads ? a.off_q + h * QD + a.dim : a.off_c + C) + d;
+    T* src = (h < a.heads ? qr + h * QD + a.dim : pr + a.off_c + C) + d;
     T* dst = (h < a.heads ? (T*)a.q + row * a.ld_q + (int64_t)h * KD : entry) + C + d;
     Run<T, V>::load(f, src);
     if (u < turned) {
@@ -76,7 +114,8 @@ int latent_prepare(cudaStream_t st, const LatentPrep& a, int64_t rows, hb_dtype 
     return fail(HB_ERR_INVALID_ARG, "latent_prepare: %d pairs of %d channels", a.pairs, a.rot_dim);
   const int n = (int)(16 / dtype_size(dtype));
   auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-  const bool vec = a.dim % n == 0 && a.rot_dim % n == 0 && a.rank % n == 0 && a.pairs % n == 0 && a.off_q % n == 0 &&
+  const bool vec = a.dim % n == 0 && a.rot_dim % n == 0 && a.rank % n == 0 && (a.halves ? a.pairs % n == 0 : 2 * a.pairs % n == 0) &&
+                   (a.qs ? a.ld_qs % n == 0 && al(a.qs) : a.off_q % n == 0) &&
                    a.off_c % n == 0 && a.ld % n == 0 && a.ld_q % n == 0 && al(a.p) && al(a.q) && al(a.kc);
   auto launch = [&](auto* k) -> int {
     HB_CUDA_CHECK(launch_pdl(k, dim3((unsigned)rows), dim3(kPrepThreads), (size_t)a.pairs * 2 * sizeof(float), st, a));
@@ -448,7 +487,7 @@ latent_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ rows, in
               p[col] = x;
             } else {
               x *= inv;
-              if (a.gate) x *= sigmoid_of(((const uint16_t*)a.gate)[row * a.ld_gate + head * VD + col]);
+              if (a.gate) x *= sigmoid_of(((const uint16_t*)a.gate)[a.gate_at(row, head, col)]);
               ((__nv_bfloat16*)a.out)[row * a.ld_out + head * VD + col] = __float2bfloat16_rn(x);
             }
           }

@@ -145,11 +145,11 @@ span_attention_rows_kernel(const SpanAttention a, const int32_t* __restrict__ ro
     }
   __syncthreads();
   T* out = (T*)a.out + row * a.ld_out + (int64_t)hs.first * VD;
-  const T* gate = a.gate ? (const T*)a.gate + row * a.ld_gate + (int64_t)hs.first * VD : nullptr;
+  const T* gate = a.gate ? (const T*)a.gate + a.gate_at(row, hs.first, 0) : nullptr;
   for (int i = tid; i < R * VD; i += kSpanThreads) {
     float o = s_acc[i] / s_l[i / VD];
     if (a.sink) o *= s_a[i / VD];
-    if (gate) o /= 1.f + expf(-to_f32<T>(gate[i]));
+    if (gate) o /= 1.f + expf(-to_f32<T>(gate[a.gate_per_head ? i / VD : i]));
     out[i] = from_f32<T>(o);
   }
 }

@@ -251,9 +251,13 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
   }
   const __nv_bfloat16 *g0 = nullptr, *g1 = nullptr;
   if (a.gate) {
-    const __nv_bfloat16* gate = (const __nv_bfloat16*)a.gate + (int64_t)hs.first * a.vdim + v0;
-    g0 = gate + (int64_t)(tile.row0 + r0 / R) * a.ld_gate + (r0 % R) * a.vdim;
-    g1 = gate + (int64_t)(tile.row0 + r1 / R) * a.ld_gate + (r1 % R) * a.vdim;
+    const __nv_bfloat16* gate = (const __nv_bfloat16*)a.gate;
+    g0 = gate + a.gate_at(tile.row0 + r0 / R, hs.first + r0 % R, v0);
+    g1 = gate + a.gate_at(tile.row0 + r1 / R, hs.first + r1 % R, v0);
+    if (a.gate_per_head) {
+      if (r0 < n_rows) i0 *= sigmoid_of(*reinterpret_cast<const uint16_t*>(g0));
+      if (r1 < n_rows) i1 *= sigmoid_of(*reinterpret_cast<const uint16_t*>(g1));
+    }
   }
   __nv_bfloat16* out = (__nv_bfloat16*)a.out + (int64_t)hs.first * a.vdim + v0;
   __nv_bfloat16* w0 = out + (int64_t)(tile.row0 + r0 / R) * a.ld_out + (r0 % R) * a.vdim;
@@ -263,7 +267,7 @@ span_attention_tiles_kernel(const SpanAttention a, const RowRange* __restrict__ 
     const int c = i * 8 + 2 * t;
     if (c < VW) {
       float x[4] = {o[i][0] * i0, o[i][1] * i0, o[i][2] * i1, o[i][3] * i1};
-      if (a.gate) {
+      if (a.gate && !a.gate_per_head) {
         const uint32_t z0 = r0 < n_rows ? *reinterpret_cast<const uint32_t*>(g0 + c) : 0u;
         const uint32_t z1 = r1 < n_rows ? *reinterpret_cast<const uint32_t*>(g1 + c) : 0u;
         x[0] *= sigmoid_of(z0 & 0xffffu); x[1] *= sigmoid_of(z0 >> 16);
@@ -514,7 +518,7 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
       for (int w = 0; w < kWarps; ++w) acc = fmaf(f[w], s_o[((size_t)w * R + h) * OS + c], acc);
       if (n_splits == 1) {
         acc *= inv;
-        if (a.gate) acc *= sigmoid_of(((const uint16_t*)a.gate)[row * a.ld_gate + head * a.vdim + v0 + c]);
+        if (a.gate) acc *= sigmoid_of(((const uint16_t*)a.gate)[a.gate_at(row, head, v0 + c)]);
         ((__nv_bfloat16*)a.out)[row * a.ld_out + head * a.vdim + v0 + c] = __float2bfloat16_rn(acc);
       } else if (clustered) {
         s_o[(size_t)h * OS + c] = acc;  // the place of warp 0, read by this lane above
@@ -553,7 +557,7 @@ span_attention_tokens_kernel(const SpanAttention a, const int32_t* __restrict__ 
       }
     }
     acc /= ls;
-    if (a.gate) acc *= sigmoid_of(((const uint16_t*)a.gate)[row * a.ld_gate + head * a.vdim + v0 + c]);
+    if (a.gate) acc *= sigmoid_of(((const uint16_t*)a.gate)[a.gate_at(row, head, v0 + c)]);
     ((__nv_bfloat16*)a.out)[row * a.ld_out + head * a.vdim + v0 + c] = __float2bfloat16_rn(acc);
   }
   cluster_sync_all();  // nobody leaves while a partner still reads its shared memory
@@ -596,7 +600,7 @@ span_attention_merge_kernel(const SpanAttention a, const int32_t* __restrict__ r
       acc = f > 0.f ? fmaf(f, p[s * ld + c], acc) : acc;
     }
     acc *= s_scale;
-    if (a.gate) acc *= sigmoid_of(((const uint16_t*)a.gate)[row * a.ld_gate + (int64_t)head * a.vdim + c]);
+    if (a.gate) acc *= sigmoid_of(((const uint16_t*)a.gate)[a.gate_at(row, head, c)]);
     ((__nv_bfloat16*)a.out)[row * a.ld_out + (int64_t)head * a.vdim + c] = __float2bfloat16_rn(acc);
   }
 }
@@ -621,7 +625,7 @@ bool span_attention_mma_ok(const SpanAttention& a, hb_dtype dtype) {
   auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   static const bool simt = [] { const char* e = getenv("HB_ATTN"); return e && e[0] == 's'; }();
   return !simt && dtype == HB_BF16 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ld_q % 8 == 0 && a.ld_out % 2 == 0 && al(a.q) &&
-         al(a.out) && (!a.gate || (a.ld_gate % 2 == 0 && (reinterpret_cast<uintptr_t>(a.gate) & 3) == 0)) &&
+         al(a.out) && (!a.gate || a.gate_per_head || (a.ld_gate % 2 == 0 && (reinterpret_cast<uintptr_t>(a.gate) & 3) == 0)) &&
          (a.vc || a.vdim <= a.dim) && (!a.key_scale || (a.dim == a.vdim && !a.vc && al(a.key_scale)));
 }
 

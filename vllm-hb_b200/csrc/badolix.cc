@@ -14,37 +14,6 @@ namespace hb {
 
 bool is_badolix(const Json& config) { return config.string_or("architecture", "") == "Badolix"; }
 
-// Frequencies base^(-2i / dims) of channel pairs (i, i + dims / 2).  Scaling by a factor alone divides
-// them all.  `ramped` (YaRN): pairs that turn more than `fast` times within `original` positions keep
-// theirs, those that turn less than `slow` times are divided, a ramp over the pair's number lies between
-// them, and sines and cosines grow with the logarithm of the factor.
-static int read_rotation(const Json* rot, const std::string& t, int width, bool ramped, AttentionSpec* a) {
-  const double pi = 3.14159265358979323846;
-  const double base = rot->number_or("base", 0);
-  const int64_t dims = int_of(rot, "dims");
-  if (base <= 0 || dims < 0 || dims % 2 || dims > width) return fail(HB_ERR_INVALID_ARG, "%s: bad rotation", t.c_str());
-  const Json* s = object_of(*rot, "scaling");
-  const double factor = s ? s->number_or("factor", 0) : 1;
-  if (!(factor > 0)) return fail(HB_ERR_INVALID_ARG, "%s: bad rotation scaling", t.c_str());
-  a->rotation_halves = true;
-  double lo = 0, hi = 0;
-  const bool ramp = ramped && s;
-  if (ramp) {
-    const double original = s->number_or("original", 0), fast = s->number_or("fast", 0), slow = s->number_or("slow", 0);
-    if (!(original > 0) || !(fast > 0) || !(slow > 0) || base == 1) return fail(HB_ERR_INVALID_ARG, "%s: bad rotation scaling", t.c_str());
-    auto pair_of = [&](double turns) { return (double)dims * std::log(original / (2.0 * pi * turns)) / (2.0 * std::log(base)); };
-    lo = std::max(std::floor(pair_of(fast)), 0.0);
-    hi = std::min(std::ceil(pair_of(slow)), (double)dims - 1.0);
-    a->rotation_gain = (float)(0.1 * std::log(factor) + 1.0);
-  }
-  for (int64_t i = 0; i < dims / 2; ++i) {
-    const double f = std::pow(base, -2.0 * (double)i / (double)dims);
-    const double slowed = ramp ? std::min(1.0, std::max(0.0, ((double)i - lo) / std::max(hi - lo, 0.001))) : 1.0;
-    a->rotation.push_back(f / factor * slowed + f * (1.0 - slowed));
-  }
-  return HB_OK;
-}
-
 static int read_attention(const Json* m, const std::string& t, size_t layer, const LayeredSpec& spec, MixerSpec* out) {
   AttentionSpec& a = out->attn;
   out->has_attn = true;
@@ -77,7 +46,7 @@ static int read_attention(const Json* m, const std::string& t, size_t layer, con
   }
   out->attn_o = t + "o";
   const Json* rot = object_of(*m, "rot");
-  return rot ? read_rotation(rot, t, a.dim, false, &a) : HB_OK;
+  return rot ? read_rotation(rot, t, a.dim, false, true, &a) : HB_OK;
 }
 
 static int read_latent(const Json* m, const std::string& t, MixerSpec* out) {
@@ -99,7 +68,7 @@ static int read_latent(const Json* m, const std::string& t, MixerSpec* out) {
   out->attn_uv = t + "uv";
   out->attn_o = t + "o";
   const Json* rot = object_of(*m, "rot");
-  return rot ? read_rotation(rot, t, a.rot_dim, true, &a) : HB_OK;
+  return rot ? read_rotation(rot, t, a.rot_dim, true, true, &a) : HB_OK;
 }
 
 static int read_mamba2(const Json* m, const std::string& t, MixerSpec* out) {

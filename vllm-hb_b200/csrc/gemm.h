@@ -14,15 +14,22 @@ int gemm_simt(cudaStream_t st, void* Y, const void* X, const void* W, int64_t M,
               int64_t K, hb_dtype dtype, bool out_f32);
 
 // Gated activation of a feed-forward: with g clipped from above and u to both sides at `limit`,
-//   act(g, u) = g * sigmoid(slope * (g + cubic * g^3)) * (u + shift).
+//   act(g, u) = g * sigmoid(slope * (g + cubic * g^3)) * (u + shift)         (kLogistic)
+//               g * (1 + erf(g / sqrt(2))) / 2 * (u + shift)                 (kErf).
 // The defaults are SiLU; gelu in its tanh form is slope = 2 sqrt(2 / pi), cubic = 0.044715, because
-// (1 + tanh(z)) / 2 = sigmoid(2 z).
+// (1 + tanh(z)) / 2 = sigmoid(2 z).  Without a gate (`single`) there is no u and its factor is 1; such a
+// form may also be limit * tanh(g / limit) (kTanh).
 struct GatedAct {
+  enum Form : int { kLogistic = 0, kErf = 1, kTanh = 2 };
   float slope = 1.f, cubic = 0.f, limit = INFINITY, shift = 0.f;
-  bool silu() const { return slope == 1.f && cubic == 0.f && limit == INFINITY && shift == 0.f; }
+  int form = kLogistic;
+  int single = 0;
+  bool silu() const {
+    return slope == 1.f && cubic == 0.f && limit == INFINITY && shift == 0.f && form == kLogistic && !single;
+  }
 };
 // out[m, i] = act(gate_up[m, i] + gate_bias[i], gate_up[m, inter + i] + up_bias[i]); rows of out have
-// stride inter, the biases may be null.
+// stride inter, the biases may be null.  (single: rows of inter numbers.)
 int gated_act(cudaStream_t st, void* out, const void* gate_up, int64_t M, int64_t inter, const GatedAct& act, hb_dtype dtype,
               const float* gate_bias = nullptr, const float* up_bias = nullptr);
 
@@ -67,6 +74,7 @@ enum TcEpilogue : int {
   kEpiSwiGLU = 1,    // W rows are [gate tile | up tile] pairs: Y = act(gate, up) (GatedAct), N_out = N/2
   kEpiResidual = 2,  // deferred RMSNorm producer (cluster plans only), see TcNormLink
   kEpiPush = 3,      // row-parallel partial pushed into the reducing ranks' staging, see TcNormLink
+  kEpiAct = 4,       // Y = act(acc), a GatedAct without a gate
 };
 
 // Deferred RMSNorm between two GEMMs of a single-rank decode step.  Instead of a separate
@@ -142,7 +150,7 @@ struct TcGemmPlan {
   int tmem_cols = 0;
   size_t smem_bytes = 0;
   int epilogue = kEpiStore;
-  GatedAct act;          // kEpiSwiGLU
+  GatedAct act;          // kEpiSwiGLU, kEpiAct
   const float *gate_bias = nullptr, *up_bias = nullptr;  // kEpiSwiGLU: [N], added before the activation
   TcHeads heads;         // heads > 0: TcHeads form
   int groups = 0;        // > 0: TcGroups form; rows of the batch operand are sorted by group

@@ -164,8 +164,10 @@ __device__ __forceinline__ void push_tile(const TcParams& p, const uint8_t* stag
 template <bool GENERAL>
 __device__ __forceinline__ float gated_f(float g, float u, const GatedAct& act) {
   if (!GENERAL) return silu_f(g) * u;
+  if (act.form == GatedAct::kTanh) return act.limit * tanhf(g / act.limit);
   g = fminf(g, act.limit);
   u = fminf(fmaxf(u, -act.limit), act.limit);
+  if (act.form == GatedAct::kErf) return g * normcdff(g) * (u + act.shift);
   const float z = act.slope * fmaf(act.cubic * g * g, g, g);
   // far below zero the gate is zero (the fast divide wants a denominator below 2^126)
   return z < -80.f ? 0.f : __fdividef(g, 1.f + __expf(-z)) * (u + act.shift);
@@ -197,6 +199,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const bool swiglu = p.epilogue == kEpiSwiGLU;
+  const bool single = GENERAL && p.epilogue == kEpiAct;
   const int n_acc = swiglu ? 2 : 1;
   TC_TRACE(tid == 0, 0);
   TC_LAUNCH_TRACE(0);
@@ -450,6 +453,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
     if (p.gate_bias) gate_b = __ldg(p.gate_bias + n_glob);
     if (p.up_bias) up_b = __ldg(p.up_bias + n_glob);
   }
+  auto alone = [&](float g) { return gated_f<GENERAL>(g, 1.f - act.shift, act); };
   auto gated = [&](float g, float u) { return BIAS ? gated_f<GENERAL>(g + gate_b, u + up_b, act) : gated_f<GENERAL>(g, u, act); };
 
   // Output tiles are staged in the (now idle) pipeline buffers as [batch row][128
@@ -569,7 +573,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           }
         }
 #pragma unroll
-        for (int j = 0; j < 16; ++j) g[j] = swiglu ? gated(g[j], u[j]) : g[j];
+        for (int j = 0; j < 16; ++j) g[j] = swiglu ? gated(g[j], u[j]) : single ? alone(g[j]) : g[j];
         if (p.post_scale) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) g[j] *= s_pscale[c0 + j];
@@ -719,6 +723,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
 #pragma unroll
           for (int j = 0; j < 16; ++j) v[j] = gated(v[j], u[j]);
         }
+        if (single) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j) v[j] = alone(v[j]);
+        }
         if (p.post_scale) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) v[j] *= s_pscale[g * 16 + j];
@@ -758,6 +766,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           tmem_ld16(t_lane + p.m_pad + c0, u);
 #pragma unroll
           for (int j = 0; j < 16; ++j) v[j] = gated(v[j], u[j]);
+        }
+        if (single) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j) v[j] = alone(v[j]);
         }
         if (n_glob < p.N) {
 #pragma unroll
@@ -814,7 +826,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           for (int j = 0; j < 8; ++j) {
             const int m = m0 + j;
             if (m < m_lim && n_glob < p.N) {
-              const float r = swiglu ? gated(g[j], u[j]) : g[j];
+              const float r = swiglu ? gated(g[j], u[j]) : single ? alone(g[j]) : g[j];
               if (p.out_f32) ((float*)p.Y)[(int64_t)(m_base + m) * p.ldy + n_glob] = r;
               else ((__nv_bfloat16*)p.Y)[(int64_t)(m_base + m) * p.ldy + n_glob] = __float2bfloat16_rn(r);
             }
@@ -961,7 +973,8 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
   pl.groups = groups ? groups->groups : 0;
   pl.group_rows = groups ? (int)N : 0;
   if (groups && (groups->groups < 1 || groups->m_pad < 16 || groups->m_pad > 128 || groups->m_pad % 16 || groups->max_tiles < 1 ||
-                 groups->likely_tiles < 1 || (int64_t)groups->max_tiles * groups->m_pad > M || epilogue > kEpiSwiGLU ||
+                 groups->likely_tiles < 1 || (int64_t)groups->max_tiles * groups->m_pad > M ||
+                 (epilogue > kEpiSwiGLU && epilogue != kEpiAct) ||
                  (groups->ldx && (groups->ldx < K || groups->ldx % 8)) || (groups->shared_w && (groups->shared_k % 8 ||
                  groups->shared_n < 1 || groups->shared_k < 8 || groups->ldx < std::max(K, groups->shared_k)))))
     return fail(HB_ERR_INVALID_ARG, "gemm_tc: bad groups");
@@ -1003,7 +1016,7 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
   // (measured: 8192 x 1024 at M = 128 15.4 -> 11.1 us, 1280 x 8192 19.0 -> 16.4 us).
   bool m_split = false;
   if (tuned && !groups && !heads && n_acc == 1 && pl.m_pad >= 128 && (int64_t)pl.n_tiles * k_chunks <= 2048 &&
-      (epilogue == kEpiStore || epilogue == kEpiPush)) {
+      (epilogue == kEpiStore || epilogue == kEpiPush || epilogue == kEpiAct)) {
     pl.m_pad = 64;
     m_split = true;
   }
@@ -1306,7 +1319,7 @@ int gemm_tc_run(const TcGemmPlan& pl, cudaStream_t st, void* Y, int64_t ldy, voi
   }
   cfg.attrs = attr;
   cfg.numAttrs = na;
-  const bool general = !pl.act.silu() || pl.gate_bias || pl.up_bias;
+  const bool general = !pl.act.silu() || pl.gate_bias || pl.up_bias || pl.epilogue == kEpiAct;
   auto* kernel = pl.groups ? gemm_tc_kernel<true, true, false>
                  : pl.heads.heads ? gemm_tc_kernel<false, false, true>
                  : general ? gemm_tc_kernel<false, true, false> : gemm_tc_kernel<false, false, false>;

@@ -22,7 +22,8 @@ struct LayeredDesign {
   bool (*serves)(const Json&);
   int (*read)(const Json&, LayeredSpec*);
 };
-static const LayeredDesign kDesigns[] = {{is_latarax, read_latarax}, {is_biberax, read_biberax}, {is_badolix, read_badolix}};
+static const LayeredDesign kDesigns[] = {{is_latarax, read_latarax}, {is_biberax, read_biberax}, {is_badolix, read_badolix},
+                                          {is_muzopel, read_muzopel}};
 
 static const LayeredDesign* design_of(const Json& config) {
   for (const LayeredDesign& d : kDesigns)
@@ -101,6 +102,25 @@ struct Loader {
     HB_CUDA_CHECK(cudaStreamSynchronize(e->stream));
     return HB_OK;
   }
+  // a convolution's weights [channels, taps] as [taps, channels]
+  int taps(float** dst, const std::string& name, int64_t channels, int taps) {
+    int rc;
+    if ((rc = dev_alloc(e, (void**)dst, (size_t)channels * taps * 4))) return rc;
+    m->params += channels * taps;
+    float* rows = nullptr;
+    HB_CUDA_CHECK(cudaMalloc((void**)&rows, (size_t)channels * taps * 4));
+    rc = src.fetch_all(name, channels, taps, rows, HB_F32);
+    if (!rc) rc = transpose_matrices(e->stream, *dst, rows, 1, channels, taps, 4);
+    const cudaError_t ce = cudaStreamSynchronize(e->stream);
+    cudaFree(rows);
+    if (rc) return rc;
+    HB_CUDA_CHECK(ce);
+    return HB_OK;
+  }
+  int sublayer(SublayerMix* q, const std::string& norm, const std::string& conv) {  // post_norm
+    const int rc = small(&q->norm, norm, 1, m->spec.width, 1.f);
+    return rc || conv.empty() ? rc : taps(&q->conv, conv, m->spec.width, m->spec.input_taps);
+  }
   int sublayer(SublayerMix* q, const std::string& in, const std::string& out, const std::string& mix,
                const std::string& norm) {
     const int S = m->spec.streams;
@@ -154,6 +174,10 @@ struct Loader {
     if ((rc = vector(&l->latent_norm, mx.attn_latent_norm, C, 1.f))) return rc;
     if ((rc = dev_alloc(e, &l->uk_t, uk)) || (rc = dev_alloc(e, &l->ukv, uk + (size_t)H * a.vdim * C * e->es))) return rc;
     l->uv = (uint8_t*)l->ukv + uk;
+    if (a.q_rank) {
+      if ((rc = vector(&l->q_latent_norm, mx.attn_q_latent_norm, a.q_rank, 1.f))) return rc;
+      if ((rc = linear(&l->uq, mx.attn_uq, H * (a.dim + a.rot_dim), a.q_rank))) return rc;
+    }
     if ((rc = src.fetch_all(mx.attn_uv, H * a.vdim, C, l->uv, e->dtype))) return rc;
     e->named[mx.attn_uv] = {l->uv, H * a.vdim, C};
     m->params += H * (a.dim + a.vdim) * C;
@@ -166,16 +190,7 @@ struct Loader {
     const RecurrenceSpec& r = mx.rec;
     const int64_t n = r.conv_channels();
     int rc;
-    if ((rc = dev_alloc(e, (void**)&l->conv_w, (size_t)n * r.conv_taps * 4))) return rc;
-    m->params += n * r.conv_taps;
-    float* rows = nullptr;
-    HB_CUDA_CHECK(cudaMalloc((void**)&rows, (size_t)n * r.conv_taps * 4));
-    rc = src.fetch_all(mx.rec_conv, n, r.conv_taps, rows, HB_F32);
-    if (!rc) rc = transpose_matrices(e->stream, l->conv_w, rows, 1, n, r.conv_taps, 4);
-    const cudaError_t ce = cudaStreamSynchronize(e->stream);
-    cudaFree(rows);
-    if (rc) return rc;
-    HB_CUDA_CHECK(ce);
+    if ((rc = taps(&l->conv_w, mx.rec_conv, n, r.conv_taps))) return rc;
     if ((rc = vector(&l->conv_b, mx.rec_conv_bias, n, 0.f))) return rc;
     if ((rc = vector(&l->dt_bias, mx.rec_dt_bias, r.heads, 0.f))) return rc;
     if ((rc = vector(&l->a_log, mx.rec_a_log, r.heads, 0.f))) return rc;
@@ -203,27 +218,30 @@ struct Loader {
     return linear(down, f.down, W, f.ff);
   }
   int experts(LayeredExperts* x, const ExpertsSpec& s, const FeedForwardSpec& shared) {
-    const int64_t W = m->spec.width, E = s.experts;
+    const int64_t W = m->spec.width, E = s.experts, halves = s.act.single ? 1 : 2;
     int rc;
     x->ffp = pad8(s.ff);
+    if (s.act.single && shared.ff) return fail(HB_ERR_INVALID_ARG, "experts without gates beside a shared one");
     LayeredLinear all_up, all_down;
-    if ((rc = alloc(&all_up, E * 2 * x->ffp, W)) || (rc = alloc(&all_down, E * pad8(W), s.ff))) return rc;
+    if ((rc = alloc(&all_up, E * halves * x->ffp, W)) || (rc = alloc(&all_down, E * pad8(W), s.ff))) return rc;
     for (int64_t i = 0; i < E; ++i) {
       const std::string t = s.prefix + std::to_string(i) + ".";
-      if ((rc = part(all_up, t + "gate", i * 2 * x->ffp, s.ff, W))) return rc;
-      if ((rc = part(all_up, t + "up", (i * 2 + 1) * x->ffp, s.ff, W))) return rc;
+      if (halves == 2 && (rc = part(all_up, t + "gate", i * 2 * x->ffp, s.ff, W))) return rc;
+      if ((rc = part(all_up, t + "up", (i * halves + halves - 1) * x->ffp, s.ff, W))) return rc;
       if ((rc = part(all_down, t + "down", i * pad8(W), W, s.ff))) return rc;
     }
     x->gate_up = all_up;
-    x->gate_up.N = 2 * x->ffp;
+    x->gate_up.N = halves * x->ffp;
     x->down = all_down;
     x->down.N = pad8(W);
-    if ((rc = dev_alloc(e, &x->router, (size_t)E * W * e->es))) return rc;
-    if ((rc = src.fetch_all(s.router, E, W, x->router, e->dtype))) return rc;
-    e->named[s.router] = {x->router, E, W};
-    m->params += E * W;
+    const int64_t O = s.outputs();
+    if ((rc = dev_alloc(e, &x->router, (size_t)O * W * e->es))) return rc;
+    if ((rc = src.fetch_all(s.router, O, W, x->router, e->dtype))) return rc;
+    e->named[s.router] = {x->router, O, W};
+    m->params += O * W;
+    if ((rc = vector(&x->correction, s.correction, O, 0.f))) return rc;
     if (shared.ff && (rc = gated(&x->shared_gate_up, &x->shared_down, &x->shared_ffp, shared))) return rc;
-    return vector(&x->router_bias, s.router_bias, E, 0.f);
+    return vector(&x->router_bias, s.router_bias, O, 0.f);
   }
 };
 }  // namespace
@@ -257,6 +275,7 @@ static int layered_load(hb_engine* e, TensorSource& src) {
     if ((rc = src.fetch_all(s.embed, s.vocab, W, m->head.w, e->dtype, m->head.K))) return rc;
   }
   if ((rc = ld.small(&m->final_norm, s.final_norm, 1, W, 1.f - s.norm_offset))) return rc;
+  if ((rc = ld.vector(&m->embed_norm, s.embed_norm, W, 1.f))) return rc;
   m->layers.resize(s.layers.size());
   for (size_t i = 0; i < s.layers.size(); ++i) {
     LayerSpec& sp = s.layers[i];
@@ -299,13 +318,24 @@ static int layered_load(hb_engine* e, TensorSource& src) {
       if ((rc = ld.small(&l.attn_out_norm, mx.attn_out_norm, 1, W, 1.f))) return rc;
       if ((rc = ld.small(&l.rec_out_norm, mx.rec_out_norm, 1, W, 1.f))) return rc;
     }
-    if ((rc = ld.sublayer(&l.sub1, sp.hc1_in, sp.hc1_out, sp.hc1_mix, sp.norm1))) return rc;
+    if (s.post_norm) rc = ld.sublayer(&l.sub1, sp.norm1, sp.conv1);
+    else rc = ld.sublayer(&l.sub1, sp.hc1_in, sp.hc1_out, sp.hc1_mix, sp.norm1);
+    if (rc) return rc;
+    if (!sp.depth.empty()) {  // generated: the newest result alone
+      const int64_t n = (int64_t)i + 2;
+      if ((rc = ld.vector(&l.depth, sp.depth, n, 0.f))) return rc;
+      std::vector<float> newest((size_t)n, 0.f);
+      newest.back() = 1.f;
+      if (src.generated() && (rc = ld.upload(l.depth, newest))) return rc;
+    }
     if (sp.moe.experts) rc = ld.experts(&l.moe, sp.moe, sp.ffn);
     else if (sp.ffn.ff) rc = ld.gated(&l.gate_up, &l.down, &l.ffp, sp.ffn);
     if (!rc && sp.ffn.ff && !sp.moe.experts) rc = ld.biases(&l, sp.ffn);
     if (rc) return rc;
     if (sp.has_ffn()) {
-      if ((rc = ld.sublayer(&l.sub2, sp.hc2_in, sp.hc2_out, sp.hc2_mix, sp.norm2))) return rc;
+      if (s.post_norm) rc = ld.sublayer(&l.sub2, sp.norm2, sp.conv2);
+      else rc = ld.sublayer(&l.sub2, sp.hc2_in, sp.hc2_out, sp.hc2_mix, sp.norm2);
+      if (rc) return rc;
     }
   }
   return HB_OK;
@@ -334,6 +364,7 @@ static size_t layered_layout(const hb_engine* e, LayeredStep* s) {
   s->off_chunk = l.take((size_t)s->n_chunks * sizeof(RowRange));
   for (int k = 0; k < kTileKinds; ++k) s->off_tile[k] = l.take((size_t)s->n_tiles[k] * sizeof(RowRange));
   s->off_row_list = l.take((size_t)s->rows * 4);
+  s->off_run = l.take((size_t)s->n_runs * sizeof(RowRange));
   s->off_tables = l.take((size_t)s->segs * e->max_blocks_per_seq * 4);
   s->off_expand_base = l.take(s->n_expand ? (size_t)s->segs * 4 : 0);
   s->off_expand_list = l.take((size_t)s->n_expand * 4);
@@ -348,6 +379,8 @@ constexpr int kExpandTokens = 32;
 constexpr size_t kExpandBytes = (size_t)512 << 20;
 // Decoded tokens: with fewer (row, kv head) units than this the keys may be split over several CTAs.
 constexpr int kSplitUnits = 592;
+// Most tokens of a run of the residual kernel: long runs repeat less, short ones fill the SMs.
+static int residual_run(int rows) { return rows <= 256 ? 4 : rows <= 1024 ? 8 : 16; }
 
 static SpanAttention span_args(const hb_engine* e, size_t i, const LayeredStep& s) {
   const LayeredModel* m = e->lm.get();
@@ -376,6 +409,7 @@ static SpanAttention span_args(const hb_engine* e, size_t i, const LayeredStep& 
   a.dist_bias = l.dist_bias; a.dist_len = l.dist_len;
   a.err = e->d_err;
   a.sink = l.sink;
+  a.gate_per_head = as.gate_per_head ? 1 : 0;
   if (mx.ag.rows) {
     a.gate = (const uint8_t*)m->proj + mx.ag.offset * e->es;
     a.ld_gate = l.proj.N;
@@ -397,8 +431,18 @@ static LatentPrep latent_args(const hb_engine* e, size_t i, const LayeredStep& s
   p.kc = e->kc[l.kv_pool]; p.num_blocks = e->num_blocks;
   p.norm = l.latent_norm; p.eps = m->spec.eps;
   p.rotation = l.rotation; p.pairs = (int)as.rotation.size(); p.rotation_gain = as.rotation_gain;
+  p.halves = as.rotation_halves ? 1 : 0;
+  if (as.q_rank) { p.qs = m->q; p.ld_qs = l.uq.N; }
   return p;
 }
+
+// The heads' queries as projected: part of the input projection, or out of a latent of their own.
+static const void* query_rows(const hb_engine* e, size_t i) {
+  const LayeredModel* m = e->lm.get();
+  const MixerSpec& mx = m->spec.layers[i].mixer;
+  return mx.attn.q_rank ? m->q : (const uint8_t*)m->proj + mx.aq.offset * e->es;
+}
+static int64_t query_stride(const LayeredLayer& l, const AttentionSpec& a) { return a.q_rank ? l.uq.N : l.proj.N; }
 
 // Attention of expanded segments: every head its own keys [dim | shared part] and values.
 static SpanAttention expanded_args(const hb_engine* e, size_t i, const LayeredStep& s) {
@@ -407,7 +451,7 @@ static SpanAttention expanded_args(const hb_engine* e, size_t i, const LayeredSt
   const AttentionSpec& as = mx.attn;
   const LayeredLayer& l = m->layers[i];
   SpanAttention a = span_args(e, i, s);
-  a.q = (const uint8_t*)m->proj + mx.aq.offset * e->es; a.ld_q = l.proj.N;
+  a.q = query_rows(e, i); a.ld_q = query_stride(l, as);
   a.out = m->attn; a.ld_out = l.attn_o.K;
   a.kv_heads = as.heads; a.dim = as.dim + as.rot_dim; a.vdim = as.vdim;
   const int64_t row = (int64_t)as.heads * (as.dim + as.vdim);
@@ -431,7 +475,7 @@ static TcHeads expand_rows(const AttentionSpec& a) {
 static TcHeads latent_q_heads(const LayeredLayer& l, const AttentionSpec& a) {
   TcHeads h;
   h.heads = a.heads;
-  h.ldx = l.proj.N; h.x_step = a.dim + a.rot_dim;
+  h.ldx = query_stride(l, a); h.x_step = a.dim + a.rot_dim;
   h.ldy = (int64_t)a.heads * a.key_width(); h.y_step = a.key_width();
   return h;
 }
@@ -501,11 +545,11 @@ static TcGroups moe_groups(const ExpertsSpec& x, bool shared, int rows, bool tc)
   TcGroups g;
   const int64_t n = (int64_t)rows * x.top;
   g.groups = x.experts;
-  g.m_pad = tc ? (int)std::min<int64_t>(128, pad_to((n * 3 / 2 + x.experts - 1) / x.experts, 16)) : 16;
+  g.m_pad = tc ? (int)std::min<int64_t>(128, pad_to(((int64_t)(rows * x.picks() * 1.5) + x.experts - 1) / x.experts, 16)) : 16;
   g.max_tiles = (int)(std::min<int64_t>(x.experts, n) + n / g.m_pad);
   // experts that some row of a random batch chooses, and their tiles
-  const double active = x.experts * (1.0 - std::pow(1.0 - 1.0 / x.experts, (double)n));
-  const double tiles = active * std::max(1.0, std::ceil((double)n / std::max(1.0, active) / g.m_pad));
+  const double picks = rows * x.picks(), active = x.experts * (1.0 - std::pow(1.0 - 1.0 / x.experts, picks));
+  const double tiles = active * std::max(1.0, std::ceil(picks / std::max(1.0, active) / g.m_pad));
   g.likely_tiles = (int)std::max<int64_t>(1, std::min<int64_t>((int64_t)tiles, g.max_tiles));
   if (shared) {
     const int more = (rows + g.m_pad - 1) / g.m_pad;
@@ -529,9 +573,12 @@ static TcGroups down_groups(TcGroups g, const LayeredExperts& w) {
   return g;
 }
 
-static MoeRouting moe_args(const LayeredModel* m, const ExpertsSpec& x, bool shared, const TcGroups& g) {
+static MoeRouting moe_args(const LayeredModel* m, const ExpertsSpec& x, const LayeredExperts& w, const TcGroups& g) {
+  const bool shared = w.shared_ffp > 0;
   MoeRouting r;
+  r.correction = w.correction;
   r.experts = x.experts; r.top = x.top; r.shared = shared ? 1 : 0;
+  r.softmax_all = x.softmax_all ? 1 : 0; r.identity = x.identity;
   r.sigmoid = x.sigmoid ? 1 : 0; r.groups = x.groups; r.keep = x.keep;
   r.m_pad = g.m_pad; r.max_tiles = g.max_tiles;
   r.ids = m->moe_ids; r.rank = m->moe_rank; r.place = m->moe_place; r.weight = m->moe_weight;
@@ -617,10 +664,22 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   for (int64_t b = 0; b < e->num_blocks; ++b) e->free_blocks.push_back(b);
   const int64_t R = pad_to(e->max_batch, 128);
   m->row_cap = R;
+  if (s.post_norm) {
+    for (size_t i = 0; i < s.layers.size(); ++i) {
+      const int64_t n = (int64_t)m->max_segs * (s.input_taps - 1) * s.width;
+      if (n <= 0) break;
+      e->num_state_slots = m->max_segs;
+      if ((rc = dev_alloc(e, (void**)&m->layers[i].sub1.conv_state, (size_t)n * 4, true))) return rc;
+      if (s.layers[i].has_ffn() && (rc = dev_alloc(e, (void**)&m->layers[i].sub2.conv_state, (size_t)n * 4, true))) return rc;
+    }
+    if ((rc = dev_alloc(e, &m->h2, (size_t)R * m->Hp * es, true))) return rc;
+    if ((rc = dev_alloc(e, (void**)&m->x2, (size_t)R * s.width * 4, true))) return rc;
+    if ((rc = dev_alloc(e, (void**)&m->results, (size_t)(s.layers.size() + 1) * R * s.width * 4, true))) return rc;
+  }
   m->max_chunks = e->max_batch / kRecChunk + std::min(m->max_segs, e->max_batch / (kShortSegment + 1)) + 1;
   int64_t max_attn = 0, max_rec = 0, max_o = 0, max_ffp = 0, max_cum = 0, max_state = 0, max_part = 0;
   int64_t max_experts = 0, max_top = 0, max_eff = 0, max_tiles = 0, max_conv = 0, max_latent_q = 0, max_latent_o = 0, max_expand_row = 0,
-          max_expand_latent = 0;
+          max_expand_latent = 0, max_q_latent = 0, max_q = 0;
   for (size_t i = 0; i < s.layers.size(); ++i) {
     LayeredLayer& l = m->layers[i];
     const MixerSpec& mx = s.layers[i].mixer;
@@ -649,6 +708,8 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
       if (a.rank) {
         max_latent_q = std::max(max_latent_q, (int64_t)a.heads * a.key_width());
         max_latent_o = std::max(max_latent_o, (int64_t)a.heads * a.rank);
+        max_q_latent = std::max(max_q_latent, l.uq.K);
+        max_q = std::max(max_q, l.uq.N);
         l.latent_tc = e->use_tc && gemm_tc_heads_supported(a.rank, a.dim, false, latent_q_heads(l, a)) &&
                       gemm_tc_heads_supported(a.vdim, a.rank, false, latent_v_heads(l, a));
         // over the latent a row and key cost more than with a head's own keys and values
@@ -662,7 +723,7 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
       if (l.rel && (rc = build_distance_bias(e, &l, a, e->max_blocks_per_seq * HB_BLOCK_SIZE))) return rc;
     }
     if (const ExpertsSpec& x = s.layers[i].moe; x.experts) {
-      if (x.experts > kMoeMaxExperts) return fail(HB_ERR_INVALID_ARG, "%d experts (at most %d)", x.experts, kMoeMaxExperts);
+      if (x.outputs() > kMoeMaxExperts) return fail(HB_ERR_INVALID_ARG, "%d experts (at most %d)", x.outputs(), kMoeMaxExperts);
       max_experts = std::max<int64_t>(max_experts, x.experts);
       max_top = std::max<int64_t>(max_top, x.top + 1);
       max_eff = std::max(max_eff, l.moe.ld());
@@ -707,6 +768,8 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   }
   if (max_conv && (rc = dev_alloc(e, &m->conv, (size_t)R * max_conv * es, true))) return rc;
   if (max_latent_q && (rc = dev_alloc(e, &m->latent_q, (size_t)R * max_latent_q * es, true))) return rc;
+  if (max_q && (rc = dev_alloc(e, &m->q_latent, (size_t)R * max_q_latent * es, true))) return rc;
+  if (max_q && (rc = dev_alloc(e, &m->q, (size_t)R * max_q * es, true))) return rc;
   if (max_latent_o && (rc = dev_alloc(e, &m->latent_o, (size_t)R * max_latent_o * es, true))) return rc;
   if (e->use_tc) {
     if ((rc = dev_alloc(e, (void**)&m->cum, (size_t)R * max_cum * 4))) return rc;
@@ -753,6 +816,7 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
   cap.n_chunks = m->max_chunks;
   for (size_t k = 0; k < m->tile_kinds.size(); ++k) cap.n_tiles[k] = e->max_batch / m->tile_kinds[k].positions + m->max_segs;
   cap.n_expand = (int)m->expand_blocks;
+  if (s.post_norm) cap.n_runs = e->max_batch / residual_run(1) + m->max_segs;
   e->inputs_bytes = layered_layout(e, &cap);
   if ((rc = dev_alloc(e, (void**)&e->d_inputs, e->inputs_bytes, true))) return rc;
   HB_CUDA_CHECK(cudaMallocHost((void**)&e->h_inputs, e->inputs_bytes));
@@ -778,7 +842,7 @@ static int layered_plans(hb_engine* e, int rows, LayeredPlans** out) {
   if (it != m->plans.end()) { *out = &it->second; return HB_OK; }
   LayeredPlans p;
   const size_t L = m->layers.size();
-  for (auto* v : {&p.proj, &p.latent_q, &p.latent_v, &p.attn_o, &p.rec_o, &p.gate_up, &p.down, &p.moe_gate_up, &p.moe_down}) v->resize(L);
+  for (auto* v : {&p.proj, &p.uq, &p.latent_q, &p.latent_v, &p.attn_o, &p.rec_o, &p.gate_up, &p.down, &p.moe_gate_up, &p.moe_down}) v->resize(L);
   size_t ws = 0;
   int rc;
   auto plan = [&](TcGemmPlan* pl, const void* X, const LayeredLinear& w, int epi, bool f32) -> int {
@@ -790,18 +854,18 @@ static int layered_plans(hb_engine* e, int rows, LayeredPlans** out) {
   for (size_t i = 0; i < L; ++i) {
     LayeredLayer& l = m->layers[i];
     if ((rc = plan(&p.proj[i], m->h, l.proj, kEpiStore, false))) return rc;
+    if ((rc = plan(&p.uq[i], m->q_latent, l.uq, kEpiStore, false))) return rc;
     if (l.latent_tc) {
-      const MixerSpec& mx = m->spec.layers[i].mixer;
-      const AttentionSpec& a = mx.attn;
+      const AttentionSpec& a = m->spec.layers[i].mixer.attn;
       const TcHeads q = latent_q_heads(l, a), v = latent_v_heads(l, a);
-      const void* X = (const uint8_t*)m->proj + mx.aq.offset * e->es;
-      if ((rc = gemm_tc_plan(&p.latent_q[i], X, l.uk_t, M, a.rank, a.dim, kEpiStore, false, e->device, 0, nullptr, &q))) return rc;
+      if ((rc = gemm_tc_plan(&p.latent_q[i], query_rows(e, i), l.uk_t, M, a.rank, a.dim, kEpiStore, false, e->device, 0, nullptr, &q))) return rc;
       if ((rc = gemm_tc_plan(&p.latent_v[i], m->latent_o, l.uv, M, a.vdim, a.rank, kEpiStore, false, e->device, 0, nullptr, &v))) return rc;
       ws = std::max(ws, std::max(p.latent_q[i].workspace_bytes(), p.latent_v[i].workspace_bytes()));
     }
     if ((rc = plan(&p.attn_o[i], m->attn, l.attn_o, kEpiStore, true))) return rc;
     if ((rc = plan(&p.rec_o[i], m->rec, l.rec_o, kEpiStore, true))) return rc;
-    if ((rc = plan(&p.gate_up[i], m->h, l.gate_up, kEpiSwiGLU, false))) return rc;
+    const void* ffn_in = m->spec.post_norm ? m->h2 : m->h;
+    if ((rc = plan(&p.gate_up[i], ffn_in, l.gate_up, kEpiSwiGLU, false))) return rc;
     p.gate_up[i].act = m->spec.layers[i].ffn.act;
     p.gate_up[i].gate_bias = l.gate_b; p.gate_up[i].up_bias = l.up_b;
     if ((rc = plan(&p.down[i], m->act, l.down, kEpiStore, true))) return rc;
@@ -811,7 +875,7 @@ static int layered_plans(hb_engine* e, int rows, LayeredPlans** out) {
     const TcGroups up = up_groups(g, l.moe, m->spec.layers[i].ffn.act), down = down_groups(g, l.moe);
     if ((int64_t)g.max_tiles * g.m_pad > m->moe_places) return fail(HB_ERR_INVALID_ARG, "experts of %d rows need more places", M);
     if ((rc = gemm_tc_plan(&p.moe_gate_up[i], m->moe_x, l.moe.gate_up.w, m->moe_places, l.moe.gate_up.N, l.moe.gate_up.K,
-                           kEpiSwiGLU, false, e->device, 0, &up))) return rc;
+                           x.act.single ? kEpiAct : kEpiSwiGLU, false, e->device, 0, &up))) return rc;
     p.moe_gate_up[i].act = x.act;
     if ((rc = gemm_tc_plan(&p.moe_down[i], m->moe_act, l.moe.down.w, m->moe_places, l.moe.down.N, l.moe.down.K, kEpiStore, false,
                            e->device, 0, &down))) return rc;
@@ -842,14 +906,24 @@ static int layered_expand_plans(hb_engine* e, int blocks, std::vector<TcGemmPlan
   return HB_OK;
 }
 
+// cap * tanh(z / cap), the logits' last step
+static GatedAct logit_act(const LayeredSpec& s) {
+  GatedAct a;
+  a.form = GatedAct::kTanh;
+  a.limit = s.logit_cap;
+  a.single = 1;
+  return a;
+}
+
 static int layered_head_plan(hb_engine* e, int want, TcGemmPlan** out) {
   LayeredModel* m = e->lm.get();
   const int M = (int)std::min<int64_t>(row_bucket(want), pad_to(e->max_logits_rows, 16));
   auto it = m->head_plans.find(M);
   if (it != m->head_plans.end()) { *out = &it->second; return HB_OK; }
   TcGemmPlan p;
-  int rc = gemm_tc_plan(&p, m->hf, m->head.w, M, m->head.N, m->head.K, kEpiStore, true, e->device);
+  int rc = gemm_tc_plan(&p, m->hf, m->head.w, M, m->head.N, m->head.K, m->spec.logit_cap > 0.f ? kEpiAct : kEpiStore, true, e->device);
   if (rc) return rc;
+  if (m->spec.logit_cap > 0.f) p.act = logit_act(m->spec);
   if ((rc = ensure_gemm_workspace(e, p.workspace_bytes()))) return rc;
   *out = &m->head_plans.emplace(M, p).first->second;
   return HB_OK;
@@ -887,6 +961,10 @@ static int layered_prepare(hb_engine* e, const StepBatch& batch, StepExec* x) {
   for (int g = 0; g < s.segs; ++g)
     for (size_t k = 0; k < m->tile_kinds.size(); ++k)
       if (cut(g, m->tile_kinds[k])) s.n_tiles[k] += (batch.segs[g].n + m->tile_kinds[k].positions - 1) / m->tile_kinds[k].positions;
+  if (m->spec.post_norm) {
+    s.run_rows = residual_run(s.rows);
+    for (const StepSeg& t : batch.segs) s.n_runs += (t.n + s.run_rows - 1) / s.run_rows;
+  }
   x->rows = batch.rows;
   x->logits_compact = true;
   x->input_bytes = layered_layout(e, &s);
@@ -903,6 +981,8 @@ static int layered_prepare(hb_engine* e, const StepBatch& batch, StepExec* x) {
   int32_t* row_list = (int32_t*)(in + s.off_row_list);
   int at_short = 0, at_long = s.n_short, n_long = 0, n_chunks = 0, n_tiles[kTileKinds] = {0}, at_token = 0, at_row = s.n_token_rows;
   int32_t* tables = (int32_t*)(in + s.off_tables);
+  RowRange* runs = (RowRange*)(in + s.off_run);
+  int n_runs = 0;
   for (int g = 0; g < s.segs; ++g) {
     const StepSeg& t = batch.segs[g];
     seg[g] = {t.row0, t.n, (int32_t)t.pos0, t.state_slot};
@@ -915,6 +995,8 @@ static int layered_prepare(hb_engine* e, const StepBatch& batch, StepExec* x) {
       for (int i = 0; i < t.n; i += kRecChunk)
         chunks[n_chunks++] = {g, t.row0 + i, std::min(kRecChunk, t.n - i), l.n++};
     }
+    if (s.run_rows)
+      for (int i = 0; i < t.n; i += s.run_rows) runs[n_runs++] = {g, t.row0 + i, std::min(s.run_rows, t.n - i), i / s.run_rows};
     for (size_t k = 0; k < m->tile_kinds.size(); ++k) {
       if (!cut(g, m->tile_kinds[k])) continue;
       RowRange* tiles = (RowRange*)(in + s.off_tile[k]);
@@ -979,23 +1061,24 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
     return gemm_simt_grouped(st, Y, X, w.w, w.N, w.K, e->dtype, false, g, m->moe_tiles);
   };
   // the experts' outputs of every row, side by side in moe_y
+  const void* ffn_in = sp.post_norm ? m->h2 : m->h;
   auto experts = [&](size_t i, const ExpertsSpec& x, const LayeredExperts& w, const GatedAct& shared_act) -> int {
     const bool shared = w.shared_ffp > 0;
     const TcGroups g = moe_groups(x, shared, e->use_tc ? row_bucket((int)rows) : (int)rows, e->use_tc);
     const TcGroups up = up_groups(g, w, shared_act), down = down_groups(g, w);
-    const MoeRouting r = moe_args(m, x, shared, g);
+    const MoeRouting r = moe_args(m, x, w, g);
     prof_mark(e, kCatRouting);
-    if ((rc = moe_route_top(st, r, m->h, m->Hp, w.router, w.router_bias, rows, W, e->dtype))) return rc;
-    if ((rc = moe_gather(st, r, m->moe_x, m->h, m->Hp, rows, e->dtype))) return rc;
+    if ((rc = moe_route_top(st, r, ffn_in, m->Hp, w.router, w.router_bias, rows, W, e->dtype))) return rc;
+    if ((rc = moe_gather(st, r, m->moe_x, ffn_in, m->Hp, rows, e->dtype))) return rc;
     e->last_launches += 2;
     prof_mark(e, kCatExpertsUp);
     if (e->use_tc) {
       if ((rc = grouped(&pl->moe_gate_up, i, m->moe_act, m->moe_x, w.gate_up, up))) return rc;
     } else {
       TcGroups raw = up;
-      raw.ldy = 2 * w.ld();
+      raw.ldy = (x.act.single ? 1 : 2) * w.ld();
       if ((rc = grouped(nullptr, i, m->moe_gu, m->moe_x, w.gate_up, raw))) return rc;
-      if ((rc = gated_act_grouped(st, m->moe_act, w.ld(), m->moe_gu, 2 * w.ld(), w.ffp, x.act, e->dtype, up, m->moe_tiles))) return rc;
+      if ((rc = gated_act_grouped(st, m->moe_act, w.ld(), m->moe_gu, raw.ldy, w.ffp, x.act, e->dtype, up, m->moe_tiles))) return rc;
       ++e->last_launches;
     }
     prof_mark(e, kCatExpertsDown);
@@ -1003,8 +1086,45 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
   };
   auto at = [&](void* p, int64_t elements) { return (void*)((uint8_t*)p + (size_t)elements * es); };
 
+  // post_norm: one boundary, and what lies ahead of it
+  const RowRange* runs = (const RowRange*)(in + s.off_run);
+  float *x_now = m->results, *x_next = m->x;  // the residual, where the next boundary leaves it
+  const SublayerMix* read = nullptr;          // the sublayer whose input was formed last
+  auto residual = [&](ResidualStep r, const float* norm, const SublayerMix* next, void* h) -> int {
+    r.ld_y = m->Hp;
+    r.norm = norm; r.groups = sp.norm_groups; r.eps = sp.eps;
+    r.taps = std::max(1, sp.input_taps);
+    if (read) r.past = read->conv_state;
+    if (next) {
+      r.conv = next->conv; r.state = next->conv_state;
+      r.h = h; r.ld_h = m->Hp;
+    }
+    read = next;
+    ++e->last_launches;
+    prof_mark(e, kCatNorm);
+    return residual_step(st, r, runs, s.n_runs, seg, W, e->dtype);
+  };
+  // the sublayer's output back into the residual; `layer` >= 0: it ends this layer
+  auto post = [&](ResidualStep r, const float* norm, int64_t layer, const SublayerMix* next, void* h) -> int {
+    r.x = x_now;
+    r.x_out = x_next;
+    if (layer >= 0 && m->layers[layer].depth) {
+      r.earlier = m->results; r.step = m->row_cap * W; r.n_earlier = (int)layer + 1;
+      r.depth = m->layers[layer].depth;
+      r.result = m->results + (layer + 1) * r.step;
+    }
+    x_now = x_next;
+    x_next = x_next == m->x ? m->x2 : m->x;
+    return residual(r, norm, next, h);
+  };
+
   prof_mark(e, kCatOther);
-  if ((rc = streams_embed(st, m->x, m->h, m->embed, m->pos, ids, pos, m->layers[0].sub1.in, m->layers[0].sub1.norm, sp.norm_offset,
+  if (sp.post_norm) {
+    ResidualStep r;
+    r.embed = m->embed; r.ids = ids; r.vocab = sp.vocab;
+    r.x_out = m->results;
+    if ((rc = residual(r, m->embed_norm, &m->layers[0].sub1, m->h))) return rc;
+  } else if ((rc = streams_embed(st, m->x, m->h, m->embed, m->pos, ids, pos, m->layers[0].sub1.in, m->layers[0].sub1.norm, sp.norm_offset,
                           rows, S, W, m->Hp, sp.vocab, sp.max_positions, sp.eps, e->dtype, sp.embed_scale))) return rc;
   ++e->last_launches;
   for (size_t i = 0; i < m->layers.size(); ++i) {
@@ -1026,8 +1146,16 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
         if (l.latent_tc) return gemm_tc_run((*plans)[i], st, Y, h.ldy, e->d_gemm_ws, e->d_err);
         return gemm_simt_heads(st, Y, X, w, rows, N, K, e->dtype, false, h);
       };
+      if (as.q_rank) {
+        prof_mark(e, kCatNorm);
+        if ((rc = parts_norm(st, m->q_latent, l.uq.K, at(m->proj, mx.aq.offset), ldp, false, nullptr, l.q_latent_norm, rows, 1, as.q_rank,
+                             sp.eps, e->dtype))) return rc;
+        ++e->last_launches;
+        prof_mark(e, kCatGemm);
+        if ((rc = gemm(pl ? &pl->uq : nullptr, i, m->q, m->q_latent, l.uq, false))) return rc;
+      }
       const bool expand = l.expand && s.n_expand, latent = as.rank && !(expand && s.n_not_expanded == 0);
-      if (latent && (rc = heads(pl ? &pl->latent_q : nullptr, m->latent_q, at(m->proj, mx.aq.offset), l.uk_t, as.rank, as.dim,
+      if (latent && (rc = heads(pl ? &pl->latent_q : nullptr, m->latent_q, query_rows(e, i), l.uk_t, as.rank, as.dim,
                                  latent_q_heads(l, as)))) return rc;
       prof_mark(e, kCatRopeKv);
       AttentionPrep prep;
@@ -1105,9 +1233,19 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
       prof_mark(e, kCatNorm);
       return streams_mix(st, m->x, m->h, y, two ? m->y2 : nullptr, m->Hp, sm, rows, S, W, m->Hp, sp.eps, e->dtype);
     };
+    const bool more = i + 1 < m->layers.size();
+    if (sp.post_norm) {
+      ResidualStep r;
+      r.y = m->y1;
+      if (!lsp.has_ffn()) {
+        if ((rc = post(r, l.sub1.norm, (int64_t)i, more ? &m->layers[i + 1].sub1 : nullptr, m->h))) return rc;
+        continue;
+      }
+      if ((rc = post(r, l.sub1.norm, -1, &l.sub2, m->h2))) return rc;
+    }
     StreamMix mixed{};
     mixed.bias = l.o_bias;
-    if ((rc = boundary(l.sub1, m->y1, both, mixed))) return rc;
+    if (!sp.post_norm && (rc = boundary(l.sub1, m->y1, both, mixed))) return rc;
     if (!lsp.has_ffn()) continue;
     next = i + 1 < m->layers.size() ? &m->layers[i + 1].sub1 : nullptr;
     StreamMix fed{};
@@ -1118,26 +1256,44 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
     } else {
       prof_mark(e, kCatGemmGateUp);
       if (e->use_tc) {
-        if ((rc = gemm(&pl->gate_up, i, m->act, m->h, l.gate_up, false))) return rc;
+        if ((rc = gemm(&pl->gate_up, i, m->act, ffn_in, l.gate_up, false))) return rc;
       } else {
-        if ((rc = gemm(nullptr, i, m->gu, m->h, l.gate_up, false))) return rc;
+        if ((rc = gemm(nullptr, i, m->gu, ffn_in, l.gate_up, false))) return rc;
         if ((rc = gated_act(st, m->act, m->gu, rows, l.ffp, lsp.ffn.act, e->dtype, l.gate_b, l.up_b))) return rc;
         ++e->last_launches;
       }
       prof_mark(e, kCatGemmDown);
       if ((rc = gemm(pl ? &pl->down : nullptr, i, m->y1, m->act, l.down, true))) return rc;
     }
+    if (sp.post_norm) {
+      ResidualStep r;
+      if (lsp.moe.experts) {
+        r.expert_y = fed.expert_y; r.expert_place = fed.expert_place; r.expert_weight = fed.expert_weight; r.top = fed.top;
+        r.input = m->h2; r.ld_input = m->Hp;
+      } else {
+        r.y = m->y1;
+      }
+      if ((rc = post(r, l.sub2.norm, (int64_t)i, more ? &m->layers[i + 1].sub1 : nullptr, m->h))) return rc;
+      continue;
+    }
     fed.bias = l.down_b;
     if ((rc = boundary(l.sub2, lsp.moe.experts ? nullptr : m->y1, false, fed))) return rc;
   }
   if (s.want) {
     prof_mark(e, kCatNorm);
-    if ((rc = streams_final(st, m->hf, m->x, (const int32_t*)(in + s.off_want), m->final_norm, sp.norm_offset, s.want, S, W, m->Hp, sp.eps,
+    if (sp.post_norm) {
+      if ((rc = parts_norm(st, m->hf, m->Hp, x_now, W, true, (const int32_t*)(in + s.off_want), m->final_norm, s.want, sp.norm_groups,
+                           W / sp.norm_groups, sp.eps, e->dtype))) return rc;
+    } else if ((rc = streams_final(st, m->hf, m->x, (const int32_t*)(in + s.off_want), m->final_norm, sp.norm_offset, s.want, S, W, m->Hp, sp.eps,
                             e->dtype, sp.logit_scale))) return rc;
     prof_mark(e, kCatGemmLmHead);
     if (e->use_tc) rc = gemm_tc_run(*s.head_plan, st, e->d_logits, sp.vocab, e->d_gemm_ws, e->d_err);
     else rc = gemm_simt(st, e->d_logits, m->hf, m->head.w, s.want, m->head.N, m->head.K, e->dtype, true);
     if (rc) return rc;
+    if (!e->use_tc && sp.logit_cap > 0.f) {
+      if ((rc = gated_act(st, e->d_logits, e->d_logits, s.want, sp.vocab, logit_act(sp), HB_F32))) return rc;
+      ++e->last_launches;
+    }
     prof_mark(e, kCatOther);
     if ((rc = hb_argmax(st, e->d_next, e->d_logits, s.want, sp.vocab, HB_F32))) return rc;
     e->last_launches += 3;
@@ -1154,7 +1310,7 @@ static double layered_step_bytes(const hb_engine* e, const int32_t* ctx_lens, in
   double w = (double)m->head.N * m->head.K * es + 2.0 * n * s.width * es;
   for (size_t i = 0; i < s.layers.size(); ++i) {
     const LayeredLayer& l = m->layers[i];
-    for (const LayeredLinear* q : {&l.proj, &l.attn_o, &l.rec_o, &l.gate_up, &l.down}) w += (double)q->N * q->K * es;
+    for (const LayeredLinear* q : {&l.proj, &l.uq, &l.attn_o, &l.rec_o, &l.gate_up, &l.down}) w += (double)q->N * q->K * es;
     const MixerSpec& mx = s.layers[i].mixer;
     if (mx.has_attn) {
       const AttentionSpec& a = mx.attn;
@@ -1171,10 +1327,12 @@ static double layered_step_bytes(const hb_engine* e, const int32_t* ctx_lens, in
     if (mx.has_rec && mx.rec.per_token_decay) w += n * 2.0 * (mx.rec.conv_taps - 1) * mx.rec.conv_channels() * es;
     if (mx.has_rec) w += n * 2.0 * mx.rec.heads * mx.rec.dim * mx.rec.vdim * 4.0;
     w += n * (s.layers[i].has_ffn() ? 2.0 : 1.0) * 2.0 * s.streams * s.width * 4.0;
+    if (s.input_taps) w += n * (s.layers[i].has_ffn() ? 2.0 : 1.0) * s.input_taps * s.width * 4.0;
+    if (l.depth) w += n * ((double)i + 2.0) * s.width * 4.0;
     if (const ExpertsSpec& x = s.layers[i].moe; x.experts)  // the experts a random batch chooses
-      w += x.experts * (1.0 - std::pow(1.0 - 1.0 / x.experts, n * x.top)) *
+      w += x.experts * (1.0 - std::pow(1.0 - 1.0 / x.experts, n * x.picks())) *
                ((double)l.moe.gate_up.N * l.moe.gate_up.K + (double)l.moe.down.N * l.moe.down.K) * es +
-           ((double)x.experts * s.width + (double)l.moe.shared_gate_up.N * l.moe.shared_gate_up.K +
+           ((double)x.outputs() * s.width + (double)l.moe.shared_gate_up.N * l.moe.shared_gate_up.K +
             (double)l.moe.shared_down.N * l.moe.shared_down.K) * es;
   }
   return w;
@@ -1192,10 +1350,10 @@ static double layered_gemm_bytes(const hb_engine* e, int64_t rows) {
   double t = lin(m->head, (double)m->head.N, 4.0);
   for (size_t i = 0; i < m->layers.size(); ++i) {
     const LayeredLayer& l = m->layers[i];
-    t += lin(l.proj, (double)l.proj.N, es) + lin(l.attn_o, (double)l.attn_o.N, 4.0) + lin(l.rec_o, (double)l.rec_o.N, 4.0) +
+    t += lin(l.proj, (double)l.proj.N, es) + lin(l.uq, (double)l.uq.N, es) + lin(l.attn_o, (double)l.attn_o.N, 4.0) + lin(l.rec_o, (double)l.rec_o.N, 4.0) +
          (m->spec.layers[i].mixer.attn.rank ? latent(m->spec.layers[i].mixer.attn) : 0.0) + lin(l.gate_up, (double)l.ffp, es) + lin(l.down, (double)l.down.N, 4.0);
     if (const ExpertsSpec& x = m->spec.layers[i].moe; x.experts) {
-      const double picks = b * x.top, active = x.experts * (1.0 - std::pow(1.0 - 1.0 / x.experts, picks));
+      const double picks = b * x.picks(), active = x.experts * (1.0 - std::pow(1.0 - 1.0 / x.experts, picks));
       const LayeredExperts& w = l.moe;
       t += active * ((double)w.gate_up.N * w.gate_up.K + (double)w.down.N * w.down.K) * es +
            picks * ((double)w.gate_up.K + 2.0 * w.ffp + (double)w.down.N) * es +

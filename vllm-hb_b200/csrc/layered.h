@@ -1,7 +1,7 @@
 // Models described layer by layer: every layer has a mixer (attention, a gated linear
 // recurrence, or both side by side) and possibly a feed-forward (one gated layer, or a mixture of
 // them), over one or several residual streams held in fp32.  The mechanisms and their constants are
-// data (LayeredSpec); a design's reader (latarax.cc, biberax.cc, badolix.cc) turns its config.json and tensor
+// data (LayeredSpec); a design's reader (latarax.cc, biberax.cc, badolix.cc, muzopel.cc) turns its config.json and tensor
 // names into it.
 #pragma once
 
@@ -39,6 +39,8 @@ struct AttentionSpec {
   // attention runs over the latent itself (as keys and as values, with the heads' matrices applied to
   // queries and outputs).
   int rank = 0, rot_dim = 0;
+  int q_rank = 0;                   // > 0: the queries are a product of a normed latent of their own
+  bool gate_per_head = false;       // the output gate is one number per head (else one per channel)
   int cached_heads() const { return rank ? 1 : kv_heads; }
   int key_width() const { return rank ? rank + rot_dim : dim; }
   int value_width() const { return rank ? rank : vdim; }
@@ -65,10 +67,17 @@ struct ExpertsSpec {
   int experts = 0, top = 0;         // 0: no mixture
   bool sigmoid = false;
   int groups = 1, keep = 1;
+  // softmax_all: weighted by the softmax over all outputs of the router, chosen by that plus `correction`;
+  // the last `identity` outputs are no experts, they hand the input on
+  bool softmax_all = false;
+  int identity = 0;
   int64_t ff = 0;
-  GatedAct act;
-  std::string router, router_bias;
+  GatedAct act;                     // single: W_down act(W_up h)
+  std::string router, router_bias, correction;
   std::string prefix;               // expert e: prefix + "<e>." + gate | up | down
+  int outputs() const { return experts + identity; }
+  // experts a random row chooses
+  double picks() const { return (double)top * experts / outputs(); }
 };
 
 // S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per head, fp32 state of [dim, vdim].
@@ -113,6 +122,7 @@ struct MixerSpec {
   ProjPart rx, rdt;                          // selective state space: [v | k | q] before the convolution, steps
   std::string rec_conv, rec_conv_bias, rec_dt_bias, rec_a_log, rec_skip;
   std::string attn_latent_norm, attn_uk, attn_uv;  // latent attention (ak: [latent | shared key part])
+  std::string attn_q_latent_norm, attn_uq;         // with q_rank (aq: the queries' latent)
   std::string attn_o, rec_o, rec_norm, rec_a2, rec_a2_bias;
   // attention, empty where the design has none: biases of the projections, norms over the whole
   // query and key projections, distance bias table, learned sinks [heads]
@@ -124,6 +134,8 @@ struct LayerSpec {
   std::string prefix;                        // tensor name prefix, "l0."
   MixerSpec mixer;
   std::string norm1, norm2;
+  std::string conv1, conv2;                  // convolutions of the sublayers' inputs (input_taps)
+  std::string depth;                         // weights of the sum over all results so far (empty: none)
   std::string hc1_in, hc1_out, hc1_mix, hc2_in, hc2_out, hc2_mix;  // empty: one plain residual stream
   FeedForwardSpec ffn;                       // the layer's feed-forward, or what every token takes beside `moe`
   ExpertsSpec moe;
@@ -138,6 +150,14 @@ struct LayeredSpec {
   float norm_offset = 0.f;                   // of norm1, norm2, final norm: 0 stored as they apply, 1 around zero
   float embed_scale = 1.f, residual_mult = 1.f, logit_scale = 1.f;  // residual_mult: of designs with one plain stream
   std::string embed, pos, final_norm, head;  // pos empty: no learned positions; head empty: the embedding table
+  // post_norm: the norms are on the sublayers' outputs (and on the embedding), in norm_groups equal parts;
+  // the sublayers read the residual itself, to which a causal convolution of input_taps taps per channel is
+  // added (0: none).  One stream, residual.cu.
+  bool post_norm = false;
+  int norm_groups = 1;
+  int input_taps = 0;
+  std::string embed_norm;
+  float logit_cap = 0.f;                     // > 0: logits z become cap * tanh(z / cap)
   std::vector<LayerSpec> layers;
 };
 
@@ -148,6 +168,8 @@ bool is_biberax(const Json& config);
 int read_biberax(const Json& config, LayeredSpec* out);
 bool is_badolix(const Json& config);
 int read_badolix(const Json& config, LayeredSpec* out);
+bool is_muzopel(const Json& config);
+int read_muzopel(const Json& config, LayeredSpec* out);
 
 // ---------------------------------------------------------------------------- weights
 struct LayeredLinear {
@@ -160,15 +182,17 @@ struct SublayerMix {        // how a sublayer's output goes back into the stream
   float* out = nullptr;     // [streams]
   float* mix = nullptr;     // [streams from, streams to]
   float* norm = nullptr;    // [width]
+  // convolution of the sublayer's input: [taps, width]; inputs of earlier steps [slots, taps - 1, width]
+  float *conv = nullptr, *conv_state = nullptr;
 };
 
 struct LayeredExperts {     // experts' matrices one after another; the expert every token passes through
-  LayeredLinear gate_up, down;   // one expert's [2 * ffp, K] and [N, ffp]
+  LayeredLinear gate_up, down;   // one expert's [2 * ffp, K] (without a gate [ffp, K]) and [N, ffp]
   LayeredLinear shared_gate_up, shared_down;
   int64_t ffp = 0, shared_ffp = 0;
   int64_t ld() const { return ffp > shared_ffp ? ffp : shared_ffp; }  // row stride of the activations
-  void* router = nullptr;        // [experts, width] engine dtype
-  float* router_bias = nullptr;  // [experts]
+  void* router = nullptr;        // [outputs, width] engine dtype
+  float *router_bias = nullptr, *correction = nullptr;  // [outputs]
 };
 
 struct LayeredLayer {
@@ -187,6 +211,8 @@ struct LayeredLayer {
   void *uk_t = nullptr, *ukv = nullptr, *uv = nullptr;  // ukv [heads * dim | heads * vdim, rank]: W_uk, then W_uv
   bool expand = false;                       // prompts attend to keys and values of the heads grown out of the latents
   float* latent_norm = nullptr;
+  LayeredLinear uq;                          // queries out of their latent
+  float* q_latent_norm = nullptr;
   bool latent_tc = false;
   // selective state space
   float *conv_w = nullptr, *conv_b = nullptr, *dt_bias = nullptr, *a_log = nullptr, *skip = nullptr;
@@ -197,11 +223,12 @@ struct LayeredLayer {
   int tile_kind = -1, expand_kind = -1;      // indices into LayeredModel::tile_kinds (-1: row by row)
   float* state = nullptr;                    // [slots, heads, dim, vdim]
   SublayerMix sub1, sub2;
+  float* depth = nullptr;                    // [layers before this one + 2]
 };
 
 // Plans of all matrix products for one bucket of batch rows.
 struct LayeredPlans {
-  std::vector<TcGemmPlan> proj, latent_q, latent_v, attn_o, rec_o, gate_up, down, moe_gate_up, moe_down;
+  std::vector<TcGemmPlan> proj, uq, latent_q, latent_v, attn_o, rec_o, gate_up, down, moe_gate_up, moe_down;
 };
 
 struct LayeredGraph {
@@ -226,10 +253,12 @@ struct LayeredStep {
   int n_tiles[kTileKinds] = {0};  // query tiles of the tiled attention kernel, by tile size
   int n_expand = 0;       // blocks of the contexts whose keys and values are grown out of latents
   int n_not_expanded = 0; // rows of the other segments
+  int n_runs = 0;         // runs of tokens of the residual kernel, run_rows each at most
+  int run_rows = 0;
   int n_token_rows = 0;   // rows that are single decoded tokens (first in the list of rows)
   bool decode = false;    // every segment is one token
   size_t off_ids = 0, off_pos = 0, off_slots = 0, off_row_seg = 0, off_want = 0, off_seg = 0, off_short = 0,
-         off_long = 0, off_chunk = 0, off_tile[kTileKinds] = {0}, off_row_list = 0, off_tables = 0,
+         off_long = 0, off_chunk = 0, off_tile[kTileKinds] = {0}, off_row_list = 0, off_tables = 0, off_run = 0,
          off_expand_base = 0, off_expand_list = 0;
   LayeredPlans* plans = nullptr;
   TcGemmPlan* head_plan = nullptr;
@@ -241,7 +270,7 @@ struct LayeredModel {
   std::vector<LayeredLayer> layers;
   void *embed = nullptr, *pos = nullptr;     // [vocab, width], [max_positions, width] engine dtype, dense rows
   LayeredLinear head;                        // [vocab (padded), width (padded)]
-  float* final_norm = nullptr;
+  float *final_norm = nullptr, *embed_norm = nullptr;
   float* ones = nullptr;                     // [streams] of 1
   int64_t Hp = 0;                            // width padded to a multiple of 8
   int64_t params = 0;                        // elements of all tensors
@@ -250,6 +279,11 @@ struct LayeredModel {
   int64_t max_proj = 0;                      // widest projection row
   float* x = nullptr;                        // [rows, streams, width]
   void* h = nullptr;                         // [rows, Hp]
+  // post_norm: the feed-forward's input [rows, Hp], a second x, results of the embedding and all layers
+  // [layers + 1, row_cap, width]
+  void* h2 = nullptr;
+  float *x2 = nullptr, *results = nullptr;
+  void *q_latent = nullptr, *q = nullptr;    // queries out of a latent: [rows, q_rank], [rows, heads * (dim + rot_dim)]
   void* proj = nullptr;                      // [rows, max_proj]
   void *attn = nullptr, *rec = nullptr;      // branch outputs before their output projection
   float* o = nullptr;                        // [rows, heads * vdim] recurrence outputs

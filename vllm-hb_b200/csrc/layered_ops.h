@@ -59,6 +59,53 @@ struct GroupNorm {
 int gated_group_norm(cudaStream_t st, void* out, int64_t ld_out, const float* o, int64_t ld_o, const void* gate,
                      int64_t ld_gate, const float* weight, int64_t rows, const GroupNorm& n, hb_dtype dtype);
 
+// ------------------------------------- residual with normed sublayer outputs (residual.cu)
+// Rows of `tiles` (runs of consecutive tokens of a segment that together are all rows of the step):
+//   v = the output of a row: its embedding row, or y plus the weighted outputs of its experts (place -1:
+//       the row of `input` itself);
+//   x' = x + rms(v in `groups` equal parts of the width) * norm       (x null: zero) -> result
+//   x' = sum_l depth[l] earlier[l] + depth[n_earlier] x'                (depth null: as it is) -> x_out
+//   h = x' + sum_j conv[j] x'[t - (taps - 1) + j]                        (conv null: x')
+// with zeros before the sequence's start.  x_out, result and h may be null; none of them is a buffer that
+// is read here.  state [slots, taps - 1, width]: what earlier steps left of the convolution's inputs, the
+// one of position p at entry p mod (taps - 1); past: the same of the convolution that read x, which is
+// brought up to date here.
+constexpr int kResidualMaxTaps = 32;
+struct ResidualStep {
+  const float* y = nullptr;            // rows of stride ld_y
+  int64_t ld_y = 0;
+  const void* expert_y = nullptr;      // rows of the step's dtype, stride ld_y
+  const int32_t* expert_place = nullptr;
+  const float* expert_weight = nullptr;
+  int top = 0;
+  const void* input = nullptr;
+  int64_t ld_input = 0;
+  const void* embed = nullptr;         // [vocab, width]
+  const uint32_t* ids = nullptr;
+  int64_t vocab = 0;
+  const float* norm = nullptr;
+  int groups = 1;
+  float eps = 0.f;
+  const float* x = nullptr;            // [rows, width]
+  float *result = nullptr, *x_out = nullptr;
+  const float* earlier = nullptr;      // n_earlier times [rows, width], `step` elements apart
+  int64_t step = 0;
+  int n_earlier = 0;
+  const float* depth = nullptr;
+  const float* conv = nullptr;         // [taps, width]
+  int taps = 1;
+  const float* state = nullptr;
+  float* past = nullptr;
+  void* h = nullptr;
+  int64_t ld_h = 0;
+};
+int residual_step(cudaStream_t st, const ResidualStep& a, const RowRange* tiles, int n_tiles, const SegInfo* segs, int64_t width,
+                  hb_dtype dtype);
+// out[r] = rms of in[list ? list[r] : r] in `groups` parts of `size` channels * weight [groups * size]; in
+// rows of `dtype`, or (in_f32) fp32.
+int parts_norm(cudaStream_t st, void* out, int64_t ld_out, const void* in, int64_t ld_in, bool in_f32, const int32_t* list,
+               const float* weight, int64_t rows, int groups, int64_t size, float eps, hb_dtype dtype);
+
 // --------------------------------------------------------------- attention (attention_span.cu)
 // Paged attention whose queries see the last `window` positions (0 = all) and the first
 // `keep_first`, or (chunk > 0) the positions of their own chunk; keys and values of different
@@ -68,7 +115,8 @@ int gated_group_norm(cudaStream_t st, void* out, int64_t ld_out, const float* o,
 // values are the first vdim channels of the keys (a latent that both are made of); with key_scale
 // [num_blocks * 16] the K pool then holds the values, and a key is its value times a scale of its own
 // (a norm over the whole projection; the norm's weight is part of q).  sink [heads]: one more member of the softmax with this score and no value.  gate (row r,
-// head h at gate + r * ld_gate + h * vdim): the output is multiplied by its sigmoid.
+// head h at gate + r * ld_gate + h * vdim): the output is multiplied by its sigmoid.  With gate_per_head
+// a head has one number, at gate + r * ld_gate + h.
 struct SpanAttention {
   const void* q = nullptr;     // row r, head h at q + r * ld_q + h * dim
   int64_t ld_q = 0;
@@ -88,6 +136,11 @@ struct SpanAttention {
   const float* sink = nullptr;
   const void* gate = nullptr;
   int64_t ld_gate = 0;
+  int gate_per_head = 0;
+  // element of `gate` that meets channel c of a head
+  __host__ __device__ __forceinline__ int64_t gate_at(int64_t row, int64_t head, int c) const {
+    return row * ld_gate + (gate_per_head ? head : head * vdim + c);
+  }
   // Where keys and values lie, in elements: token j of a block at block * step.block + head * step.head +
   // j * step.token (all zero: the pools above).  With `linear` tables holds one number per segment and
   // its blocks follow one another from there.  The last `tail` channels of every key are one vector per
@@ -177,12 +230,15 @@ struct AttentionPrep {
 // `rank` channels and a key part of rot_dim channels that all heads share.  The latent is RMS-normed
 // (weight norm), the key part rotated, and both go to the token's slot of kc [num_blocks, 16, rank +
 // rot_dim]; the rotated parts of the queries go back to their place and to q, head h at q + r * ld_q + h *
-// (rank + rot_dim) + rank.  (The other `rank` channels there come from a product of heads: W_uk^T on the first dim
+// (rank + rot_dim) + rank.  With qs the queries lie there instead, head h of row r at qs + r * ld_qs + h * (dim +
+// rot_dim).  (The other `rank` channels there come from a product of heads: W_uk^T on the first dim
 // channels, so that a query meets the latent itself.)
 struct LatentPrep {
   void* p = nullptr;
   int64_t ld = 0;
   int off_q = 0, off_c = 0;
+  void* qs = nullptr;
+  int64_t ld_qs = 0;
   int heads = 0, dim = 0, rot_dim = 0, rank = 0;
   void* q = nullptr;
   int64_t ld_q = 0;
@@ -192,8 +248,8 @@ struct LatentPrep {
   int64_t num_blocks = 0;
   const float* norm = nullptr;
   float eps = 0.f;
-  const double* rotation = nullptr;    // [pairs], halves
-  int pairs = 0;
+  const double* rotation = nullptr;    // [pairs]
+  int pairs = 0, halves = 1;           // channel i with i + pairs, or (0) 2i with 2i + 1
   float rotation_gain = 1.f;
 };
 int latent_prepare(cudaStream_t st, const LatentPrep& a, int64_t rows, hb_dtype dtype);
@@ -215,6 +271,11 @@ struct MoeRouting {
   // the chosen logits); only experts of the `keep` best of `groups` equal groups of neighbours can be
   // chosen, a group counting the sum of its two largest scores
   int sigmoid = 0, groups = 1, keep = 1;
+  // softmax_all: scores and weights are the softmax over all outputs, the choice is by score + correction
+  // [experts + identity] (may be null)
+  int softmax_all = 0;
+  const float* correction = nullptr;
+  int identity = 0;                    // router outputs behind the experts that hand the row on: place -1
   int m_pad = 0, max_tiles = 0;        // TcGroups
   int32_t *ids = nullptr, *rank = nullptr, *place = nullptr;  // [rows, picks()]
   float* weight = nullptr;             // [rows, picks()]
@@ -222,13 +283,14 @@ struct MoeRouting {
   int32_t* first = nullptr;            // [experts + shared] first place of an expert
   int32_t* tile_group = nullptr;       // [max_tiles]
   __host__ __device__ __forceinline__ int picks() const { return top + shared; }
+  __host__ __device__ __forceinline__ int outputs() const { return experts + identity; }
 };
 // Router logits h . router^T (+ bias) in fp32; the `top` largest per row (the lower expert among
 // equals), their weights, every chosen (row, expert) a rank among the expert's rows, and
 // the batch tiles of the experts: expert e has tiles of m_pad places from first[e] on.
 int moe_route_top(cudaStream_t st, const MoeRouting& m, const void* h, int64_t ld_h, const void* router, const float* bias,
                   int64_t rows, int64_t width, hb_dtype dtype);
-// place[r, k] = first[expert] + rank, and row r of h goes to these places of x (rows of ld elements).
+// place[r, k] = first[expert] + rank (-1: no expert, the row itself), and row r of h goes to these places of x (rows of ld elements).
 int moe_gather(cudaStream_t st, const MoeRouting& m, void* x, const void* h, int64_t ld, int64_t rows, hb_dtype dtype);
 
 // ------------------------------------------------------------ linear recurrence (recurrence.cu)

@@ -1,5 +1,6 @@
-// Mixture of experts with top-k routing (softmax over the chosen logits, or sigmoid scores with the
-// choice limited to the best groups of experts), each expert run on its own rows only.
+// Mixture of experts with top-k routing (softmax over the chosen logits; sigmoid scores with the choice
+// limited to the best groups of experts; or softmax over all with a corrected choice, where some outputs
+// may hand the row itself on), each expert run on its own rows only.
 //
 //   route   logits, the top experts of every row and their weights; every (row, expert) draws a rank
 //           among the expert's rows; the last CTA turns the counts into batch tiles
@@ -24,15 +25,15 @@ __global__ void __launch_bounds__(kRouteThreads)
 moe_route_top_kernel(const MoeRouting m, const T* __restrict__ h, int64_t ld_h, const T* __restrict__ router,
                      const float* __restrict__ bias, int64_t rows, int64_t width) {
   pdl_trigger();
-  extern __shared__ float s_logit[];  // [RB][experts], then [RB][groups]
+  extern __shared__ float s_logit[];  // [RB][outputs], then [RB][groups] and (softmax_all) [RB][outputs] scores
   __shared__ int s_last;
   pdl_grid_wait();
   constexpr int N = Vec16<T>::N;
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, E = m.experts;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, E = m.experts, O = m.outputs();
   const int64_t row0 = (int64_t)blockIdx.x * RB;
   const int nr = (int)min((int64_t)RB, rows - row0);
   const bool vec = width % N == 0 && ld_h % N == 0;
-  for (int e = warp; e < E; e += kRouteWarps) {
+  for (int e = warp; e < O; e += kRouteWarps) {
     const T* w = router + (int64_t)e * width;
     float acc[RB];
 #pragma unroll
@@ -67,18 +68,18 @@ moe_route_top_kernel(const MoeRouting m, const T* __restrict__ h, int64_t ld_h, 
       const float s = warp_sum(acc[r]);
       if (lane == 0) {
         const float z = bias ? s + bias[e] : s;
-        s_logit[r * E + e] = m.sigmoid ? 1.f / (1.f + expf(-z)) : z;
+        s_logit[r * O + e] = m.sigmoid ? 1.f / (1.f + expf(-z)) : z;
       }
     }
   }
   __syncthreads();
   // one warp per row: the largest logit `top` times, the lower expert among equals
   for (int r = warp; r < nr; r += kRouteWarps) {
-    float* z = s_logit + r * E;
+    float *z = s_logit + r * O, *score = s_logit + RB * (O + m.groups) + r * O;
     const int64_t at = (row0 + r) * m.picks();
     if (m.keep < m.groups) {
       // groups by the sum of their two largest scores; experts of the others cannot be chosen
-      float* gs = s_logit + RB * E + r * m.groups;
+      float* gs = s_logit + RB * O + r * m.groups;
       const int size = E / m.groups;
       for (int g = lane; g < m.groups; g += 32) {
         float a = -INFINITY, b = -INFINITY;
@@ -98,25 +99,40 @@ moe_route_top_kernel(const MoeRouting m, const T* __restrict__ h, int64_t ld_h, 
       }
       __syncwarp();
     }
+    if (m.softmax_all) {
+      float mx = -INFINITY, total = 0.f;
+      for (int e = lane; e < O; e += 32) mx = fmaxf(mx, z[e]);
+      mx = warp_max(mx);
+      for (int e = lane; e < O; e += 32) {
+        score[e] = expf(z[e] - mx);
+        total += score[e];
+      }
+      total = warp_sum(total);
+      for (int e = lane; e < O; e += 32) {
+        score[e] /= total;
+        z[e] = m.correction ? score[e] + m.correction[e] : score[e];
+      }
+      __syncwarp();
+    }
     float first = 0.f, sum = 0.f;
     int mine = 0;        // lane k keeps choice k (of every 32) and its unscaled weight
     float mine_p = 0.f;
     for (int k = 0; k < m.top; ++k) {
       float best = -INFINITY;
-      int who = E;
-      for (int e = lane; e < E; e += 32)
-        if (z[e] > best || who == E) {
+      int who = O;
+      for (int e = lane; e < O; e += 32)
+        if (z[e] > best || who == O) {
           if (!isnan(z[e])) { best = z[e]; who = e; }
         }
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) {
         const float b = __shfl_xor_sync(0xffffffffu, best, o);
         const int w = __shfl_xor_sync(0xffffffffu, who, o);
-        if (w < E && (who == E || b > best || (b == best && w < who))) { best = b; who = w; }
+        if (w < O && (who == O || b > best || (b == best && w < who))) { best = b; who = w; }
       }
-      const int e = min(who, E - 1);  // a row of NaNs still names an expert
+      const int e = min(who, O - 1);  // a row of NaNs still names an expert
       if (k == 0) first = best;
-      const float p = m.sigmoid ? best : expf(best - first);
+      const float p = m.softmax_all ? score[e] : m.sigmoid ? best : expf(best - first);
       sum += p;
       if (lane == 0) z[e] = __int_as_float(0x7fc00000);  // taken
       if (lane == (k & 31)) {
@@ -129,12 +145,13 @@ moe_route_top_kernel(const MoeRouting m, const T* __restrict__ h, int64_t ld_h, 
         if (at_k <= k) {
           m.ids[at + at_k] = mine;
           m.weight[at + at_k] = mine_p;
-          m.rank[at + at_k] = atomicAdd(m.count + mine, 1);
+          m.rank[at + at_k] = mine < E ? atomicAdd(m.count + mine, 1) : 0;
         }
       }
     }
     __syncwarp();
-    for (int k = lane; k < m.top; k += 32) m.weight[at + k] /= m.sigmoid ? sum + 1e-20f : sum;  // written by this lane
+    if (!m.softmax_all)
+      for (int k = lane; k < m.top; k += 32) m.weight[at + k] /= m.sigmoid ? sum + 1e-20f : sum;  // written by this lane
     if (m.shared && lane == 0) {
       m.ids[at + m.top] = E;
       m.weight[at + m.top] = 1.f;
@@ -190,28 +207,35 @@ moe_gather_kernel(const MoeRouting m, T* __restrict__ x, const T* __restrict__ h
   if (v < ld / N) a.load(h + row * ld + v * N);  // on its way while the places are looked up
   for (int k = threadIdx.x; k < picks; k += kRouteThreads) {
     const int64_t at = row * picks + k;
-    const int p = m.first[m.ids[at]] + m.rank[at];
+    const int id = m.ids[at];
+    const bool expert = id < m.experts || (m.shared && k == m.top);
+    const int p = expert ? m.first[id] + m.rank[at] : -1;
     s_place[k] = p < places ? p : 0;  // never outside the buffer
     m.place[at] = s_place[k];
   }
   __syncthreads();
   for (; v < ld / N; v += kRouteThreads) {
     if (v >= kRouteThreads) a.load(h + row * ld + v * N);
-    for (int k = 0; k < picks; ++k) a.store(x + (int64_t)s_place[k] * ld + v * N);
+    for (int k = 0; k < picks; ++k)
+      if (s_place[k] >= 0) a.store(x + (int64_t)s_place[k] * ld + v * N);
   }
 }
 
 int moe_route_top(cudaStream_t st, const MoeRouting& m, const void* h, int64_t ld_h, const void* router, const float* bias,
                   int64_t rows, int64_t width, hb_dtype dtype) {
   if (rows == 0) return HB_OK;
-  if (m.experts < 1 || m.experts > kMoeMaxExperts || m.top < 1 || m.top > m.experts || m.m_pad < 1)
-    return fail(HB_ERR_INVALID_ARG, "moe_route_top: %d of %d experts (at most %d)", m.top, m.experts, kMoeMaxExperts);
-  if (m.groups < 1 || m.experts % m.groups || m.keep < 1 || m.keep > m.groups || m.top > m.experts / m.groups * m.keep)
+  if (m.experts < 1 || m.identity < 0 || m.outputs() > kMoeMaxExperts || m.top < 1 || m.top > m.outputs() || m.m_pad < 1)
+    return fail(HB_ERR_INVALID_ARG, "moe_route_top: %d of %d experts (at most %d)", m.top, m.outputs(), kMoeMaxExperts);
+  if (((m.identity || m.softmax_all) && m.groups > 1) || (m.identity && m.shared) || (m.correction && !m.softmax_all) ||
+      (m.sigmoid && m.softmax_all))
+    return fail(HB_ERR_INVALID_ARG, "moe_route_top: scores, groups, identity and shared experts do not go together");
+  if (m.groups < 1 || m.experts % m.groups || m.keep < 1 || m.keep > m.groups ||
+      (m.groups > 1 && m.top > m.experts / m.groups * m.keep))
     return fail(HB_ERR_INVALID_ARG, "moe_route_top: %d of %d groups of %d experts, top %d", m.keep, m.groups, m.experts, m.top);
   auto launch = [&](auto* k, int rb, auto* t) -> int {
     using T = std::remove_pointer_t<decltype(t)>;
     HB_CUDA_CHECK(launch_pdl(k, dim3((unsigned)((rows + rb - 1) / rb)), dim3(kRouteThreads),
-                             (size_t)rb * (m.experts + m.groups) * sizeof(float), st, m, (const T*)h, ld_h, (const T*)router, bias, rows, width));
+                             (size_t)rb * (m.outputs() * (m.softmax_all ? 2 : 1) + m.groups) * sizeof(float), st, m, (const T*)h, ld_h, (const T*)router, bias, rows, width));
     return HB_OK;
   };
   const bool few = rows <= 296;
@@ -258,11 +282,22 @@ __global__ void gated_act_kernel(T* __restrict__ out, int64_t ld_out, const T* _
       act = act2;
     }
   }
+  if (act.single) {
+    for (int64_t i = threadIdx.x; i < inter; i += blockDim.x) {
+      const float z = to_f32<T>(gu[row * ld_gu + i]), g = fminf(z, act.limit);
+      const float f = act.form == GatedAct::kTanh ? act.limit * tanhf(z / act.limit)
+                      : act.form == GatedAct::kErf ? g * normcdff(g)
+                                                   : g / (1.f + expf(-act.slope * (g + act.cubic * g * g * g)));
+      out[row * ld_out + i] = from_f32<T>(f);
+    }
+    return;
+  }
   for (int64_t i = threadIdx.x; i < inter; i += blockDim.x) {
     const float gb = gate_bias ? gate_bias[i] : 0.f, ub = up_bias ? up_bias[i] : 0.f;
     const float g = fminf(to_f32<T>(gu[row * ld_gu + i]) + gb, act.limit);
     const float u = fminf(fmaxf(to_f32<T>(gu[row * ld_gu + inter + i]) + ub, -act.limit), act.limit);
-    out[row * ld_out + i] = from_f32<T>(g / (1.f + expf(-act.slope * (g + act.cubic * g * g * g))) * (u + act.shift));
+    const float f = act.form == GatedAct::kErf ? g * normcdff(g) : g / (1.f + expf(-act.slope * (g + act.cubic * g * g * g)));
+    out[row * ld_out + i] = from_f32<T>(f * (u + act.shift));
   }
 }
 
@@ -270,8 +305,8 @@ int gated_act(cudaStream_t st, void* out, const void* gate_up, int64_t M, int64_
               const float* gate_bias, const float* up_bias) {
   if (M == 0) return HB_OK;
   HB_DISPATCH_DTYPE(dtype, T, {
-    HB_CUDA_CHECK(launch_pdl(gated_act_kernel<T>, dim3((unsigned)M), dim3(256), 0, st, (T*)out, inter, (const T*)gate_up, 2 * inter,
-                             inter, act, nullptr, 1, -1, 0, act, gate_bias, up_bias));
+    HB_CUDA_CHECK(launch_pdl(gated_act_kernel<T>, dim3((unsigned)M), dim3(256), 0, st, (T*)out, inter, (const T*)gate_up,
+                             act.single ? inter : 2 * inter, inter, act, nullptr, 1, -1, 0, act, gate_bias, up_bias));
   });
   return HB_OK;
 }
@@ -282,7 +317,7 @@ int gated_act_grouped(cudaStream_t st, void* out, int64_t ld_out, const void* ga
   if (rows == 0) return HB_OK;
   HB_DISPATCH_DTYPE(dtype, T, {
     HB_CUDA_CHECK(launch_pdl(gated_act_kernel<T>, dim3((unsigned)rows), dim3(256), 0, st, (T*)out, ld_out, (const T*)gate_up,
-                             ld_gu, inter, act, tile_group, g.m_pad, g.shared_w ? g.groups : -1, g.shared_n / 2, g.shared_act,
+                             ld_gu, inter, act, tile_group, g.m_pad, g.shared_w ? g.groups : -1, act.single ? g.shared_n : g.shared_n / 2, g.shared_act,
                              nullptr, nullptr));
   });
   return HB_OK;
