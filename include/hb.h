@@ -236,7 +236,8 @@ int hb_sample(void* stream, uint32_t* tokens, float* probs_workspace, const floa
  * (p / chunk == j / chunk); keys and values may differ in width.  Optional (NULL / 0: none):
  * dist_bias [heads, dist_len] is added to the scaled score by distance (the last entry also beyond
  * it); sink [heads] is the score of one more softmax member without a value; gate: the output is
- * multiplied by sigmoid(gate), row r, head h at gate + r*ld_gate + h*vdim (`dtype`); softcap: a scaled
+ * multiplied by sigmoid(gate), row r, head h at gate + r*ld_gate + h*vdim (`dtype`), or with gate_per_head
+ * by one number per head, at gate + r*ld_gate + h; softcap: a scaled
  * score s becomes softcap * tanh(s / softcap) (before the bias).
  * v_cache NULL: the values are the first vdim channels of the keys; with key_scale [num_blocks*16] (and
  * vdim == dim, v_cache unused) the K pool holds the values and a key is its value times the scale of its
@@ -266,6 +267,7 @@ typedef struct hb_span_attention_args {
   const void* gate;
   int64_t ld_gate;
   float softcap;
+  int gate_per_head;
 } hb_span_attention_args;
 int hb_span_attention_tile_positions(const hb_span_attention_args* a, hb_dtype dtype);
 int hb_span_attention(void* stream, const hb_span_attention_args* a, const int32_t* tiles, int n_tiles, const int32_t* rows,
@@ -302,9 +304,9 @@ int hb_attention_prepare(void* stream, const hb_attention_prep_args* a, int64_t 
 /* Attention over a latent that all heads share (hb_span_attention with kv_heads 1, dim = rank+rot_dim,
  * vdim = rank and no V pool).  Row r of p holds at off_q the heads' queries [dim | rot_dim] and at off_c
  * [latent of rank | key part of rot_dim].  The latent is RMS-normed (weight norm [rank]), the key part
- * rotated (channel i with i+pairs), both go to the row's slot of k_cache [num_blocks, 16, rank+rot_dim];
+ * rotated (channel i with i+pairs; neighbours: 2i with 2i+1), both go to the row's slot of k_cache [num_blocks, 16, rank+rot_dim];
  * the queries' rotated parts go back to their place and to q, head h at q + r*ld_q + h*(rank+rot_dim) +
- * rank.  fp32 inside. */
+ * rank.  With q_rows the queries lie there (row r at q_rows + r*ld_q_rows) and not in p.  fp32 inside. */
 typedef struct hb_latent_prep_args {
   void* p;
   int64_t ld;
@@ -320,6 +322,9 @@ typedef struct hb_latent_prep_args {
   const double* rotation;
   int pairs;
   float rotation_gain;
+  void* q_rows;
+  int64_t ld_q_rows;
+  int neighbours;
 } hb_latent_prep_args;
 int hb_latent_prepare(void* stream, const hb_latent_prep_args* a, int64_t rows, hb_dtype dtype);
 /* One product per head: Y_h[M, N] = X_h . W_h^T with the heads' [N, K] matrices one after another in W,
@@ -337,12 +342,16 @@ int hb_gemm_heads(void* stream, void* Y, const void* X, const void* W, int64_t M
  * sigmoid: scores sigmoid(logit), the chosen ones over their sum as weights; groups > 1: only experts of
  * the `keep` best of that many equal groups of neighbours are chosen, a group counting the sum of its
  * two largest scores.
+ * softmax_all: scores and weights are the softmax over all outputs, chosen by score + correction [experts +
+ * identity] (NULL: none).  The router's `identity` outputs behind the experts hand the row itself on: their
+ * choices have no rank, and place -1.
  * With `shared` every row has one pick more: group number `experts`, weight 1, tiles after all
  * others (ceil(rows / m_pad) of them, counted in max_tiles).
  * hb_moe_gather: row r of h (stride ld) to place[r,k] = first + rank in x.
  * hb_gemm_grouped: Y[r] = X[r] . W[group of r]^T with [N, K] weights per group, on the sorted rows
  * (X, Y: max_tiles*m_pad rows of strides ldx, ldy; bf16 with K % 8 == 0 and m_pad % 16 == 0 on tensor
- * cores); gated: the N rows are [gate | up] and Y = act(gate, up), N/2 wide (bf16 only). */
+ * cores); gated: the N rows are [gate | up] and Y = act(gate, up), N/2 wide, or (act.single) Y = act(X . W^T)
+ * (both bf16 only). */
 typedef struct hb_moe_routing {
   int experts, top, m_pad, max_tiles;
   int32_t *ids, *rank, *place; /* [rows, top + shared] */
@@ -350,14 +359,22 @@ typedef struct hb_moe_routing {
   int32_t *count, *first, *tile_group; /* [experts + 1], [experts + shared], [max_tiles] */
   int shared;
   int sigmoid, groups, keep; /* groups 0: one */
+  int identity, softmax_all;
+  const float* correction;
 } hb_moe_routing;
 int hb_moe_route_top(void* stream, const hb_moe_routing* m, const void* h, int64_t ld_h, const void* router,
                      const float* bias, int64_t rows, int64_t width, hb_dtype dtype);
 int hb_moe_gather(void* stream, const hb_moe_routing* m, void* x, const void* h, int64_t ld, int64_t rows, hb_dtype dtype);
 /* g clipped from above, u to both sides at `limit`: g * sigmoid(slope * (g + cubic * g^3)) * (u + shift).
- * SiLU: 1, 0, INFINITY, 0; gelu in its tanh form: 2 sqrt(2/pi), 0.044715, INFINITY, 0. */
+ * SiLU: 1, 0, INFINITY, 0; gelu in its tanh form: 2 sqrt(2/pi), 0.044715, INFINITY, 0.
+ * form HB_ACT_ERF: g * (1 + erf(g / sqrt(2))) / 2 * (u + shift).  single: there is no u, its factor is 1
+ * (rows of inter numbers); HB_ACT_TANH, single only: limit * tanh(g / limit). */
+#define HB_ACT_LOGISTIC 0
+#define HB_ACT_ERF 1
+#define HB_ACT_TANH 2
 typedef struct hb_gated_act_spec {
   float slope, cubic, limit, shift;
+  int form, single;
 } hb_gated_act_spec;
 int hb_gated_act(void* stream, void* out, const void* gate_up, int64_t M, int64_t inter, const hb_gated_act_spec* act,
                  hb_dtype dtype);
@@ -460,6 +477,49 @@ int hb_streams_mix_ex(void* stream, float* x, void* h, const float* y, const flo
                       hb_dtype dtype);
 int hb_streams_final(void* stream, void* h, const float* x, const int32_t* want, const float* norm, int64_t n_want,
                      int streams, int64_t width, int64_t ld_h, float eps, hb_dtype dtype);
+/* Residual x [rows, width] in fp32 of designs that norm what a sublayer puts out; `tiles` {segment, first
+ * row, rows, -}: runs of consecutive tokens, all rows of the step.  Per row
+ *   v = embed[ids], or y (NULL: zero) + sum_k expert_weight[r,k] * expert_y[expert_place[r,k]] (place -1: the
+ *       row of `input`);  x' = x (NULL: zero) + rms(v in `groups` equal parts of the width) * norm -> result;
+ *   x' = sum_l depth[l] * earlier[l*step + ..] + depth[n_earlier] * x' (depth NULL: as it is) -> x_out;
+ *   h = x' + sum_j conv[j] * x'[t - (taps-1) + j] (conv [taps, width]; NULL: x'), zeros before position 0.
+ * y and expert_y have rows of ld_y elements; x_out, result and h may be NULL and are not among what is read.
+ * state [slots, taps-1, width]: earlier inputs of the convolution, position p at entry p mod (taps-1); past
+ * (NULL: none): the same of the convolution that read x, brought up to date here.  taps <= 32. */
+typedef struct hb_residual_args {
+  const float* y;
+  int64_t ld_y;
+  const void* expert_y;
+  const int32_t* expert_place;
+  const float* expert_weight;
+  int top;
+  const void* input;
+  int64_t ld_input;
+  const void* embed;
+  const uint32_t* ids;
+  int64_t vocab;
+  const float* norm;
+  int groups;
+  float eps;
+  const float* x;
+  float *result, *x_out;
+  const float* earlier;
+  int64_t step;
+  int n_earlier;
+  const float* depth;
+  const float* conv;
+  int taps;
+  const float* state;
+  float* past;
+  void* h;
+  int64_t ld_h;
+} hb_residual_args;
+int hb_residual_step(void* stream, const hb_residual_args* a, const int32_t* tiles, int n_tiles, const int32_t* segments,
+                     int64_t width, hb_dtype dtype);
+/* out[r] = row list[r] (list NULL: r) of in, every one of `groups` parts of `size` channels over its rms, times
+ * weight [groups*size]; in is fp32 (in_f32) or `dtype`, out `dtype`. */
+int hb_parts_norm(void* stream, void* out, int64_t ld_out, const void* in, int64_t ld_in, int in_f32, const int32_t* list,
+                  const float* weight, int64_t rows, int groups, int64_t size, float eps, hb_dtype dtype);
 /* out[r, g*size + i] = o / rms over group g * weight[i] * act(gate); the weight [size] is shared by the
  * groups; act: SiLU with bit 0 of gate_mode, else sigmoid.  Bit 1: the product o * act(gate) is what is
  * normed, and weight is [groups*size]. */

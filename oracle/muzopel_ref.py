@@ -181,8 +181,9 @@ def tensor_shapes(config: dict) -> dict:
 
 def steady_routers(config: dict, weights: dict, channels: int = 6) -> dict:
     """The same model with routers that read only the last `channels` of the width, which the embedding
-    sets and no sublayer writes to (their norms' weights are zero there): rounding inside the layers
-    then hardly moves a score, and a 16-bit run chooses the experts an exact one does."""
+    sets and no sublayer writes to (their norms' weights are zero there, and so is the convolution ahead of
+    the router): rounding inside the layers then hardly moves a score, a token alone decides its experts,
+    and a 16-bit run chooses those an exact one does."""
     w = {k: v.copy() for k, v in weights.items()}
     rng = np.random.default_rng(7)
     w["embed"][:, -channels:] = rng.choice([-3.0, -2.0, -1.0, 1.0, 2.0, 3.0], w["embed"][:, -channels:].shape)
@@ -190,7 +191,7 @@ def steady_routers(config: dict, weights: dict, channels: int = 6) -> dict:
         if name.endswith(".router"):
             a[:, :-channels] = 0.0
             a[:, -channels:] = round_bf16((a[:, -channels:] * (a.shape[1] / channels) ** 0.5).astype(np.float32))
-        elif name.endswith((".norm1", ".norm2")):
+        elif name.endswith((".norm1", ".norm2", ".canon2")):
             a[-channels:] = 0.0
     return w
 

@@ -104,6 +104,7 @@ class SpanAttentionArgs(C.Structure):
         ("keep_first", C.c_int), ("scale", C.c_float),
         ("chunk", C.c_int), ("key_scale", C.c_void_p), ("dist_bias", C.c_void_p), ("dist_len", C.c_int),
         ("sink", C.c_void_p), ("gate", C.c_void_p), ("ld_gate", C.c_int64), ("softcap", C.c_float),
+        ("gate_per_head", C.c_int),
     ]
 
 
@@ -124,7 +125,8 @@ class LatentPrepArgs(C.Structure):
         ("p", C.c_void_p), ("ld", C.c_int64), ("off_q", C.c_int), ("off_c", C.c_int), ("heads", C.c_int), ("dim", C.c_int),
         ("rot_dim", C.c_int), ("rank", C.c_int), ("q", C.c_void_p), ("ld_q", C.c_int64), ("positions", C.c_void_p),
         ("slots", C.c_void_p), ("k_cache", C.c_void_p), ("num_blocks", C.c_int64), ("norm", C.c_void_p), ("eps", C.c_float),
-        ("rotation", C.c_void_p), ("pairs", C.c_int), ("rotation_gain", C.c_float),
+        ("rotation", C.c_void_p), ("pairs", C.c_int), ("rotation_gain", C.c_float), ("q_rows", C.c_void_p),
+        ("ld_q_rows", C.c_int64), ("neighbours", C.c_int),
     ]
 
 
@@ -142,12 +144,14 @@ class MoeRouting(C.Structure):
         ("experts", C.c_int), ("top", C.c_int), ("m_pad", C.c_int), ("max_tiles", C.c_int), ("ids", C.c_void_p),
         ("rank", C.c_void_p), ("place", C.c_void_p), ("weight", C.c_void_p), ("count", C.c_void_p), ("first", C.c_void_p),
         ("tile_group", C.c_void_p), ("shared", C.c_int), ("sigmoid", C.c_int), ("groups", C.c_int), ("keep", C.c_int),
+        ("identity", C.c_int), ("softmax_all", C.c_int), ("correction", C.c_void_p),
     ]
 
 
 class GatedActSpec(C.Structure):
-    """hb_gated_act_spec: g * sigmoid(slope * (g + cubic * g^3)) * (u + shift), clipped at limit."""
-    _fields_ = [("slope", C.c_float), ("cubic", C.c_float), ("limit", C.c_float), ("shift", C.c_float)]
+    """hb_gated_act_spec: g * sigmoid(slope * (g + cubic * g^3)) * (u + shift), clipped at limit, and other forms."""
+    _fields_ = [("slope", C.c_float), ("cubic", C.c_float), ("limit", C.c_float), ("shift", C.c_float), ("form", C.c_int),
+                ("single", C.c_int)]
 
 
 class GroupedGemm(C.Structure):
@@ -166,6 +170,18 @@ class StreamMixArgs(C.Structure):
         ("mix", C.c_void_p), ("out", C.c_void_p), ("next_in", C.c_void_p), ("next_norm", C.c_void_p), ("w1", C.c_void_p),
         ("w2", C.c_void_p), ("norm_offset", C.c_float), ("bias", C.c_void_p), ("expert_y", C.c_void_p),
         ("expert_place", C.c_void_p), ("expert_weight", C.c_void_p), ("top", C.c_int),
+    ]
+
+
+class ResidualArgs(C.Structure):
+    """hb_residual_args: a residual whose sublayers' outputs are normed, up to the next sublayer's input."""
+    _fields_ = [
+        ("y", C.c_void_p), ("ld_y", C.c_int64), ("expert_y", C.c_void_p), ("expert_place", C.c_void_p),
+        ("expert_weight", C.c_void_p), ("top", C.c_int), ("input", C.c_void_p), ("ld_input", C.c_int64), ("embed", C.c_void_p),
+        ("ids", C.c_void_p), ("vocab", C.c_int64), ("norm", C.c_void_p), ("groups", C.c_int), ("eps", C.c_float),
+        ("x", C.c_void_p), ("result", C.c_void_p), ("x_out", C.c_void_p), ("earlier", C.c_void_p), ("step", C.c_int64),
+        ("n_earlier", C.c_int), ("depth", C.c_void_p), ("conv", C.c_void_p), ("taps", C.c_int), ("state", C.c_void_p),
+        ("past", C.c_void_p), ("h", C.c_void_p), ("ld_h", C.c_int64),
     ]
 
 
@@ -208,6 +224,8 @@ _SIGS = {
     "hb_streams_embed": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i, _i64, _i64, _i64, _i64, _f, _i]),
     "hb_streams_mix": (_i, [_vp, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i, _i64, _i64, _f, _i]),
     "hb_streams_mix_ex": (_i, [_vp, _vp, _vp, _vp, _vp, _i64, _vp, _i64, _i, _i64, _i64, _f, _i]),
+    "hb_residual_step": (_i, [_vp, _vp, _vp, _i, _vp, _i64, _i]),
+    "hb_parts_norm": (_i, [_vp, _vp, _i64, _vp, _i64, _i, _vp, _vp, _i64, _i, _i64, _f, _i]),
     "hb_attention_prepare": (_i, [_vp, _vp, _i64, _i]),
     "hb_latent_prepare": (_i, [_vp, _vp, _i64, _i]),
     "hb_gemm_heads": (_i, [_vp, _vp, _vp, _vp, _i64, _i64, _i64, _i, _i64, _i64, _i64, _i64, _i]),

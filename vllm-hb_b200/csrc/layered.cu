@@ -545,7 +545,7 @@ static TcGroups moe_groups(const ExpertsSpec& x, bool shared, int rows, bool tc)
   TcGroups g;
   const int64_t n = (int64_t)rows * x.top;
   g.groups = x.experts;
-  g.m_pad = tc ? (int)std::min<int64_t>(128, pad_to(((int64_t)(rows * x.picks() * 1.5) + x.experts - 1) / x.experts, 16)) : 16;
+  g.m_pad = tc ? (int)std::min<int64_t>(128, pad_to(std::max<int64_t>(1, ((int64_t)(rows * x.picks() * 1.5) + x.experts - 1) / x.experts), 16)) : 16;
   g.max_tiles = (int)(std::min<int64_t>(x.experts, n) + n / g.m_pad);
   // experts that some row of a random batch chooses, and their tiles
   const double picks = rows * x.picks(), active = x.experts * (1.0 - std::pow(1.0 - 1.0 / x.experts, picks));

@@ -15,6 +15,7 @@ static SpanAttention span_of(const hb_span_attention_args* p) {
   a.key_scale = p->key_scale; a.dist_bias = p->dist_bias; a.dist_len = p->dist_len; a.sink = p->sink;
   a.gate = p->gate; a.ld_gate = p->ld_gate;
   a.softcap = p->softcap;
+  a.gate_per_head = p->gate_per_head;
   if (a.key_scale) a.vc = nullptr;
   return a;
 }
@@ -170,6 +171,7 @@ int hb_latent_prepare(void* stream, const hb_latent_prep_args* p, int64_t rows, 
   a.q = p->q; a.ld_q = p->ld_q; a.pos = p->positions; a.slots = p->slots; a.kc = p->k_cache; a.num_blocks = p->num_blocks;
   a.norm = p->norm; a.eps = p->eps; a.rotation = p->rotation; a.pairs = p->pairs;
   a.rotation_gain = p->rotation_gain == 0.f ? 1.f : p->rotation_gain;
+  a.qs = p->q_rows; a.ld_qs = p->ld_q_rows; a.halves = p->neighbours ? 0 : 1;
   return hb::latent_prepare((cudaStream_t)stream, a, rows, dtype);
 }
 
@@ -207,6 +209,7 @@ static hb::MoeRouting routing_of(const hb_moe_routing* p) {
   m.count = p->count; m.first = p->first; m.tile_group = p->tile_group;
   m.sigmoid = p->sigmoid;
   if (p->groups) { m.groups = p->groups; m.keep = p->keep; }
+  m.identity = p->identity; m.softmax_all = p->softmax_all; m.correction = p->correction;
   return m;
 }
 
@@ -214,6 +217,7 @@ int hb_moe_route_top(void* stream, const hb_moe_routing* m, const void* h, int64
                      const float* bias, int64_t rows, int64_t width, hb_dtype dtype) {
   HB_CHECK_ARG(m && h && router && m->ids && m->rank && m->weight && m->count && m->first && m->tile_group,
                "hb_moe_route_top: null argument");
+  HB_CHECK_ARG(m->identity >= 0, "hb_moe_route_top: a negative number of identities");
   HB_CHECK_ARG(rows >= 0 && width > 0 && m->m_pad > 0 &&
                m->max_tiles >= (rows * m->top < m->experts ? rows * m->top : m->experts) + rows * m->top / m->m_pad +
                                    (m->shared ? (rows + m->m_pad - 1) / m->m_pad : 0),
@@ -229,12 +233,20 @@ int hb_moe_gather(void* stream, const hb_moe_routing* m, void* x, const void* h,
 static hb::GatedAct act_of(const hb_gated_act_spec* p) {
   hb::GatedAct a;
   a.slope = p->slope; a.cubic = p->cubic; a.limit = p->limit; a.shift = p->shift;
+  a.form = p->form; a.single = p->single;
   return a;
+}
+
+static int check_act(const hb_gated_act_spec* p) {
+  HB_CHECK_ARG(p->form >= HB_ACT_LOGISTIC && p->form <= HB_ACT_TANH && (p->form != HB_ACT_TANH || p->single),
+               "activation: unknown form %d", p->form);
+  return HB_OK;
 }
 
 int hb_gated_act(void* stream, void* out, const void* gate_up, int64_t M, int64_t inter, const hb_gated_act_spec* act,
                  hb_dtype dtype) {
   HB_CHECK_ARG(out && gate_up && act && M >= 0 && inter > 0, "hb_gated_act: bad argument");
+  if (int rc = check_act(act)) return rc;
   return hb::gated_act((cudaStream_t)stream, out, gate_up, M, inter, act_of(act), dtype);
 }
 
@@ -251,14 +263,15 @@ static int check_grouped(const hb_grouped_gemm* p) {
   HB_CHECK_ARG(p && p->tile_group && p->groups > 0 && p->N > 0 && p->K > 0 && p->m_pad > 0 && p->max_tiles > 0 &&
                p->likely_tiles > 0 && p->ldx >= p->K && (!p->shared_w || (p->shared_n > 0 && p->shared_k > 0 && p->ldx >= p->shared_k)),
                "grouped gemm: bad argument");
-  return HB_OK;
+  HB_CHECK_ARG(!p->shared_w || !p->act.single == !p->shared_act.single, "grouped gemm: one activation with a gate, one without");
+  return check_act(&p->act);
 }
 
 int hb_gemm_grouped(void* stream, void* Y, const void* X, const void* W, const hb_grouped_gemm* p, hb_dtype dtype) {
   int rc = check_grouped(p);
   if (rc) return rc;
   const int64_t wide = p->shared_n > p->N ? p->shared_n : p->N;
-  HB_CHECK_ARG(Y && X && W && p->ldy >= (p->gated ? wide / 2 : wide), "hb_gemm_grouped: bad output");
+  HB_CHECK_ARG(Y && X && W && p->ldy >= (p->gated && !p->act.single ? wide / 2 : wide), "hb_gemm_grouped: bad output");
   const hb::TcGroups g = groups_of(p);
   const int64_t M = (int64_t)p->max_tiles * p->m_pad;
   auto st = (cudaStream_t)stream;
@@ -266,7 +279,7 @@ int hb_gemm_grouped(void* stream, void* Y, const void* X, const void* W, const h
     int dev = 0;
     HB_CUDA_CHECK(cudaGetDevice(&dev));
     hb::TcGemmPlan plan;
-    rc = hb::gemm_tc_plan(&plan, X, W, M, p->N, p->K, p->gated ? hb::kEpiSwiGLU : hb::kEpiStore, p->out_f32 != 0, dev, 0, &g);
+    rc = hb::gemm_tc_plan(&plan, X, W, M, p->N, p->K, !p->gated ? hb::kEpiStore : p->act.single ? hb::kEpiAct : hb::kEpiSwiGLU, p->out_f32 != 0, dev, 0, &g);
     if (rc) return rc;
     if (p->gated) plan.act = act_of(&p->act);
     return hb::gemm_tc_run(plan, st, Y, p->ldy, nullptr, nullptr, nullptr, p->tile_group);
@@ -278,10 +291,38 @@ int hb_gemm_grouped(void* stream, void* Y, const void* X, const void* W, const h
 int hb_gated_act_grouped(void* stream, void* out, const void* gate_up, int64_t ld_gu, const hb_grouped_gemm* p, hb_dtype dtype) {
   int rc = check_grouped(p);
   if (rc) return rc;
-  HB_CHECK_ARG(out && gate_up && ld_gu >= p->N && ld_gu >= p->shared_n && p->ldy >= p->N / 2 && p->ldy >= p->shared_n / 2,
+  const int per = p->act.single ? 1 : 2;
+  HB_CHECK_ARG(out && gate_up && ld_gu >= p->N && ld_gu >= p->shared_n && p->ldy >= p->N / per && p->ldy >= p->shared_n / per,
                "hb_gated_act_grouped: bad argument");
-  return hb::gated_act_grouped((cudaStream_t)stream, out, p->ldy, gate_up, ld_gu, p->N / 2, act_of(&p->act), dtype, groups_of(p),
+  return hb::gated_act_grouped((cudaStream_t)stream, out, p->ldy, gate_up, ld_gu, p->N / per, act_of(&p->act), dtype, groups_of(p),
                                p->tile_group);
+}
+
+int hb_residual_step(void* stream, const hb_residual_args* p, const int32_t* tiles, int n_tiles, const int32_t* segments,
+                     int64_t width, hb_dtype dtype) {
+  HB_CHECK_ARG(p && p->norm && (tiles || !n_tiles) && n_tiles >= 0 && segments, "hb_residual_step: null argument");
+  HB_CHECK_ARG((p->embed ? p->ids && p->vocab > 0 : p->y || p->top > 0) && p->top >= 0 &&
+               (!p->top || (p->expert_y && p->expert_place && p->expert_weight)), "hb_residual_step: no output of a sublayer");
+  HB_CHECK_ARG(p->n_earlier >= 0 && (!p->depth || p->earlier || !p->n_earlier), "hb_residual_step: bad sum over earlier results");
+  HB_CHECK_ARG(p->taps >= 1 && (!p->conv || p->taps == 1 || p->state) && (!p->past || p->x), "hb_residual_step: bad convolution");
+  hb::ResidualStep a;
+  a.y = p->y; a.ld_y = p->ld_y;
+  a.expert_y = p->expert_y; a.expert_place = p->expert_place; a.expert_weight = p->expert_weight; a.top = p->top;
+  a.input = p->input; a.ld_input = p->ld_input;
+  a.embed = p->embed; a.ids = p->ids; a.vocab = p->vocab;
+  a.norm = p->norm; a.groups = p->groups; a.eps = p->eps;
+  a.x = p->x; a.result = p->result; a.x_out = p->x_out;
+  a.earlier = p->earlier; a.step = p->step; a.n_earlier = p->n_earlier; a.depth = p->depth;
+  a.conv = p->conv; a.taps = p->taps; a.state = p->state; a.past = p->past;
+  a.h = p->h; a.ld_h = p->ld_h;
+  return hb::residual_step((cudaStream_t)stream, a, (const hb::RowRange*)tiles, n_tiles, (const hb::SegInfo*)segments, width, dtype);
+}
+
+int hb_parts_norm(void* stream, void* out, int64_t ld_out, const void* in, int64_t ld_in, int in_f32, const int32_t* list,
+                  const float* weight, int64_t rows, int groups, int64_t size, float eps, hb_dtype dtype) {
+  HB_CHECK_ARG(out && in && weight && rows >= 0 && groups > 0 && size > 0 && ld_in >= groups * size && ld_out >= groups * size,
+               "hb_parts_norm: bad argument");
+  return hb::parts_norm((cudaStream_t)stream, out, ld_out, in, ld_in, in_f32 != 0, list, weight, rows, groups, size, eps, dtype);
 }
 
 int hb_streams_final(void* stream, void* h, const float* x, const int32_t* want, const float* norm, int64_t n_want,

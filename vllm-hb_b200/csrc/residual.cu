@@ -111,21 +111,22 @@ residual_kernel(const ResidualStep a, const RowRange* __restrict__ tiles, const 
     }
   };
 
-  float win[HELD ? kHeldTaps - 1 : 1][NC][VEC];  // inputs of the last tokens, oldest first
+  const int i0 = max(-first, -back);
+  float win[HELD ? kHeldTaps - 1 : 1][NC][VEC];  // inputs of the tokens ahead of i0, oldest first
   auto held = [&](int b, int k, int j) -> float& {  // b tokens back (from 1), not HELD
     return s_win[((b - 1) * NC * VEC + k * VEC + j) * blockDim.x + threadIdx.x];
   };
   if (a.conv) {
 #pragma unroll
     for (int b = 1; b < (HELD ? kHeldTaps : a.taps); ++b) {
-      const int64_t p = (int64_t)seg.pos0 + first - b;
+      const int64_t p = (int64_t)seg.pos0 - b;
 #pragma unroll
       for (int k = 0; k < NC; ++k) {
         float f[VEC];
 #pragma unroll
         for (int j = 0; j < VEC; ++j) f[j] = 0.f;
-        // (tokens of this step are worked out below)
-        if (b <= back && first - b < 0 && p >= 0 && live(k))
+        // where the run's past reaches back beyond this step (else it is all worked out below)
+        if (b <= back && first + i0 == 0 && p >= 0 && live(k))
           load_row<float, VEC>(f, a.state + ((int64_t)seg.slot * ring + p % ring) * W + c0 + chan(k));
 #pragma unroll
         for (int j = 0; j < VEC; ++j) {
@@ -136,7 +137,6 @@ residual_kernel(const ResidualStep a, const RowRange* __restrict__ tiles, const 
     }
   }
 
-  const int i0 = max(-first, -back);
   float next[NC][VEC];
 #pragma unroll
   for (int k = 0; k < NC; ++k)
