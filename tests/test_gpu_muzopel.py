@@ -1,0 +1,444 @@
+"""Muzopel through the engine: whole prompts, portions, token by token, mixed batches, reused blocks and
+state slots, long decoding, greedy generation — against the plain NumPy form of the whole model."""
+import json
+import subprocess
+import sys
+from pathlib import Path
+
+import numpy as np
+import pytest
+
+from oracle import muzopel_ref as R
+from tests.test_gpu_biberax import LIMIT, check, errors, feed, greedy_margin, load
+
+pytestmark = pytest.mark.gpu
+ROOT = Path(__file__).resolve().parent.parent
+
+
+def moe(experts, identity, top, ff):
+    return {"kind": "moe", "expert": dict(ff=ff), "router": dict(experts=experts, identity=identity, top=top)}
+
+
+def latent(heads, dim, rot_dim, vdim, rank, scale, base, mlp, q_rank=None, scaling=None):
+    """With q_rank: queries out of a latent, gated heads."""
+    rot = dict(base=base, dims=rot_dim)
+    if scaling:
+        rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    m = dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=rank, scale=scale, rot=rot)
+    if q_rank:
+        m["q_rank"] = q_rank
+    return {"type": "latent_attention" if q_rank else "latent_attention_2", "mlp": mlp, "mixer": m}
+
+
+def model(width, parts, taps, vocab, layers, cap=20.0, eps=1e-5):
+    return {"architecture": "Muzopel", "width": width, "vocab": vocab, "norm": {"eps": eps, "groups": parts}, "canon": {"taps": taps},
+            "logit_softcap": cap, "layers": layers}
+
+
+YARN = (8.0, 96, 12.0, 1.0)
+
+CONFIGS = {
+    "narrow": model(72, 3, 3, 61, [latent(4, 24, 8, 40, 40, 0.25, 1e3, moe(6, 2, 2, 40)),
+                                   latent(3, 16, 8, 24, 48, 0.3, 50.0, None, 24, YARN),
+                                   latent(5, 8, 16, 8, 24, 0.4, 1e2, moe(4, 4, 3, 24), 40)], 12.0),
+    # sizes that are multiples of nothing
+    "odd": model(75, 5, 2, 63, [latent(5, 9, 6, 7, 11, 0.3, 50.0, moe(9, 3, 2, 11), 13, (3.0, 40, 7.0, 2.0)),
+                                latent(3, 7, 2, 5, 19, 0.4, 9.0, moe(7, 1, 1, 20)),
+                                latent(2, 9, 4, 15, 21, 0.4, 30.0, None)], 7.5, 1e-3),
+    "one": model(64, 1, 1, 48, [latent(1, 8, 2, 8, 8, 0.5, 10.0, moe(1, 0, 1, 16)),
+                                latent(1, 16, 2, 8, 16, 0.5, 10.0, moe(1, 1, 1, 8), 1)], 50.0),
+    "wide": model(128, 2, 4, 200, [latent(8, 64, 32, 64, 256, 0.06, 1e4, moe(12, 4, 3, 24), 96, (4.0, 64, 20.0, 2.0)),
+                                   latent(16, 32, 64, 128, 512, 0.08, 1e4, moe(16, 16, 5, 40)),
+                                   latent(8, 128, 64, 128, 192, 0.05, 2e3, moe(3, 2, 2, 264), 64)], 30.0, 1e-6),
+    # plans whose last K chunk and last feature tile are ragged
+    "broad": model(520, 4, 5, 1001, [latent(6, 48, 16, 40, 320, 0.1, 2e4, moe(9, 3, 3, 296), 200),
+                                     latent(10, 40, 24, 72, 136, 0.1, 2e4, moe(4, 0, 2, 1100))], 9.0),
+    # more heads than a tile or a row's CTA takes
+    "many": model(72, 12, 6, 56, [latent(70, 8, 8, 8, 24, 0.4, 80.0, moe(40, 24, 6, 16), 56, (2.0, 32, 5.0, 1.0)),
+                                  latent(34, 8, 4, 16, 160, 0.4, 50.0, moe(10, 2, 9, 24))], 15.0),
+}
+
+
+@pytest.fixture(scope="module")
+def models(tmp_path_factory):
+    out = {}
+    for i, (name, config) in enumerate(CONFIGS.items()):
+        w = R.steady_routers(config, R.random_weights(config, seed=70 + i))
+        path = tmp_path_factory.mktemp("muzopel_" + name)
+        R.write_model(str(path), config, w)
+        out[name] = (config, w, str(path))
+    return out
+
+
+_clear = {}
+
+
+def prompt(models, name, n, seed):
+    """Random tokens whose experts hang on no close call: a choice that rounding turns over would be felt
+    by all later tokens."""
+    if name not in _clear:
+        config, w, _ = models[name]
+        margins = []
+        for t in range(config["vocab"]):
+            own = []
+            R.forward(config, w, [t], margins_out=own)
+            margins.append(min((float(m[0]) for m in own), default=np.inf))
+        _clear[name] = np.flatnonzero(np.array(margins) > 0.06)
+        assert len(_clear[name]) >= 12, name
+    return np.random.default_rng(seed).choice(_clear[name], n)
+
+
+_expected = {}
+
+
+def expected(models, name, tokens):
+    """(logits, least router margin of every position over the layers)"""
+    key = (name, tuple(int(t) for t in tokens))
+    if key not in _expected:
+        margins = []
+        logits = R.forward(models[name][0], models[name][1], tokens, margins_out=margins)
+        _expected[key] = logits, np.min(margins, axis=0) if margins else np.full(len(tokens), np.inf)
+    return _expected[key]
+
+
+@pytest.mark.parametrize("dtype", ["f32", "bf16"])
+@pytest.mark.parametrize("name", CONFIGS)
+def test_whole_prompt(hb, cuda, models, name, dtype):
+    eng = load(hb, models[name][2], dtype)
+    assert eng.num_layers() == len(models[name][0]["layers"]) and eng.hidden_size() == models[name][0]["width"]
+    assert eng.param_count() == sum(v.size for v in models[name][1].values())
+    for n in (1, 2, 17, 301):
+        toks = prompt(models, name, n, n)
+        seq = eng.create_kv_cache()
+        check(feed(eng, seq, toks, [n]), expected(models, name, toks), dtype, n)
+        assert len(seq) == n
+        seq.free()
+    eng.close()
+
+
+@pytest.mark.parametrize("dtype", ["f32", "bf16"])
+@pytest.mark.parametrize("name", CONFIGS)
+def test_portions_and_single_tokens(hb, cuda, models, name, dtype):
+    """The same prompt in portions of many sizes, and token by token: prefill against decoding."""
+    eng = load(hb, models[name][2], dtype)
+    toks = prompt(models, name, 210, 3)
+    want = expected(models, name, toks)
+    for sizes in ([2], [3, 61], [16], [64, 1, 2], [9, 130], [1]):
+        seq = eng.create_kv_cache()
+        check(feed(eng, seq, toks, sizes), want, dtype, sizes)
+        seq.free()
+    eng.close()
+
+
+@pytest.mark.parametrize("seed", [1, 2])
+def test_routers_that_read_everything(hb, cuda, tmp_path, seed):
+    """Weights as they are drawn, in 32-bit: experts that depend on what came before."""
+    for name in ("narrow", "odd", "many"):
+        config = CONFIGS[name]
+        w = R.random_weights(config, seed=200 + seed)
+        R.write_model(str(tmp_path), config, w)
+        eng = load(hb, str(tmp_path), "f32")
+        toks, margins = np.random.default_rng(seed).integers(0, config["vocab"], 90), []
+        want = R.forward(config, w, toks, margins_out=margins)
+        assert np.min(margins) > 1e-4
+        for sizes in ([90], [2, 7], [1]):
+            seq = eng.create_kv_cache()
+            check(feed(eng, seq, toks, sizes), want, "f32", (name, sizes))
+            seq.free()
+        eng.close()
+
+
+@pytest.mark.parametrize("dtype", ["f32", "bf16"])
+def test_long_decoding(hb, cuda, models, dtype):
+    eng = load(hb, models["narrow"][2], dtype)
+    toks = prompt(models, "narrow", 480, 8)
+    want = expected(models, "narrow", toks)
+    seq = eng.create_kv_cache()
+    check(feed(eng, seq, toks[:30], [30]), want, dtype, rows=slice(0, 30))
+    logits = np.empty((1, 61), dtype=np.float32)
+    rows = []
+    for t in toks[30:]:
+        nxt = eng.decode_batch([seq], [t], logits=logits)
+        assert nxt[0] == np.argmax(logits[0])
+        rows.append(logits[0].copy())
+    check(np.stack(rows), want, dtype, rows=slice(30, None))
+    eng.close()
+
+
+@pytest.mark.parametrize("dtype", ["f32", "bf16"])
+@pytest.mark.parametrize("name", ["narrow", "wide", "odd", "many"])
+def test_mixed_batches_and_reuse(hb, cuda, models, name, dtype):
+    """Unequal requests come and go: portions beside single tokens, some left out of a step, pool and
+    slots just large enough, so that later requests get what earlier ones held."""
+    rng = np.random.default_rng(11)
+    lengths = [150, 5, 33, 97, 64, 16, 201, 2, 120, 80]
+    reqs = [prompt(models, name, n, 100 + i) for i, n in enumerate(lengths)]
+    live_cap, blocks = 4, 40
+    eng = load(hb, models[name][2], dtype, tokens=blocks * 16, max_seqs=live_cap)
+    waiting, live, got = list(range(len(reqs))), {}, {i: [] for i in range(len(reqs))}
+    held = lambda: sum(-(-len(reqs[i]) // 16) for i in live)
+    while waiting or live:
+        while waiting and len(live) < live_cap and held() + -(-len(reqs[waiting[0]]) // 16) <= blocks:
+            i = waiting.pop(0)
+            live[i] = [eng.create_kv_cache(), 0]
+        entries, plan = [], []
+        for i, (seq, at) in live.items():
+            if len(live) > 1 and rng.random() < 0.2:
+                continue
+            n = int(min(len(reqs[i]) - at, rng.choice([1, 1, 1, 2, 3, 15, 16, 31, 70, 128])))
+            entries.append((seq, reqs[i][at:at + n], range(n)))
+            plan.append((i, n))
+        if not entries:
+            continue
+        logits = eng.step(entries)[1]
+        at = 0
+        for i, n in plan:
+            got[i].append(logits[at:at + n])
+            at += n
+            live[i][1] += n
+            if live[i][1] == len(reqs[i]):
+                live.pop(i)[0].free()
+    for i, toks in enumerate(reqs):
+        check(np.concatenate(got[i]), expected(models, name, toks), dtype, i)
+    assert eng.num_free_blocks() == blocks
+    assert sum(-(-n // 16) for n in lengths) > blocks  # something was used twice
+    assert eng.num_free_state_slots() == live_cap
+    eng.close()
+
+
+@pytest.mark.parametrize("dtype", ["f32", "bf16"])
+@pytest.mark.parametrize("name", ["wide", "many"])
+def test_batch_against_each_alone(hb, cuda, models, name, dtype):
+    """Decoding a batch of unequal contexts gives what each gives alone."""
+    eng = load(hb, models[name][2], dtype, tokens=2048)
+    reqs = [prompt(models, name, n, 40 + n) for n in (3, 70, 71, 130, 220)]
+    seqs = [eng.create_kv_cache() for _ in reqs]
+    for s, r in zip(seqs, reqs):
+        eng.step([(s, r[:-2], [])])
+    logits = np.empty((len(reqs), models[name][0]["vocab"]), dtype=np.float32)
+    for k in (-2, -1):
+        eng.decode_batch(seqs, [r[k] for r in reqs], logits=logits)
+        for i, r in enumerate(reqs):
+            check(logits[i:i + 1], expected(models, name, r), dtype, (k, i), rows=slice(len(r) + k, len(r) + k + 1))
+    eng.close()
+
+
+def test_a_wide_batch_of_decoded_tokens(hb, cuda, models):
+    name = "narrow"
+    eng = load(hb, models[name][2], "f32", tokens=8192, max_seqs=150)
+    base = prompt(models, name, 60, 77)
+    want = expected(models, name, base)
+    lens = [3 + i % 50 for i in range(150)]
+    seqs = [eng.create_kv_cache() for _ in lens]
+    for s, n in zip(seqs, lens):
+        eng.step([(s, base[:n], [])])
+    logits = np.empty((150, 61), dtype=np.float32)
+    eng.decode_batch(seqs, [base[n] for n in lens], logits=logits)
+    assert errors(logits, want[0][lens]).max() < LIMIT["f32"]
+    eng.close()
+
+
+def strong_key(config, seed, token, gain, strength):
+    """Layer 0 with one latent channel that only `token` fills and every query asks for: column 0 of the
+    embedding drives the queries' channel, column 1 (set for that token alone) the latent's."""
+    w = R.random_weights(config, seed=seed)
+    m = config["layers"][0]["mixer"]
+    D, QD = m["dim"], m["dim"] + m["rot_dim"]
+    w["embed"][:, 0], w["embed"][:, 1], w["embed"][token, 1] = 4.0, 0.0, 40.0
+    w["embed.norm"][:2] = 1.0
+    w["l0.canon1"][:2] = 0.0
+    p = "l0.mix."
+    w[p + "dkv"][3, :] = 0.0
+    w[p + "dkv"][3, 1] = gain
+    w[p + "dkv.norm"][3] = 1.0
+    w[p + "uk"][:, 3] = 0.0
+    if "q_rank" in m:
+        w[p + "dq"][2, :] = 0.0
+        w[p + "dq"][2, 0] = 2.0
+        w[p + "uq"][:, 2] = 0.0
+    for h in range(m["heads"]):
+        w[p + "uk"][h * D + D - 1, :] = 0.0
+        w[p + "uk"][h * D + D - 1, 3] = 1.0
+        name = p + ("uq" if "q_rank" in m else "q")
+        w[name][h * QD + D - 1, :] = 0.0
+        w[name][h * QD + D - 1, 2 if "q_rank" in m else 0] = strength
+    return w
+
+
+@pytest.mark.parametrize("q_rank", [None, 24])
+@pytest.mark.parametrize("dtype", ["f32", "bf16"])
+def test_a_standing_out_far_key(hb, cuda, tmp_path, q_rank, dtype):
+    """A single strong key hundreds of positions away, met through the latent; at the ends of blocks, in
+    prompts and in decoding."""
+    config = model(64, 4, 3, 40, [latent(4, 16, 8, 16, 24, 1.0, 100.0, None, q_rank, YARN if q_rank else None)])
+    w = strong_key(config, 10, 7, 3.0, 1.5)
+    R.write_model(str(tmp_path), config, w)
+    eng = load(hb, str(tmp_path), dtype)
+    for at in (0, 1, 15, 16, 31, 100):
+        toks = np.random.default_rng(at).integers(8, 40, 350)
+        toks[at] = 7
+        want = R.forward(config, w, toks)
+        for sizes in ([350], [190, 2, 3], [280] + [1] * 70):
+            seq = eng.create_kv_cache()
+            check(feed(eng, seq, toks, sizes), want, dtype, (at, sizes[0]))
+            seq.free()
+    toks[100] = 8
+    assert errors(R.forward(config, w, toks), want)[280:].max() > 4 * LIMIT["bf16"]
+    eng.close()
+
+
+@pytest.mark.parametrize("taps", [2, 4, 7])
+@pytest.mark.parametrize("dtype", ["f32", "bf16"])
+def test_inputs_of_earlier_tokens_are_remembered_and_forgotten(hb, cuda, tmp_path, taps, dtype):
+    """Wide convolutions: another first token is felt by the next taps - 1 tokens however the prompt is cut,
+    and never by the sequence that takes over the slot."""
+    config = model(64, 2, taps, 40, [latent(2, 16, 4, 16, 24, 0.25, 100.0, moe(2, 1, 3, 32)), latent(2, 16, 4, 16, 24, 0.25, 100.0, None, 16)])
+    w = R.random_weights(config, seed=12)
+    for name in w:
+        if ".canon" in name:
+            w[name] *= 4.0
+    R.write_model(str(tmp_path), config, w)
+    eng = load(hb, str(tmp_path), dtype, max_seqs=1)
+    toks = np.random.default_rng(1).integers(8, 40, 60)
+    plain = toks.copy()
+    plain[0] = 7
+    want, without = R.forward(config, w, toks), R.forward(config, w, plain)
+    assert errors(without, want)[1:taps].min() > 4 * LIMIT["bf16"]
+    for sizes in ([60], [2], [1], [1, 58], [3, 1, 2], [17, 16]):
+        for t, e in ((toks, want), (plain, without)):
+            seq = eng.create_kv_cache()
+            check(feed(eng, seq, t, sizes), e, dtype, sizes[0])
+            seq.free()
+    eng.close()
+
+
+def test_steps_of_any_cut_agree_to_the_last_bits(hb, cuda, models):
+    """32-bit: the same tokens in one step, in portions and beside another request."""
+    name = "narrow"
+    eng = load(hb, models[name][2], "f32")
+    toks, other = prompt(models, name, 120, 30), prompt(models, name, 50, 31)
+    seq = eng.create_kv_cache()
+    whole = feed(eng, seq, toks, [120])
+    seq.free()
+    a, b = eng.create_kv_cache(), eng.create_kv_cache()
+    eng.step([(b, other[:20], [])])
+    got, at, at_b = [], 0, 20
+    for n, m in ((33, 1), (2, 1), (1, 9), (40, 1), (44, 0)):
+        entries = [(a, toks[at:at + n], range(n))] + ([(b, other[at_b:at_b + m], [])] if m else [])
+        got.append(eng.step(entries)[1])
+        at, at_b = at + n, at_b + m
+    assert np.abs(np.concatenate(got) - whole).max() < 1e-4
+    eng.close()
+
+
+def test_greedy_generation_through_the_scheduler(hb, cuda, models):
+    from vllm_hb_b200 import serve
+
+    name = "narrow"
+    config, w, path = models[name]
+    prompts = [prompt(models, name, n, 60 + n).tolist() for n in (5, 40, 1, 23, 90, 17)]
+    want = [R.greedy_generate(config, w, p, 12) for p in prompts]
+    eng = load(hb, path, "f32", tokens=400, max_seqs=3)
+    got = serve.generate(eng, prompts, 12, max_live=3, step_tokens=24)
+    for g, (toks, rows), p in zip(got, want, prompts):
+        clear = greedy_margin(rows) > 1e-3
+        first_unclear = len(clear) if clear.all() else int(np.argmin(clear))
+        assert g[:first_unclear] == toks[:first_unclear], len(p)
+    assert eng.num_free_blocks() == 25
+    one = serve.generate(eng, prompts[:1], 10, max_live=3, temperature=0.8, top_p=0.9, seed=4)
+    many = serve.generate(eng, prompts, 10, max_live=3, temperature=0.8, top_p=0.9, seed=4)
+    assert one[0] == many[0] and max(max(o) for o in many) < config["vocab"]
+    eng.close()
+
+
+def test_generate_and_replay_commands(hb, cuda, models, tmp_path):
+    config, w, path = models["odd"]
+    p = prompt(models, "odd", 21, 5)
+    out = subprocess.run([sys.executable, str(ROOT / "bin" / "generate"), "--model", path, "--dtype", "float32", "--max-tokens",
+                          "6"], input=json.dumps(p.tolist()) + "\n", capture_output=True, text=True, timeout=120)
+    assert out.returncode == 0, out.stderr
+    toks, rows = R.greedy_generate(config, w, p.tolist(), 6)
+    if (greedy_margin(rows) > 1e-3).all():
+        assert json.loads(out.stdout) == toks
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": p[:9].tolist(), "want": [0, 8]}], "end": []},
+             {"step": 1, "entries": [{"id": "a", "tokens": p[9:20].tolist(), "want": []}], "end": []},
+             {"step": 2, "entries": [{"id": "a", "tokens": p[20:].tolist(), "want": [0]}], "end": ["a"]}]
+    out = subprocess.run([str(ROOT / "bin" / "trace_run"), "--model", path, "--dtype", "float32", "--out", str(tmp_path),
+                          "--max-tokens", "64"], input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True,
+                         text=True, timeout=120)
+    assert out.returncode == 0 and out.stdout.split("\n")[:3] == ["done 0", "done 1", "done 2"], out.stderr
+    want = expected(models, "odd", p)[0]
+    check(np.fromfile(tmp_path / "0.f32", dtype="<f4").reshape(2, -1), want[[0, 8]], "f32")
+    check(np.fromfile(tmp_path / "2.f32", dtype="<f4").reshape(1, -1), want[[20]], "f32")
+    assert not (tmp_path / "1.f32").exists()
+
+
+@pytest.mark.parametrize("dtype", ["f32", "bf16"])
+def test_without_state_blocks_are_copied_and_sequences_wound_back(hb, cuda, models, dtype):
+    """A model whose convolutions have one tap keeps nothing besides its blocks."""
+    config, w, path = models["one"]
+    eng = load(hb, path, dtype, tokens=640)
+    toks = prompt(models, "one", 70, 21)
+    other = np.concatenate([toks[:40], prompt(models, "one", 30, 22)])
+    want, want2 = expected(models, "one", toks), expected(models, "one", other)
+    table = [30, 5, 17, 2, 9]
+    check(eng.forward_tables(toks[:40], 0, table)[None], want, dtype, rows=slice(39, 40))
+    eng.kv_copy_blocks([(17, 21)])
+    table2 = [30, 5, 21, 3, 4]
+    check(eng.forward_tables(toks[40:], 40, table)[None], want, dtype, rows=slice(69, 70))
+    check(eng.forward_tables(other[40:], 40, table2)[None], want2, dtype, rows=slice(69, 70))
+    seq = eng.create_kv_cache()
+    feed(eng, seq, toks[:61], [61])
+    eng.truncate(seq, 40)
+    check(feed(eng, seq, other[40:], [7]), want2, dtype, rows=slice(40, None))
+    eng.close()
+
+
+def test_refusals(hb, cuda, models, tmp_path):
+    config, w, path = models["narrow"]
+    with pytest.raises(hb.HbError, match="f16"):
+        hb.Engine.load(path, bf16=False)
+    eng = load(hb, path, "bf16")
+    with pytest.raises(hb.HbError, match="recurrent state"):
+        eng.kv_copy_blocks([(1, 2)])
+    seqs = [eng.create_kv_cache() for _ in range(7)]
+    eng.step([(s, [1, 2], []) for s in seqs[:6]])
+    with pytest.raises(hb.HbError, match="state slot"):
+        eng.step([(seqs[6], [1], [])])
+    eng.close()
+
+    def altered(layer, key="mixer", **change):
+        c = json.loads(json.dumps(config))
+        c["layers"][layer][key].update(change)
+        return c
+
+    router = lambda **k: dict(dict(experts=6, identity=2, top=2), **k)
+    cases = [(dict(config, norm={}), "eps"), (dict(config, norm=dict(eps=1e-5, groups=5)), "parts"), (dict(config, canon={}), "taps"),
+             (dict(config, canon=dict(taps=4)), "canon1"), (dict(config, width=66), "shape"), (dict(config, layers=[]), "no layers"),
+             (dict(config, layers=[dict(config["layers"][0], type="other")]), "unknown type"), (dict(config, logit_softcap=-1.0), "parts"),
+             (altered(0, heads=0), "sizes"), (altered(0, kv_rank=0), "sizes"), (altered(1, q_rank=0), "sizes"), (altered(1, q_rank=25), "dq"),
+             (altered(0, rot=dict(base=9.0, dims=10)), "rotation"), (altered(0, rot=dict(base=9.0, dims=5)), "rotation"),
+             (altered(1, rot=dict(base=10.0, dims=4, scaling=dict(factor=0))), "scaling"), (altered(0, vdim=41), "l0.mix"),
+             (altered(0, "mlp", kind="other"), "unknown kind"), (altered(0, "mlp", router=router(top=9)), "experts"),
+             (altered(0, "mlp", router=router(identity=-1)), "identit"), (altered(0, "mlp", router=router(identity=3)), "router"),
+             (altered(0, "mlp", router=router(experts=7, identity=1)), "l0.mlp.e6")]
+    for bad, text in cases:
+        R.write_model(str(tmp_path), bad, w)
+        with pytest.raises(hb.HbError, match=text):
+            load(hb, str(tmp_path), "bf16")
+    for missing in ("embed.norm", "l0.canon1", "l2.canon2", "l1.dwa", "l1.mix.dq.norm", "l1.mix.uq", "l1.mix.g", "l0.mix.dkv.norm",
+                    "l0.mlp.correction", "l0.mlp.e5.up", "l2.norm2", "final.norm", "head"):
+        R.write_model(str(tmp_path), config, {k: v for k, v in w.items() if k != missing})
+        with pytest.raises(hb.HbError, match=missing):
+            load(hb, str(tmp_path), "bf16")
+
+
+def test_random_engine_and_profile(hb, cuda):
+    eng = hb.Engine.create_random_config(CONFIGS["wide"], max_seq_len=128, max_batch=128, max_seqs=4)
+    seqs = [eng.create_kv_cache() for _ in range(4)]
+    eng.step([(s, np.arange(20) + i, []) for i, s in enumerate(seqs)])
+    nxt, ms = eng.profile_step(seqs, np.arange(4))
+    assert len(nxt) == 4
+    assert min(ms[k] for k in ("routing", "experts_gate_up", "experts_down", "attention", "gemm", "latent", "norm")) > 0
+    assert eng.step_bytes([20] * 4) > 0 and eng.gemm_bytes(4) > 0 and eng.last_step_launches() > 10
+    eng.close()
