@@ -612,10 +612,10 @@ def main() -> None:
     ap.add_argument("--skip-checks", action="store_true",
                     help="N > 1: skip the untimed parity checks, the single-GPU base point and the row-parallel points")
     ap.add_argument("--tp1-layers", type=int, default=8, help="layers of the single-GPU base point of the N > 1 shape")
-    ap.add_argument("--workload", default="auto", choices=["auto", "mixtral", "latarax", "biberax", "badolix"],
+    ap.add_argument("--workload", default="auto", choices=["auto", "mixtral", "latarax", "biberax", "badolix", "muzopel"],
                     help="auto: Llama-3.1-8B shape on one GPU, 70B shape on several; mixtral: Mixtral-8x7B shape; "
-                         "latarax, biberax, badolix: that design beside the Llama family at equal size, one GPU")
-    ap.add_argument("--size", default="", help="latarax, biberax, badolix: only the sizes whose name contains this text")
+                         "latarax, biberax, badolix, muzopel: that design beside the Llama family at equal size, one GPU")
+    ap.add_argument("--size", default="", help="latarax, biberax, badolix, muzopel: only the sizes whose name contains this text")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
@@ -628,7 +628,7 @@ def main() -> None:
         if args.gpus != 1 or world != 1:
             raise SystemExit(f"--gpus {args.gpus} needs torchrun with {args.gpus} ranks (WORLD_SIZE={world})")
     args.warmup = max(args.warmup, 3)
-    if args.workload in ("latarax", "biberax", "badolix"):
+    if args.workload in ("latarax", "biberax", "badolix", "muzopel"):
         run_layered(args)
         return
     run_gpu_arm(args, rank, world, local_rank)

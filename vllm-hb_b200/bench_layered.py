@@ -1,7 +1,7 @@
 """Models described layer by layer beside the Llama family (and, for a mixture of experts, its
 Mixtral form) at equal width, feed-forward, depth and vocabulary.
 
-`python bench.py --workload latarax`, `biberax` or `badolix` runs it on one GPU: prefill of one long prompt and
+`python bench.py --workload latarax`, `biberax`, `badolix` or `muzopel` runs it on one GPU: prefill of one long prompt and
 of several shorter ones, decode at several batch sizes, random weights and tokens.  For every kind of
 kernel it reports the time of a profiled step and the fraction of the roofline (the larger of bytes /
 measured HBM bandwidth and FLOPs / measured bf16 throughput, over the time).
@@ -55,8 +55,33 @@ def badolix_layers(heads, window, keep, dense_ff, experts, top, ff, layers):
     return out
 
 
+def muzopel_layers(heads, q_rank, experts, identity, top, ff, layers):
+    """Latent attention with queries from a latent and gated heads, and without, in turn; experts without
+    gates in every layer."""
+    latent = dict(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5)
+    rot = dict(base=10000.0, dims=64)
+    yarn = dict(rot, scaling=dict(factor=4.0, original=4096, fast=32.0, slow=1.0))
+    mixers = [("latent_attention", dict(latent, q_rank=q_rank, rot=yarn)), ("latent_attention_2", dict(latent, rot=rot))]
+    moe = {"kind": "moe", "expert": dict(ff=ff), "router": dict(experts=experts, identity=identity, top=top)}
+    return [{"type": mixers[i % 2][0], "mixer": mixers[i % 2][1], "mlp": moe} for i in range(layers)]
+
+
 def sizes(design: str) -> list[dict]:
     """Layers of about 1.3B- and 8B-parameter models (dense ones; a mixture has more)."""
+    if design == "muzopel":  # beside Badolix with the same latent attention and (gated) experts in every layer
+        out = []
+        for small in sizes("badolix"):
+            llama, bad = small["llama"], small["badolix"]
+            width, layers = llama["hidden_size"], llama["num_hidden_layers"]
+            mixer, f = bad["layers"][0]["mixer"], bad["layers"][1]["mlp"]
+            experts, top, ff = f["router"]["experts"], f["router"]["top"], f["expert"]["ff"]
+            out.append({"name": small["name"],
+                        "muzopel": {"architecture": "Muzopel", "width": width, "vocab": VOCAB, "norm": {"eps": 1e-6, "groups": 4},
+                                    "canon": {"taps": 4}, "logit_softcap": 30.0,
+                                    "layers": muzopel_layers(width // 128, 3 * width // 8, experts, experts // 4, top, ff, layers)},
+                        "badolix": dict(bad, layers=[{"type": "latent_attention", "mixer": mixer, "mlp": f}] * layers),
+                        "llama": llama})
+        return out
     if design == "badolix":  # beside the designs its kernels are shared with or like
         out = []
         for small, other in zip(sizes("biberax"), sizes("latarax")):
@@ -124,7 +149,12 @@ def work(shape: dict, family: str, positions: list[np.ndarray], wanted: int) -> 
 
     def latent(m, H):
         h, d, r, v, c = (m[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank"))
-        gemm("gemm_qkv", h * (d + r) + c + r, H)
+        if m.get("q_rank"):
+            gemm("gemm_qkv", m["q_rank"] + c + r + h, H)
+            add("norm", 4.0 * rows * m["q_rank"])
+            gemm("gemm_qkv", h * (d + r), m["q_rank"])
+        else:
+            gemm("gemm_qkv", h * (d + r) + c + r, H)
         add("rope_kv", 4.0 * rows * (h * r + c + r))
         for p in positions:
             n, span, seen = len(p), float(p[-1] + 1), keys_seen(p, 0, 0)
@@ -222,6 +252,28 @@ def work(shape: dict, family: str, positions: list[np.ndarray], wanted: int) -> 
                 add("experts_gate_up", 4.0 * active * F * H + 2.0 * picks * (H + F), 4.0 * picks * F * H)
                 add("experts_down", 2.0 * active * F * H + 2.0 * picks * (H + F), 2.0 * picks * F * H)
                 add("norm", (2.0 * picks - 2.0 * rows) * H)
+        add("norm", wanted * H * 6.0)
+        gemm("gemm_lm_head", shape["vocab"], H, m=wanted, out=4)
+        return w
+    if family == "muzopel":
+        H, held = shape["width"], shape["canon"]["taps"] - 1
+        # a boundary: output, residual in and out, next input, inputs of earlier tokens
+        past = sum(held + min(len(p), held) for p in positions)
+        add("norm", rows * H * (2.0 + 4.0 + 2.0) + 4.0 * held * H * len(positions))  # the embedding
+        for i, layer in enumerate(shape["layers"]):
+            f = layer["mlp"]
+            latent(layer["mixer"], H)
+            add("norm", rows * H * 14.0 + 4.0 * past * H)
+            E, top, F = f["router"]["experts"], f["router"]["top"], f["expert"]["ff"]
+            O = E + f["router"]["identity"]
+            picks = rows * top * E / O
+            active = E * (1.0 - (1.0 - top / O) ** rows)
+            add("routing", 2.0 * O * H + 2.0 * rows * H + 2.0 * (rows + picks) * H)
+            add("experts_gate_up", 2.0 * active * F * H + 2.0 * picks * (H + F), 2.0 * picks * F * H)
+            add("experts_down", 2.0 * active * F * H + 2.0 * picks * (H + F), 2.0 * picks * F * H)
+            # the weighted outputs in place of a product's rows, and the sum over depth
+            add("norm", 2.0 * (picks + (rows if picks < rows * top else 0)) * H + rows * H * 10.0 + 4.0 * past * H)
+            add("norm", rows * H * 4.0 * (i + 2))
         add("norm", wanted * H * 6.0)
         gemm("gemm_lm_head", shape["vocab"], H, m=wanted, out=4)
         return w
@@ -329,7 +381,7 @@ def run(hb, hbm_gbs: float, tflops: float, steps: int, warmup: int, design: str 
         if only and only not in size["name"]:
             continue
         entry = report[size["name"]] = {}
-        for family in [design] + [f for f in ("biberax", "latarax", "llama", "mixtral") if f != design]:
+        for family in [design] + [f for f in ("badolix", "biberax", "latarax", "llama", "mixtral") if f != design]:
             shape = size.get(family)
             if not shape:
                 continue
