@@ -160,14 +160,48 @@ __device__ __forceinline__ void push_tile(const TcParams& p, const uint8_t* stag
     peer_st_release(&reinterpret_cast<CommFlags*>(p.push_peer[q])->tflag[(row_block * R + me) * T + ti], seq + 1);
 }
 
+// Standard normal distribution function by formula 7.1.26 of Abramowitz and Stegun, Handbook of
+// Mathematical Functions, for erfc (within 1.5e-7 of the exact value), without branches.
+__device__ __forceinline__ float normal_cdf(float g) {
+  const float a = fabsf(g) * 0.70710678f;
+  const float t = __fdividef(1.f, fmaf(0.3275911f, a, 1.f));
+  float p = fmaf(1.061405429f, t, -1.453152027f);
+  p = fmaf(p, t, 1.421413741f);
+  p = fmaf(p, t, -0.284496736f);
+  p = fmaf(p, t, 0.254829592f);
+  const float half_erfc = 0.5f * p * t * __expf(-a * a);
+  return g < 0.f ? half_erfc : 1.f - half_erfc;
+}
+
+// An activation without a gate, on 16 outputs: the form is looked up once.
+__device__ __forceinline__ void single_16(float (&v)[16], const GatedAct& act) {
+  if (act.form == GatedAct::kErf) {
+#pragma unroll
+    for (int j = 0; j < 16; ++j) {
+      const float g = fminf(v[j], act.limit);
+      v[j] = g * normal_cdf(g);
+    }
+  } else if (act.form == GatedAct::kTanh) {
+    const float k = __fdividef(2.f, act.limit);
+#pragma unroll
+    for (int j = 0; j < 16; ++j)  // tanh(y) = 1 - 2 / (1 + e^2y)
+      v[j] = act.limit - __fdividef(2.f * act.limit, 1.f + __expf(fminf(v[j] * k, 80.f)));
+  } else {
+#pragma unroll
+    for (int j = 0; j < 16; ++j) {
+      const float g = fminf(v[j], act.limit), z = act.slope * fmaf(act.cubic * g * g, g, g);
+      v[j] = z < -80.f ? 0.f : __fdividef(g, 1.f + __expf(-z));
+    }
+  }
+}
+
 // Gated activation of one output element (fast divide and exponential, as silu_f).
 template <bool GENERAL>
 __device__ __forceinline__ float gated_f(float g, float u, const GatedAct& act) {
   if (!GENERAL) return silu_f(g) * u;
-  if (act.form == GatedAct::kTanh) return act.limit * tanhf(g / act.limit);
   g = fminf(g, act.limit);
   u = fminf(fmaxf(u, -act.limit), act.limit);
-  if (act.form == GatedAct::kErf) return g * normcdff(g) * (u + act.shift);
+  if (act.form == GatedAct::kErf) return g * normal_cdf(g) * (u + act.shift);
   const float z = act.slope * fmaf(act.cubic * g * g, g, g);
   // far below zero the gate is zero (the fast divide wants a denominator below 2^126)
   return z < -80.f ? 0.f : __fdividef(g, 1.f + __expf(-z)) * (u + act.shift);
@@ -453,7 +487,6 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
     if (p.gate_bias) gate_b = __ldg(p.gate_bias + n_glob);
     if (p.up_bias) up_b = __ldg(p.up_bias + n_glob);
   }
-  auto alone = [&](float g) { return gated_f<GENERAL>(g, 1.f - act.shift, act); };
   auto gated = [&](float g, float u) { return BIAS ? gated_f<GENERAL>(g + gate_b, u + up_b, act) : gated_f<GENERAL>(g, u, act); };
 
   // Output tiles are staged in the (now idle) pipeline buffers as [batch row][128
@@ -573,7 +606,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           }
         }
 #pragma unroll
-        for (int j = 0; j < 16; ++j) g[j] = swiglu ? gated(g[j], u[j]) : single ? alone(g[j]) : g[j];
+        for (int j = 0; j < 16; ++j) g[j] = swiglu ? gated(g[j], u[j]) : g[j];
+        if (single) single_16(g, act);
         if (p.post_scale) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) g[j] *= s_pscale[c0 + j];
@@ -723,10 +757,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
 #pragma unroll
           for (int j = 0; j < 16; ++j) v[j] = gated(v[j], u[j]);
         }
-        if (single) {
-#pragma unroll
-          for (int j = 0; j < 16; ++j) v[j] = alone(v[j]);
-        }
+        if (single) single_16(v, act);
         if (p.post_scale) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) v[j] *= s_pscale[g * 16 + j];
@@ -767,10 +798,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
 #pragma unroll
           for (int j = 0; j < 16; ++j) v[j] = gated(v[j], u[j]);
         }
-        if (single) {
-#pragma unroll
-          for (int j = 0; j < 16; ++j) v[j] = alone(v[j]);
-        }
+        if (single) single_16(v, act);
         if (n_glob < p.N) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
@@ -809,9 +837,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
         // eight batch rows at a time: 8 (16 with SwiGLU) independent loads are in
         // flight per split instead of one dependent chain per row
         for (int m0 = 0; m0 < m_lim; m0 += 8) {
-          float g[8], u[8];
+          float g[16], u[8];  // (eight rows; room for single_16)
 #pragma unroll
-          for (int j = 0; j < 8; ++j) g[j] = u[j] = 0.f;
+          for (int j = 0; j < 8; ++j) g[j] = g[j + 8] = u[j] = 0.f;
           for (int s = 0; s < p.splits; ++s) {
             const float* ps = base + s * sstride + row;
 #pragma unroll
@@ -822,11 +850,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
               }
             }
           }
+          if (single) single_16(g, act);
 #pragma unroll
           for (int j = 0; j < 8; ++j) {
             const int m = m0 + j;
             if (m < m_lim && n_glob < p.N) {
-              const float r = swiglu ? gated(g[j], u[j]) : single ? alone(g[j]) : g[j];
+              const float r = swiglu ? gated(g[j], u[j]) : g[j];
               if (p.out_f32) ((float*)p.Y)[(int64_t)(m_base + m) * p.ldy + n_glob] = r;
               else ((__nv_bfloat16*)p.Y)[(int64_t)(m_base + m) * p.ldy + n_glob] = __float2bfloat16_rn(r);
             }
@@ -1025,9 +1054,10 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
   const int acc_cols = pl.m_pad * n_acc;
   pl.tmem_cols = acc_cols <= 32 ? 32 : acc_cols <= 64 ? 64 : acc_cols <= 128 ? 128 : acc_cols <= 256 ? 256 : 512;
   const size_t stage = (size_t)kTileN * kTileK * 2 * n_acc + (size_t)pl.m_pad * kTileK * 2;
-  // Two pipeline depths: ~110 KB, so that two CTAs share an SM and one's epilogue hides under
+  // Two pipeline depths: ~109 KB, so that two CTAs share an SM and one's epilogue hides under
   // the other's loads, or ~200 KB with the SM to itself.
-  const size_t small_budget = 110 * 1024, big_budget = 200 * 1024;
+  // (110 KB beside the static part would be a few hundred bytes too much for two)
+  const size_t small_budget = 109 * 1024, big_budget = 200 * 1024;
   auto stages_for = [&](size_t budget) { return (int)std::max<size_t>(2, std::min<size_t>(kMaxStages, budget / stage)); };
   const int small_stages = stages_for(small_budget);
   const int big_stages = (size_t)stages_for(big_budget) * stage + 1024 <= di.smem_optin ? stages_for(big_budget) : small_stages;
@@ -1040,7 +1070,7 @@ int gemm_tc_plan(TcGemmPlan* plan, const void* X, const void* W, int64_t M, int6
   } else if (!want_cluster) {
     pl.splits = pick_splits(units, k_chunks, slots);
   } else if (tuned && n_acc == 2 && units <= di.sm_count) {
-    // SwiGLU tiles carry two weight slabs per stage: the 110 KB budget holds two stages, too
+    // SwiGLU tiles carry two weight slabs per stage: the 109 KB budget holds two stages, too
     // shallow to keep HBM busy.  One CTA per SM with the deep pipeline, and the largest split
     // that still fits one wave (measured: 14336 x 8192 at M = 128 68.6 -> 51.0 us)
     int sp = 1;
