@@ -379,8 +379,9 @@ constexpr int kExpandTokens = 32;
 constexpr size_t kExpandBytes = (size_t)512 << 20;
 // Decoded tokens: with fewer (row, kv head) units than this the keys may be split over several CTAs.
 constexpr int kSplitUnits = 592;
-// Most tokens of a run of the residual kernel: long runs repeat less, short ones fill the SMs.
-static int residual_run(int rows) { return rows <= 256 ? 4 : rows <= 1024 ? 8 : 16; }
+// Most tokens of a run of the residual kernels: long runs repeat less, short ones fill the SMs.
+static int residual_run(int rows) { return rows <= 256 ? 4 : kResidualRun; }
+constexpr int kResidualTwo = 256;  // more rows than this: the residual in two kernels
 
 static SpanAttention span_args(const hb_engine* e, size_t i, const LayeredStep& s) {
   const LayeredModel* m = e->lm.get();
@@ -674,6 +675,7 @@ static int layered_alloc_runtime(hb_engine* e, const hb_model_config* cfg) {
     }
     if ((rc = dev_alloc(e, &m->h2, (size_t)R * m->Hp * es, true))) return rc;
     if ((rc = dev_alloc(e, (void**)&m->x2, (size_t)R * s.width * 4, true))) return rc;
+    if ((rc = dev_alloc(e, (void**)&m->part_scale, (size_t)R * s.norm_groups * 4, true))) return rc;
     if ((rc = dev_alloc(e, (void**)&m->results, (size_t)(s.layers.size() + 1) * R * s.width * 4, true))) return rc;
   }
   m->max_chunks = e->max_batch / kRecChunk + std::min(m->max_segs, e->max_batch / (kShortSegment + 1)) + 1;
@@ -1100,7 +1102,9 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
       r.h = h; r.ld_h = m->Hp;
     }
     read = next;
-    ++e->last_launches;
+    r.rows = rows;
+    if (rows > kResidualTwo) r.scale = m->part_scale;
+    e->last_launches += residual_in_two(r) ? 2 : 1;
     prof_mark(e, kCatNorm);
     return residual_step(st, r, runs, s.n_runs, seg, W, e->dtype);
   };

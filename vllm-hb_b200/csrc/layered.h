@@ -283,6 +283,7 @@ struct LayeredModel {
   // [layers + 1, row_cap, width]
   void* h2 = nullptr;
   float *x2 = nullptr, *results = nullptr;
+  float* part_scale = nullptr;               // [rows, norm_groups]
   void *q_latent = nullptr, *q = nullptr;    // queries out of a latent: [rows, q_rank], [rows, heads * (dim + rot_dim)]
   void* proj = nullptr;                      // [rows, max_proj]
   void *attn = nullptr, *rec = nullptr;      // branch outputs before their output projection

@@ -64,6 +64,34 @@ struct Team {
   }
 };
 
+// The sublayer's output of a row, VEC channels from c on.
+template <typename T, int VEC>
+__device__ __forceinline__ void sublayer_output(float (&f)[VEC], const ResidualStep& a, int64_t W, int64_t row, int64_t c) {
+  if (a.embed) {
+    const int64_t id = min((int64_t)a.ids[row], a.vocab - 1);  // never outside the table
+    load_row<T, VEC>(f, (const T*)a.embed + id * W + c);
+    return;
+  }
+  if (a.y) {
+    load_row<float, VEC>(f, a.y + row * a.ld_y + c);
+  } else {
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) f[j] = 0.f;
+  }
+  const int32_t* place = a.expert_place + row * a.top;
+  const float* weight = a.expert_weight + row * a.top;
+#pragma unroll 4
+  for (int k = 0; k < a.top; ++k) {
+    const int p = place[k];
+    const T* src = p < 0 ? (const T*)a.input + row * a.ld_input : (const T*)a.expert_y + (int64_t)p * a.ld_y;
+    float e[VEC];
+    load_row<T, VEC>(e, src + c);
+    const float w = weight[k];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) f[j] = fmaf(w, e[j], f[j]);
+  }
+}
+
 // NC: runs of VEC channels a thread owns.  HELD: at most kHeldTaps taps; else `win` [taps - 1][NC * VEC]
 // per thread lies in shared memory.
 template <typename T, int VEC, int NC, bool HELD>
@@ -84,32 +112,7 @@ residual_kernel(const ResidualStep a, const RowRange* __restrict__ tiles, const 
   auto chan = [&](int k) { return (team.rank + k * team.size) * VEC; };  // of the part
   auto live = [&](int k) { return member && chan(k) < size; };
 
-  // the sublayer's output of a row
-  auto output = [&](float (&f)[VEC], int64_t row, int64_t c) {
-    if (a.embed) {
-      const int64_t id = min((int64_t)a.ids[row], a.vocab - 1);  // never outside the table
-      load_row<T, VEC>(f, (const T*)a.embed + id * W + c);
-      return;
-    }
-    if (a.y) {
-      load_row<float, VEC>(f, a.y + row * a.ld_y + c);
-    } else {
-#pragma unroll
-      for (int j = 0; j < VEC; ++j) f[j] = 0.f;
-    }
-    const int32_t* place = a.expert_place + row * a.top;
-    const float* weight = a.expert_weight + row * a.top;
-#pragma unroll 4
-    for (int k = 0; k < a.top; ++k) {
-      const int p = place[k];
-      const T* src = p < 0 ? (const T*)a.input + row * a.ld_input : (const T*)a.expert_y + (int64_t)p * a.ld_y;
-      float e[VEC];
-      load_row<T, VEC>(e, src + c);
-      const float w = weight[k];
-#pragma unroll
-      for (int j = 0; j < VEC; ++j) f[j] = fmaf(w, e[j], f[j]);
-    }
-  };
+  auto output = [&](float (&f)[VEC], int64_t row, int64_t c) { sublayer_output<T, VEC>(f, a, W, row, c); };
 
   const int i0 = max(-first, -back);
   float win[HELD ? kHeldTaps - 1 : 1][NC][VEC];  // inputs of the tokens ahead of i0, oldest first
@@ -241,6 +244,128 @@ residual_kernel(const ResidualStep a, const RowRange* __restrict__ tiles, const 
   }
 }
 
+// The same in two kernels, for many rows: the factors of all parts of all rows first; then a thread takes
+// four channels of a run and all of the run's rows at once, with nothing to wait for but its loads.
+template <typename T>
+__global__ void __launch_bounds__(kResidualThreads)
+residual_scale_kernel(const ResidualStep a, int64_t W, int team_size) {
+  __shared__ float red[kResidualThreads / 32];
+  pdl_trigger();
+  pdl_grid_wait();
+  const Team team(team_size);
+  const int size = (int)(W / a.groups), group = blockIdx.y * (blockDim.x / team_size) + threadIdx.x / team_size;
+  const int64_t row = blockIdx.x;
+  float ss = 0.f;
+  if (group < a.groups)
+    for (int i = team.rank * 4; i < size; i += team.size * 4) {
+      float f[4];
+      sublayer_output<T, 4>(f, a, W, row, (int64_t)group * size + i);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) ss = fmaf(f[j], f[j], ss);
+    }
+  const float r = 1.f / sqrtf(team.sum(ss, red) / (float)size + a.eps);
+  if (group < a.groups && team.rank == 0) a.scale[row * a.groups + group] = r;
+}
+
+constexpr int kRunThreads = 128;
+template <typename T>
+__global__ void __launch_bounds__(kRunThreads)
+residual_run_kernel(const ResidualStep a, const RowRange* __restrict__ tiles, const SegInfo* __restrict__ segs, int64_t W) {
+  constexpr int H = kHeldTaps - 1, N = H + kResidualRun;  // rows ahead of the run, all rows
+  pdl_trigger();
+  pdl_grid_wait();
+  const int64_t c = ((int64_t)blockIdx.y * kRunThreads + threadIdx.x) * 4;
+  if (c >= W) return;
+  const RowRange tile = tiles[blockIdx.x];
+  const SegInfo seg = segs[tile.seg];
+  const int back = a.conv ? a.taps - 1 : 0, ring = a.taps - 1, first = tile.row0 - seg.row0, group = (int)(c / (W / a.groups));
+  // row i is token first + i - H of the segment: of this step, and wanted for itself or for the convolution
+  auto here = [&](int i) { return i >= H ? i - H < tile.n : H - i <= back && first + i - H >= 0; };
+  const int64_t row0 = (int64_t)tile.row0 - H;
+  float x[N][4];
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) x[i][j] = 0.f;
+    if (here(i)) sublayer_output<T, 4>(x[i], a, W, row0 + i, c);
+  }
+  float w[4];
+  load_row<float, 4>(w, a.norm + c);
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    if (!here(i)) continue;
+    const float r = a.scale[(row0 + i) * a.groups + group];
+    float f[4] = {0.f, 0.f, 0.f, 0.f};
+    if (a.x) load_row<float, 4>(f, a.x + (row0 + i) * W + c);
+    const int token = first + i - H;
+    if (a.past && ring > 0 && i >= H && token >= seg.n - ring)
+      store_row<float, 4>(a.past + ((int64_t)seg.slot * ring + ((int64_t)seg.pos0 + token) % ring) * W + c, f);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) x[i][j] = fmaf(x[i][j] * r, w[j], f[j]);
+    if (a.result && i >= H) store_row<float, 4>(a.result + (row0 + i) * W + c, x[i]);
+  }
+  if (a.depth) {
+    float s[N][4];
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) s[i][j] = 0.f;
+    const float* e = a.earlier + row0 * W + c;
+    for (int l = 0; l < a.n_earlier; ++l, e += a.step) {
+      const float d = a.depth[l];
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        if (!here(i)) continue;
+        float f[4];
+        load_row<float, 4>(f, e + i * W);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) s[i][j] = fmaf(d, f[j], s[i][j]);
+      }
+    }
+    const float d = a.depth[a.n_earlier];
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) x[i][j] = fmaf(d, x[i][j], s[i][j]);
+  }
+  if (a.x_out) {
+#pragma unroll
+    for (int i = H; i < N; ++i)
+      if (here(i)) store_row<float, 4>(a.x_out + (row0 + i) * W + c, x[i]);
+  }
+  if (!a.h) return;
+  if (a.conv) {
+    float tap[kHeldTaps][4];  // by distance
+#pragma unroll
+    for (int b = 0; b < kHeldTaps; ++b) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) tap[b][j] = 0.f;
+      if (b <= back) load_row<float, 4>(tap[b], a.conv + (int64_t)(back - b) * W + c);
+    }
+#pragma unroll
+    for (int i = 0; i < H; ++i) {  // what earlier steps left
+      const int token = first + i - H;
+      if (H - i <= back && token < 0 && seg.pos0 + token >= 0)
+        load_row<float, 4>(x[i], a.state + ((int64_t)seg.slot * ring + ((int64_t)seg.pos0 + token) % ring) * W + c);
+    }
+#pragma unroll
+    for (int i = N - 1; i >= H; --i) {  // the last row first: it is the one no other row needs any more
+      float acc[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[j] = tap[0][j] * x[i][j];
+#pragma unroll
+      for (int b = 1; b < kHeldTaps; ++b)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[j] = fmaf(tap[b][j], x[i - b][j], acc[j]);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) x[i][j] += acc[j];
+    }
+  }
+#pragma unroll
+  for (int i = H; i < N; ++i)
+    if (here(i)) store_row<T, 4>((T*)a.h + (row0 + i) * a.ld_h + c, x[i]);
+}
+
 // Rows normed in parts, wherever they lie: CTA = (row, one or several parts).
 template <typename T, typename IN, int VEC>
 __global__ void __launch_bounds__(kResidualThreads)
@@ -297,6 +422,16 @@ int residual_step(cudaStream_t st, const ResidualStep& a, const RowRange* tiles,
   const int threads = std::max(team, 128), teams = threads / team;
   const bool held = a.taps <= kHeldTaps;
   const dim3 grid((unsigned)n_tiles, (unsigned)((a.groups + teams - 1) / teams));
+  if (residual_in_two(a) && vec) {
+    auto two = [&](auto* scale, auto* run) -> int {
+      HB_CUDA_CHECK(launch_pdl(scale, dim3((unsigned)a.rows, grid.y), dim3((unsigned)threads), 0, st, a, width, team));
+      HB_CUDA_CHECK(launch_pdl(run, dim3((unsigned)n_tiles, (unsigned)((width / 4 + kRunThreads - 1) / kRunThreads)), dim3(kRunThreads), 0, st,
+                               a, tiles, segs, width));
+      return HB_OK;
+    };
+    if (dtype == HB_F32) return two(residual_scale_kernel<float>, residual_run_kernel<float>);
+    if (dtype == HB_BF16) return two(residual_scale_kernel<__nv_bfloat16>, residual_run_kernel<__nv_bfloat16>);
+  }
   auto launch = [&](auto* k, int nc) -> int {
     const size_t smem = held || !a.conv ? 0 : (size_t)(a.taps - 1) * nc * v * threads * sizeof(float);
     if (smem > 200 * 1024) return fail(HB_ERR_INVALID_ARG, "residual_step: %d taps of parts of %lld channels are not supported", a.taps, (long long)size);
