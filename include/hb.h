@@ -486,7 +486,7 @@ int hb_streams_final(void* stream, void* h, const float* x, const int32_t* want,
  * y and expert_y have rows of ld_y elements; x_out, result and h may be NULL and are not among what is read.
  * state [slots, taps-1, width]: earlier inputs of the convolution, position p at entry p mod (taps-1); past
  * (NULL: none): the same of the convolution that read x, brought up to date here.  taps <= 32.
- * With scale [rows, groups] (scratch), rows of the step and runs of at most 8 rows: the form for many rows
+ * With scale [rows, groups], mixed [rows, ld_y] (scratch, needed with experts), rows of the step and runs of at most 16 rows: the form for many rows
  * (up to four taps). */
 typedef struct hb_residual_args {
   const float* y;
@@ -515,7 +515,7 @@ typedef struct hb_residual_args {
   float* past;
   void* h;
   int64_t ld_h;
-  float* scale;
+  float *scale, *mixed;
   int64_t rows;
 } hb_residual_args;
 int hb_residual_step(void* stream, const hb_residual_args* a, const int32_t* tiles, int n_tiles, const int32_t* segments,

@@ -87,9 +87,10 @@ class Boundary:
 
         s = ints(segs)
         runs = [(g, r0 + i, min(run_rows, n - i), 0) for g, (r0, n, _, _) in enumerate(segs) for i in range(0, n, run_rows)]
-        t, scale = ints(runs), put(np.zeros((self.n, self.parts)))
+        t, scale, mixed = ints(runs), put(np.zeros((self.n, self.parts))), put(np.zeros((self.n, self.ld)))
         for args in (self.a, self.b):
-            args.scale, args.rows = (scale.data_ptr(), max(r0 + n for r0, n, _, _ in segs)) if two else (None, 0)
+            args.scale, args.mixed = (scale.data_ptr(), mixed.data_ptr()) if two else (None, None)
+            args.rows = max(r0 + n for r0, n, _, _ in segs)
             self.hb.check(self.hb.lib.hb_residual_step(None, C.byref(args), t.data_ptr(), len(runs), s.data_ptr(), self.width,
                                                        dt(self.hb, self.dtype)))
         torch.cuda.synchronize()
@@ -110,7 +111,7 @@ def test_residual_of_a_whole_sequence(hb, cuda, width, parts, taps, kind, dtype)
     b = Boundary(hb, width, parts, taps, n, dtype, kind, depth=3 if kind == "experts" else 0)
     made, x, h = b.expected(0, n)
     first = None
-    for run_rows, two in ((n, False), (16, False), (5, False), (2, False), (1, False), (8, True), (3, True), (1, True)):
+    for run_rows, two in ((n, False), (16, False), (5, False), (2, False), (1, False), (16, True), (8, True), (3, True), (1, True)):
         got = b.run([(0, n, 0, 1)], run_rows, two)  # (also runs shorter than the convolution)
         assert rms_err(got[0], made) < 2e-6 and rms_err(got[1], x) < 2e-6 and rms_err(got[2], h) < tight(dtype), run_rows
         first = first or got
@@ -128,7 +129,7 @@ def test_portions_meet_in_the_state(hb, cuda, width, parts, taps, dtype):
     shorter and longer than the convolution."""
     b = Boundary(hb, width, parts, taps, 130, dtype, depth=2)
     one, other = b.expected(0, 100), b.expected(100, 130)
-    for run_rows, two in ((16, False), (3, False), (4, False), (8, True), (2, True)):
+    for run_rows, two in ((16, False), (3, False), (4, False), (16, True), (2, True)):
         at = 0
         for n in (2, 1, 9, 1, 1, 1, 40, 3, 2, 40):
             segs = [(at, n, at, 1)] + ([(100, 30, 0, 2)] if at == 2 else [])
@@ -156,7 +157,7 @@ def test_an_input_is_felt_for_exactly_its_taps(hb, cuda):
         for portions, two in (((40,), 0), ((40,), 1), ((16, 24), 0), ((16, 24), 1), ((14, 1, 1, 1, 23), 0), ((1,) * 40, 1)):
             pos, h = 0, None
             for p in portions:
-                h = b.run([(pos, p, pos, 0)], 8 if two else 16, two)[2]
+                h = b.run([(pos, p, pos, 0)], 16, two)[2]
                 pos += p
             felt = np.flatnonzero(np.abs(h).max(axis=1))
             assert felt.tolist() == [t for t in range(at, at + taps) if t < n], (at, portions[:2], felt)

@@ -181,7 +181,8 @@ class ResidualArgs(C.Structure):
         ("ids", C.c_void_p), ("vocab", C.c_int64), ("norm", C.c_void_p), ("groups", C.c_int), ("eps", C.c_float),
         ("x", C.c_void_p), ("result", C.c_void_p), ("x_out", C.c_void_p), ("earlier", C.c_void_p), ("step", C.c_int64),
         ("n_earlier", C.c_int), ("depth", C.c_void_p), ("conv", C.c_void_p), ("taps", C.c_int), ("state", C.c_void_p),
-        ("past", C.c_void_p), ("h", C.c_void_p), ("ld_h", C.c_int64), ("scale", C.c_void_p), ("rows", C.c_int64),
+        ("past", C.c_void_p), ("h", C.c_void_p), ("ld_h", C.c_int64), ("scale", C.c_void_p),
+        ("mixed", C.c_void_p), ("rows", C.c_int64),
     ]
 
 

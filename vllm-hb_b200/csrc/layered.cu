@@ -1103,7 +1103,10 @@ static int layered_issue(hb_engine* e, const StepExec& x) {
     }
     read = next;
     r.rows = rows;
-    if (rows > kResidualTwo) r.scale = m->part_scale;
+    if (rows > kResidualTwo) {
+      r.scale = m->part_scale;
+      r.mixed = m->y2;
+    }
     e->last_launches += residual_in_two(r) ? 2 : 1;
     prof_mark(e, kCatNorm);
     return residual_step(st, r, runs, s.n_runs, seg, W, e->dtype);

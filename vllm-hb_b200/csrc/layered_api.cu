@@ -315,7 +315,7 @@ int hb_residual_step(void* stream, const hb_residual_args* p, const int32_t* til
   a.earlier = p->earlier; a.step = p->step; a.n_earlier = p->n_earlier; a.depth = p->depth;
   a.conv = p->conv; a.taps = p->taps; a.state = p->state; a.past = p->past;
   a.h = p->h; a.ld_h = p->ld_h;
-  a.scale = p->scale; a.rows = p->rows;
+  a.scale = p->scale; a.mixed = p->mixed; a.rows = p->rows;
   return hb::residual_step((cudaStream_t)stream, a, (const hb::RowRange*)tiles, n_tiles, (const hb::SegInfo*)segments, width, dtype);
 }
 

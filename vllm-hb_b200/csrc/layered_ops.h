@@ -71,7 +71,7 @@ int gated_group_norm(cudaStream_t st, void* out, int64_t ld_out, const float* o,
 // one of position p at entry p mod (taps - 1); past: the same of the convolution that read x, which is
 // brought up to date here.
 constexpr int kResidualMaxTaps = 32;
-constexpr int kResidualRun = 8;        // most rows of a run where the step goes in two kernels
+constexpr int kResidualRun = 16;       // most rows of a run where the step goes in two kernels
 struct ResidualStep {
   const float* y = nullptr;            // rows of stride ld_y
   int64_t ld_y = 0;
@@ -99,12 +99,12 @@ struct ResidualStep {
   float* past = nullptr;
   void* h = nullptr;
   int64_t ld_h = 0;
-  // With scale [rows, groups] (scratch) and up to four taps the step goes in two kernels, the faster form for
+  // With scale [rows, groups] and, for experts, mixed [rows, ld_y] (scratch) and up to four taps the step goes in two kernels, the faster form for
   // many rows: rows of the step, none of the runs longer than kResidualRun.
-  float* scale = nullptr;
+  float *scale = nullptr, *mixed = nullptr;
   int64_t rows = 0;
 };
-inline bool residual_in_two(const ResidualStep& a) { return a.scale && a.rows > 0 && a.taps <= 4; }
+inline bool residual_in_two(const ResidualStep& a) { return a.scale && a.rows > 0 && a.taps <= 4 && (a.mixed || !a.top); }
 int residual_step(cudaStream_t st, const ResidualStep& a, const RowRange* tiles, int n_tiles, const SegInfo* segs, int64_t width,
                   hb_dtype dtype);
 // out[r] = rms of in[list ? list[r] : r] in `groups` parts of `size` channels * weight [groups * size]; in

@@ -24,6 +24,12 @@ template <typename T, int VEC>
 __device__ __forceinline__ void load_row(float (&f)[VEC], const T* p) {
   if constexpr (VEC == 1) {
     f[0] = to_f32<T>(*p);
+  } else if constexpr (VEC == 2 && sizeof(T) == 4) {
+    const float2 v = *reinterpret_cast<const float2*>(p);
+    f[0] = v.x; f[1] = v.y;
+  } else if constexpr (VEC == 2) {
+    const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+    f[0] = v.x; f[1] = v.y;
   } else if constexpr (sizeof(T) == 4) {
     const float4 v = *reinterpret_cast<const float4*>(p);
     f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
@@ -38,6 +44,10 @@ template <typename T, int VEC>
 __device__ __forceinline__ void store_row(T* p, const float (&f)[VEC]) {
   if constexpr (VEC == 1) {
     *p = from_f32<T>(f[0]);
+  } else if constexpr (VEC == 2 && sizeof(T) == 4) {
+    *reinterpret_cast<float2*>(p) = make_float2(f[0], f[1]);
+  } else if constexpr (VEC == 2) {
+    *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(f[0], f[1]);
   } else if constexpr (sizeof(T) == 4) {
     *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
   } else {
@@ -179,9 +189,9 @@ residual_kernel(const ResidualStep a, const RowRange* __restrict__ tiles, const 
       for (int j = 0; j < VEC; ++j) x[k][j] = fmaf(v[k][j] * r, w[j], x[k][j]);
       if (a.result && i >= 0) store_row<float, VEC>(a.result + row * W + c, x[k]);
       if (a.depth) {
-        float s[VEC];
+        const float own = a.depth[a.n_earlier];
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) s[j] = 0.f;
+        for (int j = 0; j < VEC; ++j) x[k][j] *= own;
         const float* e = a.earlier + row * W + c;
 #pragma unroll 4
         for (int l = 0; l < a.n_earlier; ++l, e += a.step) {
@@ -189,11 +199,8 @@ residual_kernel(const ResidualStep a, const RowRange* __restrict__ tiles, const 
           load_row<float, VEC>(f, e);
           const float d = a.depth[l];
 #pragma unroll
-          for (int j = 0; j < VEC; ++j) s[j] = fmaf(d, f[j], s[j]);
+          for (int j = 0; j < VEC; ++j) x[k][j] = fmaf(d, f[j], x[k][j]);
         }
-        const float d = a.depth[a.n_earlier];
-#pragma unroll
-        for (int j = 0; j < VEC; ++j) x[k][j] = fmaf(d, x[k][j], s[j]);
       }
       if (a.x_out && i >= 0) store_row<float, VEC>(a.x_out + row * W + c, x[k]);
       if (!a.h) continue;
@@ -244,8 +251,9 @@ residual_kernel(const ResidualStep a, const RowRange* __restrict__ tiles, const 
   }
 }
 
-// The same in two kernels, for many rows: the factors of all parts of all rows first; then a thread takes
-// four channels of a run and all of the run's rows at once, with nothing to wait for but its loads.
+// The same in two kernels, for many rows: the factors of all parts of all rows first (and the experts' outputs
+// summed up); then a thread takes
+// two channels of a run and all of the run's rows at once, with nothing to wait for but its loads.
 template <typename T>
 __global__ void __launch_bounds__(kResidualThreads)
 residual_scale_kernel(const ResidualStep a, int64_t W, int team_size) {
@@ -260,6 +268,7 @@ residual_scale_kernel(const ResidualStep a, int64_t W, int team_size) {
     for (int i = team.rank * 4; i < size; i += team.size * 4) {
       float f[4];
       sublayer_output<T, 4>(f, a, W, row, (int64_t)group * size + i);
+      if (a.top) store_row<float, 4>(a.mixed + row * a.ld_y + (int64_t)group * size + i, f);
 #pragma unroll
       for (int j = 0; j < 4; ++j) ss = fmaf(f[j], f[j], ss);
     }
@@ -271,99 +280,109 @@ constexpr int kRunThreads = 128;
 template <typename T>
 __global__ void __launch_bounds__(kRunThreads)
 residual_run_kernel(const ResidualStep a, const RowRange* __restrict__ tiles, const SegInfo* __restrict__ segs, int64_t W) {
-  constexpr int H = kHeldTaps - 1, N = H + kResidualRun;  // rows ahead of the run, all rows
+  constexpr int H = kHeldTaps - 1, N = H + kResidualRun, V = 2;  // rows ahead of the run, all rows, channels
   pdl_trigger();
   pdl_grid_wait();
-  const int64_t c = ((int64_t)blockIdx.y * kRunThreads + threadIdx.x) * 4;
+  const int64_t c = ((int64_t)blockIdx.y * kRunThreads + threadIdx.x) * V;
   if (c >= W) return;
   const RowRange tile = tiles[blockIdx.x];
   const SegInfo seg = segs[tile.seg];
   const int back = a.conv ? a.taps - 1 : 0, ring = a.taps - 1, first = tile.row0 - seg.row0, group = (int)(c / (W / a.groups));
-  // row i is token first + i - H of the segment: of this step, and wanted for itself or for the convolution
-  auto here = [&](int i) { return i >= H ? i - H < tile.n : H - i <= back && first + i - H >= 0; };
-  const int64_t row0 = (int64_t)tile.row0 - H;
-  float x[N][4];
+  // row i is token first + i - H of the segment; rows that are not there are read as the run's first one, so
+  // that no load waits for a branch, and come to nothing
+  auto row = [&](int i) { return (int64_t)tile.row0 + (i < H ? (first + i < H ? 0 : i - H) : i - H < tile.n ? i - H : 0); };
+  float x[N][V];
+  const float* y = a.top ? a.mixed : a.y;
 #pragma unroll
   for (int i = 0; i < N; ++i) {
-#pragma unroll
-    for (int j = 0; j < 4; ++j) x[i][j] = 0.f;
-    if (here(i)) sublayer_output<T, 4>(x[i], a, W, row0 + i, c);
+    if (a.embed) load_row<T, V>(x[i], (const T*)a.embed + min((int64_t)a.ids[row(i)], a.vocab - 1) * W + c);
+    else load_row<float, V>(x[i], y + row(i) * a.ld_y + c);
   }
-  float w[4];
-  load_row<float, 4>(w, a.norm + c);
+  float w[V], f[N][V];
+  load_row<float, V>(w, a.norm + c);
 #pragma unroll
   for (int i = 0; i < N; ++i) {
-    if (!here(i)) continue;
-    const float r = a.scale[(row0 + i) * a.groups + group];
-    float f[4] = {0.f, 0.f, 0.f, 0.f};
-    if (a.x) load_row<float, 4>(f, a.x + (row0 + i) * W + c);
-    const int token = first + i - H;
-    if (a.past && ring > 0 && i >= H && token >= seg.n - ring)
-      store_row<float, 4>(a.past + ((int64_t)seg.slot * ring + ((int64_t)seg.pos0 + token) % ring) * W + c, f);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) x[i][j] = fmaf(x[i][j] * r, w[j], f[j]);
-    if (a.result && i >= H) store_row<float, 4>(a.result + (row0 + i) * W + c, x[i]);
+    for (int j = 0; j < V; ++j) f[i][j] = 0.f;
+    if (a.x) load_row<float, V>(f[i], a.x + row(i) * W + c);
+  }
+  if (a.past && ring > 0 && first + tile.n > seg.n - ring) {  // (the end of the segment)
+#pragma unroll
+    for (int i = H; i < N; ++i) {
+      const int token = first + i - H;
+      if (i - H < tile.n && token >= seg.n - ring)
+        store_row<float, V>(a.past + ((int64_t)seg.slot * ring + ((int64_t)seg.pos0 + token) % ring) * W + c, f[i]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    const float r = a.scale[row(i) * a.groups + group];
+#pragma unroll
+    for (int j = 0; j < V; ++j) x[i][j] = fmaf(x[i][j] * r, w[j], f[i][j]);
+  }
+  if (a.result) {
+#pragma unroll
+    for (int i = H; i < N; ++i)
+      if (i - H < tile.n) store_row<float, V>(a.result + row(i) * W + c, x[i]);
   }
   if (a.depth) {
-    float s[N][4];
-#pragma unroll
-    for (int i = 0; i < N; ++i)
-#pragma unroll
-      for (int j = 0; j < 4; ++j) s[i][j] = 0.f;
-    const float* e = a.earlier + row0 * W + c;
-    for (int l = 0; l < a.n_earlier; ++l, e += a.step) {
-      const float d = a.depth[l];
-#pragma unroll
-      for (int i = 0; i < N; ++i) {
-        if (!here(i)) continue;
-        float f[4];
-        load_row<float, 4>(f, e + i * W);
-#pragma unroll
-        for (int j = 0; j < 4; ++j) s[i][j] = fmaf(d, f[j], s[i][j]);
-      }
-    }
     const float d = a.depth[a.n_earlier];
 #pragma unroll
     for (int i = 0; i < N; ++i)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) x[i][j] = fmaf(d, x[i][j], s[i][j]);
+      for (int j = 0; j < V; ++j) x[i][j] *= d;
+    const float* e = a.earlier + c;
+    for (int l = 0; l < a.n_earlier; ++l, e += a.step) {
+#pragma unroll
+      for (int i = 0; i < N; ++i) load_row<float, V>(f[i], e + row(i) * W);
+      const float d = a.depth[l];
+#pragma unroll
+      for (int i = 0; i < N; ++i)
+#pragma unroll
+        for (int j = 0; j < V; ++j) x[i][j] = fmaf(d, f[i][j], x[i][j]);
+    }
   }
   if (a.x_out) {
 #pragma unroll
     for (int i = H; i < N; ++i)
-      if (here(i)) store_row<float, 4>(a.x_out + (row0 + i) * W + c, x[i]);
+      if (i - H < tile.n) store_row<float, V>(a.x_out + row(i) * W + c, x[i]);
   }
   if (!a.h) return;
   if (a.conv) {
-    float tap[kHeldTaps][4];  // by distance
+    float tap[kHeldTaps][V];  // by distance
 #pragma unroll
     for (int b = 0; b < kHeldTaps; ++b) {
 #pragma unroll
-      for (int j = 0; j < 4; ++j) tap[b][j] = 0.f;
-      if (b <= back) load_row<float, 4>(tap[b], a.conv + (int64_t)(back - b) * W + c);
+      for (int j = 0; j < V; ++j) tap[b][j] = 0.f;
+      if (b <= back) load_row<float, V>(tap[b], a.conv + (int64_t)(back - b) * W + c);
     }
+    if (first < H) {  // the run's past reaches back beyond this step
 #pragma unroll
-    for (int i = 0; i < H; ++i) {  // what earlier steps left
-      const int token = first + i - H;
-      if (H - i <= back && token < 0 && seg.pos0 + token >= 0)
-        load_row<float, 4>(x[i], a.state + ((int64_t)seg.slot * ring + ((int64_t)seg.pos0 + token) % ring) * W + c);
+      for (int i = 0; i < H; ++i) {
+        const int token = first + i - H;
+        if (token >= 0) continue;
+#pragma unroll
+        for (int j = 0; j < V; ++j) x[i][j] = 0.f;
+        if (H - i <= back && seg.pos0 + token >= 0)
+          load_row<float, V>(x[i], a.state + ((int64_t)seg.slot * ring + ((int64_t)seg.pos0 + token) % ring) * W + c);
+      }
     }
 #pragma unroll
     for (int i = N - 1; i >= H; --i) {  // the last row first: it is the one no other row needs any more
-      float acc[4];
+      float acc[V];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) acc[j] = tap[0][j] * x[i][j];
+      for (int j = 0; j < V; ++j) acc[j] = tap[0][j] * x[i][j];
 #pragma unroll
       for (int b = 1; b < kHeldTaps; ++b)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[j] = fmaf(tap[b][j], x[i - b][j], acc[j]);
+        for (int j = 0; j < V; ++j) acc[j] = fmaf(tap[b][j], x[i - b][j], acc[j]);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) x[i][j] += acc[j];
+      for (int j = 0; j < V; ++j) x[i][j] += acc[j];
     }
   }
 #pragma unroll
   for (int i = H; i < N; ++i)
-    if (here(i)) store_row<T, 4>((T*)a.h + (row0 + i) * a.ld_h + c, x[i]);
+    if (i - H < tile.n) store_row<T, V>((T*)a.h + row(i) * a.ld_h + c, x[i]);
 }
 
 // Rows normed in parts, wherever they lie: CTA = (row, one or several parts).
@@ -415,7 +434,7 @@ int residual_step(cudaStream_t st, const ResidualStep& a, const RowRange* tiles,
   const size_t es = 4 * dtype_size(dtype);
   const bool vec = size % 4 == 0 && a.ld_y % 4 == 0 && a.ld_input % 4 == 0 && a.ld_h % 4 == 0 && a.step % 4 == 0 && al(a.y, 16) &&
                    al(a.norm, 16) && al(a.x, 16) && al(a.x_out, 16) && al(a.result, 16) && al(a.earlier, 16) && al(a.conv, 16) &&
-                   al(a.state, 16) && al(a.past, 16) && al(a.expert_y, es) && al(a.input, es) && al(a.embed, es) && al(a.h, es);
+                   al(a.state, 16) && al(a.past, 16) && al(a.mixed, 16) && al(a.expert_y, es) && al(a.input, es) && al(a.embed, es) && al(a.h, es);
   const int v = vec ? 4 : 1, team = team_threads(size, v, 2);
   const int runs = (int)((size + (int64_t)team * v - 1) / ((int64_t)team * v));
   if (runs > 8) return fail(HB_ERR_INVALID_ARG, "residual_step: parts of %lld channels are not supported", (long long)size);
@@ -425,7 +444,7 @@ int residual_step(cudaStream_t st, const ResidualStep& a, const RowRange* tiles,
   if (residual_in_two(a) && vec) {
     auto two = [&](auto* scale, auto* run) -> int {
       HB_CUDA_CHECK(launch_pdl(scale, dim3((unsigned)a.rows, grid.y), dim3((unsigned)threads), 0, st, a, width, team));
-      HB_CUDA_CHECK(launch_pdl(run, dim3((unsigned)n_tiles, (unsigned)((width / 4 + kRunThreads - 1) / kRunThreads)), dim3(kRunThreads), 0, st,
+      HB_CUDA_CHECK(launch_pdl(run, dim3((unsigned)n_tiles, (unsigned)((width / 2 + kRunThreads - 1) / kRunThreads)), dim3(kRunThreads), 0, st,
                                a, tiles, segs, width));
       return HB_OK;
     };
