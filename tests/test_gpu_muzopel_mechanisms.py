@@ -423,3 +423,19 @@ def test_capped_products(hb, cuda, rows, N, K, m_pad):
     hb.check(hb.lib.hb_gemm_grouped(None, ty.data_ptr(), tx.data_ptr(), tw.data_ptr(), C.byref(g), hb.BF16))
     torch.cuda.synchronize()
     assert rms_err(back(ty), 15.0 * np.tanh(x @ w.T / 15.0)) < 1e-4
+
+
+def test_gelu_of_a_product_within_the_formulas_bound(hb, cuda):
+    """The error function inside the product: 1.5e-7 of the distribution function, so 2e-7 of z and of 1."""
+    import torch
+
+    z = rounded(np.concatenate([np.linspace(-12, 12, 4000), [0.0, -0.0, 1e-8, -1e-8, 60.0, -60.0, 1e4, -1e4] * 12]), "bf16")
+    n = len(z) // 16 * 16
+    x, w = np.zeros((n, 16)), np.zeros((8, 16))
+    x[:, 3], w[:, 3] = z[:n], 1.0
+    tx, tw, ty, tg = put(x, "bf16"), put(w, "bf16"), put(np.zeros((n, 8))), ints(np.zeros(n // 16))
+    g = hb.GroupedGemm(1, 8, 16, 16, n // 16, n // 16, tg.data_ptr(), 16, 8, 1, 1, hb.GatedActSpec(1.0, 0.0, np.inf, 0.0, 1, 1))
+    hb.check(hb.lib.hb_gemm_grouped(None, ty.data_ptr(), tx.data_ptr(), tw.data_ptr(), C.byref(g), hb.BF16))
+    torch.cuda.synchronize()
+    got = back(ty)
+    assert (np.abs(got - R.gelu(z[:n])[:, None]) <= 2e-7 * np.maximum(1.0, np.abs(z[:n]))[:, None] * 2).all()
